@@ -1,0 +1,770 @@
+// Layer-list engine (see nfn_engine.h): a decoder described layer by layer, served from paged caches in steps that run any mix of
+// prompt portions and single tokens as one batch.
+//
+// Cache manager. Every layer that owns keys and values has page pools (keys [page][kv_heads][64][dim], values transposed
+// [page][kv_heads][vdim][64]); layers that read an earlier layer's cache have none. Owner layers whose readers look equally far
+// back form a group with one free list and one page table per slot, so a page number means the same tokens in all of them. When
+// all readers of a group have windows, pages behind the widest one go back to the free list as the sequence moves on. The short
+// convolutions keep taps - 1 projected rows per slot and layer in two halves: a step reads one half and writes the other, so no
+// launch reads what it overwrites.
+//
+// A step lays its rows out short entries first (single tokens and portions below kTileMin rows: one query row at a time), then
+// the long ones (tcgen05 tiles). Per layer it launches: input projection (q | k | v | gates | feed-forward in one product), the
+// row mix (convolution, temperature, cache append, feed-forward gate), attention with the output gate, one output product that
+// adds mixer and feed-forward to the 32-bit residual stream, and the token input's two products with their norm, which also
+// produces the next layer's normalised rows. Steps of single tokens run with a padded row count and are replayed as CUDA graphs.
+#include <cmath>
+#include <cstring>
+#include <memory>
+
+#include "engine_core.h"
+
+using nfn_eng::efail;
+
+namespace {
+
+constexpr int kPage = NFN_KV_PAGE, kTileMin = 16, kMixRows = 16;
+
+int up(int v, int m) { return (v + m - 1) / m * m; }
+
+struct Layer {
+  nfn_layer_desc d{};
+  int dp = 0, vp = 0, ff = 0;                       // padded head sizes and feed-forward width
+  int nq = 0, nk = 0, nv = 0, off_g = 0, off_gate = 0, off_up = 0, n_in = 0, n_cat = 0;
+  int owner = 0, group = 0;
+  void *k_pool = nullptr, *v_pool = nullptr, *state = nullptr;
+  long long state_half = 0;
+  float* slopes = nullptr;
+  const void *norm1 = nullptr, *w_in = nullptr, *conv = nullptr, *w_out = nullptr, *side_gate = nullptr, *side_proj = nullptr, *side_norm = nullptr;
+  int tile_rows = 0;                                // query rows per tcgen05 tile, 0: one row at a time
+};
+
+struct Group {
+  int window = 0;                                   // widest reader, 0: everything stays
+  int pages = 0;
+  std::vector<int> free_pages;
+  int* d_table = nullptr;                           // [slots][max_pages]
+  int* h_table = nullptr;                           // pinned mirror
+  std::vector<int> first, next;                     // per slot: pages [first, next) of the sequence are held
+};
+
+struct layered_engine final : nfn_engine {
+  nfn_layered_config c{};
+  std::vector<Layer> layers;
+  std::vector<Group> groups;
+  std::vector<int> tile_kinds;                      // distinct tile heights
+  int es = 2;                                       // bytes per activation
+  int wp = 0, vp = 0, sp = 0, max_pages = 0, rows_max = 0, logit_rows = 0, n_in_max = 0, nq_max = 0, cat_max = 0;
+  float* x = nullptr;
+  void *xb = nullptr, *h = nullptr, *in = nullptr, *q = nullptr, *cat = nullptr, *s_act = nullptr, *y = nullptr, *hw = nullptr;
+  float *s_gate = nullptr, *logits = nullptr, *saved = nullptr;
+  void *att_ws = nullptr, *gemm_ws = nullptr;
+  long long att_ws_bytes = 0, gemm_ws_bytes = 0;
+  std::vector<uint8_t> parity;                      // per slot: the half that holds its convolution history
+  std::vector<int> logit_at;                        // per slot: row of `logits`, -1: none, -2: `saved`
+  // per-step block, one copy to the device: offsets in bytes
+  struct { long long tok, slot, pos, want, params, offset, mix, att, out, total; } io{};
+  unsigned char *h_io = nullptr, *d_io = nullptr;
+  std::map<int, cudaGraphExec_t> graphs;            // by padded row count
+  std::map<int, long long> graph_launches;
+  std::map<int, int> graph_calls;
+
+  ~layered_engine() override;
+  int build();
+  int finalize() override;
+  int release(int slot) override;
+  int prefill(int slot, const int32_t* tokens, int n, const nfn_sampling* s, int32_t* next_token) override;
+  int decode(const int32_t* tokens_in, const uint8_t* active, const nfn_sampling* s, const nfn_sampling* per_slot, int32_t* next_tokens) override;
+  int step(const nfn_step_entry* entries, int n_entries, const int32_t* tokens, const int32_t* want_rows, int n_want, const nfn_sampling* want_sampling,
+           int32_t* want_tokens, float* want_logits) override;
+  int last_logits(int slot, float* out_vocab) override;
+  int truncate(int slot, int n) override;
+  int fork(int src_slot, int dst_slot, int n) override;
+  long long free_tokens() const override;
+
+  int add(void** p, long long n) {
+    if (alloc(p, n)) return -1;
+    owned.push_back(*p);
+    return 0;
+  }
+  std::vector<void*> owned;
+  template <typename P>
+  P* dev(long long off) const { return reinterpret_cast<P*>(d_io + off); }
+  template <typename P>
+  P* host(long long off) const { return reinterpret_cast<P*>(h_io + off); }
+
+  int reserve(int slot, int upto);                  // pages for positions < upto
+  void trim(int slot);                              // pages no later query of this slot can see
+  int lin(const void* a, int lda, const void* w, int rows, int n, int k, void* out, int ldo, int kind);
+  int pass(int rows, int short_rows, int n_mix, const std::vector<int>& att_off, const std::vector<int>& att_n);
+  int head(const int* src_rows, int rows);
+  int sample(int rows);
+  int run(const std::vector<nfn_step_entry>& part, const int32_t* const* part_tokens, std::vector<int>& row_of, bool single);
+};
+
+enum { kOutAct = 0, kOutF32 = 1, kOutResidual = 2 };
+
+std::string lname(int l, const char* s) { return "layers." + std::to_string(l) + "." + s; }
+
+}  // namespace
+
+layered_engine::~layered_engine() {
+  for (auto& g : graphs) cudaGraphExecDestroy(g.second);
+  for (void* p : owned) cudaFree(p);
+  for (Group& g : groups)
+    if (g.h_table) cudaFreeHost(g.h_table);
+  if (h_io) cudaFreeHost(h_io);
+}
+
+// sizes, tensor names and groups; no device memory yet
+int layered_engine::build() {
+  es = c.dtype == 1 ? 4 : 2;
+  wp = up(c.width, 16);
+  vp = up(c.vocab, 16);
+  sp = c.side_dim > 0 ? up(c.side_dim, 16) : 0;
+  max_pages = (c.max_seq + kPage - 1) / kPage;
+  auto want = [&](const std::string& n, long long numel) { expected.emplace_back(n, numel); };
+  want("embed", (long long)vp * wp);
+  if (sp) want("side_embed", (long long)c.vocab * c.n_layer * sp);
+  for (int l = 0; l < c.n_layer; ++l) {
+    Layer& L = layers[l];
+    const nfn_layer_desc& d = L.d;
+    L.dp = up(d.dim, 16);
+    L.vp = up(d.vdim, 16);
+    L.ff = d.ff > 0 ? up(d.ff, 16) : 0;
+    L.owner = l;
+    if (d.kv_from >= 0) {
+      const Layer& o = layers[d.kv_from];
+      if (d.kv_from >= l || o.d.kv_from >= 0) return efail("engine: layer " + std::to_string(l) + " must read an earlier layer with keys and values of its own");
+      if (o.d.kv_heads != d.kv_heads || o.d.dim != d.dim || o.d.vdim != d.vdim)
+        return efail("engine: layer " + std::to_string(l) + " and the layer whose cache it reads have different key / value heads");
+      L.owner = d.kv_from;
+    }
+    const bool own = L.owner == l;
+    L.nq = d.heads * L.dp;
+    L.nk = own ? d.kv_heads * L.dp : 0;
+    L.nv = own ? d.kv_heads * L.vp : 0;
+    L.off_g = L.nq + L.nk + L.nv;
+    L.off_gate = L.off_g + (d.out_gate ? d.heads * L.vp : 0);
+    L.off_up = L.off_gate + L.ff;
+    L.n_in = L.off_up + L.ff;
+    L.n_cat = d.heads * L.vp + L.ff;
+    n_in_max = std::max(n_in_max, L.n_in);
+    nq_max = std::max(nq_max, L.nq);
+    cat_max = std::max(cat_max, L.n_cat);
+    want(lname(l, "norm1"), wp);
+    want(lname(l, "w_in"), (long long)L.n_in * wp);
+    if (d.conv_taps > 1) want(lname(l, "conv"), (long long)d.conv_taps * (L.nq + L.nk + L.nv));
+    want(lname(l, "w_out"), (long long)wp * L.n_cat);
+    if (sp) {
+      want(lname(l, "side_gate"), (long long)sp * wp);
+      want(lname(l, "side_proj"), (long long)wp * sp);
+      want(lname(l, "side_norm"), wp);
+    }
+    L.tile_rows = nfn_paged_tile_rows(c.dtype, d.heads, d.kv_heads, L.dp, L.vp);
+    if (L.tile_rows > 0 && std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) == tile_kinds.end()) tile_kinds.push_back(L.tile_rows);
+  }
+  want("final_norm", wp);
+  // how far back the readers of each owner look, and one group per distinct answer
+  for (int l = 0; l < c.n_layer; ++l) {
+    if (layers[l].owner != l) continue;
+    int w = 0;
+    bool all = false;
+    for (const Layer& r : layers)
+      if (r.owner == l) {
+        all |= r.d.window <= 0;
+        w = std::max(w, r.d.window);
+      }
+    if (all) w = 0;
+    int g = 0;
+    while (g < (int)groups.size() && groups[g].window != w) ++g;
+    if (g == (int)groups.size()) {
+      groups.emplace_back();
+      groups.back().window = w;
+    }
+    for (Layer& r : layers)
+      if (r.owner == l) r.group = g;
+  }
+  len.assign(c.max_batch, 0);
+  parity.assign(c.max_batch, 0);
+  logit_at.assign(c.max_batch, -1);
+  return 0;
+}
+
+extern "C" nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, const nfn_layer_desc* layers, int device) {
+  if (!cfg || !layers) {
+    efail("engine_create: null config");
+    return nullptr;
+  }
+  const nfn_layered_config& c = *cfg;
+  if (c.n_layer <= 0 || c.width <= 0 || c.vocab <= 0 || c.side_dim < 0 || (c.dtype != 0 && c.dtype != 1) || c.max_seq <= 0 || c.max_batch <= 0 ||
+      c.kv_tokens < 0 || c.max_step_rows <= 0 || !(c.norm_eps >= 0.f)) {
+    efail("engine_create: invalid geometry");
+    return nullptr;
+  }
+  auto e = std::make_unique<layered_engine>();
+  e->c = c;
+  if (e->c.kv_tokens == 0) e->c.kv_tokens = (int)std::min<long long>((long long)c.max_batch * up(c.max_seq, kPage), 0x7fffffc0LL);
+  e->layers.resize(c.n_layer);
+  for (int l = 0; l < c.n_layer; ++l) {
+    const nfn_layer_desc& d = layers[l];
+    if (d.heads <= 0 || d.kv_heads <= 0 || d.heads % d.kv_heads || d.dim <= 0 || d.vdim <= 0 || d.conv_taps < 0 || d.ff < 0 || d.window < 0 ||
+        d.q_temp_every < 0 || (d.ff_act != NFN_ACT_RELU && d.ff_act != NFN_ACT_SILU && d.ff_act != NFN_ACT_GELU_TANH)) {
+      efail("engine_create: invalid sizes in layer " + std::to_string(l));
+      return nullptr;
+    }
+    e->layers[l].d = d;
+  }
+  e->device = device;
+  if (cudaSetDevice(device) != cudaSuccess || cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking) != cudaSuccess) {
+    efail("engine_create: cannot select the device or create a stream");
+    return nullptr;
+  }
+  if (e->build()) return nullptr;
+  return e.release();
+}
+
+int layered_engine::finalize() {
+  CU(cudaSetDevice(device));
+  if (missing_tensor()) return -1;
+  rows_max = up(std::max(std::min(c.max_step_rows, std::max(c.max_seq, c.max_batch)), c.max_batch), 16);
+  logit_rows = std::max(c.max_batch, 64);
+  const long long R = rows_max, S = c.max_batch;
+  auto zero = [&](void** p, long long n) -> int {
+    if (add(p, n)) return -1;
+    CU(cudaMemset(*p, 0, (size_t)n));
+    return 0;
+  };
+  if (zero((void**)&x, R * wp * 4) || zero(&h, R * wp * es) || zero(&in, R * n_in_max * es) || zero(&q, R * nq_max * es) || zero(&cat, R * cat_max * es) ||
+      zero(&hw, (long long)logit_rows * wp * es) || zero((void**)&logits, (long long)logit_rows * vp * 4) || zero((void**)&saved, S * vp * 4))
+    return -1;
+  if (c.dtype == 0 && zero(&xb, R * wp * 2)) return -1;
+  if (sp && (zero((void**)&s_gate, R * sp * 4) || zero(&s_act, R * sp * es) || zero(&y, R * wp * es))) return -1;
+  for (Group& g : groups) {
+    g.pages = (c.kv_tokens + kPage - 1) / kPage;
+    if (g.window > 0) g.pages = (int)std::min<long long>(g.pages, S * ((g.window + R) / kPage + 2));
+    for (int p = g.pages - 1; p >= 0; --p) g.free_pages.push_back(p);
+    g.first.assign(S, 0);
+    g.next.assign(S, 0);
+    if (zero((void**)&g.d_table, S * max_pages * 4)) return -1;
+    CU(cudaMallocHost((void**)&g.h_table, (size_t)S * max_pages * 4));
+    std::memset(g.h_table, 0, (size_t)S * max_pages * 4);
+  }
+  long long ws = 0;
+  for (int l = 0; l < c.n_layer; ++l) {
+    Layer& L = layers[l];
+    const nfn_layer_desc& d = L.d;
+    if (L.owner == l) {
+      const long long tiles = (long long)groups[L.group].pages * d.kv_heads * kPage;
+      if (zero(&L.k_pool, tiles * L.dp * es) || zero(&L.v_pool, tiles * L.vp * es)) return -1;
+    } else {
+      L.k_pool = layers[L.owner].k_pool;
+      L.v_pool = layers[L.owner].v_pool;
+    }
+    if (d.conv_taps > 1) {
+      L.state_half = S * (d.conv_taps - 1) * (L.nq + L.nk + L.nv);
+      if (zero(&L.state, 2 * L.state_half * es)) return -1;
+      L.conv = W(lname(l, "conv"));
+    }
+    if (d.alibi != 0.f) {
+      std::vector<float> sl(d.heads);
+      for (int i = 0; i < d.heads; ++i) sl[i] = (float)std::exp2(-(double)d.alibi * (i + 1) / d.heads);
+      if (zero((void**)&L.slopes, 4LL * d.heads)) return -1;
+      CU(cudaMemcpy(L.slopes, sl.data(), sl.size() * 4, cudaMemcpyHostToDevice));
+    }
+    L.norm1 = W(lname(l, "norm1"));
+    L.w_in = W(lname(l, "w_in"));
+    L.w_out = W(lname(l, "w_out"));
+    if (sp) {
+      L.side_gate = W(lname(l, "side_gate"));
+      L.side_proj = W(lname(l, "side_proj"));
+      L.side_norm = W(lname(l, "side_norm"));
+    }
+    ws = std::max(ws, nfn_paged_attention_workspace_bytes(rows_max, d.heads, L.vp));
+  }
+  att_ws_bytes = ws;
+  gemm_ws_bytes = 64LL << 20;
+  if (zero(&att_ws, att_ws_bytes) || add(&gemm_ws, gemm_ws_bytes)) return -1;
+  auto up256 = [](long long v) { return (v + 255) / 256 * 256; };
+  const long long kinds = (long long)tile_kinds.size();
+  io.tok = 0;
+  io.slot = io.tok + up256(R * 4);
+  io.pos = io.slot + up256(R * 4);
+  io.want = io.pos + up256(R * 4);
+  io.params = io.want + up256(R * 4);
+  io.offset = io.params + up256((long long)logit_rows * 12);
+  io.mix = io.offset + 256;
+  io.att = io.mix + up256(R * (long long)sizeof(nfn_row_tile));
+  io.out = io.att + up256(kinds * R * 16);
+  io.total = io.out + up256((long long)logit_rows * 4);
+  CU(cudaMallocHost((void**)&h_io, (size_t)io.total));
+  std::memset(h_io, 0, (size_t)io.total);
+  if (zero((void**)&d_io, io.total)) return -1;
+  CU(cudaDeviceSynchronize());
+  finalized = true;
+  return 0;
+}
+
+// ---- cache manager ------------------------------------------------------------------------------------
+
+long long layered_engine::free_tokens() const {
+  long long n = -1;
+  for (const Group& g : groups) {
+    const long long t = (long long)g.free_pages.size() * kPage;
+    n = n < 0 ? t : std::min(n, t);
+  }
+  return n;
+}
+
+// Pages for every position below `upto` of the slot; the new table entries go to the device. All groups or none.
+int layered_engine::reserve(int slot, int upto) {
+  const int need = (upto + kPage - 1) / kPage;
+  for (const Group& g : groups)
+    if (need - g.next[slot] > (int)g.free_pages.size())
+      return efail("engine_step: the cache pool is full (slot " + std::to_string(slot) + " needs " + std::to_string(need - g.next[slot]) + " more pages)");
+  for (Group& g : groups) {
+    const int from = g.next[slot];
+    if (need <= from) continue;
+    int* row = g.h_table + (size_t)slot * max_pages;
+    for (int p = from; p < need; ++p) {
+      row[p] = g.free_pages.back();
+      g.free_pages.pop_back();
+    }
+    g.next[slot] = need;
+    CU(cudaMemcpyAsync(g.d_table + (size_t)slot * max_pages + from, row + from, (size_t)(need - from) * 4, cudaMemcpyHostToDevice, stream));
+  }
+  return 0;
+}
+
+// The next query of the slot sits at len[slot] and sees keys from len - window + 1 on.
+void layered_engine::trim(int slot) {
+  for (Group& g : groups) {
+    if (g.window <= 0) continue;
+    const int live = std::max(0, len[slot] - g.window + 1) / kPage;
+    for (; g.first[slot] < std::min(live, g.next[slot]); ++g.first[slot])
+      g.free_pages.push_back(g.h_table[(size_t)slot * max_pages + g.first[slot]]);
+  }
+}
+
+int layered_engine::release(int slot) {
+  for (Group& g : groups) {
+    for (int p = g.first[slot]; p < g.next[slot]; ++p) g.free_pages.push_back(g.h_table[(size_t)slot * max_pages + p]);
+    g.first[slot] = g.next[slot] = 0;
+  }
+  len[slot] = 0;
+  logit_at[slot] = -1;
+  return 0;
+}
+
+int layered_engine::truncate(int slot, int n) {
+  if (n == len[slot]) return 0;
+  if (n == 0) return release(slot);
+  return efail("engine_truncate: the short convolutions keep the newest rows only; a shorter prefix has to be run again");
+}
+
+int layered_engine::fork(int src, int dst, int n) {
+  if (n != len[src]) return efail("engine_fork: the short convolutions keep the newest rows only; a shorter prefix has to be run again");
+  CU(cudaSetDevice(device));
+  release(dst);
+  if (n == 0) return 0;
+  for (Group& g : groups)   // pages the source gave back hold nothing the copy needs
+    if (g.next[src] - g.first[src] > (int)g.free_pages.size()) return efail("engine_fork: the cache pool is full");
+  for (size_t gi = 0; gi < groups.size(); ++gi) {
+    Group& g = groups[gi];
+    int *from = g.h_table + (size_t)src * max_pages, *to = g.h_table + (size_t)dst * max_pages;
+    g.first[dst] = g.first[src];
+    g.next[dst] = g.next[src];
+    for (int p = g.first[src]; p < g.next[src]; ++p) {
+      to[p] = g.free_pages.back();
+      g.free_pages.pop_back();
+      for (int l = 0; l < c.n_layer; ++l) {
+        const Layer& L = layers[l];
+        if (L.owner != l || L.group != (int)gi) continue;
+        const size_t kb = (size_t)L.d.kv_heads * kPage * L.dp * es, vb = (size_t)L.d.kv_heads * kPage * L.vp * es;
+        CU(cudaMemcpyAsync(static_cast<char*>(L.k_pool) + to[p] * kb, static_cast<char*>(L.k_pool) + from[p] * kb, kb, cudaMemcpyDeviceToDevice, stream));
+        CU(cudaMemcpyAsync(static_cast<char*>(L.v_pool) + to[p] * vb, static_cast<char*>(L.v_pool) + from[p] * vb, vb, cudaMemcpyDeviceToDevice, stream));
+      }
+    }
+    CU(cudaMemcpyAsync(g.d_table + (size_t)dst * max_pages, to, (size_t)max_pages * 4, cudaMemcpyHostToDevice, stream));
+  }
+  parity[dst] = parity[src];
+  for (const Layer& L : layers) {
+    if (!L.state) continue;
+    const size_t row = (size_t)(L.d.conv_taps - 1) * (L.nq + L.nk + L.nv) * es;
+    char* half = static_cast<char*>(L.state) + (size_t)parity[src] * L.state_half * es;
+    CU(cudaMemcpyAsync(half + dst * row, half + src * row, row, cudaMemcpyDeviceToDevice, stream));
+  }
+  CU(cudaStreamSynchronize(stream));
+  len[dst] = n;
+  return 0;
+}
+
+// ---- one pass over the rows of a step -----------------------------------------------------------------
+
+// out = a . w^T: kOutAct in the activation type, kOutF32 in fp32, kOutResidual added to the residual stream x
+int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n, int k, void* out, int ldo, int kind) {
+  if (c.dtype == 1) {
+    K(nfn_gemm_f32(static_cast<const float*>(a), lda, wt, k, static_cast<float*>(out), ldo, rows, n, k, kind == kOutResidual, stream));
+    return 0;
+  }
+  nfn_gemm_args g{};
+  g.a = a; g.b = wt; g.c = out;
+  g.m = rows; g.n = n; g.k = k;
+  g.lda = lda; g.ldb = k; g.ldc = ldo;
+  g.alpha = 1.f;
+  g.flags = kind == kOutAct ? 0 : NFN_EPI_OUT_F32;
+  if (kind == kOutResidual) {
+    g.flags |= NFN_EPI_ACCUM | NFN_EPI_COPY_BF16;
+    g.aux_out = xb;
+    g.ld_aux_out = wp;
+  }
+  g.workspace = gemm_ws;
+  g.workspace_bytes = gemm_ws_bytes;
+  K(nfn_gemm_bf16(&g, stream));
+  return 0;
+}
+
+int layered_engine::pass(int rows, int short_rows, int n_mix, const std::vector<int>& att_off, const std::vector<int>& att_n) {
+  const int f32 = c.dtype == 1;
+  nfn_row_norm_args rn{};
+  rn.f32 = f32; rn.rows = rows; rn.width = c.width; rn.ld = wp; rn.eps = c.norm_eps;
+  rn.tokens = dev<int>(io.tok); rn.embed = W("embed"); rn.embed_scale = c.embed_scale; rn.vocab = c.vocab;
+  rn.x_out = x; rn.h = h; rn.weight = layers[0].norm1;
+  K(nfn_row_norm(&rn, stream));
+  rn.tokens = nullptr; rn.embed = nullptr; rn.x = x;
+  for (int l = 0; l < c.n_layer; ++l) {
+    const Layer& L = layers[l];
+    const nfn_layer_desc& d = L.d;
+    if (lin(h, wp, L.w_in, rows, L.n_in, wp, in, L.n_in, kOutAct)) return -1;
+
+    char* ff_out = static_cast<char*>(cat) + (size_t)d.heads * L.vp * es;
+    nfn_mix_args m{};
+    m.f32 = f32; m.in = in; m.ld_in = L.n_in;
+    m.nq = L.nq; m.nk = L.nk; m.nv = L.nv; m.off_gate = L.off_gate; m.off_up = L.off_up; m.ff = L.ff; m.act = d.ff_act;
+    m.conv = L.conv; m.taps = d.conv_taps; m.state = L.state; m.state_half = L.state_half;
+    m.q_out = q; m.ld_q = L.nq;
+    m.k_pool = L.k_pool; m.v_pool = L.v_pool; m.kv_heads = d.kv_heads; m.dim_p = L.dp; m.vdim_p = L.vp;
+    m.table = groups[L.group].d_table; m.table_ld = max_pages;
+    m.temp_coef = d.q_temp_coef; m.temp_every = d.q_temp_every;
+    m.ff_out = ff_out; m.ld_ff = L.n_cat;
+    m.tiles = dev<nfn_row_tile>(io.mix); m.n_tiles = n_mix;
+    K(nfn_mix_rows(&m, stream));
+
+    nfn_paged_attention_args a{};
+    a.f32 = f32; a.q = q; a.ld_q = L.nq; a.total_rows = rows_max;
+    a.k_pool = L.k_pool; a.v_pool = L.v_pool; a.kv_heads = d.kv_heads; a.dim_p = L.dp; a.vdim_p = L.vp; a.pages = groups[L.group].pages;
+    a.table = m.table; a.table_ld = max_pages;
+    a.heads = d.heads; a.window = d.window; a.scale = d.scale; a.slopes = L.slopes;
+    a.gate = d.out_gate ? static_cast<char*>(in) + (size_t)L.off_g * es : nullptr; a.ld_gate = L.n_in;
+    a.out = cat; a.ld_o = L.n_cat;
+    a.row_slot = dev<int>(io.slot); a.row_pos = dev<int>(io.pos);
+    a.max_keys = d.window > 0 ? std::min(d.window, c.max_seq) : c.max_seq;
+    a.workspace = att_ws; a.workspace_bytes = att_ws_bytes;
+    const int single = L.tile_rows > 0 ? short_rows : rows;
+    if (single > 0) {
+      a.rows = single;
+      K(nfn_paged_attention_rows(&a, stream));
+    }
+    if (L.tile_rows > 0 && rows > short_rows) {
+      const int k = (int)(std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) - tile_kinds.begin());
+      a.tiles = dev<int>(io.att) + att_off[k] * 4;
+      a.n_tiles = att_n[k];
+      K(nfn_paged_attention_tiles(&a, stream));
+    }
+
+    if (lin(cat, L.n_cat, L.w_out, rows, wp, L.n_cat, x, wp, kOutResidual)) return -1;
+    const bool last = l + 1 == c.n_layer;
+    if (sp) {
+      if (lin(f32 ? (const void*)x : xb, wp, L.side_gate, rows, sp, wp, s_gate, sp, kOutF32)) return -1;
+      K(nfn_side_mul(f32, s_gate, dev<int>(io.tok), W("side_embed"), (long long)c.n_layer * sp, l * sp, c.vocab, s_act, sp, rows, sp, stream));
+      if (lin(s_act, sp, L.side_proj, rows, wp, sp, y, wp, kOutAct)) return -1;
+    }
+    if (sp || !last) {
+      rn.y = sp ? y : nullptr; rn.y_weight = L.side_norm;
+      rn.x_out = sp ? x : nullptr;
+      rn.h = last ? nullptr : h; rn.weight = last ? nullptr : layers[l + 1].norm1;
+      K(nfn_row_norm(&rn, stream));
+    }
+  }
+  return 0;
+}
+
+// output norm and tied head of `rows` rows of x (src_rows: device indices, NULL: the first ones) -> logits
+int layered_engine::head(const int* src_rows, int rows) {
+  nfn_row_norm_args rn{};
+  rn.f32 = c.dtype == 1; rn.rows = rows; rn.width = c.width; rn.ld = wp; rn.eps = c.norm_eps;
+  rn.x = x; rn.src_rows = src_rows; rn.h = hw; rn.weight = W("final_norm");
+  K(nfn_row_norm(&rn, stream));
+  return lin(hw, wp, W("embed"), rows, vp, wp, logits, vp, kOutF32);
+}
+
+int layered_engine::sample(int rows) {
+  K(nfn_sample_rows(logits, 1, vp, rows, c.vocab, dev<int>(io.out), nullptr, 1.f, 0, 1.f, dev<float>(io.params), 0x5eedULL, 0ULL,
+                    dev<unsigned long long>(io.offset), 0, stream));
+  return 0;
+}
+
+// Runs one batch of at most rows_max rows. row_of[i]: row of the i-th token (in the order of the entries). single: every entry
+// brings one token, and the pass, the head over all rows and the sampling run as one (replayed) launch sequence.
+int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* const* part_tokens, std::vector<int>& row_of, bool single) {
+  int total = 0, short_rows = 0;
+  std::vector<int> first(part.size());
+  for (size_t i = 0; i < part.size(); ++i) {
+    if (reserve(part[i].slot, len[part[i].slot] + part[i].count)) return -1;
+    if (part[i].count < kTileMin) {
+      first[i] = short_rows;
+      short_rows += part[i].count;
+    }
+    total += part[i].count;
+  }
+  int at = short_rows;
+  for (size_t i = 0; i < part.size(); ++i)
+    if (part[i].count >= kTileMin) {
+      first[i] = at;
+      at += part[i].count;
+    }
+  int *tok = host<int>(io.tok), *slot = host<int>(io.slot), *pos = host<int>(io.pos);
+  nfn_row_tile* mix = host<nfn_row_tile>(io.mix);
+  int n_mix = 0, hist_max = 0;
+  for (const Layer& L : layers) hist_max = std::max(hist_max, L.d.conv_taps - 1);
+  row_of.clear();
+  for (size_t i = 0; i < part.size(); ++i) {
+    const int s = part[i].slot, p0 = len[s], n = part[i].count;
+    for (int r = 0; r < n; ++r) {
+      tok[first[i] + r] = part_tokens[i][r];
+      slot[first[i] + r] = s;
+      pos[first[i] + r] = p0 + r;
+      row_of.push_back(first[i] + r);
+    }
+    for (int r = 0; r < n;) {
+      const int k = std::min(n - r, kMixRows - (p0 + r) % kMixRows);
+      mix[n_mix++] = nfn_row_tile{first[i] + r, k, first[i], n, p0, s, parity[s], 0};
+      r += k;
+    }
+  }
+  int rows = total;
+  if (single) {
+    rows = 1;
+    while (rows < total) rows *= 2;
+    rows = std::min(rows, c.max_batch);
+    for (int r = total; r < rows; ++r) {
+      tok[r] = 0; slot[r] = -1; pos[r] = 0;
+      mix[n_mix++] = nfn_row_tile{r, 1, r, 1, 0, -1, 0, 0};
+    }
+    short_rows = rows;
+  }
+  std::vector<int> att_off(tile_kinds.size(), 0), att_n(tile_kinds.size(), 0);
+  int* att = host<int>(io.att);
+  int n_att = 0;
+  for (size_t k = 0; k < tile_kinds.size(); ++k) {
+    att_off[k] = n_att;
+    for (size_t i = 0; i < part.size(); ++i) {
+      if (part[i].count < kTileMin) continue;
+      for (int r = 0; r < part[i].count; r += tile_kinds[k]) {
+        int* t = att + (size_t)n_att++ * 4;
+        t[0] = first[i] + r; t[1] = std::min(tile_kinds[k], part[i].count - r); t[2] = part[i].slot; t[3] = len[part[i].slot] + r;
+      }
+    }
+    att_n[k] = n_att - att_off[k];
+  }
+  // row metadata, then the tile lists
+  CU(cudaMemcpyAsync(d_io + io.tok, h_io + io.tok, (size_t)(io.pos - io.tok) + (size_t)rows * 4, cudaMemcpyHostToDevice, stream));
+  CU(cudaMemcpyAsync(d_io + io.mix, h_io + io.mix, (size_t)n_mix * sizeof(nfn_row_tile), cudaMemcpyHostToDevice, stream));
+  if (n_att > 0) CU(cudaMemcpyAsync(d_io + io.att, h_io + io.att, (size_t)n_att * 16, cudaMemcpyHostToDevice, stream));
+
+  const long long before = nfn_launch_count();
+  auto body = [&]() -> int {
+    if (pass(rows, short_rows, n_mix, att_off, att_n)) return -1;
+    return single ? (head(nullptr, rows) || sample(rows) ? -1 : 0) : 0;
+  };
+  if (!single || !c.use_cuda_graph) {
+    if (body()) return -1;
+    launches += nfn_launch_count() - before;
+  } else if (graphs.count(rows)) {
+    CU(cudaGraphLaunch(graphs[rows], stream));
+    launches += graph_launches[rows];
+  } else if (graph_calls[rows]++ == 0) {
+    if (body()) return -1;                          // first call with this row count: attributes and tensor maps get set up
+    launches += nfn_launch_count() - before;
+  } else {
+    cudaGraph_t g = nullptr;
+    CU(cudaStreamBeginCapture(stream, cudaStreamCaptureModeThreadLocal));
+    const int rc = body();
+    const cudaError_t ce = cudaStreamEndCapture(stream, &g);
+    if (rc != 0 || ce != cudaSuccess || !g) {
+      if (g) cudaGraphDestroy(g);
+      return rc != 0 ? -1 : efail("engine_step: stream capture failed");
+    }
+    cudaGraphExec_t ge = nullptr;
+    CU(cudaGraphInstantiate(&ge, g, 0));
+    cudaGraphDestroy(g);
+    graphs[rows] = ge;
+    graph_launches[rows] = nfn_launch_count() - before;
+    CU(cudaGraphLaunch(ge, stream));
+    launches += graph_launches[rows];
+  }
+  for (const nfn_step_entry& p : part) {
+    len[p.slot] += p.count;
+    parity[p.slot] ^= hist_max > 0;
+    trim(p.slot);
+  }
+  return 0;
+}
+
+int layered_engine::step(const nfn_step_entry* entries, int n_entries, const int32_t* tokens, const int32_t* want_rows, int n_want,
+                         const nfn_sampling* want_sampling, int32_t* want_tokens, float* want_logits) {
+  CU(cudaSetDevice(device));
+  if ((want_sampling == nullptr) != (want_tokens == nullptr)) return efail("engine_step: sampling parameters and a place for the tokens go together");
+  std::vector<uint8_t> seen(c.max_batch, 0);
+  long long total = 0;
+  bool single = n_entries > 0;
+  for (int i = 0; i < n_entries; ++i) {
+    const nfn_step_entry& e = entries[i];
+    if (e.slot < 0 || e.slot >= c.max_batch || seen[e.slot]) return efail("engine_step: bad or repeated slot");
+    if (e.count <= 0 || e.count > c.max_seq || len[e.slot] + e.count > c.max_seq) return efail("engine_step: slot " + std::to_string(e.slot) + " would pass max_seq");
+    seen[e.slot] = 1;
+    total += e.count;
+    single &= e.count == 1;
+  }
+  for (long long i = 0; i < total; ++i)
+    if (tokens[i] < 0 || tokens[i] >= c.vocab) return efail("engine_step: token id outside the vocabulary");
+  for (int i = 0; i < n_want; ++i)
+    if (want_rows[i] < 0 || want_rows[i] >= total || (i > 0 && want_rows[i] <= want_rows[i - 1])) return efail("engine_step: wanted places must ascend inside the step");
+  {
+    // enough pages for the whole step before anything runs (portions longer than a pass get pages back on the way: see run)
+    if (total <= rows_max)
+      for (const Group& g : groups) {
+        long long need = 0;
+        for (int i = 0; i < n_entries; ++i) need += std::max(0, (len[entries[i].slot] + entries[i].count + kPage - 1) / kPage - g.next[entries[i].slot]);
+        if (need > (long long)g.free_pages.size()) return efail("engine_step: the cache pool is full");
+      }
+  }
+  for (int b = 0; b < c.max_batch; ++b)
+    if (seen[b]) logit_at[b] = -1;
+
+  auto stash = [&]() -> int {   // logits of slots that are not part of what comes next
+    for (int b = 0; b < c.max_batch; ++b)
+      if (logit_at[b] >= 0) {
+        CU(cudaMemcpyAsync(saved + (size_t)b * vp, logits + (size_t)logit_at[b] * vp, (size_t)vp * 4, cudaMemcpyDeviceToDevice, stream));
+        logit_at[b] = -2;
+      }
+    return 0;
+  };
+  auto draw_params = [&](int row, const nfn_sampling* s) {
+    float* rp = host<float>(io.params) + 3 * row;
+    rp[0] = s ? s->temperature : 0.f;
+    rp[1] = s ? (float)s->top_k : 0.f;
+    rp[2] = s ? s->top_p : 1.f;
+  };
+  auto send_params = [&](int rows, const nfn_sampling* s) -> int {
+    *host<unsigned long long>(io.offset) = ((s ? s->seed : 0ull) << 20) ^ (++steps);
+    CU(cudaMemcpyAsync(d_io + io.params, h_io + io.params, (size_t)rows * 12, cudaMemcpyHostToDevice, stream));
+    CU(cudaMemcpyAsync(d_io + io.offset, h_io + io.offset, 8, cudaMemcpyHostToDevice, stream));
+    return 0;
+  };
+  auto fetch = [&](int want0, int n, const std::vector<int>& at) -> int {   // results of wants [want0, want0 + n), rows `at` of logits / out
+    if (want_logits)
+      for (int i = 0; i < n; ++i)
+        CU(cudaMemcpyAsync(want_logits + (size_t)(want0 + i) * c.vocab, logits + (size_t)at[i] * vp, (size_t)c.vocab * 4, cudaMemcpyDeviceToHost, stream));
+    if (want_tokens) CU(cudaMemcpyAsync(h_io + io.out, d_io + io.out, (size_t)logit_rows * 4, cudaMemcpyDeviceToHost, stream));
+    CU(cudaStreamSynchronize(stream));
+    if (want_tokens)
+      for (int i = 0; i < n; ++i) want_tokens[want0 + i] = host<int>(io.out)[at[i]];
+    return 0;
+  };
+
+  int ei = 0, used = 0, w = 0;       // entry, its tokens already run, next want
+  long long base = 0;                // tokens run by earlier passes
+  const int32_t* cursor = tokens;
+  while (ei < n_entries) {
+    std::vector<nfn_step_entry> part;
+    std::vector<const int32_t*> ptok;
+    int rows = 0;
+    while (ei < n_entries && rows < rows_max) {
+      const int n = std::min(entries[ei].count - used, rows_max - rows);
+      part.push_back(nfn_step_entry{entries[ei].slot, n});
+      ptok.push_back(cursor);
+      cursor += n;
+      rows += n;
+      used += n;
+      if (used == entries[ei].count) { ++ei; used = 0; }
+    }
+    std::vector<int> row_of, slot_of;
+    for (const nfn_step_entry& p : part) slot_of.insert(slot_of.end(), p.count, p.slot);
+    if (single) {
+      if (stash()) return -1;
+      std::vector<int> want_of(rows, -1);
+      for (int i = 0; i < n_want; ++i) want_of[want_rows[i]] = i;
+      for (int r = 0; r < logit_rows; ++r) draw_params(r, (r < rows && want_sampling && want_of[r] >= 0) ? &want_sampling[want_of[r]] : nullptr);
+      if (send_params(logit_rows, (want_sampling && n_want > 0) ? want_sampling : nullptr)) return -1;
+      if (run(part, ptok.data(), row_of, true)) return -1;
+      for (int r = 0; r < rows; ++r) logit_at[slot_of[r]] = row_of[r];
+      std::vector<int> at;
+      for (int i = 0; i < n_want; ++i) at.push_back(row_of[want_rows[i]]);
+      if (fetch(0, n_want, at)) return -1;
+      break;
+    }
+    if (run(part, ptok.data(), row_of, false)) return -1;
+    while (w < n_want && want_rows[w] < base + rows) {
+      if (stash()) return -1;
+      int n = 0;
+      std::vector<int> at;
+      for (; w + n < n_want && n < logit_rows && want_rows[w + n] < base + rows; ++n) {
+        host<int>(io.want)[n] = row_of[want_rows[w + n] - base];
+        logit_at[slot_of[want_rows[w + n] - base]] = n;
+        at.push_back(n);
+        draw_params(n, want_sampling ? &want_sampling[w + n] : nullptr);
+      }
+      CU(cudaMemcpyAsync(d_io + io.want, h_io + io.want, (size_t)n * 4, cudaMemcpyHostToDevice, stream));
+      const long long before = nfn_launch_count();
+      if (head(dev<int>(io.want), n)) return -1;
+      if (want_sampling && (send_params(n, &want_sampling[w]) || sample(n))) return -1;
+      launches += nfn_launch_count() - before;
+      if (fetch(w, n, at)) return -1;
+      w += n;
+    }
+    base += rows;
+    CU(cudaStreamSynchronize(stream));   // the pinned blocks are written again by the next pass
+  }
+  if (nfn_status_peek() != 0) return efail("engine_step: a kernel reported error code " + std::to_string(nfn_status_read_reset()));
+  return 0;
+}
+
+// ---- the one-sequence and all-slots forms ---------------------------------------------------------------
+
+int layered_engine::prefill(int slot, const int32_t* tokens, int n, const nfn_sampling* s, int32_t* next_token) {
+  if (n <= 0 || n >= c.max_seq) return efail("engine_prefill: the prompt must hold between 1 and max_seq - 1 tokens");
+  release(slot);
+  const nfn_step_entry e{slot, n};
+  const int32_t want = n - 1;
+  return step(&e, 1, tokens, &want, 1, s, next_token, nullptr);
+}
+
+int layered_engine::decode(const int32_t* tokens_in, const uint8_t* active, const nfn_sampling* s, const nfn_sampling* per_slot, int32_t* next_tokens) {
+  std::vector<nfn_step_entry> entries;
+  std::vector<int32_t> tok, want, out;
+  std::vector<nfn_sampling> sam;
+  for (int b = 0; b < c.max_batch; ++b) {
+    if (!active[b]) continue;
+    if (len[b] <= 0) return efail("engine_decode: slot " + std::to_string(b) + " is active but was never prefilled");
+    if (len[b] + 1 > c.max_seq) return efail("engine_decode: slot " + std::to_string(b) + " reached max_seq");
+    want.push_back((int32_t)entries.size());
+    entries.push_back(nfn_step_entry{b, 1});
+    tok.push_back(tokens_in[b]);
+    sam.push_back(per_slot ? per_slot[b] : *s);
+    sam.back().seed = s->seed;
+  }
+  if (entries.empty()) return 0;
+  out.resize(entries.size());
+  if (step(entries.data(), (int)entries.size(), tok.data(), want.data(), (int)want.size(), sam.data(), out.data(), nullptr)) return -1;
+  for (size_t i = 0; i < entries.size(); ++i) next_tokens[entries[i].slot] = out[i];
+  return 0;
+}
+
+int layered_engine::last_logits(int slot, float* out_vocab) {
+  if (logit_at[slot] == -1) return efail("engine_last_logits: the slot's newest tokens were run without asking for logits");
+  CU(cudaSetDevice(device));
+  const float* src = logit_at[slot] == -2 ? saved + (size_t)slot * vp : logits + (size_t)logit_at[slot] * vp;
+  CU(cudaMemcpy(out_vocab, src, (size_t)c.vocab * 4, cudaMemcpyDeviceToHost));
+  return 0;
+}

@@ -7,6 +7,9 @@
 // (split-KV decode attention with fused QK-norm + RoPE + cache append, on-device sampling)
 // which is captured into a CUDA graph on first use and replayed afterwards.
 //
+// `step` (layer-list engines) is the general form: any mix of prompt portions and single tokens of
+// different slots in one batch.
+//
 // Families: 0 = GPT-2 style (LayerNorm, learned positions, GELU MLP, biases, MHA, tied head),
 //           1 = Llama style (RMSNorm, RoPE, grouped-query attention, SwiGLU, optional per-head
 //               QK norm with weights, optional sliding-window layers with ring caches).
@@ -55,6 +58,44 @@ typedef struct {
   uint64_t seed;
 } nfn_sampling;
 
+// ---- layer-list engine ------------------------------------------------------------------------------
+// A decoder given as a list of layers, each with its own sizes and constants. Layer: h = RMS(x) * norm1; x += mixer(h) + ff(h)
+// (both branches read h; one product adds both to the 32-bit residual stream); then, with side_dim > 0, a per-layer token
+// input: x += RMS(proj(gelu_tanh(gate x) * side_embed[token, layer])) * side_norm. The output norm and the tied head follow.
+typedef struct {
+  int heads, kv_heads;   // query head h reads key / value head h / (heads / kv_heads)
+  int dim, vdim;         // per-head query / key size and value size
+  int conv_taps;         // causal depthwise convolution on the projected q, k, v (<= 1: none)
+  int window;            // key j is visible to query i when 0 <= i - j < window (0: every earlier key)
+  int kv_from;           // >= 0: keys and values are those of that earlier layer (this one has none); -1: its own
+  float scale;           // score = q . k * scale - slope_h * (i - j)
+  float alibi;           // slope_h = 2^(-alibi (h + 1) / heads); 0: no distance bias
+  float q_temp_coef;     // q *= 1 + coef * ln(floor((pos + 1) / every) + 1); every = 0: off
+  int q_temp_every;
+  int out_gate;          // heads *= sigmoid(W_g h)
+  int ff;                // width of the gated feed-forward down(act(gate h) * (up h)); 0: none
+  int ff_act;            // NFN_ACT_RELU, NFN_ACT_SILU, NFN_ACT_GELU_TANH
+} nfn_layer_desc;
+
+typedef struct {
+  int n_layer, width, vocab;
+  int side_dim;          // per-layer token input size (0: none)
+  float embed_scale, norm_eps;
+  int dtype;             // 0: bf16 products and activations (norms, softmax, residual in 32-bit); 1: everything in 32-bit
+  int max_seq;           // most tokens of one sequence
+  int max_batch;         // slots
+  int kv_tokens;         // cache pool: tokens all live sequences hold together, each rounded up to a page (0: max_batch * max_seq)
+  int max_step_rows;     // most rows one internal pass runs; longer steps are cut
+  int use_cuda_graph;
+} nfn_layered_config;
+
+enum { NFN_KV_PAGE = 64 };   // tokens per cache page
+
+typedef struct {
+  int32_t slot;          // sequence
+  int32_t count;         // its next tokens in this step
+} nfn_step_entry;
+
 int nfn_engine_abi_version(void);
 const char* nfn_engine_last_error(void);
 nfn_engine* nfn_engine_create(const nfn_engine_config* cfg, int device);
@@ -88,6 +129,15 @@ int nfn_engine_prefill_rows(nfn_engine* e, int slot, const void* rows_bf16, int 
 // next_tokens[slot] receives its successor. per_slot (optional, max_batch entries) overrides `s`.
 int nfn_engine_decode(nfn_engine* e, const int32_t* tokens_in, const uint8_t* active, const nfn_sampling* s,
                       const nfn_sampling* per_slot, int32_t* next_tokens);
+// Layer-list engines: `layers` has cfg->n_layer entries.
+nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, const nfn_layer_desc* layers, int device);
+// Runs the next tokens of any number of slots as one batch: `tokens` holds the entries' tokens one after another, want_rows
+// (ascending places in `tokens`) the ones whose logits are asked for. want_sampling (n_want) and want_tokens (n_want) are given
+// together or not at all: the token drawn after each wanted place. want_logits (optional): fp32 [n_want, vocab].
+int nfn_engine_step(nfn_engine* e, const nfn_step_entry* entries, int n_entries, const int32_t* tokens, const int32_t* want_rows, int n_want,
+                    const nfn_sampling* want_sampling, int32_t* want_tokens, float* want_logits);
+// Tokens the page pool still has room for (whole free pages); -1 for engines without pages.
+long long nfn_engine_free_tokens(const nfn_engine* e);
 int nfn_engine_release(nfn_engine* e, int slot);
 int nfn_engine_slot_length(const nfn_engine* e, int slot);
 // Copies the bf16 logits of the last step for `slot` to the host as fp32 (vocab entries).

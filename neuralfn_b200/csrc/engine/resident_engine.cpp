@@ -21,8 +21,7 @@
 #include <string>
 #include <vector>
 
-#include "../kernels/nfn_kernels.h"
-#include "nfn_engine.h"
+#include "engine_core.h"
 
 extern "C" {
 // kernel-library entry points that nfn_kernels.h does not declare
@@ -40,32 +39,12 @@ int nfn_kv_cache_write(const void* qkv, int ld, void* k_cache, void* v_cache, in
 int nfn_sigmoid_gate_inplace(void* att, int ld_att, const void* gate, int ld_gate, long long rows, int width, nfn_stream_t stream);
 int nfn_rmsnorm_residual(const void* x, const void* weight, const void* resid, void* out, long long rows, int C, float eps, int centered,
                          nfn_stream_t stream);
-long long nfn_launch_count(void);
 }
+
+using nfn_eng::DevTensor;
+using nfn_eng::efail;
 
 namespace {
-
-thread_local std::string t_err;
-int efail(const std::string& m) {
-  t_err = m;
-  return -1;
-}
-#define CU(call)                                                                                       \
-  do {                                                                                                 \
-    cudaError_t e__ = (call);                                                                          \
-    if (e__ != cudaSuccess) return efail(std::string(#call) + ": " + cudaGetErrorString(e__));         \
-  } while (0)
-#define K(call)                                                                        \
-  do {                                                                                 \
-    int rc__ = (call);                                                                 \
-    if (rc__ != 0) return efail(std::string(#call) + " failed: " + nfn_last_error()); \
-  } while (0)
-
-struct DevTensor {
-  void* ptr = nullptr;
-  long long numel = 0;
-  int qtype = 0;  // 0: bf16 values; NFN_QTYPE_Q4_K / Q5_K / Q6_K: packed super-blocks of 256 values, rows back to back
-};
 
 struct StepIO {  // layout of the pinned per-step block; device mirror has the same layout
   long long tokens, lengths, positions, row_params, offset, tq_seq, tq_slot_local, tq_slot_global, out_tokens, total;
@@ -73,14 +52,8 @@ struct StepIO {  // layout of the pinned per-step block; device mirror has the s
 
 }  // namespace
 
-struct nfn_engine {
+struct block_engine final : nfn_engine {
   nfn_engine_config c{};
-  int device = 0;
-  cudaStream_t stream = nullptr;
-  std::map<std::string, DevTensor> w;
-  std::vector<std::pair<std::string, long long>> expected;
-  bool finalized = false;
-  long long bytes = 0;
   // activations
   void *x = nullptr, *xn = nullptr, *qkv = nullptr, *att = nullptr, *ff = nullptr, *ffa = nullptr, *logits = nullptr;
   float *cosT = nullptr, *sinT = nullptr;
@@ -101,10 +74,8 @@ struct nfn_engine {
   unsigned char* h_io = nullptr;
   unsigned char* d_io = nullptr;
   StepIO io{};
-  std::vector<int> len;  // tokens held per slot
-  unsigned long long steps = 0;
   cudaGraphExec_t graph = nullptr;
-  long long launches = 0, graph_launches = 0;
+  long long graph_launches = 0;
   // block verification (speculative decoding, appends at a position > 0); set up by nfn_engine_enable_verify
   int v_rows_max = 0, v_rows = 0;         // rows per slot: capacity / of the last verification
   std::vector<void*> stage_k, stage_v;    // per layer [max_batch * v_rows_max, n_kv_head * head_dim]
@@ -130,13 +101,24 @@ struct nfn_engine {
   long long wq_max_numel = 0;
   void* wq_scratch = nullptr;
 
-  int alloc(void** p, long long nbytes) {
-    CU(cudaMalloc(p, (size_t)nbytes));
-    bytes += nbytes;
-    return 0;
-  }
-  const void* W(const std::string& n) const { return w.at(n).ptr; }
-  bool has(const std::string& n) const { return w.count(n) != 0; }
+  ~block_engine() override;
+  int set_tensor_kquant(const char* name, int qtype, const void* host_blocks, long long nbytes, long long numel) override;
+  int load_dense_v5(const char* path) override;
+  int set_turboquant(const void* tq_tables) override;
+  int finalize() override;
+  int release(int slot) override;
+  int prefill(int slot, const int32_t* tokens, int n, const nfn_sampling* s, int32_t* next_token) override;
+  int prefill_rows(int slot, const void* rows_bf16, int n, int rows_on_device, const nfn_sampling* s, int32_t* next_token) override;
+  int decode(const int32_t* tokens_in, const uint8_t* active, const nfn_sampling* s, const nfn_sampling* per_slot, int32_t* next_tokens) override;
+  int last_logits(int slot, float* out_vocab) override;
+  int enable_verify(int max_rows) override;
+  int verify(const int32_t* tokens, const int32_t* n_rows, int rows, int32_t* argmax_out) override;
+  int verify_logits(int slot, int row, float* out_vocab) override;
+  int commit(const int32_t* accepted) override;
+  int truncate(int slot, int n) override;
+  int fork(int src_slot, int dst_slot, int n) override;
+  int enable_taps(const int32_t* layers, int n) override;
+  int read_taps(int slot, int pos0, int n, void* dst, int dst_on_device) override;
 };
 
 namespace {
@@ -155,7 +137,7 @@ bool layer_is_local(const nfn_engine_config& c, int l) {
   return ((l + 1) % c.global_every) != 0;
 }
 
-void build_expected(nfn_engine& e) {
+void build_expected(block_engine& e) {
   const nfn_engine_config& c = e.c;
   const long long C = c.d_model, F = c.d_ff, Vp = c.padded_vocab, HD = c.head_dim;
   const long long ATT = (long long)c.n_head * HD;
@@ -192,7 +174,7 @@ void build_expected(nfn_engine& e) {
 }
 
 // C[M, N] = A[M, K] . B[N, K]^T with the epilogue selected by flags
-int gemm(nfn_engine& e, const void* a, int lda, const void* b, void* cdst, int ldc, int m, int n, int k, int flags, const void* bias,
+int gemm(block_engine& e, const void* a, int lda, const void* b, void* cdst, int ldc, int m, int n, int k, int flags, const void* bias,
          const void* resid, int ld_resid, float act_param = 0.f, float alpha = 1.f) {
   if (!e.qtype_of.empty()) {
     const auto it = e.qtype_of.find(b);
@@ -233,7 +215,7 @@ int gemm(nfn_engine& e, const void* a, int lda, const void* b, void* cdst, int l
 // block_rows > 0 (and decode = false) the rows are max_batch blocks of block_rows rows that
 // continue each slot at d_lengths[slot]: attention reads the caches plus the block, the
 // block's K/V go to the staging buffers, the caches stay untouched.
-int forward_layers(nfn_engine& e, int rows, bool decode, int slot, const int* d_lengths, int block_rows = 0, const int* d_block_pos = nullptr,
+int forward_layers(block_engine& e, int rows, bool decode, int slot, const int* d_lengths, int block_rows = 0, const int* d_block_pos = nullptr,
                    const int* d_block_live = nullptr) {
   const nfn_engine_config& c = e.c;
   const int C = c.d_model, F = c.d_ff, HD = c.head_dim, Hq = c.n_head, Hkv = c.n_kv_head, ATT = Hq * HD;
@@ -371,7 +353,7 @@ int forward_layers(nfn_engine& e, int rows, bool decode, int slot, const int* d_
 }
 
 // final norm of rows [row0, row0 + n) -> logits[n, padded_vocab]
-int head(nfn_engine& e, int row0, int n, void* logits_dst = nullptr) {
+int head(block_engine& e, int row0, int n, void* logits_dst = nullptr) {
   const nfn_engine_config& c = e.c;
   const int C = c.d_model;
   const char* xin = static_cast<const char*>(e.x) + (size_t)row0 * C * 2;
@@ -385,13 +367,13 @@ int head(nfn_engine& e, int row0, int n, void* logits_dst = nullptr) {
   return gemm(e, e.xn, C, wh, logits_dst ? logits_dst : e.logits, c.padded_vocab, n, c.padded_vocab, C, flags, nullptr, nullptr, 0, c.logit_softcap, mult);
 }
 
-int sample(nfn_engine& e, int rows, const float* d_row_params, const unsigned long long* d_offset, int* d_out) {
+int sample(block_engine& e, int rows, const float* d_row_params, const unsigned long long* d_offset, int* d_out) {
   // every row carries its own (temperature, top_k, top_p); the Philox offset is a device word
   K(nfn_sample_rows(e.logits, 0, e.c.padded_vocab, rows, e.c.vocab, d_out, nullptr, 1.f, 0, 1.f, d_row_params, 0x5eedULL, 0ULL, d_offset, 0, e.stream));
   return 0;
 }
 
-int decode_body(nfn_engine& e) {
+int decode_body(block_engine& e) {
   const int B = e.c.max_batch;
   const int* d_tok = reinterpret_cast<const int*>(e.d_io + e.io.tokens);
   const int* d_len = reinterpret_cast<const int*>(e.d_io + e.io.lengths);
@@ -410,7 +392,7 @@ int decode_body(nfn_engine& e) {
   return sample(e, B, d_rp, d_off, d_out);
 }
 
-void fill_params(const nfn_engine& e, float* rp, int row, const nfn_sampling& s) {
+void fill_params(const block_engine& e, float* rp, int row, const nfn_sampling& s) {
   rp[3 * row] = s.temperature;
   rp[3 * row + 1] = (float)s.top_k;
   rp[3 * row + 2] = s.top_p;
@@ -421,8 +403,6 @@ void fill_params(const nfn_engine& e, float* rp, int row, const nfn_sampling& s)
 
 extern "C" {
 
-int nfn_engine_abi_version(void) { return 1; }
-const char* nfn_engine_last_error(void) { return t_err.c_str(); }
 
 nfn_engine* nfn_engine_create(const nfn_engine_config* cfg, int device) {
   if (!cfg) {
@@ -440,7 +420,7 @@ nfn_engine* nfn_engine_create(const nfn_engine_config* cfg, int device) {
     efail("engine_create: the GPT-2 family needs n_kv_head == n_head and n_head * head_dim == d_model");
     return nullptr;
   }
-  auto e = std::make_unique<nfn_engine>();
+  auto e = std::make_unique<block_engine>();
   e->c = c;
   if (e->c.embed_scale == 0.f) e->c.embed_scale = 1.f;
   e->device = device;
@@ -456,45 +436,23 @@ nfn_engine* nfn_engine_create(const nfn_engine_config* cfg, int device) {
   return e.release();
 }
 
-void nfn_engine_destroy(nfn_engine* e) {
-  if (!e) return;
-  cudaSetDevice(e->device);
-  if (e->stream) cudaStreamSynchronize(e->stream);
-  if (e->graph) cudaGraphExecDestroy(e->graph);
-  for (auto& kv : e->w) cudaFree(kv.second.ptr);
-  for (void* p : {e->x, e->xn, e->qkv, e->att, e->ff, e->ffa, e->logits, (void*)e->cosT, (void*)e->sinT, e->dec_ws, (void*)e->d_io, e->rstd, e->branch, e->ones, e->zero_pos})
-    if (p) cudaFree(p);
-  for (void* p : e->kc) cudaFree(p);
-  for (void* p : e->vc) cudaFree(p);
-  if (e->wq_scratch) cudaFree(e->wq_scratch);
-  if (e->h_io) cudaFreeHost(e->h_io);
-  if (e->stream) cudaStreamDestroy(e->stream);
-  delete e;
-}
+}  // extern "C"
 
-int nfn_engine_set_tensor(nfn_engine* e, const char* name, const void* host_bf16, long long numel) {
-  if (!e || !name || !host_bf16 || numel <= 0) return efail("engine_set_tensor: bad arguments");
-  CU(cudaSetDevice(e->device));
-  long long want = -1;
-  for (const auto& kv : e->expected)
-    if (kv.first == name) want = kv.second;
-  if (want < 0) return efail(std::string("engine_set_tensor: this configuration has no tensor named ") + name);
-  if (want != numel) return efail(std::string("engine_set_tensor: ") + name + " has " + std::to_string(numel) + " elements, expected " + std::to_string(want));
-  DevTensor& t = e->w[name];
-  if (t.qtype) return efail(std::string("engine_set_tensor: ") + name + " holds K-quant blocks");
-  if (!t.ptr) {
-    if (e->alloc(&t.ptr, numel * 2)) return -1;
-    t.numel = numel;
-  }
-  CU(cudaMemcpyAsync(t.ptr, host_bf16, (size_t)numel * 2, cudaMemcpyHostToDevice, e->stream));
-  CU(cudaStreamSynchronize(e->stream));
-  return 0;
+block_engine::~block_engine() {
+  if (graph) cudaGraphExecDestroy(graph);
+  for (void* p : {x, xn, qkv, att, ff, ffa, logits, (void*)cosT, (void*)sinT, dec_ws, gemm_ws, (void*)d_io, rstd, branch, ones, zero_pos})
+    if (p) cudaFree(p);
+  for (void* p : kc) cudaFree(p);
+  for (void* p : vc) cudaFree(p);
+  if (wq_scratch) cudaFree(wq_scratch);
+  if (h_io) cudaFreeHost(h_io);
 }
 
 // A projection weight kept in its K-quant blocks (Q4_K / Q5_K / Q6_K: `numel` values = rows of K / 256 super-blocks, rows back
 // to back, the GGUF layout). Only 2-D projection weights qualify (the embedding is gathered, norms and biases are vectors);
 // the row length must be a multiple of 256.
-int nfn_engine_set_tensor_kquant(nfn_engine* e, const char* name, int qtype, const void* host_blocks, long long nbytes, long long numel) {
+int block_engine::set_tensor_kquant(const char* name, int qtype, const void* host_blocks, long long nbytes, long long numel) {
+  block_engine* const e = this;
   if (!e || !name || !host_blocks || numel <= 0) return efail("engine_set_tensor_kquant: bad arguments");
   if (e->finalized) return efail("engine_set_tensor_kquant: call before nfn_engine_finalize");
   const int bb = nfn_quant_block_bytes(qtype);
@@ -532,19 +490,8 @@ int nfn_engine_set_tensor_kquant(nfn_engine* e, const char* name, int qtype, con
   return 0;
 }
 
-int nfn_engine_expected_tensors(const nfn_engine* e, char* buf, int cap) {
-  if (!e) return efail("engine_expected_tensors: null engine");
-  std::string s;
-  for (const auto& kv : e->expected) s += kv.first + " " + std::to_string(kv.second) + "\n";
-  if (buf && cap > 0) {
-    const size_t n = std::min<size_t>(s.size(), (size_t)cap - 1);
-    std::memcpy(buf, s.data(), n);
-    buf[n] = 0;
-  }
-  return (int)s.size();
-}
-
-int nfn_engine_load_dense_v5(nfn_engine* e, const char* path) {
+int block_engine::load_dense_v5(const char* path) {
+  block_engine* const e = this;
   if (!e || !path) return efail("engine_load_dense_v5: bad arguments");
   if (e->c.family != 0) return efail("engine_load_dense_v5: dense GPT checkpoints load into family 0 engines");
   std::ifstream in(path, std::ios::binary);
@@ -560,13 +507,14 @@ int nfn_engine_load_dense_v5(nfn_engine* e, const char* path) {
     stage.resize((size_t)kv.second * 2);
     in.read(stage.data(), (std::streamsize)stage.size());
     if (in.gcount() != (std::streamsize)stage.size()) return efail("engine_load_dense_v5: payload is truncated at " + kv.first);
-    if (nfn_engine_set_tensor(e, kv.first.c_str(), stage.data(), kv.second)) return -1;
+    if (set_tensor(kv.first.c_str(), stage.data(), kv.second)) return -1;
   }
   if (in.peek() != std::ifstream::traits_type::eof()) return efail("engine_load_dense_v5: trailing bytes after the last tensor");
   return 0;
 }
 
-int nfn_engine_set_turboquant(nfn_engine* e, const void* tq_tables) {
+int block_engine::set_turboquant(const void* tq_tables) {
+  block_engine* const e = this;
   if (!e || !tq_tables) return efail("engine_set_turboquant: null argument");
   if (e->finalized) return efail("engine_set_turboquant: call it before nfn_engine_finalize (the caches are allocated there)");
   const nfn_tq_tables* t = static_cast<const nfn_tq_tables*>(tq_tables);
@@ -581,7 +529,8 @@ int nfn_engine_set_turboquant(nfn_engine* e, const void* tq_tables) {
   return 0;
 }
 
-int nfn_engine_finalize(nfn_engine* e) {
+int block_engine::finalize() {
+  block_engine* const e = this;
   if (!e) return efail("engine_finalize: null engine");
   if (e->finalized) return 0;
   if (e->c.kv_cache_mode == 1 && !e->tq) return efail("engine_finalize: kv_cache_mode 1 needs nfn_engine_set_turboquant first");
@@ -657,20 +606,15 @@ int nfn_engine_finalize(nfn_engine* e) {
   return 0;
 }
 
-long long nfn_engine_device_bytes(const nfn_engine* e) { return e ? e->bytes : -1; }
-int nfn_engine_slot_length(const nfn_engine* e, int slot) { return (e && slot >= 0 && slot < e->c.max_batch) ? e->len[slot] : -1; }
-long long nfn_engine_launches(const nfn_engine* e) { return e ? e->launches : -1; }
-
-int nfn_engine_release(nfn_engine* e, int slot) {
+int block_engine::release(int slot) {
+  block_engine* const e = this;
   if (!e || slot < 0 || slot >= e->c.max_batch) return efail("engine_release: bad slot");
   e->len[slot] = 0;
   return 0;
 }
 
-}  // extern "C"
-
 // layers, head on the last row, sampling and bookkeeping of a prompt whose layer-0 inputs sit in e->x
-static int run_prompt_rows(nfn_engine* e, int slot, int n, const nfn_sampling* s, int32_t* next_token, long long before) {
+static int run_prompt_rows(block_engine* e, int slot, int n, const nfn_sampling* s, int32_t* next_token, long long before) {
   const nfn_engine_config& c = e->c;
   if (forward_layers(*e, n, false, slot, nullptr)) return -1;
   if (head(*e, n - 1, 1)) return -1;
@@ -695,8 +639,8 @@ static int run_prompt_rows(nfn_engine* e, int slot, int n, const nfn_sampling* s
 }
 
 
-extern "C" {
-int nfn_engine_prefill(nfn_engine* e, int slot, const int32_t* tokens, int n, const nfn_sampling* s, int32_t* next_token) {
+int block_engine::prefill(int slot, const int32_t* tokens, int n, const nfn_sampling* s, int32_t* next_token) {
+  block_engine* const e = this;
   if (!e || !tokens || !s || !next_token) return efail("engine_prefill: null argument");
   if (!e->finalized) return efail("engine_prefill: call nfn_engine_finalize first");
   const nfn_engine_config& c = e->c;
@@ -721,7 +665,8 @@ int nfn_engine_prefill(nfn_engine* e, int slot, const int32_t* tokens, int n, co
   return run_prompt_rows(e, slot, n, s, next_token, before);
 }
 
-int nfn_engine_prefill_rows(nfn_engine* e, int slot, const void* rows_bf16, int n, int rows_on_device, const nfn_sampling* s, int32_t* next_token) {
+int block_engine::prefill_rows(int slot, const void* rows_bf16, int n, int rows_on_device, const nfn_sampling* s, int32_t* next_token) {
+  block_engine* const e = this;
   if (!e || !rows_bf16 || !s || !next_token) return efail("engine_prefill_rows: null argument");
   if (!e->finalized) return efail("engine_prefill_rows: call nfn_engine_finalize first");
   const nfn_engine_config& c = e->c;
@@ -734,8 +679,9 @@ int nfn_engine_prefill_rows(nfn_engine* e, int slot, const void* rows_bf16, int 
   return run_prompt_rows(e, slot, n, s, next_token, before);
 }
 
-int nfn_engine_decode(nfn_engine* e, const int32_t* tokens_in, const uint8_t* active, const nfn_sampling* s, const nfn_sampling* per_slot,
+int block_engine::decode(const int32_t* tokens_in, const uint8_t* active, const nfn_sampling* s, const nfn_sampling* per_slot,
                       int32_t* next_tokens) {
+  block_engine* const e = this;
   if (!e || !tokens_in || !active || !s || !next_tokens) return efail("engine_decode: null argument");
   if (!e->finalized) return efail("engine_decode: call nfn_engine_finalize first");
   const nfn_engine_config& c = e->c;
@@ -804,7 +750,8 @@ int nfn_engine_decode(nfn_engine* e, const int32_t* tokens_in, const uint8_t* ac
   return 0;
 }
 
-int nfn_engine_last_logits(nfn_engine* e, int slot, float* out_vocab) {
+int block_engine::last_logits(int slot, float* out_vocab) {
+  block_engine* const e = this;
   if (!e || !out_vocab || slot < 0 || slot >= e->c.max_batch || !e->finalized) return efail("engine_last_logits: bad arguments");
   CU(cudaSetDevice(e->device));
   std::vector<uint16_t> tmp(e->c.vocab);
@@ -819,7 +766,8 @@ int nfn_engine_last_logits(nfn_engine* e, int slot, float* out_vocab) {
 
 // ---- block verification, commit, truncate, fork -------------------------------------------------
 
-int nfn_engine_enable_verify(nfn_engine* e, int max_rows) {
+int block_engine::enable_verify(int max_rows) {
+  block_engine* const e = this;
   if (!e || !e->finalized) return efail("engine_enable_verify: finalize the engine first");
   if (e->tq) return efail("engine_enable_verify: verification blocks are not available with the TurboQuant cache (decode only)");
   if (e->v_rows_max > 0) return max_rows <= e->v_rows_max ? 0 : efail("engine_enable_verify: already enabled with fewer rows");
@@ -853,7 +801,8 @@ int nfn_engine_enable_verify(nfn_engine* e, int max_rows) {
   return 0;
 }
 
-int nfn_engine_verify(nfn_engine* e, const int32_t* tokens, const int32_t* n_rows, int rows, int32_t* argmax_out) {
+int block_engine::verify(const int32_t* tokens, const int32_t* n_rows, int rows, int32_t* argmax_out) {
+  block_engine* const e = this;
   if (!e || !tokens || !n_rows || !argmax_out) return efail("engine_verify: null argument");
   if (e->v_rows_max <= 0) return efail("engine_verify: call nfn_engine_enable_verify first");
   if (rows < 1 || rows > e->v_rows_max) return efail("engine_verify: rows outside [1, max_rows]");
@@ -898,7 +847,8 @@ int nfn_engine_verify(nfn_engine* e, const int32_t* tokens, const int32_t* n_row
   return 0;
 }
 
-int nfn_engine_verify_logits(nfn_engine* e, int slot, int row, float* out_vocab) {
+int block_engine::verify_logits(int slot, int row, float* out_vocab) {
+  block_engine* const e = this;
   if (!e || !out_vocab || e->v_rows <= 0 || slot < 0 || slot >= e->c.max_batch || row < 0 || row >= e->h_vrows[slot])
     return efail("engine_verify_logits: no such verification row");
   CU(cudaSetDevice(e->device));
@@ -912,7 +862,8 @@ int nfn_engine_verify_logits(nfn_engine* e, int slot, int row, float* out_vocab)
   return 0;
 }
 
-int nfn_engine_commit(nfn_engine* e, const int32_t* accepted) {
+int block_engine::commit(const int32_t* accepted) {
+  block_engine* const e = this;
   if (!e || !accepted) return efail("engine_commit: null argument");
   if (e->v_rows <= 0) return efail("engine_commit: no verification to commit");
   const nfn_engine_config& c = e->c;
@@ -947,14 +898,15 @@ int nfn_engine_commit(nfn_engine* e, const int32_t* accepted) {
 
 // A ring cache keeps only the newest `cap` positions: once it has wrapped, the rows an earlier
 // length would need have been overwritten, so such a slot can only be truncated to its own length.
-static bool ring_prefix_intact(const nfn_engine& e, int slot, int n) {
+static bool ring_prefix_intact(const block_engine& e, int slot, int n) {
   if (n == e.len[slot]) return true;
   for (int l = 0; l < e.c.n_layer; ++l)
     if (layer_is_local(e.c, l) && e.len[slot] > e.cap[l]) return false;
   return true;
 }
 
-int nfn_engine_truncate(nfn_engine* e, int slot, int n) {
+int block_engine::truncate(int slot, int n) {
+  block_engine* const e = this;
   if (!e || slot < 0 || slot >= e->c.max_batch) return efail("engine_truncate: bad slot");
   if (n < 0 || n > e->len[slot]) return efail("engine_truncate: length outside [0, current length]");
   if (n > 0 && !ring_prefix_intact(*e, slot, n)) return efail("engine_truncate: a sliding-window cache of this slot has wrapped; only a reset is possible");
@@ -962,7 +914,8 @@ int nfn_engine_truncate(nfn_engine* e, int slot, int n) {
   return 0;
 }
 
-int nfn_engine_fork(nfn_engine* e, int src_slot, int dst_slot, int n) {
+int block_engine::fork(int src_slot, int dst_slot, int n) {
+  block_engine* const e = this;
   if (!e || !e->finalized) return efail("engine_fork: engine not ready");
   const nfn_engine_config& c = e->c;
   if (src_slot < 0 || src_slot >= c.max_batch || dst_slot < 0 || dst_slot >= c.max_batch || src_slot == dst_slot) return efail("engine_fork: bad slots");
@@ -991,7 +944,8 @@ int nfn_engine_fork(nfn_engine* e, int src_slot, int dst_slot, int n) {
   return 0;
 }
 
-int nfn_engine_enable_taps(nfn_engine* e, const int32_t* layers, int n) {
+int block_engine::enable_taps(const int32_t* layers, int n) {
+  block_engine* const e = this;
   if (!e || !e->finalized || !layers) return efail("engine_enable_taps: finalize the engine first");
   if (!e->taps.empty()) return efail("engine_enable_taps: taps are already enabled");
   if (e->graph || e->decode_calls > 0) return efail("engine_enable_taps: enable taps before the first decode step (the step is captured once)");
@@ -1011,7 +965,8 @@ int nfn_engine_enable_taps(nfn_engine* e, const int32_t* layers, int n) {
   return 0;
 }
 
-int nfn_engine_read_taps(nfn_engine* e, int slot, int pos0, int n, void* dst, int dst_on_device) {
+int block_engine::read_taps(int slot, int pos0, int n, void* dst, int dst_on_device) {
+  block_engine* const e = this;
   if (!e || !dst || e->taps.empty()) return efail("engine_read_taps: taps are not enabled");
   const nfn_engine_config& c = e->c;
   if (slot < 0 || slot >= c.max_batch || pos0 < 0 || n < 0 || pos0 + n > e->len[slot]) return efail("engine_read_taps: positions outside the slot's cached tokens");
@@ -1027,4 +982,3 @@ int nfn_engine_read_taps(nfn_engine* e, int slot, int pos0, int n, void* dst, in
   return 0;
 }
 
-}  // extern "C"

@@ -266,7 +266,8 @@ static int launch_gemm_pair(const nfn_gemm_args& a, cudaStream_t stream) {
   } else {
     if (!make_tmap_2d(&tb, a.b, 2, (uint64_t)a.n, (uint64_t)a.k, (uint64_t)a.ldb, 64, P2_BK, 128)) return -3;
   }
-  if (!make_tmap_2d(&tc, a.c, 2, (uint64_t)a.n, (uint64_t)a.m, (uint64_t)a.ldc, 64, P2_BM, 128)) return -3;
+  if (a.flags & NFN_EPI_OUT_F32) tc = ta;  // fp32 outputs are stored straight from registers
+  else if (!make_tmap_2d(&tc, a.c, 2, (uint64_t)a.n, (uint64_t)a.m, (uint64_t)a.ldc, 64, P2_BM, 128)) return -3;
   tx = tc;
   if ((a.flags & NFN_EPI_SAVE_PRE) &&
       !make_tmap_2d(&tx, a.aux_out, 2, (uint64_t)a.n, (uint64_t)a.m, (uint64_t)a.ld_aux_out, 64, P2_BM, 128))
@@ -296,7 +297,9 @@ static int launch_gemm_pair(const nfn_gemm_args& a, cudaStream_t stream) {
 // Returns 1 when the problem was launched on CTA pairs, 0 when it is not eligible, < 0 on error.
 int try_launch_gemm_pair(const nfn_gemm_args& a, cudaStream_t stream) {
   const bool out_f32 = a.flags & NFN_EPI_OUT_F32, accum = a.flags & NFN_EPI_ACCUM;
-  if (a.a_mn || out_f32 || accum || a.split_k > 1) return 0;
+  // fp32 outputs: only the residual-stream form (C += product, bf16 copy), whose epilogue is compiled as straight-line code
+  const bool residual = out_f32 && accum && (a.flags & NFN_EPI_COPY_BF16);
+  if (a.a_mn || ((out_f32 || accum) && !residual) || a.split_k > 1) return 0;
   if (a.m < 512 || a.n < 256 || a.k < 256) return 0;
   return a.b_mn ? launch_gemm_pair<true>(a, stream) : launch_gemm_pair<false>(a, stream);
 }

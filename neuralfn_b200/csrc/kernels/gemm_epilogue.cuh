@@ -147,17 +147,19 @@ enum : int {
   EPI_K_DGELU,           // C = acc * gelu_tanh'(aux_in)
   EPI_K_TANHCAP,         // C = cap * tanh(acc / cap)
   EPI_K_F32_PLAIN,       // fp32 C = acc (split-K partial slices)
+  EPI_K_F32_ACC_COPY,    // fp32 C += acc; aux_out = bf16(C) (32-bit residual streams)
 };
 
 __device__ __forceinline__ int epi_classify(const GemmParams& p) {
   if (p.alpha != 1.f) return EPI_K_GENERIC;
   const int act = (p.flags >> NFN_EPI_ACT_SHIFT) & 0xF;
-  const int base = p.flags & 0x3F;
+  const int base = p.flags & 0x7F;
   if (act == NFN_ACT_NONE) {
     if (base == 0) return EPI_K_PLAIN;
     if (base == NFN_EPI_BIAS) return EPI_K_BIAS;
     if (base == (NFN_EPI_BIAS | NFN_EPI_RESID)) return EPI_K_BIAS_RESID;
     if (base == NFN_EPI_OUT_F32) return EPI_K_F32_PLAIN;
+    if (base == (NFN_EPI_OUT_F32 | NFN_EPI_ACCUM | NFN_EPI_COPY_BF16)) return EPI_K_F32_ACC_COPY;
   } else if (act == NFN_ACT_GELU_TANH) {
     if (base == (NFN_EPI_BIAS | NFN_EPI_SAVE_PRE)) return EPI_K_BIAS_GELU_SAVE;
     if (base == NFN_EPI_DACT) return EPI_K_DGELU;
@@ -196,10 +198,32 @@ __device__ __forceinline__ void epi_chunk32(const GemmParams& p, uint32_t taddr,
 #pragma unroll
     for (int g = 0; g < 4; ++g) bias[g] = __ldg(bp + g);
   }
+  float4 held[8];
+  if (KIND == EPI_K_F32_ACC_COPY && row_ok) {
+    const float4* cp = reinterpret_cast<const float4*>(reinterpret_cast<const float*>(p.c) + (size_t)row * p.ldc + nc);
+#pragma unroll
+    for (int g = 0; g < 8; ++g) held[g] = cp[g];
+  }
   uint32_t r[32];
   tmem_ld_32x32(taddr, r);
   tmem_ld_wait();
   if (!row_ok) return;
+  if (KIND == EPI_K_F32_ACC_COPY) {
+    float4* cp = reinterpret_cast<float4*>(reinterpret_cast<float*>(p.c) + (size_t)row * p.ldc + nc);
+    uint4 o[4];
+#pragma unroll
+    for (int g = 0; g < 8; ++g) {
+      held[g].x += __uint_as_float(r[4 * g]);
+      held[g].y += __uint_as_float(r[4 * g + 1]);
+      held[g].z += __uint_as_float(r[4 * g + 2]);
+      held[g].w += __uint_as_float(r[4 * g + 3]);
+      cp[g] = held[g];
+      const uint32_t lo = pack_bf16x2(held[g].x, held[g].y), hi = pack_bf16x2(held[g].z, held[g].w);
+      if (g & 1) { o[g >> 1].z = lo; o[g >> 1].w = hi; } else { o[g >> 1].x = lo; o[g >> 1].y = hi; }
+    }
+    st_row32_bf16(p.aux_out + (size_t)row * p.ld_aux_out + nc, o, wide_aux);
+    return;
+  }
   if (KIND == EPI_K_F32_PLAIN) {
     float4* cp = reinterpret_cast<float4*>(reinterpret_cast<float*>(p.c) + (size_t)sp * p.split_stride + (size_t)row * p.ldc + nc);
 #pragma unroll

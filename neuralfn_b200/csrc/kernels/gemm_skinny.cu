@@ -30,11 +30,12 @@ constexpr int SK_WARPS = 8, SK_THREADS = SK_WARPS * 32, SK_NT = 4, SK_ROWS = SK_
 struct SkinnyParams {
   const __nv_bfloat16* a;
   const __nv_bfloat16* b;
-  __nv_bfloat16* c;
+  void* c;                // bf16, or fp32 with out_f32
+  __nv_bfloat16* copy;    // out_f32: optional bf16 copy of the result
   const __nv_bfloat16* bias;
   const __nv_bfloat16* resid;
-  int m, n, k, lda, ldb, ldc, ld_resid;
-  int act, accum;
+  int m, n, k, lda, ldb, ldc, ld_resid, ld_copy;
+  int act, accum, out_f32;
   float alpha, act_param;
 };
 
@@ -57,6 +58,20 @@ __device__ __forceinline__ float sk_act(float v, int act, float prm) {
     case NFN_ACT_RELU: return fmaxf(v, 0.f);
     case NFN_ACT_TANH_CAP: return prm * fast_tanh(v / prm);
     default: return v;
+  }
+}
+
+// accumulate and store one finished value
+__device__ __forceinline__ void sk_store(const SkinnyParams& p, int r, int n, float v) {
+  if (p.out_f32) {
+    float* cp = static_cast<float*>(p.c) + (size_t)r * p.ldc + n;
+    if (p.accum) v += *cp;
+    *cp = v;
+    if (p.copy) p.copy[(size_t)r * p.ld_copy + n] = __float2bfloat16(v);
+  } else {
+    __nv_bfloat16* cp = static_cast<__nv_bfloat16*>(p.c) + (size_t)r * p.ldc + n;
+    if (p.accum) v += __bfloat162float(*cp);
+    *cp = __float2bfloat16(v);
   }
 }
 
@@ -141,9 +156,7 @@ gemm_skinny_kernel(const SkinnyParams p) {
     if (p.bias) v += __bfloat162float(p.bias[n]);
     v = sk_act(v, p.act, p.act_param);
     if (p.resid) v += __bfloat162float(p.resid[(size_t)r * p.ld_resid + n]);
-    __nv_bfloat16* cp = p.c + (size_t)r * p.ldc + n;
-    if (p.accum) v += __bfloat162float(*cp);
-    *cp = __float2bfloat16(v);
+    sk_store(p, r, n, v);
   }
 }
 
@@ -320,9 +333,7 @@ gemm_skinny_resident_kernel(const SkinnyParams p, const int S, const int pass_co
       if (p.bias) v += __bfloat162float(p.bias[n]);
       v = sk_act(v, p.act, p.act_param);
       if (p.resid) v += __bfloat162float(p.resid[(size_t)r * p.ld_resid + n]);
-      __nv_bfloat16* cp = p.c + (size_t)r * p.ldc + n;
-      if (p.accum) v += __bfloat162float(*cp);
-      *cp = __float2bfloat16(v);
+      sk_store(p, r, n, v);
     }
     rs_cluster_sync();                                                    // nobody overwrites a strip a peer still reads
   }
@@ -387,7 +398,7 @@ static int g_skinny_mode = 1;
 // Returns 1 when it launched, 0 when the product is not one of its cases (the caller continues with the tcgen05 path),
 // negative on a launch error.
 int try_launch_skinny(const nfn_gemm_args& a, cudaStream_t stream) {
-  const int unsupported = NFN_EPI_SAVE_PRE | NFN_EPI_DACT | NFN_EPI_OUT_F32;
+  const int unsupported = NFN_EPI_SAVE_PRE | NFN_EPI_DACT;
   if (!g_skinny_mode || a.m < 3 || a.m > 64 || a.a_mn || a.b_mn || (a.flags & unsupported) || (a.k & 31) || a.k < 256 || (a.lda & 7) || (a.ldb & 7))
     return 0;
   // measured (12288 x 6656 weights, L2 flushed): 8 rows 49 us against 52 us on the tcgen05 split-K path, 32 rows 65 against
@@ -403,7 +414,10 @@ int try_launch_skinny(const nfn_gemm_args& a, cudaStream_t stream) {
   SkinnyParams p;
   p.a = static_cast<const __nv_bfloat16*>(a.a);
   p.b = static_cast<const __nv_bfloat16*>(a.b);
-  p.c = static_cast<__nv_bfloat16*>(a.c);
+  p.c = a.c;
+  p.out_f32 = (a.flags & NFN_EPI_OUT_F32) ? 1 : 0;
+  p.copy = (a.flags & NFN_EPI_COPY_BF16) ? static_cast<__nv_bfloat16*>(a.aux_out) : nullptr;
+  p.ld_copy = a.ld_aux_out;
   p.bias = (a.flags & NFN_EPI_BIAS) ? static_cast<const __nv_bfloat16*>(a.bias) : nullptr;
   p.resid = (a.flags & NFN_EPI_RESID) ? static_cast<const __nv_bfloat16*>(a.aux_in) : nullptr;
   p.m = a.m; p.n = a.n; p.k = a.k; p.lda = a.lda; p.ldb = a.ldb; p.ldc = a.ldc; p.ld_resid = a.ld_aux_in;

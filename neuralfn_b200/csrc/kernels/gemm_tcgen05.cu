@@ -16,7 +16,7 @@ namespace nfn {
 // out[m, n] = alpha * sum_s part[s][m][n] (+ out when accumulate); bf16 or fp32 output
 __global__ void __launch_bounds__(256)
 splitk_reduce_kernel(const float* __restrict__ part, long long slice, int splits, void* out, int ldc,
-                     int m, int n, float alpha, int out_f32, int accumulate) {
+                     int m, int n, float alpha, int out_f32, int accumulate, __nv_bfloat16* copy, int ld_copy) {
   const int vec_per_row = n / 8;
   const long long idx = (long long)blockIdx.x * 256 + threadIdx.x;
   if (idx >= (long long)m * vec_per_row) return;
@@ -38,6 +38,7 @@ splitk_reduce_kernel(const float* __restrict__ part, long long slice, int splits
     }
     reinterpret_cast<float4*>(cp)[0] = make_float4(v[0], v[1], v[2], v[3]);
     reinterpret_cast<float4*>(cp)[1] = make_float4(v[4], v[5], v[6], v[7]);
+    if (copy) *reinterpret_cast<uint4*>(copy + (size_t)row * ld_copy + col) = pack8_bf16(v);
   } else {
     __nv_bfloat16* cp = static_cast<__nv_bfloat16*>(out) + (size_t)row * ldc + col;
     if (accumulate) {
@@ -144,7 +145,7 @@ static int launch_gemm(const nfn_gemm_args& a, int split_k, cudaStream_t stream,
     const long long total = (long long)a.m * (a.n / 8);
     splitk_reduce_kernel<<<(unsigned)((total + 255) / 256), 256, 0, stream>>>(
         static_cast<const float*>(a.workspace), (long long)a.m * a.n, split_k, a.c, a.ldc, a.m, a.n,
-        a.alpha, out_f32 ? 1 : 0, accum ? 1 : 0);
+        a.alpha, out_f32 ? 1 : 0, accum ? 1 : 0, (a.flags & NFN_EPI_COPY_BF16) ? static_cast<__nv_bfloat16*>(a.aux_out) : nullptr, a.ld_aux_out);
     launched = 2;
   }
   return launch_check("gemm", launched);
@@ -230,6 +231,9 @@ extern "C" int nfn_gemm_bf16(const nfn_gemm_args* args, nfn_stream_t stream_) {
   if ((a.flags & NFN_EPI_SAVE_PRE) &&
       (!a.aux_out || (a.ld_aux_out & 7) || (reinterpret_cast<uintptr_t>(a.aux_out) & 15)))
     return fail(-1, "gemm: aux_out missing or misaligned");
+  if ((a.flags & NFN_EPI_COPY_BF16) && (!(a.flags & NFN_EPI_OUT_F32) || (a.flags & NFN_EPI_SAVE_PRE) || !a.aux_out || (a.ld_aux_out & 7) ||
+                                        (reinterpret_cast<uintptr_t>(a.aux_out) & 15)))
+    return fail(-1, "gemm: the bf16 copy goes with an fp32 output and its own aligned aux_out");
 
   if (a.m <= 2 && gemv_mode() != 0) {  // one or two rows: pure weight streaming (gemv_bf16.cu)
     const int rc = try_launch_gemv(a, stream);

@@ -18,11 +18,12 @@ namespace nfn {
 struct GemvParams {
   const __nv_bfloat16* a;
   const __nv_bfloat16* b;
-  __nv_bfloat16* c;
+  void* c;                // bf16, or fp32 with out_f32
+  __nv_bfloat16* copy;    // out_f32: optional bf16 copy of the result
   const __nv_bfloat16* bias;
   const __nv_bfloat16* resid;
-  int n, k, lda, ldb, ldc, ld_resid;
-  int act, accum;
+  int n, k, lda, ldb, ldc, ld_resid, ld_copy;
+  int act, accum, out_f32;
   float alpha, act_param;
 };
 
@@ -111,9 +112,16 @@ gemv_bf16_kernel(const GemvParams p) {
         if (p.bias) v += __bfloat162float(p.bias[n]);
         v = gemv_act(v, p.act, p.act_param);
         if (p.resid) v += __bfloat162float(p.resid[(size_t)m * p.ld_resid + n]);
-        __nv_bfloat16* cp = p.c + (size_t)m * p.ldc + n;
-        if (p.accum) v += __bfloat162float(*cp);
-        *cp = __float2bfloat16(v);
+        if (p.out_f32) {
+          float* cp = static_cast<float*>(p.c) + (size_t)m * p.ldc + n;
+          if (p.accum) v += *cp;
+          *cp = v;
+          if (p.copy) p.copy[(size_t)m * p.ld_copy + n] = __float2bfloat16(v);
+        } else {
+          __nv_bfloat16* cp = static_cast<__nv_bfloat16*>(p.c) + (size_t)m * p.ldc + n;
+          if (p.accum) v += __bfloat162float(*cp);
+          *cp = __float2bfloat16(v);
+        }
       }
     }
   }
@@ -122,12 +130,15 @@ gemv_bf16_kernel(const GemvParams p) {
 // Returns 1 when it launched, 0 when the product is not a GEMV case (the caller continues with the
 // tensor-core path), negative on a launch error.
 int try_launch_gemv(const nfn_gemm_args& a, cudaStream_t stream) {
-  const int unsupported = NFN_EPI_SAVE_PRE | NFN_EPI_DACT | NFN_EPI_OUT_F32;
+  const int unsupported = NFN_EPI_SAVE_PRE | NFN_EPI_DACT;
   if (a.m > 2 || a.a_mn || a.b_mn || (a.flags & unsupported) || (a.k & 7) || a.k < 256) return 0;
   GemvParams p;
   p.a = static_cast<const __nv_bfloat16*>(a.a);
   p.b = static_cast<const __nv_bfloat16*>(a.b);
-  p.c = static_cast<__nv_bfloat16*>(a.c);
+  p.c = a.c;
+  p.out_f32 = (a.flags & NFN_EPI_OUT_F32) ? 1 : 0;
+  p.copy = (a.flags & NFN_EPI_COPY_BF16) ? static_cast<__nv_bfloat16*>(a.aux_out) : nullptr;
+  p.ld_copy = a.ld_aux_out;
   p.bias = (a.flags & NFN_EPI_BIAS) ? static_cast<const __nv_bfloat16*>(a.bias) : nullptr;
   p.resid = (a.flags & NFN_EPI_RESID) ? static_cast<const __nv_bfloat16*>(a.aux_in) : nullptr;
   p.n = a.n; p.k = a.k; p.lda = a.lda; p.ldb = a.ldb; p.ldc = a.ldc; p.ld_resid = a.ld_aux_in;

@@ -43,6 +43,7 @@ enum {
   NFN_EPI_DACT = 1 << 3,      // multiply by act'(aux_in[M,N]) (aux_in = saved pre-activation)
   NFN_EPI_ACCUM = 1 << 4,     // C += result
   NFN_EPI_OUT_F32 = 1 << 5,   // C is fp32
+  NFN_EPI_COPY_BF16 = 1 << 6, // with OUT_F32: also write bf16 of the final C to aux_out (ld = ld_aux_out)
   NFN_EPI_ACT_SHIFT = 8,      // activation id in bits 8..11
 };
 enum { NFN_ACT_NONE = 0, NFN_ACT_GELU_TANH = 1, NFN_ACT_GELU_ERF = 2, NFN_ACT_SILU = 3,
@@ -295,6 +296,80 @@ int nfn_diff_combine(const void* a, const void* lambda, float out_scale, float e
                      long long tokens, int H, int D, nfn_stream_t stream);
 int nfn_diff_combine_backward(const void* dout, const void* a, const void* lambda, float out_scale, const float* rstd,
                               void* da, float* partial, void* dlambda, long long tokens, int H, int D, nfn_stream_t stream);
+
+// ---- steps of mixed batches over paged caches (paged_rows.cu, paged_decode.cu, paged_prefill.cu) ----------------------------
+// A step's rows are the next tokens of several sequences, one sequence ("entry") after another. Activations are bf16 (f32 = 0)
+// or fp32 (f32 = 1), weights bf16, the residual stream fp32. Row widths are multiples of 16.
+// Cache pages hold NFN_KV_PAGE = 64 tokens: keys [page][kv_heads][64][dim_p], values transposed [page][kv_heads][vdim_p][64];
+// table[slot * table_ld + position / 64] names the page.
+typedef struct {
+  int row0, n;         // rows of this tile (at most 16, not crossing a multiple of 16 positions)
+  int e_row0, e_n;     // first row and row count of the entry it belongs to
+  int e_pos0;          // position of the entry's first row
+  int slot;            // < 0: padding, skipped
+  int parity;          // which half of the convolution state holds the entry's history (the other one is written)
+  int pad;
+} nfn_row_tile;
+// Row pass: base = embed[token] * embed_scale (tokens != NULL) or x[src_rows ? src_rows[r] : r]; with y: base += y / rms(y) *
+// y_weight; x_out (optional) = base; h (optional) = base / rms(base) * weight. rms(z) = sqrt(sum z^2 / width + eps).
+typedef struct {
+  int f32, rows, width, ld;               // ld: row pitch of x, y, h and of the embedding table
+  const float* x; float* x_out; const int* src_rows;
+  const int* tokens; const void* embed; float embed_scale; int vocab;
+  const void* y; const void* y_weight;
+  void* h; const void* weight;
+  float eps;
+} nfn_row_norm_args;
+int nfn_row_norm(const nfn_row_norm_args* args, nfn_stream_t stream);
+// After the input projection [q | k | v | g | gate | up] of a layer: causal depthwise convolution on q, k, v over the entry's
+// rows and the stored history (conv: bf16 [taps][nq + nk + nv], NULL when taps <= 1), query temperature, keys and values into
+// their pages, ff_out = act(gate) * up. nk = nv = 0: the layer reads another layer's cache.
+typedef struct {
+  int f32;
+  const void* in; int ld_in;
+  int nq, nk, nv, off_gate, off_up, ff, act;
+  const void* conv; int taps;
+  void* state; long long state_half;      // [2][slots][taps - 1][nq + nk + nv]; elements between the halves
+  void* q_out; int ld_q;
+  void* k_pool; void* v_pool; int kv_heads, dim_p, vdim_p;
+  const int* table; int table_ld;
+  float temp_coef; int temp_every;
+  void* ff_out; int ld_ff;
+  const nfn_row_tile* tiles; int n_tiles;
+} nfn_mix_args;
+int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream);
+// Attention of a step's rows over the pages. score = q . k * scale - slopes[h] * (i - j), keys 0 <= i - j < window (0: all),
+// softmax, out = P V * sigmoid(gate) (gate optional). q: [rows, heads * dim_p]; out: row pitch ld_o, head pitch vdim_p.
+typedef struct {
+  int f32;
+  const void* q; int ld_q;
+  const void* k_pool; const void* v_pool; int kv_heads, dim_p, vdim_p; long long pages;
+  const int* table; int table_ld;
+  int heads, window;
+  float scale; const float* slopes;       // fp32 [heads], NULL: no distance bias
+  const void* gate; int ld_gate;
+  void* out; int ld_o;
+  const int* row_slot; const int* row_pos; // per row (slot < 0: skipped)
+  int rows;                               // nfn_paged_attention_rows: rows [row0, row0 + rows)
+  int row0;
+  int max_keys;                           // most keys a row of this call sees (sizes the split)
+  void* workspace; long long workspace_bytes;   // split partials; the first 64 KB are counters, zeroed once
+  const int* tiles; int n_tiles;          // nfn_paged_attention_tiles: {row0, rows, slot, pos0} each
+  int total_rows;                         // rows of the q buffer
+} nfn_paged_attention_args;
+// One query row at a time (single tokens, very short portions): bf16 goes to the tensor cores in 32-key steps, fp32 and sizes
+// outside its limits to the plain kernel.
+int nfn_paged_attention_rows(const nfn_paged_attention_args* args, nfn_stream_t stream);
+long long nfn_paged_attention_workspace_bytes(int rows, int heads, int vdim_p);
+// Tiles of consecutive rows of one sequence (prompt portions), tcgen05. nfn_paged_tile_rows: rows per tile for these sizes, 0 when
+// the sizes need nfn_paged_attention_rows.
+int nfn_paged_tile_rows(int f32, int heads, int kv_heads, int dim_p, int vdim_p);
+int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, nfn_stream_t stream);
+// out = gelu_tanh(gate) * side_embed[token][col0 + c]: gate fp32 [rows, ld], out bf16 / fp32 with the same pitch.
+int nfn_side_mul(int f32, const float* gate, const int* tokens, const void* side_embed, long long ld_embed, int col0, int vocab, void* out,
+                 int ld, int rows, int width, nfn_stream_t stream);
+// C[M, N] (fp32) (+)= A[M, K] (fp32) . B[N, K]^T (bf16), true 32-bit arithmetic. K, leading dimensions multiples of 4.
+int nfn_gemm_f32(const float* a, int lda, const void* b, int ldb, float* c, int ldc, int m, int n, int k, int accumulate, nfn_stream_t stream);
 
 #ifdef __cplusplus
 }

@@ -62,28 +62,64 @@ def _compile_one(src: Path, obj: Path, extra: list[str], verbose: bool) -> str:
     return proc.stderr if verbose else ""
 
 
-def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool = False) -> Path:
-    """Compile the CUDA kernel library; returns the path of the shared object."""
-    LIB_DIR.mkdir(parents=True, exist_ok=True)
-    OBJ_DIR.mkdir(parents=True, exist_ok=True)
-    out = LIB_DIR / "libnfn_b200_kernels.so"
-    # the resident inference engine (host C++ driving the kernels) lives in the same library,
-    # so it shares the library's CUDA runtime instance and needs no extra link step
-    sources = sorted(KERNEL_SRC.glob("*.cu")) + sorted(ENGINE_SRC.glob("*.cpp"))
+# Components: the sources one kind of model needs, built into a library of their own by ``ensure_component``. "all" is the whole library.
+COMPONENTS: dict[str, tuple[str, ...]] = {
+    "layered": ("common.cu", "gemm_tcgen05.cu", "gemm_2cta.cu", "gemv_bf16.cu", "gemm_skinny.cu", "sampling.cu", "paged_rows.cu", "paged_decode.cu",
+                "paged_prefill.cu", "engine_core.cpp", "layered_engine.cpp"),
+}
+
+
+def _sources(component: str = "all") -> list[Path]:
+    # the resident inference engines (host C++ driving the kernels) live in the same library,
+    # so they share the library's CUDA runtime instance and need no extra link step
+    every = sorted(KERNEL_SRC.glob("*.cu")) + sorted(ENGINE_SRC.glob("*.cpp"))
+    if component == "all":
+        return every
+    wanted = set(COMPONENTS[component])
+    return [s for s in every if s.name in wanted]
+
+
+def _library(component: str) -> Path:
+    return LIB_DIR / ("libnfn_b200_kernels.so" if component == "all" else f"libnfn_b200_{component}.so")
+
+
+def _object_plan(sources: list[Path]) -> list[tuple[Path, Path, Path, str, bool]]:
+    """(source, object, stamp, digest, up to date) per source."""
     headers = sorted(list(KERNEL_SRC.glob("*.h")) + list(KERNEL_SRC.glob("*.cuh")) + list(KERNEL_SRC.glob("*.inc")) +
                      list(ENGINE_SRC.glob("*.h")))
     hdr_digest = _digest(headers)
-    extra = ["-Xptxas", "-v"] if ptxas_info else []
-    jobs = []
-    objs = []
+    plan = []
     for src in sources:
-        obj = OBJ_DIR / (src.stem + ".o")
-        stamp = OBJ_DIR / (src.stem + ".sha")
+        obj, stamp = OBJ_DIR / (src.stem + ".o"), OBJ_DIR / (src.stem + ".sha")
         want = hashlib.sha256((hdr_digest + _digest([src])).encode()).hexdigest()
-        objs.append(obj)
-        if not force and obj.exists() and stamp.exists() and stamp.read_text() == want:
-            continue
-        jobs.append((src, obj, stamp, want))
+        plan.append((src, obj, stamp, want, obj.exists() and stamp.exists() and stamp.read_text() == want))
+    return plan
+
+
+def ensure_component(component: str) -> Path:
+    """The library a model of this component runs on: the whole kernel library when it is there and up to date, else the component's
+    own, built (or brought up to date) first. One build at a time; others wait for it."""
+    import fcntl
+    whole = _library("all")
+    if whole.exists() and all(p[4] for p in _object_plan(_sources("all"))):
+        return whole
+    if component == "all":
+        return build_kernels()
+    OBJ_DIR.mkdir(parents=True, exist_ok=True)
+    with open(OBJ_DIR / ".lock", "w") as lock:
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return build_kernels(component=component)
+
+
+def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool = False, component: str = "all") -> Path:
+    """Compile the CUDA kernel library (or one component of it); returns the path of the shared object."""
+    LIB_DIR.mkdir(parents=True, exist_ok=True)
+    OBJ_DIR.mkdir(parents=True, exist_ok=True)
+    out = _library(component)
+    extra = ["-Xptxas", "-v"] if ptxas_info else []
+    plan = _object_plan(_sources(component))
+    objs = [p[1] for p in plan]
+    jobs = [p[:4] for p in plan if force or not p[4]]
     if jobs:
         with concurrent.futures.ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             futs = {ex.submit(_compile_one, s, o, extra, ptxas_info): (s, st, w) for s, o, st, w in jobs}
@@ -95,12 +131,14 @@ def build_kernels(force: bool = False, verbose: bool = False, ptxas_info: bool =
                     print(f"[build] {s.name}", file=sys.stderr)
                 if ptxas_info and log:
                     print(log, file=sys.stderr)
-    if jobs or not out.exists():
-        cmd = [_nvcc(), "-shared", "-o", str(out), *map(str, objs),
+    if jobs or not out.exists() or any(o.stat().st_mtime > out.stat().st_mtime for o in objs):
+        part = out.with_suffix(f".{os.getpid()}.part")
+        cmd = [_nvcc(), "-shared", "-o", str(part), *map(str, objs),
                "-gencode", "arch=compute_100a,code=sm_100a", "-Xcompiler", "-fPIC"]
         proc = subprocess.run(cmd, capture_output=True, text=True)
         if proc.returncode != 0:
             raise RuntimeError(f"link failed:\n{proc.stdout}\n{proc.stderr}")
+        os.replace(part, out)
     return out
 
 

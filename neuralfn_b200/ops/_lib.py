@@ -33,8 +33,18 @@ class GemmArgs(ctypes.Structure):
     ]
 
 
+_CHOSEN: Path | None = None
+
+
 def lib_path() -> Path:
-    return Path(os.environ.get("NFN_B200_KERNEL_LIB", _LIB_PATH))
+    return Path(os.environ.get("NFN_B200_KERNEL_LIB", _CHOSEN or _LIB_PATH))
+
+
+def use_library(path) -> None:
+    """Choose the shared object to load (a component built for one kind of model, see ``_build.ensure_component``). Has no effect
+    once a library is loaded."""
+    global _CHOSEN
+    _CHOSEN = Path(path)
 
 
 def available() -> bool:

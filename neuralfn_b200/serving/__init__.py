@@ -1,8 +1,8 @@
 """Serving: resident inference engine bindings, generation loop, HTTP endpoints."""
-from .engine import (EngineConfig, EngineError, ResidentEngine, Sampling, resident_inference_abi_version,
+from .engine import (EngineConfig, EngineError, LayeredEngineConfig, LayerSpec, ResidentEngine, Sampling, StepEntry, resident_inference_abi_version,
                      resident_inference_capabilities)
 
-__all__ = ["EngineConfig", "EngineError", "ResidentEngine", "Sampling", "resident_inference_abi_version",
+__all__ = ["EngineConfig", "EngineError", "LayerSpec", "LayeredEngineConfig", "ResidentEngine", "StepEntry", "Sampling", "resident_inference_abi_version",
            "resident_inference_capabilities"]
 
 from .chat import (AssistantResponse, ByteTextCodec, ChatConfigurationError, ChatMessage, ChatRenderer, HuggingFaceTokenizerJSONCodec,  # noqa: E402,F401

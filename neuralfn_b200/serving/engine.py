@@ -6,7 +6,10 @@ activations stay on the GPU; Python passes token ids in and gets token ids back.
     out = eng.generate([[15496, 11], [40]], max_new_tokens=32, sampling=Sampling(temperature=0.8, top_p=0.95))
 
 ``generate`` is a continuous-batching loop: prompts are prefetched into free slots as
-earlier sequences finish, and every decode step advances all live slots at once.
+earlier sequences finish, and every decode step advances all live slots at once. Engines of
+layer-list models (``LayeredEngineConfig``) also run arbitrary steps - portions of some prompts
+beside single tokens of other sequences, ``ResidentEngine.step`` - and ``generate`` drives them
+through the scheduler of ``serving.scheduler``.
 Counterpart of the reference's ``_native_inference`` module and its Python wrapper
 (``csrc/native_gpt2/resident_binding.cpp``, ``neuralfn/native_inference.py``).
 """
@@ -20,7 +23,7 @@ import torch
 
 from ..ops import _lib
 
-__all__ = ["EngineConfig", "Sampling", "ResidentEngine", "resident_inference_abi_version", "resident_inference_capabilities"]
+__all__ = ["EngineConfig", "LayerSpec", "LayeredEngineConfig", "StepEntry", "Sampling", "ResidentEngine", "resident_inference_abi_version", "resident_inference_capabilities"]
 
 
 class _CConfig(C.Structure):
@@ -47,6 +50,121 @@ class Sampling:
 
     def c(self) -> _CSampling:
         return _CSampling(self.temperature, self.top_k, self.top_p, self.seed)
+
+
+class _CLayer(C.Structure):
+    _fields_ = [("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("conv_taps", C.c_int), ("window", C.c_int),
+                ("kv_from", C.c_int), ("scale", C.c_float), ("alibi", C.c_float), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int),
+                ("out_gate", C.c_int), ("ff", C.c_int), ("ff_act", C.c_int)]
+
+
+class _CLayeredConfig(C.Structure):
+    _fields_ = [("n_layer", C.c_int), ("width", C.c_int), ("vocab", C.c_int), ("side_dim", C.c_int), ("embed_scale", C.c_float),
+                ("norm_eps", C.c_float), ("dtype", C.c_int), ("max_seq", C.c_int), ("max_batch", C.c_int), ("kv_tokens", C.c_int),
+                ("max_step_rows", C.c_int), ("use_cuda_graph", C.c_int)]
+
+
+class _CEntry(C.Structure):
+    _fields_ = [("slot", C.c_int32), ("count", C.c_int32)]
+
+
+KV_PAGE = 64   # tokens per cache page of a layer-list engine
+
+
+@dataclass(frozen=True)
+class LayerSpec:
+    """One layer of a layer-list model (field meanings: ``nfn_layer_desc`` in csrc/engine/nfn_engine.h)."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    conv_taps: int = 1
+    window: int = 0
+    kv_from: int = -1
+    alibi: float = 0.0
+    q_temp_coef: float = 0.0
+    q_temp_every: int = 0
+    out_gate: int = 0
+    ff: int = 0
+    ff_act: str = "relu"
+
+    FF_ACT_IDS = {"gelu": 1, "silu": 3, "relu": 6}
+
+    def c(self) -> _CLayer:
+        return _CLayer(self.heads, self.kv_heads, self.dim, self.vdim, self.conv_taps, self.window, self.kv_from, self.scale, self.alibi,
+                       self.q_temp_coef, self.q_temp_every, self.out_gate, self.ff, self.FF_ACT_IDS[self.ff_act])
+
+
+@dataclass(frozen=True)
+class LayeredEngineConfig:
+    """A model given layer by layer, served from paged caches. ``dtype`` "bfloat16": products and activations in bf16, norms, softmax,
+    residual stream and constants in 32-bit; "float32": everything in 32-bit (no TF32). ``kv_tokens``: tokens the cache pool holds for
+    all sequences together, each rounded up to a page of 64 (0: ``max_batch`` sequences of ``max_seq``)."""
+    layers: tuple[LayerSpec, ...]
+    width: int
+    vocab: int
+    side_dim: int = 0
+    embed_scale: float = 1.0
+    norm_eps: float = 1e-5
+    dtype: str = "bfloat16"
+    max_seq: int = 4096
+    max_batch: int = 8
+    kv_tokens: int = 0
+    max_step_rows: int = 8192
+    use_cuda_graph: int = 1
+
+    family = 2
+    kv_cache_mode = 0
+
+    def __post_init__(self) -> None:
+        if self.dtype not in ("bfloat16", "float32"):
+            raise ValueError("dtype must be bfloat16 or float32")
+
+    @property
+    def d_model(self) -> int:
+        return self.width
+
+    @property
+    def n_layer(self) -> int:
+        return len(self.layers)
+
+    @property
+    def window(self) -> int:
+        """Widest window when every layer has one, else 0."""
+        return 0 if any(y.window == 0 for y in self.layers) else max(y.window for y in self.layers)
+
+    def create(self, lib, device: int):
+        cc = _CLayeredConfig(len(self.layers), self.width, self.vocab, self.side_dim, self.embed_scale, self.norm_eps,
+                             int(self.dtype == "float32"), self.max_seq, self.max_batch, self.kv_tokens, self.max_step_rows, self.use_cuda_graph)
+        arr = (_CLayer * len(self.layers))(*[y.c() for y in self.layers])
+        return lib.nfn_engine_create_layered(C.byref(cc), arr, device)
+
+    def estimate_device_bytes(self) -> int:
+        """Weights, page pools and activations of an engine with this configuration."""
+        up = lambda v: (v + 15) // 16 * 16  # noqa: E731
+        es, wp = (4 if self.dtype == "float32" else 2), up(self.width)
+        rows = min(self.max_step_rows, max(self.max_seq, self.max_batch))
+        pool = self.kv_tokens or self.max_batch * ((self.max_seq + KV_PAGE - 1) // KV_PAGE * KV_PAGE)
+        weights, cache, widest = wp * up(self.vocab) + self.vocab * self.n_layer * up(self.side_dim), 0, 0
+        for y in self.layers:
+            q, v = y.heads * up(y.dim), y.heads * up(y.vdim)
+            kv = 0 if y.kv_from >= 0 else y.kv_heads * (up(y.dim) + up(y.vdim))
+            n_in = q + kv + (v if y.out_gate else 0) + 2 * up(y.ff)
+            weights += wp * (n_in + v + up(y.ff) + 2 * up(self.side_dim))
+            cache += kv * pool * es
+            widest = max(widest, n_in + q + v + up(y.ff))
+        acts = rows * (es * (3 * wp + widest + up(self.side_dim)) + 4 * (wp + up(self.side_dim))) + 4 * 2 * max(self.max_batch, 64) * up(self.vocab)
+        return int(2 * weights + cache + acts)
+
+
+@dataclass(frozen=True)
+class StepEntry:
+    """The next tokens of one slot in a step; ``want``: places among them whose logits (and, with sampling, successors) are asked for."""
+    slot: int
+    tokens: Sequence[int]
+    want: Sequence[int] = ()
+    sampling: Sampling | None = None
 
 
 @dataclass
@@ -116,37 +234,30 @@ class EngineConfig:
     def c(self) -> _CConfig:
         return _CConfig(*[getattr(self, f.name) for f in fields(self)])
 
+    def create(self, lib, device: int):
+        return lib.nfn_engine_create(C.byref(self.c()), device)
+
 
 def _api():
     L = _lib.load()
     if getattr(L, "_engine_ready", False):
         return L
-    vp, ip = C.c_void_p, C.c_int
-    L.nfn_engine_last_error.restype = C.c_char_p
-    L.nfn_engine_create.restype, L.nfn_engine_create.argtypes = vp, [C.POINTER(_CConfig), ip]
-    L.nfn_engine_destroy.restype, L.nfn_engine_destroy.argtypes = None, [vp]
-    L.nfn_engine_set_tensor.argtypes = [vp, C.c_char_p, vp, C.c_longlong]
-    L.nfn_engine_set_tensor_kquant.argtypes = [vp, C.c_char_p, ip, vp, C.c_longlong, C.c_longlong]
-    L.nfn_engine_expected_tensors.argtypes = [vp, C.c_char_p, ip]
-    L.nfn_engine_load_dense_v5.argtypes = [vp, C.c_char_p]
-    L.nfn_engine_finalize.argtypes = [vp]
-    L.nfn_engine_set_turboquant.argtypes = [vp, vp]
-    L.nfn_engine_device_bytes.restype, L.nfn_engine_device_bytes.argtypes = C.c_longlong, [vp]
-    L.nfn_engine_prefill.argtypes = [vp, ip, vp, ip, C.POINTER(_CSampling), vp]
-    L.nfn_engine_decode.argtypes = [vp, vp, vp, C.POINTER(_CSampling), vp, vp]
-    L.nfn_engine_release.argtypes = [vp, ip]
-    L.nfn_engine_slot_length.argtypes = [vp, ip]
-    L.nfn_engine_last_logits.argtypes = [vp, ip, vp]
-    L.nfn_engine_launches.restype, L.nfn_engine_launches.argtypes = C.c_longlong, [vp]
-    L.nfn_engine_enable_verify.argtypes = [vp, ip]
-    L.nfn_engine_verify.argtypes = [vp, vp, vp, ip, vp]
-    L.nfn_engine_verify_logits.argtypes = [vp, ip, ip, vp]
-    L.nfn_engine_commit.argtypes = [vp, vp]
-    L.nfn_engine_truncate.argtypes = [vp, ip, ip]
-    L.nfn_engine_fork.argtypes = [vp, ip, ip, ip]
-    L.nfn_engine_prefill_rows.argtypes = [vp, ip, vp, ip, ip, C.POINTER(_CSampling), vp]
-    L.nfn_engine_enable_taps.argtypes = [vp, vp, ip]
-    L.nfn_engine_read_taps.argtypes = [vp, ip, ip, ip, vp, ip]
+    vp, ip, ll, sp = C.c_void_p, C.c_int, C.c_longlong, C.POINTER(_CSampling)
+    table = {
+        "last_error": (C.c_char_p, []), "create": (vp, [C.POINTER(_CConfig), ip]), "create_layered": (vp, [C.POINTER(_CLayeredConfig), C.POINTER(_CLayer), ip]),
+        "destroy": (None, [vp]), "set_tensor": (ip, [vp, C.c_char_p, vp, ll]), "set_tensor_kquant": (ip, [vp, C.c_char_p, ip, vp, ll, ll]),
+        "expected_tensors": (ip, [vp, C.c_char_p, ip]), "load_dense_v5": (ip, [vp, C.c_char_p]), "finalize": (ip, [vp]), "set_turboquant": (ip, [vp, vp]),
+        "device_bytes": (ll, [vp]), "prefill": (ip, [vp, ip, vp, ip, sp, vp]), "decode": (ip, [vp, vp, vp, sp, vp, vp]), "release": (ip, [vp, ip]),
+        "step": (ip, [vp, vp, ip, vp, vp, ip, vp, vp, vp]), "free_tokens": (ll, [vp]),
+        "slot_length": (ip, [vp, ip]), "last_logits": (ip, [vp, ip, vp]), "launches": (ll, [vp]), "enable_verify": (ip, [vp, ip]),
+        "verify": (ip, [vp, vp, vp, ip, vp]), "verify_logits": (ip, [vp, ip, ip, vp]), "commit": (ip, [vp, vp]), "truncate": (ip, [vp, ip, ip]),
+        "fork": (ip, [vp, ip, ip, ip]), "prefill_rows": (ip, [vp, ip, vp, ip, ip, sp, vp]), "enable_taps": (ip, [vp, vp, ip]),
+        "read_taps": (ip, [vp, ip, ip, ip, vp, ip]),
+    }
+    for name, (res, args) in table.items():
+        fn = getattr(L, "nfn_engine_" + name, None)       # a library built for one kind of model has no creator for the other
+        if fn is not None:
+            fn.restype, fn.argtypes = res, args
     L._engine_ready = True
     return L
 
@@ -156,7 +267,9 @@ def resident_inference_abi_version() -> int:
 
 
 def resident_inference_capabilities() -> dict:
-    return {"abi_version": resident_inference_abi_version(), "families": ["gpt2", "llama"], "kv_cache": "bf16",
+    return {"abi_version": resident_inference_abi_version(), "families": ["gpt2", "llama", "layered"], "kv_cache": "bf16",
+            # layer-list models: paged caches, steps of mixed prompt portions and single tokens, bf16 or true 32-bit
+            "paged_kv_cache": ["layered"], "mixed_steps": ["layered"], "float32": ["layered"],
             "hybrid_local_global": True, "qk_norm": True, "rope": ["hf", "legacy"], "continuous_batching": True,
             "cuda_graph_decode": True, "on_device_sampling": ["greedy", "temperature", "top_k", "top_p"],
             # projection weights may stay resident in K-quant blocks (``set_tensor_kquant``: quantised GEMV for up to eight rows,
@@ -171,12 +284,11 @@ class EngineError(RuntimeError):
 
 
 class ResidentEngine:
-    def __init__(self, config: EngineConfig, device: int = 0, *, turboquant_profile: str = "mse-3.5", turboquant_seed: int = 0) -> None:
+    def __init__(self, config: "EngineConfig | LayeredEngineConfig", device: int = 0, *, turboquant_profile: str = "mse-3.5", turboquant_seed: int = 0) -> None:
         self.config = config
         self.device = int(device)
         self._L = _api()
-        cc = config.c()
-        self._h = self._L.nfn_engine_create(C.byref(cc), device)
+        self._h = config.create(self._L, device)
         if not self._h:
             raise EngineError(self._err())
         self._finalized = False
@@ -201,8 +313,10 @@ class ResidentEngine:
 
     @property
     def kv_bytes_per_token(self) -> int:
-        """Cache bytes one token occupies in a global (full-context) layer."""
+        """Cache bytes one token occupies in a global (full-context) layer; in all layers together for a layer-list model."""
         c = self.config
+        if c.family == 2:
+            return sum(y.kv_heads * (y.dim + y.vdim) for y in c.layers if y.kv_from < 0) * (4 if c.dtype == "float32" else 2)
         if c.kv_cache_mode == 1:
             return c.n_kv_head * (self.turboquant.key_layout.record_bytes + self.turboquant.value_layout.record_bytes)
         return 2 * c.n_kv_head * c.head_dim * 2
@@ -335,6 +449,45 @@ class ResidentEngine:
                                               C.cast(ps, C.c_void_p) if ps is not None else None, C.cast(out, C.c_void_p)))
         return {slot: int(out[slot]) for slot in tokens_in}
 
+    # ---- steps of mixed batches (layer-list models) ----------------------------------------
+    @property
+    def has_steps(self) -> bool:
+        return self.config.family == 2
+
+    @property
+    def has_verify(self) -> bool:
+        """Block verification (speculative decoding) and truncation to any prefix."""
+        return self.config.family != 2
+
+    @property
+    def free_tokens(self) -> int:
+        """Tokens the cache pool still has whole pages for."""
+        return int(self._L.nfn_engine_free_tokens(self._h))
+
+    def step(self, entries: Sequence[StepEntry], *, logits: bool = False) -> tuple[list[list[int]], torch.Tensor | None]:
+        """Runs the next tokens of several slots as one batch. Returns, per entry, the token drawn after each wanted place (greedy
+        unless the entry has its own sampling), and with ``logits`` the fp32 rows [wanted places of all entries, vocab]."""
+        tokens: list[int] = []
+        want: list[int] = []
+        sam: list[_CSampling] = []
+        for e in entries:
+            sampling = (e.sampling or Sampling()).c()
+            for w in e.want:
+                if not 0 <= w < len(e.tokens):
+                    raise EngineError("a wanted place lies outside its entry")
+                want.append(len(tokens) + w)
+                sam.append(sampling)
+            tokens.extend(int(t) for t in e.tokens)
+        n, k = len(entries), len(want)
+        ce = (_CEntry * n)(*[_CEntry(e.slot, len(e.tokens)) for e in entries])
+        tok, wr, out, ps = (C.c_int32 * len(tokens))(*tokens), (C.c_int32 * k)(*want), (C.c_int32 * k)(), (_CSampling * k)(*sam)
+        lg = torch.empty(k, self.config.vocab, dtype=torch.float32) if logits else None
+        addr = lambda a: C.cast(a, C.c_void_p)  # noqa: E731
+        self._check(self._L.nfn_engine_step(self._h, addr(ce), n, addr(tok), addr(wr), k, addr(ps), addr(out),
+                                            C.c_void_p(lg.data_ptr()) if lg is not None and k else None))
+        drawn = iter(out)
+        return [[int(next(drawn)) for _ in e.want] for e in entries], lg
+
     def release(self, slot: int) -> None:
         self._check(self._L.nfn_engine_release(self._h, slot))
 
@@ -402,6 +555,8 @@ class ResidentEngine:
     def append(self, slot: int, tokens: Sequence[int], chunk: int | None = None) -> int:
         """Extends a slot that already holds tokens (``prefill`` only starts at position 0).
         Returns the most likely next token."""
+        if self.has_steps:
+            return self.step([StepEntry(slot, tokens, (len(tokens) - 1,))])[0][0][0]
         if not getattr(self, "_verify_rows", 0):
             self.enable_verify()
         chunk = min(chunk or self._verify_rows, self._verify_rows)
@@ -422,6 +577,12 @@ class ResidentEngine:
                  eos_token: int | None = None) -> list[list[int]]:
         """Continuous batching over ``max_batch`` slots; returns the generated ids per prompt."""
         prompts = [list(p) for p in prompts]
+        if self.has_steps:
+            from .scheduler import StepScheduler
+            sched = StepScheduler(self)
+            ids = [sched.submit(p, max_new_tokens, sampling, eos_token) for p in prompts]
+            done = sched.run()
+            return [done[i] for i in ids]
         results: list[list[int]] = [[] for _ in prompts]
         pending = list(range(len(prompts)))[::-1]
         live: dict[int, int] = {}       # slot -> prompt index
