@@ -237,7 +237,17 @@ def _infer_artifact(a) -> int:
                    allow_unauthenticated_remote=a.allow_unauthenticated_remote, sessions=a.max_batch, state_db=a.state_db)
         return 0
     from ..serving import GenerationConfig, NativeInferenceModel, NativeModelLoadConfig, NGramProposer
-    model = NativeInferenceModel.load(a.checkpoint, NativeModelLoadConfig(session_count=1, speculative_decoding=a.speculative_decoding))
+    prompts = [[int(t) for t in p.split(",") if t] for p in a.prompt_tokens.split(";") if p]
+    model = NativeInferenceModel.load(a.checkpoint, NativeModelLoadConfig(session_count=max(1, min(len(prompts), a.max_batch)), dtype=a.dtype,
+                                                                         context_tokens=a.context_tokens or None, speculative_decoding=a.speculative_decoding))
+    if len(prompts) > 1:
+        from ..serving import Sampling
+        out = model.engine.generate(prompts, max_new_tokens=a.max_new_tokens, eos_token=a.eos_token if a.eos_token >= 0 else None,
+                                    sampling=Sampling(temperature=a.temperature, top_k=a.top_k, top_p=a.top_p, seed=a.seed))
+        print(json.dumps({"status": "ok", "prompts": prompts, "generated": out, "device_bytes": model.engine.device_bytes,
+                          "kernel_launches": model.engine.launches}))
+        model.close()
+        return 0
     if getattr(a, "companion_checkpoint", ""):
         model.attach_dflash(a.companion_checkpoint)                    # a DFlash assistant exported by the distillation trainer
     if a.chat:
@@ -436,7 +446,7 @@ def build_parser() -> argparse.ArgumentParser:
     mig = sub.add_parser("migrate", help="lower a graph (and weights) to a native execution artifact: nfn migrate graph-to-native --graph G --output-dir D")
     graph_cli.add_migrate_arguments(mig)
     mig.set_defaults(fn=graph_cli.cmd_migrate)
-    i = sub.add_parser("infer", help="generate from a dense checkpoint file or an artifact directory; --serve starts the HTTP server")
+    i = sub.add_parser("infer", help="generate from a dense checkpoint file, an artifact directory or a model directory (config.json + safetensors); --serve starts the HTTP server")
     i.add_argument("--checkpoint", required=True)
     i.add_argument("--prompt-tokens", default="", help="comma-separated ids; ';' separates prompts")
     i.add_argument("--prompt", default=None, help="text prompt (artifact directories with a text codec)")
@@ -456,6 +466,8 @@ def build_parser() -> argparse.ArgumentParser:
     i.add_argument("--seed", type=int, default=1337)
     i.add_argument("--eos-token", type=int, default=-1)
     i.add_argument("--max-batch", type=int, default=8)
+    i.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16", help="model directories: number format of the engine")
+    i.add_argument("--context-tokens", type=int, default=0, help="directories: longest sequence (0: the model's own or the engine's default)")
     i.set_defaults(fn=cmd_infer)
     c = sub.add_parser("inspect-checkpoint", help="validate and checksum a dense checkpoint")
     c.add_argument("path")

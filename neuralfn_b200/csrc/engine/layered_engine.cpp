@@ -154,7 +154,7 @@ int layered_engine::build() {
     cat_max = std::max(cat_max, L.n_cat);
     want(lname(l, "norm1"), wp);
     want(lname(l, "w_in"), (long long)L.n_in * wp);
-    if (d.conv_taps > 1) want(lname(l, "conv"), (long long)d.conv_taps * (L.nq + L.nk + L.nv));
+    if (d.conv_taps > 0) want(lname(l, "conv"), (long long)d.conv_taps * (L.nq + L.nk + L.nv));
     want(lname(l, "w_out"), (long long)wp * L.n_cat);
     if (sp) {
       want(lname(l, "side_gate"), (long long)sp * wp);
@@ -264,8 +264,8 @@ int layered_engine::finalize() {
     if (d.conv_taps > 1) {
       L.state_half = S * (d.conv_taps - 1) * (L.nq + L.nk + L.nv);
       if (zero(&L.state, 2 * L.state_half * es)) return -1;
-      L.conv = W(lname(l, "conv"));
     }
+    if (d.conv_taps > 0) L.conv = W(lname(l, "conv"));
     if (d.alibi != 0.f) {
       std::vector<float> sl(d.heads);
       for (int i = 0; i < d.heads; ++i) sl[i] = (float)std::exp2(-(double)d.alibi * (i + 1) / d.heads);

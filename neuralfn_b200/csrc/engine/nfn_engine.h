@@ -65,7 +65,7 @@ typedef struct {
 typedef struct {
   int heads, kv_heads;   // query head h reads key / value head h / (heads / kv_heads)
   int dim, vdim;         // per-head query / key size and value size
-  int conv_taps;         // causal depthwise convolution on the projected q, k, v (<= 1: none)
+  int conv_taps;         // causal depthwise convolution on the projected q, k, v (0: none; 1: a factor per channel)
   int window;            // key j is visible to query i when 0 <= i - j < window (0: every earlier key)
   int kv_from;           // >= 0: keys and values are those of that earlier layer (this one has none); -1: its own
   float scale;           // score = q . k * scale - slope_h * (i - j)

@@ -322,7 +322,7 @@ typedef struct {
 } nfn_row_norm_args;
 int nfn_row_norm(const nfn_row_norm_args* args, nfn_stream_t stream);
 // After the input projection [q | k | v | g | gate | up] of a layer: causal depthwise convolution on q, k, v over the entry's
-// rows and the stored history (conv: bf16 [taps][nq + nk + nv], NULL when taps <= 1), query temperature, keys and values into
+// rows and the stored history (conv: bf16 [taps][nq + nk + nv], NULL and taps = 0: none), query temperature, keys and values into
 // their pages, ff_out = act(gate) * up. nk = nv = 0: the layer reads another layer's cache.
 typedef struct {
   int f32;

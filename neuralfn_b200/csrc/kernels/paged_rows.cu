@@ -135,7 +135,7 @@ mix_rows_kernel(const nfn_mix_args p) {
     }
   }
   auto convolve = [&](int ti, float (&acc)[8]) {
-    if (taps <= 1) {
+    if (!p.conv) {
       load8(static_cast<const T*>(p.in) + (size_t)(t.e_row0 + ti) * p.ld_in + col, acc);
       return;
     }
@@ -393,7 +393,7 @@ extern "C" int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream) {
   if (a.n_tiles <= 0) return 0;
   if ((a.nq | a.nk | a.nv | a.ff | a.ld_in | a.ld_q | a.ld_ff | a.off_gate | a.off_up | a.dim_p | a.vdim_p) & 7)
     return fail(-1, "mix_rows: widths and offsets must be multiples of 8");
-  if (a.taps > 1 && (!a.conv || !a.state)) return fail(-1, "mix_rows: a convolution needs its weights and history");
+  if ((a.taps > 0) != (a.conv != nullptr) || (a.taps > 1 && !a.state)) return fail(-1, "mix_rows: a convolution needs its weights and history");
   if (a.n_tiles > 65535) return fail(-1, "mix_rows: too many row tiles in one launch");
   const int vecs = (a.nq + a.nk + a.nv + a.ff) / 8;
   const dim3 grid(ceil_div(vecs, MIX_THREADS), a.n_tiles);

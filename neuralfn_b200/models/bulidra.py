@@ -90,7 +90,7 @@ class BulidraConfig:
                 if kv_from >= i or layers[kv_from].kv_from is not None:
                     raise BulidraError(f"{where}: kv_from must name an earlier layer that has keys and values of its own")
             layers.append(BulidraLayer(
-                heads, kv_heads, _int(_need(m, "dim", where), where), _int(_need(m, "vdim", where), where), _int(m.get("conv", 1), where),
+                heads, kv_heads, _int(_need(m, "dim", where), where), _int(_need(m, "vdim", where), where), _int(m.get("conv") or 0, where, 0),
                 float(_need(m, "scale", where)), _int(_need(mask, "size", where), where) if mask is not None else 0,
                 float(_need(temp, "coef", where)) if temp is not None else 0.0, _int(_need(temp, "every", where), where) if temp is not None else 0,
                 kv_from, _int(_need(mlp, "ff", where), where) if mlp is not None else 0))
@@ -132,7 +132,8 @@ def expected_shapes(cfg: BulidraConfig) -> dict[str, tuple[int, ...]]:
             rows.update(k=y.kv_heads * y.dim, v=y.kv_heads * y.vdim)
         for n, r in rows.items():
             out[p + f"mix.{n}"] = (r, w)
-            out[p + f"mix.{n}.conv"] = (r, y.conv)
+            if y.conv:
+                out[p + f"mix.{n}.conv"] = (r, y.conv)
         out[p + "mix.g"], out[p + "mix.o"] = (y.heads * y.vdim, w), (w, y.heads * y.vdim)
         if y.ff:
             out[p + "mlp.gate"], out[p + "mlp.up"], out[p + "mlp.down"] = (y.ff, w), (y.ff, w), (w, y.ff)
@@ -198,7 +199,7 @@ def pack_tensors(cfg: BulidraConfig, tensors: Mapping[str, torch.Tensor]) -> dic
             o.append(_pad_rows(T[p + "mlp.down"].T, 1, fp))
         out[q + "norm1"] = vec(p + "norm1")
         out[q + "w_in"] = torch.cat(rows)
-        if y.conv > 1:
+        if y.conv:
             out[q + "conv"] = torch.cat([_pad_rows(T[p + f"mix.{n}.conv"], g, to) for n, g, to in heads]).T.contiguous()
         out[q + "w_out"] = _pad_rows(torch.cat(o).T.contiguous(), 1, wp)
         if sp:

@@ -10,6 +10,7 @@ Execution routes in this framework:
   * ``native-gpt``    - ``models/gpt2.py`` + ``trainers/dense_gpt.py`` (explicit forward/backward
                         on the tcgen05 kernel library, one CUDA graph per step, DP/TP)
   * ``native-llama``  - ``models/llama.py`` (same trainer; DP, PP stages)
+  * ``serving-only``  - the layer-list resident engine (``serving/architectures.py``); no trainer
   * ``tensor-runtime``- the graph compiler + ``TorchTrainer`` (every preset runs here; the hot
                         stages call the kernel library)
 The reference ships one native binary per family (``nfn_<family>_native_train``); the family
@@ -30,7 +31,7 @@ class NativeTrainerSpec:
     aliases: tuple[str, ...]
     reference_binary: str
     presets: tuple[str, ...]
-    route: str                      # native-gpt | native-llama | native-moe | tensor-runtime
+    route: str                      # native-gpt | native-llama | native-moe | serving-only | tensor-runtime
     resident_inference: bool = False
     parallel: tuple[str, ...] = ()
     checkpoint_formats: tuple[str, ...] = ()
@@ -72,6 +73,7 @@ NATIVE_FAMILIES: dict[str, NativeTrainerSpec] = {s.family: s for s in (
     _spec("muse-glimmer", ("glimmer",), ("muse_glimmer",), resident_inference=True, checkpoint_formats=("named-tensors", "gguf")),
     _spec("deepseek-v4", (), ("deepseek_v4",)), _spec("jepa", (), ("jepa",)), _spec("semantic-dense-jepa", (), ("semantic_dense_jepa",)),
     _spec("moe-jepa-evo", (), ("moe_jepa_evo",)), _spec("semantic-router-moe", (), ("semantic_router_moe",)), _spec("jamba", (), ("jamba",)),
+    NativeTrainerSpec("bulidra", (), "", (), "serving-only", resident_inference=True, checkpoint_formats=("model-directory",)),
     _spec("seq2seq", (), ("seq2seq",)), _spec("diffusion", (), ("diffusion",)), _spec("ttt-llama", (), ("ttt_llama",)),
     _spec("hnet-lm", (), ("hnet_lm",)), _spec("universal-llama", (), ("universal_llama",)),
 )}
@@ -123,7 +125,9 @@ def capability_proof_for(name: str) -> NativeCapabilityProof:
         route = "tensor-runtime"
         reasons.append(f"preset {preset} uses blocks outside the expert-parallel MoE Llama (shared experts, aux-free balancing, MLA)")
     native_training = route in ("native-gpt", "native-llama", "native-moe")
-    if not native_training and not reasons:
+    if route == "serving-only":
+        reasons.append("served from model directories by the layer-list engine; the reference has no such family and no trainer is built for it")
+    elif not native_training and not reasons:
         reasons.append("the family trains through the graph compiler and TorchTrainer; its hot stages call the kernel library")
     if not spec.resident_inference:
         reasons.append("no resident-engine block layout for this family; inference runs through the tensor runtime")

@@ -79,7 +79,7 @@ class LayerSpec:
     dim: int
     vdim: int
     scale: float
-    conv_taps: int = 1
+    conv_taps: int = 0
     window: int = 0
     kv_from: int = -1
     alibi: float = 0.0

@@ -30,7 +30,7 @@ from typing import Any, Callable, Protocol, Sequence
 import torch
 
 from .chat import IncrementalTokenDecoder, TextCodec, TokenIdTextCodec, load_text_codec
-from .engine import EngineConfig, ResidentEngine, Sampling, resident_inference_abi_version
+from .engine import EngineConfig, LayeredEngineConfig, LayerSpec, ResidentEngine, Sampling, resident_inference_abi_version
 
 __all__ = ["InferenceError", "NativeInferenceCapabilities", "GenerationConfig", "KVCacheConfig", "NativeModelLoadConfig", "GenerationEvent",
            "GenerationResult", "Proposer", "NGramProposer", "DraftEngineProposer", "DFlashProposer", "target_embed_and_head", "NativeInferenceModel", "NativeInferenceSession",
@@ -124,6 +124,7 @@ class NativeModelLoadConfig:
     session_count: int = 1
     companion_checkpoints: tuple[str, ...] = ()
     speculative_decoding: str = "auto"  # off | auto | required
+    dtype: str = "bfloat16"            # model directories whose engine has it: float32 runs everything in 32-bit
 
     def __post_init__(self) -> None:
         if self.weight_precision not in ("auto", "bf16", "k-quant-dynamic", "k-quant-17gb"):
@@ -134,6 +135,8 @@ class NativeModelLoadConfig:
             raise ValueError("speculative_decoding must be off, auto or required")
         if self.session_count < 1:
             raise ValueError("session_count must be >= 1")
+        if self.dtype not in ("bfloat16", "float32"):
+            raise ValueError("dtype must be bfloat16 or float32")
 
 
 @dataclass(frozen=True)
@@ -347,7 +350,10 @@ class NativeInferenceModel:
         root = Path(artifact_dir)
         path = root / MANIFEST_NAME
         if not path.is_file():
-            raise InferenceError(f"{root} has no {MANIFEST_NAME}")
+            from .architectures import architecture_of, is_model_directory, read_model_config
+            if is_model_directory(root):
+                return cls._load_model_directory(root, architecture_of(read_model_config(root)), load_config or NativeModelLoadConfig(), **kw)
+            raise InferenceError(f"{root} has no {MANIFEST_NAME} and no config.json of a known architecture")
         manifest = json.loads(path.read_text(encoding="utf-8"))
         if manifest.get("schema") != MANIFEST_SCHEMA:
             raise InferenceError(f"unsupported manifest schema {manifest.get('schema')!r}")
@@ -356,17 +362,49 @@ class NativeInferenceModel:
         fields["max_batch"] = max(int(fields.get("max_batch", 1)), lc.session_count)
         if lc.context_tokens:
             fields["max_seq"] = min(int(fields["max_seq"]), int(lc.context_tokens))
-        cfg = EngineConfig(**fields)
-        if torch.cuda.is_available():
-            free, _total = torch.cuda.mem_get_info(lc.cuda_device)
-            need = cls.estimate_device_bytes(cfg)
-            if need + (lc.vram_reserve_bytes or 0) > free:
-                raise InferenceError(f"artifact needs ~{need >> 20} MiB on the device, {free >> 20} MiB free (reserve {lc.vram_reserve_bytes or 0})")
+        if "layers" in fields:
+            fields["layers"] = tuple(LayerSpec(**y) for y in fields["layers"])
+            cfg = LayeredEngineConfig(**fields)
+        else:
+            cfg = EngineConfig(**fields)
+        cls._check_fits(cfg, lc)
         engine = ResidentEngine(cfg, device=lc.cuda_device)
         from ..checkpoint.named import read_named_tensors
         engine.load_named_tensors(read_named_tensors(root / manifest["weights"])[0])
         codec = load_text_codec(manifest.get("text_codec"), root)
         return cls(engine, codec=codec, manifest=manifest, artifact_root=root, load_config=lc, **kw)
+
+    @classmethod
+    def _load_model_directory(cls, root: Path, arch, lc: NativeModelLoadConfig, **kw) -> "NativeInferenceModel":
+        """A directory with ``config.json`` + safetensors of a registered architecture (``serving.architectures``)."""
+        from .architectures import read_model_config
+        raw = read_model_config(root)
+        limits: dict[str, Any] = {"max_batch": lc.session_count, "dtype": lc.dtype}
+        if lc.context_tokens:
+            limits["max_seq"] = int(lc.context_tokens)
+        cfg, tensors = arch.build(root, raw, **limits)
+        cls._check_fits(cfg, lc)
+        engine = ResidentEngine(cfg, device=lc.cuda_device)
+        engine.load_named_tensors(tensors)
+        return cls(engine, manifest={"architecture": arch.name, "family": arch.family}, artifact_root=root, load_config=lc, **kw)
+
+    @classmethod
+    def _check_fits(cls, cfg, lc: NativeModelLoadConfig) -> None:
+        if torch.cuda.is_available():
+            free, _total = torch.cuda.mem_get_info(lc.cuda_device)
+            need = cls.estimate_device_bytes(cfg)
+            if need + (lc.vram_reserve_bytes or 0) > free:
+                raise InferenceError(f"artifact needs ~{need >> 20} MiB on the device, {free >> 20} MiB free (reserve {lc.vram_reserve_bytes or 0})")
+
+    def _shorten(self, slot: int, tokens: Sequence[int]) -> None:
+        """Leaves ``slot`` with exactly ``tokens``, a prefix of what it holds: cut where the engine's state can be cut, run again where
+        it cannot (short-convolution histories hold the newest rows only)."""
+        if getattr(self.engine, "has_verify", True):
+            self.engine.truncate(slot, len(tokens))
+        elif not tokens:
+            self.engine.release(slot)
+        elif len(tokens) != self.engine.slot_length(slot):
+            self.engine.prefill(slot, list(tokens))
 
     def attach_dflash(self, assistant, *, target_tensors: dict[str, torch.Tensor] | None = None) -> None:
         """Makes a DFlash (block-diffusion) draft the model's speculative proposer. ``assistant``: the file written by
@@ -408,6 +446,8 @@ class NativeInferenceModel:
     @staticmethod
     def estimate_device_bytes(cfg: EngineConfig) -> int:
         """Weights + KV caches + activations of an engine with this configuration."""
+        if isinstance(cfg, LayeredEngineConfig):
+            return cfg.estimate_device_bytes()
         hd, kvw = cfg.head_dim, cfg.n_kv_head * cfg.head_dim
         att = cfg.n_head * hd
         per_layer = (att + 2 * kvw) * cfg.d_model + att * cfg.d_model + (3 if cfg.family == 1 else 2) * cfg.d_model * cfg.d_ff
@@ -423,7 +463,7 @@ class NativeInferenceModel:
     @property
     def capabilities(self) -> NativeInferenceCapabilities:
         return NativeInferenceCapabilities(resident_inference_abi=resident_inference_abi_version(),
-                                           speculative_decoding=self.load_config.speculative_decoding != "off")
+                                           speculative_decoding=self.load_config.speculative_decoding != "off" and getattr(self.engine, "has_verify", True))
 
     @property
     def closed(self) -> bool:
@@ -489,7 +529,10 @@ class NativeInferenceModel:
             origin = child._origin
             try:
                 if origin is not None:
-                    self.engine.fork(origin[0].slot, slot, origin[1])
+                    if getattr(self.engine, "has_verify", True) or self.engine.slot_length(origin[0].slot) == origin[1]:
+                        self.engine.fork(origin[0].slot, slot, origin[1])
+                    else:
+                        self.engine.prefill(slot, child._tokens)      # the state at the prefix's end is gone: run it again
                     self._counters["fork_copies"] = self._counters.get("fork_copies", 0) + 1
             except Exception:
                 self._free.append(slot)
@@ -511,7 +554,7 @@ class NativeInferenceModel:
                 heir = max(session._dependants, key=lambda c: c._origin[1])
                 slot, rows = session._slot, heir._origin[1]
                 if rows < self.engine.slot_length(slot):
-                    self.engine.truncate(slot, rows)
+                    self._shorten(slot, heir._tokens)
                 for other in session._dependants:
                     if other is not heir:
                         other._origin = (heir, other._origin[1])
@@ -714,7 +757,7 @@ class NativeInferenceSession:
             # keep n - 1 tokens cached and make the n-th the pending one: running it again is what
             # yields the logits that follow the shortened history
             if n - 1 < len(self._tokens):
-                self.model.engine.truncate(self.slot, n - 1)
+                self.model._shorten(self.slot, every[:n - 1])
             self._tokens, self._pending, self._next_greedy = every[:n - 1], every[n - 1], None
 
     def reset(self) -> None:
@@ -764,6 +807,8 @@ class NativeInferenceSession:
             proposer = self.model.dflash_proposer(self)
         if proposer is None and self.model.proposer_factory is not None and spec_mode != "off":
             proposer = self.model.proposer_factory()
+        if not getattr(self.model.engine, "has_verify", True):
+            proposer = None
         if spec_mode == "required" and proposer is None:
             raise InferenceError("speculative decoding is required but no proposer is available")
         if allowed_tokens is not None:
