@@ -5,6 +5,7 @@ per GPU, synthetic uniform-random token ids, gpt2-normal random init.
 
     python bench.py --gpus N --steps K --warmup W            # this framework
     python bench.py --impl reference --gpus N --steps K ...  # unmodified reference (Torch path)
+    python bench.py --serving bulidra                        # prefill / decode of a served design beside the closest existing model
 
 For N > 1 launch under ``python -m torch.distributed.run --nproc-per-node N``. Rank 0
 prints one JSON line. ``value`` is device-timed (CUDA events, max over ranks) over K
@@ -213,7 +214,13 @@ def main() -> None:
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--check-fused", action="store_true",
                     help="run the fused-collective kernel self-check also on one GPU (always on for N > 1)")
+    ap.add_argument("--serving", choices=["bulidra"], default=None,
+                    help="instead of the training benchmark: prefill and decode throughput of this design and of Glimmer blocks of equal size")
     args = ap.parse_args()
+    if args.serving:
+        from neuralfn_b200.bench.serving_bench import run as run_serving
+        run_serving(args, ClockSampler)
+        return
     out = run_reference(args) if args.impl == "reference" else run_ours(args)
     if out:
         print(json.dumps(out), flush=True)

@@ -1,0 +1,106 @@
+"""Prefill and decode throughput of Bulidra and, at equal size, of Glimmer blocks - the closest model the engine served before: grouped
+heads, sliding windows, gated attention, gated feed-forward. Random bf16 weights; one JSON line per model, size and phase.
+
+``ms`` is device time (CUDA events on the engine's stream, median over repetitions of the public ``prefill`` / ``decode`` call,
+including its host-to-device copy of tokens and the read-back of the drawn token); weights and caches are larger than L2. Beside it
+stand the bytes (decode) or floating-point operations (prefill) the phase cannot avoid and the fraction of the measured peaks.
+"""
+from __future__ import annotations
+
+import json
+import os
+import statistics
+
+import torch
+
+SIZES = {
+    "w2048": dict(width=2048, heads=16, kv_heads=4, dim=128, ff=5632, window=1024, layers=8, vocab=32768),
+    "w4096": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=14336, window=1024, layers=6, vocab=32768),
+    "w4096_wide_window": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=14336, window=4096, layers=6, vocab=32768),
+}
+SIDE_DIM = 256
+
+
+def _peaks() -> tuple[float, float]:
+    path = os.path.join(os.path.dirname(__file__), "..", "..", "MEASURED_PEAKS.json")
+    if os.path.exists(path):
+        p = json.load(open(path))
+        return p["hbm_gbs"] * 1e9, p["bf16_tflops"] * 1e12
+    return 6.65e12, 1.59e15
+
+
+def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
+    from ..models.bulidra import BulidraConfig, BulidraLayer, engine_config
+    from ..serving import EngineConfig, ResidentEngine
+    if kind == "bulidra":
+        L = z["layers"]
+        layers = tuple(BulidraLayer(z["heads"], z["kv_heads"], z["dim"], z["dim"], 4, z["dim"] ** -0.5, z["window"], 0.1, 1024, None, z["ff"]) for _ in range(L))
+        cfg = engine_config(BulidraConfig(z["vocab"], z["width"], 1.0, 1e-5, SIDE_DIM, layers), max_batch=max_batch, max_seq=max_seq, max_step_rows=max_seq)
+    else:
+        cfg = EngineConfig.glimmer(n_layer=z["layers"], d_model=z["width"], n_head=z["heads"], n_kv_head=z["kv_heads"], head_dim=z["dim"], d_ff=z["ff"],
+                                   vocab=z["vocab"], max_seq=max_seq, window=z["window"], max_batch=max_batch, global_every=0, tie_embeddings=1)
+    eng = ResidentEngine(cfg)
+    g = torch.Generator(device="cuda").manual_seed(0)
+    for n, k in eng.expected_tensors().items():
+        t = torch.ones(k, device="cuda") if "norm" in n else torch.randn(k, generator=g, device="cuda") * 0.02
+        eng.set_tensor(n, t.bfloat16())
+    eng.finalize()
+    return eng
+
+
+def _time(eng, fn, n: int, warmup: int) -> float:
+    for _ in range(warmup):
+        fn()
+    pairs = [(torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)) for _ in range(n)]
+    with torch.cuda.stream(eng.stream):
+        for a, b in pairs:
+            a.record()
+            fn()
+            b.record()
+    torch.cuda.synchronize()
+    return statistics.median(a.elapsed_time(b) for a, b in pairs)
+
+
+def _work(z: dict, kind: str, prompt: int, batch: int, context: int) -> tuple[float, float]:
+    """(FLOPs of a prompt, bytes of a decode step): products and attention over visible keys; weights and visible cache rows."""
+    w, q, kv = z["width"], z["heads"] * z["dim"], z["kv_heads"] * z["dim"]
+    per = w * (q + 2 * kv + q + 2 * z["ff"]) + w * (q + z["ff"]) + (2 * w * SIDE_DIM if kind == "bulidra" else 0)
+    win = min(z["window"], prompt)
+    keys = win * (win + 1) / 2 + (prompt - win) * win
+    flops = z["layers"] * (2.0 * per * prompt + 4.0 * q * keys)
+    seen = min(z["window"], context)
+    return flops, 2.0 * z["layers"] * (per + batch * seen * 2 * kv) + 2.0 * z["vocab"] * w
+
+
+def run(args, clock_sampler, sizes=None) -> None:
+    hbm, tf = _peaks()
+    for name in sizes or SIZES:
+        z = SIZES[name]
+        for kind in ("glimmer", "bulidra"):
+            prompt, context = 8192, 4096
+            eng = _engine(kind, z, 1, prompt + 64)
+            g = torch.Generator().manual_seed(1)
+            ids = torch.randint(0, z["vocab"], (prompt,), generator=g).tolist()
+            with clock_sampler(0) as clocks:
+                ms = _time(eng, lambda: eng.prefill(0, ids), max(args.steps // 2, 3), 3)
+            flops, _ = _work(z, kind, prompt, 1, 0)
+            print(json.dumps({"serving": kind, "size": name, "phase": "prefill", "prompt": prompt, "ms": round(ms, 3), "tokens_per_s": round(prompt / ms * 1e3),
+                              "fraction_of_measured_bf16": round(flops / ms * 1e3 / tf, 3), "device_bytes": eng.device_bytes, "clocks": clocks.summary()}), flush=True)
+            eng.close()
+            del eng
+            for batch in (1, 8, 32):
+                eng = _engine(kind, z, batch, context + 128)
+                last = {b: eng.prefill(b, ids[:context]) for b in range(batch)}
+
+                def step():
+                    nonlocal last
+                    last = eng.decode(last)
+
+                with clock_sampler(0) as clocks:
+                    ms = _time(eng, step, max(3 * args.steps, 30), 5)
+                _, byts = _work(z, kind, 1, batch, context)
+                print(json.dumps({"serving": kind, "size": name, "phase": "decode", "batch": batch, "context": context, "ms": round(ms, 4),
+                                  "tokens_per_s": round(batch / ms * 1e3), "fraction_of_measured_hbm": round(byts / ms * 1e3 / hbm, 3),
+                                  "clocks": clocks.summary()}), flush=True)
+                eng.close()
+                del eng

@@ -96,6 +96,7 @@ int nfn_engine_finalize(nfn_engine* e) {
 long long nfn_engine_device_bytes(const nfn_engine* e) { return e ? e->bytes : -1; }
 int nfn_engine_slot_length(const nfn_engine* e, int slot) { return (e && slot >= 0 && slot < e->slots()) ? e->len[slot] : -1; }
 long long nfn_engine_launches(const nfn_engine* e) { return e ? e->launches : -1; }
+void* nfn_engine_stream(const nfn_engine* e) { return e ? e->stream : nullptr; }
 long long nfn_engine_free_tokens(const nfn_engine* e) { return e ? e->free_tokens() : -1; }
 
 int nfn_engine_release(nfn_engine* e, int slot) {

@@ -138,6 +138,8 @@ int nfn_engine_step(nfn_engine* e, const nfn_step_entry* entries, int n_entries,
                     const nfn_sampling* want_sampling, int32_t* want_tokens, float* want_logits);
 // Tokens the page pool still has room for (whole free pages); -1 for engines without pages.
 long long nfn_engine_free_tokens(const nfn_engine* e);
+// The CUDA stream the engine launches on (for events around its calls).
+void* nfn_engine_stream(const nfn_engine* e);
 int nfn_engine_release(nfn_engine* e, int slot);
 int nfn_engine_slot_length(const nfn_engine* e, int slot);
 // Copies the bf16 logits of the last step for `slot` to the host as fp32 (vocab entries).

@@ -248,7 +248,7 @@ def _api():
         "destroy": (None, [vp]), "set_tensor": (ip, [vp, C.c_char_p, vp, ll]), "set_tensor_kquant": (ip, [vp, C.c_char_p, ip, vp, ll, ll]),
         "expected_tensors": (ip, [vp, C.c_char_p, ip]), "load_dense_v5": (ip, [vp, C.c_char_p]), "finalize": (ip, [vp]), "set_turboquant": (ip, [vp, vp]),
         "device_bytes": (ll, [vp]), "prefill": (ip, [vp, ip, vp, ip, sp, vp]), "decode": (ip, [vp, vp, vp, sp, vp, vp]), "release": (ip, [vp, ip]),
-        "step": (ip, [vp, vp, ip, vp, vp, ip, vp, vp, vp]), "free_tokens": (ll, [vp]),
+        "step": (ip, [vp, vp, ip, vp, vp, ip, vp, vp, vp]), "free_tokens": (ll, [vp]), "stream": (vp, [vp]),
         "slot_length": (ip, [vp, ip]), "last_logits": (ip, [vp, ip, vp]), "launches": (ll, [vp]), "enable_verify": (ip, [vp, ip]),
         "verify": (ip, [vp, vp, vp, ip, vp]), "verify_logits": (ip, [vp, ip, ip, vp]), "commit": (ip, [vp, vp]), "truncate": (ip, [vp, ip, ip]),
         "fork": (ip, [vp, ip, ip, ip]), "prefill_rows": (ip, [vp, ip, vp, ip, ip, sp, vp]), "enable_taps": (ip, [vp, vp, ip]),
@@ -448,6 +448,11 @@ class ResidentEngine:
         self._check(self._L.nfn_engine_decode(self._h, C.cast(tok, C.c_void_p), C.cast(act, C.c_void_p), C.byref(s),
                                               C.cast(ps, C.c_void_p) if ps is not None else None, C.cast(out, C.c_void_p)))
         return {slot: int(out[slot]) for slot in tokens_in}
+
+    @property
+    def stream(self) -> "torch.cuda.ExternalStream":
+        """The stream the engine launches on, for events around its calls."""
+        return torch.cuda.ExternalStream(self._L.nfn_engine_stream(self._h), device=self.device)
 
     # ---- steps of mixed batches (layer-list models) ----------------------------------------
     @property
