@@ -46,7 +46,7 @@ struct PagedDecodeParams {
 // DC: 32-channel chunks of a query / key head; VT: 16-channel tiles of a value head; NT: 8-head tiles (upper bounds, the actual
 // sizes are checked inside)
 template <int DC, int VT, int NT>
-__global__ void __launch_bounds__(PD_THREADS, (DC * NT <= 4 && VT <= 8) ? 3 : 2)
+__global__ void __launch_bounds__(PD_THREADS, 2)
 paged_decode_kernel(const PagedDecodeParams p) {
   constexpr int NH = NT * 8;
   extern __shared__ float pd_smem[];   // [PD_WARPS][NH][vdim_p] values, then [PD_WARPS][NH] maxima, [PD_WARPS][NH] sums
@@ -98,12 +98,34 @@ paged_decode_kernel(const PagedDecodeParams p) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[v][nt][e] = 0.f;
 
+  // row g of score tile t is key 8 (g / 2) + g % 2 + 4 t of the 32, row g + 8 the key two further
+  const int key0 = 8 * (g >> 1) + (g & 1);
+  uint4 kf[2][2][DC];                                       // key fragments of the chunk at hand: [tile][row g, row g + 8]
+  auto load_keys = [&](int c) {
+    const int base = c * PD_KEYS, in_page = base % NFN_PAGE;
+    const size_t tile = (size_t)table[base / NFN_PAGE] * a.kv_heads + hk;
+    const __nv_bfloat16* krow = kp + (tile * NFN_PAGE + in_page + key0) * DP + 8 * j;
+#pragma unroll
+    for (int t = 0; t < 2; ++t)
+#pragma unroll
+      for (int half = 0; half < 2; ++half)
+#pragma unroll
+        for (int d = 0; d < DC; ++d)
+          kf[t][half][d] = d * 32 + 8 * j < DP ? __ldg(reinterpret_cast<const uint4*>(krow + (size_t)(4 * t + 2 * half) * DP + d * 32)) : zero4;
+  };
+  if (c_lo + warp < c_hi) load_keys(c_lo + warp);
   for (int c = c_lo + warp; c < c_hi; c += PD_WARPS) {
     const int base = c * PD_KEYS, in_page = base % NFN_PAGE;
     const size_t tile = (size_t)table[base / NFN_PAGE] * a.kv_heads + hk;
-    // row g of tile s is key 8 (g / 2) + g % 2 + 4 s of the 32, row g + 8 the key two further
-    const int key0 = 8 * (g >> 1) + (g & 1);
-    const __nv_bfloat16* krow = kp + (tile * NFN_PAGE + in_page + key0) * DP + 8 * j;
+    // this chunk's values are on their way while the scores are formed, the next chunk's keys while these are used
+    constexpr int VF = (NT == 1 && VT <= 8) ? VT : 2;                    // value tiles held ahead
+    const __nv_bfloat16* vrow = vp + (tile * VP + g) * NFN_PAGE + in_page + 8 * j;
+    uint4 vf[VF][2];
+#pragma unroll
+    for (int v = 0; v < VF; ++v)
+#pragma unroll
+      for (int half = 0; half < 2; ++half)
+        vf[v][half] = v * 16 < VP ? __ldg(reinterpret_cast<const uint4*>(vrow + (size_t)(v * 16 + 8 * half) * NFN_PAGE)) : zero4;
     float s[2][NT][4];
 #pragma unroll
     for (int t = 0; t < 2; ++t)
@@ -112,24 +134,18 @@ paged_decode_kernel(const PagedDecodeParams p) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) s[t][nt][e] = 0.f;
 #pragma unroll
-    for (int t = 0; t < 2; ++t) {
-      uint4 k0[DC], k1[DC];
-#pragma unroll
-      for (int d = 0; d < DC; ++d) {
-        const bool in = d * 32 + 8 * j < DP;
-        k0[d] = in ? __ldg(reinterpret_cast<const uint4*>(krow + (size_t)(4 * t) * DP + d * 32)) : zero4;
-        k1[d] = in ? __ldg(reinterpret_cast<const uint4*>(krow + (size_t)(4 * t + 2) * DP + d * 32)) : zero4;
-      }
+    for (int t = 0; t < 2; ++t)
 #pragma unroll
       for (int d = 0; d < DC; ++d) {
         if (d * 32 >= DP) break;
+        const uint4 k0 = kf[t][0][d], k1 = kf[t][1][d];
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
-          pd_mma(s[t][nt], k0[d].x, k1[d].x, k0[d].y, k1[d].y, qf[d][nt].x, qf[d][nt].y);
-          pd_mma(s[t][nt], k0[d].z, k1[d].z, k0[d].w, k1[d].w, qf[d][nt].z, qf[d][nt].w);
+          pd_mma(s[t][nt], k0.x, k1.x, k0.y, k1.y, qf[d][nt].x, qf[d][nt].y);
+          pd_mma(s[t][nt], k0.z, k1.z, k0.w, k1.w, qf[d][nt].z, qf[d][nt].w);
         }
       }
-    }
+    if (c + PD_WARPS < c_hi) load_keys(c + PD_WARPS);
     // scaled and biased scores in units of log2, invisible keys out
     const int rel = pos - base - key0;      // distance of this lane's first key
 #pragma unroll
@@ -179,12 +195,11 @@ paged_decode_kernel(const PagedDecodeParams p) {
 #pragma unroll
         for (int half = 0; half < 2; ++half) b[t][nt][half] = pd_transpose(pack_bf16x2(s[t][nt][2 * half], s[t][nt][2 * half + 1]));
     }
-    const __nv_bfloat16* vrow = vp + (tile * VP + g) * NFN_PAGE + in_page + 8 * j;
 #pragma unroll
     for (int v = 0; v < VT; ++v) {
       if (v * 16 >= VP) break;
-      const uint4 v0 = __ldg(reinterpret_cast<const uint4*>(vrow + (size_t)(v * 16) * NFN_PAGE));
-      const uint4 v1 = __ldg(reinterpret_cast<const uint4*>(vrow + (size_t)(v * 16 + 8) * NFN_PAGE));
+      const uint4 v0 = v < VF ? vf[v < VF ? v : 0][0] : __ldg(reinterpret_cast<const uint4*>(vrow + (size_t)(v * 16) * NFN_PAGE));
+      const uint4 v1 = v < VF ? vf[v < VF ? v : 0][1] : __ldg(reinterpret_cast<const uint4*>(vrow + (size_t)(v * 16 + 8) * NFN_PAGE));
 #pragma unroll
       for (int t = 0; t < 2; ++t)
 #pragma unroll
@@ -287,8 +302,8 @@ static int launch_paged_decode(const nfn_paged_attention_args& a, cudaStream_t s
   const long long cells = (long long)a.rows * cells_y;
   p.counters = static_cast<int*>(a.workspace);
   p.partial = reinterpret_cast<float*>(static_cast<char*>(a.workspace) + PAGED_COUNTER_BYTES);
-  // enough CTAs for the GPU, at least 256 keys each
-  long long splits = std::min<long long>(ceil_div(a.max_keys, PD_KEYS * PD_WARPS * 2), (4LL * sm_count() + cells - 1) / cells);
+  // about two CTAs per SM (what is resident at a time), at least one chunk of keys per warp
+  long long splits = std::min<long long>(ceil_div(a.max_keys, PD_KEYS * PD_WARPS), std::max<long long>(1, 2LL * sm_count() / cells));
   const long long per_split = cells * NT * 8 * (a.vdim_p + 2) * 4;
   splits = std::min<long long>(splits, (a.workspace_bytes - PAGED_COUNTER_BYTES) / per_split);
   if (cells > PD_COUNTERS || splits < 1) splits = 1;

@@ -6,7 +6,8 @@
 // stores channel-major, as [channels][64 tokens]; both are K-major operands, and the page table only enters the TMA coordinates.
 // Roles as in attention_fwd2.cu: four softmax warps (one thread per accumulator row), one MMA warp, one TMA warp, two stages of
 // keys and values; S of the next page is issued as soon as this one is in registers, the output is rescaled in TMEM only when a
-// row maximum grew by more than 2^8.
+// row maximum grew by more than 2^8. Pages are visited from the newest to the oldest: under a distance bias the maximum then
+// settles in the first page instead of growing with every one.
 //
 // Head sizes are run-time values (multiples of 16 up to 256; channels past a head's end are zero-filled by TMA). The distance
 // bias and the window are applied to the fp32 scores in registers; the output gate is applied on the way out.
@@ -64,7 +65,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   const int hk = blockIdx.y;
   const int* table = a.table + (size_t)slot * a.table_ld;
   const int k_lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
-  const int jb_lo = k_lo / PP_BN, nblk = (pos0 + n_rows - 1) / PP_BN + 1 - jb_lo;
+  const int jb_hi = (pos0 + n_rows - 1) / PP_BN, nblk = jb_hi + 1 - k_lo / PP_BN;   // visited from the newest page back
 
   if (threadIdx.x == 0) {
     *cta_abort = 0;
@@ -96,14 +97,14 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       auto load_k = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_k[stage]);
         const uint32_t sk = smem_u32(sKV + stage * kv_stage);
-        const int r = (table[jb_lo + j] * a.kv_heads + hk) * PP_BN;
+        const int r = (table[jb_hi - j] * a.kv_heads + hk) * PP_BN;
         mbar_expect_tx(fb, p.k_bytes);
         for (int d = 0; d < p.panels; ++d) tma_load_2d(sk + d * (PP_BN * 128), &tm_k, fb, d * 64, r);
       };
       auto load_v = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_v[stage]);
         mbar_expect_tx(fb, p.v_bytes);
-        tma_load_2d(smem_u32(sKV + stage * kv_stage + p.k_bytes), &tm_v, fb, 0, (table[jb_lo + j] * a.kv_heads + hk) * a.vdim_p);
+        tma_load_2d(smem_u32(sKV + stage * kv_stage + p.k_bytes), &tm_v, fb, 0, (table[jb_hi - j] * a.kv_heads + hk) * a.vdim_p);
       };
       mbar_expect_tx(smem_u32(bar_q), p.q_tx);
       for (int d = 0; d < p.panels; ++d) tma_load_3d(smem_u32(sQ) + d * (PP_BM * 128), &tm_q, smem_u32(bar_q), d * 64, hk * p.hg, row0);
@@ -126,6 +127,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       auto issue_s = [&](int stage) {
         const uint32_t sq = smem_u32(sQ);
         const uint32_t sk = smem_u32(sKV + stage * kv_stage);
+#pragma unroll 4
         for (int kk = 0; kk < k_steps; ++kk) {
           const uint32_t a_off = (kk / 4) * (PP_BM * 128) + (kk % 4) * 32;
           const uint32_t b_off = (kk / 4) * (PP_BN * 128) + (kk % 4) * 32;
@@ -188,7 +190,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(bar_sfree));
 
-      const int kbase = (jb_lo + j) * PP_BN;
+      const int kbase = (jb_hi - j) * PP_BN;
       const float b0 = slope * (float)(kbase - pos);
 #pragma unroll
       for (int i = 0; i < PP_BN; i += 2) {
@@ -270,7 +272,16 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(bar_p));
     }
-    // ---- O / l, output gate -> global ----
+    // ---- O / l, output gate -> global: 64 channels at a time, their gates on the way before O is waited for ----
+    __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(a.out) + (size_t)(row0 + qi) * a.ld_o + (size_t)h * a.vdim_p;
+    const __nv_bfloat16* grow_ = (a.gate && row_ok) ? static_cast<const __nv_bfloat16*>(a.gate) + (size_t)(row0 + qi) * a.ld_gate + (size_t)h * a.vdim_p : nullptr;
+    uint4 gv[8];
+    auto fetch_gate = [&](int c0) {
+#pragma unroll
+      for (int g = 0; g < 8; ++g)
+        if (grow_ && c0 + g * 8 < a.vdim_p) gv[g] = __ldg(reinterpret_cast<const uint4*>(grow_ + c0 + g * 8));
+    };
+    fetch_gate(0);
     if (ok) {
       ok = mbar_wait_bounded(smem_u32(bar_o), (nblk - 1) & 1, cta_abort, p.status, 0x600 + 11);
       ok = __all_sync(0xffffffffu, ok);
@@ -278,26 +289,28 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     if (ok) {
       tc_fence_after();
       const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
-      __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(a.out) + (size_t)(row0 + qi) * a.ld_o + (size_t)h * a.vdim_p;
-      const __nv_bfloat16* grow_ = a.gate ? static_cast<const __nv_bfloat16*>(a.gate) + (size_t)(row0 + qi) * a.ld_gate + (size_t)h * a.vdim_p : nullptr;
 #pragma unroll 1
-      for (int c = 0; c < a.vdim_p / 16; ++c) {
-        uint32_t o[16];
-        tmem_ld_32x16(t_row + p.o_col + c * 16, o);  // warp-collective: every lane issues it
+      for (int c0 = 0; c0 < a.vdim_p; c0 += 64) {
+        if (c0 > 0) fetch_gate(c0);
+        uint32_t o[64];
+#pragma unroll
+        for (int c = 0; c < 4; ++c)                                     // warp-collective: every lane issues them
+          if (c0 + c * 16 < a.vdim_p) tmem_ld_32x16(t_row + p.o_col + c0 + c * 16, *reinterpret_cast<uint32_t(*)[16]>(&o[c * 16]));
         tmem_ld_wait();
         if (row_ok) {
 #pragma unroll
-          for (int g = 0; g < 2; ++g) {
+          for (int g = 0; g < 8; ++g) {
+            if (c0 + g * 8 >= a.vdim_p) break;
             float v[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(o[g * 8 + i]) * inv;
             if (grow_) {
-              float gv[8];
-              load8(grow_ + c * 16 + g * 8, gv);
+              const float2 g0 = unpack_bf16x2(gv[g].x), g1 = unpack_bf16x2(gv[g].y), g2 = unpack_bf16x2(gv[g].z), g3 = unpack_bf16x2(gv[g].w);
+              const float gf[8] = {g0.x, g0.y, g1.x, g1.y, g2.x, g2.y, g3.x, g3.y};
 #pragma unroll
-              for (int i = 0; i < 8; ++i) v[i] *= 1.f / (1.f + __expf(-gv[i]));
+              for (int i = 0; i < 8; ++i) v[i] *= 1.f / (1.f + __expf(-gf[i]));
             }
-            store8(orow + c * 16 + g * 8, v);
+            store8(orow + c0 + g * 8, v);
           }
         }
       }

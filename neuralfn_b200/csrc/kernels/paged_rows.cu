@@ -36,17 +36,6 @@ row_norm_kernel(const nfn_row_norm_args p) {
   const int r = blockIdx.x;
   const int vecs = p.ld / 4;
   const float inv_w = 1.f / (float)p.width;
-  float ry = 0.f;
-  if (p.y) {
-    float ss = 0.f;
-    const T* y = static_cast<const T*>(p.y) + (size_t)r * p.ld;
-    for (int v = threadIdx.x; v < vecs; v += ROW_THREADS) {
-      const float4 f = load4(y + 4 * v);
-      reinterpret_cast<float4*>(yrow)[v] = f;
-      ss += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;
-    }
-    ry = 1.f / sqrtf(block_sum(ss, red) * inv_w + p.eps);
-  }
   const __nv_bfloat16* emb = nullptr;
   const float* x = nullptr;
   if (p.tokens) {
@@ -55,6 +44,18 @@ row_norm_kernel(const nfn_row_norm_args p) {
   } else {
     x = p.x + (size_t)(p.src_rows ? p.src_rows[r] : r) * p.ld;
   }
+  float ry = 0.f;
+  if (p.y) {
+    float ss = 0.f;
+    const T* y = static_cast<const T*>(p.y) + (size_t)r * p.ld;
+    for (int v = threadIdx.x; v < vecs; v += ROW_THREADS) {
+      const float4 f = load4(y + 4 * v);
+      if (x) reinterpret_cast<float4*>(base)[v] = load4(x + 4 * v);      // both rows are on their way together
+      reinterpret_cast<float4*>(yrow)[v] = f;
+      ss += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;
+    }
+    ry = 1.f / sqrtf(block_sum(ss, red) * inv_w + p.eps);
+  }
   float ss = 0.f;
   for (int v = threadIdx.x; v < vecs; v += ROW_THREADS) {
     float4 b;
@@ -62,7 +63,7 @@ row_norm_kernel(const nfn_row_norm_args p) {
       b = load4(emb + 4 * v);
       b.x *= p.embed_scale; b.y *= p.embed_scale; b.z *= p.embed_scale; b.w *= p.embed_scale;
     } else {
-      b = load4(x + 4 * v);
+      b = p.y ? reinterpret_cast<const float4*>(base)[v] : load4(x + 4 * v);
     }
     if (p.y) {
       const float4 f = reinterpret_cast<const float4*>(yrow)[v];
@@ -84,7 +85,7 @@ row_norm_kernel(const nfn_row_norm_args p) {
 }
 
 // ----------------------------------------------------------------------------- after the input projection --
-constexpr int MIX_THREADS = 128, MIX_ROWS = 16;
+constexpr int MIX_THREADS = 128, MIX_ROWS = 16, MIX_FF_ROWS = 4;   // MIX_FF_ROWS: rows in flight per thread
 
 // Projected value row `back` positions before row index ti of the entry: this step's rows, the stored history, or zero before
 // the sequence's start.
@@ -100,68 +101,136 @@ __device__ __forceinline__ bool mix_source(const nfn_mix_args& p, const nfn_row_
   return true;
 }
 
-template <typename T>
-__global__ void __launch_bounds__(MIX_THREADS)
+// Convolved values of up to N consecutive rows of a tile, starting at row index ti of the entry. TAPS > 0: the window slides through
+// registers, so every projected row is read once; TAPS = 0: any number of taps, rows are read again (they stay in L1).
+template <typename T, int TAPS, int N>
+struct MixWindow {
+  float hist[TAPS > 1 ? TAPS - 1 : 1][8], w[TAPS > 0 ? TAPS : 1][8];
+  __device__ __forceinline__ void start(const nfn_mix_args& p, const nfn_row_tile& t, int ti, int col) {
+    if (TAPS > 0) {
+      const int C = p.nq + p.nk + p.nv;
+#pragma unroll
+      for (int j = 0; j < TAPS; ++j) load8(static_cast<const __nv_bfloat16*>(p.conv) + (size_t)j * C + col, w[j]);
+#pragma unroll
+      for (int j = 0; j < TAPS - 1; ++j)
+        if (!mix_source<T>(p, t, ti - (TAPS - 1) + j, col, hist[j]))
+#pragma unroll
+          for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
+    }
+  }
+  // rows [ti, ti + n), n <= N; rows past n are left undefined
+  __device__ __forceinline__ void next(const nfn_mix_args& p, const nfn_row_tile& t, int ti, int n, int col, float (&out)[N][8]) {
+    if (TAPS == 0 && p.conv) {
+      const int C = p.nq + p.nk + p.nv;
+#pragma unroll
+      for (int i = 0; i < N; ++i) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) out[i][e] = 0.f;
+        if (i < n)
+          for (int j = 0; j < p.taps; ++j) {
+            float u[8], wj[8];
+            if (!mix_source<T>(p, t, ti + i - (p.taps - 1) + j, col, u)) continue;
+            load8(static_cast<const __nv_bfloat16*>(p.conv) + (size_t)j * C + col, wj);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) out[i][e] += wj[e] * u[e];
+          }
+      }
+      return;
+    }
+    const T* in = static_cast<const T*>(p.in) + (size_t)(t.e_row0 + ti) * p.ld_in + col;
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (i < n) load8(in + (size_t)i * p.ld_in, out[i]);
+    if (TAPS == 0) return;
+#pragma unroll
+    for (int i = 0; i < N; ++i)
+      if (i < n) {
+#pragma unroll
+        for (int e = 0; e < 8; ++e) {
+          const float u = out[i][e];
+          float acc = w[TAPS - 1][e] * u;
+#pragma unroll
+          for (int j = 0; j < TAPS - 1; ++j) acc += w[j][e] * hist[j][e];
+#pragma unroll
+          for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][e] = hist[j + 1][e];
+          if (TAPS > 1) hist[TAPS > 1 ? TAPS - 2 : 0][e] = u;
+          out[i][e] = acc;
+        }
+      }
+  }
+};
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(MIX_THREADS, 4)
 mix_rows_kernel(const nfn_mix_args p) {
+  constexpr int N = MIX_FF_ROWS;
   const nfn_row_tile t = p.tiles[blockIdx.y];
   if (t.slot < 0) return;
   const int C = p.nq + p.nk + p.nv;
   const int vec = blockIdx.x * MIX_THREADS + threadIdx.x;
   const int ti0 = t.row0 - t.e_row0;                       // first row's index inside the entry
   if (vec * 8 >= C) {
-    // feed-forward columns: ff_out = act(gate) * up
-    const int c = vec * 8 - C;
-    if (c >= p.ff) return;
+    // feed-forward columns: ff_out = act(gate) * up, N rows per thread
+    const int fv = vec - C / 8, c = fv % (p.ff / 8) * 8, i_lo = fv / (p.ff / 8) * N;
+    if (i_lo >= t.n) return;
     const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
     T* out = static_cast<T*>(p.ff_out) + (size_t)t.row0 * p.ld_ff + c;
-    for (int i = 0; i < t.n; ++i) {
-      float g[8], u[8];
-      load8(in + (size_t)i * p.ld_in + p.off_gate + c, g);
-      load8(in + (size_t)i * p.ld_in + p.off_up + c, u);
+    {
+      const int i0 = i_lo;
+      float g[N][8], u[N][8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) g[e] = ff_act(g[e], p.act) * u[e];
-      store8(out + (size_t)i * p.ld_ff, g);
+      for (int i = 0; i < N; ++i)
+        if (i0 + i < t.n) {
+          load8(in + (size_t)(i0 + i) * p.ld_in + p.off_gate + c, g[i]);
+          load8(in + (size_t)(i0 + i) * p.ld_in + p.off_up + c, u[i]);
+        }
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+        if (i0 + i < t.n) {
+#pragma unroll
+          for (int e = 0; e < 8; ++e) g[i][e] = ff_act(g[i][e], p.act) * u[i][e];
+          store8(out + (size_t)(i0 + i) * p.ld_ff, g[i]);
+        }
     }
     return;
   }
   const int col = vec * 8, taps = p.taps;
-  // the history the entry leaves behind: its newest taps - 1 projected rows (older ones move up when it brought fewer)
-  if (taps > 1 && t.row0 + t.n == t.e_row0 + t.e_n) {
-    T* st = static_cast<T*>(p.state) + (size_t)(1 - t.parity) * p.state_half + (size_t)t.slot * (taps - 1) * C + col;
+  // the history the entry leaves behind: its newest taps - 1 projected rows (older ones move up when it brought fewer). The
+  // register window holds exactly these rows after the tile's last row; otherwise they are gathered.
+  const bool last = taps > 1 && t.row0 + t.n == t.e_row0 + t.e_n;
+  T* st = static_cast<T*>(p.state) + (size_t)(1 - t.parity) * p.state_half + (size_t)t.slot * (taps - 1) * C + col;
+  if (TAPS == 0 && last) {
     for (int i = 0; i < taps - 1; ++i) {
       float v[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
       mix_source<T>(p, t, t.e_n - (taps - 1) + i, col, v);
       store8(st + (size_t)i * C, v);
     }
   }
-  auto convolve = [&](int ti, float (&acc)[8]) {
-    if (!p.conv) {
-      load8(static_cast<const T*>(p.in) + (size_t)(t.e_row0 + ti) * p.ld_in + col, acc);
-      return;
-    }
+  MixWindow<T, TAPS, N> win;
+  win.start(p, t, ti0, col);
+  auto leave = [&]() {
+    if (TAPS > 1 && last)
 #pragma unroll
-    for (int e = 0; e < 8; ++e) acc[e] = 0.f;
-    for (int j = 0; j < taps; ++j) {
-      float u[8], w[8];
-      if (!mix_source<T>(p, t, ti - (taps - 1) + j, col, u)) continue;
-      load8(static_cast<const __nv_bfloat16*>(p.conv) + (size_t)j * C + col, w);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) acc[e] += w[e] * u[e];
-    }
+      for (int i = 0; i < TAPS - 1; ++i) store8(st + (size_t)i * C, win.hist[i]);
   };
+  float v[N][8];
   if (col < p.nq) {
     T* out = static_cast<T*>(p.q_out) + (size_t)t.row0 * p.ld_q + col;
-    for (int i = 0; i < t.n; ++i) {
-      float acc[8];
-      convolve(ti0 + i, acc);
-      if (p.temp_every > 0) {
-        const int pos = t.e_pos0 + ti0 + i;
-        const float f = 1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every + 1));
+    for (int i0 = 0; i0 < t.n; i0 += N) {
+      win.next(p, t, ti0 + i0, t.n - i0, col, v);
 #pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] *= f;
-      }
-      store8(out + (size_t)i * p.ld_q, acc);
+      for (int i = 0; i < N; ++i)
+        if (i0 + i < t.n) {
+          if (p.temp_every > 0) {
+            const int pos = t.e_pos0 + ti0 + i0 + i;
+            const float f = 1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every + 1));
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[i][e] *= f;
+          }
+          store8(out + (size_t)(i0 + i) * p.ld_q, v[i]);
+        }
     }
+    leave();
     return;
   }
   // keys and values: the tile lies inside one page
@@ -171,37 +240,57 @@ mix_rows_kernel(const nfn_mix_args p) {
   if (col < p.nq + p.nk) {
     const int c = col - p.nq, head = c / p.dim_p, d = c % p.dim_p;
     T* out = static_cast<T*>(p.k_pool) + ((page * p.kv_heads + head) * NFN_PAGE + in_page) * p.dim_p + d;
-    for (int i = 0; i < t.n; ++i) {
-      float acc[8];
-      convolve(ti0 + i, acc);
-      store8(out + (size_t)i * p.dim_p, acc);
+    for (int i0 = 0; i0 < t.n; i0 += N) {
+      win.next(p, t, ti0 + i0, t.n - i0, col, v);
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+        if (i0 + i < t.n) store8(out + (size_t)(i0 + i) * p.dim_p, v[i]);
     }
+    leave();
     return;
   }
   const int c = col - p.nq - p.nk, head = c / p.vdim_p, d = c % p.vdim_p;
   T* out = static_cast<T*>(p.v_pool) + ((page * p.kv_heads + head) * p.vdim_p + d) * NFN_PAGE + in_page;   // [vdim_p][64]
   if (t.n == MIX_ROWS) {
-    // whole tile: 16 consecutive tokens of every channel go out as full sectors
-    T buf[8][MIX_ROWS];
+    // whole tile: eight consecutive tokens of every channel at a time, in 16-byte stores
+#pragma unroll 1
+    for (int i0 = 0; i0 < MIX_ROWS; i0 += 8) {
+      T buf[8][8];
 #pragma unroll
-    for (int i = 0; i < MIX_ROWS; ++i) {
-      float acc[8];
-      convolve(ti0 + i, acc);
+      for (int q = 0; q < 2; ++q) {
+        win.next(p, t, ti0 + i0 + q * N, N, col, v);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) buf[e][i] = from_float<T>(acc[e]);
+        for (int i = 0; i < N; ++i)
+#pragma unroll
+          for (int e = 0; e < 8; ++e) buf[e][q * N + i] = from_float<T>(v[i][e]);
+      }
+#pragma unroll
+      for (int e = 0; e < 8; ++e)
+#pragma unroll
+        for (int q = 0; q < (int)(sizeof(T) / 2); ++q)
+          reinterpret_cast<uint4*>(out + (size_t)e * NFN_PAGE + i0)[q] = pack16(&buf[e][q * (16 / sizeof(T))]);
     }
-#pragma unroll
-    for (int e = 0; e < 8; ++e)
-#pragma unroll
-      for (int q = 0; q < (int)(MIX_ROWS * sizeof(T) / 16); ++q)
-        reinterpret_cast<uint4*>(out + (size_t)e * NFN_PAGE)[q] = pack16(&buf[e][q * (16 / sizeof(T))]);
+    leave();
     return;
   }
-  for (int i = 0; i < t.n; ++i) {
-    float acc[8];
-    convolve(ti0 + i, acc);
+  for (int i0 = 0; i0 < t.n; i0 += N) {
+    win.next(p, t, ti0 + i0, t.n - i0, col, v);
 #pragma unroll
-    for (int e = 0; e < 8; ++e) out[(size_t)e * NFN_PAGE + i] = from_float<T>(acc[e]);
+    for (int i = 0; i < N; ++i)
+      if (i0 + i < t.n)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) out[(size_t)e * NFN_PAGE + i0 + i] = from_float<T>(v[i][e]);
+  }
+  leave();
+}
+
+template <typename T>
+static void launch_mix_rows(const nfn_mix_args& a, const dim3& grid, cudaStream_t st) {
+  switch (a.taps) {
+    case 2: mix_rows_kernel<T, 2><<<grid, MIX_THREADS, 0, st>>>(a); break;
+    case 3: mix_rows_kernel<T, 3><<<grid, MIX_THREADS, 0, st>>>(a); break;
+    case 4: mix_rows_kernel<T, 4><<<grid, MIX_THREADS, 0, st>>>(a); break;
+    default: mix_rows_kernel<T, 0><<<grid, MIX_THREADS, 0, st>>>(a); break;
   }
 }
 
@@ -395,11 +484,12 @@ extern "C" int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream) {
     return fail(-1, "mix_rows: widths and offsets must be multiples of 8");
   if ((a.taps > 0) != (a.conv != nullptr) || (a.taps > 1 && !a.state)) return fail(-1, "mix_rows: a convolution needs its weights and history");
   if (a.n_tiles > 65535) return fail(-1, "mix_rows: too many row tiles in one launch");
-  const int vecs = (a.nq + a.nk + a.nv + a.ff) / 8;
+  if (a.tile_rows < 1 || a.tile_rows > MIX_ROWS) return fail(-1, "mix_rows: tiles hold 1 to 16 rows");
+  const int vecs = (a.nq + a.nk + a.nv + a.ff * ceil_div(a.tile_rows, MIX_FF_ROWS)) / 8;
   const dim3 grid(ceil_div(vecs, MIX_THREADS), a.n_tiles);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (a.f32) mix_rows_kernel<float><<<grid, MIX_THREADS, 0, st>>>(a);
-  else mix_rows_kernel<__nv_bfloat16><<<grid, MIX_THREADS, 0, st>>>(a);
+  if (a.f32) launch_mix_rows<float>(a, grid, st);
+  else launch_mix_rows<__nv_bfloat16>(a, grid, st);
   return launch_check("mix_rows");
 }
 
