@@ -107,15 +107,14 @@ template <typename T, int TAPS, int N>
 struct MixWindow {
   float hist[TAPS > 1 ? TAPS - 1 : 1][8], w[TAPS > 0 ? TAPS : 1][8];
   __device__ __forceinline__ void start(const nfn_mix_args& p, const nfn_row_tile& t, int ti, int col) {
-    if (TAPS > 0) {
+    if constexpr (TAPS > 0) {
       const int C = p.nq + p.nk + p.nv;
 #pragma unroll
       for (int j = 0; j < TAPS; ++j) load8(static_cast<const __nv_bfloat16*>(p.conv) + (size_t)j * C + col, w[j]);
 #pragma unroll
       for (int j = 0; j < TAPS - 1; ++j)
         if (!mix_source<T>(p, t, ti - (TAPS - 1) + j, col, hist[j]))
-#pragma unroll
-          for (int e = 0; e < 8; ++e) hist[j][e] = 0.f;
+          for (float& f : hist[j]) f = 0.f;
     }
   }
   // rows [ti, ti + n), n <= N; rows past n are left undefined
@@ -141,22 +140,23 @@ struct MixWindow {
 #pragma unroll
     for (int i = 0; i < N; ++i)
       if (i < n) load8(in + (size_t)i * p.ld_in, out[i]);
-    if (TAPS == 0) return;
+    if constexpr (TAPS > 0) {
 #pragma unroll
-    for (int i = 0; i < N; ++i)
-      if (i < n) {
+      for (int i = 0; i < N; ++i)
+        if (i < n) {
 #pragma unroll
-        for (int e = 0; e < 8; ++e) {
-          const float u = out[i][e];
-          float acc = w[TAPS - 1][e] * u;
+          for (int e = 0; e < 8; ++e) {
+            const float u = out[i][e];
+            float acc = w[TAPS - 1][e] * u;
 #pragma unroll
-          for (int j = 0; j < TAPS - 1; ++j) acc += w[j][e] * hist[j][e];
+            for (int j = 0; j < TAPS - 1; ++j) acc += w[j][e] * hist[j][e];
 #pragma unroll
-          for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][e] = hist[j + 1][e];
-          if (TAPS > 1) hist[TAPS > 1 ? TAPS - 2 : 0][e] = u;
-          out[i][e] = acc;
+            for (int j = 0; j + 1 < TAPS - 1; ++j) hist[j][e] = hist[j + 1][e];
+            if constexpr (TAPS > 1) hist[TAPS - 2][e] = u;
+            out[i][e] = acc;
+          }
         }
-      }
+    }
   }
 };
 
@@ -171,6 +171,7 @@ mix_rows_kernel(const nfn_mix_args p) {
   const int ti0 = t.row0 - t.e_row0;                       // first row's index inside the entry
   if (vec * 8 >= C) {
     // feed-forward columns: ff_out = act(gate) * up, N rows per thread
+    if (p.ff == 0) return;                                 // the grid is rounded up
     const int fv = vec - C / 8, c = fv % (p.ff / 8) * 8, i_lo = fv / (p.ff / 8) * N;
     if (i_lo >= t.n) return;
     const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
@@ -209,9 +210,12 @@ mix_rows_kernel(const nfn_mix_args p) {
   MixWindow<T, TAPS, N> win;
   win.start(p, t, ti0, col);
   auto leave = [&]() {
-    if (TAPS > 1 && last)
+    if constexpr (TAPS > 1) {
+      if (last) {
 #pragma unroll
-      for (int i = 0; i < TAPS - 1; ++i) store8(st + (size_t)i * C, win.hist[i]);
+        for (int i = 0; i < TAPS - 1; ++i) store8(st + (size_t)i * C, win.hist[i]);
+      }
+    }
   };
   float v[N][8];
   if (col < p.nq) {
