@@ -447,7 +447,7 @@ int layered_engine::pass(int rows, int short_rows, int n_mix, const std::vector<
     m.table = groups[L.group].d_table; m.table_ld = max_pages;
     m.temp_coef = d.q_temp_coef; m.temp_every = d.q_temp_every;
     m.ff_out = ff_out; m.ld_ff = L.n_cat;
-    m.tiles = dev<nfn_row_tile>(io.mix); m.n_tiles = n_mix; m.tile_rows = n_mix == rows ? 1 : kMixRows;
+    m.tiles = dev<nfn_row_tile>(io.mix); m.n_tiles = n_mix; m.tile_rows = n_mix == rows ? 1 : kMixRows; m.rows = rows;
     K(nfn_mix_rows(&m, stream));
 
     nfn_paged_attention_args a{};

@@ -337,6 +337,7 @@ typedef struct {
   void* ff_out; int ld_ff;
   const nfn_row_tile* tiles; int n_tiles;
   int tile_rows;                          // most rows of a tile of this call
+  int rows;                               // rows of the call
 } nfn_mix_args;
 int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream);
 // Attention of a step's rows over the pages. score = q . k * scale - slopes[h] * (i - j), keys 0 <= i - j < window (0: all),

@@ -85,7 +85,7 @@ row_norm_kernel(const nfn_row_norm_args p) {
 }
 
 // ----------------------------------------------------------------------------- after the input projection --
-constexpr int MIX_THREADS = 128, MIX_ROWS = 16, MIX_FF_ROWS = 4;   // MIX_FF_ROWS: rows in flight per thread
+constexpr int MIX_THREADS = 128, MIX_ROWS = 16;
 
 // Projected value row `back` positions before row index ti of the entry: this step's rows, the stored history, or zero before
 // the sequence's start.
@@ -163,36 +163,24 @@ struct MixWindow {
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(MIX_THREADS, 4)
 mix_rows_kernel(const nfn_mix_args p) {
-  constexpr int N = MIX_FF_ROWS;
+  constexpr int N = 4;                                     // rows in flight per thread
   const nfn_row_tile t = p.tiles[blockIdx.y];
   if (t.slot < 0) return;
   const int C = p.nq + p.nk + p.nv;
   const int vec = blockIdx.x * MIX_THREADS + threadIdx.x;
   const int ti0 = t.row0 - t.e_row0;                       // first row's index inside the entry
   if (vec * 8 >= C) {
-    // feed-forward columns: ff_out = act(gate) * up, N rows per thread
-    if (p.ff == 0) return;                                 // the grid is rounded up
-    const int fv = vec - C / 8, c = fv % (p.ff / 8) * 8, i_lo = fv / (p.ff / 8) * N;
-    if (i_lo >= t.n) return;
+    // feed-forward columns of single-row tiles: ff_out = act(gate) * up (larger calls: ff_rows_kernel)
+    const int c = vec * 8 - C;
+    if (p.tile_rows != 1 || c >= p.ff) return;
     const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
     T* out = static_cast<T*>(p.ff_out) + (size_t)t.row0 * p.ld_ff + c;
-    {
-      const int i0 = i_lo;
-      float g[N][8], u[N][8];
+    float g[8], u[8];
+    load8(in + p.off_gate + c, g);
+    load8(in + p.off_up + c, u);
 #pragma unroll
-      for (int i = 0; i < N; ++i)
-        if (i0 + i < t.n) {
-          load8(in + (size_t)(i0 + i) * p.ld_in + p.off_gate + c, g[i]);
-          load8(in + (size_t)(i0 + i) * p.ld_in + p.off_up + c, u[i]);
-        }
-#pragma unroll
-      for (int i = 0; i < N; ++i)
-        if (i0 + i < t.n) {
-#pragma unroll
-          for (int e = 0; e < 8; ++e) g[i][e] = ff_act(g[i][e], p.act) * u[i][e];
-          store8(out + (size_t)(i0 + i) * p.ld_ff, g[i]);
-        }
-    }
+    for (int e = 0; e < 8; ++e) g[e] = ff_act(g[e], p.act) * u[e];
+    store8(out, g);
     return;
   }
   const int col = vec * 8, taps = p.taps;
@@ -286,6 +274,31 @@ mix_rows_kernel(const nfn_mix_args p) {
         for (int e = 0; e < 8; ++e) out[(size_t)e * NFN_PAGE + i0 + i] = from_float<T>(v[i][e]);
   }
   leave();
+}
+
+// ff_out = act(gate) * up over all rows of a call: two rows per thread, few registers
+template <typename T>
+__global__ void __launch_bounds__(256)
+ff_rows_kernel(const nfn_mix_args p) {
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 8, r0 = blockIdx.y * 2;
+  if (c >= p.ff) return;
+  const T* in = static_cast<const T*>(p.in) + (size_t)r0 * p.ld_in + c;
+  T* out = static_cast<T*>(p.ff_out) + (size_t)r0 * p.ld_ff + c;
+  const bool two = r0 + 1 < p.rows;
+  float g[2][8], u[2][8];
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+    if (i == 0 || two) {
+      load8(in + (size_t)i * p.ld_in + p.off_gate, g[i]);
+      load8(in + (size_t)i * p.ld_in + p.off_up, u[i]);
+    }
+#pragma unroll
+  for (int i = 0; i < 2; ++i)
+    if (i == 0 || two) {
+#pragma unroll
+      for (int e = 0; e < 8; ++e) g[i][e] = ff_act(g[i][e], p.act) * u[i][e];
+      store8(out + (size_t)i * p.ld_ff, g[i]);
+    }
 }
 
 template <typename T>
@@ -489,12 +502,19 @@ extern "C" int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream) {
   if ((a.taps > 0) != (a.conv != nullptr) || (a.taps > 1 && !a.state)) return fail(-1, "mix_rows: a convolution needs its weights and history");
   if (a.n_tiles > 65535) return fail(-1, "mix_rows: too many row tiles in one launch");
   if (a.tile_rows < 1 || a.tile_rows > MIX_ROWS) return fail(-1, "mix_rows: tiles hold 1 to 16 rows");
-  const int vecs = (a.nq + a.nk + a.nv + a.ff * ceil_div(a.tile_rows, MIX_FF_ROWS)) / 8;
+  const bool split = a.ff > 0 && a.tile_rows > 1;
+  if (split && (a.rows < 1 || ceil_div(a.rows, 2) > 65535)) return fail(-1, "mix_rows: too many rows in one launch");
+  const int vecs = (a.nq + a.nk + a.nv + (a.tile_rows == 1 ? a.ff : 0)) / 8;
   const dim3 grid(ceil_div(vecs, MIX_THREADS), a.n_tiles);
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (a.f32) launch_mix_rows<float>(a, grid, st);
   else launch_mix_rows<__nv_bfloat16>(a, grid, st);
-  return launch_check("mix_rows");
+  if (split) {
+    const dim3 ffg(ceil_div(a.ff, 256 * 8), ceil_div(a.rows, 2));
+    if (a.f32) ff_rows_kernel<float><<<ffg, 256, 0, st>>>(a);
+    else ff_rows_kernel<__nv_bfloat16><<<ffg, 256, 0, st>>>(a);
+  }
+  return launch_check("mix_rows", split ? 2 : 1);
 }
 
 extern "C" int nfn_side_mul(int f32, const float* gate, const int* tokens, const void* side_embed, long long ld_embed, int col0, int vocab,
