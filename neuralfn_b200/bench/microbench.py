@@ -306,7 +306,59 @@ def case_engine_decode(args):
                           "kernel_launches_per_step": eng.launches // (steps + 8 + B) if hasattr(eng, "launches") else None})
 
 
-CASES = {"gemm": case_gemm, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
+def case_paged(args):
+    """Kernels of the layer-list engine beside their closest counterparts, at one layer of ``--heads`` / ``--kv-heads`` x ``--head-dim`` with
+    ``--window``: prompt attention over pages (``--seq`` rows) against flash attention, decode attention (``--batch`` rows) against the ring
+    cache kernel, the row mix against SwiGLU, the residual row pass against RMS norm + residual."""
+    from neuralfn_b200.ops import infer as I, kernels as K, paged as P
+    dev = torch.device("cuda")
+    H, G, D, T, B, W = args.heads, args.kv_heads or args.heads, args.head_dim, args.seq, args.batch, args.window
+    slopes = torch.tensor([2.0 ** (-8 * (h + 1) / H) for h in range(H)], device=dev)
+    kw = dict(heads=H, window=W, scale=D ** -0.5, slopes=slopes)
+    rand = lambda *s: torch.randn(*s, device=dev).bfloat16()  # noqa: E731
+    extra = {"H": H, "G": G, "D": D, "window": W}
+    t = lambda fn: time_kernel(fn, args.iters, args.warmup, args.flush)  # noqa: E731
+    w = min(W or T, T)
+    flops = 4.0 * H * D * (w * (w + 1) / 2 + (T - w) * w)
+    c = P.PagedCache(1, T, G, D, D, dev)
+    c.k.normal_(), c.v.normal_()
+    q, gate, out = rand(T, H * D), rand(T, H * D), torch.empty(T, H * D, device=dev, dtype=torch.bfloat16)
+    step = P.tile_rows(c, H)
+    tiles = torch.tensor([[r, min(step, T - r), 0, r] for r in range(0, T, step)], dtype=torch.int32, device=dev)
+    _report("paged_attention_tiles", t(lambda: P.attention_tiles(c, q, tiles, out, gate=gate, **kw)), flops=flops, args=args, extra={**extra, "T": T})
+    k, v = rand(T, G * D), rand(T, G * D)
+    fa = dict(B=1, T=T, n_q_heads=H, n_kv_heads=G, head_dim=D, causal=True, window=W)
+    o, lse = K.attention_forward(q, k, v, **fa)
+    _report("attention_fwd", t(lambda: K.attention_forward(q, k, v, out=o, lse=lse, **fa)), flops=flops, args=args, extra={**extra, "T": T})
+    F = args.n
+    x = rand(T, 2 * H * D + 2 * G * D + 2 * F)
+    ch = H * D + 2 * G * D
+    conv, state = rand(4, ch), torch.zeros(2, 1, 3, ch, device=dev, dtype=torch.bfloat16)
+    cat, rt = torch.empty(T, H * D + F, device=dev, dtype=torch.bfloat16), P.row_tiles([(0, 0, T, 0)], dev)
+    _report("mix_rows", t(lambda: P.mix_rows(c, x, rt, q, cat[:, H * D:], heads=H, off_gate=ch + H * D, off_up=ch + H * D + F, ff=F, conv=conv, state=state, temp=(0.1, 1024))),
+            bytes_=4.0 * T * ch + 6.0 * T * F, args=args, extra={**extra, "T": T, "ff": F, "taps": 4})
+    gu = rand(T, 2 * F)
+    ffo = torch.empty(T, F, device=dev, dtype=torch.bfloat16)
+    _report("swiglu", t(lambda: I.swiglu_forward(gu, F, out=ffo)), bytes_=6.0 * T * F, args=args, extra={"T": T, "ff": F})
+    C = args.k
+    xs, y, h, wt = torch.randn(T, C, device=dev), rand(T, C), torch.empty(T, C, device=dev, dtype=torch.bfloat16), rand(C)
+    _report("row_norm (fp32 residual)", t(lambda: P.row_norm(xs, wt, h, eps=1e-5, y=y, y_weight=wt, x_out=xs)), bytes_=12.0 * T * C, args=args, extra={"T": T, "width": C})
+    del c, q, gate, out, k, v, x, gu
+    ctx = args.context
+    c = P.PagedCache(B, ctx, G, D, D, dev)
+    c.k.normal_(), c.v.normal_()
+    q1, g1, o1 = rand(B, H * D), rand(B, H * D), torch.empty(B, H * D, device=dev, dtype=torch.bfloat16)
+    slot, pos = torch.arange(B, dtype=torch.int32, device=dev), torch.full((B,), ctx - 1, dtype=torch.int32, device=dev)
+    seen = min(W or ctx, ctx)
+    _report("paged_attention_rows", t(lambda: P.attention_rows(c, q1, slot, pos, o1, gate=g1, **kw)), bytes_=4.0 * B * G * seen * D, args=args,
+            extra={**extra, "B": B, "context": ctx})
+    kc, vc, ws = rand(B, G, seen, D), rand(B, G, seen, D), I.DecodeAttentionWorkspace(B, H, G, D, dev)
+    qkv, lens, (cos, sin) = rand(B, (H + 2 * G) * D), torch.full((B,), seen, dtype=torch.int32, device=dev), I.rope_tables(seen, D, device=dev)
+    _report("decode_attention", t(lambda: I.decode_attention(qkv, kc, vc, lens, n_q_heads=H, n_kv_heads=G, head_dim=D, workspace=ws, cos=cos, sin=sin, qk_norm=True, out=o1)),
+            bytes_=4.0 * B * G * seen * D, args=args, extra={**extra, "B": B, "context": ctx})
+
+
+CASES = {"gemm": case_gemm, "paged": case_paged, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
          "cross_entropy": case_cross_entropy, "norm": case_norm, "adamw": case_adamw, "decode_attention": case_decode_attention,
          "skinny": case_skinny, "grouped_k": case_grouped_k, "kquant_gemv": case_kquant_gemv, "gemm_kquant": case_gemm_kquant, "block_attention": case_block_attention,
          "turboquant_attention": case_turboquant_attention, "engine_decode": case_engine_decode}
@@ -342,6 +394,8 @@ def main(argv=None):
     ap.add_argument("--head-dim", type=int, default=64)
     ap.add_argument("--vocab", type=int, default=50257)
     ap.add_argument("--params", type=int, default=124 * 1000 * 1000)
+    ap.add_argument("--window", type=int, default=0, help="paged case: sliding window")
+    ap.add_argument("--context", type=int, default=4096, help="paged case: cached tokens per decode row")
     ap.add_argument("--iters", type=int, default=20)
     ap.add_argument("--experts", type=int, default=16, help="grouped_k case")
     ap.add_argument("--no-baseline", action="store_true", help="grouped_k case: skip the per-expert loop (profiler captures)")

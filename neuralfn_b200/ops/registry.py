@@ -41,6 +41,12 @@ KERNELS: tuple[KernelEntry, ...] = (
     _k("attention_backward", "nfn_attention_backward", ("bf16",), True, "dQ dK dV, delta pre-pass"),
     _k("block_attention", "nfn_block_attention", ("bf16",), True, "cache prefix + block, staging of block K/V, split-KV merge"),
     _k("decode_attention", "nfn_decode_attention", ("bf16",), False, "QK-norm, RoPE, cache append, split-KV merge"),
+    _k("paged attention, prompt tiles", "nfn_paged_attention_tiles", ("bf16",), True, "page table, window, distance bias, GQA packing, output gate"),
+    _k("paged attention, single rows", "nfn_paged_attention_rows", ("bf16", "fp32"), False, "page table, window, distance bias, split-KV merge, output gate"),
+    _k("short convolution + cache append + feed-forward gate", "nfn_mix_rows", ("bf16", "fp32"), False, "per-sequence history, query temperature, transposed value pages"),
+    _k("residual row pass", "nfn_row_norm", ("bf16", "fp32"), False, "embedding, branch norm + residual, next norm, row gather"),
+    _k("per-layer token input gate", "nfn_side_mul", ("bf16", "fp32"), False, "GELU, embedding gather"),
+    _k("gemm, 32-bit", "nfn_gemm_f32", ("fp32",), False, "accumulate"),
     _k("turboquant_attention", "nfn_turboquant_attention", ("tq-3.5",), False, "attention on compressed records"),
     _k("turboquant_encode", "nfn_turboquant_encode", ("tq-3.5",)),
     _k("kv_commit", "nfn_kv_commit_layers"), _k("kv_cache_write", "nfn_kv_cache_write"),
