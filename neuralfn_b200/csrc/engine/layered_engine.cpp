@@ -8,11 +8,15 @@
 // convolutions keep taps - 1 projected rows per slot and layer in two halves: a step reads one half and writes the other, so no
 // launch reads what it overwrites.
 //
+// Delta-rule layers have no pages: a slot keeps one fp32 state per head, read and written in place. Layers of a loop share tensors and
+// have caches and states of their own.
+//
 // A step lays its rows out short entries first (single tokens and portions below kTileMin rows: one query row at a time), then
 // the long ones (tcgen05 tiles). Per layer it launches: input projection (q | k | v | gates | feed-forward in one product), the
 // row mix (convolution, temperature, cache append, feed-forward gate), attention with the output gate, one output product that
 // adds mixer and feed-forward to the 32-bit residual stream, and the token input's two products with their norm, which also
-// produces the next layer's normalised rows. Steps of single tokens run with a padded row count and are replayed as CUDA graphs.
+// produces the next layer's normalised rows. `chained` models run mixer and feed-forward as two sublayers with a stream pass after each
+// (chained_pass). Steps of single tokens run with a padded row count and are replayed as CUDA graphs.
 #include <cmath>
 #include <cstring>
 #include <memory>
@@ -32,16 +36,25 @@ struct Layer {
   int dp = 0, vp = 0, ff = 0;                       // padded head sizes and feed-forward width
   int nq = 0, nk = 0, nv = 0, off_g = 0, off_gate = 0, off_up = 0, n_in = 0, n_cat = 0;
   int owner = 0, group = 0;
+  int n_conv = 0;                                   // channels that pass the convolution
+  int off_b = 0, off_a1 = 0, off_g1 = 0, ra = 0, rg = 0;   // delta: step size, decay and gate projections inside the input product
+  int ep = 0, ef = 0;                               // padded number of experts (router rows) and expert width
   void *k_pool = nullptr, *v_pool = nullptr, *state = nullptr;
   long long state_half = 0;
+  float* memory = nullptr;                          // delta: [slots][heads][dp][vp]
   float* slopes = nullptr;
   const void *norm1 = nullptr, *w_in = nullptr, *conv = nullptr, *w_out = nullptr, *side_gate = nullptr, *side_proj = nullptr, *side_norm = nullptr;
+  const void *norm2 = nullptr, *bias_in = nullptr, *w_a2 = nullptr, *w_g2 = nullptr, *a_log = nullptr, *dt_bias = nullptr, *out_norm = nullptr;
+  const void *router = nullptr, *w_gate_up = nullptr, *w_down = nullptr;
+  struct { const void *in = nullptr, *out = nullptr, *mix = nullptr; } hc[2];   // streams: mixer, feed-forward
   int tile_rows = 0;                                // query rows per tcgen05 tile, 0: one row at a time
 };
 
 struct Group {
   int window = 0;                                   // widest reader, 0: everything stays
+  int keep = 0;                                     // first pages that stay whatever the window
   int pages = 0;
+  bool held(int slot, int p) const { return p < keep || p >= first[slot]; }   // of pages below next[slot]
   std::vector<int> free_pages;
   int* d_table = nullptr;                           // [slots][max_pages]
   int* h_table = nullptr;                           // pinned mirror
@@ -58,12 +71,17 @@ struct layered_engine final : nfn_engine {
   float* x = nullptr;
   void *xb = nullptr, *h = nullptr, *in = nullptr, *q = nullptr, *cat = nullptr, *s_act = nullptr, *y = nullptr, *hw = nullptr;
   float *s_gate = nullptr, *logits = nullptr, *saved = nullptr;
+  float *decay = nullptr, *d_o = nullptr;           // delta: projected decays, read-outs
+  void* d_gate = nullptr;
+  struct { float *logits = nullptr, *weight = nullptr, *row_w = nullptr; int *idx = nullptr, *order = nullptr, *offsets = nullptr, *active = nullptr, *counts = nullptr,
+           *cursor = nullptr, *tile_expert = nullptr, *plan = nullptr, *row_of = nullptr; void *xs = nullptr, *gate_up = nullptr, *mid = nullptr, *y = nullptr; } ex;
+  nfn_stream_args pend{};                           // chained: the last sublayer's update, applied on the way to the head
   void *att_ws = nullptr, *gemm_ws = nullptr;
   long long att_ws_bytes = 0, gemm_ws_bytes = 0;
   std::vector<uint8_t> parity;                      // per slot: the half that holds its convolution history
   std::vector<int> logit_at;                        // per slot: row of `logits`, -1: none, -2: `saved`
   // per-step block, one copy to the device: offsets in bytes
-  struct { long long tok, slot, pos, want, params, offset, mix, att, out, total; } io{};
+  struct { long long tok, slot, pos, want, params, offset, mix, att, seq, out, total; } io{};
   unsigned char *h_io = nullptr, *d_io = nullptr;
   std::map<int, cudaGraphExec_t> graphs;            // by padded row count
   std::map<int, long long> graph_launches;
@@ -95,8 +113,16 @@ struct layered_engine final : nfn_engine {
 
   int reserve(int slot, int upto);                  // pages for positions < upto
   void trim(int slot);                              // pages no later query of this slot can see
-  int lin(const void* a, int lda, const void* w, int rows, int n, int k, void* out, int ldo, int kind);
-  int pass(int rows, int short_rows, int n_mix, const std::vector<int>& att_off, const std::vector<int>& att_n);
+  int lin(const void* a, int lda, const void* w, int rows, int n, int k, void* out, int ldo, int kind, const void* bias = nullptr);
+  // the rows of one pass: short entries first, then the long ones
+  struct Batch { int rows = 0, short_rows = 0, n_mix = 0, n_seq = 0, n_short_seq = 0; std::vector<int> att_off, att_n; };
+  int mix_rows(const Layer& L, const Batch& b, void* ff_out);
+  int attention(const Layer& L, const Batch& b);
+  int delta(const Layer& L, const Batch& b);
+  bool grouped(const Layer& L, int rows) const { return c.dtype == 0 && L.d.experts <= 256 && L.d.top <= 32 && (long long)rows * L.d.top > 8LL * L.d.experts; }
+  int experts(const Layer& L, int rows, nfn_stream_args* sp);
+  int pass(const Batch& b);
+  int chained_pass(const Batch& b);
   int head(const int* src_rows, int rows);
   int sample(int rows);
   int run(const std::vector<nfn_step_entry>& part, const int32_t* const* part_tokens, std::vector<int>& row_of, bool single);
@@ -126,9 +152,22 @@ int layered_engine::build() {
   auto want = [&](const std::string& n, long long numel) { expected.emplace_back(n, numel); };
   want("embed", (long long)vp * wp);
   if (sp) want("side_embed", (long long)c.vocab * c.n_layer * sp);
+  if (c.untied_head) want("head", (long long)vp * wp);
   for (int l = 0; l < c.n_layer; ++l) {
     Layer& L = layers[l];
     const nfn_layer_desc& d = L.d;
+    const std::string bad = "engine: layer " + std::to_string(l);
+    if (d.weights_of >= 0) {
+      if (d.weights_of >= l || layers[d.weights_of].d.weights_of >= 0) return efail(bad + " must take its tensors from an earlier layer that has its own");
+      nfn_layer_desc a = d, o = layers[d.weights_of].d;
+      a.weights_of = o.weights_of = -1;
+      if (std::memcmp(&a, &o, sizeof a)) return efail(bad + " and the layer whose tensors it uses differ");
+    }
+    if (c.chained ? (d.ff > 0 || d.out_gate || d.kv_from >= 0) : (d.mixer != NFN_MIXER_ATTENTION || d.experts > 0 || d.qkv_bias))
+      return efail(bad + (c.chained ? ": sublayers one after another have routed experts, no output gate and caches of their own"
+                                    : ": delta mixers, experts and biases need sublayers one after another"));
+    L.ep = d.experts > 0 ? up(d.experts, 16) : 0;
+    L.ef = d.experts > 0 ? up(d.expert_ff, 16) : 0;
     L.dp = up(d.dim, 16);
     L.vp = up(d.vdim, 16);
     L.ff = d.ff > 0 ? up(d.ff, 16) : 0;
@@ -141,50 +180,87 @@ int layered_engine::build() {
       L.owner = d.kv_from;
     }
     const bool own = L.owner == l;
-    L.nq = d.heads * L.dp;
-    L.nk = own ? d.kv_heads * L.dp : 0;
-    L.nv = own ? d.kv_heads * L.vp : 0;
-    L.off_g = L.nq + L.nk + L.nv;
-    L.off_gate = L.off_g + (d.out_gate ? d.heads * L.vp : 0);
-    L.off_up = L.off_gate + L.ff;
-    L.n_in = L.off_up + L.ff;
+    if (d.mixer == NFN_MIXER_DELTA) {   // q, k, v leave the convolution as one row; no pages
+      L.nq = 2 * d.kv_heads * L.dp + d.heads * L.vp;
+      L.ra = up(d.rank_decay, 16);
+      L.rg = up(d.rank_gate, 16);
+      L.off_b = L.nq;
+      L.off_a1 = L.off_b + up(d.heads, 16);
+      L.off_g1 = L.off_a1 + L.ra;
+      L.off_gate = L.off_up = L.n_in = L.off_g1 + L.rg;
+    } else {
+      L.nq = d.heads * L.dp;
+      L.nk = own ? d.kv_heads * L.dp : 0;
+      L.nv = own ? d.kv_heads * L.vp : 0;
+      L.off_g = L.nq + L.nk + L.nv;
+      L.off_gate = L.off_g + (d.out_gate ? d.heads * L.vp : 0);
+      L.off_up = L.off_gate + L.ff;
+      L.n_in = L.off_up + L.ff;
+    }
+    L.n_conv = L.nq + L.nk + L.nv;
     L.n_cat = d.heads * L.vp + L.ff;
     n_in_max = std::max(n_in_max, L.n_in);
     nq_max = std::max(nq_max, L.nq);
     cat_max = std::max(cat_max, L.n_cat);
-    want(lname(l, "norm1"), wp);
-    want(lname(l, "w_in"), (long long)L.n_in * wp);
-    if (d.conv_taps > 0) want(lname(l, "conv"), (long long)d.conv_taps * (L.nq + L.nk + L.nv));
-    want(lname(l, "w_out"), (long long)wp * L.n_cat);
-    if (sp) {
-      want(lname(l, "side_gate"), (long long)sp * wp);
-      want(lname(l, "side_proj"), (long long)wp * sp);
-      want(lname(l, "side_norm"), wp);
+    if (d.weights_of < 0) {
+      want(lname(l, "norm1"), wp);
+      want(lname(l, "w_in"), (long long)L.n_in * wp);
+      if (d.conv_taps > 0) want(lname(l, "conv"), (long long)d.conv_taps * L.n_conv);
+      want(lname(l, "w_out"), (long long)wp * L.n_cat);
+      if (sp) {
+        want(lname(l, "side_gate"), (long long)sp * wp);
+        want(lname(l, "side_proj"), (long long)wp * sp);
+        want(lname(l, "side_norm"), wp);
+      }
+      if (d.qkv_bias) want(lname(l, "bias_in"), L.n_in);
+      if (d.mixer == NFN_MIXER_DELTA) {
+        want(lname(l, "w_a2"), (long long)d.heads * L.dp * L.ra);
+        want(lname(l, "w_g2"), (long long)d.heads * L.vp * L.rg);
+        want(lname(l, "a_log"), d.heads);
+        want(lname(l, "dt_bias"), (long long)d.heads * L.dp);
+        want(lname(l, "out_norm"), L.vp);
+      }
+      if (d.experts > 0) {
+        want(lname(l, "norm2"), wp);
+        want(lname(l, "router"), (long long)L.ep * wp);
+        want(lname(l, "w_gate_up"), (long long)d.experts * 2 * L.ef * wp);
+        want(lname(l, "w_down"), (long long)d.experts * wp * L.ef);
+      }
+      for (int q = 0; q < (c.streams > 0 ? (d.experts > 0 ? 2 : 1) : 0); ++q) {
+        const std::string hc = q ? "hc2_" : "hc1_";
+        want(lname(l, (hc + "in").c_str()), c.streams);
+        want(lname(l, (hc + "out").c_str()), c.streams);
+        want(lname(l, (hc + "mix").c_str()), (long long)c.streams * c.streams);
+      }
     }
+    if (d.mixer == NFN_MIXER_DELTA) continue;
     L.tile_rows = nfn_paged_tile_rows(c.dtype, d.heads, d.kv_heads, L.dp, L.vp);
     if (L.tile_rows > 0 && std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) == tile_kinds.end()) tile_kinds.push_back(L.tile_rows);
   }
   want("final_norm", wp);
   // how far back the readers of each owner look, and one group per distinct answer
   for (int l = 0; l < c.n_layer; ++l) {
-    if (layers[l].owner != l) continue;
-    int w = 0;
+    if (layers[l].owner != l || layers[l].d.mixer == NFN_MIXER_DELTA) continue;
+    int w = 0, keep = 0;
     bool all = false;
     for (const Layer& r : layers)
       if (r.owner == l) {
         all |= r.d.window <= 0;
         w = std::max(w, r.d.window);
+        keep = std::max(keep, (r.d.keep_first + kPage - 1) / kPage);
       }
-    if (all) w = 0;
+    if (all) w = keep = 0;
     int g = 0;
-    while (g < (int)groups.size() && groups[g].window != w) ++g;
+    while (g < (int)groups.size() && (groups[g].window != w || groups[g].keep != keep)) ++g;
     if (g == (int)groups.size()) {
       groups.emplace_back();
       groups.back().window = w;
+      groups.back().keep = keep;
     }
     for (Layer& r : layers)
       if (r.owner == l) r.group = g;
   }
+  if (groups.empty()) groups.emplace_back();   // no layer has pages: the pool still counts tokens
   len.assign(c.max_batch, 0);
   parity.assign(c.max_batch, 0);
   logit_at.assign(c.max_batch, -1);
@@ -198,7 +274,8 @@ extern "C" nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, 
   }
   const nfn_layered_config& c = *cfg;
   if (c.n_layer <= 0 || c.width <= 0 || c.vocab <= 0 || c.side_dim < 0 || (c.dtype != 0 && c.dtype != 1) || c.max_seq <= 0 || c.max_batch <= 0 ||
-      c.kv_tokens < 0 || c.max_step_rows <= 0 || !(c.norm_eps >= 0.f)) {
+      c.kv_tokens < 0 || c.max_step_rows <= 0 || !(c.norm_eps >= 0.f) || c.streams < 0 || c.streams > NFN_MAX_STREAMS || (c.streams > 0 && !c.chained) ||
+      (c.chained && c.side_dim > 0) || !(c.logit_softcap >= 0.f) || (!c.chained && c.norm_offset != 0.f)) {
     efail("engine_create: invalid geometry");
     return nullptr;
   }
@@ -209,7 +286,9 @@ extern "C" nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, 
   for (int l = 0; l < c.n_layer; ++l) {
     const nfn_layer_desc& d = layers[l];
     if (d.heads <= 0 || d.kv_heads <= 0 || d.heads % d.kv_heads || d.dim <= 0 || d.vdim <= 0 || d.conv_taps < 0 || d.ff < 0 || d.window < 0 ||
-        d.q_temp_every < 0 || (d.ff_act != NFN_ACT_RELU && d.ff_act != NFN_ACT_SILU && d.ff_act != NFN_ACT_GELU_TANH)) {
+        d.q_temp_every < 0 || d.keep_first < 0 || d.softcap < 0.f || d.experts < 0 || (d.experts > 0 && (d.top < 1 || d.top > d.experts || d.expert_ff < 1)) ||
+        (d.mixer != NFN_MIXER_ATTENTION && d.mixer != NFN_MIXER_DELTA) ||
+        (d.mixer == NFN_MIXER_DELTA && (d.conv_taps < 1 || d.rank_decay < 1 || d.rank_gate < 1 || d.dim > 512)) || (d.ff_act != NFN_ACT_RELU && d.ff_act != NFN_ACT_SILU && d.ff_act != NFN_ACT_GELU_TANH)) {
       efail("engine_create: invalid sizes in layer " + std::to_string(l));
       return nullptr;
     }
@@ -235,14 +314,45 @@ int layered_engine::finalize() {
     CU(cudaMemset(*p, 0, (size_t)n));
     return 0;
   };
-  if (zero((void**)&x, R * wp * 4) || zero(&h, R * wp * es) || zero(&in, R * n_in_max * es) || zero(&q, R * nq_max * es) || zero(&cat, R * cat_max * es) ||
+  if (zero((void**)&x, R * wp * 4 * std::max(c.streams, 1)) || zero(&h, R * wp * es) || zero(&in, R * n_in_max * es) || zero(&q, R * nq_max * es) || zero(&cat, R * cat_max * es) ||
       zero(&hw, (long long)logit_rows * wp * es) || zero((void**)&logits, (long long)logit_rows * vp * 4) || zero((void**)&saved, S * vp * 4))
     return -1;
   if (c.dtype == 0 && zero(&xb, R * wp * 2)) return -1;
-  if (sp && (zero((void**)&s_gate, R * sp * 4) || zero(&s_act, R * sp * es) || zero(&y, R * wp * es))) return -1;
+  if (sp && (zero((void**)&s_gate, R * sp * 4) || zero(&s_act, R * sp * es))) return -1;
+  if ((sp || c.chained) && zero(&y, R * wp * es)) return -1;
+  // scratch of the delta mixers and of the experts: the largest any layer asks for
+  long long n_dec = 0, n_do = 0, e_log = 0, e_max = 0, e_items = 0, e_sorted = 0, e_gu = 0, e_mid = 0, e_rows = 0;
+  for (const Layer& L : layers) {
+    const nfn_layer_desc& d = L.d;
+    if (d.mixer == NFN_MIXER_DELTA) {
+      n_dec = std::max(n_dec, R * d.heads * L.dp);
+      n_do = std::max(n_do, R * d.heads * L.vp);
+    }
+    if (d.experts > 0) {
+      const bool g = grouped(L, (int)R);
+      const long long sorted = g ? (R * d.top + d.experts * 127LL + 127) / 128 * 128 : 0;
+      const long long single = std::min(R * d.top, c.dtype == 0 && g ? 8LL * d.experts : R * d.top);   // items of the largest step outside the sorted form
+      e_log = std::max(e_log, R * L.ep);
+      e_max = std::max<long long>(e_max, d.experts);
+      e_items = std::max(e_items, R * d.top);
+      e_sorted = std::max(e_sorted, sorted);
+      e_gu = std::max(e_gu, sorted * 2 * L.ef);
+      e_mid = std::max(e_mid, std::max(sorted, single) * L.ef);
+      e_rows = std::max(e_rows, std::max(sorted, single));
+    }
+  }
+  if (n_dec && (zero((void**)&decay, n_dec * 4) || zero((void**)&d_o, n_do * 4) || zero(&d_gate, n_do * es))) return -1;
+  if (e_max && (zero((void**)&ex.logits, e_log * 4) || zero((void**)&ex.weight, e_items * 4) || zero((void**)&ex.idx, e_items * 4) ||
+                zero((void**)&ex.order, e_items * 4) || zero((void**)&ex.row_of, e_items * 4) || zero((void**)&ex.offsets, (e_max + 1) * 4) ||
+                zero((void**)&ex.active, (e_max + 1) * 4) || zero((void**)&ex.counts, e_max * 4) || zero((void**)&ex.cursor, e_max * 4) ||
+                zero((void**)&ex.plan, 16) || zero(&ex.mid, e_mid * es) || zero(&ex.y, e_rows * wp * es)))
+    return -1;
+  if (e_sorted && (zero((void**)&ex.row_w, e_sorted * 4) || zero((void**)&ex.tile_expert, e_sorted / 128 * 4) || zero(&ex.xs, e_sorted * wp * 2) ||
+                   zero(&ex.gate_up, e_gu * 2)))
+    return -1;
   for (Group& g : groups) {
     g.pages = (c.kv_tokens + kPage - 1) / kPage;
-    if (g.window > 0) g.pages = (int)std::min<long long>(g.pages, S * ((g.window + R) / kPage + 2));
+    if (g.window > 0) g.pages = (int)std::min<long long>(g.pages, S * ((g.window + R) / kPage + 2 + g.keep));
     for (int p = g.pages - 1; p >= 0; --p) g.free_pages.push_back(p);
     g.first.assign(S, 0);
     g.next.assign(S, 0);
@@ -254,7 +364,9 @@ int layered_engine::finalize() {
   for (int l = 0; l < c.n_layer; ++l) {
     Layer& L = layers[l];
     const nfn_layer_desc& d = L.d;
-    if (L.owner == l) {
+    if (d.mixer == NFN_MIXER_DELTA) {
+      if (zero((void**)&L.memory, S * d.heads * L.dp * L.vp * 4)) return -1;
+    } else if (L.owner == l) {
       const long long tiles = (long long)groups[L.group].pages * d.kv_heads * kPage;
       if (zero(&L.k_pool, tiles * L.dp * es) || zero(&L.v_pool, tiles * L.vp * es)) return -1;
     } else {
@@ -262,23 +374,44 @@ int layered_engine::finalize() {
       L.v_pool = layers[L.owner].v_pool;
     }
     if (d.conv_taps > 1) {
-      L.state_half = S * (d.conv_taps - 1) * (L.nq + L.nk + L.nv);
+      L.state_half = S * (d.conv_taps - 1) * L.n_conv;
       if (zero(&L.state, 2 * L.state_half * es)) return -1;
     }
-    if (d.conv_taps > 0) L.conv = W(lname(l, "conv"));
+    const int wl = d.weights_of >= 0 ? d.weights_of : l;
+    if (d.conv_taps > 0) L.conv = W(lname(wl, "conv"));
     if (d.alibi != 0.f) {
       std::vector<float> sl(d.heads);
       for (int i = 0; i < d.heads; ++i) sl[i] = (float)std::exp2(-(double)d.alibi * (i + 1) / d.heads);
       if (zero((void**)&L.slopes, 4LL * d.heads)) return -1;
       CU(cudaMemcpy(L.slopes, sl.data(), sl.size() * 4, cudaMemcpyHostToDevice));
     }
-    L.norm1 = W(lname(l, "norm1"));
-    L.w_in = W(lname(l, "w_in"));
-    L.w_out = W(lname(l, "w_out"));
+    L.norm1 = W(lname(wl, "norm1"));
+    L.w_in = W(lname(wl, "w_in"));
+    L.w_out = W(lname(wl, "w_out"));
+    if (d.qkv_bias) L.bias_in = W(lname(wl, "bias_in"));
+    if (d.mixer == NFN_MIXER_DELTA) {
+      L.w_a2 = W(lname(wl, "w_a2"));
+      L.w_g2 = W(lname(wl, "w_g2"));
+      L.a_log = W(lname(wl, "a_log"));
+      L.dt_bias = W(lname(wl, "dt_bias"));
+      L.out_norm = W(lname(wl, "out_norm"));
+    }
+    if (d.experts > 0) {
+      L.norm2 = W(lname(wl, "norm2"));
+      L.router = W(lname(wl, "router"));
+      L.w_gate_up = W(lname(wl, "w_gate_up"));
+      L.w_down = W(lname(wl, "w_down"));
+    }
+    for (int q = 0; q < (c.streams > 0 ? (d.experts > 0 ? 2 : 1) : 0); ++q) {
+      const std::string hc = q ? "hc2_" : "hc1_";
+      L.hc[q].in = W(lname(wl, (hc + "in").c_str()));
+      L.hc[q].out = W(lname(wl, (hc + "out").c_str()));
+      L.hc[q].mix = W(lname(wl, (hc + "mix").c_str()));
+    }
     if (sp) {
-      L.side_gate = W(lname(l, "side_gate"));
-      L.side_proj = W(lname(l, "side_proj"));
-      L.side_norm = W(lname(l, "side_norm"));
+      L.side_gate = W(lname(wl, "side_gate"));
+      L.side_proj = W(lname(wl, "side_proj"));
+      L.side_norm = W(lname(wl, "side_norm"));
     }
     ws = std::max(ws, nfn_paged_attention_workspace_bytes(rows_max, d.heads, L.vp));
   }
@@ -295,7 +428,8 @@ int layered_engine::finalize() {
   io.offset = io.params + up256((long long)logit_rows * 12);
   io.mix = io.offset + 256;
   io.att = io.mix + up256(R * (long long)sizeof(nfn_row_tile));
-  io.out = io.att + up256(kinds * R * 16);
+  io.seq = io.att + up256(kinds * R * 16);
+  io.out = io.seq + up256(S * (long long)sizeof(nfn_seq_rows));
   io.total = io.out + up256((long long)logit_rows * 4);
   CU(cudaMallocHost((void**)&h_io, (size_t)io.total));
   std::memset(h_io, 0, (size_t)io.total);
@@ -342,13 +476,14 @@ void layered_engine::trim(int slot) {
     if (g.window <= 0) continue;
     const int live = std::max(0, len[slot] - g.window + 1) / kPage;
     for (; g.first[slot] < std::min(live, g.next[slot]); ++g.first[slot])
-      g.free_pages.push_back(g.h_table[(size_t)slot * max_pages + g.first[slot]]);
+      if (g.first[slot] >= g.keep) g.free_pages.push_back(g.h_table[(size_t)slot * max_pages + g.first[slot]]);
   }
 }
 
 int layered_engine::release(int slot) {
   for (Group& g : groups) {
-    for (int p = g.first[slot]; p < g.next[slot]; ++p) g.free_pages.push_back(g.h_table[(size_t)slot * max_pages + p]);
+    for (int p = 0; p < g.next[slot]; ++p)
+      if (g.held(slot, p)) g.free_pages.push_back(g.h_table[(size_t)slot * max_pages + p]);
     g.first[slot] = g.next[slot] = 0;
   }
   len[slot] = 0;
@@ -359,27 +494,28 @@ int layered_engine::release(int slot) {
 int layered_engine::truncate(int slot, int n) {
   if (n == len[slot]) return 0;
   if (n == 0) return release(slot);
-  return efail("engine_truncate: the short convolutions keep the newest rows only; a shorter prefix has to be run again");
+  return efail("engine_truncate: recurrent state and short convolutions keep the newest rows only; a shorter prefix has to be run again");
 }
 
 int layered_engine::fork(int src, int dst, int n) {
-  if (n != len[src]) return efail("engine_fork: the short convolutions keep the newest rows only; a shorter prefix has to be run again");
+  if (n != len[src]) return efail("engine_fork: recurrent state and short convolutions keep the newest rows only; a shorter prefix has to be run again");
   CU(cudaSetDevice(device));
   release(dst);
   if (n == 0) return 0;
   for (Group& g : groups)   // pages the source gave back hold nothing the copy needs
-    if (g.next[src] - g.first[src] > (int)g.free_pages.size()) return efail("engine_fork: the cache pool is full");
+    if (g.next[src] - g.first[src] + std::min(g.first[src], g.keep) > (int)g.free_pages.size()) return efail("engine_fork: the cache pool is full");
   for (size_t gi = 0; gi < groups.size(); ++gi) {
     Group& g = groups[gi];
     int *from = g.h_table + (size_t)src * max_pages, *to = g.h_table + (size_t)dst * max_pages;
     g.first[dst] = g.first[src];
     g.next[dst] = g.next[src];
-    for (int p = g.first[src]; p < g.next[src]; ++p) {
+    for (int p = 0; p < g.next[src]; ++p) {
+      if (!g.held(src, p)) continue;
       to[p] = g.free_pages.back();
       g.free_pages.pop_back();
       for (int l = 0; l < c.n_layer; ++l) {
         const Layer& L = layers[l];
-        if (L.owner != l || L.group != (int)gi) continue;
+        if (L.owner != l || L.group != (int)gi || L.d.mixer == NFN_MIXER_DELTA) continue;
         const size_t kb = (size_t)L.d.kv_heads * kPage * L.dp * es, vb = (size_t)L.d.kv_heads * kPage * L.vp * es;
         CU(cudaMemcpyAsync(static_cast<char*>(L.k_pool) + to[p] * kb, static_cast<char*>(L.k_pool) + from[p] * kb, kb, cudaMemcpyDeviceToDevice, stream));
         CU(cudaMemcpyAsync(static_cast<char*>(L.v_pool) + to[p] * vb, static_cast<char*>(L.v_pool) + from[p] * vb, vb, cudaMemcpyDeviceToDevice, stream));
@@ -389,8 +525,12 @@ int layered_engine::fork(int src, int dst, int n) {
   }
   parity[dst] = parity[src];
   for (const Layer& L : layers) {
+    if (L.memory) {
+      const size_t n = (size_t)L.d.heads * L.dp * L.vp;
+      CU(cudaMemcpyAsync(L.memory + dst * n, L.memory + src * n, n * 4, cudaMemcpyDeviceToDevice, stream));
+    }
     if (!L.state) continue;
-    const size_t row = (size_t)(L.d.conv_taps - 1) * (L.nq + L.nk + L.nv) * es;
+    const size_t row = (size_t)(L.d.conv_taps - 1) * L.n_conv * es;
     char* half = static_cast<char*>(L.state) + (size_t)parity[src] * L.state_half * es;
     CU(cudaMemcpyAsync(half + dst * row, half + src * row, row, cudaMemcpyDeviceToDevice, stream));
   }
@@ -402,9 +542,9 @@ int layered_engine::fork(int src, int dst, int n) {
 // ---- one pass over the rows of a step -----------------------------------------------------------------
 
 // out = a . w^T: kOutAct in the activation type, kOutF32 in fp32, kOutResidual added to the residual stream x
-int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n, int k, void* out, int ldo, int kind) {
+int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n, int k, void* out, int ldo, int kind, const void* bias) {
   if (c.dtype == 1) {
-    K(nfn_gemm_f32(static_cast<const float*>(a), lda, wt, k, static_cast<float*>(out), ldo, rows, n, k, kind == kOutResidual, stream));
+    K(nfn_gemm_f32(static_cast<const float*>(a), lda, wt, k, static_cast<float*>(out), ldo, rows, n, k, kind == kOutResidual, bias, stream));
     return 0;
   }
   nfn_gemm_args g{};
@@ -418,14 +558,120 @@ int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n,
     g.aux_out = xb;
     g.ld_aux_out = wp;
   }
+  if (bias) {
+    g.flags |= NFN_EPI_BIAS;
+    g.bias = bias;
+  }
   g.workspace = gemm_ws;
   g.workspace_bytes = gemm_ws_bytes;
   K(nfn_gemm_bf16(&g, stream));
   return 0;
 }
 
-int layered_engine::pass(int rows, int short_rows, int n_mix, const std::vector<int>& att_off, const std::vector<int>& att_n) {
-  const int f32 = c.dtype == 1;
+// The step between a layer's input product and its mixer. Delta layers: the convolved and activated [q | k | v] rows stay in `q`.
+int layered_engine::mix_rows(const Layer& L, const Batch& b, void* ff_out) {
+  const nfn_layer_desc& d = L.d;
+  nfn_mix_args m{};
+  m.f32 = c.dtype == 1; m.in = in; m.ld_in = L.n_in;
+  m.nq = L.nq; m.nk = L.nk; m.nv = L.nv; m.off_gate = L.off_gate; m.off_up = L.off_up; m.ff = L.ff; m.act = d.ff_act;
+  m.conv = L.conv; m.taps = d.conv_taps; m.state = L.state; m.state_half = L.state_half;
+  m.conv_act = d.mixer == NFN_MIXER_DELTA ? NFN_ACT_SILU : NFN_ACT_NONE;
+  m.q_out = q; m.ld_q = L.nq;
+  m.k_pool = L.k_pool; m.v_pool = L.v_pool; m.kv_heads = d.kv_heads; m.dim_p = L.dp; m.vdim_p = L.vp;
+  m.table = groups[L.group].d_table; m.table_ld = max_pages;
+  m.temp_coef = d.q_temp_coef; m.temp_every = d.q_temp_every;
+  m.ff_out = ff_out; m.ld_ff = L.n_cat;
+  m.tiles = dev<nfn_row_tile>(io.mix); m.n_tiles = b.n_mix; m.tile_rows = b.n_mix == b.rows ? 1 : kMixRows; m.rows = b.rows;
+  K(nfn_mix_rows(&m, stream));
+  return 0;
+}
+
+// q rows over the layer's pages -> the first columns of `cat`
+int layered_engine::attention(const Layer& L, const Batch& b) {
+  const nfn_layer_desc& d = L.d;
+  nfn_paged_attention_args a{};
+  a.f32 = c.dtype == 1; a.q = q; a.ld_q = L.nq; a.total_rows = rows_max;
+  a.k_pool = L.k_pool; a.v_pool = L.v_pool; a.kv_heads = d.kv_heads; a.dim_p = L.dp; a.vdim_p = L.vp; a.pages = groups[L.group].pages;
+  a.table = groups[L.group].d_table; a.table_ld = max_pages;
+  a.heads = d.heads; a.window = d.window; a.scale = d.scale; a.slopes = L.slopes;
+  a.keep_first = d.window > 0 ? d.keep_first : 0; a.softcap = d.softcap; a.sink = d.sink;
+  a.gate = d.out_gate ? static_cast<char*>(in) + (size_t)L.off_g * es : nullptr; a.ld_gate = L.n_in;
+  a.out = cat; a.ld_o = L.n_cat;
+  a.row_slot = dev<int>(io.slot); a.row_pos = dev<int>(io.pos);
+  a.max_keys = d.window > 0 ? std::min(d.window + d.keep_first, c.max_seq) : c.max_seq;
+  a.workspace = att_ws; a.workspace_bytes = att_ws_bytes;
+  const int single = L.tile_rows > 0 ? b.short_rows : b.rows;
+  if (single > 0) {
+    a.rows = single;
+    K(nfn_paged_attention_rows(&a, stream));
+  }
+  if (L.tile_rows > 0 && b.rows > b.short_rows) {
+    const int k = (int)(std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) - tile_kinds.begin());
+    a.tiles = dev<int>(io.att) + b.att_off[k] * 4;
+    a.n_tiles = b.att_n[k];
+    K(nfn_paged_attention_tiles(&a, stream));
+  }
+  return 0;
+}
+
+// Gated delta rule over the convolved rows -> the first columns of `cat`
+int layered_engine::delta(const Layer& L, const Batch& b) {
+  const nfn_layer_desc& d = L.d;
+  const int n_dec = d.heads * L.dp, n_o = d.heads * L.vp;
+  const char* low = static_cast<const char*>(in);
+  if (lin(low + (size_t)L.off_a1 * es, L.n_in, L.w_a2, b.rows, n_dec, L.ra, decay, n_dec, kOutF32)) return -1;
+  if (lin(low + (size_t)L.off_g1 * es, L.n_in, L.w_g2, b.rows, n_o, L.rg, d_gate, n_o, kOutAct)) return -1;
+  nfn_delta_args a{};
+  a.f32 = c.dtype == 1; a.qkv = q; a.ld_qkv = L.nq;
+  a.beta = low + (size_t)L.off_b * es; a.ld_beta = L.n_in;
+  a.decay = decay; a.ld_decay = n_dec; a.a_log = L.a_log; a.dt_bias = L.dt_bias;
+  a.heads = d.heads; a.kv_heads = d.kv_heads; a.dim = d.dim; a.dim_p = L.dp; a.vdim_p = L.vp; a.unit_eps = 1e-6f;
+  a.state = L.memory; a.o = d_o; a.ld_o = n_o;
+  a.seqs = dev<nfn_seq_rows>(io.seq); a.n_seqs = b.n_seq;
+  K(nfn_delta_rows(&a, stream));
+  K(nfn_delta_out(a.f32, d_o, n_o, d_gate, n_o, L.out_norm, c.norm_eps, cat, L.n_cat, b.rows, d.heads, d.vdim, L.vp, stream));
+  return 0;
+}
+
+// Routed experts on the normalised rows h; says in `sp` where the next stream pass finds each row's outputs.
+int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
+  const nfn_layer_desc& d = L.d;
+  if (lin(h, wp, L.router, rows, L.ep, wp, ex.logits, L.ep, kOutF32)) return -1;
+  sp->y = ex.y;
+  sp->y_rows = d.top;
+  if (!grouped(L, rows)) {
+    nfn_moe_rows_args a{};
+    a.f32 = c.dtype == 1; a.rows = rows; a.width = wp; a.ff = L.ef; a.experts = d.experts; a.top = d.top; a.act = d.ff_act;
+    a.logits = ex.logits; a.ld_logits = L.ep; a.h = h; a.ld_h = wp; a.w_gate_up = L.w_gate_up; a.w_down = L.w_down;
+    a.idx = ex.idx; a.weight = ex.weight; a.order = ex.order; a.offsets = ex.offsets; a.active = ex.active;
+    a.mid = ex.mid; a.y = ex.y; a.ld_y = wp;
+    K(nfn_moe_rows(&a, stream));
+    sp->y_index = nullptr;
+    return 0;
+  }
+  const int cap = (int)(((long long)rows * d.top + d.experts * 127LL + 127) / 128 * 128);
+  CU(cudaMemsetAsync(ex.counts, 0, (size_t)d.experts * 4, stream));
+  K(nfn_moe_route(ex.logits, L.ep, rows, d.experts, d.top, 1, 0, 1.f, ex.idx, ex.weight, ex.counts, stream));
+  K(nfn_moe_plan(ex.counts, d.experts, cap / 128, ex.offsets, ex.cursor, ex.tile_expert, ex.plan, stream));
+  K(nfn_moe_permute_weighted(h, wp, rows, d.top, wp, ex.idx, ex.weight, ex.offsets, ex.cursor, cap, ex.xs, ex.row_of, ex.row_w, stream));
+  nfn_gemm_tp_args g{};
+  g.mode = NFN_TP_GROUPED;
+  g.tile_group = ex.tile_expert; g.num_m_tiles_dev = ex.plan; g.groups = d.experts; g.m = cap;
+  g.a = ex.xs; g.b = L.w_gate_up; g.c = ex.gate_up;
+  g.n = 2 * L.ef; g.k = g.lda = g.ldb = wp; g.ldc = 2 * L.ef;
+  K(nfn_gemm_tp(&g, stream));
+  K(nfn_moe_act_rows(ex.gate_up, ex.row_w, ex.plan, cap, L.ef, d.ff_act, ex.mid, stream));
+  g.a = ex.mid; g.b = L.w_down; g.c = ex.y;
+  g.n = wp; g.k = g.lda = g.ldb = L.ef; g.ldc = wp;
+  K(nfn_gemm_tp(&g, stream));
+  sp->y_index = ex.row_of;
+  return 0;
+}
+
+// Layers whose mixer and feed-forward read one norm
+int layered_engine::pass(const Batch& b) {
+  if (c.chained) return chained_pass(b);
+  const int f32 = c.dtype == 1, rows = b.rows;
   nfn_row_norm_args rn{};
   rn.f32 = f32; rn.rows = rows; rn.width = c.width; rn.ld = wp; rn.eps = c.norm_eps;
   rn.tokens = dev<int>(io.tok); rn.embed = W("embed"); rn.embed_scale = c.embed_scale; rn.vocab = c.vocab;
@@ -434,44 +680,8 @@ int layered_engine::pass(int rows, int short_rows, int n_mix, const std::vector<
   rn.tokens = nullptr; rn.embed = nullptr; rn.x = x;
   for (int l = 0; l < c.n_layer; ++l) {
     const Layer& L = layers[l];
-    const nfn_layer_desc& d = L.d;
     if (lin(h, wp, L.w_in, rows, L.n_in, wp, in, L.n_in, kOutAct)) return -1;
-
-    char* ff_out = static_cast<char*>(cat) + (size_t)d.heads * L.vp * es;
-    nfn_mix_args m{};
-    m.f32 = f32; m.in = in; m.ld_in = L.n_in;
-    m.nq = L.nq; m.nk = L.nk; m.nv = L.nv; m.off_gate = L.off_gate; m.off_up = L.off_up; m.ff = L.ff; m.act = d.ff_act;
-    m.conv = L.conv; m.taps = d.conv_taps; m.state = L.state; m.state_half = L.state_half;
-    m.q_out = q; m.ld_q = L.nq;
-    m.k_pool = L.k_pool; m.v_pool = L.v_pool; m.kv_heads = d.kv_heads; m.dim_p = L.dp; m.vdim_p = L.vp;
-    m.table = groups[L.group].d_table; m.table_ld = max_pages;
-    m.temp_coef = d.q_temp_coef; m.temp_every = d.q_temp_every;
-    m.ff_out = ff_out; m.ld_ff = L.n_cat;
-    m.tiles = dev<nfn_row_tile>(io.mix); m.n_tiles = n_mix; m.tile_rows = n_mix == rows ? 1 : kMixRows; m.rows = rows;
-    K(nfn_mix_rows(&m, stream));
-
-    nfn_paged_attention_args a{};
-    a.f32 = f32; a.q = q; a.ld_q = L.nq; a.total_rows = rows_max;
-    a.k_pool = L.k_pool; a.v_pool = L.v_pool; a.kv_heads = d.kv_heads; a.dim_p = L.dp; a.vdim_p = L.vp; a.pages = groups[L.group].pages;
-    a.table = m.table; a.table_ld = max_pages;
-    a.heads = d.heads; a.window = d.window; a.scale = d.scale; a.slopes = L.slopes;
-    a.gate = d.out_gate ? static_cast<char*>(in) + (size_t)L.off_g * es : nullptr; a.ld_gate = L.n_in;
-    a.out = cat; a.ld_o = L.n_cat;
-    a.row_slot = dev<int>(io.slot); a.row_pos = dev<int>(io.pos);
-    a.max_keys = d.window > 0 ? std::min(d.window, c.max_seq) : c.max_seq;
-    a.workspace = att_ws; a.workspace_bytes = att_ws_bytes;
-    const int single = L.tile_rows > 0 ? short_rows : rows;
-    if (single > 0) {
-      a.rows = single;
-      K(nfn_paged_attention_rows(&a, stream));
-    }
-    if (L.tile_rows > 0 && rows > short_rows) {
-      const int k = (int)(std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) - tile_kinds.begin());
-      a.tiles = dev<int>(io.att) + att_off[k] * 4;
-      a.n_tiles = att_n[k];
-      K(nfn_paged_attention_tiles(&a, stream));
-    }
-
+    if (mix_rows(L, b, static_cast<char*>(cat) + (size_t)L.d.heads * L.vp * es) || attention(L, b)) return -1;
     if (lin(cat, L.n_cat, L.w_out, rows, wp, L.n_cat, x, wp, kOutResidual)) return -1;
     const bool last = l + 1 == c.n_layer;
     if (sp) {
@@ -489,13 +699,54 @@ int layered_engine::pass(int rows, int short_rows, int n_mix, const std::vector<
   return 0;
 }
 
-// output norm and tied head of `rows` rows of x (src_rows: device indices, NULL: the first ones) -> logits
+// Layers of two sublayers. A stream pass after each one applies its output to the residual and norms the next one's input; the last
+// update is left to the head, which needs it for the wanted rows only.
+int layered_engine::chained_pass(const Batch& b) {
+  nfn_stream_args s{};
+  s.f32 = c.dtype == 1; s.rows = b.rows; s.width = c.width; s.ld = wp; s.streams = std::max(c.streams, 1);
+  s.eps = c.norm_eps; s.weight_offset = c.norm_offset;
+  s.tokens = dev<int>(io.tok); s.embed = W("embed"); s.embed_scale = c.embed_scale; s.vocab = c.vocab;
+  s.x = x; s.x_out = x; s.h = h;
+  s.in = layers[0].hc[0].in; s.weight = layers[0].norm1;
+  K(nfn_stream_pass(&s, stream));
+  s.tokens = nullptr; s.embed = nullptr;
+  for (int l = 0; l < c.n_layer; ++l) {
+    const Layer& L = layers[l];
+    if (lin(h, wp, L.w_in, b.rows, L.n_in, wp, in, L.n_in, kOutAct, L.bias_in) || mix_rows(L, b, nullptr)) return -1;
+    if (L.d.mixer == NFN_MIXER_DELTA ? delta(L, b) : attention(L, b)) return -1;
+    if (lin(cat, L.n_cat, L.w_out, b.rows, wp, L.n_cat, y, wp, kOutAct)) return -1;
+    s.y = y; s.y_rows = 1; s.y_index = nullptr; s.mix = L.hc[0].mix; s.out = L.hc[0].out;
+    if (L.d.experts > 0) {
+      s.in = L.hc[1].in; s.weight = L.norm2;
+      K(nfn_stream_pass(&s, stream));
+      if (experts(L, b.rows, &s)) return -1;
+      s.mix = L.hc[1].mix; s.out = L.hc[1].out;
+    }
+    if (l + 1 < c.n_layer) {
+      s.in = layers[l + 1].hc[0].in; s.weight = layers[l + 1].norm1;
+      K(nfn_stream_pass(&s, stream));
+    }
+  }
+  pend = s;
+  return 0;
+}
+
+// output norm and head of `rows` rows of x (src_rows: device indices, NULL: the first ones) -> logits
 int layered_engine::head(const int* src_rows, int rows) {
-  nfn_row_norm_args rn{};
-  rn.f32 = c.dtype == 1; rn.rows = rows; rn.width = c.width; rn.ld = wp; rn.eps = c.norm_eps;
-  rn.x = x; rn.src_rows = src_rows; rn.h = hw; rn.weight = W("final_norm");
-  K(nfn_row_norm(&rn, stream));
-  return lin(hw, wp, W("embed"), rows, vp, wp, logits, vp, kOutF32);
+  if (c.chained) {
+    nfn_stream_args s = pend;
+    s.rows = rows; s.src_rows = src_rows; s.x_out = nullptr;
+    s.in = nullptr; s.h = hw; s.weight = W("final_norm");
+    K(nfn_stream_pass(&s, stream));
+  } else {
+    nfn_row_norm_args rn{};
+    rn.f32 = c.dtype == 1; rn.rows = rows; rn.width = c.width; rn.ld = wp; rn.eps = c.norm_eps;
+    rn.x = x; rn.src_rows = src_rows; rn.h = hw; rn.weight = W("final_norm");
+    K(nfn_row_norm(&rn, stream));
+  }
+  if (lin(hw, wp, W(c.untied_head ? "head" : "embed"), rows, vp, wp, logits, vp, kOutF32)) return -1;
+  if (c.logit_softcap > 0.f || c.logit_scale != 1.f) K(nfn_logit_cap(logits, vp, rows, vp, c.logit_scale, c.logit_softcap, stream));
+  return 0;
 }
 
 int layered_engine::sample(int rows) {
@@ -508,6 +759,7 @@ int layered_engine::sample(int rows) {
 // brings one token, and the pass, the head over all rows and the sampling run as one (replayed) launch sequence.
 int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* const* part_tokens, std::vector<int>& row_of, bool single) {
   int total = 0, short_rows = 0;
+  Batch b;
   std::vector<int> first(part.size());
   for (size_t i = 0; i < part.size(); ++i) {
     if (reserve(part[i].slot, len[part[i].slot] + part[i].count)) return -1;
@@ -553,7 +805,18 @@ int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* 
     }
     short_rows = rows;
   }
-  std::vector<int> att_off(tile_kinds.size(), 0), att_n(tile_kinds.size(), 0);
+  nfn_seq_rows* seq = host<nfn_seq_rows>(io.seq);
+  for (int longs = 0; longs < 2; ++longs) {
+    for (size_t i = 0; i < part.size(); ++i)
+      if ((part[i].count >= kTileMin) == (longs == 1)) seq[b.n_seq++] = nfn_seq_rows{first[i], part[i].count, part[i].slot, len[part[i].slot]};
+    if (!longs) {
+      for (int r = total; r < rows; ++r) seq[b.n_seq++] = nfn_seq_rows{r, 1, -1, 0};
+      b.n_short_seq = b.n_seq;
+    }
+  }
+  std::vector<int>&att_off = b.att_off, &att_n = b.att_n;
+  att_off.assign(tile_kinds.size(), 0);
+  att_n.assign(tile_kinds.size(), 0);
   int* att = host<int>(io.att);
   int n_att = 0;
   for (size_t k = 0; k < tile_kinds.size(); ++k) {
@@ -572,9 +835,14 @@ int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* 
   CU(cudaMemcpyAsync(d_io + io.mix, h_io + io.mix, (size_t)n_mix * sizeof(nfn_row_tile), cudaMemcpyHostToDevice, stream));
   if (n_att > 0) CU(cudaMemcpyAsync(d_io + io.att, h_io + io.att, (size_t)n_att * 16, cudaMemcpyHostToDevice, stream));
 
+  CU(cudaMemcpyAsync(d_io + io.seq, h_io + io.seq, (size_t)b.n_seq * sizeof(nfn_seq_rows), cudaMemcpyHostToDevice, stream));
+
+  b.rows = rows;
+  b.short_rows = short_rows;
+  b.n_mix = n_mix;
   const long long before = nfn_launch_count();
   auto body = [&]() -> int {
-    if (pass(rows, short_rows, n_mix, att_off, att_n)) return -1;
+    if (pass(b)) return -1;
     return single ? (head(nullptr, rows) || sample(rows) ? -1 : 0) : 0;
   };
   if (!single || !c.use_cuda_graph) {

@@ -61,7 +61,10 @@ typedef struct {
 // ---- layer-list engine ------------------------------------------------------------------------------
 // A decoder given as a list of layers, each with its own sizes and constants. Layer: h = RMS(x) * norm1; x += mixer(h) + ff(h)
 // (both branches read h; one product adds both to the 32-bit residual stream); then, with side_dim > 0, a per-layer token
-// input: x += RMS(proj(gelu_tanh(gate x) * side_embed[token, layer])) * side_norm. The output norm and the tied head follow.
+// input: x += RMS(proj(gelu_tanh(gate x) * side_embed[token, layer])) * side_norm. The output norm and the head follow.
+// With `chained` set in the configuration mixer and feed-forward are two sublayers, each with a norm of its own, and the residual may be
+// several streams: u = sum_s in[s] x_s, y = sublayer(RMS(u) * norm), x_t <- sum_s mix[s][t] x_s + out[t] y.
+enum { NFN_MIXER_ATTENTION = 0, NFN_MIXER_DELTA = 1 };
 typedef struct {
   int heads, kv_heads;   // query head h reads key / value head h / (heads / kv_heads)
   int dim, vdim;         // per-head query / key size and value size
@@ -75,6 +78,14 @@ typedef struct {
   int out_gate;          // heads *= sigmoid(W_g h)
   int ff;                // width of the gated feed-forward down(act(gate h) * (up h)); 0: none
   int ff_act;            // NFN_ACT_RELU, NFN_ACT_SILU, NFN_ACT_GELU_TANH
+  int mixer;             // NFN_MIXER_*. Delta: gated delta rule with a decay per key channel (nfn_delta_rows); conv_taps >= 1 with SiLU after it
+  int qkv_bias;          // biases on the projected q, k, v
+  int keep_first;        // with a window: the sequence's first keys stay visible
+  float softcap;         // score <- softcap * tanh(score / softcap); 0: off
+  int sink;              // one more score of 0, without a value, in the softmax
+  int rank_decay, rank_gate;   // delta: inner sizes of the decay and output-gate projections
+  int experts, top, expert_ff; // chained: routed experts instead of a dense feed-forward (sigmoid scores, weight on the expert's input)
+  int weights_of;        // >= 0: this layer runs with the tensors of that earlier one (a loop over layers); -1: its own
 } nfn_layer_desc;
 
 typedef struct {
@@ -87,6 +98,12 @@ typedef struct {
   int kv_tokens;         // cache pool: tokens all live sequences hold together, each rounded up to a page (0: max_batch * max_seq)
   int max_step_rows;     // most rows one internal pass runs; longer steps are cut
   int use_cuda_graph;
+  int chained;           // two sublayers per layer
+  int streams;           // residual streams (chained only); 0: one plain residual
+  int untied_head;       // head of its own instead of the embedding table
+  float norm_offset;     // norms multiply by weight + norm_offset
+  float logit_scale;     // logits *= logit_scale
+  float logit_softcap;   // logits <- cap * tanh(logits / cap); 0: off
 } nfn_layered_config;
 
 enum { NFN_KV_PAGE = 64 };   // tokens per cache page

@@ -1,0 +1,189 @@
+// Gated delta rule with a decay per key channel, token after token: single tokens, short portions, and any length in 32-bit mode.
+// (Prompt portions in bf16 take the chunked form of delta_chunk.cu.)
+//
+// The columns of a head's state never meet: S^T k, the correction and the read-out of value column c use S[:, c] only. So a warp owns
+// eight columns of one head for all tokens of its entry - four lanes across, two columns each, eight lanes down the key channels -
+// keeps them in registers from the first token to the last, and needs nothing but shuffles. Everything past the convolved q, k, v is
+// fp32: unit vectors, decays (softplus, exponentials), step sizes, the state.
+#include "common.h"
+#include "delta.cuh"
+
+namespace nfn {
+
+constexpr int DR_WARPS = 4, DR_COLS = 8;
+
+// NR: key channels per lane (dim_p <= 8 NR)
+template <typename T, int NR>
+__global__ void __launch_bounds__(DR_WARPS * 32)
+delta_rows_kernel(const nfn_delta_args p) {
+  extern __shared__ float dr_smem[];                        // [DR_WARPS][3][dim_p]: q, k, g of the token at hand
+  const nfn_seq_rows seq = p.seqs[blockIdx.z];
+  if (seq.slot < 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, rg = lane >> 2, cl = lane & 3;
+  const int h = blockIdx.y, hk = h / (p.heads / p.kv_heads), DP = p.dim_p, VP = p.vdim_p;
+  const int col0 = (blockIdx.x * DR_WARPS + warp) * DR_COLS;
+  if (col0 >= VP) return;
+  const int col = col0 + 2 * cl;
+  float* sq = dr_smem + warp * 3 * DP;
+  float *sk = sq + DP, *sg = sk + DP;
+  float* st = p.state + ((size_t)seq.slot * p.heads + h) * DP * VP + col;
+  float s[NR][2];
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = rg + 8 * i;
+    float2 v = make_float2(0.f, 0.f);
+    if (seq.pos0 > 0 && d < DP) v = *reinterpret_cast<const float2*>(st + (size_t)d * VP);
+    s[i][0] = v.x;
+    s[i][1] = v.y;
+  }
+  const float rate = -expf(__bfloat162float(static_cast<const __nv_bfloat16*>(p.a_log)[h]));
+  const __nv_bfloat16* bias = static_cast<const __nv_bfloat16*>(p.dt_bias) + (size_t)h * DP;
+  const float q_scale = 1.f / sqrtf((float)p.dim);
+  const int off_k = p.kv_heads * DP, off_v = 2 * off_k;
+  for (int t = 0; t < seq.n; ++t) {
+    const size_t row = (size_t)(seq.row0 + t);
+    const T* x = static_cast<const T*>(p.qkv) + row * p.ld_qkv;
+    const float* dec = p.decay + row * p.ld_decay + (size_t)h * DP;
+    float nq = 0.f, nk = 0.f;
+    for (int d = lane; d < DP; d += 32) {
+      const float q = to_float(x[hk * DP + d]), k = to_float(x[off_k + hk * DP + d]);
+      nq += q * q;
+      nk += k * k;
+      sq[d] = q;
+      sk[d] = k;
+      sg[d] = delta_decay(dec[d] + __bfloat162float(bias[d]), rate);
+    }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      nq += __shfl_xor_sync(0xffffffffu, nq, o);
+      nk += __shfl_xor_sync(0xffffffffu, nk, o);
+    }
+    const float fq = q_scale / sqrtf(nq + p.unit_eps), fk = 1.f / sqrtf(nk + p.unit_eps);
+    const float beta = sigmoid_exact(to_float(static_cast<const T*>(p.beta)[row * p.ld_beta + h]));
+    const float v0 = to_float(x[off_v + h * VP + col]), v1 = to_float(x[off_v + h * VP + col + 1]);
+    __syncwarp();
+    float a0 = 0.f, a1 = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int d = rg + 8 * i;
+      if (d < DP) {
+        const float g = sg[d], k = sk[d] * fk;
+        s[i][0] *= g;
+        s[i][1] *= g;
+        a0 += s[i][0] * k;
+        a1 += s[i][1] * k;
+      }
+    }
+#pragma unroll
+    for (int o = 4; o < 32; o <<= 1) {
+      a0 += __shfl_xor_sync(0xffffffffu, a0, o);
+      a1 += __shfl_xor_sync(0xffffffffu, a1, o);
+    }
+    const float u0 = beta * (v0 - a0), u1 = beta * (v1 - a1);
+    float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+      const int d = rg + 8 * i;
+      if (d < DP) {
+        const float k = sk[d] * fk, q = sq[d] * fq;
+        s[i][0] += k * u0;
+        s[i][1] += k * u1;
+        o0 += s[i][0] * q;
+        o1 += s[i][1] * q;
+      }
+    }
+#pragma unroll
+    for (int o = 4; o < 32; o <<= 1) {
+      o0 += __shfl_xor_sync(0xffffffffu, o0, o);
+      o1 += __shfl_xor_sync(0xffffffffu, o1, o);
+    }
+    if (rg == 0) *reinterpret_cast<float2*>(p.o + row * p.ld_o + (size_t)h * VP + col) = make_float2(o0, o1);
+    __syncwarp();
+  }
+#pragma unroll
+  for (int i = 0; i < NR; ++i) {
+    const int d = rg + 8 * i;
+    if (d < DP) *reinterpret_cast<float2*>(st + (size_t)d * VP) = make_float2(s[i][0], s[i][1]);
+  }
+}
+
+// One warp per (row, head): o / rms(o) * weight * sigmoid(gate).
+template <typename T>
+__global__ void __launch_bounds__(256)
+delta_out_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_gate, const __nv_bfloat16* __restrict__ weight, float eps,
+                 T* __restrict__ out, int ld_out, int rows, int heads, int vdim, int vdim_p) {
+  const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
+  const int lane = threadIdx.x & 31;
+  if (item >= (long long)rows * heads) return;
+  const int row = (int)(item / heads), h = (int)(item % heads);
+  const float* src = o + (size_t)row * ld_o + (size_t)h * vdim_p;
+  float ss = 0.f;
+  for (int c = lane * 4; c < vdim_p; c += 128) {
+    const float4 f = load4(src + c);
+    ss += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;
+  }
+#pragma unroll
+  for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  const float r = 1.f / sqrtf(ss / (float)vdim + eps);
+  const T* g = gate + (size_t)row * ld_gate + (size_t)h * vdim_p;
+  T* dst = out + (size_t)row * ld_out + (size_t)h * vdim_p;
+  for (int c = lane * 4; c < vdim_p; c += 128) {
+    const float4 f = load4(src + c), z = load4(g + c), w = load4(weight + c);
+    store4(dst + c, make_float4(f.x * r * w.x * sigmoid_exact(z.x), f.y * r * w.y * sigmoid_exact(z.y), f.z * r * w.z * sigmoid_exact(z.z),
+                                f.w * r * w.w * sigmoid_exact(z.w)));
+  }
+}
+
+template <typename T, int NR>
+static int launch_delta_rows(const nfn_delta_args& a, cudaStream_t st) {
+  const size_t smem = (size_t)DR_WARPS * 3 * a.dim_p * sizeof(float);
+  const dim3 grid(ceil_div(a.vdim_p, DR_WARPS * DR_COLS), a.heads, a.n_seqs);
+  delta_rows_kernel<T, NR><<<grid, DR_WARPS * 32, smem, st>>>(a);
+  return launch_check("delta_rows");
+}
+
+template <typename T>
+static int pick_delta_rows(const nfn_delta_args& a, cudaStream_t st) {
+  if (a.dim_p <= 64) return launch_delta_rows<T, 8>(a, st);
+  if (a.dim_p <= 128) return launch_delta_rows<T, 16>(a, st);
+  if (a.dim_p <= 256) return launch_delta_rows<T, 32>(a, st);
+  return launch_delta_rows<T, 64>(a, st);
+}
+
+const char* delta_args_problem(const nfn_delta_args& a) {
+  if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads) return "delta rule: heads must divide into query / key heads";
+  if (((a.dim_p | a.vdim_p) & 15) || a.dim <= 0 || a.dim > a.dim_p) return "delta rule: head sizes must be padded to multiples of 16";
+  if (a.dim_p > 512) return "delta rule: more than 512 key channels per head";
+  if (a.heads > 65535 || a.n_seqs > 65535) return "delta rule: too many heads or sequences for one launch";
+  if (!a.qkv || !a.beta || !a.decay || !a.a_log || !a.dt_bias || !a.state || !a.o || !a.seqs) return "delta rule: null operand";
+  if ((a.ld_o & 3) || (a.ld_decay & 3) || (a.ld_qkv & 7)) return "delta rule: misaligned rows";
+  return nullptr;
+}
+
+}  // namespace nfn
+
+using namespace nfn;
+
+extern "C" int nfn_delta_rows(const nfn_delta_args* args, nfn_stream_t stream) {
+  if (!args) return fail(-1, "delta rule: null args");
+  if (args->n_seqs <= 0) return 0;
+  if (const char* why = delta_args_problem(*args)) return fail(-1, why);
+  return args->f32 ? pick_delta_rows<float>(*args, static_cast<cudaStream_t>(stream)) : pick_delta_rows<__nv_bfloat16>(*args, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int nfn_delta_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, float eps, void* out, int ld_out, int rows,
+                             int heads, int vdim, int vdim_p, nfn_stream_t stream) {
+  if (rows <= 0) return 0;
+  if ((vdim_p & 15) || vdim <= 0 || vdim > vdim_p || ((ld_o | ld_gate | ld_out) & 7)) return fail(-1, "delta_out: misaligned rows or head sizes");
+  const long long blocks = ((long long)rows * heads + 7) / 8;
+  if (blocks > 0x7fffffffLL) return fail(-1, "delta_out: too many rows for one launch");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(weight);
+  if (f32)
+    delta_out_kernel<float><<<(unsigned)blocks, 256, 0, st>>>(o, ld_o, static_cast<const float*>(gate), ld_gate, w, eps, static_cast<float*>(out), ld_out, rows,
+                                                              heads, vdim, vdim_p);
+  else
+    delta_out_kernel<__nv_bfloat16><<<(unsigned)blocks, 256, 0, st>>>(o, ld_o, static_cast<const __nv_bfloat16*>(gate), ld_gate, w, eps,
+                                                                      static_cast<__nv_bfloat16*>(out), ld_out, rows, heads, vdim, vdim_p);
+  return launch_check("delta_out");
+}

@@ -1,7 +1,7 @@
 // Mixture-of-experts routing around the grouped tcgen05 GEMM (NFN_TP_GROUPED):
 //
 //   route    router logits [T, E] (fp32) -> softmax (or sigmoid) scores -> top-k experts and
-//            weights per token, per-expert token counts (one warp per token, E <= 256, k <= 8);
+//            weights per token, per-expert token counts (one warp per token, E <= 256, k <= 32);
 //   plan     counts -> 128-row-padded expert offsets, the tile -> expert table and the live
 //            tile count the grouped GEMM reads from device memory (no host round trip);
 //   permute  token rows -> expert-sorted, tile-padded buffer; remembers where each
@@ -19,7 +19,7 @@
 
 namespace nfn {
 
-constexpr int MOE_MAX_E = 256, MOE_MAX_K = 8, MOE_TILE = 128;
+constexpr int MOE_MAX_E = 256, MOE_MAX_K = 32, MOE_TILE = 128;
 
 __global__ void __launch_bounds__(256)
 moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, int score_fn, int norm_topk, float route_scale,
@@ -42,7 +42,7 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, 
   for (int i = 0; i < PER; ++i) {
     const int e = i * 32 + lane;
     if (e < E) {
-      v[i] = score_fn == 1 ? 1.f / (1.f + __expf(-v[i])) : __expf(v[i] - mx);
+      v[i] = score_fn == 1 ? 1.f / (1.f + expf(-v[i])) : expf(v[i] - mx);
       sum += v[i];
     } else {
       v[i] = -1.f;  // scores are >= 0: never selected
@@ -51,9 +51,8 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, 
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
   const float inv = score_fn == 1 ? 1.f : 1.f / sum;
-  float wsel[MOE_MAX_K];
-  int isel[MOE_MAX_K];
-  float wsum = 0.f;
+  float wsel = 0.f, wsum = 0.f;      // lane j keeps choice j
+  int isel = 0;
   for (int j = 0; j < k; ++j) {
     float best = -1.f;
     int bi = 0x7fffffff;
@@ -68,20 +67,20 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, 
       const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
       if (ob > best || (ob == best && oi < bi)) { best = ob; bi = oi; }
     }
-    wsel[j] = best * inv;
-    isel[j] = bi;
-    wsum += wsel[j];
+    if (lane == j) {
+      wsel = best * inv;
+      isel = bi;
+    }
+    wsum += best * inv;
 #pragma unroll
     for (int i = 0; i < PER; ++i)
       if (i * 32 + lane == bi) v[i] = -1.f;
   }
-  if (lane == 0) {
+  if (lane < k) {
     const float norm = (norm_topk && wsum > 0.f) ? route_scale / wsum : route_scale;
-    for (int j = 0; j < k; ++j) {
-      topk_idx[(long long)tok * k + j] = isel[j];
-      topk_w[(long long)tok * k + j] = wsel[j] * norm;
-      atomicAdd(&counts[isel[j]], 1);
-    }
+    topk_idx[(long long)tok * k + lane] = isel;
+    topk_w[(long long)tok * k + lane] = wsel * norm;
+    atomicAdd(&counts[isel], 1);
   }
 }
 
@@ -112,7 +111,7 @@ __global__ void moe_plan_kernel(const int* __restrict__ counts, int E, int max_t
 __global__ void __launch_bounds__(256)
 moe_permute_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int T, int k, int d, const int* __restrict__ topk_idx,
                    const int* __restrict__ offsets, int* __restrict__ cursor, int capacity_rows, __nv_bfloat16* __restrict__ xs,
-                   int* __restrict__ row_of) {
+                   int* __restrict__ row_of, const float* __restrict__ topk_w, float* __restrict__ row_w) {
   const long long item = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (item >= (long long)T * k) return;
@@ -123,6 +122,7 @@ moe_permute_kernel(const __nv_bfloat16* __restrict__ x, int ldx, int T, int k, i
     row = offsets[e] + atomicAdd(&cursor[e], 1);
     if (row >= capacity_rows) row = -1;  // cannot happen with a worst-case buffer; dropped if it does
     row_of[item] = row;
+    if (row_w && row >= 0) row_w[row] = topk_w[item];
   }
   row = __shfl_sync(0xffffffffu, row, 0);
   if (row < 0) return;
@@ -169,7 +169,7 @@ extern "C" int nfn_moe_route(const float* logits, int ld, int T, int E, int k, i
                              int* topk_idx, float* topk_w, int* counts, nfn_stream_t stream) {
   if (T <= 0) return 0;
   if (!logits || !topk_idx || !topk_w || !counts) return fail(-1, "moe_route: null operand");
-  if (E <= 0 || E > MOE_MAX_E || k <= 0 || k > MOE_MAX_K || k > E || ld < E) return fail(-1, "moe_route: need 1 <= k <= 8, k <= E <= 256, ld >= E");
+  if (E <= 0 || E > MOE_MAX_E || k <= 0 || k > MOE_MAX_K || k > E || ld < E) return fail(-1, "moe_route: need 1 <= k <= 32, k <= E <= 256, ld >= E");
   moe_route_kernel<<<(T + 7) / 8, 256, 0, static_cast<cudaStream_t>(stream)>>>(logits, ld, T, E, k, score_fn, norm_topk, route_scale, topk_idx,
                                                                                topk_w, counts);
   return launch_check("moe_route", 1);
@@ -183,15 +183,22 @@ extern "C" int nfn_moe_plan(const int* counts, int E, int max_tiles, int* offset
   return launch_check("moe_plan", 1);
 }
 
-extern "C" int nfn_moe_permute(const void* x, int ldx, int T, int k, int d, const int* topk_idx, const int* offsets, int* cursor,
-                               int capacity_rows, void* xs, int* row_of, nfn_stream_t stream) {
+// row_w (optional, with topk_w): the routing weight of every sorted row.
+extern "C" int nfn_moe_permute_weighted(const void* x, int ldx, int T, int k, int d, const int* topk_idx, const float* topk_w, const int* offsets, int* cursor,
+                                        int capacity_rows, void* xs, int* row_of, float* row_w, nfn_stream_t stream) {
   if (T <= 0) return 0;
   if (!x || !topk_idx || !offsets || !cursor || !xs || !row_of || (d & 7) || (ldx & 7) || ldx < d || capacity_rows <= 0) return fail(-1, "moe_permute: bad arguments");
   const long long items = (long long)T * k, grid = (items + 7) / 8;
   if (grid > 0x7fffffffLL) return fail(-1, "moe_permute: too many rows for one launch");
   moe_permute_kernel<<<(unsigned)grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(
-      static_cast<const __nv_bfloat16*>(x), ldx, T, k, d, topk_idx, offsets, cursor, capacity_rows, static_cast<__nv_bfloat16*>(xs), row_of);
+      static_cast<const __nv_bfloat16*>(x), ldx, T, k, d, topk_idx, offsets, cursor, capacity_rows, static_cast<__nv_bfloat16*>(xs), row_of, topk_w,
+      topk_w ? row_w : nullptr);
   return launch_check("moe_permute", 1);
+}
+
+extern "C" int nfn_moe_permute(const void* x, int ldx, int T, int k, int d, const int* topk_idx, const int* offsets, int* cursor, int capacity_rows,
+                               void* xs, int* row_of, nfn_stream_t stream) {
+  return nfn_moe_permute_weighted(x, ldx, T, k, d, topk_idx, nullptr, offsets, cursor, capacity_rows, xs, row_of, nullptr, stream);
 }
 
 extern "C" int nfn_moe_combine(const void* ys, int d, int T, int k, const int* row_of, const float* topk_w, const void* resid,

@@ -329,6 +329,7 @@ typedef struct {
   const void* in; int ld_in;
   int nq, nk, nv, off_gate, off_up, ff, act;
   const void* conv; int taps;
+  int conv_act;                           // NFN_ACT_NONE or NFN_ACT_SILU on the convolved values
   void* state; long long state_half;      // [2][slots][taps - 1][nq + nk + nv]; elements between the halves
   void* q_out; int ld_q;
   void* k_pool; void* v_pool; int kv_heads, dim_p, vdim_p;
@@ -340,8 +341,9 @@ typedef struct {
   int rows;                               // rows of the call
 } nfn_mix_args;
 int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream);
-// Attention of a step's rows over the pages. score = q . k * scale - slopes[h] * (i - j), keys 0 <= i - j < window (0: all),
-// softmax, out = P V * sigmoid(gate) (gate optional). q: [rows, heads * dim_p]; out: row pitch ld_o, head pitch vdim_p.
+// Attention of a step's rows over the pages. score = q . k * scale, capped to softcap * tanh(score / softcap) (0: off), minus
+// slopes[h] * (i - j); keys 0 <= i - j < window (0: all) and the first keep_first ones of the sequence; softmax, with sink != 0 over
+// one more score of 0 that has no value; out = P V * sigmoid(gate) (gate optional). q: [rows, heads * dim_p]; out: row pitch ld_o, head pitch vdim_p.
 typedef struct {
   int f32;
   const void* q; int ld_q;
@@ -358,6 +360,7 @@ typedef struct {
   void* workspace; long long workspace_bytes;   // split partials; the first 64 KB are counters, zeroed once
   const int* tiles; int n_tiles;          // nfn_paged_attention_tiles: {row0, rows, slot, pos0} each
   int total_rows;                         // rows of the q buffer
+  int keep_first; float softcap; int sink;
 } nfn_paged_attention_args;
 // One query row at a time (single tokens, very short portions): bf16 goes to the tensor cores in 32-key steps, fp32 and sizes
 // outside its limits to the plain kernel.
@@ -370,8 +373,77 @@ int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, nfn_stream_t
 // out = gelu_tanh(gate) * side_embed[token][col0 + c]: gate fp32 [rows, ld], out bf16 / fp32 with the same pitch.
 int nfn_side_mul(int f32, const float* gate, const int* tokens, const void* side_embed, long long ld_embed, int col0, int vocab, void* out,
                  int ld, int rows, int width, nfn_stream_t stream);
-// C[M, N] (fp32) (+)= A[M, K] (fp32) . B[N, K]^T (bf16), true 32-bit arithmetic. K, leading dimensions multiples of 4.
-int nfn_gemm_f32(const float* a, int lda, const void* b, int ldb, float* c, int ldc, int m, int n, int k, int accumulate, nfn_stream_t stream);
+// C[M, N] (fp32) (+)= A[M, K] (fp32) . B[N, K]^T (bf16) + bias[N] (bf16, optional), true 32-bit arithmetic. K, leading dimensions
+// multiples of 4.
+int nfn_gemm_f32(const float* a, int lda, const void* b, int ldb, float* c, int ldc, int m, int n, int k, int accumulate, const void* bias,
+                 nfn_stream_t stream);
+// logits <- cap * tanh(scale * logits / cap) (cap = 0: scale only) on fp32 rows.
+int nfn_logit_cap(float* logits, int ld, int rows, int cols, float scale, float cap, nfn_stream_t stream);
+
+// ---- residual streams (stream_rows.cu) -------------------------------------------------------------------------------------
+// A row's residual is `streams` fp32 rows of pitch ld, x [rows][streams][ld]. One pass finishes a sublayer and starts the next:
+// all streams at once, x_t <- sum_s mix[s][t] x_s + out[t] y (mix, out: bf16; NULL: identity, ones; y = NULL: no update), then
+// u = sum_s in[s] x_s (in: bf16; NULL: ones) and h = u / rms(u) * (weight + weight_offset), rms(z) = sqrt(sum z^2 / width + eps).
+// The base is embed[token] * embed_scale in every stream (tokens != NULL) or row src_rows[r] (NULL: r) of x; y is the row of the
+// same number, or with y_rows > 1 the sum of rows y_index[r * y_rows + j] (y_index NULL: r * y_rows + j).
+enum { NFN_MAX_STREAMS = 16 };
+typedef struct {
+  int f32, rows, width, ld, streams;
+  const float* x; float* x_out; const int* src_rows;
+  const int* tokens; const void* embed; float embed_scale; int vocab;
+  const void* y; int y_rows; const int* y_index;
+  const void* mix; const void* out;
+  const void* in; void* h; const void* weight;
+  float eps, weight_offset;
+} nfn_stream_args;
+int nfn_stream_pass(const nfn_stream_args* args, nfn_stream_t stream);
+
+// ---- gated delta rule with a decay per key channel (delta_rows.cu, delta_chunk.cu) -------------------------------------------
+// Per head (query / key head h / (heads / kv_heads)), with the fp32 state S [dim][vdim] of the sequence:
+//   q, k made unit vectors, z / sqrt(sum z^2 + unit_eps), q also times dim^-1/2;  g = exp(-exp(a_log_h) softplus(decay + dt_bias)) per channel;
+//   S <- g * S;  u = sigmoid(beta) (v - S^T k);  S <- S + k u^T;  o = S^T q.
+// qkv: rows [q: kv_heads * dim_p | k | v: heads * vdim_p] after convolution and activation; state [slots][heads][dim_p][vdim_p]; a
+// sequence at position 0 starts from zero whatever the slot holds. o: fp32 rows of heads * vdim_p. Padded channels are zero in q, k, v.
+typedef struct { int row0, n, slot, pos0; } nfn_seq_rows;   // slot < 0: skipped
+typedef struct {
+  int f32;
+  const void* qkv; int ld_qkv;
+  const void* beta; int ld_beta;          // projected, before the sigmoid
+  const float* decay; int ld_decay;       // [rows][heads * dim_p]
+  const void* a_log; const void* dt_bias; // bf16 [heads], [heads * dim_p]
+  int heads, kv_heads, dim, dim_p, vdim_p;
+  float unit_eps;
+  float* state;
+  float* o; int ld_o;
+  const nfn_seq_rows* seqs; int n_seqs;
+} nfn_delta_args;
+int nfn_delta_rows(const nfn_delta_args* args, nfn_stream_t stream);     // token after token, any length
+// out = o / rms(o) * weight * sigmoid(gate) per head of vdim values (pitch vdim_p); weight bf16 [vdim_p], out and gate in the activation type.
+int nfn_delta_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, float eps, void* out, int ld_out, int rows,
+                  int heads, int vdim, int vdim_p, nfn_stream_t stream);
+
+// ---- mixture of experts for the rows of a step (moe.cu, moe_rows.cu) ----------------------------------------------------------
+// item i = token i / top, choice i % top. The routing weight multiplies the expert's INPUT: mid = act(w G h) * (w U h).
+int nfn_moe_route(const float* logits, int ld, int T, int E, int k, int score_fn, int norm_topk, float route_scale, int* topk_idx, float* topk_w,
+                  int* counts, nfn_stream_t stream);
+int nfn_moe_plan(const int* counts, int E, int max_tiles, int* offsets, int* cursor, int* tile_expert, int* plan, nfn_stream_t stream);
+// nfn_moe_permute that also leaves each sorted row's routing weight in row_w.
+int nfn_moe_permute_weighted(const void* x, int ldx, int T, int k, int d, const int* topk_idx, const float* topk_w, const int* offsets, int* cursor,
+                             int capacity_rows, void* xs, int* row_of, float* row_w, nfn_stream_t stream);
+// mid[r] = act(w G) * (w U) over the first plan[1] rows of gate_up [rows][2 * ff] (bf16), w = row_w[r].
+int nfn_moe_act_rows(const void* gate_up, const float* row_w, const int* plan, int capacity_rows, int ff, int act, void* mid, nfn_stream_t stream);
+// Few rows: routing and a list of items per expert in one launch (order: items by expert; offsets: experts + 1; active: experts with items,
+// active[experts] their number), then the products of the chosen experts only, item by item. w_gate_up [E][2 ff][width], w_down [E][width][ff].
+typedef struct {
+  int f32, rows, width, ff, experts, top, act;
+  const float* logits; int ld_logits;
+  const void* h; int ld_h;
+  const void* w_gate_up; const void* w_down;
+  int* idx; float* weight; int* order; int* offsets; int* active;
+  void* mid;                              // [rows * top][ff]
+  void* y; int ld_y;                      // [rows * top][ld_y]
+} nfn_moe_rows_args;
+int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream);
 
 #ifdef __cplusplus
 }

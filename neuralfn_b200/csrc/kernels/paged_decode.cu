@@ -60,8 +60,11 @@ paged_decode_kernel(const PagedDecodeParams p) {
   const int hg = a.heads / a.kv_heads, h_lo = hb * NH, n_heads = min(NH, hg - h_lo), h0 = hk * hg + h_lo;
   const int pos = a.row_pos[row];
   const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  const int c_first = lo / PD_KEYS, n_chunks = pos / PD_KEYS + 1 - c_first;
-  const int c_lo = c_first + (int)((long long)n_chunks * blockIdx.x / p.splits), c_hi = c_first + (int)((long long)n_chunks * (blockIdx.x + 1) / p.splits);
+  // chunks in the order kept tokens, window: number i of them is chunk i of the sequence, or c_first + i - n_keep
+  const int keep = min(a.keep_first, pos + 1);
+  const int c_first = lo / PD_KEYS, n_keep = min(c_first, (keep + PD_KEYS - 1) / PD_KEYS), n_chunks = n_keep + pos / PD_KEYS + 1 - c_first;
+  const int c_lo = (int)((long long)n_chunks * blockIdx.x / p.splits), c_hi = (int)((long long)n_chunks * (blockIdx.x + 1) / p.splits);
+  auto chunk_base = [&](int i) { return (i < n_keep ? i : c_first + i - n_keep) * PD_KEYS; };
   const int DP = a.dim_p, VP = a.vdim_p;
   const int* table = a.table + (size_t)slot * a.table_ld;
   const __nv_bfloat16* kp = static_cast<const __nv_bfloat16*>(a.k_pool);
@@ -80,6 +83,8 @@ paged_decode_kernel(const PagedDecodeParams p) {
   // this lane's two heads per tile: columns 2 j, 2 j + 1
   const float LOG2E = 1.4426950408889634f;
   const float mul = a.scale * LOG2E;
+  // cap tanh(s / cap) = cap (1 - 2 / (1 + e^(2 s / cap)))
+  const float cap = a.softcap * LOG2E, cap_in = a.softcap > 0.f ? 2.f * mul / a.softcap : 0.f;
   float slope[NT][2], m[NT][2], l[NT][2];
   float acc[VT][NT][4];
 #pragma unroll
@@ -102,7 +107,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
   const int key0 = 8 * (g >> 1) + (g & 1);
   uint4 kf[2][2][DC];                                       // key fragments of the chunk at hand: [tile][row g, row g + 8]
   auto load_keys = [&](int c) {
-    const int base = c * PD_KEYS, in_page = base % NFN_PAGE;
+    const int base = chunk_base(c), in_page = base % NFN_PAGE;
     const size_t tile = (size_t)table[base / NFN_PAGE] * a.kv_heads + hk;
     const __nv_bfloat16* krow = kp + (tile * NFN_PAGE + in_page + key0) * DP + 8 * j;
 #pragma unroll
@@ -115,7 +120,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
   };
   if (c_lo + warp < c_hi) load_keys(c_lo + warp);
   for (int c = c_lo + warp; c < c_hi; c += PD_WARPS) {
-    const int base = c * PD_KEYS, in_page = base % NFN_PAGE;
+    const int base = chunk_base(c), in_page = base % NFN_PAGE;
     const size_t tile = (size_t)table[base / NFN_PAGE] * a.kv_heads + hk;
     // this chunk's values are on their way while the scores are formed, the next chunk's keys while these are used
     constexpr int VF = (NT == 1 && VT <= 8) ? VT : 2;                    // value tiles held ahead
@@ -153,13 +158,14 @@ paged_decode_kernel(const PagedDecodeParams p) {
 #pragma unroll
       for (int half = 0; half < 2; ++half) {
         const int dist = rel - 4 * t - 2 * half;
-        const bool seen = dist >= 0 && pos - dist >= lo;
+        const bool seen = dist >= 0 && (pos - dist >= lo || pos - dist < keep);
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
             float& x = s[t][nt][2 * half + e];
-            x = seen ? x * mul - slope[nt][e] * (float)dist : -INFINITY;
+            const float y = cap > 0.f ? cap * (1.f - __fdividef(2.f, 1.f + exp2f(x * cap_in))) : x * mul;
+            x = seen ? y - slope[nt][e] * (float)dist : -INFINITY;
           }
       }
     uint32_t b[2][NT][2];
@@ -245,7 +251,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
   float* part = p.partial + (cell * p.splits + blockIdx.x) * NH * (VP + 2);
   for (int i = threadIdx.x; i < n_heads * VP; i += PD_THREADS) {
     const int h = i / VP, ch = i % VP;
-    float mx = -INFINITY;
+    float mx = p.splits == 1 && a.sink ? 0.f : -INFINITY;
 #pragma unroll
     for (int w = 0; w < PD_WARPS; ++w) mx = fmaxf(mx, sm[w * NH + h]);
     float o = 0.f, sum = 0.f;
@@ -258,6 +264,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
       }
     }
     if (p.splits == 1) {
+      if (a.sink) sum += exp2f(-mx);
       finish(h, ch, o / sum);
     } else {
       part[(size_t)h * (VP + 2) + ch] = o;
@@ -278,7 +285,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
   const float* all = p.partial + cell * p.splits * NH * (VP + 2);
   for (int i = threadIdx.x; i < n_heads * VP; i += PD_THREADS) {
     const int h = i / VP, ch = i % VP;
-    float mx = -INFINITY;
+    float mx = a.sink ? 0.f : -INFINITY;
     for (int s2 = 0; s2 < p.splits; ++s2) mx = fmaxf(mx, __ldcg(&all[((size_t)s2 * NH + h) * (VP + 2) + VP]));
     float o = 0.f, sum = 0.f;
     for (int s2 = 0; s2 < p.splits; ++s2) {
@@ -287,6 +294,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
       o += f * __ldcg(q + ch);
       sum += f * __ldcg(q + VP + 1);
     }
+    if (a.sink) sum += exp2f(-mx);
     finish(h, ch, o / sum);
   }
   if (threadIdx.x == 0) p.counters[cell] = 0;

@@ -65,7 +65,10 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   const int hk = blockIdx.y;
   const int* table = a.table + (size_t)slot * a.table_ld;
   const int k_lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
-  const int jb_hi = (pos0 + n_rows - 1) / PP_BN, nblk = jb_hi + 1 - k_lo / PP_BN;   // visited from the newest page back
+  // visited from the newest page back to the window's edge, then the pages of the kept first tokens that lie before it
+  const int jb_hi = (pos0 + n_rows - 1) / PP_BN, n_win = jb_hi + 1 - k_lo / PP_BN;
+  const int n_keep = min(k_lo / PP_BN, (a.keep_first + PP_BN - 1) / PP_BN), nblk = n_win + n_keep;
+  auto page_at = [&](int j) { return j < n_win ? jb_hi - j : n_keep - 1 - (j - n_win); };
 
   if (threadIdx.x == 0) {
     *cta_abort = 0;
@@ -97,14 +100,14 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       auto load_k = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_k[stage]);
         const uint32_t sk = smem_u32(sKV + stage * kv_stage);
-        const int r = (table[jb_hi - j] * a.kv_heads + hk) * PP_BN;
+        const int r = (table[page_at(j)] * a.kv_heads + hk) * PP_BN;
         mbar_expect_tx(fb, p.k_bytes);
         for (int d = 0; d < p.panels; ++d) tma_load_2d(sk + d * (PP_BN * 128), &tm_k, fb, d * 64, r);
       };
       auto load_v = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_v[stage]);
         mbar_expect_tx(fb, p.v_bytes);
-        tma_load_2d(smem_u32(sKV + stage * kv_stage + p.k_bytes), &tm_v, fb, 0, (table[jb_hi - j] * a.kv_heads + hk) * a.vdim_p);
+        tma_load_2d(smem_u32(sKV + stage * kv_stage + p.k_bytes), &tm_v, fb, 0, (table[page_at(j)] * a.kv_heads + hk) * a.vdim_p);
       };
       mbar_expect_tx(smem_u32(bar_q), p.q_tx);
       for (int d = 0; d < p.panels; ++d) tma_load_3d(smem_u32(sQ) + d * (PP_BM * 128), &tm_q, smem_u32(bar_q), d * 64, hk * p.hg, row0);
@@ -171,12 +174,14 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     const uint32_t t_row = tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
     const float LOG2E = 1.4426950408889634f;
     const float c_mul = a.scale * LOG2E;
+    const float cap = a.softcap * LOG2E, cap_in = a.softcap > 0.f ? 2.f * c_mul / a.softcap : 0.f;
     const float slope = (a.slopes && row_ok) ? a.slopes[h] * LOG2E : 0.f;
     // visible keys of this row: [v_lo, v_hi)
     const int v_hi = row_ok ? pos + 1 : 0;
     const int v_lo = (row_ok && a.window > 0) ? max(0, pos - a.window + 1) : 0;
     const int pos_last = pos0 + n_rows - 1;
-    float m_run = -INFINITY, l_run = 0.f;  // units of log2
+    const int v_keep = min(a.keep_first, v_hi);
+    float m_run = a.sink ? 0.f : -INFINITY, l_run = a.sink ? 1.f : 0.f;  // units of log2; the sink counts as seen before all keys
     bool ok = true;
     for (int j = 0; j < nblk; ++j) {
       ok = mbar_wait_bounded(smem_u32(bar_s), j & 1, cta_abort, p.status, 0x600 + 9);
@@ -190,22 +195,34 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(bar_sfree));
 
-      const int kbase = (jb_hi - j) * PP_BN;
+      const int kbase = page_at(j) * PP_BN;
+      float mul = c_mul;
+      if (a.softcap > 0.f) {
+        // cap tanh(x) = cap (1 - 2 / (1 + e^(2x))), two scores per reciprocal
+#pragma unroll
+        for (int i = 0; i < PP_BN; i += 2) {
+          const float e0 = 1.f + fast_exp2(fminf(__uint_as_float(s[i]) * cap_in, 60.f)), e1 = 1.f + fast_exp2(fminf(__uint_as_float(s[i + 1]) * cap_in, 60.f));
+          const float r2 = cap * -2.f * fast_rcp(e0 * e1);
+          s[i] = __float_as_uint(fmaf(r2, e1, cap));
+          s[i + 1] = __float_as_uint(fmaf(r2, e0, cap));
+        }
+        mul = 1.f;
+      }
       const float b0 = slope * (float)(kbase - pos);
 #pragma unroll
       for (int i = 0; i < PP_BN; i += 2) {
         float t0, t1, y0, y1;
         fma2_bcast(t0, t1, (float)i, (float)(i + 1), slope, b0);
-        fma2(y0, y1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]), c_mul, c_mul, t0, t1);
+        fma2(y0, y1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]), mul, mul, t0, t1);
         s[i] = __float_as_uint(y0);
         s[i + 1] = __float_as_uint(y1);
       }
       if (kbase + PP_BN - 1 > pos0 || (a.window > 0 && kbase <= pos_last - a.window)) {
-        const int lo_rel = v_lo - kbase;
+        const int lo_rel = v_lo - kbase, keep_rel = v_keep - kbase;
         const unsigned span = (unsigned)max(0, v_hi - v_lo);
 #pragma unroll
         for (int i = 0; i < PP_BN; ++i)
-          if ((unsigned)(i - lo_rel) >= span) s[i] = 0xff800000u;  // -inf
+          if ((unsigned)(i - lo_rel) >= span && i >= keep_rel) s[i] = 0xff800000u;  // -inf
       }
       float mx0 = -INFINITY, mx1 = -INFINITY, mx2 = -INFINITY, mx3 = -INFINITY;
 #pragma unroll

@@ -213,6 +213,10 @@ mix_rows_kernel(const nfn_mix_args p) {
 #pragma unroll
       for (int i = 0; i < N; ++i)
         if (i0 + i < t.n) {
+          if (p.conv_act == NFN_ACT_SILU) {
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[i][e] = v[i][e] / (1.f + expf(-v[i][e]));
+          }
           if (p.temp_every > 0) {
             const int pos = t.e_pos0 + ti0 + i0 + i;
             const float f = 1.f + p.temp_coef * logf((float)((pos + 1) / p.temp_every + 1));
@@ -334,24 +338,28 @@ paged_attention_plain_kernel(const nfn_paged_attention_args p) {
   __syncwarp();
   const float slope = p.slopes ? p.slopes[h] : 0.f;
   const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int keep = min(p.keep_first, pos + 1);
   const int* table = p.table + (size_t)slot * p.table_ld;
   const int nvec = (p.vdim_p + 31) / 32;
   float acc[PLAIN_MAX_VEC];
 #pragma unroll
   for (int i = 0; i < PLAIN_MAX_VEC; ++i) acc[i] = 0.f;
-  float m = -INFINITY, l = 0.f;
-  for (int base = lo / 32 * 32; base <= pos; base += 32) {   // a chunk never crosses a page
+  float m = p.sink ? 0.f : -INFINITY, l = p.sink ? 1.f : 0.f;      // the sink is an element seen before all others
+  for (int base = keep > 0 ? 0 : lo / 32 * 32; base <= pos; base += 32) {   // a chunk never crosses a page
+    if (base >= keep && base + 32 <= lo) base = lo / 32 * 32;      // from the kept tokens to the window
     const size_t tile = (size_t)table[base / NFN_PAGE] * p.kv_heads + hk;
     const int in_page = base % NFN_PAGE, j = base + lane;
     float s = -INFINITY;
-    if (j >= lo && j <= pos) {
+    if ((j >= lo || j < keep) && j <= pos) {
       const T* k = static_cast<const T*>(p.k_pool) + (tile * NFN_PAGE + in_page + lane) * p.dim_p;
       float d0 = 0.f, d1 = 0.f, d2 = 0.f, d3 = 0.f;
       for (int d = 0; d < p.dim_p; d += 4) {
         const float4 kv = load4(k + d);
         d0 += kv.x * q[d]; d1 += kv.y * q[d + 1]; d2 += kv.z * q[d + 2]; d3 += kv.w * q[d + 3];
       }
-      s = ((d0 + d1) + (d2 + d3)) * p.scale - slope * (float)(pos - j);
+      s = ((d0 + d1) + (d2 + d3)) * p.scale;
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      s -= slope * (float)(pos - j);
     }
     float mx = s;
 #pragma unroll
@@ -428,7 +436,7 @@ constexpr int SG_BM = 64, SG_BN = 64, SG_BK = 16;
 
 __global__ void __launch_bounds__(256)
 gemm_f32_kernel(const float* __restrict__ a, int lda, const __nv_bfloat16* __restrict__ b, int ldb, float* c, int ldc, int m, int n, int k,
-                int accumulate) {
+                int accumulate, const __nv_bfloat16* __restrict__ bias) {
   __shared__ float sa[SG_BK][SG_BM + 4], sb[SG_BK][SG_BN + 4];
   const int m0 = blockIdx.y * SG_BM, n0 = blockIdx.x * SG_BN;
   const int tx = threadIdx.x & 15, ty = threadIdx.x >> 4;
@@ -463,15 +471,36 @@ gemm_f32_kernel(const float* __restrict__ a, int lda, const __nv_bfloat16* __res
       const int col = n0 + tx * 4 + j;
       if (col < n) {
         float* cp = c + (size_t)r * ldc + col;
-        *cp = accumulate ? *cp + acc[i][j] : acc[i][j];
+        const float v = acc[i][j] + (bias ? __bfloat162float(bias[col]) : 0.f);
+        *cp = accumulate ? *cp + v : v;
       }
     }
   }
 }
 
+__global__ void logit_cap_kernel(float* logits, int ld, int rows, int vecs, float scale, float cap) {
+  const int i = blockIdx.x * blockDim.x + threadIdx.x;
+  if (i >= rows * vecs) return;
+  float* p = logits + (size_t)(i / vecs) * ld + (i % vecs) * 4;
+  const float4 f = load4(p);
+  float v[4] = {f.x, f.y, f.z, f.w};
+#pragma unroll
+  for (float& x : v) x = cap > 0.f ? cap * tanhf(x * scale / cap) : x * scale;
+  store4(p, make_float4(v[0], v[1], v[2], v[3]));
+}
+
 }  // namespace nfn
 
 using namespace nfn;
+
+extern "C" int nfn_logit_cap(float* logits, int ld, int rows, int cols, float scale, float cap, nfn_stream_t stream) {
+  if (rows <= 0) return 0;
+  if ((ld | cols) & 3) return fail(-1, "logit_cap: widths must be multiples of 4");
+  const int vecs = cols / 4;
+  if ((long long)rows * vecs > 0x7fffff00LL) return fail(-1, "logit_cap: too many values for one launch");
+  logit_cap_kernel<<<ceil_div(rows * vecs, 256), 256, 0, static_cast<cudaStream_t>(stream)>>>(logits, ld, rows, vecs, scale, cap);
+  return launch_check("logit_cap");
+}
 
 extern "C" int nfn_row_norm(const nfn_row_norm_args* args, nfn_stream_t stream) {
   if (!args) return fail(-1, "row_norm: null args");
@@ -499,6 +528,7 @@ extern "C" int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream) {
   if (a.n_tiles <= 0) return 0;
   if ((a.nq | a.nk | a.nv | a.ff | a.ld_in | a.ld_q | a.ld_ff | a.off_gate | a.off_up | a.dim_p | a.vdim_p) & 7)
     return fail(-1, "mix_rows: widths and offsets must be multiples of 8");
+  if (a.conv_act != NFN_ACT_NONE && (a.conv_act != NFN_ACT_SILU || a.nk || a.nv)) return fail(-1, "mix_rows: the activation (SiLU) goes with rows that stay out of the cache");
   if ((a.taps > 0) != (a.conv != nullptr) || (a.taps > 1 && !a.state)) return fail(-1, "mix_rows: a convolution needs its weights and history");
   if (a.n_tiles > 65535) return fail(-1, "mix_rows: too many row tiles in one launch");
   if (a.tile_rows < 1 || a.tile_rows > MIX_ROWS) return fail(-1, "mix_rows: tiles hold 1 to 16 rows");
@@ -530,10 +560,11 @@ extern "C" int nfn_side_mul(int f32, const float* gate, const int* tokens, const
 }
 
 extern "C" int nfn_gemm_f32(const float* a, int lda, const void* b, int ldb, float* c, int ldc, int m, int n, int k, int accumulate,
-                            nfn_stream_t stream) {
+                            const void* bias, nfn_stream_t stream) {
   if (m <= 0 || n <= 0 || k <= 0) return fail(-1, "gemm_f32: empty problem");
   if ((lda | ldb | k) & 3) return fail(-1, "gemm_f32: K and the leading dimensions must be multiples of 4");
   const dim3 grid(ceil_div(n, SG_BN), ceil_div(m, SG_BM));
-  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(a, lda, static_cast<const __nv_bfloat16*>(b), ldb, c, ldc, m, n, k, accumulate);
+  gemm_f32_kernel<<<grid, 256, 0, static_cast<cudaStream_t>(stream)>>>(a, lda, static_cast<const __nv_bfloat16*>(b), ldb, c, ldc, m, n, k, accumulate,
+                                                                        static_cast<const __nv_bfloat16*>(bias));
   return launch_check("gemm_f32");
 }

@@ -14,32 +14,14 @@ from typing import Any, Mapping
 import torch
 
 from ..serving.engine import LayeredEngineConfig, LayerSpec
+from .layered_common import ModelConfigError, check_tensors, known, need, pad_cols, pad_rows, positive_int, up
 
 __all__ = ["BulidraConfig", "BulidraError", "engine_config", "expected_shapes", "pack_tensors", "random_tensors"]
 
 _ALIBI = 8.0     # slope of head h (from 0): 2^(-8 (h + 1) / heads)
 
 
-class BulidraError(ValueError):
-    pass
-
-
-def _need(d: Mapping, key: str, where: str):
-    if key not in d:
-        raise BulidraError(f"{where}: {key} is missing")
-    return d[key]
-
-
-def _int(v, where: str, low: int = 1) -> int:
-    if isinstance(v, bool) or int(v) != v or int(v) < low:
-        raise BulidraError(f"{where}: expected an integer >= {low}, got {v!r}")
-    return int(v)
-
-
-def _known(d: Mapping, keys: set[str], where: str) -> None:
-    extra = set(d) - keys
-    if extra:
-        raise BulidraError(f"{where}: unknown settings {sorted(extra)}")
+BulidraError = ModelConfigError
 
 
 @dataclass(frozen=True)
@@ -69,37 +51,37 @@ class BulidraConfig:
     @classmethod
     def from_dict(cls, raw: Mapping[str, Any]) -> "BulidraConfig":
         layers = []
-        for i, entry in enumerate(_need(raw, "layers", "config")):
+        for i, entry in enumerate(need(raw, "layers", "config")):
             where = f"layer {i}"
-            if _need(entry, "type", where) != "attention":
+            if need(entry, "type", where) != "attention":
                 raise BulidraError(f"{where}: unknown layer type {entry['type']!r}")
-            m, mlp = _need(entry, "mixer", where), entry.get("mlp")
-            _known(m, {"heads", "kv_heads", "dim", "vdim", "conv", "scale", "mask", "q_temp", "kv_from"}, where)
-            heads, kv_heads = _int(_need(m, "heads", where), where), _int(_need(m, "kv_heads", where), where)
+            m, mlp = need(entry, "mixer", where), entry.get("mlp")
+            known(m, {"heads", "kv_heads", "dim", "vdim", "conv", "scale", "mask", "q_temp", "kv_from"}, where)
+            heads, kv_heads = positive_int(need(m, "heads", where), where), positive_int(need(m, "kv_heads", where), where)
             if heads % kv_heads:
                 raise BulidraError(f"{where}: {heads} query heads do not divide into {kv_heads} key / value heads")
             mask, temp, kv_from = m.get("mask"), m.get("q_temp"), m.get("kv_from")
             if mask is not None:
-                _known(mask, {"size"}, where)
+                known(mask, {"size"}, where)
             if temp is not None:
-                _known(temp, {"coef", "every"}, where)
-            if mlp is not None and _need(mlp, "kind", where) != "dense":
+                known(temp, {"coef", "every"}, where)
+            if mlp is not None and need(mlp, "kind", where) != "dense":
                 raise BulidraError(f"{where}: unknown feed-forward kind {mlp['kind']!r}")
             if kv_from is not None:
-                kv_from = _int(kv_from, where, 0)
+                kv_from = positive_int(kv_from, where, 0)
                 if kv_from >= i or layers[kv_from].kv_from is not None:
                     raise BulidraError(f"{where}: kv_from must name an earlier layer that has keys and values of its own")
             layers.append(BulidraLayer(
-                heads, kv_heads, _int(_need(m, "dim", where), where), _int(_need(m, "vdim", where), where), _int(m.get("conv") or 0, where, 0),
-                float(_need(m, "scale", where)), _int(_need(mask, "size", where), where) if mask is not None else 0,
-                float(_need(temp, "coef", where)) if temp is not None else 0.0, _int(_need(temp, "every", where), where) if temp is not None else 0,
-                kv_from, _int(_need(mlp, "ff", where), where) if mlp is not None else 0))
+                heads, kv_heads, positive_int(need(m, "dim", where), where), positive_int(need(m, "vdim", where), where), positive_int(m.get("conv") or 0, where, 0),
+                float(need(m, "scale", where)), positive_int(need(mask, "size", where), where) if mask is not None else 0,
+                float(need(temp, "coef", where)) if temp is not None else 0.0, positive_int(need(temp, "every", where), where) if temp is not None else 0,
+                kv_from, positive_int(need(mlp, "ff", where), where) if mlp is not None else 0))
         if not layers:
             raise BulidraError("config: no layers")
         side = raw.get("token_side")
-        return cls(_int(_need(raw, "vocab", "config"), "vocab"), _int(_need(raw, "width", "config"), "width"),
-                   float(_need(_need(raw, "embedding", "config"), "scale", "embedding")), float(_need(_need(raw, "norm", "config"), "eps", "norm")),
-                   _int(_need(side, "dim", "token_side"), "token_side") if side else 0, tuple(layers))
+        return cls(positive_int(need(raw, "vocab", "config"), "vocab"), positive_int(need(raw, "width", "config"), "width"),
+                   float(need(need(raw, "embedding", "config"), "scale", "embedding")), float(need(need(raw, "norm", "config"), "eps", "norm")),
+                   positive_int(need(side, "dim", "token_side"), "token_side") if side else 0, tuple(layers))
 
     def to_dict(self) -> dict:
         def layer(y: BulidraLayer) -> dict:
@@ -151,60 +133,39 @@ def engine_config(cfg: BulidraConfig, **kw) -> LayeredEngineConfig:
                                norm_eps=cfg.norm_eps, **kw)
 
 
-def _up(v: int, m: int = 16) -> int:
-    return (v + m - 1) // m * m
-
-
-def _pad_rows(t: torch.Tensor, groups: int, to: int) -> torch.Tensor:
-    """[groups * n, ...] -> [groups * to, ...]: zero rows after each group."""
-    n = t.shape[0] // groups
-    if n == to:
-        return t
-    out = t.new_zeros(groups, to, *t.shape[1:])
-    out[:, :n] = t.reshape(groups, n, *t.shape[1:])
-    return out.reshape(groups * to, *t.shape[1:])
-
-
 def pack_tensors(cfg: BulidraConfig, tensors: Mapping[str, torch.Tensor]) -> dict[str, torch.Tensor]:
     """The model's tensors under the engine's names: one input product [q | k | v | g | gate | up] and one output product [o | down] per
     layer, heads and widths padded with zeros to multiples of 16."""
-    want = expected_shapes(cfg)
-    missing, extra = sorted(set(want) - set(tensors)), sorted(set(tensors) - set(want))
-    if missing or extra:
-        raise BulidraError(f"tensors do not fit the configuration (missing {missing[:4]}, unexpected {extra[:4]})")
-    for n, shape in want.items():
-        if tuple(tensors[n].shape) != shape:
-            raise BulidraError(f"{n}: shape {tuple(tensors[n].shape)} instead of {shape}")
-    T = {n: tensors[n].to(torch.bfloat16) for n in want}
-    wp = _up(cfg.width)
+    T = check_tensors(expected_shapes(cfg), tensors)
+    wp = up(cfg.width)
 
     def cols(t: torch.Tensor) -> torch.Tensor:                   # [rows, width] -> [rows, wp]
-        return _pad_rows(t.T, 1, wp).T if t.shape[1] != wp else t
+        return pad_cols(t, 1, wp)
 
     def vec(n: str) -> torch.Tensor:
-        return _pad_rows(T[n], 1, wp)
+        return pad_rows(T[n], 1, wp)
 
-    out = {"embed": _pad_rows(cols(T["embed"]), 1, _up(cfg.vocab)), "final_norm": vec("final.norm")}
-    sp = _up(cfg.side_dim) if cfg.side_dim else 0
+    out = {"embed": pad_rows(cols(T["embed"]), 1, up(cfg.vocab)), "final_norm": vec("final.norm")}
+    sp = up(cfg.side_dim) if cfg.side_dim else 0
     if sp:
-        out["side_embed"] = _pad_rows(T["side.embed"].T, len(cfg.layers), sp).T.contiguous()
+        out["side_embed"] = pad_rows(T["side.embed"].T, len(cfg.layers), sp).T.contiguous()
     for i, y in enumerate(cfg.layers):
         p, q = f"l{i}.", f"layers.{i}."
-        dp, vp, fp = _up(y.dim), _up(y.vdim), _up(y.ff) if y.ff else 0
+        dp, vp, fp = up(y.dim), up(y.vdim), up(y.ff) if y.ff else 0
         heads = [("q", y.heads, dp)] + ([("k", y.kv_heads, dp), ("v", y.kv_heads, vp)] if y.kv_from is None else [])
-        rows = [_pad_rows(cols(T[p + f"mix.{n}"]), g, to) for n, g, to in heads] + [_pad_rows(cols(T[p + "mix.g"]), y.heads, vp)]
-        o = [_pad_rows(T[p + "mix.o"].T, y.heads, vp)]           # [heads * vp, width]
+        rows = [pad_rows(cols(T[p + f"mix.{n}"]), g, to) for n, g, to in heads] + [pad_rows(cols(T[p + "mix.g"]), y.heads, vp)]
+        o = [pad_rows(T[p + "mix.o"].T, y.heads, vp)]           # [heads * vp, width]
         if y.ff:
-            rows += [_pad_rows(cols(T[p + "mlp.gate"]), 1, fp), _pad_rows(cols(T[p + "mlp.up"]), 1, fp)]
-            o.append(_pad_rows(T[p + "mlp.down"].T, 1, fp))
+            rows += [pad_rows(cols(T[p + "mlp.gate"]), 1, fp), pad_rows(cols(T[p + "mlp.up"]), 1, fp)]
+            o.append(pad_rows(T[p + "mlp.down"].T, 1, fp))
         out[q + "norm1"] = vec(p + "norm1")
         out[q + "w_in"] = torch.cat(rows)
         if y.conv:
-            out[q + "conv"] = torch.cat([_pad_rows(T[p + f"mix.{n}.conv"], g, to) for n, g, to in heads]).T.contiguous()
-        out[q + "w_out"] = _pad_rows(torch.cat(o).T.contiguous(), 1, wp)
+            out[q + "conv"] = torch.cat([pad_rows(T[p + f"mix.{n}.conv"], g, to) for n, g, to in heads]).T.contiguous()
+        out[q + "w_out"] = pad_rows(torch.cat(o).T.contiguous(), 1, wp)
         if sp:
-            out[q + "side_gate"] = _pad_rows(cols(T[p + "side.gate"]), 1, sp)
-            out[q + "side_proj"] = _pad_rows(_pad_rows(T[p + "side.proj"].T, 1, sp).T.contiguous(), 1, wp)
+            out[q + "side_gate"] = pad_rows(cols(T[p + "side.gate"]), 1, sp)
+            out[q + "side_proj"] = pad_rows(pad_rows(T[p + "side.proj"].T, 1, sp).T.contiguous(), 1, wp)
             out[q + "side_norm"] = vec(p + "side.norm")
     return out
 

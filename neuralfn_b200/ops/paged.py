@@ -18,12 +18,13 @@ class _Attention(C.Structure):
                 ("dim_p", C.c_int), ("vdim_p", C.c_int), ("pages", C.c_longlong), ("table", C.c_void_p), ("table_ld", C.c_int), ("heads", C.c_int),
                 ("window", C.c_int), ("scale", C.c_float), ("slopes", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int), ("out", C.c_void_p),
                 ("ld_o", C.c_int), ("row_slot", C.c_void_p), ("row_pos", C.c_void_p), ("rows", C.c_int), ("row0", C.c_int), ("max_keys", C.c_int),
-                ("workspace", C.c_void_p), ("workspace_bytes", C.c_longlong), ("tiles", C.c_void_p), ("n_tiles", C.c_int), ("total_rows", C.c_int)]
+                ("workspace", C.c_void_p), ("workspace_bytes", C.c_longlong), ("tiles", C.c_void_p), ("n_tiles", C.c_int), ("total_rows", C.c_int),
+                ("keep_first", C.c_int), ("softcap", C.c_float), ("sink", C.c_int)]
 
 
 class _Mix(C.Structure):
     _fields_ = [("f32", C.c_int), ("in_", C.c_void_p), ("ld_in", C.c_int), ("nq", C.c_int), ("nk", C.c_int), ("nv", C.c_int), ("off_gate", C.c_int),
-                ("off_up", C.c_int), ("ff", C.c_int), ("act", C.c_int), ("conv", C.c_void_p), ("taps", C.c_int), ("state", C.c_void_p),
+                ("off_up", C.c_int), ("ff", C.c_int), ("act", C.c_int), ("conv", C.c_void_p), ("taps", C.c_int), ("conv_act", C.c_int), ("state", C.c_void_p),
                 ("state_half", C.c_longlong), ("q_out", C.c_void_p), ("ld_q", C.c_int), ("k_pool", C.c_void_p), ("v_pool", C.c_void_p), ("kv_heads", C.c_int),
                 ("dim_p", C.c_int), ("vdim_p", C.c_int), ("table", C.c_void_p), ("table_ld", C.c_int), ("temp_coef", C.c_float), ("temp_every", C.c_int),
                 ("ff_out", C.c_void_p), ("ld_ff", C.c_int), ("tiles", C.c_void_p), ("n_tiles", C.c_int), ("tile_rows", C.c_int), ("rows", C.c_int)]

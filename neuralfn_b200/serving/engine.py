@@ -55,13 +55,16 @@ class Sampling:
 class _CLayer(C.Structure):
     _fields_ = [("heads", C.c_int), ("kv_heads", C.c_int), ("dim", C.c_int), ("vdim", C.c_int), ("conv_taps", C.c_int), ("window", C.c_int),
                 ("kv_from", C.c_int), ("scale", C.c_float), ("alibi", C.c_float), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int),
-                ("out_gate", C.c_int), ("ff", C.c_int), ("ff_act", C.c_int)]
+                ("out_gate", C.c_int), ("ff", C.c_int), ("ff_act", C.c_int), ("mixer", C.c_int), ("qkv_bias", C.c_int), ("keep_first", C.c_int),
+                ("softcap", C.c_float), ("sink", C.c_int), ("rank_decay", C.c_int), ("rank_gate", C.c_int), ("experts", C.c_int), ("top", C.c_int),
+                ("expert_ff", C.c_int), ("weights_of", C.c_int)]
 
 
 class _CLayeredConfig(C.Structure):
     _fields_ = [("n_layer", C.c_int), ("width", C.c_int), ("vocab", C.c_int), ("side_dim", C.c_int), ("embed_scale", C.c_float),
                 ("norm_eps", C.c_float), ("dtype", C.c_int), ("max_seq", C.c_int), ("max_batch", C.c_int), ("kv_tokens", C.c_int),
-                ("max_step_rows", C.c_int), ("use_cuda_graph", C.c_int)]
+                ("max_step_rows", C.c_int), ("use_cuda_graph", C.c_int), ("chained", C.c_int), ("streams", C.c_int), ("untied_head", C.c_int),
+                ("norm_offset", C.c_float), ("logit_scale", C.c_float), ("logit_softcap", C.c_float)]
 
 
 class _CEntry(C.Structure):
@@ -88,12 +91,30 @@ class LayerSpec:
     out_gate: int = 0
     ff: int = 0
     ff_act: str = "relu"
+    mixer: str = "attention"
+    qkv_bias: int = 0
+    keep_first: int = 0
+    softcap: float = 0.0
+    sink: int = 0
+    rank_decay: int = 0
+    rank_gate: int = 0
+    experts: int = 0
+    top: int = 0
+    expert_ff: int = 0
+    weights_of: int = -1
 
     FF_ACT_IDS = {"gelu": 1, "silu": 3, "relu": 6}
+    MIXER_IDS = {"attention": 0, "delta": 1}
 
     def c(self) -> _CLayer:
         return _CLayer(self.heads, self.kv_heads, self.dim, self.vdim, self.conv_taps, self.window, self.kv_from, self.scale, self.alibi,
-                       self.q_temp_coef, self.q_temp_every, self.out_gate, self.ff, self.FF_ACT_IDS[self.ff_act])
+                       self.q_temp_coef, self.q_temp_every, self.out_gate, self.ff, self.FF_ACT_IDS[self.ff_act], self.MIXER_IDS[self.mixer], self.qkv_bias, self.keep_first,
+                       self.softcap, self.sink, self.rank_decay, self.rank_gate, self.experts, self.top, self.expert_ff, self.weights_of)
+
+    @property
+    def cache_row(self) -> int:
+        """Values one token adds to this layer's pages."""
+        return 0 if self.kv_from >= 0 or self.mixer == "delta" else self.kv_heads * (self.dim + self.vdim)
 
 
 @dataclass(frozen=True)
@@ -113,6 +134,12 @@ class LayeredEngineConfig:
     kv_tokens: int = 0
     max_step_rows: int = 8192
     use_cuda_graph: int = 1
+    chained: int = 0
+    streams: int = 0
+    untied_head: int = 0
+    norm_offset: float = 0.0
+    logit_scale: float = 1.0
+    logit_softcap: float = 0.0
 
     family = 2
     kv_cache_mode = 0
@@ -131,12 +158,17 @@ class LayeredEngineConfig:
 
     @property
     def window(self) -> int:
-        """Widest window when every layer has one, else 0."""
-        return 0 if any(y.window == 0 for y in self.layers) else max(y.window for y in self.layers)
+        """Most tokens behind a sequence's end whose pages stay (widest window plus kept first tokens, in whole pages) when every layer
+        with pages has a window, else 0."""
+        paged = [y for y in self.layers if y.mixer == "attention"]
+        if any(y.window == 0 for y in paged):
+            return 0
+        return max((y.window + (y.keep_first + KV_PAGE - 1) // KV_PAGE * KV_PAGE for y in paged), default=0)
 
     def create(self, lib, device: int):
         cc = _CLayeredConfig(len(self.layers), self.width, self.vocab, self.side_dim, self.embed_scale, self.norm_eps,
-                             int(self.dtype == "float32"), self.max_seq, self.max_batch, self.kv_tokens, self.max_step_rows, self.use_cuda_graph)
+                             int(self.dtype == "float32"), self.max_seq, self.max_batch, self.kv_tokens, self.max_step_rows, self.use_cuda_graph, self.chained,
+                             self.streams, self.untied_head, self.norm_offset, self.logit_scale, self.logit_softcap)
         arr = (_CLayer * len(self.layers))(*[y.c() for y in self.layers])
         return lib.nfn_engine_create_layered(C.byref(cc), arr, device)
 
@@ -146,16 +178,26 @@ class LayeredEngineConfig:
         es, wp = (4 if self.dtype == "float32" else 2), up(self.width)
         rows = min(self.max_step_rows, max(self.max_seq, self.max_batch))
         pool = self.kv_tokens or self.max_batch * ((self.max_seq + KV_PAGE - 1) // KV_PAGE * KV_PAGE)
-        weights, cache, widest = wp * up(self.vocab) + self.vocab * self.n_layer * up(self.side_dim), 0, 0
+        weights, cache, widest, routed = wp * up(self.vocab) * (1 + self.untied_head) + self.vocab * self.n_layer * up(self.side_dim), 0, 0, 0
         for y in self.layers:
-            q, v = y.heads * up(y.dim), y.heads * up(y.vdim)
-            kv = 0 if y.kv_from >= 0 else y.kv_heads * (up(y.dim) + up(y.vdim))
-            n_in = q + kv + (v if y.out_gate else 0) + 2 * up(y.ff)
-            weights += wp * (n_in + v + up(y.ff) + 2 * up(self.side_dim))
-            cache += kv * pool * es
-            widest = max(widest, n_in + q + v + up(y.ff))
-        acts = rows * (es * (3 * wp + widest + up(self.side_dim)) + 4 * (wp + up(self.side_dim))) + 4 * 2 * max(self.max_batch, 64) * up(self.vocab)
-        return int(2 * weights + cache + acts)
+            dim, vdim = up(y.dim), up(y.vdim)
+            q, v = y.heads * dim, y.heads * vdim
+            if y.mixer == "delta":
+                conv = 2 * y.kv_heads * dim + v
+                n_in = conv + up(y.heads) + up(y.rank_decay) + up(y.rank_gate)
+                own = q * up(y.rank_decay) + v * up(y.rank_gate)
+                cache += self.max_batch * (4 * q * vdim + 2 * es * conv * (y.conv_taps - 1))
+                widest = max(widest, n_in + conv + (4 // es) * (q + v) + 2 * v)
+            else:
+                kv = 0 if y.kv_from >= 0 else y.kv_heads * (dim + vdim)
+                n_in, own = q + kv + (v if y.out_gate else 0) + 2 * up(y.ff), 0
+                cache += kv * pool * es
+                widest = max(widest, n_in + q + v + up(y.ff))
+            if y.weights_of < 0:
+                weights += wp * (n_in + v + up(y.ff) + 2 * up(self.side_dim)) + own + wp * (up(y.experts) + 3 * y.experts * up(y.expert_ff))
+            routed = max(routed, (rows * y.top + 127 * y.experts) * es * (2 * wp + 3 * up(y.expert_ff)) if y.experts else 0)
+        acts = rows * (es * (3 * wp + widest + up(self.side_dim)) + 4 * (wp * max(self.streams, 1) + up(self.side_dim))) + 4 * 2 * max(self.max_batch, 64) * up(self.vocab)
+        return int(2 * weights + cache + acts + routed)
 
 
 @dataclass(frozen=True)
@@ -316,7 +358,7 @@ class ResidentEngine:
         """Cache bytes one token occupies in a global (full-context) layer; in all layers together for a layer-list model."""
         c = self.config
         if c.family == 2:
-            return sum(y.kv_heads * (y.dim + y.vdim) for y in c.layers if y.kv_from < 0) * (4 if c.dtype == "float32" else 2)
+            return sum(y.cache_row for y in c.layers) * (4 if c.dtype == "float32" else 2)
         if c.kv_cache_mode == 1:
             return c.n_kv_head * (self.turboquant.key_layout.record_bytes + self.turboquant.value_layout.record_bytes)
         return 2 * c.n_kv_head * c.head_dim * 2
