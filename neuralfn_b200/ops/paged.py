@@ -63,8 +63,9 @@ class PagedCache:
             self.v[page, :, :, :n] = v[part].permute(1, 2, 0).to(self.dtype)
 
 
-def _args(c: PagedCache, q, out, heads, window, scale, slopes, gate) -> _Attention:
+def _args(c: PagedCache, q, out, heads, window, scale, slopes, gate, keep_first=0, softcap=0.0, sink=False) -> _Attention:
     a = _Attention()
+    a.keep_first, a.softcap, a.sink = keep_first, softcap, int(sink)
     a.f32, a.q, a.ld_q, a.k_pool, a.v_pool = int(c.dtype == torch.float32), _p(q), q.stride(0), _p(c.k), _p(c.v)
     a.kv_heads, a.dim_p, a.vdim_p, a.pages, a.table, a.table_ld = c.kv_heads, c.dim, c.vdim, c.pages, _p(c.table), c.table.stride(0)
     a.heads, a.window, a.scale, a.slopes, a.gate, a.ld_gate = heads, window, scale, _p(slopes), _p(gate), gate.stride(0) if gate is not None else 0
@@ -73,10 +74,11 @@ def _args(c: PagedCache, q, out, heads, window, scale, slopes, gate) -> _Attenti
 
 
 def attention_rows(c: PagedCache, q: torch.Tensor, row_slot: torch.Tensor, row_pos: torch.Tensor, out: torch.Tensor, *, heads: int, window: int = 0,
-                   scale: float, slopes: torch.Tensor | None = None, gate: torch.Tensor | None = None, max_keys: int = 0) -> torch.Tensor:
-    a = _args(c, q, out, heads, window, scale, slopes, gate)
+                   scale: float, slopes: torch.Tensor | None = None, gate: torch.Tensor | None = None, max_keys: int = 0, keep_first: int = 0,
+                   softcap: float = 0.0, sink: bool = False) -> torch.Tensor:
+    a = _args(c, q, out, heads, window, scale, slopes, gate, keep_first, softcap, sink)
     a.row_slot, a.row_pos, a.rows = _p(row_slot), _p(row_pos), q.shape[0]
-    a.max_keys = max_keys or (window or c.table.shape[1] * PAGE)
+    a.max_keys = max_keys or (window + keep_first if window else c.table.shape[1] * PAGE)
     _lib.check(_lib.load().nfn_paged_attention_rows(C.byref(a), C.c_void_p(_lib.stream_ptr())), "paged_attention_rows")
     return out
 
@@ -86,9 +88,10 @@ def tile_rows(c: PagedCache, heads: int) -> int:
 
 
 def attention_tiles(c: PagedCache, q: torch.Tensor, tiles: torch.Tensor, out: torch.Tensor, *, heads: int, window: int = 0, scale: float,
-                    slopes: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
+                    slopes: torch.Tensor | None = None, gate: torch.Tensor | None = None, keep_first: int = 0, softcap: float = 0.0,
+                    sink: bool = False) -> torch.Tensor:
     """``tiles``: int32 [n, 4] = first row, rows (<= ``tile_rows``), slot, position of the first row."""
-    a = _args(c, q, out, heads, window, scale, slopes, gate)
+    a = _args(c, q, out, heads, window, scale, slopes, gate, keep_first, softcap, sink)
     a.tiles, a.n_tiles = _p(tiles), tiles.shape[0]
     _lib.check(_lib.load().nfn_paged_attention_tiles(C.byref(a), C.c_void_p(_lib.stream_ptr())), "paged_attention_tiles")
     return out
@@ -109,8 +112,9 @@ def row_tiles(entries: list[tuple[int, int, int, int]], device) -> torch.Tensor:
 
 def mix_rows(c: PagedCache, x: torch.Tensor, tiles: torch.Tensor, q_out: torch.Tensor, ff_out: torch.Tensor | None, *, heads: int, own_kv: bool = True,
              off_gate: int = 0, off_up: int = 0, ff: int = 0, act: int = 6, conv: torch.Tensor | None = None, state: torch.Tensor | None = None,
-             temp: tuple[float, int] = (0.0, 0)) -> None:
+             temp: tuple[float, int] = (0.0, 0), conv_act: int = 0) -> None:
     m = _Mix()
+    m.conv_act = conv_act
     m.f32, m.in_, m.ld_in, m.nq = int(c.dtype == torch.float32), _p(x), x.stride(0), heads * c.dim
     m.nk, m.nv = (c.kv_heads * c.dim, c.kv_heads * c.vdim) if own_kv else (0, 0)
     m.off_gate, m.off_up, m.ff, m.act, m.conv, m.taps = off_gate, off_up, ff, act, _p(conv), 0 if conv is None else conv.shape[0]

@@ -72,6 +72,13 @@ def visible(i, size, keep):
     return [j for j in range(i + 1) if not size or i - j < size or j < keep]
 
 
+def softmax_with_sink(s):
+    """Over the scores of a row and one more of 0, whose share is lost."""
+    top = s.max(-1, keepdim=True).values.clamp(min=0.0)
+    e = torch.exp(s - top)
+    return e / (e.sum(-1, keepdim=True) + torch.exp(-top))
+
+
 def attention_mixer(h, W, p, m):
     T, H, G, d, dv = h.shape[0], m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q, k, v = (h @ W[p + f"mix.{n}"].T + W[p + f"mix.{n}.b"] for n in "qkv")
@@ -79,16 +86,16 @@ def attention_mixer(h, W, p, m):
     mask = m.get("mask") or {}
     cap = m.get("softcap")
     out = torch.zeros(T, H, dv, dtype=h.dtype)
+    seen = torch.zeros(T, T, dtype=torch.bool)
     for i in range(T):
-        js = visible(i, mask.get("size", 0), mask.get("keep_first", 0))
-        for x in range(H):
-            g = x // (H // G)
-            s = k[js, g] @ q[i, x] * m["scale"]
-            if cap:
-                s = cap * torch.tanh(s / cap)
-            top = max(float(s.max()), 0.0)
-            e = torch.exp(s - top)
-            out[i, x] = (e / (e.sum() + math.exp(-top))) @ v[js, g]
+        seen[i, visible(i, mask.get("size", 0), mask.get("keep_first", 0))] = True
+    for x in range(H):
+        g = x // (H // G)
+        s = q[:, x] @ k[:, g].T * m["scale"]
+        if cap:
+            s = cap * torch.tanh(s / cap)
+        s = s.masked_fill(~seen, -math.inf)
+        out[:, x] = softmax_with_sink(s) @ v[:, g]
     return out.reshape(T, -1) @ W[p + "mix.o"].T
 
 
@@ -102,6 +109,14 @@ def experts(h, W, p, mlp):
             f = p + f"mlp.e{e}."
             out[t] += W[f + "down"] @ (silu(W[f + "gate"] @ a) * (W[f + "up"] @ a))
     return out
+
+
+def routing_gap(z, top):
+    """Smallest distance between a chosen and a left-out expert's logit over the rows (infinite when all are chosen)."""
+    if top == z.shape[1]:
+        return math.inf
+    v = torch.sort(z, -1, descending=True).values
+    return float((v[:, top - 1] - v[:, top]).min())
 
 
 def mixed_in(xs, W, p):
@@ -121,8 +136,9 @@ def layer_order(cfg):
     return list(range(loop["start"])) + body * loop["times"] + list(range(loop["stop"], n))
 
 
-def forward(cfg, weights, tokens, dtype=torch.float64):
-    """-> logits [T, vocab], residual (sum of the streams) after every layer run [runs, T, width]."""
+def forward(cfg, weights, tokens, dtype=torch.float64, gaps=None):
+    """-> logits [T, vocab], residual (sum of the streams) after every layer run [runs, T, width]. gaps: a list that receives the routing
+    gap of every layer run."""
     W = {k: v.to(dtype) for k, v in weights.items()}
     tokens = torch.as_tensor(tokens, dtype=torch.long)
     eps = cfg["norm"]["eps"]
@@ -139,6 +155,8 @@ def forward(cfg, weights, tokens, dtype=torch.float64):
             h = centred_norm(u, W[p + f"norm{q}"], eps)
             if what == "mlp":
                 y = experts(h, W, p, layer["mlp"])
+                if gaps is not None:
+                    gaps.append(routing_gap(h @ W[p + "mlp.router"].T, layer["mlp"]["router"]["top"]))
             elif layer["type"] == "channel_delta":
                 y = delta_mixer(h, W, p, layer["mixer"], eps)
             else:

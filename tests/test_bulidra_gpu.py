@@ -8,6 +8,7 @@ import torch
 
 import bulidra_oracle as oracle
 from bulidra_cases import boost_needle, layer, model, tokens_of
+from step_helpers import repeat_cuts, run_cuts, run_mixed, worst
 
 pytestmark = pytest.mark.gpu
 
@@ -23,36 +24,6 @@ def make_engine(cfg, weights, dtype="float32", **kw):
     eng = ResidentEngine(engine_config(c, dtype=dtype, **kw))
     eng.load_named_tensors(pack_tensors(c, weights))
     return eng
-
-
-def run_cuts(eng, slot, ids, cuts):
-    """One sequence in portions; returns the logits of every position."""
-    from neuralfn_b200.serving import StepEntry
-    eng.release(slot)
-    out, at = [], 0
-    for n in cuts:
-        part = ids[at:at + n]
-        out.append(eng.step([StepEntry(slot, part, range(len(part)))], logits=True)[1])
-        at += n
-    assert at == len(ids)
-    return torch.cat(out)
-
-
-def worst(got, want):
-    d = got.double() - want
-    d = d - d.mean(-1, keepdim=True)
-    spread = (want - want.mean(-1, keepdim=True)).pow(2).mean().sqrt()
-    return float((d.pow(2).mean(-1).sqrt() / spread).max())
-
-
-def repeat_cuts(n, sizes):
-    out, left, i = [], n, 0
-    while left:
-        k = min(sizes[i % len(sizes)], left)
-        out.append(k)
-        left -= k
-        i += 1
-    return out
 
 
 def sizes_grid():
@@ -143,42 +114,15 @@ def test_first_tokens(dtype):
 def test_mixed_batches_and_reuse(dtype):
     """Unequal requests together, some fed by portions and some by single tokens, left out of steps, ended and replaced, in a pool that
     holds only what is live: every logit equals the request's own."""
-    from neuralfn_b200.serving import StepEntry
     cfg, w = sizes_grid()["all"]
     lengths = [190, 70, 3, 128, 64, 41, 150, 2]
     seqs = [tokens_of(cfg, n, seed=100 + i) for i, n in enumerate(lengths)]
     want = [oracle.forward(cfg, w, s)[0] for s in seqs]
     eng = make_engine(cfg, w, dtype, max_batch=3, max_seq=256, kv_tokens=192 + 128 + 64)
     room = eng.free_tokens
-    g = torch.Generator().manual_seed(5)
-    waiting, live, free, at = list(range(len(seqs))), {}, [0, 1, 2], {}
-    got = [[] for _ in seqs]
-    held = lambda i: (lengths[i] + 63) // 64 * 64  # noqa: E731
-    while waiting or live:
-        for i in list(waiting):
-            if free and sum(held(k) for k in live) + held(i) <= 384:
-                live[i], at[i] = free.pop(), 0
-                eng.release(live[i])
-                waiting.remove(i)
-        entries, who = [], []
-        for i, slot in live.items():
-            kind = int(torch.randint(0, 5, (1,), generator=g))
-            if kind == 0 and len(live) > 1 and entries:
-                continue
-            n = min([1, 1, 2, 19, 50][kind], lengths[i] - at[i])
-            entries.append(StepEntry(slot, seqs[i][at[i]:at[i] + n], range(n)))
-            who.append((i, n))
-        rows = eng.step(entries, logits=True)[1]
-        base = 0
-        for i, n in who:
-            got[i].append(rows[base:base + n])
-            base += n
-            at[i] += n
-            if at[i] == lengths[i]:
-                eng.release(live[i])
-                free.append(live.pop(i))
+    got = run_mixed(eng, seqs, slots=3, room=384, seed=5)
     for i in range(len(seqs)):
-        assert worst(torch.cat(got[i]), want[i]) < TOL[dtype], i
+        assert worst(got[i], want[i]) < TOL[dtype], i
     assert eng.free_tokens == room
     eng.close()
 

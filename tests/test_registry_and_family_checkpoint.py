@@ -22,11 +22,12 @@ def test_registry_resolution_and_proofs():
     with pytest.raises(ValueError):
         q.require("native_training")
     assert capability_proof_for("jamba").route == "tensor-runtime"
-    assert len(native_families_report()) == len(NATIVE_FAMILIES) == 17
+    assert len(native_families_report()) == len(NATIVE_FAMILIES) == 18
     trained = [s for s in NATIVE_FAMILIES.values() if s.route != "serving-only"]
     assert len(trained) == 16 and all(s.reference_binary.startswith("nfn_") and s.reference_binary.endswith("_native_train") for s in trained)
-    b = capability_proof_for("bulidra")
-    assert b.native_inference and not b.native_training and b.route == "serving-only" and len(b.reasons) == 1
+    for name in ("bulidra", "murilorn"):
+        b = capability_proof_for(name)
+        assert b.native_inference and not b.native_training and b.route == "serving-only" and len(b.reasons) == 1
 
 
 def _tiny():
