@@ -1,5 +1,8 @@
-"""Prefill and decode throughput of Bulidra and, at equal size, of Glimmer blocks - the closest model the engine served before: grouped
-heads, sliding windows, gated attention, gated feed-forward. Random bf16 weights; one JSON line per model, size and phase.
+"""Prefill and decode throughput of Bulidra or Murilorn and, at equal size, of Glimmer blocks - the closest model the engine served before:
+grouped heads, sliding windows, gated attention, gated feed-forward. Random bf16 weights; one JSON line per model, size and phase.
+
+Murilorn at equal size: delta-rule and attention layers in turn with the same heads, the same active feed-forward width (four of thirty-two
+experts), four residual streams.
 
 ``ms`` is device time (CUDA events on the engine's stream, median over repetitions of the public ``prefill`` / ``decode`` call,
 including its host-to-device copy of tokens and the read-back of the drawn token); weights and caches are larger than L2. Beside it
@@ -19,6 +22,7 @@ SIZES = {
     "w4096_wide_window": dict(width=4096, heads=32, kv_heads=8, dim=128, ff=14336, window=4096, layers=6, vocab=32768),
 }
 SIDE_DIM = 256
+EXPERTS, TOP, STREAMS, RANK, KEEP = 32, 4, 4, 128, 4
 
 
 def _peaks() -> tuple[float, float]:
@@ -31,9 +35,16 @@ def _peaks() -> tuple[float, float]:
 
 def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
     from ..models.bulidra import BulidraConfig, BulidraLayer, engine_config
+    from ..models import murilorn as M
     from ..serving import EngineConfig, ResidentEngine
-    if kind == "bulidra":
-        L = z["layers"]
+    L = z["layers"]
+    if kind == "murilorn":
+        ex = dict(experts=EXPERTS, top=TOP, expert_ff=z["ff"] // TOP)
+        pair = (M.MurilornLayer("channel_delta", z["heads"], z["heads"], z["dim"], z["dim"], conv=4, rank_decay=RANK, rank_gate=RANK, **ex),
+                M.MurilornLayer("attention", z["heads"], z["kv_heads"], z["dim"], z["dim"], scale=z["dim"] ** -0.5, softcap=30.0, window=z["window"], keep_first=KEEP, **ex))
+        cfg = M.engine_config(M.MurilornConfig(z["vocab"], z["width"], 1.0, 1e-5, STREAMS, None, 1.0, 30.0, (pair * L)[:L]), max_batch=max_batch, max_seq=max_seq,
+                              max_step_rows=max_seq)
+    elif kind == "bulidra":
         layers = tuple(BulidraLayer(z["heads"], z["kv_heads"], z["dim"], z["dim"], 4, z["dim"] ** -0.5, z["window"], 0.1, 1024, None, z["ff"]) for _ in range(L))
         cfg = engine_config(BulidraConfig(z["vocab"], z["width"], 1.0, 1e-5, SIDE_DIM, layers), max_batch=max_batch, max_seq=max_seq, max_step_rows=max_seq)
     else:
@@ -42,7 +53,15 @@ def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
     eng = ResidentEngine(cfg)
     g = torch.Generator(device="cuda").manual_seed(0)
     for n, k in eng.expected_tensors().items():
-        t = torch.ones(k, device="cuda") if "norm" in n else torch.randn(k, generator=g, device="cuda") * 0.02
+        leaf = n.rsplit(".", 1)[-1]
+        if leaf.startswith("hc"):
+            t = torch.eye(STREAMS, device="cuda").flatten() if leaf.endswith("mix") else torch.full((k,), 1.0 / STREAMS if leaf.endswith("in") else 1.0, device="cuda")
+        elif leaf in ("a_log", "dt_bias"):
+            t = torch.full((k,), -1.0, device="cuda")
+        elif "norm" in n:
+            t = torch.full((k,), 0.0 if kind == "murilorn" and leaf != "out_norm" else 1.0, device="cuda")
+        else:
+            t = torch.randn(k, generator=g, device="cuda") * 0.02
         eng.set_tensor(n, t.bfloat16())
     eng.finalize()
     return eng
@@ -64,6 +83,8 @@ def _time(eng, fn, n: int, warmup: int) -> float:
 def _work(z: dict, kind: str, prompt: int, batch: int, context: int) -> tuple[float, float]:
     """(FLOPs of a prompt, bytes of a decode step): products and attention over visible keys; weights and visible cache rows."""
     w, q, kv = z["width"], z["heads"] * z["dim"], z["kv_heads"] * z["dim"]
+    if kind == "murilorn":
+        return _murilorn_work(z, prompt, batch, context)
     per = w * (q + 2 * kv + q + 2 * z["ff"]) + w * (q + z["ff"]) + (2 * w * SIDE_DIM if kind == "bulidra" else 0)
     win = min(z["window"], prompt)
     keys = win * (win + 1) / 2 + (prompt - win) * win
@@ -72,11 +93,28 @@ def _work(z: dict, kind: str, prompt: int, batch: int, context: int) -> tuple[fl
     return flops, 2.0 * z["layers"] * (per + batch * seen * 2 * kv) + 2.0 * z["vocab"] * w
 
 
+def _murilorn_work(z: dict, prompt: int, batch: int, context: int) -> tuple[float, float]:
+    w, q, kv, L = z["width"], z["heads"] * z["dim"], z["kv_heads"] * z["dim"], z["layers"]
+    n_delta = (L + 1) // 2
+    n_att = L - n_delta
+    delta = w * (3 * q + z["heads"] + 2 * RANK) + 2 * RANK * q + q * w
+    att = w * (q + 2 * kv) + q * w
+    expert = 3 * w * (z["ff"] // TOP)
+    win = min(z["window"], prompt)
+    keys = win * (win + 1) / 2 + (prompt - win) * win
+    rule = 7.0 * q * z["dim"]                                   # decay, correction, write, read-out
+    flops = n_delta * (2.0 * delta + rule) * prompt + n_att * (2.0 * att * prompt + 4.0 * q * keys) + L * 2.0 * (TOP * expert + EXPERTS * w) * prompt
+    chosen = EXPERTS * (1 - (1 - TOP / EXPERTS) ** batch)       # experts a batch of uniform choices touches
+    seen = min(z["window"] + KEEP, context)
+    byts = 2.0 * (n_delta * delta + n_att * (att + batch * seen * 2 * kv) + L * (chosen * expert + EXPERTS * w)) + n_delta * batch * 8.0 * q * z["dim"] + 2.0 * z["vocab"] * w
+    return flops, byts
+
+
 def run(args, clock_sampler, sizes=None) -> None:
     hbm, tf = _peaks()
     for name in sizes or SIZES:
         z = SIZES[name]
-        for kind in ("glimmer", "bulidra"):
+        for kind in ("glimmer", args.serving):
             prompt, context = 8192, 4096
             eng = _engine(kind, z, 1, prompt + 64)
             g = torch.Generator().manual_seed(1)

@@ -72,7 +72,8 @@ struct layered_engine final : nfn_engine {
   void *xb = nullptr, *h = nullptr, *in = nullptr, *q = nullptr, *cat = nullptr, *s_act = nullptr, *y = nullptr, *hw = nullptr;
   float *s_gate = nullptr, *logits = nullptr, *saved = nullptr;
   float *decay = nullptr, *d_o = nullptr;           // delta: projected decays, read-outs
-  void* d_gate = nullptr;
+  void *d_gate = nullptr, *delta_ws = nullptr;
+  long long delta_ws_bytes = 0;
   struct { float *logits = nullptr, *weight = nullptr, *row_w = nullptr; int *idx = nullptr, *order = nullptr, *offsets = nullptr, *active = nullptr, *counts = nullptr,
            *cursor = nullptr, *tile_expert = nullptr, *plan = nullptr, *row_of = nullptr; void *xs = nullptr, *gate_up = nullptr, *mid = nullptr, *y = nullptr; } ex;
   nfn_stream_args pend{};                           // chained: the last sublayer's update, applied on the way to the head
@@ -115,7 +116,7 @@ struct layered_engine final : nfn_engine {
   void trim(int slot);                              // pages no later query of this slot can see
   int lin(const void* a, int lda, const void* w, int rows, int n, int k, void* out, int ldo, int kind, const void* bias = nullptr);
   // the rows of one pass: short entries first, then the long ones
-  struct Batch { int rows = 0, short_rows = 0, n_mix = 0, n_seq = 0, n_short_seq = 0; std::vector<int> att_off, att_n; };
+  struct Batch { int rows = 0, short_rows = 0, n_mix = 0, n_seq = 0, n_short_seq = 0, longest = 0; std::vector<int> att_off, att_n; };
   int mix_rows(const Layer& L, const Batch& b, void* ff_out);
   int attention(const Layer& L, const Batch& b);
   int delta(const Layer& L, const Batch& b);
@@ -327,6 +328,7 @@ int layered_engine::finalize() {
     if (d.mixer == NFN_MIXER_DELTA) {
       n_dec = std::max(n_dec, R * d.heads * L.dp);
       n_do = std::max(n_do, R * d.heads * L.vp);
+      if (c.dtype == 0) delta_ws_bytes = std::max(delta_ws_bytes, nfn_delta_chunk_workspace_bytes(d.heads, L.dp, L.vp, c.max_batch));
     }
     if (d.experts > 0) {
       const bool g = grouped(L, (int)R);
@@ -341,6 +343,7 @@ int layered_engine::finalize() {
       e_rows = std::max(e_rows, std::max(sorted, single));
     }
   }
+  if (delta_ws_bytes > 0 && add(&delta_ws, delta_ws_bytes)) return -1;
   if (n_dec && (zero((void**)&decay, n_dec * 4) || zero((void**)&d_o, n_do * 4) || zero(&d_gate, n_do * es))) return -1;
   if (e_max && (zero((void**)&ex.logits, e_log * 4) || zero((void**)&ex.weight, e_items * 4) || zero((void**)&ex.idx, e_items * 4) ||
                 zero((void**)&ex.order, e_items * 4) || zero((void**)&ex.row_of, e_items * 4) || zero((void**)&ex.offsets, (e_max + 1) * 4) ||
@@ -627,8 +630,14 @@ int layered_engine::delta(const Layer& L, const Batch& b) {
   a.decay = decay; a.ld_decay = n_dec; a.a_log = L.a_log; a.dt_bias = L.dt_bias;
   a.heads = d.heads; a.kv_heads = d.kv_heads; a.dim = d.dim; a.dim_p = L.dp; a.vdim_p = L.vp; a.unit_eps = 1e-6f;
   a.state = L.memory; a.o = d_o; a.ld_o = n_o;
-  a.seqs = dev<nfn_seq_rows>(io.seq); a.n_seqs = b.n_seq;
-  K(nfn_delta_rows(&a, stream));
+  const bool chunks = c.dtype == 0 && L.dp <= 256;
+  a.seqs = dev<nfn_seq_rows>(io.seq); a.n_seqs = chunks ? b.n_short_seq : b.n_seq;
+  if (a.n_seqs > 0) K(nfn_delta_rows(&a, stream));
+  if (chunks && b.n_seq > b.n_short_seq) {
+    a.seqs += b.n_short_seq;
+    a.n_seqs = b.n_seq - b.n_short_seq;
+    K(nfn_delta_chunks(&a, b.longest, delta_ws, delta_ws_bytes, stream));
+  }
   K(nfn_delta_out(a.f32, d_o, n_o, d_gate, n_o, L.out_norm, c.norm_eps, cat, L.n_cat, b.rows, d.heads, d.vdim, L.vp, stream));
   return 0;
 }
@@ -808,7 +817,7 @@ int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* 
   nfn_seq_rows* seq = host<nfn_seq_rows>(io.seq);
   for (int longs = 0; longs < 2; ++longs) {
     for (size_t i = 0; i < part.size(); ++i)
-      if ((part[i].count >= kTileMin) == (longs == 1)) seq[b.n_seq++] = nfn_seq_rows{first[i], part[i].count, part[i].slot, len[part[i].slot]};
+      if ((part[i].count >= kTileMin) == (longs == 1)) b.longest = std::max(b.longest, part[i].count), seq[b.n_seq++] = nfn_seq_rows{first[i], part[i].count, part[i].slot, len[part[i].slot]};
     if (!longs) {
       for (int r = total; r < rows; ++r) seq[b.n_seq++] = nfn_seq_rows{r, 1, -1, 0};
       b.n_short_seq = b.n_seq;

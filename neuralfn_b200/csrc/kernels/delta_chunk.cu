@@ -1,0 +1,479 @@
+// Gated delta rule over prompt portions, sixteen tokens at a time (bf16 activations; state and everything that enters it fp32).
+//
+// Inside a chunk let G_r be the running sum of the log decays (per key channel), S the state before the chunk and, with unit vectors k, q,
+//   A_rj = sum_c k_rc k_jc e^(G_rc - G_jc)  (j < r),   P_rj = sum_c q_rc k_jc e^(G_rc - G_jc)  (j <= r),   T = (I + diag(beta) A)^-1 diag(beta).
+// The corrections of the chunk are U = T V - W S with W = T (e^G k), its read-outs O = P T V + Q S with Q = e^G q - P W, and the state after it
+// S' = e^G_last S + K^T U with K_j = k_j e^(G_last - G_j). Every exponent is a sum of decays between two tokens, never positive, so
+// nothing overflows however fast a channel forgets.
+//
+//   delta_prepare_kernel  one CTA per (chunk, head), all chunks at once: W, Q, K and T V, P T V. A thread owns a channel; products of
+//                         a channel with all pairs of tokens stay in its registers and are summed over channels through shared memory.
+//   delta_scan_kernel     one warp per (head, 16 value columns, 64 key channels), one chunk after another: the state, transposed, sits in
+//                         the accumulator registers of mma.m16n8k16 and is the A operand of the next chunk's W S and Q S as it stands; W, Q
+//                         and K arrive in fragment order by bulk copies through a ring of shared memory stages.
+//
+// The products with the state are formed from fp32 values split into two bf16 parts each (high x high + high x low + low x high), which
+// keeps sixteen bits of every factor. Rounds of as many chunks as the workspace holds alternate between the two kernels, small enough
+// to stay in L2.
+#include <algorithm>
+
+#include "common.h"
+#include "delta.cuh"
+
+namespace nfn {
+
+constexpr int DC_T = 16;                               // tokens of a chunk
+constexpr int DC_THREADS = 128, DC_PITCH = 130;        // partial sums: [64 values][128 threads], two threads read a row without conflicts
+constexpr int DC_STAGES = 3;
+constexpr long long DC_WORKSPACE = 96LL << 20;
+
+// bytes of a (chunk, head) block of the scan's operands: [W, Q: dk / 16 steps x 4 tiles of 8 rows][K: dk / 8 tiles] x 32 lanes x 16 bytes, then
+// e^G_last of every channel
+__host__ __device__ constexpr int dc_block_bytes(int dk) { return 48 * dk * 4 + dk * 4; }
+__host__ __device__ constexpr int dc_uo_floats(int vdim_p) { return vdim_p * 32; }      // T V and P T V: [column tile][2][2 row tiles][32 lanes][4]
+
+struct DeltaChunkParams {
+  nfn_delta_args a;
+  int dk;                     // key channels padded to the scan's 64 per warp
+  int chunk0, n_chunks;       // chunks [chunk0, chunk0 + n_chunks) of every sequence in this round
+  unsigned char* blocks;      // [seq][chunk][head][dc_block_bytes]
+  float* uo;                  // [seq][chunk][head][dc_uo_floats]
+  int* status;
+};
+
+// two fp32 values as bf16 pairs: the rounded values and what they leave out
+__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack_bf16x2(a, b);
+  const float2 f = unpack_bf16x2(hi);
+  lo = pack_bf16x2(a - f.x, b - f.y);
+}
+
+// NCH: channels per thread (key or value channels up to 128 NCH)
+template <int NCH>
+__global__ void __launch_bounds__(DC_THREADS)
+delta_prepare_kernel(const DeltaChunkParams p) {
+  extern __shared__ __align__(128) unsigned char dc_smem[];        // partial sums, then the operand block
+  __shared__ float sA[DC_T][DC_T + 4], sP[DC_T][DC_T + 4], sT[DC_T][DC_T + 4], s_norm[2][DC_T], s_beta[DC_T];
+  const nfn_delta_args& a = p.a;
+  const nfn_seq_rows seq = a.seqs[blockIdx.z];
+  const int r0 = (p.chunk0 + blockIdx.x) * DC_T, n = min(DC_T, seq.n - r0);
+  if (seq.slot < 0 || n <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  const int h = blockIdx.y, hk = h / (a.heads / a.kv_heads), DP = a.dim_p, VP = a.vdim_p;
+  const int off_k = a.kv_heads * DP, off_v = 2 * off_k;
+  const size_t row0 = (size_t)(seq.row0 + r0);
+  const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(a.qkv) + row0 * a.ld_qkv;
+
+  // ---- unit vectors, step sizes ----
+  for (int r = warp; r < DC_T; r += DC_THREADS / 32) {
+    float nq = 0.f, nk = 0.f;
+    if (r < n)
+      for (int d = lane * 2; d < DP; d += 64) {
+        const float2 q = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + (size_t)r * a.ld_qkv + hk * DP + d));
+        const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + (size_t)r * a.ld_qkv + off_k + hk * DP + d));
+        nq += q.x * q.x + q.y * q.y;
+        nk += k.x * k.x + k.y * k.y;
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      nq += __shfl_xor_sync(0xffffffffu, nq, o);
+      nk += __shfl_xor_sync(0xffffffffu, nk, o);
+    }
+    if (lane == 0) {
+      s_norm[0][r] = 1.f / (sqrtf((float)a.dim) * sqrtf(nq + a.unit_eps));
+      s_norm[1][r] = 1.f / sqrtf(nk + a.unit_eps);
+      s_beta[r] = r < n ? sigmoid_exact(__bfloat162float(static_cast<const __nv_bfloat16*>(a.beta)[(row0 + r) * a.ld_beta + h])) : 0.f;
+    }
+  }
+  __syncthreads();
+  // ---- this thread's channels: q, k and the running sum of log decays ----
+  float q[NCH][DC_T], k[NCH][DC_T], G[NCH][DC_T];
+  const float rate = -expf(__bfloat162float(static_cast<const __nv_bfloat16*>(a.a_log)[h]));
+#pragma unroll
+  for (int i = 0; i < NCH; ++i) {
+    const int c = tid + i * DC_THREADS;
+    const bool on = c < DP;
+    const float bias = on ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.dt_bias)[(size_t)h * DP + c]) : 0.f;
+    float raw[DC_T];
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      const bool live = on && r < n;
+      q[i][r] = live ? __bfloat162float(x[(size_t)r * a.ld_qkv + hk * DP + c]) : 0.f;
+      k[i][r] = live ? __bfloat162float(x[(size_t)r * a.ld_qkv + off_k + hk * DP + c]) : 0.f;
+      raw[r] = live ? a.decay[(row0 + r) * a.ld_decay + (size_t)h * DP + c] : 0.f;
+    }
+    float sum = 0.f;
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      q[i][r] *= s_norm[0][r];
+      k[i][r] *= s_norm[1][r];
+      if (on && r < n) sum += delta_log_decay(raw[r] + bias, rate);
+      G[i][r] = sum;
+    }
+  }
+  // ---- A and P: rows 2t, 15 - 2t, 2t + 1, 14 - 2t together have 64 values ----
+  float* part = reinterpret_cast<float*>(dc_smem);
+  const float LOG2E = 1.4426950408889634f;
+#pragma unroll
+  for (int t = 0; t < 4; ++t) {
+    const int rows[4] = {2 * t, 15 - 2 * t, 2 * t + 1, 14 - 2 * t};
+    int at = 0;
+#pragma unroll
+    for (int w = 0; w < 4; ++w) {
+      const int r = rows[w];
+#pragma unroll
+      for (int j = 0; j < DC_T; ++j) {
+        if (j > r) continue;
+        float va = 0.f, vp = 0.f;
+#pragma unroll
+        for (int i = 0; i < NCH; ++i) {
+          const float kj = j < r ? k[i][j] * fast_exp2((G[i][r] - G[i][j]) * LOG2E) : k[i][j];
+          va += k[i][r] * kj;
+          vp += q[i][r] * kj;
+        }
+        part[at++ * DC_PITCH + tid] = vp;
+        if (j < r) part[at++ * DC_PITCH + tid] = va;
+      }
+    }
+    __syncthreads();
+    {
+      // value `v` of the pass is summed by two threads, one per parity of the channel
+      const int v = tid >> 1;
+      float s0 = 0.f, s1 = 0.f;
+      const float* src = part + v * DC_PITCH + (tid & 1);
+#pragma unroll 8
+      for (int i = 0; i < DC_THREADS / 2; i += 2) {
+        s0 += src[2 * i];
+        s1 += src[2 * i + 2];
+      }
+      float s = s0 + s1;
+      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      // where it belongs: the rows of the pass hold 2 r + 1 values each, P_rj and A_rj in turn
+      int rest = v, r = rows[0];
+      if (rest >= 2 * r + 1) { rest -= 2 * r + 1; r = rows[1];
+        if (rest >= 2 * r + 1) { rest -= 2 * r + 1; r = rows[2];
+          if (rest >= 2 * r + 1) { rest -= 2 * r + 1; r = rows[3]; } } }
+      if ((tid & 1) == 0) ((rest & 1) ? sA : sP)[r][rest >> 1] = s;
+    }
+    __syncthreads();
+  }
+  // ---- T = (I + diag(beta) A)^-1 diag(beta): one column per lane, forward substitution ----
+  if (tid < DC_T) {
+    float y[DC_T];
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      float s = r == tid ? 1.f : 0.f;
+      const float b = s_beta[r];
+#pragma unroll
+      for (int i = 0; i < r; ++i) s -= b * sA[r][i] * y[i];
+      y[r] = s;
+    }
+    const float b = s_beta[tid];
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) sT[r][tid] = y[r] * b;
+  }
+  __syncthreads();
+  const size_t block = ((size_t)blockIdx.z * p.n_chunks + blockIdx.x) * a.heads + h;
+  // ---- W, Q, K of this thread's key channels, in the order of the scan's fragments ----
+  unsigned char* stage = dc_smem;
+  float* gamma = reinterpret_cast<float*>(stage + 48 * p.dk * 4);
+#pragma unroll
+  for (int i = 0; i < NCH; ++i) {
+    const int c = tid + i * DC_THREADS;
+    if (c >= p.dk) continue;
+    float e[DC_T], w[DC_T];
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) e[r] = fast_exp2(G[i][r] * LOG2E);
+    gamma[c] = e[DC_T - 1];
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j <= r; ++j) s += sT[r][j] * (k[i][j] * e[j]);
+      w[r] = s;
+    }
+    auto put = [&](int tile, int row, int col, float v) {      // element (row, col) of a 8 x 16 operand tile: high and low part
+      const __nv_bfloat16 hi = __float2bfloat16(v), lo = __float2bfloat16(v - __bfloat162float(hi));
+      unsigned char* d = stage + ((size_t)(tile * 32 + row * 4 + ((col & 7) >> 1)) * 16 + (col >> 3) * 4 + (col & 1) * 2);
+      *reinterpret_cast<__nv_bfloat16*>(d) = hi;
+      *reinterpret_cast<__nv_bfloat16*>(d + 8) = lo;
+    };
+    const int step = c / 16, col = c % 16, k_tile = 4 * (p.dk / 16) + c / 8;
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      float s = q[i][r] * e[r];
+#pragma unroll
+      for (int j = 0; j <= r; ++j) s -= sP[r][j] * w[j];
+      put(4 * step + r / 8, r % 8, col, w[r]);
+      put(4 * step + 2 + r / 8, r % 8, col, s);
+      put(k_tile, c % 8, r, k[i][r] * fast_exp2((G[i][DC_T - 1] - G[i][r]) * LOG2E));
+    }
+  }
+  // ---- T V and P T V of this thread's value columns ----
+  float* uo = p.uo + block * dc_uo_floats(VP);
+  for (int c = tid; c < VP; c += DC_THREADS) {
+    float v[DC_T], u[DC_T];
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) v[r] = r < n ? __bfloat162float(x[(size_t)r * a.ld_qkv + off_v + h * VP + c]) : 0.f;
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      float s = 0.f;
+#pragma unroll
+      for (int j = 0; j <= r; ++j) s += sT[r][j] * v[j];
+      u[r] = s;
+    }
+    float* dst = uo + (c / 16) * 512 + ((c & 7) * 4) * 4 + ((c & 15) >> 3) * 2;      // [2][2 row tiles][lane = column % 8, row pair][column half, row]
+#pragma unroll
+    for (int r = 0; r < DC_T; r += 2) {
+      float o0 = 0.f, o1 = 0.f;
+#pragma unroll
+      for (int j = 0; j <= r; ++j) o0 += sP[r][j] * u[j];
+#pragma unroll
+      for (int j = 0; j <= r + 1; ++j) o1 += sP[r + 1][j] * u[j];
+      const int o = (r / 8) * 128 + ((r % 8) / 2) * 4;
+      *reinterpret_cast<float2*>(dst + o) = make_float2(u[r], u[r + 1]);
+      *reinterpret_cast<float2*>(dst + 256 + o) = make_float2(o0, o1);
+    }
+  }
+  __syncthreads();
+  const int vecs = dc_block_bytes(p.dk) / 16;
+  uint4* out = reinterpret_cast<uint4*>(p.blocks + block * dc_block_bytes(p.dk));
+  for (int i = tid; i < vecs; i += DC_THREADS) out[i] = reinterpret_cast<const uint4*>(stage)[i];
+}
+
+__device__ __forceinline__ void dc_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void dc_bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
+
+// KS: warps that share a head's key channels, 64 each; the CTA's four warps take 4 / KS tiles of 16 value columns
+template <int KS>
+__global__ void __launch_bounds__(128)
+delta_scan_kernel(const DeltaChunkParams p) {
+  constexpr int DK = 64 * KS, TILES = 4 / KS, BLOCK = dc_block_bytes(DK);
+  extern __shared__ __align__(128) unsigned char dc_smem[];       // [DC_STAGES][BLOCK], then the partial sums [2][4 warps][16][32]
+  __shared__ __align__(8) uint64_t bar_full[DC_STAGES];
+  __shared__ int cta_abort_s;
+  volatile int* cta_abort = &cta_abort_s;
+  const nfn_delta_args& a = p.a;
+  const nfn_seq_rows seq = a.seqs[blockIdx.z];
+  const int total = (seq.n + DC_T - 1) / DC_T, n_chunks = min(p.n_chunks, total - p.chunk0);
+  if (seq.slot < 0 || n_chunks <= 0) return;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, j = lane & 3;
+  const int ks = warp % KS, h = blockIdx.y, DP = a.dim_p, VP = a.vdim_p;
+  const int vt = blockIdx.x * TILES + warp / KS;
+  const bool on = vt * 16 < VP;                                   // warps past the last column tile keep the others company
+  float* xch = reinterpret_cast<float*>(dc_smem + DC_STAGES * BLOCK);
+  const unsigned char* blocks = p.blocks + ((size_t)blockIdx.z * p.n_chunks * a.heads + h) * BLOCK;
+  const size_t block_step = (size_t)a.heads * BLOCK;
+  const float* uo = p.uo + ((size_t)blockIdx.z * p.n_chunks * a.heads + h) * dc_uo_floats(VP) + (on ? vt : 0) * 512 + lane * 4;
+  const size_t uo_step = (size_t)a.heads * dc_uo_floats(VP);
+
+  auto load = [&](int i) {
+    const uint32_t bar = smem_u32(&bar_full[i % DC_STAGES]);
+    mbar_expect_tx(bar, BLOCK);
+    dc_bulk_load(smem_u32(dc_smem + (i % DC_STAGES) * BLOCK), blocks + i * block_step, BLOCK, bar);
+  };
+  if (tid == 0) {
+    cta_abort_s = 0;
+    for (int s = 0; s < DC_STAGES; ++s) mbar_init(smem_u32(&bar_full[s]), 1);
+    fence_mbar_init();
+    for (int i = 0; i < min(DC_STAGES, n_chunks); ++i) load(i);
+  }
+  // S^T: rows are value columns (g, g + 8), columns key channels 64 ks + 8 t + 2 j, + 1
+  float* st = a.state + ((size_t)seq.slot * a.heads + h) * DP * VP + vt * 16 + g;
+  const bool fresh = seq.pos0 == 0 && p.chunk0 == 0;
+  float s[8][4];
+#pragma unroll
+  for (int t = 0; t < 8; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = 64 * ks + 8 * t + 2 * j + (e & 1);
+      s[t][e] = (on && !fresh && d < DP) ? st[(size_t)d * VP + (e >> 1) * 8] : 0.f;
+    }
+  float u_next[2][4], o_next[2][4];
+  auto fetch = [&](int i) {
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      const float4 u = *reinterpret_cast<const float4*>(uo + i * uo_step + nt * 128), o = *reinterpret_cast<const float4*>(uo + i * uo_step + 256 + nt * 128);
+      u_next[nt][0] = u.x; u_next[nt][1] = u.y; u_next[nt][2] = u.z; u_next[nt][3] = u.w;
+      o_next[nt][0] = o.x; o_next[nt][1] = o.y; o_next[nt][2] = o.z; o_next[nt][3] = o.w;
+    }
+  };
+  fetch(0);
+  __syncthreads();
+  bool ok = true;
+  for (int i = 0; i < n_chunks; ++i) {
+    float u[2][4], o[2][4];
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        u[nt][e] = u_next[nt][e];
+        o[nt][e] = o_next[nt][e];
+      }
+    if (i + 1 < n_chunks) fetch(i + 1);
+    ok = mbar_wait_bounded(smem_u32(&bar_full[i % DC_STAGES]), (i / DC_STAGES) & 1, cta_abort, p.status, NFN_ERR_WAIT_FULL);
+    const unsigned char* stage = dc_smem + (i % DC_STAGES) * BLOCK;
+    float acc[4][4], low[4][4];                          // (W S)^T row tiles 0, 1, then (Q S)^T: high x high, and the products with a low part
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[nt][e] = low[nt][e] = 0.f;
+    if (ok) {
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        uint32_t hi[4], lo[4];
+        split_bf16(s[2 * kk][0], s[2 * kk][1], hi[0], lo[0]);
+        split_bf16(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
+        split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lo[2]);
+        split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) {
+          const uint4 b = *reinterpret_cast<const uint4*>(stage + ((size_t)((4 * ks + kk) * 4 + nt) * 32 + lane) * 16);
+          dc_mma(acc[nt], hi, b.x, b.y);
+          dc_mma(low[nt], hi, b.z, b.w);
+          dc_mma(low[nt], lo, b.x, b.y);
+        }
+      }
+    }
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[nt][e] += low[nt][e];
+    if (KS > 1) {
+      float* mine = xch + ((i & 1) * 4 + warp) * 512 + lane * 4;
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) *reinterpret_cast<float4*>(mine + nt * 128) = make_float4(acc[nt][0], acc[nt][1], acc[nt][2], acc[nt][3]);
+    }
+    // every warp is done with chunk i - 1 here: its stage takes the next load
+    if (!__syncthreads_and(ok)) break;
+    if (tid == 0 && i > 0 && i - 1 + DC_STAGES < n_chunks) load(i - 1 + DC_STAGES);
+    if (KS > 1) {
+      const float* all = xch + ((i & 1) * 4 + warp / KS * KS) * 512 + lane * 4;
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) {
+        float4 t = *reinterpret_cast<const float4*>(all + nt * 128);
+#pragma unroll
+        for (int w = 1; w < KS; ++w) {
+          const float4 b = *reinterpret_cast<const float4*>(all + w * 512 + nt * 128);
+          t.x += b.x; t.y += b.y; t.z += b.z; t.w += b.w;
+        }
+        acc[nt][0] = t.x; acc[nt][1] = t.y; acc[nt][2] = t.z; acc[nt][3] = t.w;
+      }
+    }
+    // U^T, as the A operand of S'^T = e^G_last S^T + U^T K
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) u[nt][e] -= acc[nt][e];
+    uint32_t uh[4], ul[4];
+    split_bf16(u[0][0], u[0][1], uh[0], ul[0]);
+    split_bf16(u[0][2], u[0][3], uh[1], ul[1]);
+    split_bf16(u[1][0], u[1][1], uh[2], ul[2]);
+    split_bf16(u[1][2], u[1][3], uh[3], ul[3]);
+    const float* gamma = reinterpret_cast<const float*>(stage + 48 * DK * 4) + 64 * ks + 2 * j;
+#pragma unroll
+    for (int t = 0; t < 8; ++t) {
+      const float2 f = *reinterpret_cast<const float2*>(gamma + 8 * t);
+      const uint4 b = *reinterpret_cast<const uint4*>(stage + ((size_t)(4 * (DK / 16) + 8 * ks + t) * 32 + lane) * 16);
+      s[t][0] *= f.x; s[t][1] *= f.y; s[t][2] *= f.x; s[t][3] *= f.y;
+      dc_mma(s[t], uh, b.x, b.y);
+      dc_mma(s[t], uh, b.z, b.w);
+      dc_mma(s[t], ul, b.x, b.y);
+    }
+    // read-outs: the warps of a column tile take the row tiles in turn
+    const int r0 = (p.chunk0 + i) * DC_T;
+    float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g;
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt) {
+      if (!on || nt % KS != ks) continue;
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int r = 8 * nt + 2 * j + (e & 1);
+        if (r0 + r < seq.n) dst[(size_t)r * a.ld_o + (e >> 1) * 8] = o[nt][e] + acc[2 + nt][e];
+      }
+    }
+  }
+  if (*cta_abort) {
+    for (int i = 0; i < 64; ++i) __nanosleep(1000);     // copies in flight land
+    return;
+  }
+  if (!on) return;
+#pragma unroll
+  for (int t = 0; t < 8; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = 64 * ks + 8 * t + 2 * j + (e & 1);
+      if (d < DP) st[(size_t)d * VP + (e >> 1) * 8] = s[t][e];
+    }
+}
+
+template <int KS>
+static int launch_scan(const DeltaChunkParams& p, cudaStream_t st) {
+  constexpr int SMEM = DC_STAGES * dc_block_bytes(64 * KS) + 2 * 4 * 512 * 4;
+  auto kern = delta_scan_kernel<KS>;
+  static bool raised[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (SMEM > 48 * 1024 && !raised[dev & 63]) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return launch_check("delta_scan attr", 0);
+    raised[dev & 63] = true;
+  }
+  kern<<<dim3(ceil_div(p.a.vdim_p, 16 * (4 / KS)), p.a.heads, p.a.n_seqs), 128, SMEM, st>>>(p);
+  return launch_check("delta_scan");
+}
+
+template <int NCH>
+static int launch_prepare(const DeltaChunkParams& p, cudaStream_t st) {
+  const int smem = std::max(64 * DC_PITCH * 4, dc_block_bytes(p.dk));
+  auto kern = delta_prepare_kernel<NCH>;
+  static int raised[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (smem > 40 * 1024 && raised[dev & 63] < smem) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return launch_check("delta_prepare attr", 0);
+    raised[dev & 63] = smem;
+  }
+  kern<<<dim3(p.n_chunks, p.a.heads, p.a.n_seqs), DC_THREADS, smem, st>>>(p);
+  return launch_check("delta_prepare");
+}
+
+}  // namespace nfn
+
+using namespace nfn;
+
+extern "C" long long nfn_delta_chunk_workspace_bytes(int heads, int dim_p, int vdim_p, int max_seqs) {
+  if (dim_p > 256) return 0;
+  const int dk = dim_p <= 64 ? 64 : dim_p <= 128 ? 128 : 256;
+  // at least one chunk of every head and sequence
+  return std::max<long long>(DC_WORKSPACE, (long long)max_seqs * heads * (dc_block_bytes(dk) + dc_uo_floats(vdim_p) * 4LL));
+}
+
+extern "C" int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* workspace, long long workspace_bytes, nfn_stream_t stream) {
+  if (!args) return fail(-1, "delta rule: null args");
+  if (args->n_seqs <= 0 || max_rows <= 0) return 0;
+  if (const char* why = delta_args_problem(*args)) return fail(-1, why);
+  if (args->f32 || args->dim_p > 256) return fail(-1, "delta rule: chunks are for bf16 activations and at most 256 key channels");
+  DeltaChunkParams p;
+  p.a = *args;
+  p.dk = args->dim_p <= 64 ? 64 : args->dim_p <= 128 ? 128 : 256;
+  p.status = status_ptr();
+  const long long per_chunk = (long long)args->n_seqs * args->heads * (dc_block_bytes(p.dk) + dc_uo_floats(args->vdim_p) * 4LL);
+  const int total = ceil_div(max_rows, DC_T), round = (int)std::min<long long>(total, workspace_bytes / per_chunk);
+  if (!workspace || round < 1) return fail(-1, "delta rule: the workspace holds no chunk");
+  p.blocks = static_cast<unsigned char*>(workspace);
+  p.uo = reinterpret_cast<float*>(p.blocks + (size_t)round * args->n_seqs * args->heads * dc_block_bytes(p.dk));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  for (p.chunk0 = 0; p.chunk0 < total; p.chunk0 += round) {
+    p.n_chunks = std::min(round, total - p.chunk0);
+    int rc = p.dk <= 128 ? launch_prepare<1>(p, st) : launch_prepare<2>(p, st);
+    if (rc == 0) rc = p.dk == 64 ? launch_scan<1>(p, st) : p.dk == 128 ? launch_scan<2>(p, st) : launch_scan<4>(p, st);
+    if (rc) return rc;
+  }
+  return 0;
+}

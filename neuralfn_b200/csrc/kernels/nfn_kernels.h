@@ -418,6 +418,9 @@ typedef struct {
   const nfn_seq_rows* seqs; int n_seqs;
 } nfn_delta_args;
 int nfn_delta_rows(const nfn_delta_args* args, nfn_stream_t stream);     // token after token, any length
+// Sixteen tokens at a time on the tensor cores (bf16, dim_p <= 256), for sequences of up to max_rows rows.
+long long nfn_delta_chunk_workspace_bytes(int heads, int dim_p, int vdim_p, int max_seqs);   // 0: these sizes go token after token
+int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* workspace, long long workspace_bytes, nfn_stream_t stream);
 // out = o / rms(o) * weight * sigmoid(gate) per head of vdim values (pitch vdim_p); weight bf16 [vdim_p], out and gate in the activation type.
 int nfn_delta_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, float eps, void* out, int ld_out, int rows,
                   int heads, int vdim, int vdim_p, nfn_stream_t stream);

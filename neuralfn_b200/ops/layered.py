@@ -51,14 +51,21 @@ def stream_pass(x: torch.Tensor | None, h: torch.Tensor | None, *, width: int, s
 
 
 def delta_rule(qkv: torch.Tensor, beta: torch.Tensor, decay: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, *,
-               kv_heads: int, dim: int, unit_eps: float = 1e-6, form: str = "rows") -> torch.Tensor:
+               kv_heads: int, dim: int, unit_eps: float = 1e-6, form: str = "rows", workspace: torch.Tensor | None = None, longest: int = 0) -> torch.Tensor:
     """qkv [rows, 2 * kv_heads * dim_p + heads * vdim_p] after convolution and activation (bf16 or fp32), beta [rows, heads], decay fp32 [rows, heads * dim_p],
-    state fp32 [slots, heads, dim_p, vdim_p], seqs int32 [n, 4] = first row, rows, slot, position. Returns the read-outs, fp32 [rows, heads * vdim_p]."""
+    state fp32 [slots, heads, dim_p, vdim_p], seqs int32 [n, 4] = first row, rows, slot, position. Returns the read-outs, fp32 [rows, heads * vdim_p].
+    form: "rows" (token after token) or "chunks" (sixteen at a time, bf16; ``longest``: most rows of a sequence)."""
     _, heads, dim_p, vdim_p = state.shape
     o = torch.zeros(qkv.shape[0], heads * vdim_p, device=qkv.device)
     a = _Delta(int(qkv.dtype == torch.float32), _p(qkv), qkv.stride(0), _p(beta), beta.stride(0), _p(decay), decay.stride(0), _p(a_log), _p(dt_bias), heads, kv_heads, dim,
                dim_p, vdim_p, unit_eps, _p(state), _p(o), o.stride(0), _p(seqs), seqs.shape[0])
-    _call("delta_rows", a)
+    if form == "rows":
+        _call("delta_rows", a)
+        return o
+    lib = _lib.load()
+    lib.nfn_delta_chunk_workspace_bytes.restype = C.c_longlong
+    ws = workspace if workspace is not None else torch.empty(lib.nfn_delta_chunk_workspace_bytes(heads, dim_p, vdim_p, seqs.shape[0]), device=qkv.device, dtype=torch.uint8)
+    _lib.check(lib.nfn_delta_chunks(C.byref(a), C.c_int(longest or qkv.shape[0]), C.c_void_p(_p(ws)), C.c_longlong(ws.numel()), C.c_void_p(_lib.stream_ptr())), "delta_chunks")
     return o
 
 
