@@ -6,8 +6,8 @@
 // S' = e^G_last S + K^T U with K_j = k_j e^(G_last - G_j). Every exponent is a sum of decays between two tokens, never positive, so
 // nothing overflows however fast a channel forgets.
 //
-//   delta_prepare_kernel  one CTA per (chunk, head), all chunks at once: W, Q, K and T V, P T V. A thread owns a channel; products of
-//                         a channel with all pairs of tokens stay in its registers and are summed over channels through shared memory.
+//   delta_prepare_kernel  one CTA per (chunk, head), all chunks at once: W, Q, K and T V, P T V. A thread owns two channels; their
+//                         products for all pairs of tokens are formed in registers and summed over channels through shared memory.
 //   delta_scan_kernel     one warp per (head, 16 value columns, 64 key channels), one chunk after another: the state, transposed, sits in
 //                         the accumulator registers of mma.m16n8k16 and is the A operand of the next chunk's W S and Q S as it stands; W, Q
 //                         and K arrive in fragment order by bulk copies through a ring of shared memory stages.
@@ -23,7 +23,6 @@
 namespace nfn {
 
 constexpr int DC_T = 16;                               // tokens of a chunk
-constexpr int DC_THREADS = 128, DC_PITCH = 130;        // partial sums: [64 values][128 threads], two threads read a row without conflicts
 constexpr int DC_STAGES = 3;
 constexpr long long DC_WORKSPACE = 96LL << 20;
 
@@ -48,12 +47,29 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
   lo = pack_bf16x2(a - f.x, b - f.y);
 }
 
-// NCH: channels per thread (key or value channels up to 128 NCH)
-template <int NCH>
-__global__ void __launch_bounds__(DC_THREADS)
+// log2(1 + e^z): the series of log(1 + t) for small t = e^z keeps slow decays exact
+__device__ __forceinline__ float softplus_log2(float z) {
+  const float y = z * 1.4426950408889634f, t = fast_exp2(y);
+  const float s = t * (1.f - t * (0.5f - t * (0.33333333f - t * (0.25f - t * (0.2f - t * (0.16666667f - t * 0.14285714f))))));
+  const float l = t < 0.125f ? s * 1.4426950408889634f : __log2f(1.f + t);
+  return y > 28.f ? y : l;
+}
+
+// Where the 16-byte piece of lane `lane` lies inside operand tile `tile` of a block: the order keeps the writers of both kinds of tile, and
+// the scan's reads, on different banks.
+__device__ __forceinline__ uint32_t dc_piece(int tile, int lane, bool of_k) {
+  const int turn = of_k ? ((lane >> 3) & 3) | ((tile & 1) << 2) : ((tile >> 2) & 1) << 2;
+  return (uint32_t)(tile * 32 + (lane ^ turn)) * 16;
+}
+
+// NT threads, two neighbouring key channels each (dk = 2 NT), and value columns in pairs
+template <int NT>
+__global__ void __launch_bounds__(NT, 384 / NT)
 delta_prepare_kernel(const DeltaChunkParams p) {
-  extern __shared__ __align__(128) unsigned char dc_smem[];        // partial sums, then the operand block
-  __shared__ float sA[DC_T][DC_T + 4], sP[DC_T][DC_T + 4], sT[DC_T][DC_T + 4], s_norm[2][DC_T], s_beta[DC_T];
+  constexpr int PITCH = NT == 128 ? 136 : NT + 4;                 // partial sums [64 values][NT]; rows are read in 16-byte pieces
+  extern __shared__ __align__(128) unsigned char dc_smem[];       // partial sums, then the operand block
+  __shared__ __align__(16) float sA[DC_T][DC_T + 4], sP[DC_T][DC_T + 4], sT[DC_T][DC_T + 4];
+  __shared__ float s_norm[2][DC_T], s_beta[DC_T];
   const nfn_delta_args& a = p.a;
   const nfn_seq_rows seq = a.seqs[blockIdx.z];
   const int r0 = (p.chunk0 + blockIdx.x) * DC_T, n = min(DC_T, seq.n - r0);
@@ -63,57 +79,65 @@ delta_prepare_kernel(const DeltaChunkParams p) {
   const int off_k = a.kv_heads * DP, off_v = 2 * off_k;
   const size_t row0 = (size_t)(seq.row0 + r0);
   const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(a.qkv) + row0 * a.ld_qkv;
+  const int c0 = 2 * tid;
+  const bool on = c0 < DP;
 
-  // ---- unit vectors, step sizes ----
-  for (int r = warp; r < DC_T; r += DC_THREADS / 32) {
-    float nq = 0.f, nk = 0.f;
-    if (r < n)
-      for (int d = lane * 2; d < DP; d += 64) {
-        const float2 q = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + (size_t)r * a.ld_qkv + hk * DP + d));
-        const float2 k = unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + (size_t)r * a.ld_qkv + off_k + hk * DP + d));
-        nq += q.x * q.x + q.y * q.y;
-        nk += k.x * k.x + k.y * k.y;
-      }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      nq += __shfl_xor_sync(0xffffffffu, nq, o);
-      nk += __shfl_xor_sync(0xffffffffu, nk, o);
-    }
-    if (lane == 0) {
-      s_norm[0][r] = 1.f / (sqrtf((float)a.dim) * sqrtf(nq + a.unit_eps));
-      s_norm[1][r] = 1.f / sqrtf(nk + a.unit_eps);
-      s_beta[r] = r < n ? sigmoid_exact(__bfloat162float(static_cast<const __nv_bfloat16*>(a.beta)[(row0 + r) * a.ld_beta + h])) : 0.f;
-    }
-  }
-  __syncthreads();
-  // ---- this thread's channels: q, k and the running sum of log decays ----
-  float q[NCH][DC_T], k[NCH][DC_T], G[NCH][DC_T];
-  const float rate = -expf(__bfloat162float(static_cast<const __nv_bfloat16*>(a.a_log)[h]));
-#pragma unroll
-  for (int i = 0; i < NCH; ++i) {
-    const int c = tid + i * DC_THREADS;
-    const bool on = c < DP;
-    const float bias = on ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.dt_bias)[(size_t)h * DP + c]) : 0.f;
-    float raw[DC_T];
+  // ---- this thread's channels; unit vectors, step sizes ----
+  float q[DC_T][2], k[DC_T][2], G[DC_T][2];
+  {
+    uint32_t qw[DC_T], kw[DC_T];
 #pragma unroll
     for (int r = 0; r < DC_T; ++r) {
       const bool live = on && r < n;
-      q[i][r] = live ? __bfloat162float(x[(size_t)r * a.ld_qkv + hk * DP + c]) : 0.f;
-      k[i][r] = live ? __bfloat162float(x[(size_t)r * a.ld_qkv + off_k + hk * DP + c]) : 0.f;
-      raw[r] = live ? a.decay[(row0 + r) * a.ld_decay + (size_t)h * DP + c] : 0.f;
+      qw[r] = live ? *reinterpret_cast<const uint32_t*>(x + (size_t)r * a.ld_qkv + hk * DP + c0) : 0u;
+      kw[r] = live ? *reinterpret_cast<const uint32_t*>(x + (size_t)r * a.ld_qkv + off_k + hk * DP + c0) : 0u;
+      const float2 z = live ? *reinterpret_cast<const float2*>(a.decay + (row0 + r) * a.ld_decay + (size_t)h * DP + c0) : make_float2(0.f, 0.f);
+      G[r][0] = z.x;
+      G[r][1] = z.y;
     }
-    float sum = 0.f;
+    float* red = reinterpret_cast<float*>(dc_smem);               // [32 sums][warps]
 #pragma unroll
     for (int r = 0; r < DC_T; ++r) {
-      q[i][r] *= s_norm[0][r];
-      k[i][r] *= s_norm[1][r];
-      if (on && r < n) sum += delta_log_decay(raw[r] + bias, rate);
-      G[i][r] = sum;
+      const float2 fq = unpack_bf16x2(qw[r]), fk = unpack_bf16x2(kw[r]);
+      q[r][0] = fq.x; q[r][1] = fq.y; k[r][0] = fk.x; k[r][1] = fk.y;
+      float nq = fq.x * fq.x + fq.y * fq.y, nk = fk.x * fk.x + fk.y * fk.y;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1) {
+        nq += __shfl_xor_sync(0xffffffffu, nq, o);
+        nk += __shfl_xor_sync(0xffffffffu, nk, o);
+      }
+      if (lane == r) red[r * (NT / 32) + warp] = nq;
+      if (lane == 16 + r) red[(16 + r) * (NT / 32) + warp] = nk;
+    }
+    __syncthreads();
+    if (tid < 2 * DC_T) {
+      float t = 0.f;
+#pragma unroll
+      for (int w = 0; w < NT / 32; ++w) t += red[tid * (NT / 32) + w];
+      const float f = 1.f / sqrtf(t + a.unit_eps);
+      s_norm[tid / DC_T][tid % DC_T] = tid < DC_T ? f / sqrtf((float)a.dim) : f;
+      if (tid < DC_T) s_beta[tid] = tid < n ? sigmoid_exact(__bfloat162float(static_cast<const __nv_bfloat16*>(a.beta)[(row0 + tid) * a.ld_beta + h])) : 0.f;
+    }
+    __syncthreads();
+  }
+  {
+    const float rate = -expf(__bfloat162float(static_cast<const __nv_bfloat16*>(a.a_log)[h]));
+    const float2 bias = on ? unpack_bf16x2(*reinterpret_cast<const uint32_t*>(static_cast<const __nv_bfloat16*>(a.dt_bias) + (size_t)h * DP + c0)) : make_float2(0.f, 0.f);
+    float s0 = 0.f, s1 = 0.f;                                     // sums of log2 decays
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      const float fq = s_norm[0][r], fk = s_norm[1][r];
+      q[r][0] *= fq; q[r][1] *= fq; k[r][0] *= fk; k[r][1] *= fk;
+      if (r < n) {
+        s0 += rate * softplus_log2(G[r][0] + bias.x);
+        s1 += rate * softplus_log2(G[r][1] + bias.y);
+      }
+      G[r][0] = s0;
+      G[r][1] = s1;
     }
   }
   // ---- A and P: rows 2t, 15 - 2t, 2t + 1, 14 - 2t together have 64 values ----
   float* part = reinterpret_cast<float*>(dc_smem);
-  const float LOG2E = 1.4426950408889634f;
 #pragma unroll
   for (int t = 0; t < 4; ++t) {
     const int rows[4] = {2 * t, 15 - 2 * t, 2 * t + 1, 14 - 2 * t};
@@ -124,125 +148,138 @@ delta_prepare_kernel(const DeltaChunkParams p) {
 #pragma unroll
       for (int j = 0; j < DC_T; ++j) {
         if (j > r) continue;
-        float va = 0.f, vp = 0.f;
-#pragma unroll
-        for (int i = 0; i < NCH; ++i) {
-          const float kj = j < r ? k[i][j] * fast_exp2((G[i][r] - G[i][j]) * LOG2E) : k[i][j];
-          va += k[i][r] * kj;
-          vp += q[i][r] * kj;
+        float k0 = k[j][0], k1 = k[j][1];
+        if (j < r) {
+          k0 *= fast_exp2(G[r][0] - G[j][0]);
+          k1 *= fast_exp2(G[r][1] - G[j][1]);
         }
-        part[at++ * DC_PITCH + tid] = vp;
-        if (j < r) part[at++ * DC_PITCH + tid] = va;
+        part[at++ * PITCH + tid] = q[r][0] * k0 + q[r][1] * k1;
+        if (j < r) part[at++ * PITCH + tid] = k[r][0] * k0 + k[r][1] * k1;
       }
     }
     __syncthreads();
-    {
-      // value `v` of the pass is summed by two threads, one per parity of the channel
-      const int v = tid >> 1;
-      float s0 = 0.f, s1 = 0.f;
-      const float* src = part + v * DC_PITCH + (tid & 1);
-#pragma unroll 8
-      for (int i = 0; i < DC_THREADS / 2; i += 2) {
-        s0 += src[2 * i];
-        s1 += src[2 * i + 2];
+    // every thread sums 64 numbers: two values (NT = 32), one (64) or half of one (128)
+#pragma unroll
+    for (int v0 = 0; v0 < (NT == 32 ? 64 : 32); v0 += 32) {
+      const int v = NT == 32 ? tid + v0 : NT == 64 ? tid : tid >> 1;
+      const float* src = part + v * PITCH + (NT == 128 ? 4 * (tid & 1) : 0);
+      float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+      for (int i = 0; i < (NT == 32 ? 8 : 16); ++i) {
+        const float4 f = *reinterpret_cast<const float4*>(src + i * (NT == 128 ? 8 : 4));
+        s.x += f.x; s.y += f.y; s.z += f.z; s.w += f.w;
       }
-      float s = s0 + s1;
-      s += __shfl_xor_sync(0xffffffffu, s, 1);
+      float sum = (s.x + s.y) + (s.z + s.w);
+      if (NT == 128) sum += __shfl_xor_sync(0xffffffffu, sum, 1);
       // where it belongs: the rows of the pass hold 2 r + 1 values each, P_rj and A_rj in turn
       int rest = v, r = rows[0];
       if (rest >= 2 * r + 1) { rest -= 2 * r + 1; r = rows[1];
         if (rest >= 2 * r + 1) { rest -= 2 * r + 1; r = rows[2];
           if (rest >= 2 * r + 1) { rest -= 2 * r + 1; r = rows[3]; } } }
-      if ((tid & 1) == 0) ((rest & 1) ? sA : sP)[r][rest >> 1] = s;
+      ((rest & 1) ? sA : sP)[r][rest >> 1] = sum;
+      if (NT != 32) break;
     }
     __syncthreads();
   }
+  // powers of the decays are formed again below instead of being kept in registers
+#pragma unroll
+  for (int r = 0; r < DC_T; ++r) asm volatile("" : "+f"(G[r][0]), "+f"(G[r][1]));
   // ---- T = (I + diag(beta) A)^-1 diag(beta): one column per lane, forward substitution ----
   if (tid < DC_T) {
     float y[DC_T];
 #pragma unroll
     for (int r = 0; r < DC_T; ++r) {
-      float s = r == tid ? 1.f : 0.f;
-      const float b = s_beta[r];
+      float s0 = 0.f, s1 = 0.f;
 #pragma unroll
-      for (int i = 0; i < r; ++i) s -= b * sA[r][i] * y[i];
-      y[r] = s;
+      for (int i = 0; i < r; ++i) ((i & 1) ? s1 : s0) += sA[r][i] * y[i];
+      y[r] = (r == tid ? 1.f : 0.f) - s_beta[r] * (s0 + s1);
     }
     const float b = s_beta[tid];
 #pragma unroll
     for (int r = 0; r < DC_T; ++r) sT[r][tid] = y[r] * b;
   }
   __syncthreads();
+  // rows of T and P times two columns at once
+  auto lower = [](const float (&m)[DC_T + 4], const float (&v)[DC_T][2], int last, float& o0, float& o1) {
+#pragma unroll
+    for (int j4 = 0; j4 <= last; j4 += 4) {
+      const float4 f = *reinterpret_cast<const float4*>(&m[j4]);
+      const float t[4] = {f.x, f.y, f.z, f.w};
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        if (j4 + e <= last) fma2(o0, o1, t[e], t[e], v[j4 + e][0], v[j4 + e][1], o0, o1);
+    }
+  };
   const size_t block = ((size_t)blockIdx.z * p.n_chunks + blockIdx.x) * a.heads + h;
-  // ---- W, Q, K of this thread's key channels, in the order of the scan's fragments ----
+  // ---- W, Q, K of this thread's key channels, in the order of the scan's fragments: {first eight of the contraction: high, low; second: high, low} ----
   unsigned char* stage = dc_smem;
-  float* gamma = reinterpret_cast<float*>(stage + 48 * p.dk * 4);
+  *reinterpret_cast<float2*>(stage + 48 * p.dk * 4 + c0 * 4) = make_float2(fast_exp2(G[DC_T - 1][0]), fast_exp2(G[DC_T - 1][1]));
 #pragma unroll
-  for (int i = 0; i < NCH; ++i) {
-    const int c = tid + i * DC_THREADS;
-    if (c >= p.dk) continue;
-    float e[DC_T], w[DC_T];
+  for (int r = 0; r < DC_T; r += 2)
 #pragma unroll
-    for (int r = 0; r < DC_T; ++r) e[r] = fast_exp2(G[i][r] * LOG2E);
-    gamma[c] = e[DC_T - 1];
-#pragma unroll
-    for (int r = 0; r < DC_T; ++r) {
-      float s = 0.f;
-#pragma unroll
-      for (int j = 0; j <= r; ++j) s += sT[r][j] * (k[i][j] * e[j]);
-      w[r] = s;
+    for (int i = 0; i < 2; ++i) {
+      uint2 w;
+      split_bf16(k[r][i] * fast_exp2(G[DC_T - 1][i] - G[r][i]), k[r + 1][i] * fast_exp2(G[DC_T - 1][i] - G[r + 1][i]), w.x, w.y);
+      *reinterpret_cast<uint2*>(stage + dc_piece(4 * (p.dk / 16) + (c0 + i) / 8, (c0 + i) % 8 * 4 + (r % 8) / 2, true) + (r / 8) * 8) = w;
     }
-    auto put = [&](int tile, int row, int col, float v) {      // element (row, col) of a 8 x 16 operand tile: high and low part
-      const __nv_bfloat16 hi = __float2bfloat16(v), lo = __float2bfloat16(v - __bfloat162float(hi));
-      unsigned char* d = stage + ((size_t)(tile * 32 + row * 4 + ((col & 7) >> 1)) * 16 + (col >> 3) * 4 + (col & 1) * 2);
-      *reinterpret_cast<__nv_bfloat16*>(d) = hi;
-      *reinterpret_cast<__nv_bfloat16*>(d + 8) = lo;
-    };
-    const int step = c / 16, col = c % 16, k_tile = 4 * (p.dk / 16) + c / 8;
+  float w[DC_T][2];
 #pragma unroll
-    for (int r = 0; r < DC_T; ++r) {
-      float s = q[i][r] * e[r];
-#pragma unroll
-      for (int j = 0; j <= r; ++j) s -= sP[r][j] * w[j];
-      put(4 * step + r / 8, r % 8, col, w[r]);
-      put(4 * step + 2 + r / 8, r % 8, col, s);
-      put(k_tile, c % 8, r, k[i][r] * fast_exp2((G[i][DC_T - 1] - G[i][r]) * LOG2E));
-    }
+  for (int r = 0; r < DC_T; ++r) {
+    const float e0 = fast_exp2(G[r][0]), e1 = fast_exp2(G[r][1]);
+    q[r][0] *= e0; q[r][1] *= e1; k[r][0] *= e0; k[r][1] *= e1;
   }
+#pragma unroll
+  for (int r = 0; r < DC_T; ++r) {
+    w[r][0] = w[r][1] = 0.f;
+    lower(sT[r], k, r, w[r][0], w[r][1]);
+    float p0 = 0.f, p1 = 0.f;
+    lower(sP[r], w, r, p0, p1);
+    uint2 f;
+    const uint32_t half = ((c0 % 16) / 8) * 8;
+    const int piece_lane = r % 8 * 4 + (c0 % 8) / 2;
+    split_bf16(w[r][0], w[r][1], f.x, f.y);
+    *reinterpret_cast<uint2*>(stage + dc_piece(4 * (c0 / 16) + r / 8, piece_lane, false) + half) = f;
+    split_bf16(q[r][0] - p0, q[r][1] - p1, f.x, f.y);
+    *reinterpret_cast<uint2*>(stage + dc_piece(4 * (c0 / 16) + 2 + r / 8, piece_lane, false) + half) = f;
+  }
+  asm volatile("" ::: "memory");                                 // T and P are read again, not kept in registers
   // ---- T V and P T V of this thread's value columns ----
   float* uo = p.uo + block * dc_uo_floats(VP);
-  for (int c = tid; c < VP; c += DC_THREADS) {
-    float v[DC_T], u[DC_T];
-#pragma unroll
-    for (int r = 0; r < DC_T; ++r) v[r] = r < n ? __bfloat162float(x[(size_t)r * a.ld_qkv + off_v + h * VP + c]) : 0.f;
+  for (int c = c0; c < VP; c += 2 * NT) {
+    float v[DC_T][2], u[DC_T][2];
 #pragma unroll
     for (int r = 0; r < DC_T; ++r) {
-      float s = 0.f;
-#pragma unroll
-      for (int j = 0; j <= r; ++j) s += sT[r][j] * v[j];
-      u[r] = s;
+      const float2 f = r < n ? unpack_bf16x2(*reinterpret_cast<const uint32_t*>(x + (size_t)r * a.ld_qkv + off_v + h * VP + c)) : make_float2(0.f, 0.f);
+      v[r][0] = f.x;
+      v[r][1] = f.y;
     }
-    float* dst = uo + (c / 16) * 512 + ((c & 7) * 4) * 4 + ((c & 15) >> 3) * 2;      // [2][2 row tiles][lane = column % 8, row pair][column half, row]
+#pragma unroll
+    for (int r = 0; r < DC_T; ++r) {
+      u[r][0] = u[r][1] = 0.f;
+      lower(sT[r], v, r, u[r][0], u[r][1]);
+    }
+    float* dst = uo + (c / 16) * 512 + (c & 7) * 16 + ((c & 15) >> 3) * 2;      // [2][2 row tiles][lane = column % 8, row pair][column half, row]
 #pragma unroll
     for (int r = 0; r < DC_T; r += 2) {
-      float o0 = 0.f, o1 = 0.f;
+      float o[2][2] = {};
 #pragma unroll
-      for (int j = 0; j <= r; ++j) o0 += sP[r][j] * u[j];
+      for (int e = 0; e < 2; ++e) lower(sP[r + e], u, r + e, o[e][0], o[e][1]);
+      const int at = (r / 8) * 128 + ((r % 8) / 2) * 4;
 #pragma unroll
-      for (int j = 0; j <= r + 1; ++j) o1 += sP[r + 1][j] * u[j];
-      const int o = (r / 8) * 128 + ((r % 8) / 2) * 4;
-      *reinterpret_cast<float2*>(dst + o) = make_float2(u[r], u[r + 1]);
-      *reinterpret_cast<float2*>(dst + 256 + o) = make_float2(o0, o1);
+      for (int i = 0; i < 2; ++i) {
+        *reinterpret_cast<float2*>(dst + i * 16 + at) = make_float2(u[r][i], u[r + 1][i]);
+        *reinterpret_cast<float2*>(dst + i * 16 + 256 + at) = make_float2(o[0][i], o[1][i]);
+      }
     }
   }
   __syncthreads();
   const int vecs = dc_block_bytes(p.dk) / 16;
   uint4* out = reinterpret_cast<uint4*>(p.blocks + block * dc_block_bytes(p.dk));
-  for (int i = tid; i < vecs; i += DC_THREADS) out[i] = reinterpret_cast<const uint4*>(stage)[i];
+  for (int i = tid; i < vecs; i += NT) out[i] = reinterpret_cast<const uint4*>(stage)[i];
 }
 
 __device__ __forceinline__ void dc_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
@@ -319,11 +356,11 @@ delta_scan_kernel(const DeltaChunkParams p) {
     if (i + 1 < n_chunks) fetch(i + 1);
     ok = mbar_wait_bounded(smem_u32(&bar_full[i % DC_STAGES]), (i / DC_STAGES) & 1, cta_abort, p.status, NFN_ERR_WAIT_FULL);
     const unsigned char* stage = dc_smem + (i % DC_STAGES) * BLOCK;
-    float acc[4][4], low[4][4];                          // (W S)^T row tiles 0, 1, then (Q S)^T: high x high, and the products with a low part
+    float acc[4][4], low[4][4], low2[4][4];              // (W S)^T row tiles 0, 1, then (Q S)^T: high x high, high x low, low x high
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc[nt][e] = low[nt][e] = 0.f;
+      for (int e = 0; e < 4; ++e) acc[nt][e] = low[nt][e] = low2[nt][e] = 0.f;
     if (ok) {
 #pragma unroll
       for (int kk = 0; kk < 4; ++kk) {
@@ -332,19 +369,21 @@ delta_scan_kernel(const DeltaChunkParams p) {
         split_bf16(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
         split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lo[2]);
         split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
+        uint4 b[4];
 #pragma unroll
-        for (int nt = 0; nt < 4; ++nt) {
-          const uint4 b = *reinterpret_cast<const uint4*>(stage + ((size_t)((4 * ks + kk) * 4 + nt) * 32 + lane) * 16);
-          dc_mma(acc[nt], hi, b.x, b.y);
-          dc_mma(low[nt], hi, b.z, b.w);
-          dc_mma(low[nt], lo, b.x, b.y);
-        }
+        for (int nt = 0; nt < 4; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((4 * ks + kk) * 4 + nt, lane, false));
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) dc_mma(acc[nt], hi, b[nt].x, b[nt].z);
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) dc_mma(low[nt], hi, b[nt].y, b[nt].w);
+#pragma unroll
+        for (int nt = 0; nt < 4; ++nt) dc_mma(low2[nt], lo, b[nt].x, b[nt].z);
       }
     }
 #pragma unroll
     for (int nt = 0; nt < 4; ++nt)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) acc[nt][e] += low[nt][e];
+      for (int e = 0; e < 4; ++e) acc[nt][e] += low[nt][e] + low2[nt][e];
     if (KS > 1) {
       float* mine = xch + ((i & 1) * 4 + warp) * 512 + lane * 4;
 #pragma unroll
@@ -377,15 +416,19 @@ delta_scan_kernel(const DeltaChunkParams p) {
     split_bf16(u[1][0], u[1][1], uh[2], ul[2]);
     split_bf16(u[1][2], u[1][3], uh[3], ul[3]);
     const float* gamma = reinterpret_cast<const float*>(stage + 48 * DK * 4) + 64 * ks + 2 * j;
+    uint4 kb[8];
 #pragma unroll
     for (int t = 0; t < 8; ++t) {
       const float2 f = *reinterpret_cast<const float2*>(gamma + 8 * t);
-      const uint4 b = *reinterpret_cast<const uint4*>(stage + ((size_t)(4 * (DK / 16) + 8 * ks + t) * 32 + lane) * 16);
+      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece(4 * (DK / 16) + 8 * ks + t, lane, true));
       s[t][0] *= f.x; s[t][1] *= f.y; s[t][2] *= f.x; s[t][3] *= f.y;
-      dc_mma(s[t], uh, b.x, b.y);
-      dc_mma(s[t], uh, b.z, b.w);
-      dc_mma(s[t], ul, b.x, b.y);
     }
+#pragma unroll
+    for (int t = 0; t < 8; ++t) dc_mma(s[t], uh, kb[t].x, kb[t].z);
+#pragma unroll
+    for (int t = 0; t < 8; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
+#pragma unroll
+    for (int t = 0; t < 8; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
     // read-outs: the warps of a column tile take the row tiles in turn
     const int r0 = (p.chunk0 + i) * DC_T;
     float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g;
@@ -428,18 +471,20 @@ static int launch_scan(const DeltaChunkParams& p, cudaStream_t st) {
   return launch_check("delta_scan");
 }
 
-template <int NCH>
+template <int NT>
 static int launch_prepare(const DeltaChunkParams& p, cudaStream_t st) {
-  const int smem = std::max(64 * DC_PITCH * 4, dc_block_bytes(p.dk));
-  auto kern = delta_prepare_kernel<NCH>;
-  static int raised[64] = {};
+  constexpr int SMEM = std::max(64 * (NT == 128 ? 136 : NT + 4) * 4, dc_block_bytes(2 * NT));
+  auto kern = delta_prepare_kernel<NT>;
+  static bool raised[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  if (smem > 40 * 1024 && raised[dev & 63] < smem) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return launch_check("delta_prepare attr", 0);
-    raised[dev & 63] = smem;
+  if (!raised[dev & 63]) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess ||
+        cudaFuncSetAttribute(kern, cudaFuncAttributePreferredSharedMemoryCarveout, 100) != cudaSuccess)
+      return launch_check("delta_prepare attr", 0);
+    raised[dev & 63] = true;
   }
-  kern<<<dim3(p.n_chunks, p.a.heads, p.a.n_seqs), DC_THREADS, smem, st>>>(p);
+  kern<<<dim3(p.n_chunks, p.a.heads, p.a.n_seqs), NT, SMEM, st>>>(p);
   return launch_check("delta_prepare");
 }
 
@@ -471,7 +516,7 @@ extern "C" int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* 
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   for (p.chunk0 = 0; p.chunk0 < total; p.chunk0 += round) {
     p.n_chunks = std::min(round, total - p.chunk0);
-    int rc = p.dk <= 128 ? launch_prepare<1>(p, st) : launch_prepare<2>(p, st);
+    int rc = p.dk == 64 ? launch_prepare<32>(p, st) : p.dk == 128 ? launch_prepare<64>(p, st) : launch_prepare<128>(p, st);
     if (rc == 0) rc = p.dk == 64 ? launch_scan<1>(p, st) : p.dk == 128 ? launch_scan<2>(p, st) : launch_scan<4>(p, st);
     if (rc) return rc;
   }
