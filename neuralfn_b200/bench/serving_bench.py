@@ -128,7 +128,7 @@ def run(args, clock_sampler, sizes=None) -> None:
             del eng
             for batch in (1, 8, 32):
                 eng = _engine(kind, z, batch, context + 128)
-                last = {b: eng.prefill(b, ids[:context]) for b in range(batch)}
+                last = {b: eng.prefill(b, ids[64 * b:64 * b + context]) for b in range(batch)}      # different tokens, different experts
 
                 def step():
                     nonlocal last

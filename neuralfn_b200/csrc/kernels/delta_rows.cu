@@ -129,8 +129,8 @@ delta_out_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ ga
   T* dst = out + (size_t)row * ld_out + (size_t)h * vdim_p;
   for (int c = lane * 4; c < vdim_p; c += 128) {
     const float4 f = load4(src + c), z = load4(g + c), w = load4(weight + c);
-    store4(dst + c, make_float4(f.x * r * w.x * sigmoid_exact(z.x), f.y * r * w.y * sigmoid_exact(z.y), f.z * r * w.z * sigmoid_exact(z.z),
-                                f.w * r * w.w * sigmoid_exact(z.w)));
+    store4(dst + c, make_float4(f.x * r * w.x * sigmoid_for<T>(z.x), f.y * r * w.y * sigmoid_for<T>(z.y), f.z * r * w.z * sigmoid_for<T>(z.z),
+                                f.w * r * w.w * sigmoid_for<T>(z.w)));
   }
 }
 

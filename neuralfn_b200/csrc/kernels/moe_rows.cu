@@ -1,9 +1,11 @@
 // Mixture of experts for a handful of rows (decoding, short portions) and in 32-bit mode: one launch routes the rows and lists every
-// expert's items, then each chosen expert's weights are streamed once per group of eight items - a warp per weight row, its lanes
-// across the input width. Also the gate of the sorted prompt rows (the grouped GEMMs around it are in gemm_tp.cu).
+// expert's items, then each chosen expert's weights are streamed once per group of items: on the tensor cores in bf16, a warp per
+// weight row in 32-bit mode. Also the gate of the sorted prompt rows (the grouped GEMMs around it are in gemm_tp.cu).
 //
 // The routing weight multiplies the expert's input. Gate and up are linear, so it is applied to their fp32 results instead:
 // act(w g) * (w u).
+#include <algorithm>
+
 #include "common.h"
 #include "paged.cuh"
 
@@ -11,58 +13,73 @@ namespace nfn {
 
 constexpr int MR_MAX_EXPERTS = 1024, MR_GROUP = 8, MR_WARPS = 8;
 
-// One CTA. Scores: sigmoid of the fp32 logits; the `top` largest per row (ties: the lower index).
+// One CTA. Scores: sigmoid of the fp32 logits; the `top` largest per row (ties: the lower index). PER: logits per lane (experts <= 32 PER).
+template <int PER>
 __global__ void __launch_bounds__(1024)
 moe_route_rows_kernel(const nfn_moe_rows_args p) {
-  __shared__ int count[MR_MAX_EXPERTS], start[MR_MAX_EXPERTS + 1];
+  __shared__ int count[MR_MAX_EXPERTS], start[MR_MAX_EXPERTS], warp_sum[32], warp_live[32];
   const int E = p.experts, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int e = threadIdx.x; e < E; e += 1024) count[e] = 0;
+  count[threadIdx.x] = 0;
   __syncthreads();
   for (int r = warp; r < p.rows; r += 32) {
     const float* z = p.logits + (size_t)r * p.ld_logits;
+    float v[PER];
+#pragma unroll
+    for (int i = 0; i < PER; ++i) v[i] = lane + 32 * i < E ? z[lane + 32 * i] : -INFINITY;
+    uint32_t taken = 0;
     for (int j = 0; j < p.top; ++j) {
-      // the next one in (score falling, index rising) order after the one chosen before
       float best = -INFINITY;
       int bi = 0x7fffffff;
-      const int prev = j > 0 ? p.idx[(size_t)r * p.top + j - 1] : -1;
-      const float pz = prev >= 0 ? z[prev] : INFINITY;
-      for (int e = lane; e < E; e += 32) {
-        const float v = z[e];
-        const bool open = prev < 0 || v < pz || (v == pz && e > prev);
-        if (open && (bi == 0x7fffffff || v > best)) { best = v; bi = e; }
-      }
+#pragma unroll
+      for (int i = 0; i < PER; ++i)
+        if (lane + 32 * i < E && !((taken >> i) & 1u) && (bi == 0x7fffffff || v[i] > best)) { best = v[i]; bi = lane + 32 * i; }
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) {
         const float ov = __shfl_xor_sync(0xffffffffu, best, o);
         const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
         if (oi != 0x7fffffff && (bi == 0x7fffffff || ov > best || (ov == best && oi < bi))) { best = ov; bi = oi; }
       }
+      if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
       if (lane == 0) {
-        bi = min(bi, E - 1);
         p.idx[(size_t)r * p.top + j] = bi;
         p.weight[(size_t)r * p.top + j] = sigmoid_exact(best);
         atomicAdd(&count[bi], 1);
       }
-      __syncwarp();
     }
   }
   __syncthreads();
-  if (threadIdx.x == 0) {
-    int run = 0, live = 0;
-    for (int e = 0; e < E; ++e) {
-      start[e] = run;
-      p.offsets[e] = run;
-      run += count[e];
-      if (count[e] > 0) p.active[live++] = e;
+  // first item of every expert, and the experts that have items
+  const int e = threadIdx.x, mine = e < E ? count[e] : 0;
+  int run = mine;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const int up = __shfl_up_sync(0xffffffffu, run, o);
+    if (lane >= o) run += up;
+  }
+  const uint32_t live = __ballot_sync(0xffffffffu, mine > 0);
+  if (lane == 31) {
+    warp_sum[warp] = run;
+    warp_live[warp] = __popc(live);
+  }
+  __syncthreads();
+  int base = 0, slot = 0;
+  for (int w = 0; w < warp; ++w) {
+    base += warp_sum[w];
+    slot += warp_live[w];
+  }
+  if (e < E) {
+    start[e] = p.offsets[e] = base + run - mine;
+    if (mine > 0) p.active[slot + __popc(live & ((1u << lane) - 1u))] = e;
+    if (e == E - 1) {
+      p.offsets[E] = base + run;
+      p.active[E] = slot + __popc(live);
     }
-    p.offsets[E] = run;
-    p.active[E] = live;
   }
   __syncthreads();
   for (int i = threadIdx.x; i < p.rows * p.top; i += 1024) p.order[atomicAdd(&start[p.idx[i]], 1)] = i;
 }
 
-// DOWN = false: mid[item][f] = act(w G_f h) * (w U_f h), h of the item's row. DOWN = true: y[item][n] = D_n mid[item].
+// 32-bit mode. DOWN = false: mid[item][f] = act(w G_f h) * (w U_f h), h of the item's row. DOWN = true: y[item][n] = D_n mid[item].
 template <typename T, bool DOWN>
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_products_kernel(const nfn_moe_rows_args p) {
@@ -134,6 +151,110 @@ moe_products_kernel(const nfn_moe_rows_args p) {
   }
 }
 
+// The same on the tensor cores: a CTA takes 16 weight rows (DOWN: 32; else 16 of gate and the 16 of up beside them), its four warps a quarter
+// of the contraction each. Weight rows are the 16-row operand of mma.m16n8k16, items its eight columns; the order of the contraction is
+// free, so every fragment is one 16-byte load per lane. Weights are read once per 8 NT items.
+constexpr int MM_WARPS = 4;
+
+__device__ __forceinline__ uint4 mm_stream(const __nv_bfloat16* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+__device__ __forceinline__ void mm_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <bool DOWN, int NT>
+__global__ void __launch_bounds__(MM_WARPS * 32)
+moe_products_mma_kernel(const nfn_moe_rows_args p) {
+  constexpr int M = 8 * NT;                               // items at a time
+  constexpr int U = NT == 4 ? 2 : 4;                      // 32-channel steps in flight
+  __shared__ float part[MM_WARPS][2][16][M + 1];
+  if ((int)blockIdx.y >= p.active[p.experts]) return;
+  const int e = p.active[blockIdx.y], warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+  const int N = DOWN ? p.width : p.ff, K = DOWN ? p.ff : p.width;
+  const int n0 = blockIdx.x * (DOWN ? 32 : 16);
+  // rows of the two 16-row tiles
+  const __nv_bfloat16* w0 = (DOWN ? static_cast<const __nv_bfloat16*>(p.w_down) + ((size_t)e * N + n0) * K : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * 2 * N + n0) * K) +
+                            (size_t)g * K + 8 * j;
+  const bool two = !DOWN || n0 + 16 < N;
+  const __nv_bfloat16* w1 = two ? w0 + (size_t)(DOWN ? 16 : N) * K : w0;
+  const int steps = (K + 31) / 32, s0 = steps * warp / MM_WARPS, s1 = steps * (warp + 1) / MM_WARPS;
+  const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
+  const int i0 = p.offsets[e], i1 = p.offsets[e + 1];
+  for (int i = i0; i < i1; i += M) {
+    const __nv_bfloat16* src[NT];
+    bool on[NT];
+#pragma unroll
+    for (int t = 0; t < NT; ++t) {
+      on[t] = i + 8 * t + g < i1;
+      const int item = p.order[on[t] ? i + 8 * t + g : i0];
+      src[t] = (DOWN ? static_cast<const __nv_bfloat16*>(p.mid) + (size_t)item * p.ff : static_cast<const __nv_bfloat16*>(p.h) + (size_t)(item / p.top) * p.ld_h) + 8 * j;
+    }
+    float acc[2][NT][4];
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int t = 0; t < NT; ++t)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) acc[m][t][c] = 0.f;
+    for (int s = s0; s < s1; s += U) {
+      uint4 a[U][4], b[U][NT];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int k = (s + u) * 32;
+        const bool ok = s + u < s1 && k + 8 * j < K;
+        a[u][0] = ok ? mm_stream(w0 + k) : zero4;
+        a[u][1] = ok ? mm_stream(w0 + (size_t)8 * K + k) : zero4;
+        a[u][2] = ok ? mm_stream(w1 + k) : zero4;
+        a[u][3] = ok ? mm_stream(w1 + (size_t)8 * K + k) : zero4;
+#pragma unroll
+        for (int t = 0; t < NT; ++t) b[u][t] = ok && on[t] ? __ldg(reinterpret_cast<const uint4*>(src[t] + k)) : zero4;
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+          mm_mma(acc[0][t], a[u][0].x, a[u][1].x, a[u][0].y, a[u][1].y, b[u][t].x, b[u][t].y);
+          mm_mma(acc[1][t], a[u][2].x, a[u][3].x, a[u][2].y, a[u][3].y, b[u][t].x, b[u][t].y);
+          mm_mma(acc[0][t], a[u][0].z, a[u][1].z, a[u][0].w, a[u][1].w, b[u][t].z, b[u][t].w);
+          mm_mma(acc[1][t], a[u][2].z, a[u][3].z, a[u][2].w, a[u][3].w, b[u][t].z, b[u][t].w);
+        }
+    }
+#pragma unroll
+    for (int m = 0; m < 2; ++m)
+#pragma unroll
+      for (int t = 0; t < NT; ++t)
+#pragma unroll
+        for (int c = 0; c < 4; ++c) part[warp][m][g + (c >> 1) * 8][8 * t + 2 * j + (c & 1)] = acc[m][t][c];
+    __syncthreads();
+    const int live = min(M, i1 - i);
+    for (int x = threadIdx.x; x < (DOWN ? 32 : 16) * live; x += MM_WARPS * 32) {
+      const int col = x / (DOWN ? 32 : 16), row = x % (DOWN ? 32 : 16), item = p.order[i + col];
+      if (n0 + row >= N) continue;
+      if (DOWN) {
+        float v = 0.f;
+#pragma unroll
+        for (int w = 0; w < MM_WARPS; ++w) v += part[w][row >> 4][row & 15][col];
+        static_cast<__nv_bfloat16*>(p.y)[(size_t)item * p.ld_y + n0 + row] = __float2bfloat16(v);
+      } else {
+        float gv = 0.f, uv = 0.f;
+#pragma unroll
+        for (int w = 0; w < MM_WARPS; ++w) {
+          gv += part[w][0][row][col];
+          uv += part[w][1][row][col];
+        }
+        const float f = p.weight[item];
+        static_cast<__nv_bfloat16*>(p.mid)[(size_t)item * p.ff + n0 + row] = __float2bfloat16(ff_act(f * gv, p.act) * (f * uv));
+      }
+    }
+    __syncthreads();
+  }
+}
+
 // Sorted prompt rows: mid = act(w g) * (w u). Rows past the plan's count stay untouched.
 __global__ void __launch_bounds__(256)
 moe_act_rows_kernel(const __nv_bfloat16* __restrict__ gate_up, const float* __restrict__ row_w, const int* __restrict__ plan, int ff, int act,
@@ -149,12 +270,27 @@ moe_act_rows_kernel(const __nv_bfloat16* __restrict__ gate_up, const float* __re
   store8(mid + (size_t)r * ff + c, g);
 }
 
-template <typename T>
+template <int NT>
+static void launch_products_mma(const nfn_moe_rows_args& a, int live, cudaStream_t st) {
+  moe_products_mma_kernel<false, NT><<<dim3(ceil_div(a.ff, 16), live), MM_WARPS * 32, 0, st>>>(a);
+  moe_products_mma_kernel<true, NT><<<dim3(ceil_div(a.width, 32), live), MM_WARPS * 32, 0, st>>>(a);
+}
+
 static int launch_moe_rows(const nfn_moe_rows_args& a, cudaStream_t st) {
-  const int live = (int)min((long long)a.experts, (long long)a.rows * a.top);     // most experts that can have items
-  moe_route_rows_kernel<<<1, 1024, 0, st>>>(a);
-  moe_products_kernel<T, false><<<dim3(ceil_div(a.ff, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
-  moe_products_kernel<T, true><<<dim3(ceil_div(a.width, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
+  const int live = (int)std::min<long long>(a.experts, (long long)a.rows * a.top);     // most experts that can have items
+  if (a.experts <= 64) moe_route_rows_kernel<2><<<1, 1024, 0, st>>>(a);
+  else if (a.experts <= 256) moe_route_rows_kernel<8><<<1, 1024, 0, st>>>(a);
+  else moe_route_rows_kernel<32><<<1, 1024, 0, st>>>(a);
+  if (a.f32) {
+    moe_products_kernel<float, false><<<dim3(ceil_div(a.ff, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
+    moe_products_kernel<float, true><<<dim3(ceil_div(a.width, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
+  } else if (a.rows <= 8) {
+    launch_products_mma<1>(a, live, st);
+  } else if (a.rows <= 16) {
+    launch_products_mma<2>(a, live, st);
+  } else {
+    launch_products_mma<4>(a, live, st);
+  }
   return launch_check("moe_rows", 3);
 }
 
@@ -167,9 +303,9 @@ extern "C" int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream) 
   const nfn_moe_rows_args& a = *args;
   if (a.rows <= 0) return 0;
   if (a.experts < 1 || a.experts > MR_MAX_EXPERTS || a.top < 1 || a.top > a.experts) return fail(-1, "moe_rows: need 1 <= top <= experts <= 1024");
-  if ((a.width | a.ff | a.ld_h) & 7) return fail(-1, "moe_rows: widths must be multiples of 8");
+  if ((a.width | a.ff | a.ld_h) & 15) return fail(-1, "moe_rows: widths must be multiples of 16");
   if ((long long)a.rows * a.top > 0x7fffffffLL / 2) return fail(-1, "moe_rows: too many rows");
-  return a.f32 ? launch_moe_rows<float>(a, static_cast<cudaStream_t>(stream)) : launch_moe_rows<__nv_bfloat16>(a, static_cast<cudaStream_t>(stream));
+  return launch_moe_rows(a, static_cast<cudaStream_t>(stream));
 }
 
 extern "C" int nfn_moe_act_rows(const void* gate_up, const float* row_w, const int* plan, int capacity_rows, int ff, int act, void* mid, nfn_stream_t stream) {

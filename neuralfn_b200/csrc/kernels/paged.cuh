@@ -68,6 +68,12 @@ __device__ __forceinline__ float ff_act(float v, int act) {
   if (act == NFN_ACT_GELU_TANH) return gelu_tanh_exact(v);
   return v;
 }
+// by activation type: exact in 32-bit mode; for results that are rounded to bf16 the exponential and reciprocal units (a few ulp of fp32)
+template <typename T>
+__device__ __forceinline__ float sigmoid_for(float v) {
+  if constexpr (sizeof(T) == 4) return 1.f / (1.f + expf(-v));
+  else return fast_rcp(1.f + fast_exp2(v * -1.4426950408889634f));
+}
 __device__ __forceinline__ float sigmoid_exact(float v) { return 1.f / (1.f + expf(-v)); }
 
 }  // namespace nfn

@@ -215,7 +215,7 @@ mix_rows_kernel(const nfn_mix_args p) {
         if (i0 + i < t.n) {
           if (p.conv_act == NFN_ACT_SILU) {
 #pragma unroll
-            for (int e = 0; e < 8; ++e) v[i][e] = v[i][e] / (1.f + expf(-v[i][e]));
+            for (int e = 0; e < 8; ++e) v[i][e] *= sigmoid_for<T>(v[i][e]);
           }
           if (p.temp_every > 0) {
             const int pos = t.e_pos0 + ti0 + i0 + i;

@@ -7,8 +7,7 @@
 
 namespace nfn {
 
-constexpr int ST_THREADS = 256;
-
+template <int ST_THREADS>
 __device__ __forceinline__ float st_block_sum(float v, float* red) {
 #pragma unroll
   for (int s = 16; s > 0; s >>= 1) v += __shfl_xor_sync(0xffffffffu, v, s);
@@ -20,13 +19,39 @@ __device__ __forceinline__ float st_block_sum(float v, float* red) {
   return t;
 }
 
-// S: streams held in registers (an upper bound; the mixing weights past p.streams are zero)
-template <typename T, int S>
+// S: streams held in registers (an upper bound; the mixing weights past p.streams are zero). Few rows take many threads each, so that a
+// row's loads are all on their way at once
+template <typename T, int S, int ST_THREADS>
 __global__ void __launch_bounds__(ST_THREADS)
 stream_pass_kernel(const nfn_stream_args p) {
   extern __shared__ float st_row[];                        // [ld] u
   __shared__ float red[ST_THREADS / 32], w_mix[S][S], w_out[S], w_in[S];
   const int r = blockIdx.x, n = p.streams, vecs = p.ld / 4;
+  const int src = p.src_rows ? p.src_rows[r] : r;
+  const __nv_bfloat16* emb = nullptr;
+  if (p.tokens) emb = static_cast<const __nv_bfloat16*>(p.embed) + (size_t)min(max(p.tokens[r], 0), p.vocab - 1) * p.ld;
+  const float* x = p.x + (size_t)src * n * p.ld;
+  float* x_out = p.x_out ? p.x_out + (size_t)r * n * p.ld : nullptr;
+  const T* y = static_cast<const T*>(p.y);
+  float4 b[S], f;
+  auto fetch = [&](int v) {
+    if (emb) {
+      b[0] = load4(emb + 4 * v);
+    } else {
+#pragma unroll
+      for (int s = 0; s < S; ++s) b[s] = s < n ? load4(x + (size_t)s * p.ld + 4 * v) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    f = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (p.y) {
+#pragma unroll 4
+      for (int j = 0; j < p.y_rows; ++j) {
+        const int at = src * p.y_rows + j, yr = p.y_index ? p.y_index[at] : at;
+        const float4 g = load4(y + (size_t)yr * p.ld + 4 * v);
+        f.x += g.x; f.y += g.y; f.z += g.z; f.w += g.w;
+      }
+    }
+  };
+  if (threadIdx.x < vecs) fetch(threadIdx.x);
   if (threadIdx.x < S * S) {
     const int s = threadIdx.x / S, t = threadIdx.x % S;
     w_mix[s][t] = (s < n && t < n) ? (p.mix ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.mix)[s * n + t]) : (s == t ? 1.f : 0.f)) : 0.f;
@@ -37,31 +62,15 @@ stream_pass_kernel(const nfn_stream_args p) {
     w_in[s] = s < n ? (p.in ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.in)[s]) : 1.f) : 0.f;
   }
   __syncthreads();
-  const int src = p.src_rows ? p.src_rows[r] : r;
-  const __nv_bfloat16* emb = nullptr;
-  if (p.tokens) emb = static_cast<const __nv_bfloat16*>(p.embed) + (size_t)min(max(p.tokens[r], 0), p.vocab - 1) * p.ld;
-  const float* x = p.x + (size_t)src * n * p.ld;
-  float* x_out = p.x_out ? p.x_out + (size_t)r * n * p.ld : nullptr;
-  const T* y = static_cast<const T*>(p.y);
   float ss = 0.f;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
-    float4 b[S];
+    if (v != threadIdx.x) fetch(v);
     if (emb) {
-      float4 e = load4(emb + 4 * v);
-      e.x *= p.embed_scale; e.y *= p.embed_scale; e.z *= p.embed_scale; e.w *= p.embed_scale;
+      b[0].x *= p.embed_scale; b[0].y *= p.embed_scale; b[0].z *= p.embed_scale; b[0].w *= p.embed_scale;
 #pragma unroll
-      for (int s = 0; s < S; ++s) b[s] = e;
-    } else {
-#pragma unroll
-      for (int s = 0; s < S; ++s) b[s] = s < n ? load4(x + (size_t)s * p.ld + 4 * v) : make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int s = 1; s < S; ++s) b[s] = b[0];
     }
     if (p.y) {
-      float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
-      for (int j = 0; j < p.y_rows; ++j) {
-        const int at = src * p.y_rows + j, yr = p.y_index ? p.y_index[at] : at;
-        const float4 g = load4(y + (size_t)yr * p.ld + 4 * v);
-        f.x += g.x; f.y += g.y; f.z += g.z; f.w += g.w;
-      }
       float4 c[S];
 #pragma unroll
       for (int t = 0; t < S; ++t) {
@@ -93,7 +102,7 @@ stream_pass_kernel(const nfn_stream_args p) {
     }
   }
   if (!p.h) return;
-  const float rms = 1.f / sqrtf(st_block_sum(ss, red) / (float)p.width + p.eps);
+  const float rms = 1.f / sqrtf(st_block_sum<ST_THREADS>(ss, red) / (float)p.width + p.eps);
   T* h = static_cast<T*>(p.h) + (size_t)r * p.ld;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
     const float4 u = load4(st_row + 4 * v), w = load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * v);
@@ -102,10 +111,10 @@ stream_pass_kernel(const nfn_stream_args p) {
   }
 }
 
-template <typename T, int S>
+template <typename T, int S, int THREADS>
 static int launch_stream(const nfn_stream_args& a, cudaStream_t st) {
   const size_t smem = a.h ? (size_t)a.ld * sizeof(float) : 0;
-  auto kern = stream_pass_kernel<T, S>;
+  auto kern = stream_pass_kernel<T, S, THREADS>;
   static bool raised[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -113,18 +122,19 @@ static int launch_stream(const nfn_stream_args& a, cudaStream_t st) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return launch_check("stream_pass attr", 0);
     raised[dev & 63] = true;
   }
-  kern<<<a.rows, ST_THREADS, smem, st>>>(a);
+  kern<<<a.rows, THREADS, smem, st>>>(a);
   return launch_check("stream_pass");
 }
 
 template <typename T>
 static int pick_stream(const nfn_stream_args& a, cudaStream_t st) {
+  const bool few = a.rows <= 2 * sm_count() && a.ld >= 2048;
   switch (a.streams) {
-    case 1: return launch_stream<T, 1>(a, st);
-    case 2: return launch_stream<T, 2>(a, st);
-    case 3: return launch_stream<T, 3>(a, st);
-    case 4: return launch_stream<T, 4>(a, st);
-    default: return a.streams <= 8 ? launch_stream<T, 8>(a, st) : launch_stream<T, NFN_MAX_STREAMS>(a, st);
+    case 1: return few ? launch_stream<T, 1, 1024>(a, st) : launch_stream<T, 1, 256>(a, st);
+    case 2: return few ? launch_stream<T, 2, 1024>(a, st) : launch_stream<T, 2, 256>(a, st);
+    case 3: return few ? launch_stream<T, 3, 1024>(a, st) : launch_stream<T, 3, 256>(a, st);
+    case 4: return few ? launch_stream<T, 4, 1024>(a, st) : launch_stream<T, 4, 256>(a, st);
+    default: return a.streams <= 8 ? launch_stream<T, 8, 256>(a, st) : launch_stream<T, NFN_MAX_STREAMS, 256>(a, st);
   }
 }
 
