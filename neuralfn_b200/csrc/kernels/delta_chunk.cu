@@ -8,7 +8,7 @@
 //
 //   delta_prepare_kernel  one CTA per (chunk, head), all chunks at once: W, Q, K and T V, P T V. A thread owns two channels; their
 //                         products for all pairs of tokens are formed in registers and summed over channels through shared memory.
-//   delta_scan_kernel     one warp per (head, 16 value columns, 64 key channels), one chunk after another: the state, transposed, sits in
+//   delta_scan_kernel     one warp per (head, 16 value columns, 32 key channels), one chunk after another: the state, transposed, sits in
 //                         the accumulator registers of mma.m16n8k16 and is the A operand of the next chunk's W S and Q S as it stands; W, Q
 //                         and K arrive in fragment order by bulk copies through a ring of shared memory stages.
 //
@@ -23,7 +23,6 @@
 namespace nfn {
 
 constexpr int DC_T = 16;                               // tokens of a chunk
-constexpr int DC_STAGES = 3;
 constexpr long long DC_WORKSPACE = 96LL << 20;
 
 // bytes of a (chunk, head) block of the scan's operands: [W, Q: dk / 16 steps x 4 tiles of 8 rows][K: dk / 8 tiles] x 32 lanes x 16 bytes, then
@@ -33,7 +32,7 @@ __host__ __device__ constexpr int dc_uo_floats(int vdim_p) { return vdim_p * 32;
 
 struct DeltaChunkParams {
   nfn_delta_args a;
-  int dk;                     // key channels padded to the scan's 64 per warp
+  int dk;                     // padded key channels: 64, 128 or 256
   int chunk0, n_chunks;       // chunks [chunk0, chunk0 + n_chunks) of every sequence in this round
   unsigned char* blocks;      // [seq][chunk][head][dc_block_bytes]
   float* uo;                  // [seq][chunk][head][dc_uo_floats]
@@ -283,17 +282,27 @@ __device__ __forceinline__ void dc_mma(float (&d)[4], const uint32_t (&a)[4], ui
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+// the first product of a sum
+__device__ __forceinline__ void dc_mma0(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%10,%10,%10,%10};"
+      : "=f"(d[0]), "=f"(d[1]), "=f"(d[2]), "=f"(d[3])
+      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1), "f"(0.f));
+}
 __device__ __forceinline__ void dc_bulk_load(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 
-// KS: warps that share a head's key channels, 64 each; the CTA's four warps take 4 / KS tiles of 16 value columns
+// KS: warps that share a head's key channels, 32 each; the CTA's eight warps take 8 / KS tiles of 16 value columns
+constexpr int DS_WARPS = 8, DS_CH = 32;
+// shared memory of a stage: the head's operand block, then T V and P T V of the CTA's column tiles
+__host__ __device__ constexpr int ds_stage_bytes(int ks) { return dc_block_bytes(DS_CH * ks) + DS_WARPS / ks * 2048; }
+__host__ __device__ constexpr int ds_stages(int ks) { return ks == 8 ? 3 : 4; }
 template <int KS>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(DS_WARPS * 32)
 delta_scan_kernel(const DeltaChunkParams p) {
-  constexpr int DK = 64 * KS, TILES = 4 / KS, BLOCK = dc_block_bytes(DK);
-  extern __shared__ __align__(128) unsigned char dc_smem[];       // [DC_STAGES][BLOCK], then the partial sums [2][4 warps][16][32]
-  __shared__ __align__(8) uint64_t bar_full[DC_STAGES];
+  constexpr int DK = DS_CH * KS, TILES = DS_WARPS / KS, BLOCK = dc_block_bytes(DK), STAGE = ds_stage_bytes(KS), STAGES = ds_stages(KS);
+  extern __shared__ __align__(128) unsigned char dc_smem[];       // [STAGES][STAGE], then partial sums [2][warps][4 row tiles][32][4]
+  __shared__ __align__(8) uint64_t bar_full[STAGES];
   __shared__ int cta_abort_s;
   volatile int* cta_abort = &cta_abort_s;
   const nfn_delta_args& a = p.a;
@@ -304,143 +313,120 @@ delta_scan_kernel(const DeltaChunkParams p) {
   const int ks = warp % KS, h = blockIdx.y, DP = a.dim_p, VP = a.vdim_p;
   const int vt = blockIdx.x * TILES + warp / KS;
   const bool on = vt * 16 < VP;                                   // warps past the last column tile keep the others company
-  float* xch = reinterpret_cast<float*>(dc_smem + DC_STAGES * BLOCK);
+  float* xch = reinterpret_cast<float*>(dc_smem + STAGES * STAGE);
   const unsigned char* blocks = p.blocks + ((size_t)blockIdx.z * p.n_chunks * a.heads + h) * BLOCK;
   const size_t block_step = (size_t)a.heads * BLOCK;
-  const float* uo = p.uo + ((size_t)blockIdx.z * p.n_chunks * a.heads + h) * dc_uo_floats(VP) + (on ? vt : 0) * 512 + lane * 4;
+  const float* uo = p.uo + ((size_t)blockIdx.z * p.n_chunks * a.heads + h) * dc_uo_floats(VP) + blockIdx.x * TILES * 512;
   const size_t uo_step = (size_t)a.heads * dc_uo_floats(VP);
+  const uint32_t uo_bytes = min(TILES, VP / 16 - (int)blockIdx.x * TILES) * 2048;
 
   auto load = [&](int i) {
-    const uint32_t bar = smem_u32(&bar_full[i % DC_STAGES]);
-    mbar_expect_tx(bar, BLOCK);
-    dc_bulk_load(smem_u32(dc_smem + (i % DC_STAGES) * BLOCK), blocks + i * block_step, BLOCK, bar);
+    const uint32_t bar = smem_u32(&bar_full[i % STAGES]), dst = smem_u32(dc_smem + (i % STAGES) * STAGE);
+    mbar_expect_tx(bar, BLOCK + uo_bytes);
+    dc_bulk_load(dst, blocks + i * block_step, BLOCK, bar);
+    dc_bulk_load(dst + BLOCK, uo + i * uo_step, uo_bytes, bar);
   };
   if (tid == 0) {
     cta_abort_s = 0;
-    for (int s = 0; s < DC_STAGES; ++s) mbar_init(smem_u32(&bar_full[s]), 1);
+    for (int s = 0; s < STAGES; ++s) mbar_init(smem_u32(&bar_full[s]), 1);
     fence_mbar_init();
-    for (int i = 0; i < min(DC_STAGES, n_chunks); ++i) load(i);
+    for (int i = 0; i < min(STAGES, n_chunks); ++i) load(i);
   }
-  // S^T: rows are value columns (g, g + 8), columns key channels 64 ks + 8 t + 2 j, + 1
+  // S^T: rows are value columns (g, g + 8), columns key channels 32 ks + 8 t + 2 j, + 1
   float* st = a.state + ((size_t)seq.slot * a.heads + h) * DP * VP + vt * 16 + g;
   const bool fresh = seq.pos0 == 0 && p.chunk0 == 0;
-  float s[8][4];
+  float s[4][4];
 #pragma unroll
-  for (int t = 0; t < 8; ++t)
+  for (int t = 0; t < 4; ++t)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = 64 * ks + 8 * t + 2 * j + (e & 1);
+      const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
       s[t][e] = (on && !fresh && d < DP) ? st[(size_t)d * VP + (e >> 1) * 8] : 0.f;
     }
-  float u_next[2][4], o_next[2][4];
-  auto fetch = [&](int i) {
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt) {
-      const float4 u = *reinterpret_cast<const float4*>(uo + i * uo_step + nt * 128), o = *reinterpret_cast<const float4*>(uo + i * uo_step + 256 + nt * 128);
-      u_next[nt][0] = u.x; u_next[nt][1] = u.y; u_next[nt][2] = u.z; u_next[nt][3] = u.w;
-      o_next[nt][0] = o.x; o_next[nt][1] = o.y; o_next[nt][2] = o.z; o_next[nt][3] = o.w;
-    }
-  };
-  fetch(0);
   __syncthreads();
   bool ok = true;
+  int at = 0, phase = 0;
   for (int i = 0; i < n_chunks; ++i) {
-    float u[2][4], o[2][4];
+    ok = mbar_wait_bounded(smem_u32(&bar_full[at]), phase, cta_abort, p.status, NFN_ERR_WAIT_FULL);
+    const unsigned char* stage = dc_smem + at * STAGE;
+    float acc[4][4], low[4][4];                          // (W S)^T row tiles 0, 1, then (Q S)^T: high x high, and the products with a low part
 #pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
+    for (int kk = 0; kk < 2; ++kk) {
+      uint32_t hi[4], lo[4];
+      split_bf16(s[2 * kk][0], s[2 * kk][1], hi[0], lo[0]);
+      split_bf16(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
+      split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lo[2]);
+      split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
+      uint4 b[4];
 #pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        u[nt][e] = u_next[nt][e];
-        o[nt][e] = o_next[nt][e];
-      }
-    if (i + 1 < n_chunks) fetch(i + 1);
-    ok = mbar_wait_bounded(smem_u32(&bar_full[i % DC_STAGES]), (i / DC_STAGES) & 1, cta_abort, p.status, NFN_ERR_WAIT_FULL);
-    const unsigned char* stage = dc_smem + (i % DC_STAGES) * BLOCK;
-    float acc[4][4], low[4][4], low2[4][4];              // (W S)^T row tiles 0, 1, then (Q S)^T: high x high, high x low, low x high
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[nt][e] = low[nt][e] = low2[nt][e] = 0.f;
-    if (ok) {
-#pragma unroll
-      for (int kk = 0; kk < 4; ++kk) {
-        uint32_t hi[4], lo[4];
-        split_bf16(s[2 * kk][0], s[2 * kk][1], hi[0], lo[0]);
-        split_bf16(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
-        split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lo[2]);
-        split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
-        uint4 b[4];
-#pragma unroll
-        for (int nt = 0; nt < 4; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((4 * ks + kk) * 4 + nt, lane, false));
-#pragma unroll
-        for (int nt = 0; nt < 4; ++nt) dc_mma(acc[nt], hi, b[nt].x, b[nt].z);
-#pragma unroll
-        for (int nt = 0; nt < 4; ++nt) dc_mma(low[nt], hi, b[nt].y, b[nt].w);
-#pragma unroll
-        for (int nt = 0; nt < 4; ++nt) dc_mma(low2[nt], lo, b[nt].x, b[nt].z);
-      }
-    }
-#pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[nt][e] += low[nt][e] + low2[nt][e];
-    if (KS > 1) {
-      float* mine = xch + ((i & 1) * 4 + warp) * 512 + lane * 4;
-#pragma unroll
-      for (int nt = 0; nt < 4; ++nt) *reinterpret_cast<float4*>(mine + nt * 128) = make_float4(acc[nt][0], acc[nt][1], acc[nt][2], acc[nt][3]);
-    }
-    // every warp is done with chunk i - 1 here: its stage takes the next load
-    if (!__syncthreads_and(ok)) break;
-    if (tid == 0 && i > 0 && i - 1 + DC_STAGES < n_chunks) load(i - 1 + DC_STAGES);
-    if (KS > 1) {
-      const float* all = xch + ((i & 1) * 4 + warp / KS * KS) * 512 + lane * 4;
+      for (int nt = 0; nt < 4; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((2 * ks + kk) * 4 + nt, lane, false));
 #pragma unroll
       for (int nt = 0; nt < 4; ++nt) {
-        float4 t = *reinterpret_cast<const float4*>(all + nt * 128);
-#pragma unroll
-        for (int w = 1; w < KS; ++w) {
-          const float4 b = *reinterpret_cast<const float4*>(all + w * 512 + nt * 128);
-          t.x += b.x; t.y += b.y; t.z += b.z; t.w += b.w;
-        }
-        acc[nt][0] = t.x; acc[nt][1] = t.y; acc[nt][2] = t.z; acc[nt][3] = t.w;
+        if (kk == 0) dc_mma0(acc[nt], hi, b[nt].x, b[nt].z);
+        else dc_mma(acc[nt], hi, b[nt].x, b[nt].z);
       }
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) {
+        if (kk == 0) dc_mma0(low[nt], hi, b[nt].y, b[nt].w);
+        else dc_mma(low[nt], hi, b[nt].y, b[nt].w);
+      }
+#pragma unroll
+      for (int nt = 0; nt < 4; ++nt) dc_mma(low[nt], lo, b[nt].x, b[nt].z);
     }
+    float* mine = xch + ((i & 1) * DS_WARPS + warp) * 512 + lane * 4;
+#pragma unroll
+    for (int nt = 0; nt < 4; ++nt)
+      *reinterpret_cast<float4*>(mine + nt * 128) = make_float4(acc[nt][0] + low[nt][0], acc[nt][1] + low[nt][1], acc[nt][2] + low[nt][2], acc[nt][3] + low[nt][3]);
+    // every warp is done with chunk i - 1 here: its stage takes the next load
+    if (!__syncthreads_and(ok)) break;
+    if (tid == 0 && i > 0 && i - 1 + STAGES < n_chunks) load(i - 1 + STAGES);
+    const float* all = xch + ((i & 1) * DS_WARPS + warp / KS * KS) * 512 + lane * 4;
+    auto sum = [&](int nt) {
+      float4 t = *reinterpret_cast<const float4*>(all + nt * 128);
+#pragma unroll
+      for (int w = 1; w < KS; ++w) {
+        const float4 b = *reinterpret_cast<const float4*>(all + w * 512 + nt * 128);
+        t.x += b.x; t.y += b.y; t.z += b.z; t.w += b.w;
+      }
+      return t;
+    };
     // U^T, as the A operand of S'^T = e^G_last S^T + U^T K
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) u[nt][e] -= acc[nt][e];
+    const float* tv = reinterpret_cast<const float*>(stage + BLOCK) + (warp / KS) * 512 + lane * 4;
     uint32_t uh[4], ul[4];
-    split_bf16(u[0][0], u[0][1], uh[0], ul[0]);
-    split_bf16(u[0][2], u[0][3], uh[1], ul[1]);
-    split_bf16(u[1][0], u[1][1], uh[2], ul[2]);
-    split_bf16(u[1][2], u[1][3], uh[3], ul[3]);
-    const float* gamma = reinterpret_cast<const float*>(stage + 48 * DK * 4) + 64 * ks + 2 * j;
-    uint4 kb[8];
 #pragma unroll
-    for (int t = 0; t < 8; ++t) {
+    for (int nt = 0; nt < 2; ++nt) {
+      const float4 t = sum(nt), v = *reinterpret_cast<const float4*>(tv + nt * 128);
+      split_bf16(v.x - t.x, v.y - t.y, uh[2 * nt], ul[2 * nt]);
+      split_bf16(v.z - t.z, v.w - t.w, uh[2 * nt + 1], ul[2 * nt + 1]);
+    }
+    const float* gamma = reinterpret_cast<const float*>(stage + 48 * DK * 4) + DS_CH * ks + 2 * j;
+    uint4 kb[4];
+#pragma unroll
+    for (int t = 0; t < 4; ++t) {
       const float2 f = *reinterpret_cast<const float2*>(gamma + 8 * t);
-      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece(4 * (DK / 16) + 8 * ks + t, lane, true));
+      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece(4 * (DK / 16) + 4 * ks + t, lane, true));
       s[t][0] *= f.x; s[t][1] *= f.y; s[t][2] *= f.x; s[t][3] *= f.y;
     }
 #pragma unroll
-    for (int t = 0; t < 8; ++t) dc_mma(s[t], uh, kb[t].x, kb[t].z);
+    for (int t = 0; t < 4; ++t) dc_mma(s[t], uh, kb[t].x, kb[t].z);
 #pragma unroll
-    for (int t = 0; t < 8; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
+    for (int t = 0; t < 4; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
 #pragma unroll
-    for (int t = 0; t < 8; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
-    // read-outs: the warps of a column tile take the row tiles in turn
-    const int r0 = (p.chunk0 + i) * DC_T;
-    float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g;
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt) {
-      if (!on || nt % KS != ks) continue;
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = 8 * nt + 2 * j + (e & 1);
-        if (r0 + r < seq.n) dst[(size_t)r * a.ld_o + (e >> 1) * 8] = o[nt][e] + acc[2 + nt][e];
+    for (int t = 0; t < 4; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
+    if (on && ks < 2) {                                  // read-outs: the first two warps of a column tile take eight rows each
+      const float4 t = sum(2 + ks), o = *reinterpret_cast<const float4*>(tv + 256 + ks * 128);
+      const int r0 = (p.chunk0 + i) * DC_T + 8 * ks + 2 * j;
+      float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g;
+      if (r0 < seq.n) {
+        dst[0] = o.x + t.x;
+        dst[8] = o.z + t.z;
+      }
+      if (r0 + 1 < seq.n) {
+        dst[a.ld_o] = o.y + t.y;
+        dst[a.ld_o + 8] = o.w + t.w;
       }
     }
+    if (++at == STAGES) { at = 0; phase ^= 1; }
   }
   if (*cta_abort) {
     for (int i = 0; i < 64; ++i) __nanosleep(1000);     // copies in flight land
@@ -448,17 +434,17 @@ delta_scan_kernel(const DeltaChunkParams p) {
   }
   if (!on) return;
 #pragma unroll
-  for (int t = 0; t < 8; ++t)
+  for (int t = 0; t < 4; ++t)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
-      const int d = 64 * ks + 8 * t + 2 * j + (e & 1);
+      const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
       if (d < DP) st[(size_t)d * VP + (e >> 1) * 8] = s[t][e];
     }
 }
 
 template <int KS>
 static int launch_scan(const DeltaChunkParams& p, cudaStream_t st) {
-  constexpr int SMEM = DC_STAGES * dc_block_bytes(64 * KS) + 2 * 4 * 512 * 4;
+  constexpr int SMEM = ds_stages(KS) * ds_stage_bytes(KS) + 2 * DS_WARPS * 512 * 4;
   auto kern = delta_scan_kernel<KS>;
   static bool raised[64] = {};
   int dev = 0;
@@ -467,7 +453,7 @@ static int launch_scan(const DeltaChunkParams& p, cudaStream_t st) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return launch_check("delta_scan attr", 0);
     raised[dev & 63] = true;
   }
-  kern<<<dim3(ceil_div(p.a.vdim_p, 16 * (4 / KS)), p.a.heads, p.a.n_seqs), 128, SMEM, st>>>(p);
+  kern<<<dim3(ceil_div(p.a.vdim_p, 16 * (DS_WARPS / KS)), p.a.heads, p.a.n_seqs), DS_WARPS * 32, SMEM, st>>>(p);
   return launch_check("delta_scan");
 }
 
@@ -517,7 +503,7 @@ extern "C" int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* 
   for (p.chunk0 = 0; p.chunk0 < total; p.chunk0 += round) {
     p.n_chunks = std::min(round, total - p.chunk0);
     int rc = p.dk == 64 ? launch_prepare<32>(p, st) : p.dk == 128 ? launch_prepare<64>(p, st) : launch_prepare<128>(p, st);
-    if (rc == 0) rc = p.dk == 64 ? launch_scan<1>(p, st) : p.dk == 128 ? launch_scan<2>(p, st) : launch_scan<4>(p, st);
+    if (rc == 0) rc = p.dk == 64 ? launch_scan<2>(p, st) : p.dk == 128 ? launch_scan<4>(p, st) : launch_scan<8>(p, st);
     if (rc) return rc;
   }
   return 0;

@@ -131,7 +131,7 @@ gemv_bf16_kernel(const GemvParams p) {
 // tensor-core path), negative on a launch error.
 int try_launch_gemv(const nfn_gemm_args& a, cudaStream_t stream) {
   const int unsupported = NFN_EPI_SAVE_PRE | NFN_EPI_DACT;
-  if (a.m > 2 || a.a_mn || a.b_mn || (a.flags & unsupported) || (a.k & 7) || a.k < 256) return 0;
+  if (a.m > 2 || a.a_mn || a.b_mn || (a.flags & unsupported) || (a.k & 7) || a.k < 64) return 0;
   GemvParams p;
   p.a = static_cast<const __nv_bfloat16*>(a.a);
   p.b = static_cast<const __nv_bfloat16*>(a.b);

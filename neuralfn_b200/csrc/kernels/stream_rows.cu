@@ -51,7 +51,6 @@ stream_pass_kernel(const nfn_stream_args p) {
       }
     }
   };
-  if (threadIdx.x < vecs) fetch(threadIdx.x);
   if (threadIdx.x < S * S) {
     const int s = threadIdx.x / S, t = threadIdx.x % S;
     w_mix[s][t] = (s < n && t < n) ? (p.mix ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.mix)[s * n + t]) : (s == t ? 1.f : 0.f)) : 0.f;
@@ -61,6 +60,9 @@ stream_pass_kernel(const nfn_stream_args p) {
     w_out[s] = s < n ? (p.out ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.out)[s]) : 1.f) : 0.f;
     w_in[s] = s < n ? (p.in ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.in)[s]) : 1.f) : 0.f;
   }
+  if (threadIdx.x < vecs) fetch(threadIdx.x);
+  float4 wt = make_float4(0.f, 0.f, 0.f, 0.f);             // the norm's weights of the first piece come along
+  if (p.h && threadIdx.x < vecs) wt = load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * threadIdx.x);
   __syncthreads();
   float ss = 0.f;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
@@ -105,7 +107,7 @@ stream_pass_kernel(const nfn_stream_args p) {
   const float rms = 1.f / sqrtf(st_block_sum<ST_THREADS>(ss, red) / (float)p.width + p.eps);
   T* h = static_cast<T*>(p.h) + (size_t)r * p.ld;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
-    const float4 u = load4(st_row + 4 * v), w = load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * v);
+    const float4 u = load4(st_row + 4 * v), w = v == threadIdx.x ? wt : load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * v);
     store4(h + 4 * v, make_float4(u.x * rms * (w.x + p.weight_offset), u.y * rms * (w.y + p.weight_offset), u.z * rms * (w.z + p.weight_offset),
                                   u.w * rms * (w.w + p.weight_offset)));
   }
