@@ -28,6 +28,7 @@ using nfn_eng::efail;
 namespace {
 
 constexpr int kPage = NFN_KV_PAGE, kTileMin = 16, kMixRows = 16;
+constexpr float kUnitEps = 1e-6f;                   // of the delta rule's unit vectors
 
 int up(int v, int m) { return (v + m - 1) / m * m; }
 
@@ -116,11 +117,13 @@ struct layered_engine final : nfn_engine {
   void trim(int slot);                              // pages no later query of this slot can see
   int lin(const void* a, int lda, const void* w, int rows, int n, int k, void* out, int ldo, int kind, const void* bias = nullptr);
   // the rows of one pass: short entries first, then the long ones
-  struct Batch { int rows = 0, short_rows = 0, n_mix = 0, n_seq = 0, n_short_seq = 0, longest = 0; std::vector<int> att_off, att_n; };
+  struct Batch { int rows = 0, short_rows = 0, n_mix = 0, n_seq = 0, n_short_seq = 0, longest = 0; bool single = false; std::vector<int> att_off, att_n; };
   int mix_rows(const Layer& L, const Batch& b, void* ff_out);
   int attention(const Layer& L, const Batch& b);
   int delta(const Layer& L, const Batch& b);
   bool grouped(const Layer& L, int rows) const { return c.dtype == 0 && L.d.experts <= 256 && L.d.top <= 32 && (long long)rows * L.d.top > 8LL * L.d.experts; }
+  // single tokens of delta layers: convolution, rule, norm and gate in one launch
+  bool one_step(const Layer& L, const Batch& b) const { return b.single && L.d.mixer == NFN_MIXER_DELTA && nfn_delta_step_fits(b.rows, L.d.heads, L.dp, L.vp); }
   int experts(const Layer& L, int rows, nfn_stream_args* sp);
   int pass(const Batch& b);
   int chained_pass(const Batch& b);
@@ -624,11 +627,22 @@ int layered_engine::delta(const Layer& L, const Batch& b) {
   const char* low = static_cast<const char*>(in);
   if (lin(low + (size_t)L.off_a1 * es, L.n_in, L.w_a2, b.rows, n_dec, L.ra, decay, n_dec, kOutF32)) return -1;
   if (lin(low + (size_t)L.off_g1 * es, L.n_in, L.w_g2, b.rows, n_o, L.rg, d_gate, n_o, kOutAct)) return -1;
+  if (one_step(L, b)) {
+    nfn_delta_step_args t{};
+    t.f32 = c.dtype == 1; t.rows = b.rows; t.in = in; t.ld_in = L.n_in; t.off_beta = L.off_b;
+    t.conv = L.conv; t.taps = d.conv_taps; t.history = L.state; t.history_half = L.state_half;
+    t.decay = decay; t.ld_decay = n_dec; t.a_log = L.a_log; t.dt_bias = L.dt_bias;
+    t.heads = d.heads; t.kv_heads = d.kv_heads; t.dim = d.dim; t.vdim = d.vdim; t.dim_p = L.dp; t.vdim_p = L.vp;
+    t.unit_eps = kUnitEps; t.norm_eps = c.norm_eps; t.state = L.memory;
+    t.gate = d_gate; t.ld_gate = n_o; t.weight = L.out_norm; t.out = cat; t.ld_out = L.n_cat; t.tiles = dev<nfn_row_tile>(io.mix);
+    K(nfn_delta_step(&t, stream));
+    return 0;
+  }
   nfn_delta_args a{};
   a.f32 = c.dtype == 1; a.qkv = q; a.ld_qkv = L.nq;
   a.beta = low + (size_t)L.off_b * es; a.ld_beta = L.n_in;
   a.decay = decay; a.ld_decay = n_dec; a.a_log = L.a_log; a.dt_bias = L.dt_bias;
-  a.heads = d.heads; a.kv_heads = d.kv_heads; a.dim = d.dim; a.dim_p = L.dp; a.vdim_p = L.vp; a.unit_eps = 1e-6f;
+  a.heads = d.heads; a.kv_heads = d.kv_heads; a.dim = d.dim; a.dim_p = L.dp; a.vdim_p = L.vp; a.unit_eps = kUnitEps;
   a.state = L.memory; a.o = d_o; a.ld_o = n_o;
   const bool chunks = c.dtype == 0 && L.dp <= 256;
   a.seqs = dev<nfn_seq_rows>(io.seq); a.n_seqs = chunks ? b.n_short_seq : b.n_seq;
@@ -721,7 +735,8 @@ int layered_engine::chained_pass(const Batch& b) {
   s.tokens = nullptr; s.embed = nullptr;
   for (int l = 0; l < c.n_layer; ++l) {
     const Layer& L = layers[l];
-    if (lin(h, wp, L.w_in, b.rows, L.n_in, wp, in, L.n_in, kOutAct, L.bias_in) || mix_rows(L, b, nullptr)) return -1;
+    if (lin(h, wp, L.w_in, b.rows, L.n_in, wp, in, L.n_in, kOutAct, L.bias_in)) return -1;
+    if (!one_step(L, b) && mix_rows(L, b, nullptr)) return -1;
     if (L.d.mixer == NFN_MIXER_DELTA ? delta(L, b) : attention(L, b)) return -1;
     if (lin(cat, L.n_cat, L.w_out, b.rows, wp, L.n_cat, y, wp, kOutAct)) return -1;
     s.y = y; s.y_rows = 1; s.y_index = nullptr; s.mix = L.hc[0].mix; s.out = L.hc[0].out;
@@ -849,6 +864,7 @@ int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* 
   b.rows = rows;
   b.short_rows = short_rows;
   b.n_mix = n_mix;
+  b.single = single;
   const long long before = nfn_launch_count();
   auto body = [&]() -> int {
     if (pass(b)) return -1;

@@ -344,61 +344,102 @@ delta_scan_kernel(const DeltaChunkParams p) {
       s[t][e] = (on && !fresh && d < DP) ? st[(size_t)d * VP + (e >> 1) * 8] : 0.f;
     }
   __syncthreads();
-  bool ok = true;
+  // Products that every warp of a column tile adds up: W S of this chunk, which the next state waits for, and Q S of the chunk before, which
+  // nothing waits for and which is formed while the partial sums of W S cross shared memory.
   int at = 0, phase = 0;
-  for (int i = 0; i < n_chunks; ++i) {
-    ok = mbar_wait_bounded(smem_u32(&bar_full[at]), phase, cta_abort, p.status, NFN_ERR_WAIT_FULL);
-    const unsigned char* stage = dc_smem + at * STAGE;
-    float acc[4][4], low[4][4];                          // (W S)^T row tiles 0, 1, then (Q S)^T: high x high, and the products with a low part
+  uint32_t hi[2][4], lo[2][4];                           // S, split
+  auto product = [&](const unsigned char* stage, int nt0, float (&acc)[2][4]) {      // two row tiles of [W, Q] times S, transposed
+    float low[2][4];
 #pragma unroll
     for (int kk = 0; kk < 2; ++kk) {
-      uint32_t hi[4], lo[4];
-      split_bf16(s[2 * kk][0], s[2 * kk][1], hi[0], lo[0]);
-      split_bf16(s[2 * kk][2], s[2 * kk][3], hi[1], lo[1]);
-      split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[2], lo[2]);
-      split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
-      uint4 b[4];
+      uint4 b[2];
 #pragma unroll
-      for (int nt = 0; nt < 4; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((2 * ks + kk) * 4 + nt, lane, false));
+      for (int nt = 0; nt < 2; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((2 * ks + kk) * 4 + nt0 + nt, lane, false));
 #pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {
-        if (kk == 0) dc_mma0(acc[nt], hi, b[nt].x, b[nt].z);
-        else dc_mma(acc[nt], hi, b[nt].x, b[nt].z);
+      for (int nt = 0; nt < 2; ++nt) {
+        if (kk == 0) dc_mma0(acc[nt], hi[kk], b[nt].x, b[nt].z);
+        else dc_mma(acc[nt], hi[kk], b[nt].x, b[nt].z);
       }
 #pragma unroll
-      for (int nt = 0; nt < 4; ++nt) {
-        if (kk == 0) dc_mma0(low[nt], hi, b[nt].y, b[nt].w);
-        else dc_mma(low[nt], hi, b[nt].y, b[nt].w);
+      for (int nt = 0; nt < 2; ++nt) {
+        if (kk == 0) dc_mma0(low[nt], hi[kk], b[nt].y, b[nt].w);
+        else dc_mma(low[nt], hi[kk], b[nt].y, b[nt].w);
       }
 #pragma unroll
-      for (int nt = 0; nt < 4; ++nt) dc_mma(low[nt], lo, b[nt].x, b[nt].z);
+      for (int nt = 0; nt < 2; ++nt) dc_mma(kk == 0 ? acc[nt] : low[nt], lo[kk], b[nt].x, b[nt].z);
     }
+#pragma unroll
+    for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[nt][e] += low[nt][e];
+  };
+  auto put = [&](int i, int nt0, const float (&acc)[2][4]) {
     float* mine = xch + ((i & 1) * DS_WARPS + warp) * 512 + lane * 4;
 #pragma unroll
-    for (int nt = 0; nt < 4; ++nt)
-      *reinterpret_cast<float4*>(mine + nt * 128) = make_float4(acc[nt][0] + low[nt][0], acc[nt][1] + low[nt][1], acc[nt][2] + low[nt][2], acc[nt][3] + low[nt][3]);
-    // every warp is done with chunk i - 1 here: its stage takes the next load
-    if (!__syncthreads_and(ok)) break;
-    if (tid == 0 && i > 0 && i - 1 + STAGES < n_chunks) load(i - 1 + STAGES);
+    for (int nt = 0; nt < 2; ++nt) *reinterpret_cast<float4*>(mine + (nt0 + nt) * 128) = make_float4(acc[nt][0], acc[nt][1], acc[nt][2], acc[nt][3]);
+  };
+  auto sum = [&](int i, int nt) {
     const float* all = xch + ((i & 1) * DS_WARPS + warp / KS * KS) * 512 + lane * 4;
-    auto sum = [&](int nt) {
-      float4 t = *reinterpret_cast<const float4*>(all + nt * 128);
+    float4 t = *reinterpret_cast<const float4*>(all + nt * 128);
 #pragma unroll
-      for (int w = 1; w < KS; ++w) {
-        const float4 b = *reinterpret_cast<const float4*>(all + w * 512 + nt * 128);
-        t.x += b.x; t.y += b.y; t.z += b.z; t.w += b.w;
+    for (int w = 1; w < KS; ++w) {
+      const float4 b = *reinterpret_cast<const float4*>(all + w * 512 + nt * 128);
+      t.x += b.x; t.y += b.y; t.z += b.z; t.w += b.w;
+    }
+    return t;
+  };
+  // read-outs of chunk i, whose partial sums were exchanged with those of step `x`: the warps of a column tile take one of two row tiles and
+  // one or both column halves
+  constexpr bool SPLIT = KS >= 4;
+  auto read_out = [&](int i, int x) {
+    if (!on || ks >= (SPLIT ? 4 : 2)) return;
+    const int tile = ks & 1, half = SPLIT ? ks >> 1 : 0;
+    const float* o = reinterpret_cast<const float*>(dc_smem + (i % STAGES) * STAGE + BLOCK) + (warp / KS) * 512 + 256 + tile * 128 + lane * 4;
+    const float* all = xch + ((x & 1) * DS_WARPS + warp / KS * KS) * 512 + (2 + tile) * 128 + lane * 4;
+    const int r0 = (p.chunk0 + i) * DC_T + 8 * tile + 2 * j;
+    float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g;
+#pragma unroll
+    for (int hf = 0; hf < (SPLIT ? 1 : 2); ++hf) {
+      const int c = 2 * (half + hf);
+      float2 t = *reinterpret_cast<const float2*>(o + c);
+#pragma unroll
+      for (int w = 0; w < KS; ++w) {
+        const float2 f = *reinterpret_cast<const float2*>(all + w * 512 + c);
+        t.x += f.x; t.y += f.y;
       }
-      return t;
-    };
+      if (r0 < seq.n) dst[4 * c] = t.x;
+      if (r0 + 1 < seq.n) dst[a.ld_o + 4 * c] = t.y;
+    }
+  };
+  float qs[2][4];
+  for (int i = 0; i < n_chunks; ++i) {
+    mbar_wait_bounded(smem_u32(&bar_full[at]), phase, cta_abort, p.status, NFN_ERR_WAIT_FULL);
+    const unsigned char* stage = dc_smem + at * STAGE;
+#pragma unroll
+    for (int kk = 0; kk < 2; ++kk) {
+      split_bf16(s[2 * kk][0], s[2 * kk][1], hi[kk][0], lo[kk][0]);
+      split_bf16(s[2 * kk][2], s[2 * kk][3], hi[kk][1], lo[kk][1]);
+      split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[kk][2], lo[kk][2]);
+      split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[kk][3], lo[kk][3]);
+    }
+    float ws[2][4];
+    product(stage, 0, ws);
+    if (i > 0) put(i, 2, qs);
+    put(i, 0, ws);
+    // every warp is done with chunk i - 2 here: its stage takes the next load
+    __syncthreads();
+    const int gave_up = *cta_abort;                      // set before the barrier by a thread whose wait ran out: all leave together
+    if (tid == 0 && i > 1 && i - 2 + STAGES < n_chunks) load(i - 2 + STAGES);
+    const float4 w0 = sum(i, 0), w1 = sum(i, 1);
+    product(stage, 2, qs);
     // U^T, as the A operand of S'^T = e^G_last S^T + U^T K
     const float* tv = reinterpret_cast<const float*>(stage + BLOCK) + (warp / KS) * 512 + lane * 4;
+    const float4 v0 = *reinterpret_cast<const float4*>(tv), v1 = *reinterpret_cast<const float4*>(tv + 128);
     uint32_t uh[4], ul[4];
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt) {
-      const float4 t = sum(nt), v = *reinterpret_cast<const float4*>(tv + nt * 128);
-      split_bf16(v.x - t.x, v.y - t.y, uh[2 * nt], ul[2 * nt]);
-      split_bf16(v.z - t.z, v.w - t.w, uh[2 * nt + 1], ul[2 * nt + 1]);
-    }
+    split_bf16(v0.x - w0.x, v0.y - w0.y, uh[0], ul[0]);
+    split_bf16(v0.z - w0.z, v0.w - w0.w, uh[1], ul[1]);
+    split_bf16(v1.x - w1.x, v1.y - w1.y, uh[2], ul[2]);
+    split_bf16(v1.z - w1.z, v1.w - w1.w, uh[3], ul[3]);
     const float* gamma = reinterpret_cast<const float*>(stage + 48 * DK * 4) + DS_CH * ks + 2 * j;
     uint4 kb[4];
 #pragma unroll
@@ -413,21 +454,13 @@ delta_scan_kernel(const DeltaChunkParams p) {
     for (int t = 0; t < 4; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
 #pragma unroll
     for (int t = 0; t < 4; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
-    if (on && ks < 2) {                                  // read-outs: the first two warps of a column tile take eight rows each
-      const float4 t = sum(2 + ks), o = *reinterpret_cast<const float4*>(tv + 256 + ks * 128);
-      const int r0 = (p.chunk0 + i) * DC_T + 8 * ks + 2 * j;
-      float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g;
-      if (r0 < seq.n) {
-        dst[0] = o.x + t.x;
-        dst[8] = o.z + t.z;
-      }
-      if (r0 + 1 < seq.n) {
-        dst[a.ld_o] = o.y + t.y;
-        dst[a.ld_o + 8] = o.w + t.w;
-      }
-    }
+    if (gave_up) break;
+    if (i > 0) read_out(i - 1, i);
     if (++at == STAGES) { at = 0; phase ^= 1; }
   }
+  if (!*cta_abort) put(n_chunks, 2, qs);
+  __syncthreads();
+  if (!*cta_abort) read_out(n_chunks - 1, n_chunks);
   if (*cta_abort) {
     for (int i = 0; i < 64; ++i) __nanosleep(1000);     // copies in flight land
     return;

@@ -421,6 +421,24 @@ int nfn_delta_rows(const nfn_delta_args* args, nfn_stream_t stream);     // toke
 // Sixteen tokens at a time on the tensor cores (bf16, dim_p <= 256), for sequences of up to max_rows rows.
 long long nfn_delta_chunk_workspace_bytes(int heads, int dim_p, int vdim_p, int max_seqs);   // 0: these sizes go token after token
 int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* workspace, long long workspace_bytes, nfn_stream_t stream);
+// One token of every sequence, from the input product to the rows the output product reads: convolution with its history (tiles: one per row),
+// SiLU, the rule, the output norm and gate. in: [q | k | v] at column 0, beta at off_beta; conv [taps][channels], taps >= 1; history as in
+// nfn_mix_args. nfn_delta_step_fits: the sizes it takes, and few enough heads and rows for its large CTAs (more rows run faster as
+// nfn_mix_rows, nfn_delta_rows, nfn_delta_out).
+typedef struct {
+  int f32, rows;
+  const void* in; int ld_in, off_beta;
+  const void* conv; int taps; void* history; long long history_half;
+  const float* decay; int ld_decay; const void* a_log; const void* dt_bias;
+  int heads, kv_heads, dim, vdim, dim_p, vdim_p;
+  float unit_eps, norm_eps;
+  float* state;
+  const void* gate; int ld_gate; const void* weight;
+  void* out; int ld_out;
+  const nfn_row_tile* tiles;
+} nfn_delta_step_args;
+int nfn_delta_step_fits(int rows, int heads, int dim_p, int vdim_p);
+int nfn_delta_step(const nfn_delta_step_args* args, nfn_stream_t stream);
 // out = o / rms(o) * weight * sigmoid(gate) per head of vdim values (pitch vdim_p); weight bf16 [vdim_p], out and gate in the activation type.
 int nfn_delta_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, float eps, void* out, int ld_out, int rows,
                   int heads, int vdim, int vdim_p, nfn_stream_t stream);
