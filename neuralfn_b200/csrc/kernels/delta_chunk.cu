@@ -8,7 +8,7 @@
 //
 //   delta_prepare_kernel  one CTA per (chunk, head), all chunks at once: W, Q, K and T V, P T V. A thread owns two channels; their
 //                         products for all pairs of tokens are formed in registers and summed over channels through shared memory.
-//   delta_scan_kernel     one warp per (head, 16 value columns, 32 key channels), one chunk after another: the state, transposed, sits in
+//   delta_scan_kernel     one warp per (head, 16 value columns, 64 key channels), one chunk after another: the state, transposed, sits in
 //                         the accumulator registers of mma.m16n8k16 and is the A operand of the next chunk's W S and Q S as it stands; W, Q
 //                         and K arrive in fragment order by bulk copies through a ring of shared memory stages.
 //
@@ -292,11 +292,11 @@ __device__ __forceinline__ void dc_bulk_load(uint32_t dst, const void* src, uint
   asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 
-// KS: warps that share a head's key channels, 32 each; the CTA's eight warps take 8 / KS tiles of 16 value columns
-constexpr int DS_WARPS = 8, DS_CH = 32;
+// KS: warps that share a head's key channels, 64 each; the CTA's four warps take 4 / KS tiles of 16 value columns
+constexpr int DS_WARPS = 4, DS_CH = 64, DS_K = DS_CH / 16, DS_N = DS_CH / 8;      // a warp's steps of 16 and tiles of 8 channels
 // shared memory of a stage: the head's operand block, then T V and P T V of the CTA's column tiles
 __host__ __device__ constexpr int ds_stage_bytes(int ks) { return dc_block_bytes(DS_CH * ks) + DS_WARPS / ks * 2048; }
-__host__ __device__ constexpr int ds_stages(int ks) { return ks == 8 ? 3 : 4; }
+__host__ __device__ constexpr int ds_stages(int ks) { return ks == 4 ? 3 : 4; }
 template <int KS>
 __global__ void __launch_bounds__(DS_WARPS * 32)
 delta_scan_kernel(const DeltaChunkParams p) {
@@ -332,12 +332,12 @@ delta_scan_kernel(const DeltaChunkParams p) {
     fence_mbar_init();
     for (int i = 0; i < min(STAGES, n_chunks); ++i) load(i);
   }
-  // S^T: rows are value columns (g, g + 8), columns key channels 32 ks + 8 t + 2 j, + 1
+  // S^T: rows are value columns (g, g + 8), columns key channels 64 ks + 8 t + 2 j, + 1
   float* st = a.state + ((size_t)seq.slot * a.heads + h) * DP * VP + vt * 16 + g;
   const bool fresh = seq.pos0 == 0 && p.chunk0 == 0;
-  float s[4][4];
+  float s[DS_N][4];
 #pragma unroll
-  for (int t = 0; t < 4; ++t)
+  for (int t = 0; t < DS_N; ++t)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
@@ -347,14 +347,14 @@ delta_scan_kernel(const DeltaChunkParams p) {
   // Products that every warp of a column tile adds up: W S of this chunk, which the next state waits for, and Q S of the chunk before, which
   // nothing waits for and which is formed while the partial sums of W S cross shared memory.
   int at = 0, phase = 0;
-  uint32_t hi[2][4], lo[2][4];                           // S, split
+  uint32_t hi[DS_K][4], lo[DS_K][4];                           // S, split
   auto product = [&](const unsigned char* stage, int nt0, float (&acc)[2][4]) {      // two row tiles of [W, Q] times S, transposed
     float low[2][4];
 #pragma unroll
-    for (int kk = 0; kk < 2; ++kk) {
+    for (int kk = 0; kk < DS_K; ++kk) {
       uint4 b[2];
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((2 * ks + kk) * 4 + nt0 + nt, lane, false));
+      for (int nt = 0; nt < 2; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((DS_K * ks + kk) * 4 + nt0 + nt, lane, false));
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
         if (kk == 0) dc_mma0(acc[nt], hi[kk], b[nt].x, b[nt].z);
@@ -366,7 +366,7 @@ delta_scan_kernel(const DeltaChunkParams p) {
         else dc_mma(low[nt], hi[kk], b[nt].y, b[nt].w);
       }
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) dc_mma(kk == 0 ? acc[nt] : low[nt], lo[kk], b[nt].x, b[nt].z);
+      for (int nt = 0; nt < 2; ++nt) dc_mma((kk & 1) == 0 ? acc[nt] : low[nt], lo[kk], b[nt].x, b[nt].z);
     }
 #pragma unroll
     for (int nt = 0; nt < 2; ++nt)
@@ -388,27 +388,25 @@ delta_scan_kernel(const DeltaChunkParams p) {
     }
     return t;
   };
-  // read-outs of chunk i, whose partial sums were exchanged with those of step `x`: the warps of a column tile take one of two row tiles and
-  // one or both column halves
-  constexpr bool SPLIT = KS >= 4;
+  // read-outs of chunk i, whose partial sums were exchanged with those of step `x`, shared out among the warps of a column tile: each takes some of
+  // (row tile, column half)
+  constexpr int PARTS = 4 / KS;
   auto read_out = [&](int i, int x) {
-    if (!on || ks >= (SPLIT ? 4 : 2)) return;
-    const int tile = ks & 1, half = SPLIT ? ks >> 1 : 0;
-    const float* o = reinterpret_cast<const float*>(dc_smem + (i % STAGES) * STAGE + BLOCK) + (warp / KS) * 512 + 256 + tile * 128 + lane * 4;
-    const float* all = xch + ((x & 1) * DS_WARPS + warp / KS * KS) * 512 + (2 + tile) * 128 + lane * 4;
-    const int r0 = (p.chunk0 + i) * DC_T + 8 * tile + 2 * j;
-    float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g;
+    if (!on) return;
 #pragma unroll
-    for (int hf = 0; hf < (SPLIT ? 1 : 2); ++hf) {
-      const int c = 2 * (half + hf);
-      float2 t = *reinterpret_cast<const float2*>(o + c);
+    for (int n = 0; n < PARTS; ++n) {
+      const int tile = (ks * PARTS + n) >> 1, c = 2 * ((ks * PARTS + n) & 1);
+      float2 t = *reinterpret_cast<const float2*>(dc_smem + (i % STAGES) * STAGE + BLOCK + ((warp / KS) * 512 + 256 + tile * 128 + lane * 4 + c) * 4);
+      const float* all = xch + ((x & 1) * DS_WARPS + warp / KS * KS) * 512 + (2 + tile) * 128 + lane * 4 + c;
 #pragma unroll
       for (int w = 0; w < KS; ++w) {
-        const float2 f = *reinterpret_cast<const float2*>(all + w * 512 + c);
+        const float2 f = *reinterpret_cast<const float2*>(all + w * 512);
         t.x += f.x; t.y += f.y;
       }
-      if (r0 < seq.n) dst[4 * c] = t.x;
-      if (r0 + 1 < seq.n) dst[a.ld_o + 4 * c] = t.y;
+      const int r0 = (p.chunk0 + i) * DC_T + 8 * tile + 2 * j;
+      float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g + 4 * c;
+      if (r0 < seq.n) dst[0] = t.x;
+      if (r0 + 1 < seq.n) dst[a.ld_o] = t.y;
     }
   };
   float qs[2][4];
@@ -416,7 +414,7 @@ delta_scan_kernel(const DeltaChunkParams p) {
     mbar_wait_bounded(smem_u32(&bar_full[at]), phase, cta_abort, p.status, NFN_ERR_WAIT_FULL);
     const unsigned char* stage = dc_smem + at * STAGE;
 #pragma unroll
-    for (int kk = 0; kk < 2; ++kk) {
+    for (int kk = 0; kk < DS_K; ++kk) {
       split_bf16(s[2 * kk][0], s[2 * kk][1], hi[kk][0], lo[kk][0]);
       split_bf16(s[2 * kk][2], s[2 * kk][3], hi[kk][1], lo[kk][1]);
       split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[kk][2], lo[kk][2]);
@@ -441,19 +439,19 @@ delta_scan_kernel(const DeltaChunkParams p) {
     split_bf16(v1.x - w1.x, v1.y - w1.y, uh[2], ul[2]);
     split_bf16(v1.z - w1.z, v1.w - w1.w, uh[3], ul[3]);
     const float* gamma = reinterpret_cast<const float*>(stage + 48 * DK * 4) + DS_CH * ks + 2 * j;
-    uint4 kb[4];
+    uint4 kb[DS_N];
 #pragma unroll
-    for (int t = 0; t < 4; ++t) {
+    for (int t = 0; t < DS_N; ++t) {
       const float2 f = *reinterpret_cast<const float2*>(gamma + 8 * t);
-      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece(4 * (DK / 16) + 4 * ks + t, lane, true));
+      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece(4 * (DK / 16) + DS_N * ks + t, lane, true));
       s[t][0] *= f.x; s[t][1] *= f.y; s[t][2] *= f.x; s[t][3] *= f.y;
     }
 #pragma unroll
-    for (int t = 0; t < 4; ++t) dc_mma(s[t], uh, kb[t].x, kb[t].z);
+    for (int t = 0; t < DS_N; ++t) dc_mma(s[t], uh, kb[t].x, kb[t].z);
 #pragma unroll
-    for (int t = 0; t < 4; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
+    for (int t = 0; t < DS_N; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
 #pragma unroll
-    for (int t = 0; t < 4; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
+    for (int t = 0; t < DS_N; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
     if (gave_up) break;
     if (i > 0) read_out(i - 1, i);
     if (++at == STAGES) { at = 0; phase ^= 1; }
@@ -467,7 +465,7 @@ delta_scan_kernel(const DeltaChunkParams p) {
   }
   if (!on) return;
 #pragma unroll
-  for (int t = 0; t < 4; ++t)
+  for (int t = 0; t < DS_N; ++t)
 #pragma unroll
     for (int e = 0; e < 4; ++e) {
       const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
@@ -536,7 +534,7 @@ extern "C" int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* 
   for (p.chunk0 = 0; p.chunk0 < total; p.chunk0 += round) {
     p.n_chunks = std::min(round, total - p.chunk0);
     int rc = p.dk == 64 ? launch_prepare<32>(p, st) : p.dk == 128 ? launch_prepare<64>(p, st) : launch_prepare<128>(p, st);
-    if (rc == 0) rc = p.dk == 64 ? launch_scan<2>(p, st) : p.dk == 128 ? launch_scan<4>(p, st) : launch_scan<8>(p, st);
+    if (rc == 0) rc = p.dk == 64 ? launch_scan<1>(p, st) : p.dk == 128 ? launch_scan<2>(p, st) : launch_scan<4>(p, st);
     if (rc) return rc;
   }
   return 0;
