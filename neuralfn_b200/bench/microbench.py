@@ -358,7 +358,87 @@ def case_paged(args):
             bytes_=4.0 * B * G * seen * D, args=args, extra={**extra, "B": B, "context": ctx})
 
 
-CASES = {"gemm": case_gemm, "paged": case_paged, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
+def case_layered(args):
+    """Kernels of delta-rule layers, streams and routed experts beside their closest counterparts, at one layer of ``--heads`` / ``--kv-heads`` x
+    ``--head-dim``, width ``--k``, ``--experts`` experts of which four of ``--n`` / 4 are used, four streams, ``--window`` with four kept tokens."""
+    from neuralfn_b200.ops import infer as I, kernels as K, layered as Y, paged as P
+    from neuralfn_b200.ops.gemm import gemm
+    from neuralfn_b200.ops.moe import MoEWorkspace, _grouped_gemm, moe_forward
+    dev = torch.device("cuda")
+    H, G, D, T, B, W, C, E = args.heads, args.kv_heads or args.heads, args.head_dim, args.seq, args.batch, args.window, args.k, args.experts
+    F, S = args.n // 4, 4
+    rand = lambda *s: torch.randn(*s, device=dev).bfloat16()  # noqa: E731
+    t = lambda fn: time_kernel(fn, args.iters, args.warmup, args.flush)  # noqa: E731
+    i32 = dict(dtype=torch.int32, device=dev)
+    # attention with kept tokens, soft cap, sink
+    w = min(W or T, T)
+    flops = 4.0 * H * D * (w * (w + 1) / 2 + (T - w) * w)
+    c = P.PagedCache(1, T, G, D, D, dev)
+    c.k.normal_(), c.v.normal_()
+    q, out = rand(T, H * D), torch.empty(T, H * D, device=dev, dtype=torch.bfloat16)
+    step = P.tile_rows(c, H)
+    tiles = torch.tensor([[r, min(step, T - r), 0, r] for r in range(0, T, step)], **i32)
+    kw = dict(heads=H, window=W, scale=D ** -0.5, keep_first=4 if W else 0, softcap=30.0, sink=True)
+    _report("paged_attention_tiles (cap, kept, sink)", t(lambda: P.attention_tiles(c, q, tiles, out, **kw)), flops=flops, args=args, extra={"T": T, "window": W})
+    k, v = rand(T, G * D), rand(T, G * D)
+    fa = dict(B=1, T=T, n_q_heads=H, n_kv_heads=G, head_dim=D, causal=True, window=W)
+    o, lse = K.attention_forward(q, k, v, **fa)
+    _report("attention_fwd", t(lambda: K.attention_forward(q, k, v, out=o, lse=lse, **fa)), flops=flops, args=args, extra={"T": T, "window": W})
+    ctx = args.context
+    seen = min(W or ctx, ctx)
+    c = P.PagedCache(B, ctx, G, D, D, dev)
+    c.k.normal_(), c.v.normal_()
+    q1, o1 = rand(B, H * D), torch.empty(B, H * D, device=dev, dtype=torch.bfloat16)
+    slot, pos = torch.arange(B, **i32), torch.full((B,), ctx - 1, **i32)
+    _report("paged_attention_rows (cap, kept, sink)", t(lambda: P.attention_rows(c, q1, slot, pos, o1, **kw)), bytes_=4.0 * B * G * seen * D, args=args, extra={"B": B, "context": ctx})
+    kc, vc, ws = rand(B, G, seen, D), rand(B, G, seen, D), I.DecodeAttentionWorkspace(B, H, G, D, dev)
+    qkv, lens, (cos, sin) = rand(B, (H + 2 * G) * D), torch.full((B,), seen, **i32), I.rope_tables(seen, D, device=dev)
+    _report("decode_attention", t(lambda: I.decode_attention(qkv, kc, vc, lens, n_q_heads=H, n_kv_heads=G, head_dim=D, workspace=ws, cos=cos, sin=sin, qk_norm=True, out=o1)),
+            bytes_=4.0 * B * G * seen * D, args=args, extra={"B": B, "context": ctx})
+    del c, k, v, kc, vc, q, out, o
+    # delta rule: prompt in chunks, decode rows
+    a_log, dt = torch.full((H,), -1.0, device=dev).bfloat16(), torch.full((H * D,), -1.0, device=dev).bfloat16()
+
+    def rule(rows, seqs, slots):
+        x, beta, decay, st = rand(rows, 3 * H * D), rand(rows, H), torch.randn(rows, H * D, device=dev), torch.zeros(slots, H, D, D, device=dev)
+        return dict(qkv=x, beta=beta, decay=decay, a_log=a_log, dt_bias=dt, state=st, seqs=torch.tensor(seqs, **i32), kv_heads=H, dim=D)
+
+    r = rule(T, [[0, T, 0, 0]], 1)
+    wsp = torch.empty(96 << 20, device=dev, dtype=torch.uint8)
+    _report("delta_chunks", t(lambda: Y.delta_rule(**r, form="chunks", workspace=wsp)), flops=7.0 * T * H * D * D, bytes_=14.0 * T * H * D, args=args, extra={"T": T, "heads": H, "dim": D})
+    orow, gate, nw = torch.randn(T, H * D, device=dev), rand(T, H * D), rand(D)
+    _report("delta_out", t(lambda: Y.delta_out(orow, gate, nw, heads=H, vdim=D, eps=1e-5)), bytes_=8.0 * T * H * D, args=args, extra={"T": T})
+    cc, cx, conv, hist = P.PagedCache(1, 64, 1, 16, 16, dev), rand(T, 3 * H * D), rand(4, 3 * H * D), torch.zeros(2, 1, 3, 3 * H * D, device=dev, dtype=torch.bfloat16)
+    cc.dim, qo, rt = 3 * D, torch.empty(T, 3 * H * D, device=dev, dtype=torch.bfloat16), P.row_tiles([(0, 0, T, 0)], dev)
+    _report("mix_rows (SiLU)", t(lambda: P.mix_rows(cc, cx, rt, qo, None, heads=H, own_kv=False, conv=conv, state=hist, conv_act=3)), bytes_=4.0 * T * 3 * H * D, args=args,
+            extra={"T": T, "taps": 4})
+    r1 = rule(B, [[b, 1, b, 7] for b in range(B)], B)
+    _report("delta_rows", t(lambda: Y.delta_rule(**r1)), bytes_=8.0 * B * H * D * D, args=args, extra={"B": B})
+    del r, r1, orow, gate, cx, qo
+    # streams
+    xs, y, h, wt = torch.randn(T, S, C, device=dev), rand(T, C), torch.empty(T, C, device=dev, dtype=torch.bfloat16), rand(C)
+    mix, one = torch.eye(S, device=dev).bfloat16(), torch.ones(S, device=dev).bfloat16()
+    sp = dict(width=C, streams=S, ld=C, f32=False, weight=wt, mix=mix, out=one, into=one)
+    _report("stream_pass", t(lambda: Y.stream_pass(xs, h, rows=T, x_out=xs, y=y, **sp)), bytes_=T * C * (8.0 * S + 4), args=args, extra={"T": T, "width": C, "streams": S})
+    x1 = torch.randn(T, C, device=dev)
+    _report("row_norm (fp32 residual)", t(lambda: P.row_norm(x1, wt, h, eps=1e-5, y=y, y_weight=wt, x_out=x1)), bytes_=12.0 * T * C, args=args, extra={"T": T, "width": C})
+    del xs, x1
+    # experts: prompt (grouped products), decode rows
+    wg, wd, wr = rand(E, 2 * F, C) * C ** -0.5, rand(E, C, F) * F ** -0.5, rand(E, C) * C ** -0.5
+    mw = MoEWorkspace(T, E, 4, C, F, dev)
+    moe_forward(y, wr, wg, wd, 4, mw, score_fn="sigmoid", norm_topk=False)
+    _report("grouped gemm (gate and up)", t(lambda: _grouped_gemm(mw.xs, wg, mw.h, mw)), flops=2.0 * 4 * T * 2 * F * C, args=args, extra={"T": T, "experts": E, "ff": F})
+    wide, dense = rand(8 * F, C), torch.empty(T, 8 * F, device=dev, dtype=torch.bfloat16)
+    _report("gemm (dense, same flops)", t(lambda: gemm(y, wide, out=dense)), flops=2.0 * T * 8 * F * C, args=args, extra={"T": T})
+    y1 = rand(B, C)
+    z = torch.randn(B, E, device=dev)
+    idx, _, _ = Y.expert_rows(y1, z, wg, wd, experts=E, top=4)
+    live = int(idx.unique().numel())
+    _report("expert_rows (routing and products)", t(lambda: Y.expert_rows(y1, z, wg, wd, experts=E, top=4)), bytes_=2.0 * live * 3 * F * C, args=args, extra={"B": B, "experts_used": live})
+    _report("gemm (dense, batch rows)", t(lambda: gemm(y1, wide, out=dense[:B])), bytes_=2.0 * 8 * F * C, args=args, extra={"B": B})
+
+
+CASES = {"gemm": case_gemm, "paged": case_paged, "layered": case_layered, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
          "cross_entropy": case_cross_entropy, "norm": case_norm, "adamw": case_adamw, "decode_attention": case_decode_attention,
          "skinny": case_skinny, "grouped_k": case_grouped_k, "kquant_gemv": case_kquant_gemv, "gemm_kquant": case_gemm_kquant, "block_attention": case_block_attention,
          "turboquant_attention": case_turboquant_attention, "engine_decode": case_engine_decode}
@@ -397,7 +477,7 @@ def main(argv=None):
     ap.add_argument("--window", type=int, default=0, help="paged case: sliding window")
     ap.add_argument("--context", type=int, default=4096, help="paged case: cached tokens per decode row")
     ap.add_argument("--iters", type=int, default=20)
-    ap.add_argument("--experts", type=int, default=16, help="grouped_k case")
+    ap.add_argument("--experts", type=int, default=16, help="grouped_k and layered cases")
     ap.add_argument("--no-baseline", action="store_true", help="grouped_k case: skip the per-expert loop (profiler captures)")
     ap.add_argument("--skinny-impl", type=int, default=-1, help="gemm case: nfn_gemm_skinny_set_impl mode for products with 3 - 64 rows (-1: the default)")
     ap.add_argument("--warmup", type=int, default=5)

@@ -17,6 +17,7 @@
 // to stay in L2.
 #include <algorithm>
 
+#include "attention_v2.cuh"
 #include "common.h"
 #include "delta.cuh"
 
@@ -46,6 +47,10 @@ __device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint3
   lo = pack_bf16x2(a - f.x, b - f.y);
 }
 
+__device__ __forceinline__ void dc_bulk_store(void* dst, uint32_t src, uint32_t bytes) {
+  asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst), "r"(src), "r"(bytes) : "memory");
+}
+
 // log2(1 + e^z): the series of log(1 + t) for small t = e^z keeps slow decays exact
 __device__ __forceinline__ float softplus_log2(float z) {
   const float y = z * 1.4426950408889634f, t = fast_exp2(y);
@@ -63,7 +68,7 @@ __device__ __forceinline__ uint32_t dc_piece(int tile, int lane, bool of_k) {
 
 // NT threads, two neighbouring key channels each (dk = 2 NT), and value columns in pairs
 template <int NT>
-__global__ void __launch_bounds__(NT, 384 / NT)
+__global__ void __launch_bounds__(NT, 448 / NT)
 delta_prepare_kernel(const DeltaChunkParams p) {
   constexpr int PITCH = NT == 128 ? 136 : NT + 4;                 // partial sums [64 values][NT]; rows are read in 16-byte pieces
   extern __shared__ __align__(128) unsigned char dc_smem[];       // partial sums, then the operand block
@@ -94,29 +99,31 @@ delta_prepare_kernel(const DeltaChunkParams p) {
       G[r][0] = z.x;
       G[r][1] = z.y;
     }
-    float* red = reinterpret_cast<float*>(dc_smem);               // [32 sums][warps]
+    // squared lengths: 32 sums over the channels, NT / 32 neighbouring threads each
+    float* part = reinterpret_cast<float*>(dc_smem);
 #pragma unroll
     for (int r = 0; r < DC_T; ++r) {
       const float2 fq = unpack_bf16x2(qw[r]), fk = unpack_bf16x2(kw[r]);
       q[r][0] = fq.x; q[r][1] = fq.y; k[r][0] = fk.x; k[r][1] = fk.y;
-      float nq = fq.x * fq.x + fq.y * fq.y, nk = fk.x * fk.x + fk.y * fk.y;
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        nq += __shfl_xor_sync(0xffffffffu, nq, o);
-        nk += __shfl_xor_sync(0xffffffffu, nk, o);
-      }
-      if (lane == r) red[r * (NT / 32) + warp] = nq;
-      if (lane == 16 + r) red[(16 + r) * (NT / 32) + warp] = nk;
+      part[r * PITCH + tid] = fq.x * fq.x + fq.y * fq.y;
+      part[(DC_T + r) * PITCH + tid] = fk.x * fk.x + fk.y * fk.y;
     }
     __syncthreads();
-    if (tid < 2 * DC_T) {
-      float t = 0.f;
+    constexpr int SHARE = NT / 32;
+    const int v = tid / SHARE;
+    const float* src = part + v * PITCH + tid % SHARE * 32;
+    float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
-      for (int w = 0; w < NT / 32; ++w) t += red[tid * (NT / 32) + w];
-      const float f = 1.f / sqrtf(t + a.unit_eps);
-      s_norm[tid / DC_T][tid % DC_T] = tid < DC_T ? f / sqrtf((float)a.dim) : f;
-      if (tid < DC_T) s_beta[tid] = tid < n ? sigmoid_exact(__bfloat162float(static_cast<const __nv_bfloat16*>(a.beta)[(row0 + tid) * a.ld_beta + h])) : 0.f;
+    for (int i = 0; i < 8; ++i) {
+      const float4 g = *reinterpret_cast<const float4*>(src + 4 * i);
+      f.x += g.x; f.y += g.y; f.z += g.z; f.w += g.w;
     }
+    float t = (f.x + f.y) + (f.z + f.w);
+#pragma unroll
+    for (int o = 1; o < SHARE; o <<= 1) t += __shfl_xor_sync(0xffffffffu, t, o);
+    const float inv = 1.f / sqrtf(t + a.unit_eps);
+    s_norm[v / DC_T][v % DC_T] = v < DC_T ? inv / sqrtf((float)a.dim) : inv;
+    if (tid < DC_T) s_beta[tid] = tid < n ? sigmoid_exact(__bfloat162float(static_cast<const __nv_bfloat16*>(a.beta)[(row0 + tid) * a.ld_beta + h])) : 0.f;
     __syncthreads();
   }
   {
@@ -149,8 +156,9 @@ delta_prepare_kernel(const DeltaChunkParams p) {
         if (j > r) continue;
         float k0 = k[j][0], k1 = k[j][1];
         if (j < r) {
-          k0 *= fast_exp2(G[r][0] - G[j][0]);
-          k1 *= fast_exp2(G[r][1] - G[j][1]);
+          float d0 = G[r][0], d1 = G[r][1];
+          add2f(d0, d1, d0, d1, -G[j][0], -G[j][1]);
+          mul2(k0, k1, k0, k1, fast_exp2(d0), fast_exp2(d1));
         }
         part[at++ * PITCH + tid] = q[r][0] * k0 + q[r][1] * k1;
         if (j < r) part[at++ * PITCH + tid] = k[r][0] * k0 + k[r][1] * k1;
@@ -166,7 +174,8 @@ delta_prepare_kernel(const DeltaChunkParams p) {
 #pragma unroll
       for (int i = 0; i < (NT == 32 ? 8 : 16); ++i) {
         const float4 f = *reinterpret_cast<const float4*>(src + i * (NT == 128 ? 8 : 4));
-        s.x += f.x; s.y += f.y; s.z += f.z; s.w += f.w;
+        add2(s.x, s.y, f.x, f.y);
+        add2(s.z, s.w, f.z, f.w);
       }
       float sum = (s.x + s.y) + (s.z + s.w);
       if (NT == 128) sum += __shfl_xor_sync(0xffffffffu, sum, 1);
@@ -271,10 +280,14 @@ delta_prepare_kernel(const DeltaChunkParams p) {
       }
     }
   }
+  // the finished operand block leaves in one bulk copy
+  fence_proxy_async();
   __syncthreads();
-  const int vecs = dc_block_bytes(p.dk) / 16;
-  uint4* out = reinterpret_cast<uint4*>(p.blocks + block * dc_block_bytes(p.dk));
-  for (int i = tid; i < vecs; i += NT) out[i] = reinterpret_cast<const uint4*>(stage)[i];
+  if (tid == 0) {
+    dc_bulk_store(p.blocks + block * dc_block_bytes(p.dk), smem_u32(stage), dc_block_bytes(p.dk));
+    asm volatile("cp.async.bulk.commit_group;" ::: "memory");
+    asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
+  }
 }
 
 __device__ __forceinline__ void dc_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {

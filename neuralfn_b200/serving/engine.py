@@ -197,7 +197,8 @@ class LayeredEngineConfig:
                 weights += wp * (n_in + v + up(y.ff) + 2 * up(self.side_dim)) + own + wp * (up(y.experts) + 3 * y.experts * up(y.expert_ff))
             routed = max(routed, (rows * y.top + 127 * y.experts) * es * (2 * wp + 3 * up(y.expert_ff)) if y.experts else 0)
         acts = rows * (es * (3 * wp + widest + up(self.side_dim)) + 4 * (wp * max(self.streams, 1) + up(self.side_dim))) + 4 * 2 * max(self.max_batch, 64) * up(self.vocab)
-        return int(2 * weights + cache + acts + routed)
+        chunks = (96 << 20) if es == 2 and any(y.mixer == "delta" for y in self.layers) else 0        # operands of the delta rule's prompt chunks
+        return int(2 * weights + cache + acts + routed + chunks)
 
 
 @dataclass(frozen=True)
@@ -311,7 +312,8 @@ def resident_inference_abi_version() -> int:
 def resident_inference_capabilities() -> dict:
     return {"abi_version": resident_inference_abi_version(), "families": ["gpt2", "llama", "layered"], "kv_cache": "bf16",
             # layer-list models: paged caches, steps of mixed prompt portions and single tokens, bf16 or true 32-bit
-            "paged_kv_cache": ["layered"], "mixed_steps": ["layered"], "float32": ["layered"],
+            "paged_kv_cache": ["layered"], "mixed_steps": ["layered"], "float32": ["layered"], "mixers": {"layered": sorted(LayerSpec.MIXER_IDS)},
+            "recurrent_state": ["layered"], "routed_experts": ["layered"], "residual_streams": ["layered"],
             "hybrid_local_global": True, "qk_norm": True, "rope": ["hf", "legacy"], "continuous_batching": True,
             "cuda_graph_decode": True, "on_device_sampling": ["greedy", "temperature", "top_k", "top_p"],
             # projection weights may stay resident in K-quant blocks (``set_tensor_kquant``: quantised GEMV for up to eight rows,
