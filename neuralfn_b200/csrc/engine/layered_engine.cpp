@@ -8,8 +8,12 @@
 // convolutions keep taps - 1 projected rows per slot and layer in two halves: a step reads one half and writes the other, so no
 // launch reads what it overwrites.
 //
-// Delta-rule layers have no pages: a slot keeps one fp32 state per head, read and written in place. Layers of a loop share tensors and
-// have caches and states of their own.
+// Layers whose keys are limited to chunks of positions give pages back when a chunk ends. Latent layers cache one row per token, [latent | rotated key
+// part], for all heads; single tokens and short portions attend to the latents themselves, long portions to keys and values formed from the
+// visible latents for the pass.
+//
+// Recurrent layers have no pages: a slot keeps one fp32 state per head, read and written in place (and, for the token shift, the previous input in two
+// halves like the convolutions' history). Layers of a loop share tensors and have caches and states of their own.
 //
 // A step lays its rows out short entries first (single tokens and portions below kTileMin rows: one query row at a time), then
 // the long ones (tcgen05 tiles). Per layer it launches: input projection (q | k | v | gates | feed-forward in one product), the
@@ -47,13 +51,38 @@ struct Layer {
   const void *norm1 = nullptr, *w_in = nullptr, *conv = nullptr, *w_out = nullptr, *side_gate = nullptr, *side_proj = nullptr, *side_norm = nullptr;
   const void *norm2 = nullptr, *bias_in = nullptr, *w_a2 = nullptr, *w_g2 = nullptr, *a_log = nullptr, *dt_bias = nullptr, *out_norm = nullptr;
   const void *router = nullptr, *w_gate_up = nullptr, *w_down = nullptr;
+  int rp = 0, lr = 0, off_kv = 0;                   // latent: padded rotated part and latent size, latent columns of the input product
+  int shp = 0;                                      // padded width of the shared expert
+  float* freq = nullptr;                            // rotation: rot_dims / 2 frequencies in two parts
+  const void *q_norm = nullptr, *k_norm = nullptr, *c_norm = nullptr, *w_ukv = nullptr, *w_uk_t = nullptr, *w_uv = nullptr;
+  const void *mu = nullptr, *w1 = nullptr, *w2 = nullptr, *w0 = nullptr, *u = nullptr;
+  const void *w_shared_up = nullptr, *w_shared_down = nullptr, *correction = nullptr;
+  float* prev = nullptr;                            // token shift: [2][slots][wp]
+  bool paged() const { return d.mixer == NFN_MIXER_ATTENTION || d.mixer == NFN_MIXER_LATENT; }
+  bool latent() const { return d.mixer == NFN_MIXER_LATENT; }
+  int key_row() const { return latent() ? lr + rp : d.kv_heads * dp; }       // values of one token's key and value rows in the pages
+  int value_row() const { return latent() ? 0 : d.kv_heads * vp; }
+  int look() const { return d.chunk > 0 ? d.chunk : d.window; }              // most positions a query sees, 0: all
   struct { const void *in = nullptr, *out = nullptr, *mix = nullptr; } hc[2];   // streams: mixer, feed-forward
   int tile_rows = 0;                                // query rows per tcgen05 tile, 0: one row at a time
 };
 
 struct Group {
-  int window = 0;                                   // widest reader, 0: everything stays
+  bool all = false;                                 // a reader sees everything: everything stays
+  int window = 0;                                   // widest reader with a window
+  std::vector<int> chunks;                          // chunk sizes of the readers that have them
   int keep = 0;                                     // first pages that stay whatever the window
+  int look() const {                                // most positions a reader sees, 0: all
+    int n = window;
+    for (int k : chunks) n = std::max(n, k);
+    return all ? 0 : n;
+  }
+  int oldest(int next) const {                      // first position a query at `next` or later can see
+    int p = window > 0 ? std::max(0, next - window + 1) : next;
+    for (int k : chunks) p = std::min(p, next / k * k);
+    return all ? 0 : p;
+  }
+  bool like(const Group& o) const { return all == o.all && window == o.window && chunks == o.chunks && keep == o.keep; }
   int pages = 0;
   bool held(int slot, int p) const { return p < keep || p >= first[slot]; }   // of pages below next[slot]
   std::vector<int> free_pages;
@@ -77,13 +106,19 @@ struct layered_engine final : nfn_engine {
   long long delta_ws_bytes = 0;
   struct { float *logits = nullptr, *weight = nullptr, *row_w = nullptr; int *idx = nullptr, *order = nullptr, *offsets = nullptr, *active = nullptr, *counts = nullptr,
            *cursor = nullptr, *tile_expert = nullptr, *plan = nullptr, *row_of = nullptr; void *xs = nullptr, *gate_up = nullptr, *mid = nullptr, *y = nullptr; } ex;
+  void *q_lat = nullptr, *o_lat = nullptr, *lat_rows = nullptr, *lat_x = nullptr;   // latent: absorbed queries and outputs of short rows; gathered latents, expansion
+  int lat_cap = 0;                                  // rows of the last two
+  void *shift = nullptr, *low_act = nullptr, *shared_mid = nullptr, *y_shared = nullptr;
+  float* low = nullptr;
+  void* wkv_ws = nullptr;
+  long long wkv_ws_bytes = 0;
   nfn_stream_args pend{};                           // chained: the last sublayer's update, applied on the way to the head
   void *att_ws = nullptr, *gemm_ws = nullptr;
   long long att_ws_bytes = 0, gemm_ws_bytes = 0;
   std::vector<uint8_t> parity;                      // per slot: the half that holds its convolution history
   std::vector<int> logit_at;                        // per slot: row of `logits`, -1: none, -2: `saved`
   // per-step block, one copy to the device: offsets in bytes
-  struct { long long tok, slot, pos, want, params, offset, mix, att, seq, out, total; } io{};
+  struct { long long tok, slot, pos, want, params, offset, mix, att, seq, spans, base, out, total; } io{};
   unsigned char *h_io = nullptr, *d_io = nullptr;
   std::map<int, cudaGraphExec_t> graphs;            // by padded row count
   std::map<int, long long> graph_launches;
@@ -115,12 +150,25 @@ struct layered_engine final : nfn_engine {
 
   int reserve(int slot, int upto);                  // pages for positions < upto
   void trim(int slot);                              // pages no later query of this slot can see
-  int lin(const void* a, int lda, const void* w, int rows, int n, int k, void* out, int ldo, int kind, const void* bias = nullptr);
+  int lin(const void* a, int lda, const void* w, int rows, int n, int k, void* out, int ldo, int kind, const void* bias = nullptr, int act = NFN_ACT_NONE);
   // the rows of one pass: short entries first, then the long ones
-  struct Batch { int rows = 0, short_rows = 0, n_mix = 0, n_seq = 0, n_short_seq = 0, longest = 0; bool single = false; std::vector<int> att_off, att_n; };
+  struct Batch { int rows = 0, short_rows = 0, n_mix = 0, n_seq = 0, n_short_seq = 0, longest = 0; bool single = false; std::vector<int> att_off, att_n;
+                 // latent layers: the long entries whose latents one expansion holds, by layer
+                 struct Round { int span0, n_spans, max_pages, rows, tile0, n_tiles; };
+                 std::vector<std::vector<Round>> expand; };
   int mix_rows(const Layer& L, const Batch& b, void* ff_out);
   int attention(const Layer& L, const Batch& b);
   int delta(const Layer& L, const Batch& b);
+  int rotated_attention(const Layer& L, const Batch& b);
+  int latent_attention(const Layer& L, const Batch& b);
+  int wkv(const Layer& L, const Batch& b);
+  int mixer(const Layer& L, const Batch& b);
+  int dense_ff(const Layer& L, int rows);
+  bool rotated(const Layer& L) const { return L.d.mixer == NFN_MIXER_ATTENTION && (L.d.rot_dims > 0 || L.d.qk_norm || L.d.key_values); }
+  void attention_args(const Layer& L, nfn_paged_attention_args* a);
+  int post_pass(const Batch& b);
+  // wkv: single tokens in one launch after the products, few rows through one launch for the four projections
+  bool wkv_step(const Layer& L, const Batch& b) const { return b.single && nfn_wkv_step_fits(b.rows, L.d.heads, L.dp); }
   bool grouped(const Layer& L, int rows) const { return c.dtype == 0 && L.d.experts <= 256 && L.d.top <= 32 && (long long)rows * L.d.top > 8LL * L.d.experts; }
   // single tokens of delta layers: convolution, rule, norm and gate in one launch
   bool one_step(const Layer& L, const Batch& b) const { return b.single && L.d.mixer == NFN_MIXER_DELTA && nfn_delta_step_fits(b.rows, L.d.heads, L.dp, L.vp); }
@@ -167,9 +215,13 @@ int layered_engine::build() {
       a.weights_of = o.weights_of = -1;
       if (std::memcmp(&a, &o, sizeof a)) return efail(bad + " and the layer whose tensors it uses differ");
     }
-    if (c.chained ? (d.ff > 0 || d.out_gate || d.kv_from >= 0) : (d.mixer != NFN_MIXER_ATTENTION || d.experts > 0 || d.qkv_bias))
-      return efail(bad + (c.chained ? ": sublayers one after another have routed experts, no output gate and caches of their own"
-                                    : ": delta mixers, experts and biases need sublayers one after another"));
+    if (c.chained ? (d.out_gate || (d.ff > 0 && d.experts > 0)) : (d.mixer != NFN_MIXER_ATTENTION || d.experts > 0 || d.qkv_bias || d.rot_dims > 0 || d.qk_norm || d.key_values))
+      return efail(bad + (c.chained ? ": sublayers one after another have one feed-forward and no output gate"
+                                    : ": recurrent and latent mixers, rotation, experts and biases need sublayers one after another"));
+    if (d.mixer == NFN_MIXER_WKV && !c.post_norm) return efail(bad + ": the token shift reads the residual itself (post_norm)");
+    if ((rotated(L) || d.mixer == NFN_MIXER_LATENT) && (d.conv_taps > 0 || d.q_temp_every > 0 || d.qkv_bias))
+      return efail(bad + ": rotated and latent attention have no convolutions, query temperature or biases");
+    if (!d.expert_plain && (d.shared_ff > 0 || d.route_correction || d.route_groups > 0 || d.route_normalise)) return efail(bad + ": gated experts have plain sigmoid routing and no shared expert");
     L.ep = d.experts > 0 ? up(d.experts, 16) : 0;
     L.ef = d.experts > 0 ? up(d.expert_ff, 16) : 0;
     L.dp = up(d.dim, 16);
@@ -179,8 +231,9 @@ int layered_engine::build() {
     if (d.kv_from >= 0) {
       const Layer& o = layers[d.kv_from];
       if (d.kv_from >= l || o.d.kv_from >= 0) return efail("engine: layer " + std::to_string(l) + " must read an earlier layer with keys and values of its own");
-      if (o.d.kv_heads != d.kv_heads || o.d.dim != d.dim || o.d.vdim != d.vdim)
-        return efail("engine: layer " + std::to_string(l) + " and the layer whose cache it reads have different key / value heads");
+      if (o.d.mixer != d.mixer || (d.mixer == NFN_MIXER_LATENT ? (o.d.kv_rank != d.kv_rank || o.d.rot_dim != d.rot_dim || o.d.rot_dims != d.rot_dims || o.d.rot_base != d.rot_base)
+                                                               : (o.d.kv_heads != d.kv_heads || o.d.dim != d.dim || o.d.vdim != d.vdim)))
+        return efail("engine: layer " + std::to_string(l) + " and the layer whose cache it reads have different caches");
       L.owner = d.kv_from;
     }
     const bool own = L.owner == l;
@@ -192,23 +245,61 @@ int layered_engine::build() {
       L.off_a1 = L.off_b + up(d.heads, 16);
       L.off_g1 = L.off_a1 + L.ra;
       L.off_gate = L.off_up = L.n_in = L.off_g1 + L.rg;
+    } else if (d.mixer == NFN_MIXER_LATENT) {
+      L.lr = up(d.kv_rank, 16);
+      L.rp = up(d.rot_dim, 16);
+      L.nq = d.heads * (L.dp + L.rp);
+      L.off_kv = L.nq;
+      L.n_in = L.nq + (own ? L.lr + L.rp : 0);
+    } else if (d.mixer == NFN_MIXER_WKV) {
+      L.ra = up(d.rank_decay, 16);
+      L.nq = d.heads * L.dp;                       // each of r, k, v, g
+      L.n_in = 4 * L.nq;
     } else {
       L.nq = d.heads * L.dp;
       L.nk = own ? d.kv_heads * L.dp : 0;
-      L.nv = own ? d.kv_heads * L.vp : 0;
+      L.nv = own && !d.key_values ? d.kv_heads * L.vp : 0;
       L.off_g = L.nq + L.nk + L.nv;
       L.off_gate = L.off_g + (d.out_gate ? d.heads * L.vp : 0);
-      L.off_up = L.off_gate + L.ff;
-      L.n_in = L.off_up + L.ff;
+      L.off_up = L.off_gate + (c.chained ? 0 : L.ff);
+      L.n_in = L.off_up + (c.chained ? 0 : L.ff);
     }
+    L.shp = d.shared_ff > 0 ? up(d.shared_ff, 16) : 0;
     L.n_conv = L.nq + L.nk + L.nv;
-    L.n_cat = d.heads * L.vp + L.ff;
-    n_in_max = std::max(n_in_max, L.n_in);
-    nq_max = std::max(nq_max, L.nq);
-    cat_max = std::max(cat_max, L.n_cat);
+    L.n_cat = d.heads * L.vp + (c.chained ? 0 : L.ff);
+    n_in_max = std::max(n_in_max, std::max(L.n_in, c.chained ? 2 * L.ff : 0));
+    if (!rotated(L) && (d.mixer == NFN_MIXER_ATTENTION || d.mixer == NFN_MIXER_DELTA)) nq_max = std::max(nq_max, L.nq);      // others keep their queries in place
+    cat_max = std::max(cat_max, std::max(L.n_cat, L.ff));
     if (d.weights_of < 0) {
       want(lname(l, "norm1"), wp);
       want(lname(l, "w_in"), (long long)L.n_in * wp);
+      if (d.qk_norm) {
+        want(lname(l, "q_norm"), L.dp);
+        if (own) want(lname(l, "k_norm"), L.dp);
+      }
+      if (d.mixer == NFN_MIXER_LATENT) {
+        if (own) want(lname(l, "c_norm"), L.lr);
+        want(lname(l, "w_ukv"), (long long)d.heads * (L.dp + L.vp) * L.lr);
+        want(lname(l, "w_uk_t"), (long long)d.heads * L.lr * L.dp);
+      }
+      if (d.mixer == NFN_MIXER_WKV) {
+        want(lname(l, "mu"), 5LL * wp);
+        want(lname(l, "w1"), (long long)L.ra * wp);
+        want(lname(l, "w2"), 2LL * L.nq * L.ra);
+        want(lname(l, "w0"), L.nq);
+        want(lname(l, "u"), L.nq);
+        want(lname(l, "out_norm"), L.nq);
+      }
+      if (c.chained && d.ff > 0) {
+        want(lname(l, "norm2"), wp);
+        want(lname(l, "w_gate_up"), 2LL * L.ff * wp);
+        want(lname(l, "w_down"), (long long)wp * L.ff);
+      }
+      if (d.shared_ff > 0) {
+        want(lname(l, "w_shared_up"), (long long)L.shp * wp);
+        want(lname(l, "w_shared_down"), (long long)wp * L.shp);
+      }
+      if (d.route_correction) want(lname(l, "correction"), L.ep);
       if (d.conv_taps > 0) want(lname(l, "conv"), (long long)d.conv_taps * L.n_conv);
       want(lname(l, "w_out"), (long long)wp * L.n_cat);
       if (sp) {
@@ -227,44 +318,48 @@ int layered_engine::build() {
       if (d.experts > 0) {
         want(lname(l, "norm2"), wp);
         want(lname(l, "router"), (long long)L.ep * wp);
-        want(lname(l, "w_gate_up"), (long long)d.experts * 2 * L.ef * wp);
+        want(lname(l, "w_gate_up"), (long long)d.experts * (d.expert_plain ? 1 : 2) * L.ef * wp);
         want(lname(l, "w_down"), (long long)d.experts * wp * L.ef);
       }
-      for (int q = 0; q < (c.streams > 0 ? (d.experts > 0 ? 2 : 1) : 0); ++q) {
+      for (int q = 0; q < (c.streams > 0 ? (d.experts > 0 || d.ff > 0 ? 2 : 1) : 0); ++q) {
         const std::string hc = q ? "hc2_" : "hc1_";
         want(lname(l, (hc + "in").c_str()), c.streams);
         want(lname(l, (hc + "out").c_str()), c.streams);
         want(lname(l, (hc + "mix").c_str()), (long long)c.streams * c.streams);
       }
     }
-    if (d.mixer == NFN_MIXER_DELTA) continue;
-    L.tile_rows = nfn_paged_tile_rows(c.dtype, d.heads, d.kv_heads, L.dp, L.vp);
+    if (!L.paged()) continue;
+    L.tile_rows = L.latent() ? nfn_latent_tile_rows(c.dtype, L.dp, L.rp, L.vp) : nfn_paged_tile_rows(c.dtype, d.heads, d.kv_heads, L.dp, L.vp);
     if (L.tile_rows > 0 && std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) == tile_kinds.end()) tile_kinds.push_back(L.tile_rows);
   }
   want("final_norm", wp);
   // how far back the readers of each owner look, and one group per distinct answer
   for (int l = 0; l < c.n_layer; ++l) {
-    if (layers[l].owner != l || layers[l].d.mixer == NFN_MIXER_DELTA) continue;
-    int w = 0, keep = 0;
-    bool all = false;
+    if (layers[l].owner != l || !layers[l].paged()) continue;
+    Group n;
     for (const Layer& r : layers)
       if (r.owner == l) {
-        all |= r.d.window <= 0;
-        w = std::max(w, r.d.window);
-        keep = std::max(keep, (r.d.keep_first + kPage - 1) / kPage);
+        n.all |= r.look() <= 0;
+        if (r.d.chunk > 0) n.chunks.push_back(r.d.chunk);
+        else n.window = std::max(n.window, r.d.window);
+        n.keep = std::max(n.keep, (r.d.keep_first + kPage - 1) / kPage);
       }
-    if (all) w = keep = 0;
-    int g = 0;
-    while (g < (int)groups.size() && (groups[g].window != w || groups[g].keep != keep)) ++g;
-    if (g == (int)groups.size()) {
-      groups.emplace_back();
-      groups.back().window = w;
-      groups.back().keep = keep;
+    std::sort(n.chunks.begin(), n.chunks.end());
+    n.chunks.erase(std::unique(n.chunks.begin(), n.chunks.end()), n.chunks.end());
+    if (n.all) {
+      n.window = n.keep = 0;
+      n.chunks.clear();
     }
+    int g = 0;
+    while (g < (int)groups.size() && !groups[g].like(n)) ++g;
+    if (g == (int)groups.size()) groups.push_back(n);
     for (Layer& r : layers)
       if (r.owner == l) r.group = g;
   }
-  if (groups.empty()) groups.emplace_back();   // no layer has pages: the pool still counts tokens
+  if (groups.empty()) {   // no layer has pages: the pool still counts tokens
+    groups.emplace_back();
+    groups.back().all = true;
+  }
   len.assign(c.max_batch, 0);
   parity.assign(c.max_batch, 0);
   logit_at.assign(c.max_batch, -1);
@@ -279,7 +374,8 @@ extern "C" nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, 
   const nfn_layered_config& c = *cfg;
   if (c.n_layer <= 0 || c.width <= 0 || c.vocab <= 0 || c.side_dim < 0 || (c.dtype != 0 && c.dtype != 1) || c.max_seq <= 0 || c.max_batch <= 0 ||
       c.kv_tokens < 0 || c.max_step_rows <= 0 || !(c.norm_eps >= 0.f) || c.streams < 0 || c.streams > NFN_MAX_STREAMS || (c.streams > 0 && !c.chained) ||
-      (c.chained && c.side_dim > 0) || !(c.logit_softcap >= 0.f) || (!c.chained && c.norm_offset != 0.f)) {
+      (c.chained && c.side_dim > 0) || !(c.logit_softcap >= 0.f) || (!c.chained && c.norm_offset != 0.f) ||
+      (c.post_norm && (!c.chained || c.streams > 0 || c.norm_offset != 0.f))) {
     efail("engine_create: invalid geometry");
     return nullptr;
   }
@@ -291,8 +387,12 @@ extern "C" nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, 
     const nfn_layer_desc& d = layers[l];
     if (d.heads <= 0 || d.kv_heads <= 0 || d.heads % d.kv_heads || d.dim <= 0 || d.vdim <= 0 || d.conv_taps < 0 || d.ff < 0 || d.window < 0 ||
         d.q_temp_every < 0 || d.keep_first < 0 || d.softcap < 0.f || d.experts < 0 || (d.experts > 0 && (d.top < 1 || d.top > d.experts || d.expert_ff < 1)) ||
-        (d.mixer != NFN_MIXER_ATTENTION && d.mixer != NFN_MIXER_DELTA) ||
-        (d.mixer == NFN_MIXER_DELTA && (d.conv_taps < 1 || d.rank_decay < 1 || d.rank_gate < 1 || d.dim > 512)) || (d.ff_act != NFN_ACT_RELU && d.ff_act != NFN_ACT_SILU && d.ff_act != NFN_ACT_GELU_TANH)) {
+        d.mixer < NFN_MIXER_ATTENTION || d.mixer > NFN_MIXER_WKV || d.chunk < 0 || (d.chunk > 0 && (d.window > 0 || d.keep_first > 0)) || d.rot_dims < 0 ||
+        (d.rot_dims & 1) || (d.rot_dims > 0 && !(d.rot_base > 0.0)) || (d.mixer == NFN_MIXER_ATTENTION && (d.rot_dims > d.dim || (d.key_values && d.vdim != d.dim) || ((d.rot_dims > 0 || d.qk_norm) && d.dim > 512))) ||
+        (d.mixer == NFN_MIXER_LATENT && (d.kv_rank <= 0 || d.rot_dim <= 0 || d.rot_dims != d.rot_dim || d.rot_dim > 512 || d.kv_heads != 1 || d.keep_first > 0 || d.qk_norm || d.sink || d.softcap > 0.f || d.alibi != 0.f)) ||
+        (d.mixer == NFN_MIXER_WKV && (d.rank_decay < 1 || d.dim > 512 || d.vdim != d.dim || d.kv_heads != d.heads)) || d.shared_ff < 0 || (d.shared_ff > 0 && d.experts <= 0) ||
+        (d.route_groups > 0 && (d.experts % d.route_groups || d.route_keep < 1 || d.route_keep > d.route_groups || d.route_keep * (d.experts / d.route_groups) < d.top)) || d.route_groups < 0 ||
+        (d.mixer == NFN_MIXER_DELTA && (d.conv_taps < 1 || d.rank_decay < 1 || d.rank_gate < 1 || d.dim > 512)) || (d.ff_act != NFN_ACT_RELU && d.ff_act != NFN_ACT_SILU && d.ff_act != NFN_ACT_GELU_TANH && d.ff_act != NFN_ACT_RELU2)) {
       efail("engine_create: invalid sizes in layer " + std::to_string(l));
       return nullptr;
     }
@@ -318,13 +418,16 @@ int layered_engine::finalize() {
     CU(cudaMemset(*p, 0, (size_t)n));
     return 0;
   };
-  if (zero((void**)&x, R * wp * 4 * std::max(c.streams, 1)) || zero(&h, R * wp * es) || zero(&in, R * n_in_max * es) || zero(&q, R * nq_max * es) || zero(&cat, R * cat_max * es) ||
+  if (zero((void**)&x, R * wp * 4 * std::max(c.streams, 1)) || zero(&h, R * wp * es) || zero(&in, R * n_in_max * es) || (nq_max > 0 && zero(&q, R * nq_max * es)) || zero(&cat, R * cat_max * es) ||
       zero(&hw, (long long)logit_rows * wp * es) || zero((void**)&logits, (long long)logit_rows * vp * 4) || zero((void**)&saved, S * vp * 4))
     return -1;
   if (c.dtype == 0 && zero(&xb, R * wp * 2)) return -1;
   if (sp && (zero((void**)&s_gate, R * sp * 4) || zero(&s_act, R * sp * es))) return -1;
   if ((sp || c.chained) && zero(&y, R * wp * es)) return -1;
   // scratch of the delta mixers and of the experts: the largest any layer asks for
+  long long n_q_lat = 0, n_o_lat = 0, n_lat = 0, n_lat_x = 0, n_low = 0, n_shift = 0, n_shared = 0;
+  // rows that attend to latents themselves: short entries, or all of them where the sizes have no tiles
+  const long long r_short = std::min<long long>(R, S * (kTileMin - 1));
   long long n_dec = 0, n_do = 0, e_log = 0, e_max = 0, e_items = 0, e_sorted = 0, e_gu = 0, e_mid = 0, e_rows = 0;
   for (const Layer& L : layers) {
     const nfn_layer_desc& d = L.d;
@@ -333,6 +436,25 @@ int layered_engine::finalize() {
       n_do = std::max(n_do, R * d.heads * L.vp);
       if (c.dtype == 0) delta_ws_bytes = std::max(delta_ws_bytes, nfn_delta_chunk_workspace_bytes(d.heads, L.dp, L.vp, c.max_batch));
     }
+    if (L.latent()) {
+      const long long rows = L.tile_rows > 0 ? std::max<long long>(r_short, c.max_batch) : R;
+      n_q_lat = std::max(n_q_lat, rows * d.heads * (L.lr + L.rp));
+      n_o_lat = std::max(n_o_lat, rows * d.heads * L.lr);
+      if (L.tile_rows > 0) {   // at least the longest portion with its window; several portions per round where they fit
+        const long long look = L.look() > 0 ? std::min(L.look(), c.max_seq) : c.max_seq;
+        lat_cap = std::max(lat_cap, up((int)std::min<long long>(look + R, up(c.max_seq, kPage)) + 2 * kPage, kPage));
+        n_lat = std::max<long long>(n_lat, L.lr);
+        n_lat_x = std::max<long long>(n_lat_x, (long long)d.heads * (L.dp + L.vp));
+      }
+    }
+    if (d.mixer == NFN_MIXER_WKV) {
+      n_dec = std::max(n_dec, R * L.nq);
+      n_do = std::max(n_do, R * L.nq);
+      n_low = std::max(n_low, R * L.ra);
+      n_shift = 5 * R * wp;
+      if (c.dtype == 0) wkv_ws_bytes = std::max(wkv_ws_bytes, nfn_wkv_chunk_workspace_bytes(d.heads, L.dp, c.max_batch));
+    }
+    n_shared = std::max(n_shared, R * L.shp);
     if (d.experts > 0) {
       const bool g = grouped(L, (int)R);
       const long long sorted = g ? (R * d.top + d.experts * 127LL + 127) / 128 * 128 : 0;
@@ -346,6 +468,11 @@ int layered_engine::finalize() {
       e_rows = std::max(e_rows, std::max(sorted, single));
     }
   }
+  lat_cap = std::max(lat_cap, n_lat > 0 ? rows_max : 0);
+  if ((n_q_lat && (zero(&q_lat, n_q_lat * es) || zero(&o_lat, n_o_lat * es))) || (n_lat && (zero(&lat_rows, lat_cap * n_lat * es) || zero(&lat_x, lat_cap * n_lat_x * es)))) return -1;
+  if (n_low && (zero((void**)&low, n_low * 4) || zero(&low_act, 2 * n_low * es) || zero(&shift, n_shift * es))) return -1;
+  if (n_shared && (zero(&shared_mid, n_shared * es) || zero(&y_shared, R * wp * es))) return -1;
+  if (wkv_ws_bytes > 0 && add(&wkv_ws, wkv_ws_bytes)) return -1;
   if (delta_ws_bytes > 0 && add(&delta_ws, delta_ws_bytes)) return -1;
   if (n_dec && (zero((void**)&decay, n_dec * 4) || zero((void**)&d_o, n_do * 4) || zero(&d_gate, n_do * es))) return -1;
   if (e_max && (zero((void**)&ex.logits, e_log * 4) || zero((void**)&ex.weight, e_items * 4) || zero((void**)&ex.idx, e_items * 4) ||
@@ -358,7 +485,7 @@ int layered_engine::finalize() {
     return -1;
   for (Group& g : groups) {
     g.pages = (c.kv_tokens + kPage - 1) / kPage;
-    if (g.window > 0) g.pages = (int)std::min<long long>(g.pages, S * ((g.window + R) / kPage + 2 + g.keep));
+    if (g.look() > 0) g.pages = (int)std::min<long long>(g.pages, S * ((g.look() + R) / kPage + 2 + g.keep));
     for (int p = g.pages - 1; p >= 0; --p) g.free_pages.push_back(p);
     g.first.assign(S, 0);
     g.next.assign(S, 0);
@@ -372,9 +499,11 @@ int layered_engine::finalize() {
     const nfn_layer_desc& d = L.d;
     if (d.mixer == NFN_MIXER_DELTA) {
       if (zero((void**)&L.memory, S * d.heads * L.dp * L.vp * 4)) return -1;
+    } else if (d.mixer == NFN_MIXER_WKV) {
+      if (zero((void**)&L.memory, S * d.heads * L.dp * L.dp * 4) || zero((void**)&L.prev, 2 * S * wp * 4)) return -1;
     } else if (L.owner == l) {
-      const long long tiles = (long long)groups[L.group].pages * d.kv_heads * kPage;
-      if (zero(&L.k_pool, tiles * L.dp * es) || zero(&L.v_pool, tiles * L.vp * es)) return -1;
+      const long long tokens = (long long)groups[L.group].pages * kPage;
+      if (zero(&L.k_pool, tokens * L.key_row() * es) || (L.value_row() > 0 && zero(&L.v_pool, tokens * L.value_row() * es))) return -1;
     } else {
       L.k_pool = layers[L.owner].k_pool;
       L.v_pool = layers[L.owner].v_pool;
@@ -391,6 +520,44 @@ int layered_engine::finalize() {
       if (zero((void**)&L.slopes, 4LL * d.heads)) return -1;
       CU(cudaMemcpy(L.slopes, sl.data(), sl.size() * 4, cudaMemcpyHostToDevice));
     }
+    if (d.rot_dims > 0) {
+      std::vector<float> f(d.rot_dims);
+      for (int i = 0; i < d.rot_dims / 2; ++i) {
+        const double v = std::pow(d.rot_base, -2.0 * i / d.rot_dims);
+        f[2 * i] = (float)v;
+        f[2 * i + 1] = (float)(v - (double)f[2 * i]);
+      }
+      if (zero((void**)&L.freq, 4LL * d.rot_dims)) return -1;
+      CU(cudaMemcpy(L.freq, f.data(), f.size() * 4, cudaMemcpyHostToDevice));
+    }
+    if (d.qk_norm) {
+      L.q_norm = W(lname(wl, "q_norm"));
+      if (L.owner == l) L.k_norm = W(lname(wl, "k_norm"));
+    }
+    if (L.latent()) {
+      if (L.owner == l) L.c_norm = W(lname(wl, "c_norm"));
+      L.w_ukv = W(lname(wl, "w_ukv"));
+      L.w_uk_t = W(lname(wl, "w_uk_t"));
+      L.w_uv = static_cast<const char*>(L.w_ukv) + 2LL * d.heads * L.dp * L.lr;
+    }
+    if (d.mixer == NFN_MIXER_WKV) {
+      L.mu = W(lname(wl, "mu"));
+      L.w1 = W(lname(wl, "w1"));
+      L.w2 = W(lname(wl, "w2"));
+      L.w0 = W(lname(wl, "w0"));
+      L.u = W(lname(wl, "u"));
+      L.out_norm = W(lname(wl, "out_norm"));
+    }
+    if (c.chained && d.ff > 0) {
+      L.norm2 = W(lname(wl, "norm2"));
+      L.w_gate_up = W(lname(wl, "w_gate_up"));
+      L.w_down = W(lname(wl, "w_down"));
+    }
+    if (d.shared_ff > 0) {
+      L.w_shared_up = W(lname(wl, "w_shared_up"));
+      L.w_shared_down = W(lname(wl, "w_shared_down"));
+    }
+    if (d.route_correction) L.correction = W(lname(wl, "correction"));
     L.norm1 = W(lname(wl, "norm1"));
     L.w_in = W(lname(wl, "w_in"));
     L.w_out = W(lname(wl, "w_out"));
@@ -408,7 +575,7 @@ int layered_engine::finalize() {
       L.w_gate_up = W(lname(wl, "w_gate_up"));
       L.w_down = W(lname(wl, "w_down"));
     }
-    for (int q = 0; q < (c.streams > 0 ? (d.experts > 0 ? 2 : 1) : 0); ++q) {
+    for (int q = 0; q < (c.streams > 0 ? (d.experts > 0 || d.ff > 0 ? 2 : 1) : 0); ++q) {
       const std::string hc = q ? "hc2_" : "hc1_";
       L.hc[q].in = W(lname(wl, (hc + "in").c_str()));
       L.hc[q].out = W(lname(wl, (hc + "out").c_str()));
@@ -435,7 +602,9 @@ int layered_engine::finalize() {
   io.mix = io.offset + 256;
   io.att = io.mix + up256(R * (long long)sizeof(nfn_row_tile));
   io.seq = io.att + up256(kinds * R * 16);
-  io.out = io.seq + up256(S * (long long)sizeof(nfn_seq_rows));
+  io.spans = io.seq + up256(S * (long long)sizeof(nfn_seq_rows));
+  io.base = io.spans + up256(c.n_layer * S * (long long)sizeof(nfn_latent_span));
+  io.out = io.base + up256(c.n_layer * S * 4);
   io.total = io.out + up256((long long)logit_rows * 4);
   CU(cudaMallocHost((void**)&h_io, (size_t)io.total));
   std::memset(h_io, 0, (size_t)io.total);
@@ -476,11 +645,11 @@ int layered_engine::reserve(int slot, int upto) {
   return 0;
 }
 
-// The next query of the slot sits at len[slot] and sees keys from len - window + 1 on.
+// The next query of the slot sits at len[slot].
 void layered_engine::trim(int slot) {
   for (Group& g : groups) {
-    if (g.window <= 0) continue;
-    const int live = std::max(0, len[slot] - g.window + 1) / kPage;
+    if (g.look() <= 0) continue;
+    const int live = g.oldest(len[slot]) / kPage;
     for (; g.first[slot] < std::min(live, g.next[slot]); ++g.first[slot])
       if (g.first[slot] >= g.keep) g.free_pages.push_back(g.h_table[(size_t)slot * max_pages + g.first[slot]]);
   }
@@ -521,10 +690,10 @@ int layered_engine::fork(int src, int dst, int n) {
       g.free_pages.pop_back();
       for (int l = 0; l < c.n_layer; ++l) {
         const Layer& L = layers[l];
-        if (L.owner != l || L.group != (int)gi || L.d.mixer == NFN_MIXER_DELTA) continue;
-        const size_t kb = (size_t)L.d.kv_heads * kPage * L.dp * es, vb = (size_t)L.d.kv_heads * kPage * L.vp * es;
+        if (L.owner != l || L.group != (int)gi || !L.paged()) continue;
+        const size_t kb = (size_t)kPage * L.key_row() * es, vb = (size_t)kPage * L.value_row() * es;
         CU(cudaMemcpyAsync(static_cast<char*>(L.k_pool) + to[p] * kb, static_cast<char*>(L.k_pool) + from[p] * kb, kb, cudaMemcpyDeviceToDevice, stream));
-        CU(cudaMemcpyAsync(static_cast<char*>(L.v_pool) + to[p] * vb, static_cast<char*>(L.v_pool) + from[p] * vb, vb, cudaMemcpyDeviceToDevice, stream));
+        if (vb) CU(cudaMemcpyAsync(static_cast<char*>(L.v_pool) + to[p] * vb, static_cast<char*>(L.v_pool) + from[p] * vb, vb, cudaMemcpyDeviceToDevice, stream));
       }
     }
     CU(cudaMemcpyAsync(g.d_table + (size_t)dst * max_pages, to, (size_t)max_pages * 4, cudaMemcpyHostToDevice, stream));
@@ -534,6 +703,10 @@ int layered_engine::fork(int src, int dst, int n) {
     if (L.memory) {
       const size_t n = (size_t)L.d.heads * L.dp * L.vp;
       CU(cudaMemcpyAsync(L.memory + dst * n, L.memory + src * n, n * 4, cudaMemcpyDeviceToDevice, stream));
+    }
+    if (L.prev) {
+      float* half = L.prev + (size_t)parity[src] * c.max_batch * wp;
+      CU(cudaMemcpyAsync(half + (size_t)dst * wp, half + (size_t)src * wp, (size_t)wp * 4, cudaMemcpyDeviceToDevice, stream));
     }
     if (!L.state) continue;
     const size_t row = (size_t)(L.d.conv_taps - 1) * L.n_conv * es;
@@ -548,9 +721,10 @@ int layered_engine::fork(int src, int dst, int n) {
 // ---- one pass over the rows of a step -----------------------------------------------------------------
 
 // out = a . w^T: kOutAct in the activation type, kOutF32 in fp32, kOutResidual added to the residual stream x
-int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n, int k, void* out, int ldo, int kind, const void* bias) {
+int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n, int k, void* out, int ldo, int kind, const void* bias, int act) {
   if (c.dtype == 1) {
     K(nfn_gemm_f32(static_cast<const float*>(a), lda, wt, k, static_cast<float*>(out), ldo, rows, n, k, kind == kOutResidual, bias, stream));
+    if (act != NFN_ACT_NONE) K(nfn_ff_rows(1, out, ldo, 0, -1, n, act, out, ldo, rows, stream));
     return 0;
   }
   nfn_gemm_args g{};
@@ -558,7 +732,7 @@ int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n,
   g.m = rows; g.n = n; g.k = k;
   g.lda = lda; g.ldb = k; g.ldc = ldo;
   g.alpha = 1.f;
-  g.flags = kind == kOutAct ? 0 : NFN_EPI_OUT_F32;
+  g.flags = (kind == kOutAct ? 0 : NFN_EPI_OUT_F32) | (act << NFN_EPI_ACT_SHIFT);
   if (kind == kOutResidual) {
     g.flags |= NFN_EPI_ACCUM | NFN_EPI_COPY_BF16;
     g.aux_out = xb;
@@ -579,7 +753,7 @@ int layered_engine::mix_rows(const Layer& L, const Batch& b, void* ff_out) {
   const nfn_layer_desc& d = L.d;
   nfn_mix_args m{};
   m.f32 = c.dtype == 1; m.in = in; m.ld_in = L.n_in;
-  m.nq = L.nq; m.nk = L.nk; m.nv = L.nv; m.off_gate = L.off_gate; m.off_up = L.off_up; m.ff = L.ff; m.act = d.ff_act;
+  m.nq = L.nq; m.nk = L.nk; m.nv = L.nv; m.off_gate = L.off_gate; m.off_up = L.off_up; m.ff = c.chained ? 0 : L.ff; m.act = d.ff_act;
   m.conv = L.conv; m.taps = d.conv_taps; m.state = L.state; m.state_half = L.state_half;
   m.conv_act = d.mixer == NFN_MIXER_DELTA ? NFN_ACT_SILU : NFN_ACT_NONE;
   m.q_out = q; m.ld_q = L.nq;
@@ -592,20 +766,30 @@ int layered_engine::mix_rows(const Layer& L, const Batch& b, void* ff_out) {
   return 0;
 }
 
+// What the attention calls of a layer have in common.
+void layered_engine::attention_args(const Layer& L, nfn_paged_attention_args* out) {
+  const nfn_layer_desc& d = L.d;
+  nfn_paged_attention_args& a = *out;
+  a.f32 = c.dtype == 1; a.total_rows = rows_max;
+  a.k_pool = L.k_pool; a.v_pool = L.v_pool; a.pages = groups[L.group].pages;
+  a.table = groups[L.group].d_table; a.table_ld = max_pages;
+  a.heads = d.heads; a.window = d.window; a.chunk = d.chunk; a.scale = d.scale; a.slopes = L.slopes;
+  a.keep_first = d.window > 0 ? d.keep_first : 0; a.softcap = d.softcap; a.sink = d.sink;
+  a.row_slot = dev<int>(io.slot); a.row_pos = dev<int>(io.pos);
+  a.max_keys = L.look() > 0 ? std::min(L.look() + d.keep_first, c.max_seq) : c.max_seq;
+  a.workspace = att_ws; a.workspace_bytes = att_ws_bytes;
+}
+
 // q rows over the layer's pages -> the first columns of `cat`
 int layered_engine::attention(const Layer& L, const Batch& b) {
   const nfn_layer_desc& d = L.d;
   nfn_paged_attention_args a{};
-  a.f32 = c.dtype == 1; a.q = q; a.ld_q = L.nq; a.total_rows = rows_max;
-  a.k_pool = L.k_pool; a.v_pool = L.v_pool; a.kv_heads = d.kv_heads; a.dim_p = L.dp; a.vdim_p = L.vp; a.pages = groups[L.group].pages;
-  a.table = groups[L.group].d_table; a.table_ld = max_pages;
-  a.heads = d.heads; a.window = d.window; a.scale = d.scale; a.slopes = L.slopes;
-  a.keep_first = d.window > 0 ? d.keep_first : 0; a.softcap = d.softcap; a.sink = d.sink;
+  attention_args(L, &a);
+  const bool in_place = rotated(L);
+  a.q = in_place ? in : q; a.ld_q = in_place ? L.n_in : L.nq;
+  a.kv_heads = d.kv_heads; a.dim_p = L.dp; a.vdim_p = L.vp;
   a.gate = d.out_gate ? static_cast<char*>(in) + (size_t)L.off_g * es : nullptr; a.ld_gate = L.n_in;
   a.out = cat; a.ld_o = L.n_cat;
-  a.row_slot = dev<int>(io.slot); a.row_pos = dev<int>(io.pos);
-  a.max_keys = d.window > 0 ? std::min(d.window + d.keep_first, c.max_seq) : c.max_seq;
-  a.workspace = att_ws; a.workspace_bytes = att_ws_bytes;
   const int single = L.tile_rows > 0 ? b.short_rows : b.rows;
   if (single > 0) {
     a.rows = single;
@@ -656,34 +840,178 @@ int layered_engine::delta(const Layer& L, const Batch& b) {
   return 0;
 }
 
+// Attention whose queries and keys are normed and rotated, in place inside the input product -> the first columns of `cat`
+int layered_engine::rotated_attention(const Layer& L, const Batch& b) {
+  const nfn_layer_desc& d = L.d;
+  nfn_head_rows_args r{};
+  r.f32 = c.dtype == 1; r.in = in; r.ld_in = L.n_in; r.off_k = L.nq; r.off_v = d.key_values ? L.nq : L.nq + L.nk;
+  r.heads = d.heads; r.kv_heads = L.nk > 0 ? d.kv_heads : 0; r.dim = d.dim; r.dim_p = L.dp; r.vdim_p = L.vp;
+  r.q_norm = L.q_norm; r.k_norm = L.k_norm; r.eps = c.norm_eps; r.freq = L.freq; r.rot_dims = d.rot_dims;
+  r.q_out = in; r.ld_q = L.n_in;
+  r.k_pool = L.k_pool; r.v_pool = L.v_pool; r.table = groups[L.group].d_table; r.table_ld = max_pages;
+  r.tiles = dev<nfn_row_tile>(io.mix); r.n_tiles = b.n_mix; r.tile_rows = b.n_mix == b.rows ? 1 : kMixRows;
+  K(nfn_head_rows(&r, stream));
+  return attention(L, b);
+}
+
+// Latent attention -> the first columns of `cat`. Short entries: queries and outputs pass through the key and value projections, attention runs on
+// the cached latents. Long ones: keys and values of the visible latents are formed first, as many entries at a time as the buffers hold.
+int layered_engine::latent_attention(const Layer& L, const Batch& b) {
+  const nfn_layer_desc& d = L.d;
+  const int f32 = c.dtype == 1, H = d.heads, lp = L.lr + L.rp, qp = L.dp + L.rp, single = L.tile_rows > 0 ? b.short_rows : b.rows;
+  nfn_latent_rows_args r{};
+  r.f32 = f32; r.in = in; r.ld_in = L.n_in; r.off_kv = L.off_kv;
+  r.heads = H; r.dim_p = L.dp; r.rot_dim = d.rot_dim; r.rot_p = L.rp; r.rank = d.kv_rank; r.rank_p = L.lr;
+  r.c_norm = L.c_norm; r.eps = c.norm_eps; r.freq = L.freq;
+  r.q_out = in; r.ld_q = L.n_in; r.q_row0 = single; r.q_lat = q_lat;
+  r.k_pool = L.c_norm ? L.k_pool : nullptr;              // readers of another layer's cache leave it alone
+  r.table = groups[L.group].d_table; r.table_ld = max_pages;
+  r.tiles = dev<nfn_row_tile>(io.mix); r.n_tiles = b.n_mix; r.tile_rows = b.n_mix == b.rows ? 1 : kMixRows;
+  K(nfn_latent_rows(&r, stream));
+  nfn_paged_attention_args a{};
+  attention_args(L, &a);
+  if (single > 0) {
+    nfn_group_products_args g{};
+    g.f32 = f32; g.rows = single; g.groups = H;
+    g.n = L.lr; g.k = L.dp; g.in = in; g.ld_in = L.n_in; g.in_group = qp; g.w = L.w_uk_t; g.out = q_lat; g.ld_out = (long long)H * lp; g.out_group = lp;
+    K(nfn_group_products(&g, stream));
+    a.q = q_lat; a.ld_q = H * lp; a.kv_heads = 1; a.dim_p = lp; a.vdim_p = L.lr; a.v_pool = nullptr;
+    a.out = o_lat; a.ld_o = H * L.lr; a.rows = single;
+    K(nfn_paged_attention_rows(&a, stream));
+    g.n = L.vp; g.k = L.lr; g.in = o_lat; g.ld_in = (long long)H * L.lr; g.in_group = L.lr; g.w = L.w_uv; g.out = cat; g.ld_out = L.n_cat; g.out_group = L.vp;
+    K(nfn_group_products(&g, stream));
+  }
+  const int l = (int)(&L - layers.data()), cols = H * (L.dp + L.vp);
+  a.q = in; a.ld_q = L.n_in; a.kv_heads = H; a.dim_p = qp; a.vdim_p = L.vp; a.out = cat; a.ld_o = L.n_cat;
+  const int k = (int)(std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) - tile_kinds.begin());
+  for (const Batch::Round& o : b.expand[l]) {
+    K(nfn_latent_gather(f32, L.k_pool, lp, L.lr, groups[L.group].d_table, max_pages, dev<nfn_latent_span>(io.spans) + (size_t)l * c.max_batch + o.span0, o.n_spans, o.max_pages,
+                        lat_rows, stream));
+    if (lin(lat_rows, L.lr, L.w_ukv, o.rows, cols, L.lr, lat_x, cols, kOutAct)) return -1;
+    nfn_latent_expanded x{};
+    x.x = lat_x; x.x_rows = o.rows; x.dim_u = L.dp; x.rot_p = L.rp; x.rank_p = L.lr; x.x_base = dev<int>(io.base) + (size_t)l * c.max_batch;
+    a.tiles = dev<int>(io.att) + (size_t)(b.att_off[k] + o.tile0) * 4;
+    a.n_tiles = o.n_tiles;
+    K(nfn_latent_attention_tiles(&a, &x, stream));
+  }
+  return 0;
+}
+
+// Time mixing with the bonus recurrence -> the first columns of `cat`
+int layered_engine::wkv(const Layer& L, const Batch& b) {
+  const nfn_layer_desc& d = L.d;
+  const int f32 = c.dtype == 1, rows = b.rows, nq = L.nq;
+  const long long stride = (long long)rows_max * wp;
+  nfn_shift_args s{};
+  s.f32 = f32; s.width = c.width; s.ld = wp; s.n = 5; s.src = x; s.mu = L.mu;
+  s.prev = L.prev; s.prev_half = (long long)c.max_batch * wp; s.out = shift; s.out_stride = stride;
+  s.tiles = dev<nfn_row_tile>(io.mix); s.n_tiles = b.n_mix;
+  K(nfn_shift_rows(&s, stream));
+  auto mixed = [&](int i) { return static_cast<const char*>(shift) + (size_t)i * stride * es; };
+  if (!f32 && rows <= 32) {                              // r, k, v, gate in one launch
+    nfn_group_products_args g{};
+    g.rows = rows; g.groups = 4; g.n = nq; g.k = wp; g.in = shift; g.ld_in = wp; g.in_group = stride; g.w = L.w_in;
+    g.out = in; g.ld_out = L.n_in; g.out_group = nq;
+    K(nfn_group_products(&g, stream));
+  } else {
+    for (int i = 0; i < 4; ++i)
+      if (lin(mixed(i), wp, static_cast<const char*>(L.w_in) + 2LL * i * nq * wp, rows, nq, wp, static_cast<char*>(in) + (size_t)i * nq * es, L.n_in, kOutAct)) return -1;
+  }
+  if (lin(mixed(4), wp, L.w1, rows, L.ra, wp, low, L.ra, kOutF32)) return -1;
+  if (wkv_step(L, b)) {
+    nfn_wkv_step_args t{};
+    t.f32 = f32; t.rows = rows; t.rkvg = in; t.ld_rkvg = L.n_in; t.low = low; t.ld_low = t.rank_p = L.ra; t.w2 = L.w2; t.ld_w2 = 2 * L.ra;
+    t.w0 = L.w0; t.u = L.u; t.heads = d.heads; t.dim = d.dim; t.dim_p = L.dp; t.state = L.memory; t.weight = L.out_norm; t.eps = c.norm_eps;
+    t.out = cat; t.ld_out = L.n_cat; t.tiles = dev<nfn_row_tile>(io.mix);
+    K(nfn_wkv_step(&t, stream));
+    return 0;
+  }
+  const int ld = f32 ? L.ra : 2 * L.ra;                  // w2 rows stand twice: for the rounded tanh and for what rounding left out
+  K(nfn_tanh_split(f32, low, L.ra, low_act, ld, rows, L.ra, stream));
+  if (f32) K(nfn_gemm_f32(static_cast<const float*>(low_act), ld, L.w2, 2 * L.ra, decay, nq, rows, nq, L.ra, 0, nullptr, stream));
+  else if (lin(low_act, ld, L.w2, rows, nq, ld, decay, nq, kOutF32)) return -1;
+  nfn_wkv_args a{};
+  a.f32 = f32; a.rkv = in; a.ld_rkv = L.n_in; a.z = decay; a.ld_z = nq; a.w0 = L.w0; a.u = L.u;
+  a.heads = d.heads; a.dim = d.dim; a.dim_p = L.dp; a.state = L.memory; a.o = d_o; a.ld_o = nq;
+  const bool chunks = !f32 && L.dp <= 256;
+  a.seqs = dev<nfn_seq_rows>(io.seq); a.n_seqs = chunks ? b.n_short_seq : b.n_seq;
+  if (a.n_seqs > 0) K(nfn_wkv_rows(&a, stream));
+  if (chunks && b.n_seq > b.n_short_seq) {
+    a.seqs += b.n_short_seq;
+    a.n_seqs = b.n_seq - b.n_short_seq;
+    K(nfn_wkv_chunks(&a, b.longest, wkv_ws, wkv_ws_bytes, stream));
+  }
+  K(nfn_head_out(f32, d_o, nq, static_cast<char*>(in) + 3LL * nq * es, L.n_in, NFN_ACT_SILU, L.out_norm, L.dp, c.norm_eps, cat, L.n_cat, rows, d.heads, d.dim, L.dp, stream));
+  return 0;
+}
+
+// A chained layer's mixer on the rows h -> y
+int layered_engine::mixer(const Layer& L, const Batch& b) {
+  const int kind = L.d.mixer;
+  if (kind != NFN_MIXER_WKV && lin(h, wp, L.w_in, b.rows, L.n_in, wp, in, L.n_in, kOutAct, L.bias_in)) return -1;
+  int rc;
+  if (kind == NFN_MIXER_WKV) rc = wkv(L, b);
+  else if (kind == NFN_MIXER_LATENT) rc = latent_attention(L, b);
+  else if (rotated(L)) rc = rotated_attention(L, b);
+  else {
+    if (!one_step(L, b) && mix_rows(L, b, nullptr)) return -1;
+    rc = kind == NFN_MIXER_DELTA ? delta(L, b) : attention(L, b);
+  }
+  return rc ? -1 : lin(cat, L.n_cat, L.w_out, b.rows, wp, L.n_cat, y, wp, kOutAct);
+}
+
+// A chained layer's gated feed-forward on the rows h -> y
+int layered_engine::dense_ff(const Layer& L, int rows) {
+  if (lin(h, wp, L.w_gate_up, rows, 2 * L.ff, wp, in, 2 * L.ff, kOutAct)) return -1;
+  K(nfn_ff_rows(c.dtype == 1, in, 2 * L.ff, 0, L.ff, L.ff, L.d.ff_act, cat, L.ff, rows, stream));
+  return lin(cat, L.ff, L.w_down, rows, wp, L.ff, y, wp, kOutAct);
+}
+
 // Routed experts on the normalised rows h; says in `sp` where the next stream pass finds each row's outputs.
 int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
   const nfn_layer_desc& d = L.d;
   if (lin(h, wp, L.router, rows, L.ep, wp, ex.logits, L.ep, kOutF32)) return -1;
   sp->y = ex.y;
   sp->y_rows = d.top;
+  sp->y_item = d.expert_plain ? ex.weight : nullptr;
+  if (d.shared_ff > 0) {
+    if (lin(h, wp, L.w_shared_up, rows, L.shp, wp, shared_mid, L.shp, kOutAct, nullptr, d.ff_act) ||
+        lin(shared_mid, L.shp, L.w_shared_down, rows, wp, L.shp, y_shared, wp, kOutAct))
+      return -1;
+    sp->y_plus = y_shared;
+  }
+  nfn_route_rule rule{};
+  rule.correction = L.correction; rule.groups = d.route_groups; rule.keep_groups = d.route_keep; rule.normalise = d.route_normalise; rule.scale = d.route_scale;
   if (!grouped(L, rows)) {
     nfn_moe_rows_args a{};
     a.f32 = c.dtype == 1; a.rows = rows; a.width = wp; a.ff = L.ef; a.experts = d.experts; a.top = d.top; a.act = d.ff_act;
     a.logits = ex.logits; a.ld_logits = L.ep; a.h = h; a.ld_h = wp; a.w_gate_up = L.w_gate_up; a.w_down = L.w_down;
     a.idx = ex.idx; a.weight = ex.weight; a.order = ex.order; a.offsets = ex.offsets; a.active = ex.active;
-    a.mid = ex.mid; a.y = ex.y; a.ld_y = wp;
+    a.mid = ex.mid; a.y = ex.y; a.ld_y = wp; a.plain = d.expert_plain; a.rule = rule;
     K(nfn_moe_rows(&a, stream));
     sp->y_index = nullptr;
     return 0;
   }
   const int cap = (int)(((long long)rows * d.top + d.experts * 127LL + 127) / 128 * 128);
   CU(cudaMemsetAsync(ex.counts, 0, (size_t)d.experts * 4, stream));
-  K(nfn_moe_route(ex.logits, L.ep, rows, d.experts, d.top, 1, 0, 1.f, ex.idx, ex.weight, ex.counts, stream));
+  if (d.expert_plain) K(nfn_moe_choose(ex.logits, L.ep, rows, d.experts, d.top, &rule, ex.idx, ex.weight, ex.counts, stream));
+  else K(nfn_moe_route(ex.logits, L.ep, rows, d.experts, d.top, 1, 0, 1.f, ex.idx, ex.weight, ex.counts, stream));
   K(nfn_moe_plan(ex.counts, d.experts, cap / 128, ex.offsets, ex.cursor, ex.tile_expert, ex.plan, stream));
   K(nfn_moe_permute_weighted(h, wp, rows, d.top, wp, ex.idx, ex.weight, ex.offsets, ex.cursor, cap, ex.xs, ex.row_of, ex.row_w, stream));
   nfn_gemm_tp_args g{};
   g.mode = NFN_TP_GROUPED;
   g.tile_group = ex.tile_expert; g.num_m_tiles_dev = ex.plan; g.groups = d.experts; g.m = cap;
-  g.a = ex.xs; g.b = L.w_gate_up; g.c = ex.gate_up;
-  g.n = 2 * L.ef; g.k = g.lda = g.ldb = wp; g.ldc = 2 * L.ef;
-  K(nfn_gemm_tp(&g, stream));
-  K(nfn_moe_act_rows(ex.gate_up, ex.row_w, ex.plan, cap, L.ef, d.ff_act, ex.mid, stream));
+  g.a = ex.xs; g.b = L.w_gate_up;
+  g.k = g.lda = g.ldb = wp;
+  if (d.expert_plain) {
+    g.c = ex.mid; g.n = g.ldc = L.ef; g.flags = d.ff_act << NFN_EPI_ACT_SHIFT;
+    K(nfn_gemm_tp(&g, stream));
+    g.flags = 0;
+  } else {
+    g.c = ex.gate_up; g.n = g.ldc = 2 * L.ef;
+    K(nfn_gemm_tp(&g, stream));
+    K(nfn_moe_act_rows(ex.gate_up, ex.row_w, ex.plan, cap, L.ef, d.ff_act, ex.mid, stream));
+  }
   g.a = ex.mid; g.b = L.w_down; g.c = ex.y;
   g.n = wp; g.k = g.lda = g.ldb = L.ef; g.ldc = wp;
   K(nfn_gemm_tp(&g, stream));
@@ -693,6 +1021,7 @@ int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
 
 // Layers whose mixer and feed-forward read one norm
 int layered_engine::pass(const Batch& b) {
+  if (c.post_norm) return post_pass(b);
   if (c.chained) return chained_pass(b);
   const int f32 = c.dtype == 1, rows = b.rows;
   nfn_row_norm_args rn{};
@@ -735,21 +1064,43 @@ int layered_engine::chained_pass(const Batch& b) {
   s.tokens = nullptr; s.embed = nullptr;
   for (int l = 0; l < c.n_layer; ++l) {
     const Layer& L = layers[l];
-    if (lin(h, wp, L.w_in, b.rows, L.n_in, wp, in, L.n_in, kOutAct, L.bias_in)) return -1;
-    if (!one_step(L, b) && mix_rows(L, b, nullptr)) return -1;
-    if (L.d.mixer == NFN_MIXER_DELTA ? delta(L, b) : attention(L, b)) return -1;
-    if (lin(cat, L.n_cat, L.w_out, b.rows, wp, L.n_cat, y, wp, kOutAct)) return -1;
-    s.y = y; s.y_rows = 1; s.y_index = nullptr; s.mix = L.hc[0].mix; s.out = L.hc[0].out;
-    if (L.d.experts > 0) {
+    if (mixer(L, b)) return -1;
+    s.y = y; s.y_rows = 1; s.y_index = nullptr; s.y_item = nullptr; s.y_plus = nullptr; s.mix = L.hc[0].mix; s.out = L.hc[0].out;
+    if (L.d.experts > 0 || L.d.ff > 0) {
       s.in = L.hc[1].in; s.weight = L.norm2;
       K(nfn_stream_pass(&s, stream));
-      if (experts(L, b.rows, &s)) return -1;
+      if (L.d.experts > 0 ? experts(L, b.rows, &s) : dense_ff(L, b.rows)) return -1;
       s.mix = L.hc[1].mix; s.out = L.hc[1].out;
     }
     if (l + 1 < c.n_layer) {
       s.in = layers[l + 1].hc[0].in; s.weight = layers[l + 1].norm1;
       K(nfn_stream_pass(&s, stream));
     }
+  }
+  pend = s;
+  return 0;
+}
+
+// Layers whose sublayers read the residual itself; the stream pass after each one norms its output, adds it and leaves the new rows in the activation
+// type. The last update is left to the head.
+int layered_engine::post_pass(const Batch& b) {
+  nfn_stream_args s{};
+  s.f32 = c.dtype == 1; s.rows = b.rows; s.width = c.width; s.ld = wp; s.streams = 1;
+  s.eps = c.norm_eps; s.y_scale = c.residual_mult;
+  s.tokens = dev<int>(io.tok); s.embed = W("embed"); s.embed_scale = c.embed_scale; s.vocab = c.vocab;
+  s.x = x; s.x_out = x; s.h = h;
+  K(nfn_stream_pass(&s, stream));
+  s.tokens = nullptr; s.embed = nullptr;
+  for (int l = 0; l < c.n_layer; ++l) {
+    const Layer& L = layers[l];
+    if (mixer(L, b)) return -1;
+    s.y = y; s.y_rows = 1; s.y_index = nullptr; s.y_item = nullptr; s.y_plus = nullptr; s.y_weight = L.norm1;
+    if (L.d.experts > 0 || L.d.ff > 0) {
+      K(nfn_stream_pass(&s, stream));
+      if (L.d.experts > 0 ? experts(L, b.rows, &s) : dense_ff(L, b.rows)) return -1;
+      s.y_weight = L.norm2;
+    }
+    if (l + 1 < c.n_layer) K(nfn_stream_pass(&s, stream));
   }
   pend = s;
   return 0;
@@ -802,7 +1153,7 @@ int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* 
   int *tok = host<int>(io.tok), *slot = host<int>(io.slot), *pos = host<int>(io.pos);
   nfn_row_tile* mix = host<nfn_row_tile>(io.mix);
   int n_mix = 0, hist_max = 0;
-  for (const Layer& L : layers) hist_max = std::max(hist_max, L.d.conv_taps - 1);
+  for (const Layer& L : layers) hist_max = std::max(hist_max, L.prev ? 1 : L.d.conv_taps - 1);
   row_of.clear();
   for (size_t i = 0; i < part.size(); ++i) {
     const int s = part[i].slot, p0 = len[s], n = part[i].count;
@@ -854,12 +1205,37 @@ int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* 
     }
     att_n[k] = n_att - att_off[k];
   }
+  // what the latent layers expand: the visible pages of every long entry, in rounds that fit
+  b.expand.resize(c.n_layer);
+  for (int l = 0; l < c.n_layer; ++l) {
+    const Layer& L = layers[l];
+    if (!L.latent() || L.tile_rows <= 0) continue;
+    nfn_latent_span* spans = host<nfn_latent_span>(io.spans) + (size_t)l * c.max_batch;
+    int* base = host<int>(io.base) + (size_t)l * c.max_batch;
+    int n_spans = 0, tile = 0;
+    for (size_t i = 0; i < part.size(); ++i) {
+      if (part[i].count < kTileMin) continue;
+      const int s = part[i].slot, p0 = len[s], oldest = L.d.chunk > 0 ? p0 / L.d.chunk * L.d.chunk : L.d.window > 0 ? std::max(0, p0 - L.d.window + 1) : 0;
+      const int page0 = oldest / kPage, pages = (p0 + part[i].count - 1) / kPage + 1 - page0, tiles = (part[i].count + L.tile_rows - 1) / L.tile_rows;
+      if (b.expand[l].empty() || b.expand[l].back().rows + pages * kPage > lat_cap) b.expand[l].push_back(Batch::Round{n_spans, 0, 0, 0, tile, 0});
+      Batch::Round& o = b.expand[l].back();
+      spans[n_spans++] = nfn_latent_span{s, page0, pages, o.rows};
+      base[s] = o.rows - page0 * kPage;
+      o.n_spans += 1;
+      o.max_pages = std::max(o.max_pages, pages);
+      o.rows += pages * kPage;
+      o.n_tiles += tiles;
+      tile += tiles;
+      if (o.rows > lat_cap) return efail("engine_step: a portion's latents do not fit their buffer");
+    }
+  }
   // row metadata, then the tile lists
   CU(cudaMemcpyAsync(d_io + io.tok, h_io + io.tok, (size_t)(io.pos - io.tok) + (size_t)rows * 4, cudaMemcpyHostToDevice, stream));
   CU(cudaMemcpyAsync(d_io + io.mix, h_io + io.mix, (size_t)n_mix * sizeof(nfn_row_tile), cudaMemcpyHostToDevice, stream));
   if (n_att > 0) CU(cudaMemcpyAsync(d_io + io.att, h_io + io.att, (size_t)n_att * 16, cudaMemcpyHostToDevice, stream));
 
   CU(cudaMemcpyAsync(d_io + io.seq, h_io + io.seq, (size_t)b.n_seq * sizeof(nfn_seq_rows), cudaMemcpyHostToDevice, stream));
+  if (lat_cap > 0 && rows > short_rows) CU(cudaMemcpyAsync(d_io + io.spans, h_io + io.spans, (size_t)(io.out - io.spans), cudaMemcpyHostToDevice, stream));
 
   b.rows = rows;
   b.short_rows = short_rows;

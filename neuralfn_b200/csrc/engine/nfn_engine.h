@@ -64,7 +64,8 @@ typedef struct {
 // input: x += RMS(proj(gelu_tanh(gate x) * side_embed[token, layer])) * side_norm. The output norm and the head follow.
 // With `chained` set in the configuration mixer and feed-forward are two sublayers, each with a norm of its own, and the residual may be
 // several streams: u = sum_s in[s] x_s, y = sublayer(RMS(u) * norm), x_t <- sum_s mix[s][t] x_s + out[t] y.
-enum { NFN_MIXER_ATTENTION = 0, NFN_MIXER_DELTA = 1 };
+// With `post_norm` the sublayers of such a layer read the residual itself and their outputs are normed: x <- x + residual_mult * RMS(sublayer(x)) * norm.
+enum { NFN_MIXER_ATTENTION = 0, NFN_MIXER_DELTA = 1, NFN_MIXER_LATENT = 2, NFN_MIXER_WKV = 3 };
 typedef struct {
   int heads, kv_heads;   // query head h reads key / value head h / (heads / kv_heads)
   int dim, vdim;         // per-head query / key size and value size
@@ -86,7 +87,22 @@ typedef struct {
   int rank_decay, rank_gate;   // delta: inner sizes of the decay and output-gate projections
   int experts, top, expert_ff; // chained: routed experts instead of a dense feed-forward (sigmoid scores, weight on the expert's input)
   int weights_of;        // >= 0: this layer runs with the tensors of that earlier one (a loop over layers); -1: its own
+  int chunk;             // > 0: keys of the query's own chunk of that many positions only (counted from the sequence's start), instead of a window
+  int qk_norm;           // per-head RMS norm on queries and keys before the rotation, a weight shared by the heads
+  int rot_dims;          // rotary positions on the first rot_dims dimensions of queries and keys, pairs (2i, 2i + 1); latent: on the rot_dim part
+  double rot_base;       // frequency of pair i: rot_base^(-2i / rot_dims)
+  int key_values;        // the values are the keys as projected, before norm and rotation; no value projection
+  int kv_rank, rot_dim;  // latent: size of the cached latent and of the rotated key part all heads share; dim: the unrotated part. With kv_from the earlier
+                         // layer's latents are read through this layer's own key and value projections
+  int expert_plain;      // experts down(act(up h)), weighted at their output, instead of gated ones weighted at their input
+  int shared_ff;         // width of an expert of the same (plain) form that every token has; 0: none
+  int route_correction;  // choice scores s + correction
+  int route_groups, route_keep;   // experts in equal groups of neighbours, of which the best are kept (0: no groups)
+  int route_normalise;   // weights divided by their sum
+  float route_scale;     // times this; 0 counts as 1
 } nfn_layer_desc;
+// Latent (NFN_MIXER_LATENT): q per head [dim | rot_dim], c = RMS(W_dkv h) cached with the rotated key part; score = (q . W_uk c + q_rot . k_rot) * scale, value W_uv c.
+// Wkv (NFN_MIXER_WKV): heads x dim, vdim = dim; token shift, bonus recurrence (nfn_wkv_rows), rank_decay the inner size of the decay projection.
 
 typedef struct {
   int n_layer, width, vocab;
@@ -104,6 +120,8 @@ typedef struct {
   float norm_offset;     // norms multiply by weight + norm_offset
   float logit_scale;     // logits *= logit_scale
   float logit_softcap;   // logits <- cap * tanh(logits / cap); 0: off
+  int post_norm;         // chained, one residual: norms on the sublayers' outputs
+  float residual_mult;   // post_norm: factor of the normed output
 } nfn_layered_config;
 
 enum { NFN_KV_PAGE = 64 };   // tokens per cache page

@@ -13,43 +13,16 @@
 //                         and K arrive in fragment order by bulk copies through a ring of shared memory stages.
 //
 // The products with the state are formed from fp32 values split into two bf16 parts each (high x high + high x low + low x high), which
-// keeps sixteen bits of every factor. Rounds of as many chunks as the workspace holds alternate between the two kernels, small enough
+// keeps sixteen bits of every factor. The scan also runs recurrences without corrections (U = V, no W: wkv_chunk.cu). Rounds of as many chunks as the workspace holds alternate between the two kernels, small enough
 // to stay in L2.
 #include <algorithm>
 
 #include "attention_v2.cuh"
 #include "common.h"
+#include "chunk_scan.cuh"
 #include "delta.cuh"
 
 namespace nfn {
-
-constexpr int DC_T = 16;                               // tokens of a chunk
-constexpr long long DC_WORKSPACE = 96LL << 20;
-
-// bytes of a (chunk, head) block of the scan's operands: [W, Q: dk / 16 steps x 4 tiles of 8 rows][K: dk / 8 tiles] x 32 lanes x 16 bytes, then
-// e^G_last of every channel
-__host__ __device__ constexpr int dc_block_bytes(int dk) { return 48 * dk * 4 + dk * 4; }
-__host__ __device__ constexpr int dc_uo_floats(int vdim_p) { return vdim_p * 32; }      // T V and P T V: [column tile][2][2 row tiles][32 lanes][4]
-
-struct DeltaChunkParams {
-  nfn_delta_args a;
-  int dk;                     // padded key channels: 64, 128 or 256
-  int chunk0, n_chunks;       // chunks [chunk0, chunk0 + n_chunks) of every sequence in this round
-  unsigned char* blocks;      // [seq][chunk][head][dc_block_bytes]
-  float* uo;                  // [seq][chunk][head][dc_uo_floats]
-  int* status;
-};
-
-// two fp32 values as bf16 pairs: the rounded values and what they leave out
-__device__ __forceinline__ void split_bf16(float a, float b, uint32_t& hi, uint32_t& lo) {
-  hi = pack_bf16x2(a, b);
-  const float2 f = unpack_bf16x2(hi);
-  lo = pack_bf16x2(a - f.x, b - f.y);
-}
-
-__device__ __forceinline__ void dc_bulk_store(void* dst, uint32_t src, uint32_t bytes) {
-  asm volatile("cp.async.bulk.global.shared::cta.bulk_group [%0], [%1], %2;" ::"l"(dst), "r"(src), "r"(bytes) : "memory");
-}
 
 // log2(1 + e^z): the series of log(1 + t) for small t = e^z keeps slow decays exact
 __device__ __forceinline__ float softplus_log2(float z) {
@@ -57,13 +30,6 @@ __device__ __forceinline__ float softplus_log2(float z) {
   const float s = t * (1.f - t * (0.5f - t * (0.33333333f - t * (0.25f - t * (0.2f - t * (0.16666667f - t * 0.14285714f))))));
   const float l = t < 0.125f ? s * 1.4426950408889634f : __log2f(1.f + t);
   return y > 28.f ? y : l;
-}
-
-// Where the 16-byte piece of lane `lane` lies inside operand tile `tile` of a block: the order keeps the writers of both kinds of tile, and
-// the scan's reads, on different banks.
-__device__ __forceinline__ uint32_t dc_piece(int tile, int lane, bool of_k) {
-  const int turn = of_k ? ((lane >> 3) & 3) | ((tile & 1) << 2) : ((tile >> 2) & 1) << 2;
-  return (uint32_t)(tile * 32 + (lane ^ turn)) * 16;
 }
 
 // NT threads, two neighbouring key channels each (dk = 2 NT), and value columns in pairs
@@ -221,7 +187,7 @@ delta_prepare_kernel(const DeltaChunkParams p) {
   const size_t block = ((size_t)blockIdx.z * p.n_chunks + blockIdx.x) * a.heads + h;
   // ---- W, Q, K of this thread's key channels, in the order of the scan's fragments: {first eight of the contraction: high, low; second: high, low} ----
   unsigned char* stage = dc_smem;
-  *reinterpret_cast<float2*>(stage + 48 * p.dk * 4 + c0 * 4) = make_float2(fast_exp2(G[DC_T - 1][0]), fast_exp2(G[DC_T - 1][1]));
+  *reinterpret_cast<float2*>(stage + dc_gamma_at(p.dk, true) + c0 * 4) = make_float2(fast_exp2(G[DC_T - 1][0]), fast_exp2(G[DC_T - 1][1]));
 #pragma unroll
   for (int r = 0; r < DC_T; r += 2)
 #pragma unroll
@@ -284,7 +250,7 @@ delta_prepare_kernel(const DeltaChunkParams p) {
   fence_proxy_async();
   __syncthreads();
   if (tid == 0) {
-    dc_bulk_store(p.blocks + block * dc_block_bytes(p.dk), smem_u32(stage), dc_block_bytes(p.dk));
+    dc_bulk_store(p.blocks + block * dc_block_bytes(p.dk, true), smem_u32(stage), dc_block_bytes(p.dk, true));
     asm volatile("cp.async.bulk.commit_group;" ::: "memory");
     asm volatile("cp.async.bulk.wait_group 0;" ::: "memory");
   }
@@ -308,12 +274,12 @@ __device__ __forceinline__ void dc_bulk_load(uint32_t dst, const void* src, uint
 // KS: warps that share a head's key channels, 64 each; the CTA's four warps take 4 / KS tiles of 16 value columns
 constexpr int DS_WARPS = 4, DS_CH = 64, DS_K = DS_CH / 16, DS_N = DS_CH / 8;      // a warp's steps of 16 and tiles of 8 channels
 // shared memory of a stage: the head's operand block, then T V and P T V of the CTA's column tiles
-__host__ __device__ constexpr int ds_stage_bytes(int ks) { return dc_block_bytes(DS_CH * ks) + DS_WARPS / ks * 2048; }
+__host__ __device__ constexpr int ds_stage_bytes(int ks, bool corrections) { return dc_block_bytes(DS_CH * ks, corrections) + DS_WARPS / ks * 2048; }
 __host__ __device__ constexpr int ds_stages(int ks) { return ks == 4 ? 3 : 4; }
-template <int KS>
+template <int KS, bool CORRECTIONS>
 __global__ void __launch_bounds__(DS_WARPS * 32)
 delta_scan_kernel(const DeltaChunkParams p) {
-  constexpr int DK = DS_CH * KS, TILES = DS_WARPS / KS, BLOCK = dc_block_bytes(DK), STAGE = ds_stage_bytes(KS), STAGES = ds_stages(KS);
+  constexpr int DK = DS_CH * KS, TILES = DS_WARPS / KS, WT = CORRECTIONS ? 4 : 2, BLOCK = dc_block_bytes(DK, CORRECTIONS), STAGE = ds_stage_bytes(KS, CORRECTIONS), STAGES = ds_stages(KS);
   extern __shared__ __align__(128) unsigned char dc_smem[];       // [STAGES][STAGE], then partial sums [2][warps][4 row tiles][32][4]
   __shared__ __align__(8) uint64_t bar_full[STAGES];
   __shared__ int cta_abort_s;
@@ -367,7 +333,7 @@ delta_scan_kernel(const DeltaChunkParams p) {
     for (int kk = 0; kk < DS_K; ++kk) {
       uint4 b[2];
 #pragma unroll
-      for (int nt = 0; nt < 2; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece((DS_K * ks + kk) * 4 + nt0 + nt, lane, false));
+      for (int nt = 0; nt < 2; ++nt) b[nt] = *reinterpret_cast<const uint4*>(stage + dc_piece<CORRECTIONS>((DS_K * ks + kk) * WT + nt0 + nt, lane, false));
 #pragma unroll
       for (int nt = 0; nt < 2; ++nt) {
         if (kk == 0) dc_mma0(acc[nt], hi[kk], b[nt].x, b[nt].z);
@@ -433,16 +399,22 @@ delta_scan_kernel(const DeltaChunkParams p) {
       split_bf16(s[2 * kk + 1][0], s[2 * kk + 1][1], hi[kk][2], lo[kk][2]);
       split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[kk][3], lo[kk][3]);
     }
-    float ws[2][4];
-    product(stage, 0, ws);
     if (i > 0) put(i, 2, qs);
-    put(i, 0, ws);
+    if constexpr (CORRECTIONS) {
+      float ws[2][4];
+      product(stage, 0, ws);
+      put(i, 0, ws);
+    }
     // every warp is done with chunk i - 2 here: its stage takes the next load
     __syncthreads();
     const int gave_up = *cta_abort;                      // set before the barrier by a thread whose wait ran out: all leave together
     if (tid == 0 && i > 1 && i - 2 + STAGES < n_chunks) load(i - 2 + STAGES);
-    const float4 w0 = sum(i, 0), w1 = sum(i, 1);
-    product(stage, 2, qs);
+    float4 w0 = make_float4(0.f, 0.f, 0.f, 0.f), w1 = w0;
+    if constexpr (CORRECTIONS) {
+      w0 = sum(i, 0);
+      w1 = sum(i, 1);
+    }
+    product(stage, WT - 2, qs);
     // U^T, as the A operand of S'^T = e^G_last S^T + U^T K
     const float* tv = reinterpret_cast<const float*>(stage + BLOCK) + (warp / KS) * 512 + lane * 4;
     const float4 v0 = *reinterpret_cast<const float4*>(tv), v1 = *reinterpret_cast<const float4*>(tv + 128);
@@ -451,20 +423,22 @@ delta_scan_kernel(const DeltaChunkParams p) {
     split_bf16(v0.z - w0.z, v0.w - w0.w, uh[1], ul[1]);
     split_bf16(v1.x - w1.x, v1.y - w1.y, uh[2], ul[2]);
     split_bf16(v1.z - w1.z, v1.w - w1.w, uh[3], ul[3]);
-    const float* gamma = reinterpret_cast<const float*>(stage + 48 * DK * 4) + DS_CH * ks + 2 * j;
+    const float* gamma = reinterpret_cast<const float*>(stage + dc_gamma_at(DK, CORRECTIONS)) + DS_CH * ks + 2 * j;
     uint4 kb[DS_N];
 #pragma unroll
     for (int t = 0; t < DS_N; ++t) {
       const float2 f = *reinterpret_cast<const float2*>(gamma + 8 * t);
-      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece(4 * (DK / 16) + DS_N * ks + t, lane, true));
+      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece<CORRECTIONS>(WT * (DK / 16) + DS_N * ks + t, lane, true));
       s[t][0] *= f.x; s[t][1] *= f.y; s[t][2] *= f.x; s[t][3] *= f.y;
     }
 #pragma unroll
     for (int t = 0; t < DS_N; ++t) dc_mma(s[t], uh, kb[t].x, kb[t].z);
 #pragma unroll
     for (int t = 0; t < DS_N; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
+    if constexpr (CORRECTIONS) {                         // values on their own are bf16: nothing was left out
 #pragma unroll
-    for (int t = 0; t < DS_N; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
+      for (int t = 0; t < DS_N; ++t) dc_mma(s[t], ul, kb[t].x, kb[t].z);
+    }
     if (gave_up) break;
     if (i > 0) read_out(i - 1, i);
     if (++at == STAGES) { at = 0; phase ^= 1; }
@@ -486,10 +460,10 @@ delta_scan_kernel(const DeltaChunkParams p) {
     }
 }
 
-template <int KS>
+template <int KS, bool CORRECTIONS>
 static int launch_scan(const DeltaChunkParams& p, cudaStream_t st) {
-  constexpr int SMEM = ds_stages(KS) * ds_stage_bytes(KS) + 2 * DS_WARPS * 512 * 4;
-  auto kern = delta_scan_kernel<KS>;
+  constexpr int SMEM = ds_stages(KS) * ds_stage_bytes(KS, CORRECTIONS) + 2 * DS_WARPS * 512 * 4;
+  auto kern = delta_scan_kernel<KS, CORRECTIONS>;
   static bool raised[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -501,9 +475,14 @@ static int launch_scan(const DeltaChunkParams& p, cudaStream_t st) {
   return launch_check("delta_scan");
 }
 
+int chunk_scan(const DeltaChunkParams& p, bool corrections, cudaStream_t st) {
+  if (corrections) return p.dk == 64 ? launch_scan<1, true>(p, st) : p.dk == 128 ? launch_scan<2, true>(p, st) : launch_scan<4, true>(p, st);
+  return p.dk == 64 ? launch_scan<1, false>(p, st) : p.dk == 128 ? launch_scan<2, false>(p, st) : launch_scan<4, false>(p, st);
+}
+
 template <int NT>
 static int launch_prepare(const DeltaChunkParams& p, cudaStream_t st) {
-  constexpr int SMEM = std::max(64 * (NT == 128 ? 136 : NT + 4) * 4, dc_block_bytes(2 * NT));
+  constexpr int SMEM = std::max(64 * (NT == 128 ? 136 : NT + 4) * 4, dc_block_bytes(2 * NT, true));
   auto kern = delta_prepare_kernel<NT>;
   static bool raised[64] = {};
   int dev = 0;
@@ -526,7 +505,7 @@ extern "C" long long nfn_delta_chunk_workspace_bytes(int heads, int dim_p, int v
   if (dim_p > 256) return 0;
   const int dk = dim_p <= 64 ? 64 : dim_p <= 128 ? 128 : 256;
   // at least one chunk of every head and sequence
-  return std::max<long long>(DC_WORKSPACE, (long long)max_seqs * heads * (dc_block_bytes(dk) + dc_uo_floats(vdim_p) * 4LL));
+  return std::max<long long>(DC_WORKSPACE, (long long)max_seqs * heads * (dc_block_bytes(dk, true) + dc_uo_floats(vdim_p) * 4LL));
 }
 
 extern "C" int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* workspace, long long workspace_bytes, nfn_stream_t stream) {
@@ -538,16 +517,16 @@ extern "C" int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* 
   p.a = *args;
   p.dk = args->dim_p <= 64 ? 64 : args->dim_p <= 128 ? 128 : 256;
   p.status = status_ptr();
-  const long long per_chunk = (long long)args->n_seqs * args->heads * (dc_block_bytes(p.dk) + dc_uo_floats(args->vdim_p) * 4LL);
+  const long long per_chunk = (long long)args->n_seqs * args->heads * (dc_block_bytes(p.dk, true) + dc_uo_floats(args->vdim_p) * 4LL);
   const int total = ceil_div(max_rows, DC_T), round = (int)std::min<long long>(total, workspace_bytes / per_chunk);
   if (!workspace || round < 1) return fail(-1, "delta rule: the workspace holds no chunk");
   p.blocks = static_cast<unsigned char*>(workspace);
-  p.uo = reinterpret_cast<float*>(p.blocks + (size_t)round * args->n_seqs * args->heads * dc_block_bytes(p.dk));
+  p.uo = reinterpret_cast<float*>(p.blocks + (size_t)round * args->n_seqs * args->heads * dc_block_bytes(p.dk, true));
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   for (p.chunk0 = 0; p.chunk0 < total; p.chunk0 += round) {
     p.n_chunks = std::min(round, total - p.chunk0);
     int rc = p.dk == 64 ? launch_prepare<32>(p, st) : p.dk == 128 ? launch_prepare<64>(p, st) : launch_prepare<128>(p, st);
-    if (rc == 0) rc = p.dk == 64 ? launch_scan<1>(p, st) : p.dk == 128 ? launch_scan<2>(p, st) : launch_scan<4>(p, st);
+    if (rc == 0) rc = chunk_scan(p, true, st);
     if (rc) return rc;
   }
   return 0;

@@ -248,11 +248,11 @@ static int launch_delta_step(const nfn_delta_step_args& a, cudaStream_t st) {
   return launch_check("delta_step");
 }
 
-// One warp per (row, head): o / rms(o) * weight * sigmoid(gate).
-template <typename T>
+// One warp per (row, head): o / rms(o) * weight * sigmoid(gate), with SILU also times gate. Weights weight_pitch apart for every head (0: shared).
+template <typename T, bool SILU>
 __global__ void __launch_bounds__(256)
-delta_out_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_gate, const __nv_bfloat16* __restrict__ weight, float eps,
-                 T* __restrict__ out, int ld_out, int rows, int heads, int vdim, int vdim_p) {
+delta_out_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ gate, int ld_gate, const __nv_bfloat16* __restrict__ weight, int weight_pitch,
+                 float eps, T* __restrict__ out, int ld_out, int rows, int heads, int vdim, int vdim_p) {
   const long long item = (long long)blockIdx.x * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
   if (item >= (long long)rows * heads) return;
@@ -269,7 +269,9 @@ delta_out_kernel(const float* __restrict__ o, int ld_o, const T* __restrict__ ga
   const T* g = gate + (size_t)row * ld_gate + (size_t)h * vdim_p;
   T* dst = out + (size_t)row * ld_out + (size_t)h * vdim_p;
   for (int c = lane * 4; c < vdim_p; c += 128) {
-    const float4 f = load4(src + c), z = load4(g + c), w = load4(weight + c);
+    const float4 f = load4(src + c), z = load4(g + c);
+    float4 w = load4(weight + (size_t)h * weight_pitch + c);
+    if (SILU) { w.x *= z.x; w.y *= z.y; w.z *= z.z; w.w *= z.w; }
     store4(dst + c, make_float4(f.x * r * w.x * sigmoid_for<T>(z.x), f.y * r * w.y * sigmoid_for<T>(z.y), f.z * r * w.z * sigmoid_for<T>(z.z),
                                 f.w * r * w.w * sigmoid_for<T>(z.w)));
   }
@@ -328,19 +330,27 @@ extern "C" int nfn_delta_step(const nfn_delta_step_args* args, nfn_stream_t stre
   return a.f32 ? launch_delta_step<float>(a, static_cast<cudaStream_t>(stream)) : launch_delta_step<__nv_bfloat16>(a, static_cast<cudaStream_t>(stream));
 }
 
+template <typename T, bool SILU>
+static void launch_head_out(const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, int weight_pitch, float eps, void* out, int ld_out, int rows,
+                            int heads, int vdim, int vdim_p, cudaStream_t st) {
+  const unsigned blocks = (unsigned)(((long long)rows * heads + 7) / 8);
+  delta_out_kernel<T, SILU><<<blocks, 256, 0, st>>>(o, ld_o, static_cast<const T*>(gate), ld_gate, static_cast<const __nv_bfloat16*>(weight), weight_pitch, eps,
+                                                    static_cast<T*>(out), ld_out, rows, heads, vdim, vdim_p);
+}
+
+extern "C" int nfn_head_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, int gate_act, const void* weight, int weight_pitch, float eps, void* out,
+                            int ld_out, int rows, int heads, int vdim, int vdim_p, nfn_stream_t stream) {
+  if (rows <= 0) return 0;
+  if ((vdim_p & 15) || vdim <= 0 || vdim > vdim_p || ((ld_o | ld_gate | ld_out | weight_pitch) & 7)) return fail(-1, "head_out: misaligned rows or head sizes");
+  if (((long long)rows * heads + 7) / 8 > 0x7fffffffLL) return fail(-1, "head_out: too many rows for one launch");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  const bool silu = gate_act == NFN_ACT_SILU;
+  auto run = f32 ? (silu ? launch_head_out<float, true> : launch_head_out<float, false>) : (silu ? launch_head_out<__nv_bfloat16, true> : launch_head_out<__nv_bfloat16, false>);
+  run(o, ld_o, gate, ld_gate, weight, weight_pitch, eps, out, ld_out, rows, heads, vdim, vdim_p, st);
+  return launch_check("head_out");
+}
+
 extern "C" int nfn_delta_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, float eps, void* out, int ld_out, int rows,
                              int heads, int vdim, int vdim_p, nfn_stream_t stream) {
-  if (rows <= 0) return 0;
-  if ((vdim_p & 15) || vdim <= 0 || vdim > vdim_p || ((ld_o | ld_gate | ld_out) & 7)) return fail(-1, "delta_out: misaligned rows or head sizes");
-  const long long blocks = ((long long)rows * heads + 7) / 8;
-  if (blocks > 0x7fffffffLL) return fail(-1, "delta_out: too many rows for one launch");
-  cudaStream_t st = static_cast<cudaStream_t>(stream);
-  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(weight);
-  if (f32)
-    delta_out_kernel<float><<<(unsigned)blocks, 256, 0, st>>>(o, ld_o, static_cast<const float*>(gate), ld_gate, w, eps, static_cast<float*>(out), ld_out, rows,
-                                                              heads, vdim, vdim_p);
-  else
-    delta_out_kernel<__nv_bfloat16><<<(unsigned)blocks, 256, 0, st>>>(o, ld_o, static_cast<const __nv_bfloat16*>(gate), ld_gate, w, eps,
-                                                                      static_cast<__nv_bfloat16*>(out), ld_out, rows, heads, vdim, vdim_p);
-  return launch_check("delta_out");
+  return nfn_head_out(f32, o, ld_o, gate, ld_gate, NFN_ACT_NONE, weight, 0, eps, out, ld_out, rows, heads, vdim, vdim_p, stream);
 }

@@ -1,0 +1,385 @@
+// Between a layer's input projection and its attention, for designs with rotary positions: per-head norm and rotation of queries and keys,
+// the latent and shared key part of latent attention, cache append, the per-head products around a latent cache, and the gather of
+// visible latents in front of a prompt's expansion.
+//
+// Angles are formed in fp32 from frequencies given as two parts (high, low): position * frequency is exact to the last bit of the sum, so a
+// rotation at a far position is as good as one near the start. All arithmetic between loads and stores is fp32. Rotations may happen
+// in place: every element is read and written by one thread.
+#include <algorithm>
+
+#include "common.h"
+#include "paged.cuh"
+
+namespace nfn {
+
+constexpr int HR_THREADS = 256, HR_WARPS = HR_THREADS / 32, HR_ROWS = 16;
+
+__device__ __forceinline__ float2 rotation(int pos, const float* freq, int i) {
+  const float p = (float)pos, f = freq[2 * i], hi = p * f, lo = fmaf(p, f, -hi) + p * freq[2 * i + 1];
+  float s, c;
+  sincosf(hi, &s, &c);
+  const float q = 1.f - 0.5f * lo * lo;
+  return make_float2(c * q - s * lo, s * q + c * lo);
+}
+
+// cos and sin of every row and pair of the tile, [rows][half]
+__device__ __forceinline__ void fill_rotations(float2* cs, const float* freq, int half, int pos0, int n) {
+  for (int i = threadIdx.x; i < n * half; i += HR_THREADS) cs[i] = rotation(pos0 + i / half, freq, i % half);
+}
+
+// dimensions c .. c + 3 of a head: the pairs below rot_dims turn
+__device__ __forceinline__ float4 rotate4(const float4& v, const float2* cs, int c, int rot_dims) {
+  float4 o = v;
+  if (c + 1 < rot_dims) {
+    const float2 a = cs[c / 2];
+    o.x = v.x * a.x - v.y * a.y;
+    o.y = v.y * a.x + v.x * a.y;
+  }
+  if (c + 3 < rot_dims) {
+    const float2 a = cs[c / 2 + 1];
+    o.z = v.z * a.x - v.w * a.y;
+    o.w = v.w * a.x + v.z * a.y;
+  }
+  return o;
+}
+
+__device__ __forceinline__ float warp_sum(float v) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
+  return v;
+}
+__device__ __forceinline__ float squares(const float4& v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+
+// A warp takes one query or key head for all rows of a tile, R rows in flight. NV: 128-wide pieces of a head.
+template <typename T, int NV>
+__global__ void __launch_bounds__(HR_THREADS)
+head_rows_kernel(const nfn_head_rows_args p) {
+  extern __shared__ float2 hr_cs[];
+  constexpr int R = NV >= 4 ? 1 : 4 / NV;
+  const nfn_row_tile t = p.tiles[blockIdx.x];
+  if (t.slot < 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dims / 2;
+  const int pos0 = t.e_pos0 + t.row0 - t.e_row0;
+  fill_rotations(hr_cs, p.freq, half, pos0, t.n);
+  __syncthreads();
+  const int item = blockIdx.y * HR_WARPS + warp;
+  const bool key = item >= p.heads;
+  const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
+  const size_t page = p.kv_heads > 0 ? (size_t)p.table[(size_t)t.slot * p.table_ld + pos0 / NFN_PAGE] : 0;
+  const int in_page = pos0 % NFN_PAGE;
+  if (item < p.heads + p.kv_heads) {
+    const int head = key ? item - p.heads : item;
+    const T* src = in + (key ? p.off_k : 0) + head * p.dim_p;
+    T* dst = key ? static_cast<T*>(p.k_pool) + ((page * p.kv_heads + head) * NFN_PAGE + in_page) * p.dim_p
+                 : static_cast<T*>(p.q_out) + (size_t)t.row0 * p.ld_q + head * p.dim_p;
+    const int ld_dst = key ? p.dim_p : p.ld_q;
+    const __nv_bfloat16* weight = static_cast<const __nv_bfloat16*>(key ? p.k_norm : p.q_norm);
+    float4 w[NV];
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int c = lane * 4 + j * 128;
+      w[j] = weight && c < p.dim_p ? load4(weight + c) : make_float4(1.f, 1.f, 1.f, 1.f);
+    }
+    for (int i0 = 0; i0 < t.n; i0 += R) {
+      float4 v[R][NV];
+#pragma unroll
+      for (int i = 0; i < R; ++i)
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          const int c = lane * 4 + j * 128;
+          v[i][j] = i0 + i < t.n && c < p.dim_p ? load4(src + (size_t)(i0 + i) * p.ld_in + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+#pragma unroll
+      for (int i = 0; i < R; ++i) {
+        if (i0 + i >= t.n) break;
+        if (weight) {
+          float ss = 0.f;
+#pragma unroll
+          for (int j = 0; j < NV; ++j) ss += squares(v[i][j]);
+          const float r = 1.f / sqrtf(warp_sum(ss) / (float)p.dim + p.eps);
+#pragma unroll
+          for (int j = 0; j < NV; ++j) {
+            v[i][j].x *= r * w[j].x; v[i][j].y *= r * w[j].y; v[i][j].z *= r * w[j].z; v[i][j].w *= r * w[j].w;
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < NV; ++j) {
+          const int c = lane * 4 + j * 128;
+          if (c < p.dim_p) store4(dst + (size_t)(i0 + i) * ld_dst + c, rotate4(v[i][j], hr_cs + (i0 + i) * half, c, p.rot_dims));
+        }
+      }
+    }
+  }
+  // values, channel-major
+  const int n_v = p.kv_heads * p.vdim_p;
+  for (int ch = blockIdx.y * HR_THREADS + threadIdx.x; ch < n_v; ch += gridDim.y * HR_THREADS) {
+    const T* src = in + p.off_v + ch;
+    T* dst = static_cast<T*>(p.v_pool) + (page * n_v + ch) * NFN_PAGE + in_page;
+    if (t.n == HR_ROWS) {
+      T buf[HR_ROWS];
+#pragma unroll
+      for (int i = 0; i < HR_ROWS; ++i) buf[i] = src[(size_t)i * p.ld_in];
+#pragma unroll
+      for (int q = 0; q < HR_ROWS * (int)sizeof(T) / 16; ++q) reinterpret_cast<uint4*>(dst)[q] = pack16(&buf[q * (16 / sizeof(T))]);
+    } else {
+      for (int i = 0; i < t.n; ++i) dst[i] = src[(size_t)i * p.ld_in];
+    }
+  }
+}
+
+// A warp takes one query head, or the latent and shared key part, of all rows of a tile.
+template <typename T, int NV>
+__global__ void __launch_bounds__(HR_THREADS)
+latent_rows_kernel(const nfn_latent_rows_args p) {
+  extern __shared__ float2 hr_cs[];
+  const nfn_row_tile t = p.tiles[blockIdx.x];
+  if (t.slot < 0) return;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dim / 2;
+  const int pos0 = t.e_pos0 + t.row0 - t.e_row0;
+  fill_rotations(hr_cs, p.freq, half, pos0, t.n);
+  __syncthreads();
+  const int item = blockIdx.y * HR_WARPS + warp, pitch = p.dim_p + p.rot_p, lp = p.rank_p + p.rot_p;
+  const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
+  if (item < p.heads) {
+    const bool lat = t.row0 < p.q_row0;                    // rows of an entry are all short or all long
+    const T* src = in + item * pitch;
+    T* dst = lat ? static_cast<T*>(p.q_lat) + (size_t)t.row0 * p.heads * lp + (size_t)item * lp + p.rank_p
+                 : static_cast<T*>(p.q_out) + (size_t)t.row0 * p.ld_q + item * pitch + p.dim_p;
+    const size_t ld_dst = lat ? (size_t)p.heads * lp : (size_t)p.ld_q;
+    // pieces of four over the tile's rows: narrow rotated parts leave no lane idle
+    const int quads = p.rot_p / 4;
+    for (int x = lane; x < quads * t.n; x += 32) {
+      const int i = x / quads, c = x % quads * 4;
+      store4(dst + i * ld_dst + c, rotate4(load4(src + (size_t)i * p.ld_in + p.dim_p + c), hr_cs + i * half, c, p.rot_dim));
+    }
+    if (!lat && p.q_out != p.in)
+      for (int i = 0; i < t.n; ++i)
+        for (int c = lane * 4; c < p.dim_p; c += 128) store4(dst + i * ld_dst - p.dim_p + c, load4(src + (size_t)i * p.ld_in + c));
+    return;
+  }
+  if (item > p.heads || !p.k_pool) return;
+  const size_t page = (size_t)p.table[(size_t)t.slot * p.table_ld + pos0 / NFN_PAGE];
+  T* dst = static_cast<T*>(p.k_pool) + (page * NFN_PAGE + pos0 % NFN_PAGE) * lp;
+  const T* src = in + p.off_kv;
+  const __nv_bfloat16* weight = static_cast<const __nv_bfloat16*>(p.c_norm);
+  for (int i = 0; i < t.n; ++i) {
+    const T* row = src + (size_t)i * p.ld_in;
+    float4 v[NV];
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < NV; ++j) {
+      const int c = lane * 4 + j * 128;
+      v[j] = c < p.rank_p ? load4(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      ss += squares(v[j]);
+    }
+    for (int c = lane * 4 + NV * 128; c < p.rank_p; c += 128) ss += squares(load4(row + c));
+    const float r = 1.f / sqrtf(warp_sum(ss) / (float)p.rank + p.eps);
+    auto leave = [&](const float4& f, int c) {
+      const float4 w = load4(weight + c);
+      store4(dst + (size_t)i * lp + c, make_float4(f.x * r * w.x, f.y * r * w.y, f.z * r * w.z, f.w * r * w.w));
+    };
+#pragma unroll
+    for (int j = 0; j < NV; ++j)
+      if (lane * 4 + j * 128 < p.rank_p) leave(v[j], lane * 4 + j * 128);
+    for (int c = lane * 4 + NV * 128; c < p.rank_p; c += 128) leave(load4(row + c), c);
+    for (int c = lane * 4; c < p.rot_p; c += 128)
+      store4(dst + (size_t)i * lp + p.rank_p + c, rotate4(load4(row + p.rank_p + c), hr_cs + i * half, c, p.rot_dim));
+  }
+}
+
+// ------------------------------------------------------------------------------------------------ per-group products --
+// 32-bit mode: a warp per weight row, eight rows at a time.
+constexpr int GP_WARPS = 8, GP_ROWS = 8;
+
+__global__ void __launch_bounds__(GP_WARPS * 32)
+group_products_f32_kernel(const nfn_group_products_args p) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = blockIdx.x * GP_WARPS + warp, g = blockIdx.y, r0 = blockIdx.z * GP_ROWS;
+  if (n >= p.n) return;
+  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(p.w) + ((size_t)g * p.n + n) * p.k;
+  const float* in = static_cast<const float*>(p.in) + (size_t)r0 * p.ld_in + (size_t)g * p.in_group;
+  const int live = min(GP_ROWS, p.rows - r0);
+  float a[GP_ROWS];
+#pragma unroll
+  for (int i = 0; i < GP_ROWS; ++i) a[i] = 0.f;
+  for (int k = lane * 4; k < p.k; k += 128) {
+    const float4 f = load4(w + k);
+#pragma unroll
+    for (int i = 0; i < GP_ROWS; ++i) {
+      if (i >= live) break;
+      const float4 x = load4(in + (size_t)i * p.ld_in + k);
+      a[i] += (f.x * x.x + f.y * x.y) + (f.z * x.z + f.w * x.w);
+    }
+  }
+  float* out = static_cast<float*>(p.out) + (size_t)r0 * p.ld_out + (size_t)g * p.out_group + n;
+#pragma unroll
+  for (int i = 0; i < GP_ROWS; ++i) {
+    if (i >= live) break;
+    const float s = warp_sum(a[i]);
+    if (lane == 0) out[(size_t)i * p.ld_out] = s;
+  }
+}
+
+// bf16, on the tensor cores: a CTA takes 32 weight rows of a group, its warps a quarter of the contraction each; rows are the eight columns of
+// mma.m16n8k16. The order of a contraction is free, so every fragment is one 16-byte load per lane.
+constexpr int GM_WARPS = 4;
+
+__device__ __forceinline__ uint4 gm_stream(const __nv_bfloat16* p) {
+  uint4 v;
+  asm volatile("ld.global.nc.L1::no_allocate.v4.u32 {%0,%1,%2,%3}, [%4];" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "l"(p));
+  return v;
+}
+__device__ __forceinline__ void gm_mma(float (&d)[4], uint32_t a0, uint32_t a1, uint32_t a2, uint32_t a3, uint32_t b0, uint32_t b1) {
+  asm("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+      : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
+      : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
+}
+
+template <int NT>
+__global__ void __launch_bounds__(GM_WARPS * 32)
+group_products_mma_kernel(const nfn_group_products_args p) {
+  constexpr int M = 8 * NT, U = NT == 4 ? 2 : 4;          // rows at a time, 32-wide steps in flight
+  __shared__ float part[GM_WARPS][32][M + 1];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, j = lane & 3, g = blockIdx.y;
+  const int n0 = blockIdx.x * 32, r0 = blockIdx.z * M;
+  const bool two = n0 + 16 < p.n;
+  const __nv_bfloat16* w0 = static_cast<const __nv_bfloat16*>(p.w) + ((size_t)g * p.n + n0 + gr) * p.k + 8 * j;
+  const __nv_bfloat16* w1 = two ? w0 + (size_t)16 * p.k : w0;
+  const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
+  const __nv_bfloat16* src[NT];
+  bool on[NT];
+#pragma unroll
+  for (int t = 0; t < NT; ++t) {
+    const int r = r0 + 8 * t + gr;
+    on[t] = r < p.rows;
+    src[t] = static_cast<const __nv_bfloat16*>(p.in) + (size_t)(on[t] ? r : r0) * p.ld_in + (size_t)g * p.in_group + 8 * j;
+  }
+  float acc[2][NT][4];
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) acc[m][t][c] = 0.f;
+  const int steps = (p.k + 31) / 32, s0 = steps * warp / GM_WARPS, s1 = steps * (warp + 1) / GM_WARPS;
+  for (int s = s0; s < s1; s += U) {
+    uint4 a[U][4], b[U][NT];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int k = (s + u) * 32;
+      const bool ok = s + u < s1 && k + 8 * j < p.k;
+      a[u][0] = ok ? gm_stream(w0 + k) : zero4;
+      a[u][1] = ok ? gm_stream(w0 + (size_t)8 * p.k + k) : zero4;
+      a[u][2] = ok ? gm_stream(w1 + k) : zero4;
+      a[u][3] = ok ? gm_stream(w1 + (size_t)8 * p.k + k) : zero4;
+#pragma unroll
+      for (int t = 0; t < NT; ++t) b[u][t] = ok && on[t] ? *reinterpret_cast<const uint4*>(src[t] + k) : zero4;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+#pragma unroll
+      for (int t = 0; t < NT; ++t) {
+        gm_mma(acc[0][t], a[u][0].x, a[u][1].x, a[u][0].y, a[u][1].y, b[u][t].x, b[u][t].y);
+        gm_mma(acc[1][t], a[u][2].x, a[u][3].x, a[u][2].y, a[u][3].y, b[u][t].x, b[u][t].y);
+        gm_mma(acc[0][t], a[u][0].z, a[u][1].z, a[u][0].w, a[u][1].w, b[u][t].z, b[u][t].w);
+        gm_mma(acc[1][t], a[u][2].z, a[u][3].z, a[u][2].w, a[u][3].w, b[u][t].z, b[u][t].w);
+      }
+  }
+#pragma unroll
+  for (int m = 0; m < 2; ++m)
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+#pragma unroll
+      for (int c = 0; c < 4; ++c) part[warp][m * 16 + gr + (c >> 1) * 8][8 * t + 2 * j + (c & 1)] = acc[m][t][c];
+  __syncthreads();
+  const int live = min(M, p.rows - r0);
+  for (int x = threadIdx.x; x < 32 * live; x += GM_WARPS * 32) {
+    const int col = x / 32, row = x % 32;
+    if (n0 + row >= p.n) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int w = 0; w < GM_WARPS; ++w) v += part[w][row][col];
+    static_cast<__nv_bfloat16*>(p.out)[(size_t)(r0 + col) * p.ld_out + (size_t)g * p.out_group + n0 + row] = __float2bfloat16(v);
+  }
+}
+
+// one CTA per page: 64 rows of `vecs` 16-byte pieces
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ pool, int ld_pool, int vecs, const int* __restrict__ table, int table_ld, const nfn_latent_span* __restrict__ spans,
+                     uint4* __restrict__ out) {
+  const nfn_latent_span s = spans[blockIdx.y];
+  if (s.slot < 0 || (int)blockIdx.x >= s.n_pages) return;
+  const uint4* src = pool + (size_t)table[(size_t)s.slot * table_ld + s.first_page + blockIdx.x] * NFN_PAGE * ld_pool;
+  uint4* dst = out + ((size_t)s.row0 + (size_t)blockIdx.x * NFN_PAGE) * vecs;
+  for (int i = threadIdx.x; i < NFN_PAGE * vecs; i += 256) dst[i] = src[(size_t)(i / vecs) * ld_pool + i % vecs];
+}
+
+template <typename T>
+static int launch_head_rows(const nfn_head_rows_args& a, cudaStream_t st) {
+  const dim3 grid(a.n_tiles, ceil_div(a.heads + a.kv_heads, HR_WARPS));
+  const size_t smem = (size_t)std::max(1, a.tile_rows * (a.rot_dims / 2)) * sizeof(float2);
+  if (a.dim_p <= 128) head_rows_kernel<T, 1><<<grid, HR_THREADS, smem, st>>>(a);
+  else if (a.dim_p <= 256) head_rows_kernel<T, 2><<<grid, HR_THREADS, smem, st>>>(a);
+  else head_rows_kernel<T, 4><<<grid, HR_THREADS, smem, st>>>(a);
+  return launch_check("head_rows");
+}
+
+template <typename T>
+static int launch_latent_rows(const nfn_latent_rows_args& a, cudaStream_t st) {
+  const dim3 grid(a.n_tiles, ceil_div(a.heads + 1, HR_WARPS));
+  const size_t smem = (size_t)std::max(1, a.tile_rows * (a.rot_dim / 2)) * sizeof(float2);
+  latent_rows_kernel<T, 4><<<grid, HR_THREADS, smem, st>>>(a);
+  return launch_check("latent_rows");
+}
+
+}  // namespace nfn
+
+using namespace nfn;
+
+extern "C" int nfn_head_rows(const nfn_head_rows_args* args, nfn_stream_t stream) {
+  if (!args) return fail(-1, "head_rows: null args");
+  const nfn_head_rows_args& a = *args;
+  if (a.n_tiles <= 0) return 0;
+  if ((a.ld_in | a.off_k | a.off_v | a.dim_p | a.vdim_p | a.ld_q) & 7) return fail(-1, "head_rows: widths and offsets must be multiples of 8");
+  if (a.heads <= 0 || a.kv_heads < 0 || a.dim <= 0 || a.dim > a.dim_p || a.dim_p > 512) return fail(-1, "head_rows: heads of at most 512 dimensions");
+  if ((a.rot_dims & 1) || a.rot_dims < 0 || a.rot_dims > a.dim || (a.rot_dims > 0 && !a.freq)) return fail(-1, "head_rows: an even number of rotated dimensions, with their frequencies");
+  if (a.tile_rows < 1 || a.tile_rows > HR_ROWS) return fail(-1, "head_rows: tiles hold 1 to 16 rows");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return a.f32 ? launch_head_rows<float>(a, st) : launch_head_rows<__nv_bfloat16>(a, st);
+}
+
+extern "C" int nfn_latent_rows(const nfn_latent_rows_args* args, nfn_stream_t stream) {
+  if (!args) return fail(-1, "latent_rows: null args");
+  const nfn_latent_rows_args& a = *args;
+  if (a.n_tiles <= 0) return 0;
+  if ((a.ld_in | a.off_kv | a.dim_p | a.rot_p | a.rank_p | a.ld_q) & 7) return fail(-1, "latent_rows: widths and offsets must be multiples of 8");
+  if ((a.rot_dim & 1) || a.rot_dim <= 0 || a.rot_dim > a.rot_p || !a.freq) return fail(-1, "latent_rows: an even number of rotated dimensions, with their frequencies");
+  if (a.k_pool && (!a.c_norm || a.rank <= 0 || a.rank > a.rank_p)) return fail(-1, "latent_rows: the latent needs its norm");
+  if (a.q_row0 > 0 && !a.q_lat) return fail(-1, "latent_rows: short rows need their query buffer");
+  if (a.tile_rows < 1 || a.tile_rows > HR_ROWS || (size_t)a.tile_rows * (a.rot_dim / 2) * sizeof(float2) > 48 * 1024) return fail(-1, "latent_rows: tiles hold 1 to 16 rows of at most 768 rotated dimensions");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return a.f32 ? launch_latent_rows<float>(a, st) : launch_latent_rows<__nv_bfloat16>(a, st);
+}
+
+extern "C" int nfn_group_products(const nfn_group_products_args* args, nfn_stream_t stream) {
+  if (!args) return fail(-1, "group_products: null args");
+  const nfn_group_products_args& a = *args;
+  if (a.rows <= 0) return 0;
+  if (a.groups <= 0 || a.groups > 65535 || ((a.n | a.k) & 15) || a.n <= 0 || a.k <= 0 || ((a.ld_in | a.in_group) & 7)) return fail(-1, "group_products: sizes must be multiples of 16");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (ceil_div(a.rows, 8) > 65535) return fail(-1, "group_products: too many rows in one launch");
+  if (a.f32) group_products_f32_kernel<<<dim3(ceil_div(a.n, GP_WARPS), a.groups, ceil_div(a.rows, GP_ROWS)), GP_WARPS * 32, 0, st>>>(a);
+  else if (a.rows <= 8) group_products_mma_kernel<1><<<dim3(ceil_div(a.n, 32), a.groups, 1), GM_WARPS * 32, 0, st>>>(a);
+  else if (a.rows <= 16) group_products_mma_kernel<2><<<dim3(ceil_div(a.n, 32), a.groups, 1), GM_WARPS * 32, 0, st>>>(a);
+  else group_products_mma_kernel<4><<<dim3(ceil_div(a.n, 32), a.groups, ceil_div(a.rows, 32)), GM_WARPS * 32, 0, st>>>(a);
+  return launch_check("group_products");
+}
+
+extern "C" int nfn_latent_gather(int f32, const void* pool, int ld_pool, int cols, const int* table, int table_ld, const nfn_latent_span* spans, int n_spans,
+                                 int max_pages, void* out, nfn_stream_t stream) {
+  if (n_spans <= 0 || max_pages <= 0) return 0;
+  const int per = f32 ? 4 : 8;
+  if (ld_pool % per || cols % per || n_spans > 65535) return fail(-1, "latent_gather: rows of 16-byte pieces, at most 65535 spans");
+  latent_gather_kernel<<<dim3(max_pages, n_spans), 256, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const uint4*>(pool), ld_pool / per, cols / per, table, table_ld,
+                                                                                                 spans, static_cast<uint4*>(out));
+  return launch_check("latent_gather");
+}

@@ -14,6 +14,7 @@
 #include <cfloat>
 
 #include "common.h"
+#include "moe_choice.cuh"
 #include "nfn_kernels.h"
 #include "sm100_ptx.cuh"
 
@@ -82,6 +83,22 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, 
     topk_w[(long long)tok * k + lane] = wsel * norm;
     atomicAdd(&counts[isel], 1);
   }
+}
+
+// The same with the choice of nfn_route_rule
+__global__ void __launch_bounds__(256)
+moe_choose_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, nfn_route_rule rule, int* topk_idx, float* topk_w, int* __restrict__ counts) {
+  __shared__ int count[MOE_MAX_E];
+  const int tok = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  count[threadIdx.x] = 0;
+  __syncthreads();
+  if (tok < T) {
+    int* idx = topk_idx + (long long)tok * k;
+    choose_experts<MOE_MAX_E / 32>(logits + (long long)tok * ld, E, k, rule, lane, idx, topk_w + (long long)tok * k);
+    for (int j = lane; j < k; j += 32) atomicAdd(&count[idx[j]], 1);
+  }
+  __syncthreads();
+  if (count[threadIdx.x]) atomicAdd(&counts[threadIdx.x], count[threadIdx.x]);
 }
 
 // plan[0] = live m tiles, plan[1] = padded rows; offsets[e] = first row of expert e
@@ -173,6 +190,16 @@ extern "C" int nfn_moe_route(const float* logits, int ld, int T, int E, int k, i
   moe_route_kernel<<<(T + 7) / 8, 256, 0, static_cast<cudaStream_t>(stream)>>>(logits, ld, T, E, k, score_fn, norm_topk, route_scale, topk_idx,
                                                                                topk_w, counts);
   return launch_check("moe_route", 1);
+}
+
+extern "C" int nfn_moe_choose(const float* logits, int ld, int T, int E, int k, const nfn_route_rule* rule, int* idx, float* weight, int* counts, nfn_stream_t stream) {
+  if (T <= 0) return 0;
+  if (!logits || !rule || !idx || !weight || !counts) return fail(-1, "moe_choose: null operand");
+  if (E <= 0 || E > MOE_MAX_E || k <= 0 || k > E || ld < E) return fail(-1, "moe_choose: need 1 <= k <= E <= 256, ld >= E");
+  if (rule->groups < 0 || (rule->groups > 0 && (E % rule->groups || rule->keep_groups < 1 || rule->keep_groups * (E / rule->groups) < k)))
+    return fail(-1, "moe_choose: the kept groups must hold the chosen experts");
+  moe_choose_kernel<<<(T + 7) / 8, 256, 0, static_cast<cudaStream_t>(stream)>>>(logits, ld, T, E, k, *rule, idx, weight, counts);
+  return launch_check("moe_choose", 1);
 }
 
 // offsets: E + 1 ints, cursor: E ints, tile_expert: max_tiles ints, plan: 2 ints.

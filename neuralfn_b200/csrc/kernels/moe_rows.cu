@@ -2,18 +2,19 @@
 // expert's items, then each chosen expert's weights are streamed once per group of items: on the tensor cores in bf16, a warp per
 // weight row in 32-bit mode. Also the gate of the sorted prompt rows (the grouped GEMMs around it are in gemm_tp.cu).
 //
-// The routing weight multiplies the expert's input. Gate and up are linear, so it is applied to their fp32 results instead:
-// act(w g) * (w u).
+// For gated experts the routing weight multiplies the input. Gate and up are linear, so it is applied to their fp32 results instead:
+// act(w g) * (w u). Plain experts, act(u), leave it to the pass that sums a token's items.
 #include <algorithm>
 
 #include "common.h"
+#include "moe_choice.cuh"
 #include "paged.cuh"
 
 namespace nfn {
 
 constexpr int MR_MAX_EXPERTS = 1024, MR_GROUP = 8, MR_WARPS = 8;
 
-// One CTA. Scores: sigmoid of the fp32 logits; the `top` largest per row (ties: the lower index). PER: logits per lane (experts <= 32 PER).
+// One CTA, a warp per row. PER: experts per lane (experts <= 32 PER).
 template <int PER>
 __global__ void __launch_bounds__(1024)
 moe_route_rows_kernel(const nfn_moe_rows_args p) {
@@ -22,30 +23,9 @@ moe_route_rows_kernel(const nfn_moe_rows_args p) {
   count[threadIdx.x] = 0;
   __syncthreads();
   for (int r = warp; r < p.rows; r += 32) {
-    const float* z = p.logits + (size_t)r * p.ld_logits;
-    float v[PER];
-#pragma unroll
-    for (int i = 0; i < PER; ++i) v[i] = lane + 32 * i < E ? z[lane + 32 * i] : -INFINITY;
-    uint32_t taken = 0;
-    for (int j = 0; j < p.top; ++j) {
-      float best = -INFINITY;
-      int bi = 0x7fffffff;
-#pragma unroll
-      for (int i = 0; i < PER; ++i)
-        if (lane + 32 * i < E && !((taken >> i) & 1u) && (bi == 0x7fffffff || v[i] > best)) { best = v[i]; bi = lane + 32 * i; }
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) {
-        const float ov = __shfl_xor_sync(0xffffffffu, best, o);
-        const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
-        if (oi != 0x7fffffff && (bi == 0x7fffffff || ov > best || (ov == best && oi < bi))) { best = ov; bi = oi; }
-      }
-      if ((bi & 31) == lane) taken |= 1u << (bi >> 5);
-      if (lane == 0) {
-        p.idx[(size_t)r * p.top + j] = bi;
-        p.weight[(size_t)r * p.top + j] = sigmoid_exact(best);
-        atomicAdd(&count[bi], 1);
-      }
-    }
+    int* idx = p.idx + (size_t)r * p.top;
+    choose_experts<PER>(p.logits + (size_t)r * p.ld_logits, E, p.top, p.rule, lane, idx, p.weight + (size_t)r * p.top);
+    for (int j = lane; j < p.top; j += 32) atomicAdd(&count[idx[j]], 1);       // this lane's own entries
   }
   __syncthreads();
   // first item of every expert, and the experts that have items
@@ -79,17 +59,21 @@ moe_route_rows_kernel(const nfn_moe_rows_args p) {
   for (int i = threadIdx.x; i < p.rows * p.top; i += 1024) p.order[atomicAdd(&start[p.idx[i]], 1)] = i;
 }
 
-// 32-bit mode. DOWN = false: mid[item][f] = act(w G_f h) * (w U_f h), h of the item's row. DOWN = true: y[item][n] = D_n mid[item].
-template <typename T, bool DOWN>
+// What a launch computes. kGateUp: mid[item][f] = act(w G_f h) * (w U_f h), h of the item's row; kDown: y[item][n] = D_n mid[item]; kUp: mid[item][f] = act(U_f h).
+enum { kGateUp = 0, kDown = 1, kUp = 2 };
+
+// 32-bit mode
+template <typename T, int FORM>
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_products_kernel(const nfn_moe_rows_args p) {
   if ((int)blockIdx.y >= p.active[p.experts]) return;
   const int e = p.active[blockIdx.y], warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  constexpr bool DOWN = FORM == kDown, TWO = FORM == kGateUp;
   const int n = blockIdx.x * MR_WARPS + warp, N = DOWN ? p.width : p.ff, K = DOWN ? p.ff : p.width;
   if (n >= N) return;
   const __nv_bfloat16* wa = DOWN ? static_cast<const __nv_bfloat16*>(p.w_down) + ((size_t)e * N + n) * K
-                                 : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * 2 * N + n) * K;
-  const __nv_bfloat16* wb = DOWN ? wa : wa + (size_t)N * K;
+                                 : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * (TWO ? 2 : 1) * N + n) * K;
+  const __nv_bfloat16* wb = TWO ? wa + (size_t)N * K : wa;
   const int i0 = p.offsets[e], i1 = p.offsets[e + 1];
   for (int g = i0; g < i1; g += MR_GROUP) {
     const int m = min(MR_GROUP, i1 - g);
@@ -110,7 +94,7 @@ moe_products_kernel(const nfn_moe_rows_args p) {
         const int k = k0 + u * 256;
         if (k < K) {
           load8(wa + k, va[u]);
-          if (!DOWN) load8(wb + k, vb[u]);
+          if (TWO) load8(wb + k, vb[u]);
         }
       }
 #pragma unroll
@@ -125,7 +109,7 @@ moe_products_kernel(const nfn_moe_rows_args p) {
 #pragma unroll
           for (int c = 0; c < 8; ++c) {
             a[i] += va[u][c] * x[c];
-            if (!DOWN) b[i] += vb[u][c] * x[c];
+            if (TWO) b[i] += vb[u][c] * x[c];
           }
         }
       }
@@ -136,12 +120,14 @@ moe_products_kernel(const nfn_moe_rows_args p) {
 #pragma unroll
       for (int o = 16; o > 0; o >>= 1) {
         a[i] += __shfl_xor_sync(0xffffffffu, a[i], o);
-        if (!DOWN) b[i] += __shfl_xor_sync(0xffffffffu, b[i], o);
+        if (TWO) b[i] += __shfl_xor_sync(0xffffffffu, b[i], o);
       }
       if (lane == 0) {
         const int item = p.order[g + i];
         if (DOWN) {
           static_cast<T*>(p.y)[(size_t)item * p.ld_y + n] = from_float<T>(a[i]);
+        } else if (!TWO) {
+          static_cast<T*>(p.mid)[(size_t)item * p.ff + n] = from_float<T>(ff_act(a[i], p.act));
         } else {
           const float w = p.weight[item];
           static_cast<T*>(p.mid)[(size_t)item * p.ff + n] = from_float<T>(ff_act(w * a[i], p.act) * (w * b[i]));
@@ -151,7 +137,7 @@ moe_products_kernel(const nfn_moe_rows_args p) {
   }
 }
 
-// The same on the tensor cores: a CTA takes 16 weight rows (DOWN: 32; else 16 of gate and the 16 of up beside them), its four warps a quarter
+// The same on the tensor cores: a CTA takes 32 weight rows (kGateUp: 16 of gate and the 16 of up beside them), its four warps a quarter
 // of the contraction each. Weight rows are the 16-row operand of mma.m16n8k16, items its eight columns; the order of the contraction is
 // free, so every fragment is one 16-byte load per lane. Weights are read once per 8 NT items.
 constexpr int MM_WARPS = 4;
@@ -167,21 +153,23 @@ __device__ __forceinline__ void mm_mma(float (&d)[4], uint32_t a0, uint32_t a1, 
       : "r"(a0), "r"(a1), "r"(a2), "r"(a3), "r"(b0), "r"(b1));
 }
 
-template <bool DOWN, int NT>
+template <int FORM, int NT>
 __global__ void __launch_bounds__(MM_WARPS * 32)
 moe_products_mma_kernel(const nfn_moe_rows_args p) {
+  constexpr bool DOWN = FORM == kDown, TWO = FORM == kGateUp;
+  constexpr int TILE = TWO ? 16 : 32;
   constexpr int M = 8 * NT;                               // items at a time
   constexpr int U = NT == 4 ? 2 : 4;                      // 32-channel steps in flight
   __shared__ float part[MM_WARPS][2][16][M + 1];
   if ((int)blockIdx.y >= p.active[p.experts]) return;
   const int e = p.active[blockIdx.y], warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
   const int N = DOWN ? p.width : p.ff, K = DOWN ? p.ff : p.width;
-  const int n0 = blockIdx.x * (DOWN ? 32 : 16);
+  const int n0 = blockIdx.x * TILE;
   // rows of the two 16-row tiles
-  const __nv_bfloat16* w0 = (DOWN ? static_cast<const __nv_bfloat16*>(p.w_down) + ((size_t)e * N + n0) * K : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * 2 * N + n0) * K) +
+  const __nv_bfloat16* w0 = (DOWN ? static_cast<const __nv_bfloat16*>(p.w_down) + ((size_t)e * N + n0) * K : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * (TWO ? 2 : 1) * N + n0) * K) +
                             (size_t)g * K + 8 * j;
-  const bool two = !DOWN || n0 + 16 < N;
-  const __nv_bfloat16* w1 = two ? w0 + (size_t)(DOWN ? 16 : N) * K : w0;
+  const bool two = TWO || n0 + 16 < N;
+  const __nv_bfloat16* w1 = two ? w0 + (size_t)(TWO ? N : 16) * K : w0;
   const int steps = (K + 31) / 32, s0 = steps * warp / MM_WARPS, s1 = steps * (warp + 1) / MM_WARPS;
   const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
   const int i0 = p.offsets[e], i1 = p.offsets[e + 1];
@@ -232,14 +220,15 @@ moe_products_mma_kernel(const nfn_moe_rows_args p) {
         for (int c = 0; c < 4; ++c) part[warp][m][g + (c >> 1) * 8][8 * t + 2 * j + (c & 1)] = acc[m][t][c];
     __syncthreads();
     const int live = min(M, i1 - i);
-    for (int x = threadIdx.x; x < (DOWN ? 32 : 16) * live; x += MM_WARPS * 32) {
-      const int col = x / (DOWN ? 32 : 16), row = x % (DOWN ? 32 : 16), item = p.order[i + col];
+    for (int x = threadIdx.x; x < TILE * live; x += MM_WARPS * 32) {
+      const int col = x / TILE, row = x % TILE, item = p.order[i + col];
       if (n0 + row >= N) continue;
-      if (DOWN) {
+      if (!TWO) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < MM_WARPS; ++w) v += part[w][row >> 4][row & 15][col];
-        static_cast<__nv_bfloat16*>(p.y)[(size_t)item * p.ld_y + n0 + row] = __float2bfloat16(v);
+        if (DOWN) static_cast<__nv_bfloat16*>(p.y)[(size_t)item * p.ld_y + n0 + row] = __float2bfloat16(v);
+        else static_cast<__nv_bfloat16*>(p.mid)[(size_t)item * p.ff + n0 + row] = __float2bfloat16(ff_act(v, p.act));
       } else {
         float gv = 0.f, uv = 0.f;
 #pragma unroll
@@ -272,8 +261,9 @@ moe_act_rows_kernel(const __nv_bfloat16* __restrict__ gate_up, const float* __re
 
 template <int NT>
 static void launch_products_mma(const nfn_moe_rows_args& a, int live, cudaStream_t st) {
-  moe_products_mma_kernel<false, NT><<<dim3(ceil_div(a.ff, 16), live), MM_WARPS * 32, 0, st>>>(a);
-  moe_products_mma_kernel<true, NT><<<dim3(ceil_div(a.width, 32), live), MM_WARPS * 32, 0, st>>>(a);
+  if (a.plain) moe_products_mma_kernel<kUp, NT><<<dim3(ceil_div(a.ff, 32), live), MM_WARPS * 32, 0, st>>>(a);
+  else moe_products_mma_kernel<kGateUp, NT><<<dim3(ceil_div(a.ff, 16), live), MM_WARPS * 32, 0, st>>>(a);
+  moe_products_mma_kernel<kDown, NT><<<dim3(ceil_div(a.width, 32), live), MM_WARPS * 32, 0, st>>>(a);
 }
 
 static int launch_moe_rows(const nfn_moe_rows_args& a, cudaStream_t st) {
@@ -282,8 +272,9 @@ static int launch_moe_rows(const nfn_moe_rows_args& a, cudaStream_t st) {
   else if (a.experts <= 256) moe_route_rows_kernel<8><<<1, 1024, 0, st>>>(a);
   else moe_route_rows_kernel<32><<<1, 1024, 0, st>>>(a);
   if (a.f32) {
-    moe_products_kernel<float, false><<<dim3(ceil_div(a.ff, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
-    moe_products_kernel<float, true><<<dim3(ceil_div(a.width, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
+    if (a.plain) moe_products_kernel<float, kUp><<<dim3(ceil_div(a.ff, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
+    else moe_products_kernel<float, kGateUp><<<dim3(ceil_div(a.ff, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
+    moe_products_kernel<float, kDown><<<dim3(ceil_div(a.width, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
   } else if (a.rows <= 8) {
     launch_products_mma<1>(a, live, st);
   } else if (a.rows <= 16) {
@@ -303,6 +294,8 @@ extern "C" int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream) 
   const nfn_moe_rows_args& a = *args;
   if (a.rows <= 0) return 0;
   if (a.experts < 1 || a.experts > MR_MAX_EXPERTS || a.top < 1 || a.top > a.experts) return fail(-1, "moe_rows: need 1 <= top <= experts <= 1024");
+  if (a.rule.groups < 0 || (a.rule.groups > 0 && (a.experts % a.rule.groups || a.rule.keep_groups < 1 || (long long)a.rule.keep_groups * (a.experts / a.rule.groups) < a.top)))
+    return fail(-1, "moe_rows: the kept groups must hold the chosen experts");
   if ((a.width | a.ff | a.ld_h) & 15) return fail(-1, "moe_rows: widths must be multiples of 16");
   if ((long long)a.rows * a.top > 0x7fffffffLL / 2) return fail(-1, "moe_rows: too many rows");
   return launch_moe_rows(a, static_cast<cudaStream_t>(stream));

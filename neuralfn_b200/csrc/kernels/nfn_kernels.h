@@ -341,9 +341,12 @@ typedef struct {
   int rows;                               // rows of the call
 } nfn_mix_args;
 int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream);
+// out[r] = act(gate) * up of rows [.. off_gate: gate .. off_up: up ..]; off_up < 0: out[r] = act(gate).
+int nfn_ff_rows(int f32, const void* in, int ld_in, int off_gate, int off_up, int ff, int act, void* out, int ld_out, int rows, nfn_stream_t stream);
 // Attention of a step's rows over the pages. score = q . k * scale, capped to softcap * tanh(score / softcap) (0: off), minus
-// slopes[h] * (i - j); keys 0 <= i - j < window (0: all) and the first keep_first ones of the sequence; softmax, with sink != 0 over
-// one more score of 0 that has no value; out = P V * sigmoid(gate) (gate optional). q: [rows, heads * dim_p]; out: row pitch ld_o, head pitch vdim_p.
+// slopes[h] * (i - j); keys 0 <= i - j < window (0: all) and the first keep_first ones of the sequence, with chunk > 0 only those of the query's own
+// chunk of that many positions; softmax, with sink != 0 over one more score of 0 that has no value; out = P V * sigmoid(gate) (gate optional).
+// q: [rows, heads * dim_p]; out: row pitch ld_o, head pitch vdim_p. v_pool = NULL: a key's value is its first vdim_p channels (latent caches).
 typedef struct {
   int f32;
   const void* q; int ld_q;
@@ -361,6 +364,7 @@ typedef struct {
   const int* tiles; int n_tiles;          // nfn_paged_attention_tiles: {row0, rows, slot, pos0} each
   int total_rows;                         // rows of the q buffer
   int keep_first; float softcap; int sink;
+  int chunk;
 } nfn_paged_attention_args;
 // One query row at a time (single tokens, very short portions): bf16 goes to the tensor cores in 32-key steps, fp32 and sizes
 // outside its limits to the plain kernel.
@@ -370,6 +374,60 @@ long long nfn_paged_attention_workspace_bytes(int rows, int heads, int vdim_p);
 // the sizes need nfn_paged_attention_rows.
 int nfn_paged_tile_rows(int f32, int heads, int kv_heads, int dim_p, int vdim_p);
 int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, nfn_stream_t stream);
+
+// ---- heads of a step's rows (head_rows.cu) ---------------------------------------------------------------------------------------
+// After the input projection of an attention layer: per head of dim values (pitch dim_p), RMS norm with a weight shared by the heads (NULL: none),
+// then rotation of the first rot_dims dimensions, pairs (2i, 2i + 1) by position * freq_i; freq: rot_dims / 2 pairs (high, low part of the
+// frequency). Queries [rows][heads] -> q_out, keys and values into their pages; off_v = off_k: the values are the keys as projected.
+typedef struct {
+  int f32;
+  const void* in; int ld_in, off_k, off_v;
+  int heads, kv_heads, dim, dim_p, vdim_p;         // kv_heads = 0: queries only
+  const void* q_norm; const void* k_norm; float eps;
+  const float* freq; int rot_dims;
+  void* q_out; int ld_q;
+  void* k_pool; void* v_pool;
+  const int* table; int table_ld;
+  const nfn_row_tile* tiles; int n_tiles, tile_rows;
+} nfn_head_rows_args;
+int nfn_head_rows(const nfn_head_rows_args* args, nfn_stream_t stream);
+// The same for latent attention. in: queries [heads][dim_p + rot_p] and, with k_pool, [rank_p latent | rot_p shared key part] at off_kv. The latent is
+// normed, the key part rotated, both go into the page [64][rank_p + rot_p]. Rotated query parts go to q_out ([heads][dim_p + rot_p], with
+// the unrotated ones) from row q_row0 on and to q_lat ([heads][rank_p + rot_p], at column rank_p) before it.
+typedef struct {
+  int f32;
+  const void* in; int ld_in, off_kv;
+  int heads, dim_p, rot_dim, rot_p, rank, rank_p;
+  const void* c_norm; float eps;
+  const float* freq;
+  void* q_out; int ld_q, q_row0;
+  void* q_lat;
+  void* k_pool;
+  const int* table; int table_ld;
+  const nfn_row_tile* tiles; int n_tiles, tile_rows;
+} nfn_latent_rows_args;
+int nfn_latent_rows(const nfn_latent_rows_args* args, nfn_stream_t stream);
+// out[r][g][n] = sum_k in[r][g][k] w[g][n][k]: one small product per group and row (the per-head projections around a latent cache, several inputs
+// with a matrix each). in, out: activation type, group pitches in elements; w bf16. Sizes are multiples of 16.
+typedef struct {
+  int f32, rows, groups, n, k;
+  const void* in; long long ld_in, in_group;
+  const void* w;
+  void* out; long long ld_out, out_group;
+} nfn_group_products_args;
+int nfn_group_products(const nfn_group_products_args* args, nfn_stream_t stream);
+
+// ---- latent attention over prompt portions (paged_prefill.cu, head_rows.cu) --------------------------------------------------------
+// A portion's visible latents, page by page, as rows of one matrix: page first_page + i of the slot to rows [row0 + 64 i, ...), i < n_pages.
+typedef struct { int slot, first_page, n_pages, row0; } nfn_latent_span;
+int nfn_latent_gather(int f32, const void* pool, int ld_pool, int cols, const int* table, int table_ld, const nfn_latent_span* spans, int n_spans,
+                      int max_pages, void* out, nfn_stream_t stream);
+// nfn_paged_attention_tiles with keys and values formed from the latents: x [x_rows][heads * dim_u unrotated keys | heads * vdim_p values], the rotated
+// key part (rot_p channels at column rank_p) still in the pages. args: dim_p = dim_u + rot_p, kv_heads = heads; tiles hold 128 rows;
+// x_base[slot]: row of x that belongs to position 0 of the sequence (may be negative).
+typedef struct { const void* x; int x_rows, dim_u, rot_p, rank_p; const int* x_base; } nfn_latent_expanded;
+int nfn_latent_tile_rows(int f32, int dim_u, int rot_p, int vdim_p);
+int nfn_latent_attention_tiles(const nfn_paged_attention_args* args, const nfn_latent_expanded* x, nfn_stream_t stream);
 // out = gelu_tanh(gate) * side_embed[token][col0 + c]: gate fp32 [rows, ld], out bf16 / fp32 with the same pitch.
 int nfn_side_mul(int f32, const float* gate, const int* tokens, const void* side_embed, long long ld_embed, int col0, int vocab, void* out,
                  int ld, int rows, int width, nfn_stream_t stream);
@@ -385,7 +443,9 @@ int nfn_logit_cap(float* logits, int ld, int rows, int cols, float scale, float 
 // all streams at once, x_t <- sum_s mix[s][t] x_s + out[t] y (mix, out: bf16; NULL: identity, ones; y = NULL: no update), then
 // u = sum_s in[s] x_s (in: bf16; NULL: ones) and h = u / rms(u) * (weight + weight_offset), rms(z) = sqrt(sum z^2 / width + eps).
 // The base is embed[token] * embed_scale in every stream (tokens != NULL) or row src_rows[r] (NULL: r) of x; y is the row of the
-// same number, or with y_rows > 1 the sum of rows y_index[r * y_rows + j] (y_index NULL: r * y_rows + j).
+// same number, or with y_rows > 1 the sum of rows y_index[r * y_rows + j] (y_index NULL: r * y_rows + j), each times y_item[r * y_rows + j]
+// (NULL: 1), plus row r of y_plus (NULL: none). With y_weight the update is normed first: y <- y_scale * y / rms(y) * y_weight.
+// weight = NULL: h = u.
 enum { NFN_MAX_STREAMS = 16 };
 typedef struct {
   int f32, rows, width, ld, streams;
@@ -395,6 +455,8 @@ typedef struct {
   const void* mix; const void* out;
   const void* in; void* h; const void* weight;
   float eps, weight_offset;
+  const float* y_item; const void* y_plus;
+  const void* y_weight; float y_scale;
 } nfn_stream_args;
 int nfn_stream_pass(const nfn_stream_args* args, nfn_stream_t stream);
 
@@ -440,11 +502,68 @@ typedef struct {
 int nfn_delta_step_fits(int rows, int heads, int dim_p, int vdim_p);
 int nfn_delta_step(const nfn_delta_step_args* args, nfn_stream_t stream);
 // out = o / rms(o) * weight * sigmoid(gate) per head of vdim values (pitch vdim_p); weight bf16 [vdim_p], out and gate in the activation type.
+// nfn_head_out: the same with weights per head (weight_pitch = vdim_p; 0: shared) and gate_act NFN_ACT_SILU (silu(gate)) or NFN_ACT_NONE (sigmoid).
+int nfn_head_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, int gate_act, const void* weight, int weight_pitch, float eps, void* out,
+                 int ld_out, int rows, int heads, int vdim, int vdim_p, nfn_stream_t stream);
 int nfn_delta_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, float eps, void* out, int ld_out, int rows,
                   int heads, int vdim, int vdim_p, nfn_stream_t stream);
 
+// ---- token shift and the bonus recurrence (wkv_rows.cu, wkv_chunk.cu) --------------------------------------------------------------------
+// out[s][r] = h + (h' - h) * mu[s], s < n: h the row, h' the previous token's (the row before it in its entry, the stored one of the slot, zero at
+// position 0). src fp32 or, with src_act, in the activation type; prev fp32 [2][slots][ld], the half named by the tile's parity is read, the other written.
+typedef struct {
+  int f32, src_act, width, ld, n;
+  const void* src;
+  const void* mu;                         // bf16 [n][ld]
+  float* prev; long long prev_half;
+  void* out; long long out_stride;        // elements between the outputs; row pitch ld
+  const nfn_row_tile* tiles; int n_tiles;
+} nfn_shift_args;
+int nfn_shift_rows(const nfn_shift_args* args, nfn_stream_t stream);
+// Per head, with the fp32 state S [dim][dim] of the sequence: o = S^T r + (r . (u k)) v;  S <- w S + k v^T,  w = exp(-exp(z + w0)) per key channel.
+// rkv: rows [r | k | v] of heads * dim_p each; z fp32 [rows][heads * dim_p]; u, w0 bf16 [heads * dim_p]; state [slots][heads][dim_p][dim_p]; a sequence at
+// position 0 starts from zero. o: fp32 rows. Padded channels are zero in r, k, v.
+typedef struct {
+  int f32;
+  const void* rkv; int ld_rkv;
+  const float* z; int ld_z;
+  const void* w0; const void* u;
+  int heads, dim, dim_p;
+  float* state;
+  float* o; int ld_o;
+  const nfn_seq_rows* seqs; int n_seqs;
+} nfn_wkv_args;
+int nfn_wkv_rows(const nfn_wkv_args* args, nfn_stream_t stream);         // token after token, any length
+long long nfn_wkv_chunk_workspace_bytes(int heads, int dim_p, int max_seqs);   // 0: these sizes go token after token
+int nfn_wkv_chunks(const nfn_wkv_args* args, int max_rows, void* workspace, long long workspace_bytes, nfn_stream_t stream);
+// tanh of the inner decay projection, ready for the outer product: fp32 in; out in the activation type, [rows][2 * rank_p] = rounded value | what rounding
+// left out in bf16, [rows][rank_p] in 32-bit mode.
+int nfn_tanh_split(int f32, const float* in, int ld_in, void* out, int ld_out, int rows, int rank_p, nfn_stream_t stream);
+// One token of every sequence: decay (with its outer projection w2 [heads * dim_p][ld_w2], low fp32 [rows][rank_p] before the tanh), rule, output norm, gate.
+// rkvg: rows [r | k | v | g]; tiles: one per row. nfn_wkv_step_fits: the sizes and row counts it takes.
+typedef struct {
+  int f32, rows;
+  const void* rkvg; int ld_rkvg;
+  const float* low; int ld_low, rank_p;
+  const void* w2; int ld_w2;
+  const void* w0; const void* u;
+  int heads, dim, dim_p;
+  float* state;
+  const void* weight; float eps;
+  void* out; int ld_out;
+  const nfn_row_tile* tiles;
+} nfn_wkv_step_args;
+int nfn_wkv_step_fits(int rows, int heads, int dim_p);
+int nfn_wkv_step(const nfn_wkv_step_args* args, nfn_stream_t stream);
+
 // ---- mixture of experts for the rows of a step (moe.cu, moe_rows.cu) ----------------------------------------------------------
-// item i = token i / top, choice i % top. The routing weight multiplies the expert's INPUT: mid = act(w G h) * (w U h).
+// item i = token i / top, choice i % top. Gated experts take the routing weight at their INPUT: mid = act(w G h) * (w U h); plain ones (w_gate_up
+// [E][ff][width]) compute mid = act(U h) and leave the weight to whoever sums the items.
+// nfn_route_rule: how experts are chosen and weighted. Scores s = sigmoid(logits); choice scores s + correction (bf16, NULL: none); with groups > 0
+// (equal groups of neighbours) a group counts by the sum of its two largest choice scores and only experts of the best keep_groups can be chosen;
+// weights s, with normalise / (sum of the chosen ones + 1e-20), times scale. Ties: the lower index.
+typedef struct { const void* correction; int groups, keep_groups, normalise; float scale; } nfn_route_rule;
+int nfn_moe_choose(const float* logits, int ld, int T, int E, int k, const nfn_route_rule* rule, int* idx, float* weight, int* counts, nfn_stream_t stream);
 int nfn_moe_route(const float* logits, int ld, int T, int E, int k, int score_fn, int norm_topk, float route_scale, int* topk_idx, float* topk_w,
                   int* counts, nfn_stream_t stream);
 int nfn_moe_plan(const int* counts, int E, int max_tiles, int* offsets, int* cursor, int* tile_expert, int* plan, nfn_stream_t stream);
@@ -463,6 +582,8 @@ typedef struct {
   int* idx; float* weight; int* order; int* offsets; int* active;
   void* mid;                              // [rows * top][ff]
   void* y; int ld_y;                      // [rows * top][ld_y]
+  int plain;
+  nfn_route_rule rule;                    // scale 0 counts as 1
 } nfn_moe_rows_args;
 int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream);
 

@@ -8,6 +8,12 @@ namespace nfn {
 constexpr int NFN_PAGE = 64;   // tokens per cache page
 constexpr int PAGED_COUNTER_BYTES = 64 * 1024;
 
+// the oldest key a query sees, apart from kept first tokens
+__device__ __forceinline__ int first_visible(const nfn_paged_attention_args& a, int pos) {
+  if (a.chunk > 0) return pos / a.chunk * a.chunk;
+  return a.window > 0 ? max(0, pos - a.window + 1) : 0;
+}
+
 template <typename T>
 __device__ __forceinline__ T from_float(float v);
 template <>
@@ -66,6 +72,7 @@ __device__ __forceinline__ float ff_act(float v, int act) {
   if (act == NFN_ACT_RELU) return fmaxf(v, 0.f);
   if (act == NFN_ACT_SILU) return v / (1.f + expf(-v));
   if (act == NFN_ACT_GELU_TANH) return gelu_tanh_exact(v);
+  if (act == NFN_ACT_RELU2) return fmaxf(v, 0.f) * fmaxf(v, 0.f);
   return v;
 }
 // by activation type: exact in 32-bit mode; for results that are rounded to bf16 the exponential and reciprocal units (a few ulp of fp32)

@@ -18,6 +18,7 @@
 namespace nfn {
 
 int paged_attention_plain(const nfn_paged_attention_args& a, cudaStream_t st);  // paged_rows.cu
+int latent_decode(const nfn_paged_attention_args& a, cudaStream_t st);           // latent_decode.cu; 1: sizes outside its limits
 
 constexpr int PD_WARPS = 4, PD_THREADS = PD_WARPS * 32, PD_KEYS = 32;
 constexpr int PD_COUNTERS = PAGED_COUNTER_BYTES / 4;
@@ -59,7 +60,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
   const int hk = blockIdx.y / p.head_blocks, hb = blockIdx.y % p.head_blocks;
   const int hg = a.heads / a.kv_heads, h_lo = hb * NH, n_heads = min(NH, hg - h_lo), h0 = hk * hg + h_lo;
   const int pos = a.row_pos[row];
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = first_visible(a, pos);
   // chunks in the order kept tokens, window: number i of them is chunk i of the sequence, or c_first + i - n_keep
   const int keep = min(a.keep_first, pos + 1);
   const int c_first = lo / PD_KEYS, n_keep = min(c_first, (keep + PD_KEYS - 1) / PD_KEYS), n_chunks = n_keep + pos / PD_KEYS + 1 - c_first;
@@ -350,6 +351,11 @@ extern "C" int nfn_paged_attention_rows(const nfn_paged_attention_args* args, nf
   if (a.kv_heads <= 0 || a.heads % a.kv_heads) return fail(-1, "paged attention: query heads must divide into key / value heads");
   if ((a.dim_p | a.vdim_p | a.ld_q) & 15) return fail(-1, "paged attention: head sizes and the query pitch must be multiples of 16");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (!a.v_pool) {
+    if (a.kv_heads != 1 || a.vdim_p > a.dim_p) return fail(-1, "paged attention: values out of the keys need one key head at least as wide");
+    const int rc = a.f32 || !a.workspace ? 1 : latent_decode(a, st);
+    return rc == 1 ? paged_attention_plain(a, st) : rc;
+  }
   if (a.f32 || a.dim_p > 256 || a.vdim_p > 256 || !a.workspace) return paged_attention_plain(a, st);
   if (a.dim_p > 128 || a.vdim_p > 128) return launch_paged_decode<8, 16, 1>(a, st);
   return a.heads / a.kv_heads > 8 ? launch_paged_decode<4, 8, 2>(a, st) : launch_paged_decode<4, 8, 1>(a, st);

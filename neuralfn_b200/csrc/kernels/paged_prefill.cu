@@ -9,6 +9,10 @@
 // row maximum grew by more than 2^8. Pages are visited from the newest to the oldest: under a distance bias the maximum then
 // settles in the first page instead of growing with every one.
 //
+// Latent attention (EXPANDED): every head's unrotated keys and its values were formed from the cached latents as rows of one matrix, 64 rows per
+// page; the rotated key part, shared by the heads, still comes from the pages as further panels of the same score product. Values then
+// are [64 tokens][64 channels] panels, an MN-major operand.
+//
 // Head sizes are run-time values (multiples of 16 up to 256; channels past a head's end are zero-filled by TMA). The distance
 // bias and the window are applied to the fp32 scores in registers; the output gate is applied on the way out.
 #include "attention_v2.cuh"
@@ -21,13 +25,17 @@ constexpr int PP_BM = 128, PP_BN = NFN_PAGE;
 struct PagedPrefillParams {
   nfn_paged_attention_args a;
   int hg, nq;                 // query heads per key / value head, query rows per tile
-  int panels;                 // 64-channel panels of a query / key head
+  int panels;                 // 64-channel panels of a query / key head (EXPANDED: of its unrotated part)
+  nfn_latent_expanded x;      // EXPANDED
+  int panels_r, panels_v;     // panels of the rotated part, of a value head
   uint32_t q_bytes, k_bytes, v_bytes, q_tx;
   uint32_t o_col, tmem_cols;
   uint32_t smem;
   int* status;
 };
 
+// tm_k, tm_v: the pages (EXPANDED: the pages for the rotated key part, the matrix of unrotated keys and values)
+template <bool EXPANDED>
 __global__ void __launch_bounds__(AV2_THREADS, 2)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                      const __grid_constant__ CUtensorMap tm_v, const PagedPrefillParams p) {
@@ -64,7 +72,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   const int row0 = tile.x, n_rows = tile.y, slot = tile.z, pos0 = tile.w;
   const int hk = blockIdx.y;
   const int* table = a.table + (size_t)slot * a.table_ld;
-  const int k_lo = a.window > 0 ? max(0, pos0 - a.window + 1) : 0;
+  const int k_lo = first_visible(a, pos0);
   // visited from the newest page back to the window's edge, then the pages of the kept first tokens that lie before it
   const int jb_hi = (pos0 + n_rows - 1) / PP_BN, n_win = jb_hi + 1 - k_lo / PP_BN;
   const int n_keep = min(k_lo / PP_BN, (a.keep_first + PP_BN - 1) / PP_BN), nblk = n_win + n_keep;
@@ -97,20 +105,37 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
   if (warp == AV2_TMA_WARP) {
     // ------------------------------------------------------------ TMA producer --
     if (lane == 0) {
+      const int x_base = EXPANDED ? p.x.x_base[slot] : 0;
       auto load_k = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_k[stage]);
         const uint32_t sk = smem_u32(sKV + stage * kv_stage);
-        const int r = (table[page_at(j)] * a.kv_heads + hk) * PP_BN;
         mbar_expect_tx(fb, p.k_bytes);
-        for (int d = 0; d < p.panels; ++d) tma_load_2d(sk + d * (PP_BN * 128), &tm_k, fb, d * 64, r);
+        if (EXPANDED) {
+          const int r = x_base + page_at(j) * PP_BN;
+          for (int d = 0; d < p.panels; ++d) tma_load_2d(sk + d * (PP_BN * 128), &tm_v, fb, hk * p.x.dim_u + d * 64, r);
+          for (int d = 0; d < p.panels_r; ++d)
+            tma_load_2d(sk + (p.panels + d) * (PP_BN * 128), &tm_k, fb, p.x.rank_p + d * 64, table[page_at(j)] * PP_BN);
+        } else {
+          const int r = (table[page_at(j)] * a.kv_heads + hk) * PP_BN;
+          for (int d = 0; d < p.panels; ++d) tma_load_2d(sk + d * (PP_BN * 128), &tm_k, fb, d * 64, r);
+        }
       };
       auto load_v = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_v[stage]);
+        const uint32_t sv = smem_u32(sKV + stage * kv_stage + p.k_bytes);
         mbar_expect_tx(fb, p.v_bytes);
-        tma_load_2d(smem_u32(sKV + stage * kv_stage + p.k_bytes), &tm_v, fb, 0, (table[page_at(j)] * a.kv_heads + hk) * a.vdim_p);
+        if (EXPANDED) {
+          for (int d = 0; d < p.panels_v; ++d)
+            tma_load_2d(sv + d * (PP_BN * 128), &tm_v, fb, a.heads * p.x.dim_u + hk * a.vdim_p + d * 64, x_base + page_at(j) * PP_BN);
+        } else {
+          tma_load_2d(sv, &tm_v, fb, 0, (table[page_at(j)] * a.kv_heads + hk) * a.vdim_p);
+        }
       };
       mbar_expect_tx(smem_u32(bar_q), p.q_tx);
       for (int d = 0; d < p.panels; ++d) tma_load_3d(smem_u32(sQ) + d * (PP_BM * 128), &tm_q, smem_u32(bar_q), d * 64, hk * p.hg, row0);
+      if (EXPANDED)
+        for (int d = 0; d < p.panels_r; ++d)
+          tma_load_3d(smem_u32(sQ) + (p.panels + d) * (PP_BM * 128), &tm_q, smem_u32(bar_q), p.x.dim_u + d * 64, hk, row0);
       load_k(0, 0);
       load_v(0, 0);
       if (nblk > 1) { load_k(1, 1); load_v(1, 1); }
@@ -125,8 +150,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     // -------------------------------------------------------------- MMA issuer --
     if (lane == 0) {
       const uint32_t idesc_s = make_idesc_bf16(PP_BM, PP_BN, 0, 0);
-      const uint32_t idesc_o = make_idesc_bf16(PP_BM, a.vdim_p, 0, 0);
-      const int k_steps = a.dim_p / 16;
+      const uint32_t idesc_o = EXPANDED ? make_idesc_bf16(PP_BM, p.panels_v * 64, 0, 1) : make_idesc_bf16(PP_BM, a.vdim_p, 0, 0);   // whole panels
+      const int k_steps = (EXPANDED ? p.x.dim_u : a.dim_p) / 16;
       auto issue_s = [&](int stage) {
         const uint32_t sq = smem_u32(sQ);
         const uint32_t sk = smem_u32(sKV + stage * kv_stage);
@@ -135,6 +160,14 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           const uint32_t a_off = (kk / 4) * (PP_BM * 128) + (kk % 4) * 32;
           const uint32_t b_off = (kk / 4) * (PP_BN * 128) + (kk % 4) * 32;
           umma_bf16_ss(tmem_base, make_smem_desc_sw128(sq + a_off, 16, 1024), make_smem_desc_sw128(sk + b_off, 16, 1024), idesc_s, kk != 0);
+        }
+        if (EXPANDED) {
+          const uint32_t sqr = sq + p.panels * (PP_BM * 128), skr = sk + p.panels * (PP_BN * 128);
+          for (int kk = 0; kk < p.x.rot_p / 16; ++kk) {
+            const uint32_t a_off = (kk / 4) * (PP_BM * 128) + (kk % 4) * 32;
+            const uint32_t b_off = (kk / 4) * (PP_BN * 128) + (kk % 4) * 32;
+            umma_bf16_ss(tmem_base, make_smem_desc_sw128(sqr + a_off, 16, 1024), make_smem_desc_sw128(skr + b_off, 16, 1024), idesc_s, 1);
+          }
         }
         umma_commit(smem_u32(bar_s));
         umma_commit(smem_u32(&bar_kfree[stage]));
@@ -159,8 +192,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         const uint32_t sv = smem_u32(sKV + (j & 1) * kv_stage + p.k_bytes);
 #pragma unroll
         for (int kk = 0; kk < PP_BN / 16; ++kk)
-          umma_bf16_ss(tmem_base + p.o_col, make_smem_desc_sw128(sp + kk * 32, 16, 1024), make_smem_desc_sw128(sv + kk * 32, 16, 1024), idesc_o,
-                       (j | kk) != 0);
+          umma_bf16_ss(tmem_base + p.o_col, make_smem_desc_sw128(sp + kk * 32, 16, 1024),
+                       EXPANDED ? make_smem_desc_sw128(sv + kk * (16 * 128), PP_BN * 128, 1024) : make_smem_desc_sw128(sv + kk * 32, 16, 1024), idesc_o, (j | kk) != 0);
         umma_commit(smem_u32(bar_o));
         umma_commit(smem_u32(&bar_vfree[j & 1]));
       }
@@ -181,8 +214,8 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     const float slope = (a.slopes && row_ok) ? a.slopes[h] * LOG2E : 0.f;
     // visible keys of this row: [v_lo, v_hi)
     const int v_hi = row_ok ? pos + 1 : 0;
-    const int v_lo = (row_ok && a.window > 0) ? max(0, pos - a.window + 1) : 0;
-    const int pos_last = pos0 + n_rows - 1;
+    const int v_lo = row_ok ? first_visible(a, pos) : 0;
+    const int lo_last = first_visible(a, pos0 + n_rows - 1);
     const int v_keep = min(a.keep_first, v_hi);
     float m_run = a.sink ? 0.f : -INFINITY, l_run = a.sink ? 1.f : 0.f;  // units of log2; the sink counts as seen before all keys
     bool ok = true;
@@ -240,7 +273,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         s[i] = __float_as_uint(y0);
         s[i + 1] = __float_as_uint(y1);
       }
-      if (kbase + PP_BN - 1 > pos0 || (a.window > 0 && kbase <= pos_last - a.window)) {
+      if (kbase + PP_BN - 1 > pos0 || kbase < lo_last) {
         const int lo_rel = v_lo - kbase, keep_rel = v_keep - kbase;
         const unsigned span = (unsigned)max(0, v_hi - v_lo);
 #pragma unroll
@@ -372,23 +405,41 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
 
 using namespace nfn;
 
-// shared memory of a tile for these head sizes; the limit is what one CTA may have
-static uint32_t paged_tile_smem(int dim_p, int vdim_p) {
-  const uint32_t panels = (dim_p + 63) / 64;
-  return panels * PP_BM * 128 + 2 * (panels * PP_BN * 128 + vdim_p * 128) + PP_BM * PP_BN * 2 + 128;
+// shared memory of a tile with this many panels and bytes of values per page; the limit is what one CTA may have
+static uint32_t paged_tile_smem(uint32_t panels, uint32_t v_bytes) {
+  return panels * PP_BM * 128 + 2 * (panels * PP_BN * 128 + v_bytes) + PP_BM * PP_BN * 2 + 128;
 }
 
 extern "C" int nfn_paged_tile_rows(int f32, int heads, int kv_heads, int dim_p, int vdim_p) {
   const int hg = heads / kv_heads;
-  if (f32 || dim_p > 256 || vdim_p > 256 || hg > PP_BM || paged_tile_smem(dim_p, vdim_p) > 227 * 1024) return 0;
+  if (f32 || dim_p > 256 || vdim_p > 256 || hg > PP_BM || paged_tile_smem((dim_p + 63) / 64, vdim_p * 128) > 226 * 1024) return 0;
   return PP_BM / hg;
+}
+
+template <bool EXPANDED>
+static int launch_paged_prefill(PagedPrefillParams& p, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, cudaStream_t st) {
+  const nfn_paged_attention_args& a = p.a;
+  p.o_col = PP_BN;
+  const int cols = PP_BN + (EXPANDED ? p.panels_v * 64 : a.vdim_p);
+  p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;
+  p.status = status_ptr();
+  auto kern = paged_prefill_kernel<EXPANDED>;
+  static uint32_t raised[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (raised[dev & 63] < p.smem) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)p.smem) != cudaSuccess) return launch_check("paged_prefill attr", 0);
+    raised[dev & 63] = p.smem;
+  }
+  kern<<<dim3(a.n_tiles, a.kv_heads), AV2_THREADS, p.smem, st>>>(tq, tk, tv, p);
+  return launch_check("paged_prefill");
 }
 
 extern "C" int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, nfn_stream_t stream) {
   if (!args) return fail(-1, "paged attention: null args");
   const nfn_paged_attention_args& a = *args;
   if (a.n_tiles <= 0) return 0;
-  PagedPrefillParams p;
+  PagedPrefillParams p{};
   p.a = a;
   p.nq = nfn_paged_tile_rows(a.f32, a.heads, a.kv_heads, a.dim_p, a.vdim_p);
   if (p.nq <= 0) return fail(-1, "paged attention: these head sizes run one row at a time");
@@ -400,23 +451,47 @@ extern "C" int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, n
   // the value stage keeps the next key stage on a 1024-byte boundary
   p.v_bytes = a.vdim_p * 128;
   p.q_tx = p.panels * p.nq * p.hg * 128;
-  p.o_col = PP_BN;
-  p.tmem_cols = PP_BN + a.vdim_p <= 128 ? 128 : PP_BN + a.vdim_p <= 256 ? 256 : 512;
-  p.smem = paged_tile_smem(a.dim_p, a.vdim_p);
-  p.status = status_ptr();
+  p.smem = paged_tile_smem(p.panels, p.v_bytes);
   CUtensorMap tq, tk, tv;
   if (!make_tmap_3d(&tq, a.q, 2, a.dim_p, a.heads, a.total_rows, a.dim_p, a.ld_q, 64, p.hg, p.nq, 128)) return -3;
   const uint64_t cells = (uint64_t)a.pages * a.kv_heads;
   if (!make_tmap_2d(&tk, a.k_pool, 2, a.dim_p, cells * NFN_PAGE, a.dim_p, 64, PP_BN, 128)) return -3;
   if (!make_tmap_2d(&tv, a.v_pool, 2, NFN_PAGE, cells * a.vdim_p, NFN_PAGE, NFN_PAGE, a.vdim_p, 128)) return -3;
-  static uint32_t raised[64] = {};
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (raised[dev & 63] < p.smem) {
-    if (cudaFuncSetAttribute(paged_prefill_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)p.smem) != cudaSuccess)
-      return launch_check("paged_prefill attr", 0);
-    raised[dev & 63] = p.smem;
-  }
-  paged_prefill_kernel<<<dim3(a.n_tiles, a.kv_heads), AV2_THREADS, p.smem, static_cast<cudaStream_t>(stream)>>>(tq, tk, tv, p);
-  return launch_check("paged_prefill");
+  return launch_paged_prefill<false>(p, tq, tk, tv, static_cast<cudaStream_t>(stream));
+}
+
+static uint32_t latent_tile_smem(int dim_u, int rot_p, int vdim_p) {
+  return paged_tile_smem((dim_u + 63) / 64 + (rot_p + 63) / 64, (vdim_p + 63) / 64 * PP_BN * 128);
+}
+
+extern "C" int nfn_latent_tile_rows(int f32, int dim_u, int rot_p, int vdim_p) {
+  return f32 || vdim_p > 256 || latent_tile_smem(dim_u, rot_p, vdim_p) > 226 * 1024 ? 0 : PP_BM;
+}
+
+extern "C" int nfn_latent_attention_tiles(const nfn_paged_attention_args* args, const nfn_latent_expanded* x, nfn_stream_t stream) {
+  if (!args || !x) return fail(-1, "latent attention: null args");
+  const nfn_paged_attention_args& a = *args;
+  if (a.n_tiles <= 0) return 0;
+  if (nfn_latent_tile_rows(a.f32, x->dim_u, x->rot_p, a.vdim_p) <= 0) return fail(-1, "latent attention: these head sizes run one row at a time");
+  if (a.kv_heads != a.heads || a.dim_p != x->dim_u + x->rot_p || a.keep_first > 0) return fail(-1, "latent attention: every head has expanded keys and values of its own");
+  if ((x->dim_u | x->rot_p | x->rank_p | a.vdim_p | a.ld_q | a.ld_o) & 15 || (a.gate && (a.ld_gate & 7))) return fail(-1, "latent attention: head sizes and row pitches must be multiples of 16");
+  PagedPrefillParams p{};
+  p.a = a;
+  p.x = *x;
+  p.nq = PP_BM;
+  p.hg = 1;
+  p.panels = (x->dim_u + 63) / 64;
+  p.panels_r = (x->rot_p + 63) / 64;
+  p.panels_v = (a.vdim_p + 63) / 64;
+  const int panels = p.panels + p.panels_r;
+  p.q_bytes = p.q_tx = panels * PP_BM * 128;
+  p.k_bytes = panels * PP_BN * 128;
+  p.v_bytes = p.panels_v * PP_BN * 128;
+  p.smem = latent_tile_smem(x->dim_u, x->rot_p, a.vdim_p);
+  const int lp = x->rank_p + x->rot_p, cols = a.heads * (x->dim_u + a.vdim_p);
+  CUtensorMap tq, tk, tx;
+  if (!make_tmap_3d(&tq, a.q, 2, a.dim_p, a.heads, a.total_rows, a.dim_p, a.ld_q, 64, 1, PP_BM, 128)) return -3;
+  if (!make_tmap_2d(&tk, a.k_pool, 2, lp, (uint64_t)a.pages * NFN_PAGE, lp, 64, PP_BN, 128)) return -3;
+  if (!make_tmap_2d(&tx, x->x, 2, cols, x->x_rows, cols, 64, PP_BN, 128)) return -3;
+  return launch_paged_prefill<true>(p, tq, tk, tx, static_cast<cudaStream_t>(stream));
 }

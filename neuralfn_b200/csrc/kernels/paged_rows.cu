@@ -280,29 +280,35 @@ mix_rows_kernel(const nfn_mix_args p) {
   leave();
 }
 
-// ff_out = act(gate) * up over all rows of a call: two rows per thread, few registers
+// out = act(gate) * up over all rows of a call: two rows per thread, few registers. off_up < 0: out = act(gate)
 template <typename T>
 __global__ void __launch_bounds__(256)
-ff_rows_kernel(const nfn_mix_args p) {
+ff_rows_kernel(const T* __restrict__ src, int ld_in, int off_gate, int off_up, int ff, int act, T* __restrict__ dst, int ld_out, int rows) {
   const int c = (blockIdx.x * 256 + threadIdx.x) * 8, r0 = blockIdx.y * 2;
-  if (c >= p.ff) return;
-  const T* in = static_cast<const T*>(p.in) + (size_t)r0 * p.ld_in + c;
-  T* out = static_cast<T*>(p.ff_out) + (size_t)r0 * p.ld_ff + c;
-  const bool two = r0 + 1 < p.rows;
+  if (c >= ff) return;
+  const T* in = src + (size_t)r0 * ld_in + c;
+  T* out = dst + (size_t)r0 * ld_out + c;
+  const bool two = r0 + 1 < rows, up = off_up >= 0;
   float g[2][8], u[2][8];
 #pragma unroll
   for (int i = 0; i < 2; ++i)
     if (i == 0 || two) {
-      load8(in + (size_t)i * p.ld_in + p.off_gate, g[i]);
-      load8(in + (size_t)i * p.ld_in + p.off_up, u[i]);
+      load8(in + (size_t)i * ld_in + off_gate, g[i]);
+      if (up) load8(in + (size_t)i * ld_in + off_up, u[i]);
     }
 #pragma unroll
   for (int i = 0; i < 2; ++i)
     if (i == 0 || two) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) g[i][e] = ff_act(g[i][e], p.act) * u[i][e];
-      store8(out + (size_t)i * p.ld_ff, g[i]);
+      for (int e = 0; e < 8; ++e) g[i][e] = ff_act(g[i][e], act) * (up ? u[i][e] : 1.f);
+      store8(out + (size_t)i * ld_out, g[i]);
     }
+}
+
+template <typename T>
+static void launch_ff_rows(const void* in, int ld_in, int off_gate, int off_up, int ff, int act, void* out, int ld_out, int rows, cudaStream_t st) {
+  ff_rows_kernel<T><<<dim3(ceil_div(ff, 256 * 8), ceil_div(rows, 2)), 256, 0, st>>>(static_cast<const T*>(in), ld_in, off_gate, off_up, ff, act, static_cast<T*>(out),
+                                                                                    ld_out, rows);
 }
 
 template <typename T>
@@ -318,7 +324,7 @@ static void launch_mix_rows(const nfn_mix_args& a, const dim3& grid, cudaStream_
 // --------------------------------------------------------------------------------- plain paged attention --
 // One warp per (row, query head): 32 keys at a time, one per lane, running maximum and sum, the value sum over channels held
 // lane-wise. Any size; 32-bit throughout. The yardstick of the tensor-core kernels and the only path in 32-bit mode.
-constexpr int PLAIN_WARPS = 4, PLAIN_MAX_VEC = 16;   // values up to 32 * 16 channels per head
+constexpr int PLAIN_WARPS = 4, PLAIN_MAX_VEC = 16;   // 32 * 16 value channels of a head per CTA
 
 template <typename T>
 __global__ void __launch_bounds__(PLAIN_WARPS * 32)
@@ -337,10 +343,11 @@ paged_attention_plain_kernel(const nfn_paged_attention_args p) {
   for (int d = lane; d < p.dim_p; d += 32) q[d] = to_float(static_cast<const T*>(p.q)[(size_t)row * p.ld_q + h * p.dim_p + d]);
   __syncwarp();
   const float slope = p.slopes ? p.slopes[h] : 0.f;
-  const int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
+  const int lo = first_visible(p, pos);
   const int keep = min(p.keep_first, pos + 1);
   const int* table = p.table + (size_t)slot * p.table_ld;
-  const int nvec = (p.vdim_p + 31) / 32;
+  const int v0 = blockIdx.z * 32 * PLAIN_MAX_VEC, v_n = min(p.vdim_p - v0, 32 * PLAIN_MAX_VEC);      // this CTA's value channels
+  const int nvec = (v_n + 31) / 32;
   float acc[PLAIN_MAX_VEC];
 #pragma unroll
   for (int i = 0; i < PLAIN_MAX_VEC; ++i) acc[i] = 0.f;
@@ -374,12 +381,28 @@ paged_attention_plain_kernel(const nfn_paged_attention_args p) {
     m = m_new;
     wgt[lane] = e;
     __syncwarp();
-    const T* v = static_cast<const T*>(p.v_pool) + tile * p.vdim_p * NFN_PAGE + in_page;
+    if (!p.v_pool) {                                     // values are the keys' first channels
+      const int live = min(32, pos - base + 1);
+      const T* v = static_cast<const T*>(p.k_pool) + (tile * NFN_PAGE + in_page) * p.dim_p + v0;
+#pragma unroll
+      for (int i = 0; i < PLAIN_MAX_VEC; ++i) {
+        if (i >= nvec) break;
+        const int c = lane + 32 * i;
+        if (c < v_n) {
+          float t = 0.f;
+          for (int k = 0; k < live; ++k) t += to_float(v[(size_t)k * p.dim_p + c]) * wgt[k];
+          acc[i] = acc[i] * alpha + t;
+        }
+      }
+      __syncwarp();
+      continue;
+    }
+    const T* v = static_cast<const T*>(p.v_pool) + (tile * p.vdim_p + v0) * NFN_PAGE + in_page;
 #pragma unroll
     for (int i = 0; i < PLAIN_MAX_VEC; ++i) {
       if (i >= nvec) break;
       const int c = lane + 32 * i;
-      if (c < p.vdim_p) {
+      if (c < v_n) {
         const T* vc = v + (size_t)c * NFN_PAGE;
         float t = 0.f;
         for (int k = 0; k < 32; k += 4) {
@@ -396,19 +419,18 @@ paged_attention_plain_kernel(const nfn_paged_attention_args p) {
   for (int i = 0; i < PLAIN_MAX_VEC; ++i) {
     if (i >= nvec) break;
     const int c = lane + 32 * i;
-    if (c < p.vdim_p) {
+    if (c < v_n) {
       float o = acc[i] * inv;
-      if (p.gate) o *= sigmoid_exact(to_float(static_cast<const T*>(p.gate)[(size_t)row * p.ld_gate + h * p.vdim_p + c]));
-      static_cast<T*>(p.out)[(size_t)row * p.ld_o + h * p.vdim_p + c] = from_float<T>(o);
+      if (p.gate) o *= sigmoid_exact(to_float(static_cast<const T*>(p.gate)[(size_t)row * p.ld_gate + h * p.vdim_p + v0 + c]));
+      static_cast<T*>(p.out)[(size_t)row * p.ld_o + h * p.vdim_p + v0 + c] = from_float<T>(o);
     }
   }
 }
 
 int paged_attention_plain(const nfn_paged_attention_args& a, cudaStream_t st) {
-  if (a.vdim_p > 32 * PLAIN_MAX_VEC) return fail(-1, "paged attention: more than 512 value channels per head");
   const size_t smem = (size_t)PLAIN_WARPS * (a.dim_p + 32) * sizeof(float);
   if (smem > 48 * 1024) return fail(-1, "paged attention: query head too wide");
-  const dim3 grid(a.rows, ceil_div(a.heads, PLAIN_WARPS));
+  const dim3 grid(a.rows, ceil_div(a.heads, PLAIN_WARPS), ceil_div(a.vdim_p, 32 * PLAIN_MAX_VEC));
   if (a.f32) paged_attention_plain_kernel<float><<<grid, PLAIN_WARPS * 32, smem, st>>>(a);
   else paged_attention_plain_kernel<__nv_bfloat16><<<grid, PLAIN_WARPS * 32, smem, st>>>(a);
   return launch_check("paged_attention_plain");
@@ -540,11 +562,20 @@ extern "C" int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream) {
   if (a.f32) launch_mix_rows<float>(a, grid, st);
   else launch_mix_rows<__nv_bfloat16>(a, grid, st);
   if (split) {
-    const dim3 ffg(ceil_div(a.ff, 256 * 8), ceil_div(a.rows, 2));
-    if (a.f32) ff_rows_kernel<float><<<ffg, 256, 0, st>>>(a);
-    else ff_rows_kernel<__nv_bfloat16><<<ffg, 256, 0, st>>>(a);
+    if (a.f32) launch_ff_rows<float>(a.in, a.ld_in, a.off_gate, a.off_up, a.ff, a.act, a.ff_out, a.ld_ff, a.rows, st);
+    else launch_ff_rows<__nv_bfloat16>(a.in, a.ld_in, a.off_gate, a.off_up, a.ff, a.act, a.ff_out, a.ld_ff, a.rows, st);
   }
   return launch_check("mix_rows", split ? 2 : 1);
+}
+
+extern "C" int nfn_ff_rows(int f32, const void* in, int ld_in, int off_gate, int off_up, int ff, int act, void* out, int ld_out, int rows, nfn_stream_t stream) {
+  if (rows <= 0 || ff <= 0) return 0;
+  if ((ld_in | off_gate | ff | ld_out) & 7 || (off_up >= 0 && (off_up & 7))) return fail(-1, "ff_rows: widths and offsets must be multiples of 8");
+  if (ceil_div(rows, 2) > 65535) return fail(-1, "ff_rows: too many rows in one launch");
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  if (f32) launch_ff_rows<float>(in, ld_in, off_gate, off_up, ff, act, out, ld_out, rows, st);
+  else launch_ff_rows<__nv_bfloat16>(in, ld_in, off_gate, off_up, ff, act, out, ld_out, rows, st);
+  return launch_check("ff_rows");
 }
 
 extern "C" int nfn_side_mul(int f32, const float* gate, const int* tokens, const void* side_embed, long long ld_embed, int col0, int vocab,

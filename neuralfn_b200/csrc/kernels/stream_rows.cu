@@ -1,7 +1,8 @@
 // Residual streams: the pass between two sublayers. A row's residual is a handful of fp32 rows ("streams"); a finished sublayer's
 // output enters all of them through a small mixing matrix, the next sublayer reads a weighted sum of them through its norm. One CTA
 // per row does both: every stream is read and written once, the weighted sum waits in shared memory until its norm is known.
-// A single plain residual is the case of one stream with unit weights.
+// A single plain residual is the case of one stream with unit weights. The update may have a norm of its own (designs that norm a sublayer's output
+// instead of its input), its rows may carry weights (routed experts) and a row every token has (a shared expert).
 #include "common.h"
 #include "paged.cuh"
 
@@ -25,7 +26,7 @@ template <typename T, int S, int ST_THREADS>
 __global__ void __launch_bounds__(ST_THREADS)
 stream_pass_kernel(const nfn_stream_args p) {
   extern __shared__ float st_row[];                        // [ld] u
-  __shared__ float red[ST_THREADS / 32], w_mix[S][S], w_out[S], w_in[S];
+  __shared__ float red[ST_THREADS / 32], red_y[ST_THREADS / 32], w_mix[S][S], w_out[S], w_in[S];
   const int r = blockIdx.x, n = p.streams, vecs = p.ld / 4;
   const int src = p.src_rows ? p.src_rows[r] : r;
   const __nv_bfloat16* emb = nullptr;
@@ -34,19 +35,26 @@ stream_pass_kernel(const nfn_stream_args p) {
   float* x_out = p.x_out ? p.x_out + (size_t)r * n * p.ld : nullptr;
   const T* y = static_cast<const T*>(p.y);
   float4 b[S], f;
-  auto fetch = [&](int v) {
+  auto fetch_x = [&](int v) {
     if (emb) {
       b[0] = load4(emb + 4 * v);
     } else {
 #pragma unroll
       for (int s = 0; s < S; ++s) b[s] = s < n ? load4(x + (size_t)s * p.ld + 4 * v) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+  };
+  auto fetch_y = [&](int v) {
     f = make_float4(0.f, 0.f, 0.f, 0.f);
     if (p.y) {
 #pragma unroll 4
       for (int j = 0; j < p.y_rows; ++j) {
         const int at = src * p.y_rows + j, yr = p.y_index ? p.y_index[at] : at;
         const float4 g = load4(y + (size_t)yr * p.ld + 4 * v);
+        const float a = p.y_item ? p.y_item[at] : 1.f;
+        f.x += a * g.x; f.y += a * g.y; f.z += a * g.z; f.w += a * g.w;
+      }
+      if (p.y_plus) {
+        const float4 g = load4(static_cast<const T*>(p.y_plus) + (size_t)src * p.ld + 4 * v);
         f.x += g.x; f.y += g.y; f.z += g.z; f.w += g.w;
       }
     }
@@ -60,13 +68,36 @@ stream_pass_kernel(const nfn_stream_args p) {
     w_out[s] = s < n ? (p.out ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.out)[s]) : 1.f) : 0.f;
     w_in[s] = s < n ? (p.in ? __bfloat162float(static_cast<const __nv_bfloat16*>(p.in)[s]) : 1.f) : 0.f;
   }
-  if (threadIdx.x < vecs) fetch(threadIdx.x);
+  if (threadIdx.x < vecs) {
+    fetch_x(threadIdx.x);
+    fetch_y(threadIdx.x);
+  }
   float4 wt = make_float4(0.f, 0.f, 0.f, 0.f);             // the norm's weights of the first piece come along
-  if (p.h && threadIdx.x < vecs) wt = load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * threadIdx.x);
+  if (p.h && p.weight && threadIdx.x < vecs) wt = load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * threadIdx.x);
   __syncthreads();
+  float ry = 0.f;
+  if (p.y_weight) {                                        // the update's own norm: its pieces past the first one wait in shared memory
+    float sy = threadIdx.x < vecs ? f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w : 0.f;
+    const float4 first = f;
+    for (int v = threadIdx.x + ST_THREADS; v < vecs; v += ST_THREADS) {
+      fetch_y(v);
+      store4(st_row + 4 * v, f);
+      sy += f.x * f.x + f.y * f.y + f.z * f.z + f.w * f.w;
+    }
+    f = first;
+    ry = p.y_scale / sqrtf(st_block_sum<ST_THREADS>(sy, red_y) / (float)p.width + p.eps);
+  }
   float ss = 0.f;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
-    if (v != threadIdx.x) fetch(v);
+    if (v != threadIdx.x) {
+      fetch_x(v);
+      if (p.y_weight) f = load4(st_row + 4 * v);
+      else fetch_y(v);
+    }
+    if (p.y_weight) {
+      const float4 w = load4(static_cast<const __nv_bfloat16*>(p.y_weight) + 4 * v);
+      f.x *= ry * w.x; f.y *= ry * w.y; f.z *= ry * w.z; f.w *= ry * w.w;
+    }
     if (emb) {
       b[0].x *= p.embed_scale; b[0].y *= p.embed_scale; b[0].z *= p.embed_scale; b[0].w *= p.embed_scale;
 #pragma unroll
@@ -99,11 +130,15 @@ stream_pass_kernel(const nfn_stream_args p) {
         const float m = w_in[s];
         u.x += m * b[s].x; u.y += m * b[s].y; u.z += m * b[s].z; u.w += m * b[s].w;
       }
+      if (!p.weight) {                                     // no norm: the row leaves as it is
+        store4(static_cast<T*>(p.h) + (size_t)r * p.ld + 4 * v, u);
+        continue;
+      }
       store4(st_row + 4 * v, u);
       ss += u.x * u.x + u.y * u.y + u.z * u.z + u.w * u.w;
     }
   }
-  if (!p.h) return;
+  if (!p.h || !p.weight) return;
   const float rms = 1.f / sqrtf(st_block_sum<ST_THREADS>(ss, red) / (float)p.width + p.eps);
   T* h = static_cast<T*>(p.h) + (size_t)r * p.ld;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
@@ -115,7 +150,7 @@ stream_pass_kernel(const nfn_stream_args p) {
 
 template <typename T, int S, int THREADS>
 static int launch_stream(const nfn_stream_args& a, cudaStream_t st) {
-  const size_t smem = a.h ? (size_t)a.ld * sizeof(float) : 0;
+  const size_t smem = a.h || a.y_weight ? (size_t)a.ld * sizeof(float) : 0;
   auto kern = stream_pass_kernel<T, S, THREADS>;
   static bool raised[64] = {};
   int dev = 0;

@@ -16,7 +16,8 @@ class _Stream(C.Structure):
     _fields_ = [("f32", C.c_int), ("rows", C.c_int), ("width", C.c_int), ("ld", C.c_int), ("streams", C.c_int), ("x", C.c_void_p), ("x_out", C.c_void_p),
                 ("src_rows", C.c_void_p), ("tokens", C.c_void_p), ("embed", C.c_void_p), ("embed_scale", C.c_float), ("vocab", C.c_int), ("y", C.c_void_p),
                 ("y_rows", C.c_int), ("y_index", C.c_void_p), ("mix", C.c_void_p), ("out", C.c_void_p), ("in_", C.c_void_p), ("h", C.c_void_p),
-                ("weight", C.c_void_p), ("eps", C.c_float), ("weight_offset", C.c_float)]
+                ("weight", C.c_void_p), ("eps", C.c_float), ("weight_offset", C.c_float), ("y_item", C.c_void_p), ("y_plus", C.c_void_p), ("y_weight", C.c_void_p),
+                ("y_scale", C.c_float)]
 
 
 class _Delta(C.Structure):
@@ -25,11 +26,16 @@ class _Delta(C.Structure):
                 ("unit_eps", C.c_float), ("state", C.c_void_p), ("o", C.c_void_p), ("ld_o", C.c_int), ("seqs", C.c_void_p), ("n_seqs", C.c_int)]
 
 
+class RouteRule(C.Structure):
+    """``nfn_route_rule``"""
+    _fields_ = [("correction", C.c_void_p), ("groups", C.c_int), ("keep_groups", C.c_int), ("normalise", C.c_int), ("scale", C.c_float)]
+
+
 class _Experts(C.Structure):
     _fields_ = [("f32", C.c_int), ("rows", C.c_int), ("width", C.c_int), ("ff", C.c_int), ("experts", C.c_int), ("top", C.c_int), ("act", C.c_int),
                 ("logits", C.c_void_p), ("ld_logits", C.c_int), ("h", C.c_void_p), ("ld_h", C.c_int), ("w_gate_up", C.c_void_p), ("w_down", C.c_void_p),
                 ("idx", C.c_void_p), ("weight", C.c_void_p), ("order", C.c_void_p), ("offsets", C.c_void_p), ("active", C.c_void_p), ("mid", C.c_void_p),
-                ("y", C.c_void_p), ("ld_y", C.c_int)]
+                ("y", C.c_void_p), ("ld_y", C.c_int), ("plain", C.c_int), ("rule", RouteRule)]
 
 
 def _p(t: torch.Tensor | None):

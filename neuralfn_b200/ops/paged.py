@@ -19,7 +19,7 @@ class _Attention(C.Structure):
                 ("window", C.c_int), ("scale", C.c_float), ("slopes", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int), ("out", C.c_void_p),
                 ("ld_o", C.c_int), ("row_slot", C.c_void_p), ("row_pos", C.c_void_p), ("rows", C.c_int), ("row0", C.c_int), ("max_keys", C.c_int),
                 ("workspace", C.c_void_p), ("workspace_bytes", C.c_longlong), ("tiles", C.c_void_p), ("n_tiles", C.c_int), ("total_rows", C.c_int),
-                ("keep_first", C.c_int), ("softcap", C.c_float), ("sink", C.c_int)]
+                ("keep_first", C.c_int), ("softcap", C.c_float), ("sink", C.c_int), ("chunk", C.c_int)]
 
 
 class _Mix(C.Structure):

@@ -57,14 +57,16 @@ class _CLayer(C.Structure):
                 ("kv_from", C.c_int), ("scale", C.c_float), ("alibi", C.c_float), ("q_temp_coef", C.c_float), ("q_temp_every", C.c_int),
                 ("out_gate", C.c_int), ("ff", C.c_int), ("ff_act", C.c_int), ("mixer", C.c_int), ("qkv_bias", C.c_int), ("keep_first", C.c_int),
                 ("softcap", C.c_float), ("sink", C.c_int), ("rank_decay", C.c_int), ("rank_gate", C.c_int), ("experts", C.c_int), ("top", C.c_int),
-                ("expert_ff", C.c_int), ("weights_of", C.c_int)]
+                ("expert_ff", C.c_int), ("weights_of", C.c_int), ("chunk", C.c_int), ("qk_norm", C.c_int), ("rot_dims", C.c_int), ("rot_base", C.c_double),
+                ("key_values", C.c_int), ("kv_rank", C.c_int), ("rot_dim", C.c_int), ("expert_plain", C.c_int), ("shared_ff", C.c_int), ("route_correction", C.c_int),
+                ("route_groups", C.c_int), ("route_keep", C.c_int), ("route_normalise", C.c_int), ("route_scale", C.c_float)]
 
 
 class _CLayeredConfig(C.Structure):
     _fields_ = [("n_layer", C.c_int), ("width", C.c_int), ("vocab", C.c_int), ("side_dim", C.c_int), ("embed_scale", C.c_float),
                 ("norm_eps", C.c_float), ("dtype", C.c_int), ("max_seq", C.c_int), ("max_batch", C.c_int), ("kv_tokens", C.c_int),
                 ("max_step_rows", C.c_int), ("use_cuda_graph", C.c_int), ("chained", C.c_int), ("streams", C.c_int), ("untied_head", C.c_int),
-                ("norm_offset", C.c_float), ("logit_scale", C.c_float), ("logit_softcap", C.c_float)]
+                ("norm_offset", C.c_float), ("logit_scale", C.c_float), ("logit_softcap", C.c_float), ("post_norm", C.c_int), ("residual_mult", C.c_float)]
 
 
 class _CEntry(C.Structure):
@@ -102,19 +104,46 @@ class LayerSpec:
     top: int = 0
     expert_ff: int = 0
     weights_of: int = -1
+    chunk: int = 0
+    qk_norm: int = 0
+    rot_dims: int = 0
+    rot_base: float = 0.0
+    key_values: int = 0
+    kv_rank: int = 0
+    rot_dim: int = 0
+    expert_plain: int = 0
+    shared_ff: int = 0
+    route_correction: int = 0
+    route_groups: int = 0
+    route_keep: int = 0
+    route_normalise: int = 0
+    route_scale: float = 0.0
 
-    FF_ACT_IDS = {"gelu": 1, "silu": 3, "relu": 6}
-    MIXER_IDS = {"attention": 0, "delta": 1}
+    FF_ACT_IDS = {"gelu": 1, "silu": 3, "relu2": 4, "relu": 6}
+    MIXER_IDS = {"attention": 0, "delta": 1, "latent": 2, "wkv": 3}
 
     def c(self) -> _CLayer:
         return _CLayer(self.heads, self.kv_heads, self.dim, self.vdim, self.conv_taps, self.window, self.kv_from, self.scale, self.alibi,
                        self.q_temp_coef, self.q_temp_every, self.out_gate, self.ff, self.FF_ACT_IDS[self.ff_act], self.MIXER_IDS[self.mixer], self.qkv_bias, self.keep_first,
-                       self.softcap, self.sink, self.rank_decay, self.rank_gate, self.experts, self.top, self.expert_ff, self.weights_of)
+                       self.softcap, self.sink, self.rank_decay, self.rank_gate, self.experts, self.top, self.expert_ff, self.weights_of,
+                       self.chunk, self.qk_norm, self.rot_dims, self.rot_base, self.key_values, self.kv_rank, self.rot_dim, self.expert_plain, self.shared_ff,
+                       self.route_correction, self.route_groups, self.route_keep, self.route_normalise, self.route_scale)
+
+    @property
+    def paged(self) -> bool:
+        return self.mixer in ("attention", "latent")
+
+    @property
+    def look(self) -> int:
+        """Most positions a query sees (0: all)."""
+        return self.chunk or self.window
 
     @property
     def cache_row(self) -> int:
         """Values one token adds to this layer's pages."""
-        return 0 if self.kv_from >= 0 or self.mixer == "delta" else self.kv_heads * (self.dim + self.vdim)
+        if self.kv_from >= 0 or not self.paged:
+            return 0
+        return self.kv_rank + self.rot_dim if self.mixer == "latent" else self.kv_heads * (self.dim + self.vdim)
 
 
 @dataclass(frozen=True)
@@ -140,6 +169,8 @@ class LayeredEngineConfig:
     norm_offset: float = 0.0
     logit_scale: float = 1.0
     logit_softcap: float = 0.0
+    post_norm: int = 0
+    residual_mult: float = 1.0
 
     family = 2
     kv_cache_mode = 0
@@ -158,17 +189,17 @@ class LayeredEngineConfig:
 
     @property
     def window(self) -> int:
-        """Most tokens behind a sequence's end whose pages stay (widest window plus kept first tokens, in whole pages) when every layer
-        with pages has a window, else 0."""
-        paged = [y for y in self.layers if y.mixer == "attention"]
-        if any(y.window == 0 for y in paged):
+        """Most tokens behind a sequence's end whose pages stay (widest window or chunk plus kept first tokens, in whole pages) when every
+        layer with pages has a limit, else 0."""
+        paged = [y for y in self.layers if y.paged]
+        if any(y.look == 0 for y in paged):
             return 0
-        return max((y.window + (y.keep_first + KV_PAGE - 1) // KV_PAGE * KV_PAGE for y in paged), default=0)
+        return max((y.look + (y.keep_first + KV_PAGE - 1) // KV_PAGE * KV_PAGE for y in paged), default=0)
 
     def create(self, lib, device: int):
         cc = _CLayeredConfig(len(self.layers), self.width, self.vocab, self.side_dim, self.embed_scale, self.norm_eps,
                              int(self.dtype == "float32"), self.max_seq, self.max_batch, self.kv_tokens, self.max_step_rows, self.use_cuda_graph, self.chained,
-                             self.streams, self.untied_head, self.norm_offset, self.logit_scale, self.logit_softcap)
+                             self.streams, self.untied_head, self.norm_offset, self.logit_scale, self.logit_softcap, self.post_norm, self.residual_mult)
         arr = (_CLayer * len(self.layers))(*[y.c() for y in self.layers])
         return lib.nfn_engine_create_layered(C.byref(cc), arr, device)
 
@@ -188,16 +219,27 @@ class LayeredEngineConfig:
                 own = q * up(y.rank_decay) + v * up(y.rank_gate)
                 cache += self.max_batch * (4 * q * vdim + 2 * es * conv * (y.conv_taps - 1))
                 widest = max(widest, n_in + conv + (4 // es) * (q + v) + 2 * v)
+            elif y.mixer == "wkv":
+                n_in, own = 4 * q, up(y.rank_decay) * (wp + 2 * q)
+                cache += self.max_batch * 4 * (q * dim + 2 * wp)
+                widest = max(widest, n_in + 5 * wp + v + (4 // es) * (2 * q + up(y.rank_decay)) + 2 * up(y.rank_decay))
+            elif y.mixer == "latent":
+                rank, rot = up(y.kv_rank), up(y.rot_dim)
+                n_in, own = y.heads * (dim + rot) + (0 if y.kv_from >= 0 else rank + rot), y.heads * rank * (2 * dim + vdim)
+                cache += 0 if y.kv_from >= 0 else (rank + rot) * pool * es
+                short = rows if es == 4 else min(rows, 15 * self.max_batch)                # rows that attend to the latents, rows of the expansion
+                cache += short * y.heads * (2 * rank + rot) * es + (0 if es == 4 else (rows + min(y.look or self.max_seq, self.max_seq) + 2 * KV_PAGE) * (rank + y.heads * (dim + vdim)) * es)
+                widest = max(widest, n_in + v)
             else:
                 kv = 0 if y.kv_from >= 0 else y.kv_heads * (dim + vdim)
-                n_in, own = q + kv + (v if y.out_gate else 0) + 2 * up(y.ff), 0
+                n_in, own = q + kv + (v if y.out_gate else 0) + (0 if self.chained else 2 * up(y.ff)), 0
                 cache += kv * pool * es
                 widest = max(widest, n_in + q + v + up(y.ff))
             if y.weights_of < 0:
-                weights += wp * (n_in + v + up(y.ff) + 2 * up(self.side_dim)) + own + wp * (up(y.experts) + 3 * y.experts * up(y.expert_ff))
+                weights += wp * (n_in + v + up(y.ff) * (3 if self.chained else 1) + 2 * up(self.side_dim) + 2 * up(y.shared_ff)) + own + wp * (up(y.experts) + 3 * y.experts * up(y.expert_ff))
             routed = max(routed, (rows * y.top + 127 * y.experts) * es * (2 * wp + 3 * up(y.expert_ff)) if y.experts else 0)
         acts = rows * (es * (3 * wp + widest + up(self.side_dim)) + 4 * (wp * max(self.streams, 1) + up(self.side_dim))) + 4 * 2 * max(self.max_batch, 64) * up(self.vocab)
-        chunks = (96 << 20) if es == 2 and any(y.mixer == "delta" for y in self.layers) else 0        # operands of the delta rule's prompt chunks
+        chunks = (96 << 20) * sum(any(y.mixer == m for y in self.layers) for m in ("delta", "wkv")) if es == 2 else 0        # operands of the recurrences' prompt chunks
         return int(2 * weights + cache + acts + routed + chunks)
 
 
