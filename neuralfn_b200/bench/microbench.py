@@ -438,7 +438,128 @@ def case_layered(args):
     _report("gemm (dense, batch rows)", t(lambda: gemm(y1, wide, out=dense[:B])), bytes_=2.0 * 8 * F * C, args=args, extra={"B": B})
 
 
-CASES = {"gemm": case_gemm, "paged": case_paged, "layered": case_layered, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
+def case_mixers(args):
+    """Kernels of rotated chunk attention, latent attention, time mixing, output norms and plain experts beside their closest counterparts, at one layer of
+    ``--heads`` / ``--kv-heads`` x ``--head-dim``, width ``--k``: chunks of 1.5 x ``--window`` (queries in the middle of one), latents of 512 + 64 channels with
+    ``--window``, ``--experts`` experts of which four of ``--n`` / 4 are used beside a shared one of ``--n`` / 2."""
+    from neuralfn_b200.ops import infer as I, kernels as K, layered as Y, paged as P
+    from neuralfn_b200.ops.gemm import gemm
+    from neuralfn_b200.ops.moe import MoEWorkspace, _grouped_gemm, moe_forward
+    dev = torch.device("cuda")
+    H, G, D, T, B, W, C, E = args.heads, args.kv_heads or args.heads, args.head_dim, args.seq, args.batch, args.window, args.k, args.experts
+    F, R, RANK, HD, chunk = args.n // 4, 64, 512, args.heads * args.head_dim, W + W // 2
+    rand = lambda *s: torch.randn(*s, device=dev).bfloat16()  # noqa: E731
+    t = lambda fn: time_kernel(fn, args.iters, args.warmup, args.flush)  # noqa: E731
+    i32 = dict(dtype=torch.int32, device=dev)
+    rep = lambda name, fn, **kw: _report(name, t(fn), args=args, **kw)  # noqa: E731
+    w = min(W, T)
+    win_keys = w * (w + 1) / 2 + (T - w) * w
+    chunk_keys = sum(min(chunk, T - a) * (min(chunk, T - a) + 1) / 2 for a in range(0, T, chunk))
+
+    def tile_list(step):
+        return torch.tensor([[r, min(step, T - r), 0, r] for r in range(0, T, step)], **i32)
+
+    # ---- prompt attention ----
+    c = P.PagedCache(1, T, G, D, D, dev)
+    c.k.normal_(), c.v.normal_()
+    q, out, tiles, kw = rand(T, HD), torch.empty(T, HD, device=dev, dtype=torch.bfloat16), tile_list(P.tile_rows(c, H)), dict(heads=H, scale=D ** -0.5)
+    rep("paged_attention_tiles (chunk)", lambda: P.attention_tiles(c, q, tiles, out, chunk=chunk, **kw), flops=4.0 * HD * chunk_keys, extra={"T": T, "chunk": chunk})
+    k, v = rand(T, G * D), rand(T, G * D)
+    fa = dict(B=1, T=T, n_q_heads=H, n_kv_heads=G, head_dim=D, causal=True, window=W)
+    o, lse = K.attention_forward(q, k, v, **fa)
+    rep("attention_fwd", lambda: K.attention_forward(q, k, v, out=o, lse=lse, **fa), flops=4.0 * HD * win_keys, extra={"T": T, "window": W})
+    lc = Y.LatentCache(1, T, RANK, R, dev)
+    lc.k.normal_()
+    ql, x, ltiles, base = rand(T, H * (D + R)), rand(T, 2 * HD), tile_list(128), torch.zeros(1, **i32)
+    rep("latent_attention_tiles", lambda: Y.latent_attention_tiles(lc, ql, x, base, ltiles, out, heads=H, dim=D, vdim=D, window=W, scale=(D + R) ** -0.5),
+        flops=2.0 * H * (2 * D + R) * win_keys, extra={"T": T, "window": W})
+    spans, lat, wkvx = torch.tensor([[0, 0, T // 64, 0]], **i32), torch.empty(T, RANK, device=dev, dtype=torch.bfloat16), rand(2 * HD, RANK)
+    rep("latent_gather", lambda: Y.latent_gather(lc, spans, lat), bytes_=4.0 * T * RANK, extra={"T": T})
+    rep("gemm (expansion)", lambda: gemm(lat, wkvx, out=x), flops=4.0 * T * HD * RANK, extra={"T": T})
+    # ---- rows between products and attention ----
+    rt, freq, wn = P.row_tiles([(0, 0, T, 0)], dev), Y.frequencies(R, 1e4, dev), rand(D)
+    hx = rand(T, (H + G) * D)
+    rep("head_rows", lambda: Y.head_rows(c, hx, rt, hx, heads=H, dim=D, freq=freq, rot_dims=R, eps=1e-5, q_norm=wn, k_norm=wn, key_values=True), bytes_=2.0 * T * D * (2 * H + 3 * G), extra={"T": T})
+    lx = rand(T, H * (D + R) + RANK + R)
+    rep("latent_rows", lambda: Y.latent_rows(lc, lx, rt, heads=H, dim=D, rot_dim=R, rank=RANK, c_norm=rand(RANK), eps=1e-5, freq=freq), bytes_=4.0 * T * (H * R + RANK + R), extra={"T": T})
+    mx, mq = rand(T, (H + 2 * G) * D + 2 * 4 * F), torch.empty(T, HD, device=dev, dtype=torch.bfloat16)
+    cat = torch.empty(T, 4 * F, device=dev, dtype=torch.bfloat16)
+    rep("mix_rows (no convolution)", lambda: P.mix_rows(c, mx, rt, mq, None, heads=H), bytes_=4.0 * T * (H + 2 * G) * D, extra={"T": T})
+    rep("ff_rows", lambda: Y.ff_rows(mx, cat, off_gate=0, off_up=4 * F, act=3), bytes_=6.0 * T * 4 * F, extra={"T": T, "ff": 4 * F})
+    del c, k, v, q, o, mx, mq, cat, hx, lx, ql, x, lc
+    # ---- decode attention ----
+    seen, pos1 = W, chunk + W - 1
+    c = P.PagedCache(B, pos1 + 1, G, D, D, dev)
+    c.k.normal_(), c.v.normal_()
+    q1, o1, slot, pos = rand(B, HD), torch.empty(B, HD, device=dev, dtype=torch.bfloat16), torch.arange(B, **i32), torch.full((B,), pos1, **i32)
+    rep("paged_attention_rows (chunk)", lambda: P.attention_rows(c, q1, slot, pos, o1, chunk=chunk, **kw), bytes_=4.0 * B * G * seen * D, extra={"B": B, "keys": seen})
+    kc, vc, ws = rand(B, G, seen, D), rand(B, G, seen, D), I.DecodeAttentionWorkspace(B, H, G, D, dev)
+    qkv, lens, (cos, sin) = rand(B, (H + 2 * G) * D), torch.full((B,), seen, **i32), I.rope_tables(seen, D, device=dev)
+    rep("decode_attention", lambda: I.decode_attention(qkv, kc, vc, lens, n_q_heads=H, n_kv_heads=G, head_dim=D, workspace=ws, cos=cos, sin=sin, qk_norm=True, out=o1),
+        bytes_=4.0 * B * G * seen * D, extra={"B": B, "keys": seen})
+    lc = Y.LatentCache(B, pos1 + 1, RANK, R, dev)
+    lc.k.normal_()
+    qa, oa = rand(B, H, RANK + R), torch.empty(B, H, RANK, device=dev, dtype=torch.bfloat16)
+    rep("latent_attention_rows", lambda: Y.latent_attention_rows(lc, qa.view(B, -1), slot, pos, oa.view(B, -1), heads=H, window=W, scale=(D + R) ** -0.5),
+        bytes_=2.0 * B * seen * (RANK + R), flops=2.0 * B * H * seen * (2 * RANK + R), extra={"B": B, "keys": seen})
+    wut, wuv, ov = rand(H, RANK, D), rand(H, D, RANK), torch.empty(B, H, D, device=dev, dtype=torch.bfloat16)
+    qn = rand(B, H, D + R)
+    rep("group_products (keys)", lambda: Y.group_products(qn[..., :D], wut, qa), bytes_=2.0 * (H * RANK * D + B * H * (RANK + D)), extra={"B": B})
+    rep("group_products (values)", lambda: Y.group_products(oa, wuv, ov), bytes_=2.0 * (H * RANK * D + B * H * (RANK + D)), extra={"B": B})
+    w4, x4, y4 = rand(4, HD, C), rand(4, B, C), torch.empty(B, 4, HD, device=dev, dtype=torch.bfloat16)
+    rep("group_products (r, k, v, gate)", lambda: Y.group_products(x4.transpose(0, 1), w4, y4), bytes_=8.0 * HD * C, extra={"B": B})
+    rep("gemm (same bytes)", lambda: gemm(x4[0], w4.view(4 * HD, C), out=y4.view(B, 4 * HD)), bytes_=8.0 * HD * C, extra={"B": B})
+    del c, kc, vc, lc, w4
+    # ---- time mixing ----
+    u, w0 = rand(HD), torch.full((HD,), -1.0, device=dev).bfloat16()
+
+    def rule(rows, seqs, slots):
+        return dict(rkv=rand(rows, 4 * HD), z=torch.randn(rows, HD, device=dev), w0=w0, u=u, state=torch.zeros(slots, H, D, D, device=dev), seqs=torch.tensor(seqs, **i32), dim=D)
+
+    r, wsp = rule(T, [[0, T, 0, 0]], 1), torch.empty(96 << 20, device=dev, dtype=torch.uint8)
+    rep("wkv_chunks", lambda: Y.wkv_rule(**r, form="chunks", workspace=wsp), bytes_=14.0 * T * HD, extra={"T": T, "heads": H, "dim": D})
+    dt, a_log = w0, torch.full((H,), -1.0, device=dev).bfloat16()
+    dr = dict(qkv=rand(T, 3 * HD), beta=rand(T, H), decay=torch.randn(T, HD, device=dev), a_log=a_log, dt_bias=dt, state=torch.zeros(1, H, D, D, device=dev), seqs=torch.tensor([[0, T, 0, 0]], **i32),
+              kv_heads=H, dim=D)
+    rep("delta_chunks", lambda: Y.delta_rule(**dr, form="chunks", workspace=wsp), bytes_=14.0 * T * HD, extra={"T": T, "heads": H, "dim": D})
+    r1 = rule(B, [[b, 1, b, 7] for b in range(B)], B)
+    rep("wkv_rows", lambda: Y.wkv_rule(**r1), bytes_=8.0 * B * HD * D, extra={"B": B})
+    d1 = dict(qkv=rand(B, 3 * HD), beta=rand(B, H), decay=torch.randn(B, HD, device=dev), a_log=a_log, dt_bias=dt, state=torch.zeros(B, H, D, D, device=dev),
+              seqs=torch.tensor([[b, 1, b, 7] for b in range(B)], **i32), kv_heads=H, dim=D)
+    rep("delta_rows", lambda: Y.delta_rule(**d1), bytes_=8.0 * B * HD * D, extra={"B": B})
+    low, w2, so, n1 = torch.randn(B, 64, device=dev), rand(HD, 128) * 0.1, torch.empty(B, HD, device=dev, dtype=torch.bfloat16), rand(HD)
+    for b in sorted({1, min(8, B), B}):
+        if b * H <= 4 * 148:
+            st = P.row_tiles([(s, 7, 1, 0) for s in range(b)], dev)
+            rep("wkv_step", lambda: Y.wkv_step(r1["rkv"][:b], low[:b], w2, w0, u, r1["state"], n1, so[:b], st, dim=D, eps=1e-5), bytes_=8.0 * b * HD * D, extra={"B": b})
+    xs, mu, prev, sh = torch.randn(T, C, device=dev), rand(5, C), torch.zeros(2, 1, C, device=dev), torch.empty(5, T, C, device=dev, dtype=torch.bfloat16)
+    rep("shift_rows", lambda: Y.shift_rows(xs, mu, prev, sh, rt), bytes_=14.0 * T * C, extra={"T": T, "width": C})
+    del r, dr, d1, r1, sh
+    # ---- residual, experts ----
+    y, h, wt = rand(T, C), torch.empty(T, C, device=dev, dtype=torch.bfloat16), rand(C)
+    rep("stream_pass (norm on the update)", lambda: Y.stream_pass(xs, h, width=C, streams=1, rows=T, ld=C, f32=False, x_out=xs, y=y, y_weight=wt, y_scale=0.5), bytes_=12.0 * T * C, extra={"T": T})
+    rep("row_norm (fp32 residual)", lambda: P.row_norm(xs, wt, h, eps=1e-5, y=y, y_weight=wt, x_out=xs), bytes_=12.0 * T * C, extra={"T": T})
+    ys, item, plus, order = rand(4 * T, C), torch.rand(4 * T, device=dev), rand(T, C), torch.randperm(4 * T, device=dev).int()
+    rep("stream_pass (experts)", lambda: Y.stream_pass(xs, h, width=C, streams=1, rows=T, ld=C, f32=False, x_out=xs, y=ys, y_rows=4, y_index=order, y_item=item, y_plus=plus, y_weight=wt, y_scale=0.5),
+        bytes_=20.0 * T * C, extra={"T": T})
+    z, corr = torch.randn(T, E, device=dev), torch.zeros(E, device=dev).bfloat16()
+    choice = dict(correction=corr, groups=8 if E % 8 == 0 else 0, keep=4, normalise=True, scale=1.5)
+    rep("expert_choice", lambda: Y.expert_choice(z, 4, **choice), bytes_=4.0 * T * E + 32.0 * T, extra={"T": T})
+    up, down, wr = rand(E, F, C) * C ** -0.5, rand(E, C, F) * F ** -0.5, rand(E, C) * C ** -0.5
+    wg = rand(E, 2 * F, C) * C ** -0.5
+    mw = MoEWorkspace(T, E, 4, C, F, dev)
+    moe_forward(y, wr, wg, down, 4, mw, score_fn="sigmoid", norm_topk=False)
+    rep("grouped gemm (gate and up)", lambda: _grouped_gemm(mw.xs, wg, mw.h, mw), flops=16.0 * T * F * C, extra={"T": T, "experts": E, "ff": F})
+    mid = torch.empty(mw.xs.shape[0], F, device=dev, dtype=torch.bfloat16)
+    rep("grouped gemm (up)", lambda: _grouped_gemm(mw.xs, up, mid, mw), flops=8.0 * T * F * C, extra={"T": T, "experts": E, "ff": F})
+    y1, z1 = rand(B, C), torch.randn(B, E, device=dev)
+    live = int(Y.expert_rows(y1, z1, up, down, experts=E, top=4, act=4, plain=True, **choice)[0].unique().numel())
+    rep("expert_rows (plain)", lambda: Y.expert_rows(y1, z1, up, down, experts=E, top=4, act=4, plain=True, **choice), bytes_=4.0 * live * F * C, extra={"B": B, "experts_used": live})
+    live = int(Y.expert_rows(y1, z1, wg, down, experts=E, top=4)[0].unique().numel())
+    rep("expert_rows (gated)", lambda: Y.expert_rows(y1, z1, wg, down, experts=E, top=4), bytes_=6.0 * live * F * C, extra={"B": B, "experts_used": live})
+
+
+CASES = {"gemm": case_gemm, "paged": case_paged, "layered": case_layered, "mixers": case_mixers, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
          "cross_entropy": case_cross_entropy, "norm": case_norm, "adamw": case_adamw, "decode_attention": case_decode_attention,
          "skinny": case_skinny, "grouped_k": case_grouped_k, "kquant_gemv": case_kquant_gemv, "gemm_kquant": case_gemm_kquant, "block_attention": case_block_attention,
          "turboquant_attention": case_turboquant_attention, "engine_decode": case_engine_decode}

@@ -1,8 +1,10 @@
-"""Prefill and decode throughput of Bulidra or Murilorn and, at equal size, of Glimmer blocks - the closest model the engine served before:
+"""Prefill and decode throughput of Bulidra, Murilorn or Vopozen and, at equal size, of Glimmer blocks - the closest model the engine served before:
 grouped heads, sliding windows, gated attention, gated feed-forward. Random bf16 weights; one JSON line per model, size and phase.
 
 Murilorn at equal size: delta-rule and attention layers in turn with the same heads, the same active feed-forward width (four of thirty-two
-experts), four residual streams.
+experts), four residual streams. Vopozen at equal size: chunked attention, latent attention, time mixing and latent attention on the earlier layer's
+cache in turn, the same heads, gated and routed feed-forwards in turn with the same active weights (four of thirty-two plain experts and a shared
+one).
 
 ``ms`` is device time (CUDA events on the engine's stream, median over repetitions of the public ``prefill`` / ``decode`` call,
 including its host-to-device copy of tokens and the read-back of the drawn token); weights and caches are larger than L2. Beside it
@@ -23,6 +25,8 @@ SIZES = {
 }
 SIDE_DIM = 256
 EXPERTS, TOP, STREAMS, RANK, KEEP = 32, 4, 4, 128, 4
+LATENT, ROT, DECAY = 512, 64, 64
+VOPOZEN = ("attention", "latent", "wkv", "reader")
 
 
 def _peaks() -> tuple[float, float]:
@@ -35,7 +39,7 @@ def _peaks() -> tuple[float, float]:
 
 def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
     from ..models.bulidra import BulidraConfig, BulidraLayer, engine_config
-    from ..models import murilorn as M
+    from ..models import murilorn as M, vopozen as V
     from ..serving import EngineConfig, ResidentEngine
     L = z["layers"]
     if kind == "murilorn":
@@ -44,6 +48,8 @@ def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
                 M.MurilornLayer("attention", z["heads"], z["kv_heads"], z["dim"], z["dim"], scale=z["dim"] ** -0.5, softcap=30.0, window=z["window"], keep_first=KEEP, **ex))
         cfg = M.engine_config(M.MurilornConfig(z["vocab"], z["width"], 1.0, 1e-5, STREAMS, None, 1.0, 30.0, (pair * L)[:L]), max_batch=max_batch, max_seq=max_seq,
                               max_step_rows=max_seq)
+    elif kind == "vopozen":
+        cfg = V.engine_config(V.VopozenConfig(z["vocab"], z["width"], 1e-5, 0.5, tuple(_vopozen_layers(z))), max_batch=max_batch, max_seq=max_seq, max_step_rows=max_seq)
     elif kind == "bulidra":
         layers = tuple(BulidraLayer(z["heads"], z["kv_heads"], z["dim"], z["dim"], 4, z["dim"] ** -0.5, z["window"], 0.1, 1024, None, z["ff"]) for _ in range(L))
         cfg = engine_config(BulidraConfig(z["vocab"], z["width"], 1.0, 1e-5, SIDE_DIM, layers), max_batch=max_batch, max_seq=max_seq, max_step_rows=max_seq)
@@ -56,7 +62,7 @@ def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
         leaf = n.rsplit(".", 1)[-1]
         if leaf.startswith("hc"):
             t = torch.eye(STREAMS, device="cuda").flatten() if leaf.endswith("mix") else torch.full((k,), 1.0 / STREAMS if leaf.endswith("in") else 1.0, device="cuda")
-        elif leaf in ("a_log", "dt_bias"):
+        elif leaf in ("a_log", "dt_bias", "w0"):
             t = torch.full((k,), -1.0, device="cuda")
         elif "norm" in n:
             t = torch.full((k,), 0.0 if kind == "murilorn" and leaf != "out_norm" else 1.0, device="cuda")
@@ -65,6 +71,24 @@ def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
         eng.set_tensor(n, t.bfloat16())
     eng.finalize()
     return eng
+
+
+def _vopozen_layers(z: dict) -> list:
+    """Chunks of 1.5 windows: the decode steps at a context of 4096 then see as many keys as with the window."""
+    from ..models import vopozen as V
+    L, rot = z["layers"], dict(rot_base=1e4, scale=z["dim"] ** -0.5)
+    out: list = []
+    for i in range(L):
+        kind = VOPOZEN[i % 4]
+        f = dict(ff=z["ff"]) if i % 2 == 0 else dict(experts=EXPERTS, top=TOP, expert_ff=z["ff"] // 4, shared_ff=z["ff"] // 2, groups=8, keep=4, route_scale=1.5)
+        if kind == "attention":
+            out.append(V.VopozenLayer("attention", z["heads"], z["kv_heads"], z["dim"], z["dim"], look=3 * z["window"] // 2, rot_dims=ROT, **rot, **f))
+        elif kind == "wkv":
+            out.append(V.VopozenLayer("wkv", z["heads"], z["heads"], z["dim"], z["dim"], rank_decay=DECAY, **f))
+        else:
+            out.append(V.VopozenLayer("latent_attention", z["heads"], 1, z["dim"], z["dim"], look=z["window"], rot_dims=ROT, rot_dim=ROT, kv_rank=LATENT, kv_from=i - 2 if kind == "reader" else -1,
+                                      **rot, **f))
+    return out
 
 
 def _time(eng, fn, n: int, warmup: int) -> float:
@@ -85,6 +109,8 @@ def _work(z: dict, kind: str, prompt: int, batch: int, context: int) -> tuple[fl
     w, q, kv = z["width"], z["heads"] * z["dim"], z["kv_heads"] * z["dim"]
     if kind == "murilorn":
         return _murilorn_work(z, prompt, batch, context)
+    if kind == "vopozen":
+        return _vopozen_work(z, prompt, batch, context)
     per = w * (q + 2 * kv + q + 2 * z["ff"]) + w * (q + z["ff"]) + (2 * w * SIDE_DIM if kind == "bulidra" else 0)
     win = min(z["window"], prompt)
     keys = win * (win + 1) / 2 + (prompt - win) * win
@@ -107,6 +133,32 @@ def _murilorn_work(z: dict, prompt: int, batch: int, context: int) -> tuple[floa
     chosen = EXPERTS * (1 - (1 - TOP / EXPERTS) ** batch)       # experts a batch of uniform choices touches
     seen = min(z["window"] + KEEP, context)
     byts = 2.0 * (n_delta * delta + n_att * (att + batch * seen * 2 * kv) + L * (chosen * expert + EXPERTS * w)) + n_delta * batch * 8.0 * q * z["dim"] + 2.0 * z["vocab"] * w
+    return flops, byts
+
+
+def _vopozen_work(z: dict, prompt: int, batch: int, context: int) -> tuple[float, float]:
+    w, q, kv = z["width"], z["heads"] * z["dim"], z["kv_heads"] * z["dim"]
+    chosen = EXPERTS * (1 - (1 - TOP / EXPERTS) ** batch)       # experts a batch of uniform choices touches
+    flops, byts = 0.0, 2.0 * z["vocab"] * w
+    for y in _vopozen_layers(z):
+        if y.type == "attention":
+            per, n = w * (q + kv) + q * w, min(y.look, prompt)
+            keys = prompt / n * n * (n + 1) / 2
+            flops += 4.0 * q * keys
+            byts += 2.0 * batch * min(context % y.look or y.look, context) * 2 * kv
+        elif y.type == "wkv":
+            per = w * (4 * q + DECAY) + DECAY * q + q * w
+            flops += 5.0 * q * z["dim"] * prompt
+            byts += batch * 8.0 * q * z["dim"]
+        else:
+            row = LATENT + ROT
+            per, n = w * (z["heads"] * (z["dim"] + ROT) + (row if y.kv_from < 0 else 0)) + 2 * q * LATENT + q * w, min(y.look, prompt)
+            keys = n * (n + 1) / 2 + (prompt - n) * n
+            flops += 2.0 * z["heads"] * (2 * z["dim"] + ROT) * keys
+            byts += 2.0 * batch * min(y.look, context) * row
+        act, read = (3 * w * y.ff,) * 2 if y.ff else (w * (2 * TOP * y.expert_ff + 2 * y.shared_ff + EXPERTS), w * (2 * chosen * y.expert_ff + 2 * y.shared_ff + EXPERTS))
+        flops += 2.0 * (per + act) * prompt
+        byts += 2.0 * (per + read)
     return flops, byts
 
 

@@ -97,7 +97,7 @@ typedef struct {
   int expert_plain;      // experts down(act(up h)), weighted at their output, instead of gated ones weighted at their input
   int shared_ff;         // width of an expert of the same (plain) form that every token has; 0: none
   int route_correction;  // choice scores s + correction
-  int route_groups, route_keep;   // experts in equal groups of neighbours, of which the best are kept (0: no groups)
+  int route_groups, route_keep;   // consecutive experts form groups, the choice is limited to the best of them (nfn_route_rule; 0: no groups)
   int route_normalise;   // weights divided by their sum
   float route_scale;     // times this; 0 counts as 1
 } nfn_layer_desc;

@@ -559,9 +559,9 @@ int nfn_wkv_step(const nfn_wkv_step_args* args, nfn_stream_t stream);
 // ---- mixture of experts for the rows of a step (moe.cu, moe_rows.cu) ----------------------------------------------------------
 // item i = token i / top, choice i % top. Gated experts take the routing weight at their INPUT: mid = act(w G h) * (w U h); plain ones (w_gate_up
 // [E][ff][width]) compute mid = act(U h) and leave the weight to whoever sums the items.
-// nfn_route_rule: how experts are chosen and weighted. Scores s = sigmoid(logits); choice scores s + correction (bf16, NULL: none); with groups > 0
-// (equal groups of neighbours) a group counts by the sum of its two largest choice scores and only experts of the best keep_groups can be chosen;
-// weights s, with normalise / (sum of the chosen ones + 1e-20), times scale. Ties: the lower index.
+// nfn_route_rule: how experts are chosen and weighted. s = sigmoid(logits). The choice goes by s + correction (bf16, NULL: by s). groups > 0: group g is
+// experts [g E / groups, (g + 1) E / groups); the keep_groups whose two best members add up to most stay open, the rest are out of the choice.
+// Weights: s, with normalise / (sum of the chosen ones + 1e-20), times scale. Ties: the lower index.
 typedef struct { const void* correction; int groups, keep_groups, normalise; float scale; } nfn_route_rule;
 int nfn_moe_choose(const float* logits, int ld, int T, int E, int k, const nfn_route_rule* rule, int* idx, float* weight, int* counts, nfn_stream_t stream);
 int nfn_moe_route(const float* logits, int ld, int T, int E, int k, int score_fn, int norm_topk, float route_scale, int* topk_idx, float* topk_w,

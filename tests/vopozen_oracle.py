@@ -37,19 +37,21 @@ def rotate(x, first, dims, base):
 
 
 def in_chunk(i, j, size):
-    return j <= i and i // size == j // size
+    return (j <= i) & (i // size == j // size)
 
 
 def in_window(i, j, size):
-    return 0 <= i - j < size
+    return (j <= i) & (i - j < size)
 
 
 def seen(T, rule, size):
-    m = torch.zeros(T, T, dtype=torch.bool)
-    for i in range(T):
-        for j in range(i + 1):
-            m[i, j] = rule(i, j, size)
-    return m
+    """[T, T]: does query i see key j (size 0: every earlier key)."""
+    i, j = torch.arange(T)[:, None], torch.arange(T)[None, :]
+    return rule(i, j, size) if size else j <= i
+
+
+def size_of(m):
+    return (m.get("mask") or {}).get("size", 0)
 
 
 def attend(scores, mask, v):
@@ -62,7 +64,7 @@ def attention_mixer(h, W, p, m, eps):
     q, v = (h @ W[p + "q"].T).view(T, H, d), (h @ W[p + "k"].T).view(T, G, d)
     q, k = norm(q, W[p + "q.norm"], eps), norm(v, W[p + "k.norm"], eps)
     q, k = (rotate(t, 0, m["rot"]["dims"], m["rot"]["base"]) for t in (q, k))
-    mask = seen(T, in_chunk, m["mask"]["size"])
+    mask = seen(T, in_chunk, size_of(m))
     out = torch.stack([attend(q[:, x] @ k[:, x // (H // G)].T * m["scale"], mask, v[:, x // (H // G)]) for x in range(H)], 1)
     return out.reshape(T, -1) @ W[p + "o"].T
 
@@ -79,7 +81,7 @@ def latent_mixer(h, W, p, m, latent):
     q = (h @ W[p + "q"].T).view(T, H, d + e)
     qr = rotate(q[..., d:], 0, m["rot"]["dims"], m["rot"]["base"])
     k, v = (c @ W[p + "uk"].T).view(T, H, d), (c @ W[p + "uv"].T).view(T, H, m["vdim"])
-    mask = seen(T, in_window, m["mask"]["size"])
+    mask = seen(T, in_window, size_of(m))
     out = torch.stack([attend((q[:, x, :d] @ k[:, x].T + qr[:, x] @ kr.T) * m["scale"], mask, v[:, x]) for x in range(H)], 1)
     return out.reshape(T, -1) @ W[p + "o"].T
 
@@ -122,7 +124,7 @@ def expert(h, W, p):
 
 
 def allowed(choice, groups):
-    """Experts of the best groups; a group counts by the sum of its two largest choice scores."""
+    """Which experts are open to the choice: those of the groups whose two best members add up to most."""
     n = choice.numel() // groups["count"]
     score = choice.view(-1, n).sort(-1, descending=True).values[:, :2].sum(-1)
     best = torch.sort(score, descending=True, stable=True).indices[:groups["keep"]]
@@ -131,11 +133,15 @@ def allowed(choice, groups):
     return ok.view(-1)
 
 
+def closed(choice, ok):
+    return choice.masked_fill(~ok, -math.inf)
+
+
 def route(s, correction, router):
     """One token: chosen experts and their weights."""
     choice = s + correction
     if router.get("groups"):
-        choice = choice.masked_fill(~allowed(choice, router["groups"]), -math.inf)
+        choice = closed(choice, allowed(choice, router["groups"]))
     e = torch.topk(choice, router["top"]).indices
     return e, s[e] / (s[e].sum() + 1e-20) * router.get("scale", 1.0)
 
