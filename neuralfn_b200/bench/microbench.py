@@ -474,14 +474,15 @@ def case_mixers(args):
     rep("latent_attention_tiles", lambda: Y.latent_attention_tiles(lc, ql, x, base, ltiles, out, heads=H, dim=D, vdim=D, window=W, scale=(D + R) ** -0.5),
         flops=2.0 * H * (2 * D + R) * win_keys, extra={"T": T, "window": W})
     spans, lat, wkvx = torch.tensor([[0, 0, T // 64, 0]], **i32), torch.empty(T, RANK, device=dev, dtype=torch.bfloat16), rand(2 * HD, RANK)
-    rep("latent_gather", lambda: Y.latent_gather(lc, spans, lat), bytes_=4.0 * T * RANK, extra={"T": T})
+    rep("latent_gather", lambda: Y.latent_gather(lc, spans, lat, T // 64), bytes_=4.0 * T * RANK, extra={"T": T})
     rep("gemm (expansion)", lambda: gemm(lat, wkvx, out=x), flops=4.0 * T * HD * RANK, extra={"T": T})
     # ---- rows between products and attention ----
     rt, freq, wn = P.row_tiles([(0, 0, T, 0)], dev), Y.frequencies(R, 1e4, dev), rand(D)
     hx = rand(T, (H + G) * D)
     rep("head_rows", lambda: Y.head_rows(c, hx, rt, hx, heads=H, dim=D, freq=freq, rot_dims=R, eps=1e-5, q_norm=wn, k_norm=wn, key_values=True), bytes_=2.0 * T * D * (2 * H + 3 * G), extra={"T": T})
     lx = rand(T, H * (D + R) + RANK + R)
-    rep("latent_rows", lambda: Y.latent_rows(lc, lx, rt, heads=H, dim=D, rot_dim=R, rank=RANK, c_norm=rand(RANK), eps=1e-5, freq=freq), bytes_=4.0 * T * (H * R + RANK + R), extra={"T": T})
+    cn = rand(RANK)
+    rep("latent_rows", lambda: Y.latent_rows(lc, lx, rt, heads=H, dim=D, rot_dim=R, rank=RANK, c_norm=cn, eps=1e-5, freq=freq), bytes_=4.0 * T * (H * R + RANK + R), extra={"T": T})
     mx, mq = rand(T, (H + 2 * G) * D + 2 * 4 * F), torch.empty(T, HD, device=dev, dtype=torch.bfloat16)
     cat = torch.empty(T, 4 * F, device=dev, dtype=torch.bfloat16)
     rep("mix_rows (no convolution)", lambda: P.mix_rows(c, mx, rt, mq, None, heads=H), bytes_=4.0 * T * (H + 2 * G) * D, extra={"T": T})
@@ -507,8 +508,10 @@ def case_mixers(args):
     rep("group_products (keys)", lambda: Y.group_products(qn[..., :D], wut, qa), bytes_=2.0 * (H * RANK * D + B * H * (RANK + D)), extra={"B": B})
     rep("group_products (values)", lambda: Y.group_products(oa, wuv, ov), bytes_=2.0 * (H * RANK * D + B * H * (RANK + D)), extra={"B": B})
     w4, x4, y4 = rand(4, HD, C), rand(4, B, C), torch.empty(B, 4, HD, device=dev, dtype=torch.bfloat16)
-    rep("group_products (r, k, v, gate)", lambda: Y.group_products(x4.transpose(0, 1), w4, y4), bytes_=8.0 * HD * C, extra={"B": B})
-    rep("gemm (same bytes)", lambda: gemm(x4[0], w4.view(4 * HD, C), out=y4.view(B, 4 * HD)), bytes_=8.0 * HD * C, extra={"B": B})
+    for b in sorted({1, min(8, B), min(16, B), B}):
+        rep("group_products (r, k, v, gate)", lambda: Y.group_products(x4[:, :b].transpose(0, 1), w4, y4[:b]), bytes_=8.0 * HD * C, extra={"B": b})
+        rep("gemm (one after another)", lambda: [gemm(x4[i, :b], w4[i], out=y4.view(4, B, HD)[i, :b]) for i in range(4)], bytes_=8.0 * HD * C, extra={"B": b})
+        rep("gemm (same bytes)", lambda: gemm(x4[0, :b], w4.view(4 * HD, C), out=y4.view(B, 4 * HD)[:b]), bytes_=8.0 * HD * C, extra={"B": b})
     del c, kc, vc, lc, w4
     # ---- time mixing ----
     u, w0 = rand(HD), torch.full((HD,), -1.0, device=dev).bfloat16()
@@ -545,6 +548,7 @@ def case_mixers(args):
     z, corr = torch.randn(T, E, device=dev), torch.zeros(E, device=dev).bfloat16()
     choice = dict(correction=corr, groups=8 if E % 8 == 0 else 0, keep=4, normalise=True, scale=1.5)
     rep("expert_choice", lambda: Y.expert_choice(z, 4, **choice), bytes_=4.0 * T * E + 32.0 * T, extra={"T": T})
+    rep("expert_choice (no groups)", lambda: Y.expert_choice(z, 4), bytes_=4.0 * T * E + 32.0 * T, extra={"T": T})
     up, down, wr = rand(E, F, C) * C ** -0.5, rand(E, C, F) * F ** -0.5, rand(E, C) * C ** -0.5
     wg = rand(E, 2 * F, C) * C ** -0.5
     mw = MoEWorkspace(T, E, 4, C, F, dev)

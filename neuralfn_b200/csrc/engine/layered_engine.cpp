@@ -32,6 +32,7 @@ using nfn_eng::efail;
 namespace {
 
 constexpr int kPage = NFN_KV_PAGE, kTileMin = 16, kMixRows = 16;
+constexpr int kFewRows = 32;                        // up to here several products of a layer run as one weight-streaming launch
 constexpr float kUnitEps = 1e-6f;                   // of the delta rule's unit vectors
 
 int up(int v, int m) { return (v + m - 1) / m * m; }
@@ -908,16 +909,17 @@ int layered_engine::wkv(const Layer& L, const Batch& b) {
   s.tiles = dev<nfn_row_tile>(io.mix); s.n_tiles = b.n_mix;
   K(nfn_shift_rows(&s, stream));
   auto mixed = [&](int i) { return static_cast<const char*>(shift) + (size_t)i * stride * es; };
-  if (!f32 && rows <= 32) {                              // r, k, v, gate in one launch
+  if (!f32 && rows <= kFewRows) {                        // r, k, v, gate and the inner decay projection in one launch
     nfn_group_products_args g{};
     g.rows = rows; g.groups = 4; g.n = nq; g.k = wp; g.in = shift; g.ld_in = wp; g.in_group = stride; g.w = L.w_in;
     g.out = in; g.ld_out = L.n_in; g.out_group = nq;
+    g.tail_n = L.ra; g.tail_in = 4 * stride; g.tail_w = L.w1; g.tail_out = low; g.ld_tail = L.ra;
     K(nfn_group_products(&g, stream));
   } else {
     for (int i = 0; i < 4; ++i)
       if (lin(mixed(i), wp, static_cast<const char*>(L.w_in) + 2LL * i * nq * wp, rows, nq, wp, static_cast<char*>(in) + (size_t)i * nq * es, L.n_in, kOutAct)) return -1;
+    if (lin(mixed(4), wp, L.w1, rows, L.ra, wp, low, L.ra, kOutF32)) return -1;
   }
-  if (lin(mixed(4), wp, L.w1, rows, L.ra, wp, low, L.ra, kOutF32)) return -1;
   if (wkv_step(L, b)) {
     nfn_wkv_step_args t{};
     t.f32 = f32; t.rows = rows; t.rkvg = in; t.ld_rkvg = L.n_in; t.low = low; t.ld_low = t.rank_p = L.ra; t.w2 = L.w2; t.ld_w2 = 2 * L.ra;
@@ -970,24 +972,29 @@ int layered_engine::dense_ff(const Layer& L, int rows) {
 // Routed experts on the normalised rows h; says in `sp` where the next stream pass finds each row's outputs.
 int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
   const nfn_layer_desc& d = L.d;
-  if (lin(h, wp, L.router, rows, L.ep, wp, ex.logits, L.ep, kOutF32)) return -1;
+  const bool few = !grouped(L, rows), shared = d.shared_ff > 0;
+  if (shared && c.dtype == 0 && rows <= kFewRows) {        // router and the shared expert's first product in one launch
+    nfn_group_products_args g{};
+    g.rows = rows; g.groups = 1; g.n = L.shp; g.k = wp; g.in = h; g.ld_in = wp; g.w = L.w_shared_up; g.out = shared_mid; g.ld_out = L.shp; g.act = d.ff_act;
+    g.tail_n = L.ep; g.tail_w = L.router; g.tail_out = ex.logits; g.ld_tail = L.ep;
+    K(nfn_group_products(&g, stream));
+  } else if (lin(h, wp, L.router, rows, L.ep, wp, ex.logits, L.ep, kOutF32) || (shared && lin(h, wp, L.w_shared_up, rows, L.shp, wp, shared_mid, L.shp, kOutAct, nullptr, d.ff_act))) {
+    return -1;
+  }
+  if (shared && !few && lin(shared_mid, L.shp, L.w_shared_down, rows, wp, L.shp, y_shared, wp, kOutAct)) return -1;
   sp->y = ex.y;
   sp->y_rows = d.top;
   sp->y_item = d.expert_plain ? ex.weight : nullptr;
-  if (d.shared_ff > 0) {
-    if (lin(h, wp, L.w_shared_up, rows, L.shp, wp, shared_mid, L.shp, kOutAct, nullptr, d.ff_act) ||
-        lin(shared_mid, L.shp, L.w_shared_down, rows, wp, L.shp, y_shared, wp, kOutAct))
-      return -1;
-    sp->y_plus = y_shared;
-  }
+  sp->y_plus = shared ? y_shared : nullptr;
   nfn_route_rule rule{};
   rule.correction = L.correction; rule.groups = d.route_groups; rule.keep_groups = d.route_keep; rule.normalise = d.route_normalise; rule.scale = d.route_scale;
-  if (!grouped(L, rows)) {
+  if (few) {
     nfn_moe_rows_args a{};
     a.f32 = c.dtype == 1; a.rows = rows; a.width = wp; a.ff = L.ef; a.experts = d.experts; a.top = d.top; a.act = d.ff_act;
     a.logits = ex.logits; a.ld_logits = L.ep; a.h = h; a.ld_h = wp; a.w_gate_up = L.w_gate_up; a.w_down = L.w_down;
     a.idx = ex.idx; a.weight = ex.weight; a.order = ex.order; a.offsets = ex.offsets; a.active = ex.active;
     a.mid = ex.mid; a.y = ex.y; a.ld_y = wp; a.plain = d.expert_plain; a.rule = rule;
+    if (shared) { a.shared_ff = L.shp; a.shared_mid = shared_mid; a.w_shared_down = L.w_shared_down; a.y_shared = y_shared; }
     K(nfn_moe_rows(&a, stream));
     sp->y_index = nullptr;
     return 0;

@@ -127,42 +127,57 @@ head_rows_kernel(const nfn_head_rows_args p) {
   }
 }
 
-// A warp takes one query head, or the latent and shared key part, of all rows of a tile.
+// A warp takes the rotated part of one query head over the tile's rows; the CTAs of the last column take latents and shared key parts, a row per warp.
 template <typename T, int NV>
 __global__ void __launch_bounds__(HR_THREADS)
 latent_rows_kernel(const nfn_latent_rows_args p) {
   extern __shared__ float2 hr_cs[];
   const nfn_row_tile t = p.tiles[blockIdx.x];
-  if (t.slot < 0) return;
+  const bool of_keys = blockIdx.y == gridDim.y - 1;
+  if (t.slot < 0 || (of_keys && !p.k_pool)) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dim / 2;
   const int pos0 = t.e_pos0 + t.row0 - t.e_row0;
   fill_rotations(hr_cs, p.freq, half, pos0, t.n);
-  __syncthreads();
-  const int item = blockIdx.y * HR_WARPS + warp, pitch = p.dim_p + p.rot_p, lp = p.rank_p + p.rot_p;
+  const int pitch = p.dim_p + p.rot_p, lp = p.rank_p + p.rot_p;
   const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
-  if (item < p.heads) {
-    const bool lat = t.row0 < p.q_row0;                    // rows of an entry are all short or all long
-    const T* src = in + item * pitch;
-    T* dst = lat ? static_cast<T*>(p.q_lat) + (size_t)t.row0 * p.heads * lp + (size_t)item * lp + p.rank_p
-                 : static_cast<T*>(p.q_out) + (size_t)t.row0 * p.ld_q + item * pitch + p.dim_p;
+  if (!of_keys) {
+    const int head = blockIdx.y * HR_WARPS + warp;
+    const bool lat = t.row0 < p.q_row0, on = head < p.heads;    // rows of an entry are all short or all long
+    const T* src = in + (on ? head : 0) * pitch;
+    T* dst = lat ? static_cast<T*>(p.q_lat) + (size_t)t.row0 * p.heads * lp + (size_t)head * lp + p.rank_p
+                 : static_cast<T*>(p.q_out) + (size_t)t.row0 * p.ld_q + head * pitch + p.dim_p;
     const size_t ld_dst = lat ? (size_t)p.heads * lp : (size_t)p.ld_q;
-    // pieces of four over the tile's rows: narrow rotated parts leave no lane idle
-    const int quads = p.rot_p / 4;
-    for (int x = lane; x < quads * t.n; x += 32) {
-      const int i = x / quads, c = x % quads * 4;
-      store4(dst + i * ld_dst + c, rotate4(load4(src + (size_t)i * p.ld_in + p.dim_p + c), hr_cs + i * half, c, p.rot_dim));
+    // pieces of four over the tile's rows, four per lane in flight: narrow rotated parts leave no lane idle
+    const int quads = p.rot_p / 4, total = on ? quads * t.n : 0;
+    float4 v[4];
+    auto fetch = [&](int x0) {
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int x = x0 + 32 * e;
+        if (x < total) v[e] = load4(src + (size_t)(x / quads) * p.ld_in + p.dim_p + x % quads * 4);
+      }
+    };
+    fetch(lane);
+    __syncthreads();
+    for (int x0 = lane; x0 < total; x0 += 128) {
+      if (x0 != lane) fetch(x0);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int x = x0 + 32 * e, i = x / quads, c = x % quads * 4;
+        if (x < total) store4(dst + i * ld_dst + c, rotate4(v[e], hr_cs + i * half, c, p.rot_dim));
+      }
     }
-    if (!lat && p.q_out != p.in)
+    if (on && !lat && p.q_out != p.in)
       for (int i = 0; i < t.n; ++i)
         for (int c = lane * 4; c < p.dim_p; c += 128) store4(dst + i * ld_dst - p.dim_p + c, load4(src + (size_t)i * p.ld_in + c));
     return;
   }
-  if (item > p.heads || !p.k_pool) return;
+  __syncthreads();
   const size_t page = (size_t)p.table[(size_t)t.slot * p.table_ld + pos0 / NFN_PAGE];
   T* dst = static_cast<T*>(p.k_pool) + (page * NFN_PAGE + pos0 % NFN_PAGE) * lp;
   const T* src = in + p.off_kv;
   const __nv_bfloat16* weight = static_cast<const __nv_bfloat16*>(p.c_norm);
-  for (int i = 0; i < t.n; ++i) {
+  for (int i = warp; i < t.n; i += HR_WARPS) {
     const T* row = src + (size_t)i * p.ld_in;
     float4 v[NV];
     float ss = 0.f;
@@ -170,8 +185,9 @@ latent_rows_kernel(const nfn_latent_rows_args p) {
     for (int j = 0; j < NV; ++j) {
       const int c = lane * 4 + j * 128;
       v[j] = c < p.rank_p ? load4(row + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-      ss += squares(v[j]);
     }
+#pragma unroll
+    for (int j = 0; j < NV; ++j) ss += squares(v[j]);
     for (int c = lane * 4 + NV * 128; c < p.rank_p; c += 128) ss += squares(load4(row + c));
     const float r = 1.f / sqrtf(warp_sum(ss) / (float)p.rank + p.eps);
     auto leave = [&](const float4& f, int c) {
@@ -194,9 +210,10 @@ constexpr int GP_WARPS = 8, GP_ROWS = 8;
 __global__ void __launch_bounds__(GP_WARPS * 32)
 group_products_f32_kernel(const nfn_group_products_args p) {
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n = blockIdx.x * GP_WARPS + warp, g = blockIdx.y, r0 = blockIdx.z * GP_ROWS;
-  if (n >= p.n) return;
-  const __nv_bfloat16* w = static_cast<const __nv_bfloat16*>(p.w) + ((size_t)g * p.n + n) * p.k;
-  const float* in = static_cast<const float*>(p.in) + (size_t)r0 * p.ld_in + (size_t)g * p.in_group;
+  const bool tail = g == p.groups;
+  if (n >= (tail ? p.tail_n : p.n)) return;
+  const __nv_bfloat16* w = tail ? static_cast<const __nv_bfloat16*>(p.tail_w) + (size_t)n * p.k : static_cast<const __nv_bfloat16*>(p.w) + ((size_t)g * p.n + n) * p.k;
+  const float* in = static_cast<const float*>(p.in) + (size_t)r0 * p.ld_in + (tail ? (size_t)p.tail_in : (size_t)g * p.in_group);
   const int live = min(GP_ROWS, p.rows - r0);
   float a[GP_ROWS];
 #pragma unroll
@@ -210,12 +227,12 @@ group_products_f32_kernel(const nfn_group_products_args p) {
       a[i] += (f.x * x.x + f.y * x.y) + (f.z * x.z + f.w * x.w);
     }
   }
-  float* out = static_cast<float*>(p.out) + (size_t)r0 * p.ld_out + (size_t)g * p.out_group + n;
+  float* out = tail ? p.tail_out + (size_t)r0 * p.ld_tail + n : static_cast<float*>(p.out) + (size_t)r0 * p.ld_out + (size_t)g * p.out_group + n;
 #pragma unroll
   for (int i = 0; i < GP_ROWS; ++i) {
     if (i >= live) break;
     const float s = warp_sum(a[i]);
-    if (lane == 0) out[(size_t)i * p.ld_out] = s;
+    if (lane == 0) out[(size_t)i * (tail ? p.ld_tail : p.ld_out)] = tail ? s : ff_act(s, p.act);
   }
 }
 
@@ -237,12 +254,14 @@ __device__ __forceinline__ void gm_mma(float (&d)[4], uint32_t a0, uint32_t a1, 
 template <int NT>
 __global__ void __launch_bounds__(GM_WARPS * 32)
 group_products_mma_kernel(const nfn_group_products_args p) {
-  constexpr int M = 8 * NT, U = NT == 4 ? 2 : 4;          // rows at a time, 32-wide steps in flight
+  constexpr int M = 8 * NT, U = NT == 4 ? 1 : 2;          // rows at a time; 32-wide steps per set, two sets in flight
   __shared__ float part[GM_WARPS][32][M + 1];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, j = lane & 3, g = blockIdx.y;
-  const int n0 = blockIdx.x * 32, r0 = blockIdx.z * M;
-  const bool two = n0 + 16 < p.n;
-  const __nv_bfloat16* w0 = static_cast<const __nv_bfloat16*>(p.w) + ((size_t)g * p.n + n0 + gr) * p.k + 8 * j;
+  const bool tail = g == p.groups;
+  const int n0 = blockIdx.x * 32, r0 = blockIdx.z * M, N = tail ? p.tail_n : p.n;
+  if (n0 >= N) return;
+  const bool two = n0 + 16 < N;
+  const __nv_bfloat16* w0 = (tail ? static_cast<const __nv_bfloat16*>(p.tail_w) : static_cast<const __nv_bfloat16*>(p.w) + (size_t)g * p.n * p.k) + (size_t)(n0 + gr) * p.k + 8 * j;
   const __nv_bfloat16* w1 = two ? w0 + (size_t)16 * p.k : w0;
   const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
   const __nv_bfloat16* src[NT];
@@ -251,7 +270,7 @@ group_products_mma_kernel(const nfn_group_products_args p) {
   for (int t = 0; t < NT; ++t) {
     const int r = r0 + 8 * t + gr;
     on[t] = r < p.rows;
-    src[t] = static_cast<const __nv_bfloat16*>(p.in) + (size_t)(on[t] ? r : r0) * p.ld_in + (size_t)g * p.in_group + 8 * j;
+    src[t] = static_cast<const __nv_bfloat16*>(p.in) + (size_t)(on[t] ? r : r0) * p.ld_in + (tail ? (size_t)p.tail_in : (size_t)g * p.in_group) + 8 * j;
   }
   float acc[2][NT][4];
 #pragma unroll
@@ -261,28 +280,38 @@ group_products_mma_kernel(const nfn_group_products_args p) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) acc[m][t][c] = 0.f;
   const int steps = (p.k + 31) / 32, s0 = steps * warp / GM_WARPS, s1 = steps * (warp + 1) / GM_WARPS;
-  for (int s = s0; s < s1; s += U) {
-    uint4 a[U][4], b[U][NT];
+  uint4 a[2][U][4], b[2][U][NT];
+  auto fetch = [&](int s, uint4 (&fa)[U][4], uint4 (&fb)[U][NT]) {
 #pragma unroll
     for (int u = 0; u < U; ++u) {
       const int k = (s + u) * 32;
       const bool ok = s + u < s1 && k + 8 * j < p.k;
-      a[u][0] = ok ? gm_stream(w0 + k) : zero4;
-      a[u][1] = ok ? gm_stream(w0 + (size_t)8 * p.k + k) : zero4;
-      a[u][2] = ok ? gm_stream(w1 + k) : zero4;
-      a[u][3] = ok ? gm_stream(w1 + (size_t)8 * p.k + k) : zero4;
+      fa[u][0] = ok ? gm_stream(w0 + k) : zero4;
+      fa[u][1] = ok ? gm_stream(w0 + (size_t)8 * p.k + k) : zero4;
+      fa[u][2] = ok ? gm_stream(w1 + k) : zero4;
+      fa[u][3] = ok ? gm_stream(w1 + (size_t)8 * p.k + k) : zero4;
 #pragma unroll
-      for (int t = 0; t < NT; ++t) b[u][t] = ok && on[t] ? *reinterpret_cast<const uint4*>(src[t] + k) : zero4;
+      for (int t = 0; t < NT; ++t) fb[u][t] = ok && on[t] ? *reinterpret_cast<const uint4*>(src[t] + k) : zero4;
     }
+  };
+  auto use = [&](const uint4 (&fa)[U][4], const uint4 (&fb)[U][NT]) {
 #pragma unroll
     for (int u = 0; u < U; ++u)
 #pragma unroll
       for (int t = 0; t < NT; ++t) {
-        gm_mma(acc[0][t], a[u][0].x, a[u][1].x, a[u][0].y, a[u][1].y, b[u][t].x, b[u][t].y);
-        gm_mma(acc[1][t], a[u][2].x, a[u][3].x, a[u][2].y, a[u][3].y, b[u][t].x, b[u][t].y);
-        gm_mma(acc[0][t], a[u][0].z, a[u][1].z, a[u][0].w, a[u][1].w, b[u][t].z, b[u][t].w);
-        gm_mma(acc[1][t], a[u][2].z, a[u][3].z, a[u][2].w, a[u][3].w, b[u][t].z, b[u][t].w);
+        gm_mma(acc[0][t], fa[u][0].x, fa[u][1].x, fa[u][0].y, fa[u][1].y, fb[u][t].x, fb[u][t].y);
+        gm_mma(acc[1][t], fa[u][2].x, fa[u][3].x, fa[u][2].y, fa[u][3].y, fb[u][t].x, fb[u][t].y);
+        gm_mma(acc[0][t], fa[u][0].z, fa[u][1].z, fa[u][0].w, fa[u][1].w, fb[u][t].z, fb[u][t].w);
+        gm_mma(acc[1][t], fa[u][2].z, fa[u][3].z, fa[u][2].w, fa[u][3].w, fb[u][t].z, fb[u][t].w);
       }
+  };
+  fetch(s0, a[0], b[0]);
+  fetch(s0 + U, a[1], b[1]);
+  for (int s = s0; s < s1; s += 2 * U) {
+    use(a[0], b[0]);
+    fetch(s + 2 * U, a[0], b[0]);
+    use(a[1], b[1]);
+    fetch(s + 3 * U, a[1], b[1]);
   }
 #pragma unroll
   for (int m = 0; m < 2; ++m)
@@ -294,23 +323,26 @@ group_products_mma_kernel(const nfn_group_products_args p) {
   const int live = min(M, p.rows - r0);
   for (int x = threadIdx.x; x < 32 * live; x += GM_WARPS * 32) {
     const int col = x / 32, row = x % 32;
-    if (n0 + row >= p.n) continue;
+    if (n0 + row >= N) continue;
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < GM_WARPS; ++w) v += part[w][row][col];
-    static_cast<__nv_bfloat16*>(p.out)[(size_t)(r0 + col) * p.ld_out + (size_t)g * p.out_group + n0 + row] = __float2bfloat16(v);
+    if (tail) p.tail_out[(size_t)(r0 + col) * p.ld_tail + n0 + row] = v;
+    else static_cast<__nv_bfloat16*>(p.out)[(size_t)(r0 + col) * p.ld_out + (size_t)g * p.out_group + n0 + row] = __float2bfloat16(ff_act(v, p.act));
   }
 }
 
-// one CTA per page: 64 rows of `vecs` 16-byte pieces
+// a quarter of a page per CTA: 16 rows of `vecs` 16-byte pieces
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const uint4* __restrict__ pool, int ld_pool, int vecs, const int* __restrict__ table, int table_ld, const nfn_latent_span* __restrict__ spans,
                      uint4* __restrict__ out) {
   const nfn_latent_span s = spans[blockIdx.y];
-  if (s.slot < 0 || (int)blockIdx.x >= s.n_pages) return;
-  const uint4* src = pool + (size_t)table[(size_t)s.slot * table_ld + s.first_page + blockIdx.x] * NFN_PAGE * ld_pool;
-  uint4* dst = out + ((size_t)s.row0 + (size_t)blockIdx.x * NFN_PAGE) * vecs;
-  for (int i = threadIdx.x; i < NFN_PAGE * vecs; i += 256) dst[i] = src[(size_t)(i / vecs) * ld_pool + i % vecs];
+  const int page = blockIdx.x / 4, r0 = blockIdx.x % 4 * 16;
+  if (s.slot < 0 || page >= s.n_pages) return;
+  const uint4* src = pool + ((size_t)table[(size_t)s.slot * table_ld + s.first_page + page] * NFN_PAGE + r0) * ld_pool;
+  uint4* dst = out + ((size_t)s.row0 + (size_t)page * NFN_PAGE + r0) * vecs;
+#pragma unroll 4
+  for (int i = threadIdx.x; i < 16 * vecs; i += 256) dst[i] = src[(size_t)(i / vecs) * ld_pool + i % vecs];
 }
 
 template <typename T>
@@ -325,7 +357,7 @@ static int launch_head_rows(const nfn_head_rows_args& a, cudaStream_t st) {
 
 template <typename T>
 static int launch_latent_rows(const nfn_latent_rows_args& a, cudaStream_t st) {
-  const dim3 grid(a.n_tiles, ceil_div(a.heads + 1, HR_WARPS));
+  const dim3 grid(a.n_tiles, ceil_div(a.heads, HR_WARPS) + 1);
   const size_t smem = (size_t)std::max(1, a.tile_rows * (a.rot_dim / 2)) * sizeof(float2);
   latent_rows_kernel<T, 4><<<grid, HR_THREADS, smem, st>>>(a);
   return launch_check("latent_rows");
@@ -367,10 +399,12 @@ extern "C" int nfn_group_products(const nfn_group_products_args* args, nfn_strea
   if (a.groups <= 0 || a.groups > 65535 || ((a.n | a.k) & 15) || a.n <= 0 || a.k <= 0 || ((a.ld_in | a.in_group) & 7)) return fail(-1, "group_products: sizes must be multiples of 16");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   if (ceil_div(a.rows, 8) > 65535) return fail(-1, "group_products: too many rows in one launch");
-  if (a.f32) group_products_f32_kernel<<<dim3(ceil_div(a.n, GP_WARPS), a.groups, ceil_div(a.rows, GP_ROWS)), GP_WARPS * 32, 0, st>>>(a);
-  else if (a.rows <= 8) group_products_mma_kernel<1><<<dim3(ceil_div(a.n, 32), a.groups, 1), GM_WARPS * 32, 0, st>>>(a);
-  else if (a.rows <= 16) group_products_mma_kernel<2><<<dim3(ceil_div(a.n, 32), a.groups, 1), GM_WARPS * 32, 0, st>>>(a);
-  else group_products_mma_kernel<4><<<dim3(ceil_div(a.n, 32), a.groups, ceil_div(a.rows, 32)), GM_WARPS * 32, 0, st>>>(a);
+  if (a.tail_n < 0 || (a.tail_n > 0 && (!a.tail_w || !a.tail_out || (a.tail_in & 7)))) return fail(-1, "group_products: the tail product lacks an operand");
+  const int n = std::max(a.n, a.tail_n), g = a.groups + (a.tail_n > 0 ? 1 : 0);
+  if (a.f32) group_products_f32_kernel<<<dim3(ceil_div(n, GP_WARPS), g, ceil_div(a.rows, GP_ROWS)), GP_WARPS * 32, 0, st>>>(a);
+  else if (a.rows <= 8) group_products_mma_kernel<1><<<dim3(ceil_div(n, 32), g, 1), GM_WARPS * 32, 0, st>>>(a);
+  else if (a.rows <= 16) group_products_mma_kernel<2><<<dim3(ceil_div(n, 32), g, 1), GM_WARPS * 32, 0, st>>>(a);
+  else group_products_mma_kernel<4><<<dim3(ceil_div(n, 32), g, ceil_div(a.rows, 32)), GM_WARPS * 32, 0, st>>>(a);
   return launch_check("group_products");
 }
 
@@ -379,7 +413,7 @@ extern "C" int nfn_latent_gather(int f32, const void* pool, int ld_pool, int col
   if (n_spans <= 0 || max_pages <= 0) return 0;
   const int per = f32 ? 4 : 8;
   if (ld_pool % per || cols % per || n_spans > 65535) return fail(-1, "latent_gather: rows of 16-byte pieces, at most 65535 spans");
-  latent_gather_kernel<<<dim3(max_pages, n_spans), 256, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const uint4*>(pool), ld_pool / per, cols / per, table, table_ld,
+  latent_gather_kernel<<<dim3(4 * max_pages, n_spans), 256, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const uint4*>(pool), ld_pool / per, cols / per, table, table_ld,
                                                                                                  spans, static_cast<uint4*>(out));
   return launch_check("latent_gather");
 }

@@ -3,9 +3,10 @@
 // projection follows, so a token's row is read once for all heads and twice from shared memory: as the key operand and, transposed by
 // ldmatrix, as the value operand.
 //
-// One CTA takes one row, a block of 16 or 32 heads and a share of the visible pages. Per page: eight warps form the scores (16 keys x half of the
+// One CTA takes one row, a block of 16 or 32 heads and a share of the visible pages. Per page: sixteen warps form the scores (8 keys x half of the
 // channels each, on mma.m16n8k16), a softmax pass merges the halves, then each warp owns a slice of the latent channels of the output.
-// Pages arrive by cp.async one ahead. Scores, softmax and sums are fp32; shares are merged in a fixed order by the CTA that finishes last.
+// Pages arrive one ahead, a bulk copy per row (rows in shared memory are 16 bytes longer than in the page: no bank conflicts). Scores, softmax
+// and sums are fp32; a second launch merges the shares, in order.
 #include <algorithm>
 
 #include "common.h"
@@ -13,14 +14,14 @@
 
 namespace nfn {
 
-constexpr int LD_WARPS = 8, LD_THREADS = LD_WARPS * 32, LD_S = NFN_PAGE + 4, LD_P = NFN_PAGE + 8;
-constexpr int LD_COUNTERS = PAGED_COUNTER_BYTES / 4;
+constexpr int LD_WARPS = 16, LD_THREADS = LD_WARPS * 32, LD_S = NFN_PAGE + 4, LD_P = NFN_PAGE + 8;
 
 struct LatentDecodeParams {
   nfn_paged_attention_args a;
   int splits, pitch;           // pitch: elements between rows in shared memory (an odd number of 16-byte pieces: no bank conflicts)
-  int* counters;               // [rows][head blocks]
-  float* partial;              // [rows][head blocks][splits][heads of a block][vdim_p + 2]: values, maximum, sum
+  float* partial;              // [rows][heads][splits][vdim_p] values
+  float2* stats;               // [rows][heads][splits] maximum and sum
+  int* status;
 };
 
 __device__ __forceinline__ void ld_x4(uint32_t (&r)[4], uint32_t addr) {
@@ -34,8 +35,8 @@ __device__ __forceinline__ void ld_mma(float (&d)[4], const uint32_t (&a)[4], ui
                : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
                : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
-__device__ __forceinline__ void ld_copy16(uint32_t dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
+__device__ __forceinline__ void ld_bulk(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
 }
 
 // MT: 16-head tiles of a CTA; VN: 8-channel tiles of the output per warp (an upper bound)
@@ -45,7 +46,8 @@ latent_decode_kernel(const LatentDecodeParams p) {
   constexpr int NH = MT * 16;
   extern __shared__ __align__(16) unsigned char ld_smem[];
   __shared__ float s_alpha[NH], s_m[NH], s_l[NH];
-  __shared__ int sh_last;
+  __shared__ __align__(8) uint64_t bar_full[2];
+  __shared__ int abort_s;
   const nfn_paged_attention_args& a = p.a;
   const int row = a.row0 + blockIdx.z, slot = a.row_slot[row];
   if (slot < 0) return;
@@ -62,16 +64,22 @@ latent_decode_kernel(const LatentDecodeParams p) {
   const int* table = a.table + (size_t)slot * a.table_ld;
   const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a.k_pool);
   const int vecs = DP / 8;
-  auto load = [&](int i) {
+  auto load = [&](int i) {                                       // warp 0: two rows per lane
+    const uint32_t bar = smem_u32(&bar_full[i & 1]), dst = smem_u32(sK + (size_t)(i & 1) * NFN_PAGE * pitch);
     const __nv_bfloat16* src = pool + (size_t)table[page0 + i] * NFN_PAGE * DP;
-    const uint32_t dst = smem_u32(sK + (size_t)(i & 1) * NFN_PAGE * pitch);
-    for (int x = tid; x < NFN_PAGE * vecs; x += LD_THREADS) {
-      const int r = x / vecs, c = x - r * vecs;
-      ld_copy16(dst + (uint32_t)(r * pitch + c * 8) * 2, src + (size_t)x * 8);
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
+    if (lane == 0) mbar_expect_tx(bar, (uint32_t)(NFN_PAGE * DP * 2));
+    __syncwarp();
+#pragma unroll
+    for (int r = lane; r < NFN_PAGE; r += 32) ld_bulk(dst + (uint32_t)(r * pitch) * 2, src + (size_t)r * DP, (uint32_t)DP * 2, bar);
   };
-  if (p_lo < p_hi) load(p_lo);
+  if (tid == 0) {
+    abort_s = 0;
+    mbar_init(smem_u32(&bar_full[0]), 1);
+    mbar_init(smem_u32(&bar_full[1]), 1);
+    fence_mbar_init();
+  }
+  __syncthreads();
+  if (warp == 0 && p_lo < p_hi) load(p_lo);
   {
     const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + (size_t)row * a.ld_q + (size_t)h0 * DP;
     const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
@@ -92,51 +100,47 @@ latent_decode_kernel(const LatentDecodeParams p) {
     for (int v = 0; v < VN; ++v)
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[m][v][e] = 0.f;
-  const int kg = warp & 3, half = warp >> 2, steps = DP / 16, ks0 = steps * half / 2, ks1 = steps * (half + 1) / 2;
+  const int kg = warp & 7, half = warp >> 3, steps = DP / 16, ks0 = steps * half / 2, ks1 = steps * (half + 1) / 2;
   const uint32_t aq = smem_u32(sQ) + (uint32_t)((lane & 15) * pitch + (lane >> 4) * 8) * 2;
   const uint32_t ap = smem_u32(sP) + (uint32_t)((lane & 15) * LD_P + (lane >> 4) * 8) * 2;
-  const uint32_t bk = (uint32_t)((kg * 16 + (lane >> 4) * 8 + (lane & 7)) * pitch + ((lane >> 3) & 1) * 8) * 2;
+  const uint32_t bk = (uint32_t)((kg * 8 + (lane & 7)) * pitch + (lane >> 3) * 8) * 2;
   const uint32_t bv = (uint32_t)((((lane >> 3) & 1) * 8 + (lane & 7)) * pitch + warp * VN * 8 + (lane >> 4) * 8) * 2;
 
+  __syncthreads();                                                  // queries are in place
   for (int i = p_lo; i < p_hi; ++i) {
-    if (i + 1 < p_hi) {
-      load(i + 1);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
-    }
-    __syncthreads();
+    if (warp == 0 && i + 1 < p_hi) load(i + 1);
+    mbar_wait_bounded(smem_u32(&bar_full[i & 1]), ((i - p_lo) >> 1) & 1, &abort_s, p.status, NFN_ERR_WAIT_FULL);
     const uint32_t stage = smem_u32(sK + (size_t)(i & 1) * NFN_PAGE * pitch);
-    // ---- scores: 16 keys, half of the channels ----
-    float s[MT][2][4];
+    // ---- scores: 8 keys, half of the channels, two steps of 16 per load of keys ----
+    float s[MT][4];
 #pragma unroll
     for (int m = 0; m < MT; ++m)
 #pragma unroll
-      for (int t = 0; t < 2; ++t)
-#pragma unroll
-        for (int e = 0; e < 4; ++e) s[m][t][e] = 0.f;
+      for (int e = 0; e < 4; ++e) s[m][e] = 0.f;
 #pragma unroll 3
-    for (int k = ks0; k < ks1; ++k) {
+    for (int k = ks0; k < ks1; k += 2) {
       uint32_t b[4], q[MT][4];
       ld_x4(b, stage + bk + k * 32);
 #pragma unroll
       for (int m = 0; m < MT; ++m) ld_x4(q[m], aq + (uint32_t)(m * 16 * pitch) * 2 + k * 32);
 #pragma unroll
-      for (int m = 0; m < MT; ++m) {
-        ld_mma(s[m][0], q[m], b[0], b[1]);
-        ld_mma(s[m][1], q[m], b[2], b[3]);
+      for (int m = 0; m < MT; ++m) ld_mma(s[m], q[m], b[0], b[1]);
+      if (k + 1 < ks1) {
+#pragma unroll
+        for (int m = 0; m < MT; ++m) ld_x4(q[m], aq + (uint32_t)(m * 16 * pitch) * 2 + k * 32 + 32);
+#pragma unroll
+        for (int m = 0; m < MT; ++m) ld_mma(s[m], q[m], b[2], b[3]);
       }
     }
 #pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int t = 0; t < 2; ++t) {
-        float* dst = sS + (size_t)(half * NH + m * 16 + g) * LD_S + kg * 16 + t * 8 + 2 * j;
-        *reinterpret_cast<float2*>(dst) = make_float2(s[m][t][0], s[m][t][1]);
-        *reinterpret_cast<float2*>(dst + 8 * LD_S) = make_float2(s[m][t][2], s[m][t][3]);
-      }
+    for (int m = 0; m < MT; ++m) {
+      float* dst = sS + (size_t)(half * NH + m * 16 + g) * LD_S + kg * 8 + 2 * j;
+      *reinterpret_cast<float2*>(dst) = make_float2(s[m][0], s[m][1]);
+      *reinterpret_cast<float2*>(dst + 8 * LD_S) = make_float2(s[m][2], s[m][3]);
+    }
     __syncthreads();
-    // ---- softmax: 256 / NH threads per head, 64 NH / 256 keys each ----
+    if (*static_cast<volatile int*>(&abort_s)) break;               // a wait ran out: set before the barrier, so all leave together
+    // ---- softmax: LD_THREADS / NH threads per head, a few keys each ----
     {
       constexpr int SHARE = LD_THREADS / NH, KEYS = NFN_PAGE / SHARE;
       const int h = tid / SHARE, k0 = tid % SHARE * KEYS, key0 = (page0 + i) * NFN_PAGE + k0;
@@ -198,10 +202,13 @@ latent_decode_kernel(const LatentDecodeParams p) {
     __syncthreads();                                                // the stage takes the page after the next
   }
   __syncthreads();
+  if (abort_s) {
+    for (int i = 0; i < 64; ++i) __nanosleep(1000);                 // copies in flight land
+    return;
+  }
 
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (size_t)row * a.ld_o + (size_t)h0 * VP;
-  const size_t cell = (size_t)blockIdx.z * gridDim.y + blockIdx.y;
-  float* part = p.partial + (cell * p.splits + blockIdx.x) * NH * (VP + 2);
+  const size_t cell = (size_t)blockIdx.z * a.heads + h0;
 #pragma unroll
   for (int m = 0; m < MT; ++m)
 #pragma unroll
@@ -209,45 +216,56 @@ latent_decode_kernel(const LatentDecodeParams p) {
       const int h = m * 16 + g + 8 * e2;
       const float inv = s_l[h] > 0.f ? 1.f / s_l[h] : 0.f;
       if (h >= n_heads) continue;
+      float* part = p.partial + ((cell + h) * p.splits + blockIdx.x) * VP;
 #pragma unroll
       for (int v = 0; v < VN; ++v) {
         const int c = (warp * VN + v) * 8 + 2 * j;
         if (c >= VP) break;
         if (p.splits == 1) *reinterpret_cast<uint32_t*>(out + (size_t)h * VP + c) = pack_bf16x2(acc[m][v][2 * e2] * inv, acc[m][v][2 * e2 + 1] * inv);
-        else *reinterpret_cast<float2*>(part + (size_t)h * (VP + 2) + c) = make_float2(acc[m][v][2 * e2], acc[m][v][2 * e2 + 1]);
+        else *reinterpret_cast<float2*>(part + c) = make_float2(acc[m][v][2 * e2], acc[m][v][2 * e2 + 1]);
       }
-      if (p.splits > 1 && warp == 0 && j == 0) {
-        part[(size_t)h * (VP + 2) + VP] = s_m[h];
-        part[(size_t)h * (VP + 2) + VP + 1] = s_l[h];
-      }
+      if (p.splits > 1 && warp == 0 && j == 0) p.stats[(cell + h) * p.splits + blockIdx.x] = make_float2(s_m[h], s_l[h]);
     }
-  if (p.splits == 1) return;
-  __threadfence();
-  __syncthreads();
-  if (tid == 0) sh_last = atomicAdd(&p.counters[cell], 1) == p.splits - 1;
-  __syncthreads();
-  if (!sh_last) return;
-  __threadfence();
-  const float* all = p.partial + cell * p.splits * NH * (VP + 2);
-  const size_t step = (size_t)NH * (VP + 2);
-  for (int x = tid; x < n_heads * (VP / 2); x += LD_THREADS) {
-    const int h = x / (VP / 2), c = 2 * (x % (VP / 2));
-    const float* q = all + (size_t)h * (VP + 2);
-    float mx = -INFINITY;
-    for (int s2 = 0; s2 < p.splits; ++s2) mx = fmaxf(mx, __ldcg(q + s2 * step + VP));
-    float o0 = 0.f, o1 = 0.f, sum = 0.f;
-    for (int s2 = 0; s2 < p.splits; ++s2) {
-      const float* r = q + s2 * step;
-      const float f = exp2f(__ldcg(r + VP) - mx);
-      const float2 v = __ldcg(reinterpret_cast<const float2*>(r + c));
-      o0 += f * v.x;
-      o1 += f * v.y;
-      sum += f * __ldcg(r + VP + 1);
+}
+
+// A CTA takes one head of a row, a thread four channels.
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const LatentDecodeParams p) {
+  const nfn_paged_attention_args& a = p.a;
+  const int row = a.row0 + blockIdx.y, h = blockIdx.x, c = threadIdx.x * 4;
+  if (a.row_slot[row] < 0 || c >= a.vdim_p) return;
+  const size_t cell = (size_t)blockIdx.y * a.heads + h;
+  const float2* stats = p.stats + cell * p.splits;
+  const float* part = p.partial + cell * p.splits * a.vdim_p + c;
+  float m = -INFINITY, l = 0.f;
+  float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int s0 = 0; s0 < p.splits; s0 += 8) {
+    float2 t[8];
+    float4 v[8];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const int s = min(s0 + i, p.splits - 1);
+      t[i] = stats[s];
+      v[i] = load4(part + (size_t)s * a.vdim_p);
+      if (s0 + i >= p.splits) t[i] = make_float2(-INFINITY, 0.f);
     }
-    const float inv = 1.f / sum;
-    *reinterpret_cast<uint32_t*>(out + (size_t)h * VP + c) = pack_bf16x2(o0 * inv, o1 * inv);
+    float m_new = m;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) m_new = fmaxf(m_new, t[i].x);
+    if (m_new == -INFINITY) continue;                       // shares without pages
+    const float keep = exp2f(m - m_new);
+    l *= keep;
+    o.x *= keep; o.y *= keep; o.z *= keep; o.w *= keep;
+    m = m_new;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float f = exp2f(t[i].x - m_new);
+      l += f * t[i].y;
+      o.x += f * v[i].x; o.y += f * v[i].y; o.z += f * v[i].z; o.w += f * v[i].w;
+    }
   }
-  if (tid == 0) p.counters[cell] = 0;
+  const float inv = 1.f / l;
+  store4(static_cast<__nv_bfloat16*>(a.out) + (size_t)row * a.ld_o + (size_t)h * a.vdim_p + c, make_float4(o.x * inv, o.y * inv, o.z * inv, o.w * inv));
 }
 
 template <int MT, int VN>
@@ -264,9 +282,11 @@ static int launch_latent_decode(LatentDecodeParams p, size_t smem, cudaStream_t 
   const int blocks = ceil_div(a.heads, MT * 16);
   for (int r = 0; r < a.rows; r += 65535) {
     p.a.row0 = a.row0 + r;
-    kern<<<dim3(p.splits, blocks, std::min(a.rows - r, 65535)), LD_THREADS, smem, st>>>(p);
+    const int n = std::min(a.rows - r, 65535);
+    kern<<<dim3(p.splits, blocks, n), LD_THREADS, smem, st>>>(p);
+    if (p.splits > 1) latent_merge_kernel<<<dim3(a.heads, n), 128, 0, st>>>(p);
   }
-  return launch_check("latent_decode");
+  return launch_check("latent_decode", p.splits > 1 ? 2 : 1);
 }
 
 // 1: sizes outside the kernel's limits
@@ -275,21 +295,20 @@ int latent_decode(const nfn_paged_attention_args& a, cudaStream_t st) {
   LatentDecodeParams p;
   p.a = a;
   p.pitch = a.dim_p + 8;
+  p.status = status_ptr();
   const int mt = a.heads > 16 ? 2 : 1, nh = 16 * mt;
   const size_t smem = (size_t)(nh + 2 * NFN_PAGE) * p.pitch * 2 + (size_t)2 * nh * LD_S * 4 + (size_t)nh * LD_P * 2;
   if (smem > 220 * 1024) return 1;
-  p.counters = static_cast<int*>(a.workspace);
-  p.partial = reinterpret_cast<float*>(static_cast<char*>(a.workspace) + PAGED_COUNTER_BYTES);
-  const long long cells = (long long)a.rows * ceil_div(a.heads, nh);
   // one wave of what is resident at a time, at least one page each
+  const long long ctas = (long long)a.rows * ceil_div(a.heads, nh), cells = (long long)a.rows * a.heads;
   const int resident = (int)std::max<size_t>(1, (size_t)(220 * 1024) / smem);
-  long long splits = std::min<long long>(ceil_div(a.max_keys, NFN_PAGE), std::max<long long>(1, (long long)sm_count() * std::min(resident, 4) / cells));
-  const long long per_split = cells * nh * (a.vdim_p + 2) * 4;
-  splits = std::min<long long>(splits, (a.workspace_bytes - PAGED_COUNTER_BYTES) / per_split);
-  if (cells > LD_COUNTERS || splits < 1) splits = 1;
-  p.splits = (int)std::min<long long>(splits, 64);
-  if (mt == 1) return a.vdim_p <= 128 ? launch_latent_decode<1, 2>(p, smem, st) : a.vdim_p <= 256 ? launch_latent_decode<1, 4>(p, smem, st) : launch_latent_decode<1, 8>(p, smem, st);
-  return a.vdim_p <= 128 ? launch_latent_decode<2, 2>(p, smem, st) : a.vdim_p <= 256 ? launch_latent_decode<2, 4>(p, smem, st) : launch_latent_decode<2, 8>(p, smem, st);
+  long long splits = std::min<long long>(ceil_div(a.max_keys, NFN_PAGE) + 1, std::max<long long>(1, (long long)sm_count() * std::min(resident, 4) / ctas));
+  splits = std::min<long long>(std::min<long long>(splits, 64), (a.workspace_bytes - PAGED_COUNTER_BYTES) / (cells * (a.vdim_p * 4 + 8)));
+  p.splits = (int)std::max<long long>(splits, 1);
+  p.partial = reinterpret_cast<float*>(static_cast<char*>(a.workspace) + PAGED_COUNTER_BYTES);
+  p.stats = reinterpret_cast<float2*>(p.partial + cells * p.splits * a.vdim_p);
+  if (mt == 1) return a.vdim_p <= 256 ? launch_latent_decode<1, 2>(p, smem, st) : launch_latent_decode<1, 4>(p, smem, st);
+  return a.vdim_p <= 256 ? launch_latent_decode<2, 2>(p, smem, st) : launch_latent_decode<2, 4>(p, smem, st);
 }
 
 }  // namespace nfn

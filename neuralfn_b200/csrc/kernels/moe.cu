@@ -85,7 +85,8 @@ moe_route_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, 
   }
 }
 
-// The same with the choice of nfn_route_rule
+// The same with the choice of nfn_route_rule. PER: experts per lane
+template <int PER>
 __global__ void __launch_bounds__(256)
 moe_choose_kernel(const float* __restrict__ logits, int ld, int T, int E, int k, nfn_route_rule rule, int* topk_idx, float* topk_w, int* __restrict__ counts) {
   __shared__ int count[MOE_MAX_E];
@@ -94,7 +95,7 @@ moe_choose_kernel(const float* __restrict__ logits, int ld, int T, int E, int k,
   __syncthreads();
   if (tok < T) {
     int* idx = topk_idx + (long long)tok * k;
-    choose_experts<MOE_MAX_E / 32>(logits + (long long)tok * ld, E, k, rule, lane, idx, topk_w + (long long)tok * k);
+    choose_experts<PER>(logits + (long long)tok * ld, E, k, rule, lane, idx, topk_w + (long long)tok * k);
     for (int j = lane; j < k; j += 32) atomicAdd(&count[idx[j]], 1);
   }
   __syncthreads();
@@ -198,7 +199,8 @@ extern "C" int nfn_moe_choose(const float* logits, int ld, int T, int E, int k, 
   if (E <= 0 || E > MOE_MAX_E || k <= 0 || k > E || ld < E) return fail(-1, "moe_choose: need 1 <= k <= E <= 256, ld >= E");
   if (rule->groups < 0 || (rule->groups > 0 && (E % rule->groups || rule->keep_groups < 1 || rule->keep_groups * (E / rule->groups) < k)))
     return fail(-1, "moe_choose: the kept groups must hold the chosen experts");
-  moe_choose_kernel<<<(T + 7) / 8, 256, 0, static_cast<cudaStream_t>(stream)>>>(logits, ld, T, E, k, *rule, idx, weight, counts);
+  auto kern = E <= 32 ? moe_choose_kernel<1> : E <= 64 ? moe_choose_kernel<2> : E <= 128 ? moe_choose_kernel<4> : moe_choose_kernel<MOE_MAX_E / 32>;
+  kern<<<(T + 7) / 8, 256, 0, static_cast<cudaStream_t>(stream)>>>(logits, ld, T, E, k, *rule, idx, weight, counts);
   return launch_check("moe_choose", 1);
 }
 

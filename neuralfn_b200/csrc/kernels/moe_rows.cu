@@ -66,22 +66,24 @@ enum { kGateUp = 0, kDown = 1, kUp = 2 };
 template <typename T, int FORM>
 __global__ void __launch_bounds__(MR_WARPS * 32)
 moe_products_kernel(const nfn_moe_rows_args p) {
-  if ((int)blockIdx.y >= p.active[p.experts]) return;
-  const int e = p.active[blockIdx.y], warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   constexpr bool DOWN = FORM == kDown, TWO = FORM == kGateUp;
-  const int n = blockIdx.x * MR_WARPS + warp, N = DOWN ? p.width : p.ff, K = DOWN ? p.ff : p.width;
+  const bool shared = DOWN && p.shared_ff > 0 && blockIdx.y == 0;        // the expert of all rows comes first
+  const int at = blockIdx.y - (DOWN && p.shared_ff > 0 ? 1 : 0);
+  if (!shared && at >= p.active[p.experts]) return;
+  const int e = shared ? 0 : p.active[at], warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int n = blockIdx.x * MR_WARPS + warp, N = DOWN ? p.width : p.ff, K = DOWN ? (shared ? p.shared_ff : p.ff) : p.width;
   if (n >= N) return;
-  const __nv_bfloat16* wa = DOWN ? static_cast<const __nv_bfloat16*>(p.w_down) + ((size_t)e * N + n) * K
+  const __nv_bfloat16* wa = DOWN ? static_cast<const __nv_bfloat16*>(shared ? p.w_shared_down : p.w_down) + ((size_t)e * N + n) * K
                                  : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * (TWO ? 2 : 1) * N + n) * K;
   const __nv_bfloat16* wb = TWO ? wa + (size_t)N * K : wa;
-  const int i0 = p.offsets[e], i1 = p.offsets[e + 1];
+  const int i0 = shared ? 0 : p.offsets[e], i1 = shared ? p.rows : p.offsets[e + 1];
   for (int g = i0; g < i1; g += MR_GROUP) {
     const int m = min(MR_GROUP, i1 - g);
     const T* src[MR_GROUP];
 #pragma unroll
     for (int i = 0; i < MR_GROUP; ++i) {
-      const int item = p.order[i < m ? g + i : g];
-      src[i] = DOWN ? static_cast<const T*>(p.mid) + (size_t)item * p.ff : static_cast<const T*>(p.h) + (size_t)(item / p.top) * p.ld_h;
+      const int item = shared ? (i < m ? g + i : g) : p.order[i < m ? g + i : g];
+      src[i] = DOWN ? static_cast<const T*>(shared ? p.shared_mid : p.mid) + (size_t)item * K : static_cast<const T*>(p.h) + (size_t)(item / p.top) * p.ld_h;
     }
     float a[MR_GROUP], b[MR_GROUP];
 #pragma unroll
@@ -123,9 +125,9 @@ moe_products_kernel(const nfn_moe_rows_args p) {
         if (TWO) b[i] += __shfl_xor_sync(0xffffffffu, b[i], o);
       }
       if (lane == 0) {
-        const int item = p.order[g + i];
+        const int item = shared ? g + i : p.order[g + i];
         if (DOWN) {
-          static_cast<T*>(p.y)[(size_t)item * p.ld_y + n] = from_float<T>(a[i]);
+          static_cast<T*>(shared ? p.y_shared : p.y)[(size_t)item * p.ld_y + n] = from_float<T>(a[i]);
         } else if (!TWO) {
           static_cast<T*>(p.mid)[(size_t)item * p.ff + n] = from_float<T>(ff_act(a[i], p.act));
         } else {
@@ -161,26 +163,29 @@ moe_products_mma_kernel(const nfn_moe_rows_args p) {
   constexpr int M = 8 * NT;                               // items at a time
   constexpr int U = NT == 4 ? 2 : 4;                      // 32-channel steps in flight
   __shared__ float part[MM_WARPS][2][16][M + 1];
-  if ((int)blockIdx.y >= p.active[p.experts]) return;
-  const int e = p.active[blockIdx.y], warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
-  const int N = DOWN ? p.width : p.ff, K = DOWN ? p.ff : p.width;
+  const bool shared = DOWN && p.shared_ff > 0 && blockIdx.y == 0;        // the expert of all rows comes first
+  const int at = blockIdx.y - (DOWN && p.shared_ff > 0 ? 1 : 0);
+  if (!shared && at >= p.active[p.experts]) return;
+  const int e = shared ? 0 : p.active[at], warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, j = lane & 3;
+  const int N = DOWN ? p.width : p.ff, K = DOWN ? (shared ? p.shared_ff : p.ff) : p.width;
   const int n0 = blockIdx.x * TILE;
   // rows of the two 16-row tiles
-  const __nv_bfloat16* w0 = (DOWN ? static_cast<const __nv_bfloat16*>(p.w_down) + ((size_t)e * N + n0) * K : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * (TWO ? 2 : 1) * N + n0) * K) +
+  const __nv_bfloat16* w0 = (DOWN ? static_cast<const __nv_bfloat16*>(shared ? p.w_shared_down : p.w_down) + ((size_t)e * N + n0) * K : static_cast<const __nv_bfloat16*>(p.w_gate_up) + ((size_t)e * (TWO ? 2 : 1) * N + n0) * K) +
                             (size_t)g * K + 8 * j;
   const bool two = TWO || n0 + 16 < N;
   const __nv_bfloat16* w1 = two ? w0 + (size_t)(TWO ? N : 16) * K : w0;
   const int steps = (K + 31) / 32, s0 = steps * warp / MM_WARPS, s1 = steps * (warp + 1) / MM_WARPS;
   const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
-  const int i0 = p.offsets[e], i1 = p.offsets[e + 1];
+  const int i0 = shared ? 0 : p.offsets[e], i1 = shared ? p.rows : p.offsets[e + 1];
+  auto item_at = [&](int i) { return shared ? i : p.order[i]; };
   for (int i = i0; i < i1; i += M) {
     const __nv_bfloat16* src[NT];
     bool on[NT];
 #pragma unroll
     for (int t = 0; t < NT; ++t) {
       on[t] = i + 8 * t + g < i1;
-      const int item = p.order[on[t] ? i + 8 * t + g : i0];
-      src[t] = (DOWN ? static_cast<const __nv_bfloat16*>(p.mid) + (size_t)item * p.ff : static_cast<const __nv_bfloat16*>(p.h) + (size_t)(item / p.top) * p.ld_h) + 8 * j;
+      const int item = item_at(on[t] ? i + 8 * t + g : i0);
+      src[t] = (DOWN ? static_cast<const __nv_bfloat16*>(shared ? p.shared_mid : p.mid) + (size_t)item * K : static_cast<const __nv_bfloat16*>(p.h) + (size_t)(item / p.top) * p.ld_h) + 8 * j;
     }
     float acc[2][NT][4];
 #pragma unroll
@@ -221,13 +226,13 @@ moe_products_mma_kernel(const nfn_moe_rows_args p) {
     __syncthreads();
     const int live = min(M, i1 - i);
     for (int x = threadIdx.x; x < TILE * live; x += MM_WARPS * 32) {
-      const int col = x / TILE, row = x % TILE, item = p.order[i + col];
+      const int col = x / TILE, row = x % TILE, item = item_at(i + col);
       if (n0 + row >= N) continue;
       if (!TWO) {
         float v = 0.f;
 #pragma unroll
         for (int w = 0; w < MM_WARPS; ++w) v += part[w][row >> 4][row & 15][col];
-        if (DOWN) static_cast<__nv_bfloat16*>(p.y)[(size_t)item * p.ld_y + n0 + row] = __float2bfloat16(v);
+        if (DOWN) static_cast<__nv_bfloat16*>(shared ? p.y_shared : p.y)[(size_t)item * p.ld_y + n0 + row] = __float2bfloat16(v);
         else static_cast<__nv_bfloat16*>(p.mid)[(size_t)item * p.ff + n0 + row] = __float2bfloat16(ff_act(v, p.act));
       } else {
         float gv = 0.f, uv = 0.f;
@@ -263,18 +268,19 @@ template <int NT>
 static void launch_products_mma(const nfn_moe_rows_args& a, int live, cudaStream_t st) {
   if (a.plain) moe_products_mma_kernel<kUp, NT><<<dim3(ceil_div(a.ff, 32), live), MM_WARPS * 32, 0, st>>>(a);
   else moe_products_mma_kernel<kGateUp, NT><<<dim3(ceil_div(a.ff, 16), live), MM_WARPS * 32, 0, st>>>(a);
-  moe_products_mma_kernel<kDown, NT><<<dim3(ceil_div(a.width, 32), live), MM_WARPS * 32, 0, st>>>(a);
+  moe_products_mma_kernel<kDown, NT><<<dim3(ceil_div(a.width, 32), live + (a.shared_ff > 0)), MM_WARPS * 32, 0, st>>>(a);
 }
 
 static int launch_moe_rows(const nfn_moe_rows_args& a, cudaStream_t st) {
   const int live = (int)std::min<long long>(a.experts, (long long)a.rows * a.top);     // most experts that can have items
-  if (a.experts <= 64) moe_route_rows_kernel<2><<<1, 1024, 0, st>>>(a);
+  if (a.experts <= 32) moe_route_rows_kernel<1><<<1, 1024, 0, st>>>(a);
+  else if (a.experts <= 64) moe_route_rows_kernel<2><<<1, 1024, 0, st>>>(a);
   else if (a.experts <= 256) moe_route_rows_kernel<8><<<1, 1024, 0, st>>>(a);
   else moe_route_rows_kernel<32><<<1, 1024, 0, st>>>(a);
   if (a.f32) {
     if (a.plain) moe_products_kernel<float, kUp><<<dim3(ceil_div(a.ff, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
     else moe_products_kernel<float, kGateUp><<<dim3(ceil_div(a.ff, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
-    moe_products_kernel<float, kDown><<<dim3(ceil_div(a.width, MR_WARPS), live), MR_WARPS * 32, 0, st>>>(a);
+    moe_products_kernel<float, kDown><<<dim3(ceil_div(a.width, MR_WARPS), live + (a.shared_ff > 0)), MR_WARPS * 32, 0, st>>>(a);
   } else if (a.rows <= 8) {
     launch_products_mma<1>(a, live, st);
   } else if (a.rows <= 16) {
@@ -296,6 +302,7 @@ extern "C" int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream) 
   if (a.experts < 1 || a.experts > MR_MAX_EXPERTS || a.top < 1 || a.top > a.experts) return fail(-1, "moe_rows: need 1 <= top <= experts <= 1024");
   if (a.rule.groups < 0 || (a.rule.groups > 0 && (a.experts % a.rule.groups || a.rule.keep_groups < 1 || (long long)a.rule.keep_groups * (a.experts / a.rule.groups) < a.top)))
     return fail(-1, "moe_rows: the kept groups must hold the chosen experts");
+  if (a.shared_ff < 0 || (a.shared_ff > 0 && ((a.shared_ff & 15) || !a.shared_mid || !a.w_shared_down || !a.y_shared))) return fail(-1, "moe_rows: the shared expert lacks an operand");
   if ((a.width | a.ff | a.ld_h) & 15) return fail(-1, "moe_rows: widths must be multiples of 16");
   if ((long long)a.rows * a.top > 0x7fffffffLL / 2) return fail(-1, "moe_rows: too many rows");
   return launch_moe_rows(a, static_cast<cudaStream_t>(stream));

@@ -407,13 +407,18 @@ typedef struct {
   const nfn_row_tile* tiles; int n_tiles, tile_rows;
 } nfn_latent_rows_args;
 int nfn_latent_rows(const nfn_latent_rows_args* args, nfn_stream_t stream);
-// out[r][g][n] = sum_k in[r][g][k] w[g][n][k]: one small product per group and row (the per-head projections around a latent cache, several inputs
-// with a matrix each). in, out: activation type, group pitches in elements; w bf16. Sizes are multiples of 16.
+// out[r][g][n] = act(sum_k in[r][g][k] w[g][n][k]): one small product per group and row (the per-head projections around a latent cache, several inputs
+// with a matrix each). in, out: activation type, group pitches in elements; w bf16. Sizes are multiples of 16. tail_n > 0: one more product of the same
+// depth, from the input tail_in elements into each row, with an fp32 result and no activation.
 typedef struct {
   int f32, rows, groups, n, k;
   const void* in; long long ld_in, in_group;
   const void* w;
   void* out; long long ld_out, out_group;
+  int act, tail_n;
+  long long tail_in;
+  const void* tail_w;
+  float* tail_out; int ld_tail;
 } nfn_group_products_args;
 int nfn_group_products(const nfn_group_products_args* args, nfn_stream_t stream);
 
@@ -584,6 +589,8 @@ typedef struct {
   void* y; int ld_y;                      // [rows * top][ld_y]
   int plain;
   nfn_route_rule rule;                    // scale 0 counts as 1
+  // shared_ff > 0: the second product of an expert that every row has, y_shared [rows][ld_y] = w_shared_down shared_mid [rows][shared_ff], beside the others
+  int shared_ff; const void* shared_mid; const void* w_shared_down; void* y_shared;
 } nfn_moe_rows_args;
 int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream);
 

@@ -11,7 +11,8 @@
 //
 // Latent attention (EXPANDED): every head's unrotated keys and its values were formed from the cached latents as rows of one matrix, 64 rows per
 // page; the rotated key part, shared by the heads, still comes from the pages as further panels of the same score product. Values then
-// are [64 tokens][64 channels] panels, an MN-major operand.
+// are [64 tokens][64 channels] panels, an MN-major operand. Queries and keys take a panel more, so P stays in TMEM (a TMEM-sourced product) and
+// values have one stage where two would cost the second CTA of an SM its place.
 //
 // Head sizes are run-time values (multiples of 16 up to 256; channels past a head's end are zero-filled by TMA). The distance
 // bias and the window are applied to the fp32 scores in registers; the output gate is applied on the way out.
@@ -21,6 +22,7 @@
 namespace nfn {
 
 constexpr int PP_BM = 128, PP_BN = NFN_PAGE;
+constexpr uint32_t PP_P_COL = PP_BN;          // EXPANDED: P behind the scores, PP_BN / 2 columns
 
 struct PagedPrefillParams {
   nfn_paged_attention_args a;
@@ -29,6 +31,7 @@ struct PagedPrefillParams {
   nfn_latent_expanded x;      // EXPANDED
   int panels_r, panels_v;     // panels of the rotated part, of a value head
   uint32_t q_bytes, k_bytes, v_bytes, q_tx;
+  int v_stages;
   uint32_t o_col, tmem_cols;
   uint32_t smem;
   int* status;
@@ -50,11 +53,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     }
   }
   const nfn_paged_attention_args& a = p.a;
-  const uint32_t kv_stage = p.k_bytes + p.v_bytes;
+  const int vs = p.v_stages;
   uint8_t* sQ = smem;
-  uint8_t* sKV = sQ + p.q_bytes;
-  uint8_t* sP = sKV + 2 * kv_stage;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + PP_BM * PP_BN * 2);
+  uint8_t* sK = sQ + p.q_bytes;
+  uint8_t* sV = sK + 2 * p.k_bytes;
+  uint8_t* sP = sV + vs * p.v_bytes;
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + (EXPANDED ? 0 : PP_BM * PP_BN * 2));
   uint64_t* bar_q = bars;          // TMA: Q landed
   uint64_t* bar_k = bars + 1;      // [2] TMA: key stage landed
   uint64_t* bar_v = bars + 3;      // [2] TMA: value stage landed
@@ -108,7 +112,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       const int x_base = EXPANDED ? p.x.x_base[slot] : 0;
       auto load_k = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_k[stage]);
-        const uint32_t sk = smem_u32(sKV + stage * kv_stage);
+        const uint32_t sk = smem_u32(sK + stage * p.k_bytes);
         mbar_expect_tx(fb, p.k_bytes);
         if (EXPANDED) {
           const int r = x_base + page_at(j) * PP_BN;
@@ -122,7 +126,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       };
       auto load_v = [&](int j, int stage) {
         const uint32_t fb = smem_u32(&bar_v[stage]);
-        const uint32_t sv = smem_u32(sKV + stage * kv_stage + p.k_bytes);
+        const uint32_t sv = smem_u32(sV + stage * p.v_bytes);
         mbar_expect_tx(fb, p.v_bytes);
         if (EXPANDED) {
           for (int d = 0; d < p.panels_v; ++d)
@@ -138,12 +142,16 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           tma_load_3d(smem_u32(sQ) + (p.panels + d) * (PP_BM * 128), &tm_q, smem_u32(bar_q), p.x.dim_u + d * 64, hk, row0);
       load_k(0, 0);
       load_v(0, 0);
-      if (nblk > 1) { load_k(1, 1); load_v(1, 1); }
-      for (int j = 0; j + 2 < nblk; ++j) {
-        if (!mbar_wait_bounded(smem_u32(&bar_kfree[j & 1]), (j >> 1) & 1, cta_abort, p.status, 0x600 + 1)) break;
-        load_k(j + 2, j & 1);
-        if (!mbar_wait_bounded(smem_u32(&bar_vfree[j & 1]), (j >> 1) & 1, cta_abort, p.status, 0x600 + 2)) break;
-        load_v(j + 2, j & 1);
+      if (nblk > 1) load_k(1, 1);
+      if (nblk > 1 && vs > 1) load_v(1, 1);
+      for (int j = 0; j + vs < nblk; ++j) {
+        if (j + 2 < nblk) {
+          if (!mbar_wait_bounded(smem_u32(&bar_kfree[j & 1]), (j >> 1) & 1, cta_abort, p.status, 0x600 + 1)) break;
+          load_k(j + 2, j & 1);
+        }
+        const int st = vs > 1 ? j & 1 : 0;
+        if (!mbar_wait_bounded(smem_u32(&bar_vfree[st]), (vs > 1 ? j >> 1 : j) & 1, cta_abort, p.status, 0x600 + 2)) break;
+        load_v(j + vs, st);
       }
     }
   } else if (warp == AV2_MMA_WARP) {
@@ -154,7 +162,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       const int k_steps = (EXPANDED ? p.x.dim_u : a.dim_p) / 16;
       auto issue_s = [&](int stage) {
         const uint32_t sq = smem_u32(sQ);
-        const uint32_t sk = smem_u32(sKV + stage * kv_stage);
+        const uint32_t sk = smem_u32(sK + stage * p.k_bytes);
 #pragma unroll 4
         for (int kk = 0; kk < k_steps; ++kk) {
           const uint32_t a_off = (kk / 4) * (PP_BM * 128) + (kk % 4) * 32;
@@ -185,17 +193,21 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           issue_s(ns);
         }
         ok = mbar_wait_bounded(smem_u32(bar_p), j & 1, cta_abort, p.status, 0x600 + 7);
-        ok = ok && mbar_wait_bounded(smem_u32(&bar_v[j & 1]), (j >> 1) & 1, cta_abort, p.status, 0x600 + 8);
+        const int st = vs > 1 ? j & 1 : 0;
+        ok = ok && mbar_wait_bounded(smem_u32(&bar_v[st]), (vs > 1 ? j >> 1 : j) & 1, cta_abort, p.status, 0x600 + 8);
         if (!ok) break;
         tc_fence_after();
         const uint32_t sp = smem_u32(sP);
-        const uint32_t sv = smem_u32(sKV + (j & 1) * kv_stage + p.k_bytes);
+        const uint32_t sv = smem_u32(sV + st * p.v_bytes);
 #pragma unroll
-        for (int kk = 0; kk < PP_BN / 16; ++kk)
-          umma_bf16_ss(tmem_base + p.o_col, make_smem_desc_sw128(sp + kk * 32, 16, 1024),
-                       EXPANDED ? make_smem_desc_sw128(sv + kk * (16 * 128), PP_BN * 128, 1024) : make_smem_desc_sw128(sv + kk * 32, 16, 1024), idesc_o, (j | kk) != 0);
+        for (int kk = 0; kk < PP_BN / 16; ++kk) {
+          if (EXPANDED)  // 16 keys of P = 8 TMEM columns of bf16 pairs
+            umma_bf16_ts(tmem_base + p.o_col, tmem_base + PP_P_COL + kk * 8, make_smem_desc_sw128(sv + kk * (16 * 128), PP_BN * 128, 1024), idesc_o, (j | kk) != 0);
+          else
+            umma_bf16_ss(tmem_base + p.o_col, make_smem_desc_sw128(sp + kk * 32, 16, 1024), make_smem_desc_sw128(sv + kk * 32, 16, 1024), idesc_o, (j | kk) != 0);
+        }
         umma_commit(smem_u32(bar_o));
-        umma_commit(smem_u32(&bar_vfree[j & 1]));
+        umma_commit(smem_u32(&bar_vfree[st]));
       }
     }
   } else {
@@ -333,6 +345,13 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
           tmem_st_wait();
         }
       }
+      if (EXPANDED) {
+        // packed in place, then straight into TMEM
+#pragma unroll
+        for (int i = 0; i < PP_BN / 2; ++i) s[i] = pack_bf16x2(__uint_as_float(s[2 * i]), __uint_as_float(s[2 * i + 1]));
+        tmem_st_32x32(t_row + PP_P_COL, *reinterpret_cast<uint32_t(*)[32]>(&s[0]));
+        tmem_st_wait();
+      } else {
 #pragma unroll
       for (int c = 0; c < PP_BN / 8; ++c) {
         const uint32_t* e = &s[c * 8];
@@ -341,6 +360,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
                                          pack_bf16x2(__uint_as_float(e[4]), __uint_as_float(e[5])), pack_bf16x2(__uint_as_float(e[6]), __uint_as_float(e[7]))));
       }
       fence_proxy_async();
+      }
       tc_fence_before();
       __syncwarp();
       if (lane == 0) mbar_arrive(smem_u32(bar_p));
@@ -409,18 +429,22 @@ using namespace nfn;
 static uint32_t paged_tile_smem(uint32_t panels, uint32_t v_bytes) {
   return panels * PP_BM * 128 + 2 * (panels * PP_BN * 128 + v_bytes) + PP_BM * PP_BN * 2 + 128;
 }
+static uint32_t latent_tile_smem(int panels, int panels_v, int v_stages) {
+  return panels * PP_BM * 128 + 2 * panels * PP_BN * 128 + v_stages * panels_v * PP_BN * 128 + 128;
+}
+constexpr uint32_t PP_SMEM_MAX = 226 * 1024, PP_SMEM_HALF = 113 * 1024;     // of one CTA; so that two share an SM
 
 extern "C" int nfn_paged_tile_rows(int f32, int heads, int kv_heads, int dim_p, int vdim_p) {
   const int hg = heads / kv_heads;
-  if (f32 || dim_p > 256 || vdim_p > 256 || hg > PP_BM || paged_tile_smem((dim_p + 63) / 64, vdim_p * 128) > 226 * 1024) return 0;
+  if (f32 || dim_p > 256 || vdim_p > 256 || hg > PP_BM || paged_tile_smem((dim_p + 63) / 64, vdim_p * 128) > PP_SMEM_MAX) return 0;
   return PP_BM / hg;
 }
 
 template <bool EXPANDED>
 static int launch_paged_prefill(PagedPrefillParams& p, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, cudaStream_t st) {
   const nfn_paged_attention_args& a = p.a;
-  p.o_col = PP_BN;
-  const int cols = PP_BN + (EXPANDED ? p.panels_v * 64 : a.vdim_p);
+  p.o_col = EXPANDED ? PP_BN + PP_BN / 2 : PP_BN;
+  const int cols = (int)p.o_col + (EXPANDED ? p.panels_v * 64 : a.vdim_p);
   p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;
   p.status = status_ptr();
   auto kern = paged_prefill_kernel<EXPANDED>;
@@ -451,6 +475,7 @@ extern "C" int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, n
   // the value stage keeps the next key stage on a 1024-byte boundary
   p.v_bytes = a.vdim_p * 128;
   p.q_tx = p.panels * p.nq * p.hg * 128;
+  p.v_stages = 2;
   p.smem = paged_tile_smem(p.panels, p.v_bytes);
   CUtensorMap tq, tk, tv;
   if (!make_tmap_3d(&tq, a.q, 2, a.dim_p, a.heads, a.total_rows, a.dim_p, a.ld_q, 64, p.hg, p.nq, 128)) return -3;
@@ -460,12 +485,15 @@ extern "C" int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, n
   return launch_paged_prefill<false>(p, tq, tk, tv, static_cast<cudaStream_t>(stream));
 }
 
-static uint32_t latent_tile_smem(int dim_u, int rot_p, int vdim_p) {
-  return paged_tile_smem((dim_u + 63) / 64 + (rot_p + 63) / 64, (vdim_p + 63) / 64 * PP_BN * 128);
+// stages of values for these panels: two, or one where that lets a second CTA in or is all there is room for; 0: no room
+static int latent_v_stages(int panels, int panels_v) {
+  if (latent_tile_smem(panels, panels_v, 2) <= PP_SMEM_HALF) return 2;
+  if (latent_tile_smem(panels, panels_v, 1) <= PP_SMEM_HALF) return 1;
+  return latent_tile_smem(panels, panels_v, 2) <= PP_SMEM_MAX ? 2 : latent_tile_smem(panels, panels_v, 1) <= PP_SMEM_MAX ? 1 : 0;
 }
 
 extern "C" int nfn_latent_tile_rows(int f32, int dim_u, int rot_p, int vdim_p) {
-  return f32 || vdim_p > 256 || latent_tile_smem(dim_u, rot_p, vdim_p) > 226 * 1024 ? 0 : PP_BM;
+  return f32 || vdim_p > 256 || latent_v_stages((dim_u + 63) / 64 + (rot_p + 63) / 64, (vdim_p + 63) / 64) == 0 ? 0 : PP_BM;
 }
 
 extern "C" int nfn_latent_attention_tiles(const nfn_paged_attention_args* args, const nfn_latent_expanded* x, nfn_stream_t stream) {
@@ -487,7 +515,8 @@ extern "C" int nfn_latent_attention_tiles(const nfn_paged_attention_args* args, 
   p.q_bytes = p.q_tx = panels * PP_BM * 128;
   p.k_bytes = panels * PP_BN * 128;
   p.v_bytes = p.panels_v * PP_BN * 128;
-  p.smem = latent_tile_smem(x->dim_u, x->rot_p, a.vdim_p);
+  p.v_stages = latent_v_stages(panels, p.panels_v);
+  p.smem = latent_tile_smem(panels, p.panels_v, p.v_stages);
   const int lp = x->rank_p + x->rot_p, cols = a.heads * (x->dim_u + a.vdim_p);
   CUtensorMap tq, tk, tx;
   if (!make_tmap_3d(&tq, a.q, 2, a.dim_p, a.heads, a.total_rows, a.dim_p, a.ld_q, 64, 1, PP_BM, 128)) return -3;

@@ -38,7 +38,8 @@ class _Experts(C.Structure):
     _fields_ = [("f32", C.c_int), ("rows", C.c_int), ("width", C.c_int), ("ff", C.c_int), ("experts", C.c_int), ("top", C.c_int), ("act", C.c_int),
                 ("logits", C.c_void_p), ("ld_logits", C.c_int), ("h", C.c_void_p), ("ld_h", C.c_int), ("w_gate_up", C.c_void_p), ("w_down", C.c_void_p),
                 ("idx", C.c_void_p), ("weight", C.c_void_p), ("order", C.c_void_p), ("offsets", C.c_void_p), ("active", C.c_void_p), ("mid", C.c_void_p),
-                ("y", C.c_void_p), ("ld_y", C.c_int), ("plain", C.c_int), ("rule", RouteRule)]
+                ("y", C.c_void_p), ("ld_y", C.c_int), ("plain", C.c_int), ("rule", RouteRule), ("shared_ff", C.c_int),
+                ("shared_mid", C.c_void_p), ("w_shared_down", C.c_void_p), ("y_shared", C.c_void_p)]
 
 
 def _p(t: torch.Tensor | None):
@@ -102,15 +103,18 @@ def expert_choice(logits: torch.Tensor, top: int, **rule) -> tuple[torch.Tensor,
     return idx, weight, counts
 
 
-def expert_rows(h: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, *, experts: int, top: int, act: int = 3, plain: bool = False, **rule):
-    """Returns the chosen experts [rows, top], their weights and outputs y [rows, top, width]. plain: w_gate_up holds one matrix per expert."""
+def expert_rows(h: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, *, experts: int, top: int, act: int = 3, plain: bool = False,
+                shared_mid: torch.Tensor | None = None, shared_down: torch.Tensor | None = None, y_shared: torch.Tensor | None = None, **rule):
+    """Returns the chosen experts [rows, top], their weights and outputs y [rows, top, width]. plain: w_gate_up holds one matrix per expert. shared_mid [rows, f],
+    shared_down [width, f]: y_shared [rows, width] is their product."""
     rows, width, ff = h.shape[0], h.shape[1], w_down.shape[2]
     i32 = dict(dtype=torch.int32, device=h.device)
     idx, order, offsets, active = (torch.zeros(n, **i32) for n in (rows * top, rows * top, experts + 1, experts + 1))
     weight = torch.zeros(rows * top, device=h.device)
     mid, y = torch.zeros(rows * top, ff, device=h.device, dtype=h.dtype), torch.zeros(rows * top, width, device=h.device, dtype=h.dtype)
     a = _Experts(int(h.dtype == torch.float32), rows, width, ff, experts, top, act, _p(logits), logits.stride(0), _p(h), h.stride(0), _p(w_gate_up), _p(w_down), _p(idx),
-                 _p(weight), _p(order), _p(offsets), _p(active), _p(mid), _p(y), y.stride(0), int(plain), _rule(**rule))
+                 _p(weight), _p(order), _p(offsets), _p(active), _p(mid), _p(y), y.stride(0), int(plain), _rule(**rule), 0 if shared_mid is None else shared_mid.shape[1], _p(shared_mid),
+                 _p(shared_down), _p(y_shared))
     _call("moe_rows", a)
     return idx.view(rows, top), weight.view(rows, top), y.view(rows, top, width)
 
@@ -137,7 +141,8 @@ class _Latent(C.Structure):
 
 class _Groups(C.Structure):
     _fields_ = [("f32", C.c_int), ("rows", C.c_int), ("groups", C.c_int), ("n", C.c_int), ("k", C.c_int), ("in_", C.c_void_p), ("ld_in", C.c_longlong), ("in_group", C.c_longlong),
-                ("w", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_longlong), ("out_group", C.c_longlong)]
+                ("w", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_longlong), ("out_group", C.c_longlong), ("act", C.c_int), ("tail_n", C.c_int), ("tail_in", C.c_longlong),
+                ("tail_w", C.c_void_p), ("tail_out", C.c_void_p), ("ld_tail", C.c_int)]
 
 
 class _Expanded(C.Structure):
@@ -189,9 +194,12 @@ def latent_rows(c: LatentCache, x: torch.Tensor, tiles: torch.Tensor, *, heads: 
     _call("latent_rows", a)
 
 
-def group_products(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
-    """x [rows, groups, k], w bf16 [groups, n, k] -> out [rows, groups, n] (any strides over rows and groups)."""
-    a = _Groups(int(x.dtype == torch.float32), x.shape[0], w.shape[0], w.shape[1], w.shape[2], _p(x), x.stride(0), x.stride(1), _p(w), _p(out), out.stride(0), out.stride(1))
+def group_products(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, act: int = 0, tail_w: torch.Tensor | None = None, tail_out: torch.Tensor | None = None,
+                   tail_in: int = 0) -> torch.Tensor:
+    """x [rows, groups, k], w bf16 [groups, n, k] -> out [rows, groups, n] (any strides over rows and groups); tail_w bf16 [m, k]: one more product, of the input
+    ``tail_in`` elements into each row, into tail_out fp32 [rows, m]."""
+    a = _Groups(int(x.dtype == torch.float32), x.shape[0], w.shape[0], w.shape[1], w.shape[2], _p(x), x.stride(0), x.stride(1), _p(w), _p(out), out.stride(0), out.stride(1), act,
+                0 if tail_w is None else tail_w.shape[0], tail_in, _p(tail_w), _p(tail_out), 0 if tail_out is None else tail_out.stride(0))
     _call("group_products", a)
     return out
 
@@ -206,10 +214,10 @@ def latent_attention_rows(c: LatentCache, q: torch.Tensor, row_slot: torch.Tenso
     return out
 
 
-def latent_gather(c: LatentCache, spans: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
+def latent_gather(c: LatentCache, spans: torch.Tensor, out: torch.Tensor, max_pages: int | None = None) -> torch.Tensor:
     """spans int32 [n, 4] = slot, first page, pages, first row of ``out`` [rows, rank]."""
     _lib.check(_lib.load().nfn_latent_gather(C.c_int(int(c.dtype == torch.float32)), C.c_void_p(_p(c.k)), C.c_int(c.rank + c.rot), C.c_int(c.rank), C.c_void_p(_p(c.table)),
-                                             C.c_int(c.table.stride(0)), C.c_void_p(_p(spans)), C.c_int(spans.shape[0]), C.c_int(int(spans[:, 2].max())), C.c_void_p(_p(out)),
+                                             C.c_int(c.table.stride(0)), C.c_void_p(_p(spans)), C.c_int(spans.shape[0]), C.c_int(max_pages or int(spans[:, 2].max())), C.c_void_p(_p(out)),
                                              C.c_void_p(_lib.stream_ptr())), "latent_gather")
     return out
 

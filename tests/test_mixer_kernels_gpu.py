@@ -107,7 +107,12 @@ def test_group_products(rows, groups, n, k, dtype):
     x, w = rnd(rows, groups, k + 16, dtype=dtype)[..., :k], rnd(groups, n, k)
     out = torch.zeros(groups, rows, n, device=DEV, dtype=dtype).transpose(0, 1)
     Y.group_products(x, w, out)
-    close(out, torch.einsum("rgk,gnk->rgn", x.double(), w.double()), 0.01 if dtype == torch.bfloat16 else 2e-6)
+    want = torch.einsum("rgk,gnk->rgn", x.double(), w.double())
+    close(out, want, 0.01 if dtype == torch.bfloat16 else 2e-6)
+    tail, got = rnd(n + 32, k), torch.zeros(rows, n + 32, device=DEV)
+    Y.group_products(x, w, out, act=4, tail_w=tail, tail_out=got, tail_in=(groups - 1) * x.stride(1))
+    close(out, oracle.relu_squared(want), 0.01 if dtype == torch.bfloat16 else 2e-6)
+    close(got, x[:, -1].double() @ tail.double().T, 2e-6)
 
 
 def latent_problem(rank, rot, lengths, dtype, seed=3):
@@ -291,7 +296,10 @@ def test_expert_choice(experts, top, rule):
     z, corr = rnd(T, experts, dtype=torch.float32), (rnd(experts) * 0.5 - 0.7)
     idx, weight, counts = Y.expert_choice(z, top, correction=corr, normalise=True, scale=1.3, **rule)
     h, up, down = rnd(T, 32), rnd(experts, 16, 32) * 0.2, rnd(experts, 32, 16) * 0.2
-    idx2, weight2, y = Y.expert_rows(h, z, up, down, experts=experts, top=top, act=4, plain=True, correction=corr, normalise=True, scale=1.3, **rule)
+    mid, sd, ys = rnd(T, 48), rnd(32, 48) * 0.2, torch.zeros(T, 32, device=DEV, dtype=torch.bfloat16)
+    idx2, weight2, y = Y.expert_rows(h, z, up, down, experts=experts, top=top, act=4, plain=True, shared_mid=mid, shared_down=sd, y_shared=ys, correction=corr, normalise=True, scale=1.3,
+                                     **rule)
+    close(ys, mid.double() @ sd.double().T, 0.02)
     assert torch.equal(counts, torch.bincount(idx.long().view(-1), minlength=experts).int())
     router = {"top": top, "scale": 1.3}
     if rule:
