@@ -1,236 +1,347 @@
-// Attention of single query rows over latent caches: one cached row per token, [latent | rotated key part], is key and value of every head. The
-// queries come with the key projection folded in (q . W_uk c = W_uk^T q . c), the outputs are weighted sums of latents whose value
-// projection follows, so a token's row is read once for all heads and twice from shared memory: as the key operand and, transposed by
-// ldmatrix, as the value operand.
+// Attention of single query rows over latent caches (tcgen05): one cached row per token, [latent | rotated key part], is key and value of every
+// head. The queries come with the key projection folded in (q . W_uk c = W_uk^T q . c), the outputs are weighted sums of latents whose value
+// projection follows.
 //
-// One CTA takes one row, a block of 16 or 32 heads and a share of the visible pages. Per page: sixteen warps form the scores (8 keys x half of the
-// channels each, on mma.m16n8k16), a softmax pass merges the halves, then each warp owns a slice of the latent channels of the output.
-// Pages arrive one ahead, a bulk copy per row (rows in shared memory are 16 bytes longer than in the page: no bank conflicts). Scores, softmax
-// and sums are fp32; a second launch merges the shares, in order.
+// One CTA takes one row, a block of up to 32 heads and a share of the visible pages. A page arrives once, as 64-channel panels [64 tokens][64 channels],
+// and is used twice as it stands: as the K-major operand of the scores S = q C^T (heads are accumulator rows, the queries wait in TMEM as its
+// other operand) and as the MN-major operand of the outputs, which are transposed, O^T = C^T P^T (latent channels, 128 at a time, are accumulator
+// rows, heads the narrow side), so that few heads waste no accumulators. Roles: warp 0 turns scores into weights, a head per thread; warps 0 - 3
+// rescale outputs, only when a maximum grew by more than 2^8, and write them, a channel per thread; one MMA warp, one TMA warp. Up to three
+// pages are in shared memory or on their way.
+//
+// Scores, softmax and sums are fp32; a second launch merges the shares, in order. Sizes outside the limits take the plain kernel of paged_rows.cu.
 #include <algorithm>
 
+#include "attention_v2.cuh"
 #include "common.h"
 #include "paged.cuh"
 
 namespace nfn {
 
-constexpr int LD_WARPS = 16, LD_THREADS = LD_WARPS * 32, LD_S = NFN_PAGE + 4, LD_P = NFN_PAGE + 8;
+constexpr uint32_t LD_PANEL = NFN_PAGE * 128;      // bytes of 64 channels of a page
+constexpr int LD_MAX_STAGES = 3;
 
 struct LatentDecodeParams {
   nfn_paged_attention_args a;
-  int splits, pitch;           // pitch: elements between rows in shared memory (an odd number of 16-byte pieces: no bank conflicts)
-  float* partial;              // [rows][heads][splits][vdim_p] values
-  float2* stats;               // [rows][heads][splits] maximum and sum
+  int splits, stages;           // shares of a row's pages; pages in shared memory
+  int panels, m_tiles;          // 64-channel panels of a cached row; 128-channel tiles of the latent
+  uint32_t smem, tmem_cols;
+  float* partial;               // [rows][heads][splits][vdim_p] values
+  float2* stats;                // [rows][heads][splits] maximum and sum
   int* status;
 };
 
-__device__ __forceinline__ void ld_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ld_x4_t(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-__device__ __forceinline__ void ld_mma(float (&d)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(d[0]), "+f"(d[1]), "+f"(d[2]), "+f"(d[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void ld_bulk(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
-  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
-}
-
-// MT: 16-head tiles of a CTA; VN: 8-channel tiles of the output per warp (an upper bound)
-template <int MT, int VN>
-__global__ void __launch_bounds__(LD_THREADS)
-latent_decode_kernel(const LatentDecodeParams p) {
-  constexpr int NH = MT * 16;
-  extern __shared__ __align__(16) unsigned char ld_smem[];
-  __shared__ float s_alpha[NH], s_m[NH], s_l[NH];
-  __shared__ __align__(8) uint64_t bar_full[2];
+// NH: heads of a CTA
+template <int NH>
+__global__ void __launch_bounds__(AV2_THREADS, 1)
+latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_c, const LatentDecodeParams p) {
+  constexpr uint32_t Q_PANEL = NH * 128;
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ float s_alpha[2][NH], s_sum[NH];
+  __shared__ int s_flag[2];
+  __shared__ __align__(8) uint64_t bars[4 + 2 * LD_MAX_STAGES + 2];
+  __shared__ uint32_t tmem_slot;
   __shared__ int abort_s;
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~static_cast<uintptr_t>(1023));
   const nfn_paged_attention_args& a = p.a;
   const int row = a.row0 + blockIdx.z, slot = a.row_slot[row];
   if (slot < 0) return;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, j = lane & 3;
-  const int DP = a.dim_p, VP = a.vdim_p, pitch = p.pitch;
-  const int h0 = blockIdx.y * NH, n_heads = min(NH, a.heads - h0);
-  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(ld_smem);               // [NH][pitch]
-  __nv_bfloat16* sK = sQ + (size_t)NH * pitch;                                 // [2][64][pitch]
-  float* sS = reinterpret_cast<float*>(sK + (size_t)2 * NFN_PAGE * pitch);     // [2][NH][LD_S]: the two halves' scores
-  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(sS + 2 * NH * LD_S);    // [NH][LD_P]
+  const uint32_t stage_bytes = p.panels * LD_PANEL;
+  uint8_t* sK = smem;                                    // [stages][panels][64][128 B]
+  uint8_t* sP = sK + p.stages * stage_bytes;             // [NH][64 keys]
+  uint8_t* sQ = sK + (p.stages - 1) * stage_bytes;       // the queries pass through the last stage
+  uint64_t* bar_q = bars;          // TMA: queries landed
+  uint64_t* bar_qt = bars + 1;     // warp 0: queries are in TMEM, their stage is free
+  uint64_t* bar_s = bars + 2;      // MMA: scores complete
+  uint64_t* bar_sfree = bars + 3;  // warp 0: scores are in registers
+  uint64_t* bar_p = bars + 4;      // 4 arrivals: weights in shared memory (and O rescaled if needed)
+  uint64_t* bar_o = bars + 5;      // MMA: O += ... retired
+  uint64_t* bar_k = bars + 6;                      // [stages] TMA: page landed
+  uint64_t* bar_free = bars + 6 + LD_MAX_STAGES;   // [stages] MMA: the page's last product retired
+  volatile int* cta_abort = &abort_s;
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int h0 = blockIdx.y * NH, n_heads = min(NH, a.heads - h0), VP = a.vdim_p;
   const int pos = a.row_pos[row], lo = first_visible(a, pos);
   const int page0 = lo / NFN_PAGE, n_pages = pos / NFN_PAGE + 1 - page0;
-  const int p_lo = (int)((long long)n_pages * blockIdx.x / p.splits), p_hi = (int)((long long)n_pages * (blockIdx.x + 1) / p.splits);
+  const int p_lo = page0 + (int)((long long)n_pages * blockIdx.x / p.splits), n = page0 + (int)((long long)n_pages * (blockIdx.x + 1) / p.splits) - p_lo;
   const int* table = a.table + (size_t)slot * a.table_ld;
-  const __nv_bfloat16* pool = static_cast<const __nv_bfloat16*>(a.k_pool);
-  const int vecs = DP / 8;
-  auto load = [&](int i) {                                       // warp 0: two rows per lane
-    const uint32_t bar = smem_u32(&bar_full[i & 1]), dst = smem_u32(sK + (size_t)(i & 1) * NFN_PAGE * pitch);
-    const __nv_bfloat16* src = pool + (size_t)table[page0 + i] * NFN_PAGE * DP;
-    if (lane == 0) mbar_expect_tx(bar, (uint32_t)(NFN_PAGE * DP * 2));
-    __syncwarp();
-#pragma unroll
-    for (int r = lane; r < NFN_PAGE; r += 32) ld_bulk(dst + (uint32_t)(r * pitch) * 2, src + (size_t)r * DP, (uint32_t)DP * 2, bar);
-  };
-  if (tid == 0) {
+  const size_t cell = (size_t)blockIdx.z * a.heads + h0;
+  if (n <= 0) {                                          // more shares than pages
+    for (int x = threadIdx.x; x < n_heads * VP; x += AV2_THREADS) p.partial[((cell + x / VP) * p.splits + blockIdx.x) * VP + x % VP] = 0.f;
+    if ((int)threadIdx.x < n_heads) p.stats[(cell + threadIdx.x) * p.splits + blockIdx.x] = make_float2(-INFINITY, 0.f);
+    return;
+  }
+  {
+    uint32_t dyn;
+    asm volatile("mov.u32 %0, %%dynamic_smem_size;" : "=r"(dyn));
+    if (static_cast<uint32_t>(smem - smem_raw) + p.smem > dyn) {
+      if (threadIdx.x == 0 && p.status) atomicCAS(p.status, 0, NFN_ERR_WAIT_MISC);
+      return;
+    }
+  }
+  if (threadIdx.x == 0) {
     abort_s = 0;
-    mbar_init(smem_u32(&bar_full[0]), 1);
-    mbar_init(smem_u32(&bar_full[1]), 1);
+    mbar_init(smem_u32(bar_q), 1);
+    mbar_init(smem_u32(bar_qt), 1);
+    mbar_init(smem_u32(bar_s), 1);
+    mbar_init(smem_u32(bar_sfree), 1);
+    mbar_init(smem_u32(bar_p), AV2_MATH_WARPS);
+    mbar_init(smem_u32(bar_o), 1);
+    for (int i = 0; i < LD_MAX_STAGES; ++i) {
+      mbar_init(smem_u32(&bar_k[i]), 1);
+      mbar_init(smem_u32(&bar_free[i]), 1);
+    }
     fence_mbar_init();
   }
-  __syncthreads();
-  if (warp == 0 && p_lo < p_hi) load(p_lo);
-  {
-    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + (size_t)row * a.ld_q + (size_t)h0 * DP;
-    const uint4 zero4 = make_uint4(0u, 0u, 0u, 0u);
-    for (int x = tid; x < NH * vecs; x += LD_THREADS) {
-      const int r = x / vecs, c = x - r * vecs;
-      *reinterpret_cast<uint4*>(sQ + (size_t)r * pitch + c * 8) = r < n_heads ? *reinterpret_cast<const uint4*>(q + (size_t)x * 8) : zero4;
-    }
-    if (tid < NH) {
-      s_m[tid] = -INFINITY;
-      s_l[tid] = 0.f;
-    }
+  if (warp == AV2_MMA_WARP) {
+    tmem_alloc(smem_u32(&tmem_slot), p.tmem_cols);
+    tmem_relinquish();
   }
-  const float mul = a.scale * 1.4426950408889634f;
-  float acc[MT][VN][4];
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int v = 0; v < VN; ++v)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) acc[m][v][e] = 0.f;
-  const int kg = warp & 7, half = warp >> 3, steps = DP / 16, ks0 = steps * half / 2, ks1 = steps * (half + 1) / 2;
-  const uint32_t aq = smem_u32(sQ) + (uint32_t)((lane & 15) * pitch + (lane >> 4) * 8) * 2;
-  const uint32_t ap = smem_u32(sP) + (uint32_t)((lane & 15) * LD_P + (lane >> 4) * 8) * 2;
-  const uint32_t bk = (uint32_t)((kg * 8 + (lane & 7)) * pitch + (lane >> 3) * 8) * 2;
-  const uint32_t bv = (uint32_t)((((lane >> 3) & 1) * 8 + (lane & 7)) * pitch + warp * VN * 8 + (lane >> 4) * 8) * 2;
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem_base = tmem_slot, q_col = NFN_PAGE, o_col = q_col + a.dim_p / 2;      // scores, queries, outputs
 
-  __syncthreads();                                                  // queries are in place
-  for (int i = p_lo; i < p_hi; ++i) {
-    if (warp == 0 && i + 1 < p_hi) load(i + 1);
-    mbar_wait_bounded(smem_u32(&bar_full[i & 1]), ((i - p_lo) >> 1) & 1, &abort_s, p.status, NFN_ERR_WAIT_FULL);
-    const uint32_t stage = smem_u32(sK + (size_t)(i & 1) * NFN_PAGE * pitch);
-    // ---- scores: 8 keys, half of the channels, two steps of 16 per load of keys ----
-    float s[MT][4];
-#pragma unroll
-    for (int m = 0; m < MT; ++m)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) s[m][e] = 0.f;
-#pragma unroll 3
-    for (int k = ks0; k < ks1; k += 2) {
-      uint32_t b[4], q[MT][4];
-      ld_x4(b, stage + bk + k * 32);
-#pragma unroll
-      for (int m = 0; m < MT; ++m) ld_x4(q[m], aq + (uint32_t)(m * 16 * pitch) * 2 + k * 32);
-#pragma unroll
-      for (int m = 0; m < MT; ++m) ld_mma(s[m], q[m], b[0], b[1]);
-      if (k + 1 < ks1) {
-#pragma unroll
-        for (int m = 0; m < MT; ++m) ld_x4(q[m], aq + (uint32_t)(m * 16 * pitch) * 2 + k * 32 + 32);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) ld_mma(s[m], q[m], b[2], b[3]);
+  if (warp == AV2_TMA_WARP) {
+    // ------------------------------------------------------------ TMA producer --
+    if (lane == 0) {
+      auto load = [&](int j) {
+        const int st = j % p.stages;
+        const uint32_t fb = smem_u32(&bar_k[st]), dst = smem_u32(sK + st * stage_bytes);
+        const int r = table[p_lo + j] * NFN_PAGE;
+        mbar_expect_tx(fb, stage_bytes);
+        for (int d = 0; d < p.panels; ++d) tma_load_2d(dst + d * LD_PANEL, &tm_c, fb, d * 64, r);
+      };
+      mbar_expect_tx(smem_u32(bar_q), p.panels * Q_PANEL);
+      for (int d = 0; d < p.panels; ++d) tma_load_2d(smem_u32(sQ) + d * Q_PANEL, &tm_q, smem_u32(bar_q), d * 64, row * a.heads + h0);
+      const int ahead = min(n, p.stages - 1);
+      for (int j = 0; j < ahead; ++j) load(j);
+      for (int j = ahead; j < n; ++j) {
+        const bool ok = j == p.stages - 1 ? mbar_wait_bounded(smem_u32(bar_qt), 0, cta_abort, p.status, 0x700 + 1)
+                                          : mbar_wait_bounded(smem_u32(&bar_free[j % p.stages]), (j / p.stages - 1) & 1, cta_abort, p.status, 0x700 + 1);
+        if (!ok) break;
+        load(j);
       }
     }
+  } else if (warp == AV2_MMA_WARP) {
+    // -------------------------------------------------------------- MMA issuer --
+    if (lane == 0) {
+      const uint32_t idesc_s = make_idesc_bf16(128, NFN_PAGE, 0, 0), idesc_o = make_idesc_bf16(128, NH, 1, 0);
+      const int k_steps = a.dim_p / 16;
+      auto issue_s = [&](int j) {
+        const uint32_t sk = smem_u32(sK + (j % p.stages) * stage_bytes);
+        tc_fence_after();
+#pragma unroll 4
+        for (int kk = 0; kk < k_steps; ++kk)             // 16 channels of the queries are 8 TMEM columns
+          umma_bf16_ts(tmem_base, tmem_base + q_col + kk * 8, make_smem_desc_sw128(sk + (kk / 4) * LD_PANEL + (kk % 4) * 32, 16, 1024), idesc_s, kk != 0);
+        umma_commit(smem_u32(bar_s));
+      };
+      auto page_here = [&](int j) { return mbar_wait_bounded(smem_u32(&bar_k[j % p.stages]), (j / p.stages) & 1, cta_abort, p.status, 0x700 + 2); };
+      bool ok = mbar_wait_bounded(smem_u32(bar_qt), 0, cta_abort, p.status, 0x700 + 3) && page_here(0);
+      if (ok) issue_s(0);
+      for (int j = 0; j < n && ok; ++j) {
+        // the next scores first if their page is here, else this page's outputs
+        bool ahead = j + 1 >= n;
+        ok = mbar_wait_bounded(smem_u32(bar_sfree), j & 1, cta_abort, p.status, 0x700 + 4);
+        if (!ok) break;
+        if (!ahead && mbar_try_wait(smem_u32(&bar_k[(j + 1) % p.stages]), ((j + 1) / p.stages) & 1)) {
+          issue_s(j + 1);
+          ahead = true;
+        }
+        ok = mbar_wait_bounded(smem_u32(bar_p), j & 1, cta_abort, p.status, 0x700 + 5);
+        if (!ok) break;
+        tc_fence_after();
+        const uint32_t sv = smem_u32(sK + (j % p.stages) * stage_bytes), sp = smem_u32(sP);
+        for (int t = 0; t < p.m_tiles; ++t)
 #pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      float* dst = sS + (size_t)(half * NH + m * 16 + g) * LD_S + kg * 8 + 2 * j;
-      *reinterpret_cast<float2*>(dst) = make_float2(s[m][0], s[m][1]);
-      *reinterpret_cast<float2*>(dst + 8 * LD_S) = make_float2(s[m][2], s[m][3]);
-    }
-    __syncthreads();
-    if (*static_cast<volatile int*>(&abort_s)) break;               // a wait ran out: set before the barrier, so all leave together
-    // ---- softmax: LD_THREADS / NH threads per head, a few keys each ----
-    {
-      constexpr int SHARE = LD_THREADS / NH, KEYS = NFN_PAGE / SHARE;
-      const int h = tid / SHARE, k0 = tid % SHARE * KEYS, key0 = (page0 + i) * NFN_PAGE + k0;
-      const float *s0 = sS + (size_t)h * LD_S + k0, *s1 = s0 + (size_t)NH * LD_S;
-      float x[KEYS], mx = -INFINITY;
-#pragma unroll
-      for (int e = 0; e < KEYS; ++e) {
-        x[e] = key0 + e >= lo && key0 + e <= pos ? (s0[e] + s1[e]) * mul : -INFINITY;
-        mx = fmaxf(mx, x[e]);
-      }
-#pragma unroll
-      for (int o = 1; o < SHARE; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
-      const float m_old = s_m[h], m_new = fmaxf(m_old, mx);         // every page holds a visible key: finite
-      float sum = 0.f;
-#pragma unroll
-      for (int e = 0; e < KEYS; ++e) {
-        x[e] = exp2f(x[e] - m_new);
-        sum += x[e];
-      }
-#pragma unroll
-      for (int o = 1; o < SHARE; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
-#pragma unroll
-      for (int e = 0; e < KEYS; e += 2) *reinterpret_cast<uint32_t*>(sP + (size_t)h * LD_P + k0 + e) = pack_bf16x2(x[e], x[e + 1]);
-      __syncwarp();                                                 // a head's threads share a warp: its maximum is read by all before it changes
-      if (tid % SHARE == 0) {
-        const float alpha = exp2f(m_old - m_new);                   // 0 on the first page
-        s_alpha[h] = alpha;
-        s_l[h] = s_l[h] * alpha + sum;
-        s_m[h] = m_new;
-      }
-    }
-    __syncthreads();
-    // ---- output: this warp's latent channels ----
-#pragma unroll
-    for (int m = 0; m < MT; ++m) {
-      const float a0 = s_alpha[m * 16 + g], a1 = s_alpha[m * 16 + g + 8];
-#pragma unroll
-      for (int v = 0; v < VN; ++v) {
-        acc[m][v][0] *= a0; acc[m][v][1] *= a0; acc[m][v][2] *= a1; acc[m][v][3] *= a1;
-      }
-    }
-#pragma unroll
-    for (int kk = 0; kk < NFN_PAGE / 16; ++kk) {
-      uint32_t pf[MT][4];
-#pragma unroll
-      for (int m = 0; m < MT; ++m) ld_x4(pf[m], ap + (uint32_t)(m * 16 * LD_P) * 2 + kk * 32);
-#pragma unroll
-      for (int v = 0; v < VN; v += 2) {
-        if ((warp * VN + v) * 8 >= VP) break;                       // channels come in whole sixteens
-        uint32_t b[4];
-        ld_x4_t(b, stage + bv + (uint32_t)(kk * 16 * pitch) * 2 + v * 16);
-#pragma unroll
-        for (int m = 0; m < MT; ++m) {
-          ld_mma(acc[m][v], pf[m], b[0], b[1]);
-          ld_mma(acc[m][v + 1], pf[m], b[2], b[3]);
+          for (int kk = 0; kk < NFN_PAGE / 16; ++kk)
+            umma_bf16_ss(tmem_base + o_col + t * NH, make_smem_desc_sw128(sv + 2 * t * LD_PANEL + kk * (16 * 128), LD_PANEL, 1024),
+                         make_smem_desc_sw128(sp + kk * 32, 16, 1024), idesc_o, (j | kk) != 0);
+        umma_commit(smem_u32(bar_o));
+        umma_commit(smem_u32(&bar_free[j % p.stages]));
+        if (!ahead) {
+          ok = page_here(j + 1);
+          if (ok) issue_s(j + 1);
         }
       }
     }
-    __syncthreads();                                                // the stage takes the page after the next
-  }
-  __syncthreads();
-  if (abort_s) {
-    for (int i = 0; i < 64; ++i) __nanosleep(1000);                 // copies in flight land
-    return;
+  } else {
+    // ------------------------------------------------------------- math threads --
+    const uint32_t t_row = tmem_base + (static_cast<uint32_t>(warp * 32) << 16);
+    const float mul = a.scale * 1.4426950408889634f;
+    const int head = lane % NH;                          // of warp 0's threads
+    float m_run = -INFINITY, l_run = 0.f;
+    bool ok = true;
+    if (warp == 0) {                                     // queries to TMEM: a head's row is a lane's
+      ok = mbar_wait_bounded(smem_u32(bar_q), 0, cta_abort, p.status, 0x700 + 6);
+      ok = __all_sync(0xffffffffu, ok);
+#pragma unroll 1
+      for (int c = 0; c < a.dim_p / 32; ++c) {
+        uint32_t u[16];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int ch = c * 4 + e;                      // 16-byte piece of the row
+          *reinterpret_cast<uint4*>(&u[4 * e]) = *reinterpret_cast<const uint4*>(sQ + (ch / 8) * Q_PANEL + head * 128 + (((ch % 8) ^ (head & 7)) << 4));
+        }
+        tmem_st_32x16(t_row + q_col + c * 16, u);
+      }
+      if (a.dim_p % 32) {                                // the last sixteen channels; what is stored behind them is overwritten by the first output
+        const int c = a.dim_p / 32;
+        uint32_t u[16] = {};
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const int ch = c * 4 + e;
+          *reinterpret_cast<uint4*>(&u[4 * e]) = *reinterpret_cast<const uint4*>(sQ + (ch / 8) * Q_PANEL + head * 128 + (((ch % 8) ^ (head & 7)) << 4));
+        }
+        tmem_st_32x16(t_row + q_col + c * 16, u);
+      }
+      tmem_st_wait();
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(bar_qt));
+    }
+    for (int j = 0; j < n; ++j) {
+      uint32_t s[NFN_PAGE];
+      float m_new = m_run;
+      if (warp == 0) {
+        ok = mbar_wait_bounded(smem_u32(bar_s), j & 1, cta_abort, p.status, 0x700 + 7);
+        ok = __all_sync(0xffffffffu, ok);
+        tc_fence_after();
+        tmem_ld_row<NFN_PAGE>(t_row, s);
+        tmem_ld_wait();
+        tc_fence_before();
+        __syncwarp();
+        if (lane == 0) mbar_arrive(smem_u32(bar_sfree));
+        const int kbase = (p_lo + j) * NFN_PAGE;
+#pragma unroll
+        for (int i = 0; i < NFN_PAGE; i += 2) {
+          float x0, x1;
+          mul2(x0, x1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]), mul, mul);
+          s[i] = __float_as_uint(x0);
+          s[i + 1] = __float_as_uint(x1);
+        }
+        if (kbase < lo || kbase + NFN_PAGE - 1 > pos) {
+#pragma unroll
+          for (int i = 0; i < NFN_PAGE; ++i)
+            if (kbase + i < lo || kbase + i > pos) s[i] = 0xff800000u;      // -inf
+        }
+        float mx[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+        for (int i = 0; i < NFN_PAGE; i += 8)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) mx[e] = fmax3(mx[e], __uint_as_float(s[i + 2 * e]), __uint_as_float(s[i + 2 * e + 1]));
+        m_new = fmaxf(m_run, fmaxf(fmaxf(mx[0], mx[1]), fmaxf(mx[2], mx[3])));      // every page holds a visible key: finite
+        const bool grow = __any_sync(0xffffffffu, m_new - m_run > 8.f);
+        if (grow) s_alpha[j & 1][head] = exp2f(m_run - m_new);
+        if (lane == 0) s_flag[j & 1] = grow;
+      }
+      asm volatile("bar.sync 1, 128;" ::: "memory");
+      if (*cta_abort) ok = false;                        // set before the barrier by whoever ran out of patience
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) break;
+      const bool rescale = s_flag[j & 1];
+      if (warp == 0) {
+        if (rescale) {
+          l_run *= exp2f(m_run - m_new);
+          m_run = m_new;
+        }
+#pragma unroll
+        for (int i = 0; i < NFN_PAGE; i += 2) {
+          float x0, x1;
+          add2f(x0, x1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]), -m_run, -m_run);
+          s[i] = __float_as_uint(x0);
+          s[i + 1] = __float_as_uint(x1);
+        }
+#pragma unroll
+        for (int i = 0; i < NFN_PAGE; ++i) s[i] = __float_as_uint(fast_exp2(__uint_as_float(s[i])));
+        float l0 = 0.f, l1 = 0.f, l2 = 0.f, l3 = 0.f;
+#pragma unroll
+        for (int i = 0; i < NFN_PAGE; i += 4) {
+          add2(l0, l1, __uint_as_float(s[i]), __uint_as_float(s[i + 1]));
+          add2(l2, l3, __uint_as_float(s[i + 2]), __uint_as_float(s[i + 3]));
+        }
+        l_run += (l0 + l1) + (l2 + l3);
+      }
+      if (j > 0 && (warp == 0 || rescale)) {
+        // the last product must have retired before its weights are overwritten and O is rescaled
+        ok = mbar_wait_bounded(smem_u32(bar_o), (j - 1) & 1, cta_abort, p.status, 0x700 + 8);
+        ok = __all_sync(0xffffffffu, ok);
+        if (!ok) continue;                               // all four warps leave together, at the next barrier
+        tc_fence_after();
+        if (rescale) {
+#pragma unroll 1
+          for (int c = 0; c < p.m_tiles * (NH / 16); ++c) {
+            uint32_t o[16];
+            tmem_ld_32x16(t_row + o_col + c * 16, o);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 16; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * s_alpha[j & 1][(c * 16 + i) % NH]);
+            tmem_st_32x16(t_row + o_col + c * 16, o);
+          }
+          tmem_st_wait();
+        }
+      }
+      if (warp == 0) {
+        if (lane < NH) {
+#pragma unroll
+          for (int c = 0; c < NFN_PAGE / 8; ++c) {
+            const uint32_t* e = &s[c * 8];
+            st_swizzled_row_chunk(sP, NH, lane, c,
+                                  make_uint4(pack_bf16x2(__uint_as_float(e[0]), __uint_as_float(e[1])), pack_bf16x2(__uint_as_float(e[2]), __uint_as_float(e[3])),
+                                             pack_bf16x2(__uint_as_float(e[4]), __uint_as_float(e[5])), pack_bf16x2(__uint_as_float(e[6]), __uint_as_float(e[7]))));
+          }
+        }
+        fence_proxy_async();
+      }
+      tc_fence_before();
+      __syncwarp();
+      if (lane == 0) mbar_arrive(smem_u32(bar_p));
+    }
+    // ---- O^T: a thread holds one channel of all heads ----
+    if (warp == 0) s_sum[head] = l_run;
+    asm volatile("bar.sync 1, 128;" ::: "memory");
+    if (*cta_abort) ok = false;
+    if (ok) ok = mbar_wait_bounded(smem_u32(bar_o), (n - 1) & 1, cta_abort, p.status, 0x700 + 9);
+    ok = __all_sync(0xffffffffu, ok);
+    if (ok) {
+      tc_fence_after();
+      if (p.splits > 1 && warp == 0 && lane < n_heads) p.stats[(cell + lane) * p.splits + blockIdx.x] = make_float2(m_run, l_run);
+      __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (size_t)row * a.ld_o + (size_t)h0 * VP;
+#pragma unroll 1
+      for (int t = 0; t < p.m_tiles; ++t) {
+        uint32_t o[NH];
+#pragma unroll
+        for (int c = 0; c < NH / 16; ++c) tmem_ld_32x16(t_row + o_col + t * NH + c * 16, *reinterpret_cast<uint32_t(*)[16]>(&o[c * 16]));
+        tmem_ld_wait();
+        const int ch = t * 128 + warp * 32 + lane;
+        if (ch < VP) {
+#pragma unroll
+          for (int h = 0; h < NH; ++h) {
+            if (h >= n_heads) break;
+            if (p.splits == 1) out[(size_t)h * VP + ch] = __float2bfloat16(__uint_as_float(o[h]) / s_sum[h]);
+            else p.partial[((cell + h) * p.splits + blockIdx.x) * VP + ch] = __uint_as_float(o[h]);
+          }
+        }
+      }
+    }
   }
 
-  __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (size_t)row * a.ld_o + (size_t)h0 * VP;
-  const size_t cell = (size_t)blockIdx.z * a.heads + h0;
-#pragma unroll
-  for (int m = 0; m < MT; ++m)
-#pragma unroll
-    for (int e2 = 0; e2 < 2; ++e2) {
-      const int h = m * 16 + g + 8 * e2;
-      const float inv = s_l[h] > 0.f ? 1.f / s_l[h] : 0.f;
-      if (h >= n_heads) continue;
-      float* part = p.partial + ((cell + h) * p.splits + blockIdx.x) * VP;
-#pragma unroll
-      for (int v = 0; v < VN; ++v) {
-        const int c = (warp * VN + v) * 8 + 2 * j;
-        if (c >= VP) break;
-        if (p.splits == 1) *reinterpret_cast<uint32_t*>(out + (size_t)h * VP + c) = pack_bf16x2(acc[m][v][2 * e2] * inv, acc[m][v][2 * e2 + 1] * inv);
-        else *reinterpret_cast<float2*>(part + c) = make_float2(acc[m][v][2 * e2], acc[m][v][2 * e2 + 1]);
-      }
-      if (p.splits > 1 && warp == 0 && j == 0) p.stats[(cell + h) * p.splits + blockIdx.x] = make_float2(s_m[h], s_l[h]);
-    }
+  tc_fence_before();
+  __syncthreads();
+  if (*cta_abort) {
+    for (int i = 0; i < 64; ++i) __nanosleep(1000);       // copies in flight land
+  }
+  if (warp == AV2_MMA_WARP) {
+    tc_fence_after();
+    tmem_dealloc(tmem_base, p.tmem_cols);
+  }
 }
 
 // A CTA takes one head of a row, a thread four channels.
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const LatentDecodeParams p) {
+  constexpr int AT_ONCE = 8;
   const nfn_paged_attention_args& a = p.a;
   const int row = a.row0 + blockIdx.y, h = blockIdx.x, c = threadIdx.x * 4;
   if (a.row_slot[row] < 0 || c >= a.vdim_p) return;
@@ -239,11 +350,11 @@ latent_merge_kernel(const LatentDecodeParams p) {
   const float* part = p.partial + cell * p.splits * a.vdim_p + c;
   float m = -INFINITY, l = 0.f;
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-  for (int s0 = 0; s0 < p.splits; s0 += 8) {
-    float2 t[8];
-    float4 v[8];
+  for (int s0 = 0; s0 < p.splits; s0 += AT_ONCE) {
+    float2 t[AT_ONCE];
+    float4 v[AT_ONCE];
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < AT_ONCE; ++i) {
       const int s = min(s0 + i, p.splits - 1);
       t[i] = stats[s];
       v[i] = load4(part + (size_t)s * a.vdim_p);
@@ -251,14 +362,14 @@ latent_merge_kernel(const LatentDecodeParams p) {
     }
     float m_new = m;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) m_new = fmaxf(m_new, t[i].x);
-    if (m_new == -INFINITY) continue;                       // shares without pages
+    for (int i = 0; i < AT_ONCE; ++i) m_new = fmaxf(m_new, t[i].x);
+    if (m_new == -INFINITY) continue;                     // shares without pages
     const float keep = exp2f(m - m_new);
     l *= keep;
     o.x *= keep; o.y *= keep; o.z *= keep; o.w *= keep;
     m = m_new;
 #pragma unroll
-    for (int i = 0; i < 8; ++i) {
+    for (int i = 0; i < AT_ONCE; ++i) {
       const float f = exp2f(t[i].x - m_new);
       l += f * t[i].y;
       o.x += f * v[i].x; o.y += f * v[i].y; o.z += f * v[i].z; o.w += f * v[i].w;
@@ -268,47 +379,53 @@ latent_merge_kernel(const LatentDecodeParams p) {
   store4(static_cast<__nv_bfloat16*>(a.out) + (size_t)row * a.ld_o + (size_t)h * a.vdim_p + c, make_float4(o.x * inv, o.y * inv, o.z * inv, o.w * inv));
 }
 
-template <int MT, int VN>
-static int launch_latent_decode(LatentDecodeParams p, size_t smem, cudaStream_t st) {
-  auto kern = latent_decode_kernel<MT, VN>;
-  static size_t raised[64] = {};
+template <int NH>
+static int launch_latent_decode(LatentDecodeParams p, const CUtensorMap& tq, const CUtensorMap& tc, cudaStream_t st) {
+  auto kern = latent_decode_kernel<NH>;
+  static uint32_t raised[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
-  if (smem > 40 * 1024 && raised[dev & 63] < smem) {
-    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) return launch_check("latent_decode attr", 0);
-    raised[dev & 63] = smem;
+  if (raised[dev & 63] < p.smem + 1024) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)p.smem + 1024) != cudaSuccess) return launch_check("latent_decode attr", 0);
+    raised[dev & 63] = p.smem + 1024;
   }
-  const nfn_paged_attention_args a = p.a;
-  const int blocks = ceil_div(a.heads, MT * 16);
-  for (int r = 0; r < a.rows; r += 65535) {
-    p.a.row0 = a.row0 + r;
-    const int n = std::min(a.rows - r, 65535);
-    kern<<<dim3(p.splits, blocks, n), LD_THREADS, smem, st>>>(p);
-    if (p.splits > 1) latent_merge_kernel<<<dim3(a.heads, n), 128, 0, st>>>(p);
-  }
+  const nfn_paged_attention_args& a = p.a;
+  kern<<<dim3(p.splits, ceil_div(a.heads, NH), a.rows), AV2_THREADS, p.smem + 1024, st>>>(tq, tc, p);
+  if (p.splits > 1) latent_merge_kernel<<<dim3(a.heads, a.rows), 128, 0, st>>>(p);
   return launch_check("latent_decode", p.splits > 1 ? 2 : 1);
 }
 
+// What lies behind the stages: the weights, and at least a panel where a product over whole 128-channel tiles reads past the last panel.
+static uint32_t latent_tail(int panels, int m_tiles, int nh) { return std::max<uint32_t>(nh * 128, 2 * m_tiles > panels ? LD_PANEL : 0); }
+
 // 1: sizes outside the kernel's limits
 int latent_decode(const nfn_paged_attention_args& a, cudaStream_t st) {
-  if (a.vdim_p > 512 || (a.dim_p & 15) || (a.vdim_p & 15) || (a.ld_q & 7) || a.slopes || a.softcap > 0.f || a.sink || a.keep_first > 0 || a.gate) return 1;
-  LatentDecodeParams p;
+  constexpr uint32_t LIMIT = 227 * 1024 - 2048;            // static shared memory and the alignment of the dynamic part aside
+  if (a.vdim_p > 512 || ((a.dim_p | a.vdim_p) & 15) || a.ld_q != a.heads * a.dim_p || a.rows > 65535 || a.slopes || a.softcap > 0.f || a.sink || a.keep_first > 0 || a.gate) return 1;
+  LatentDecodeParams p{};
   p.a = a;
-  p.pitch = a.dim_p + 8;
+  p.panels = ceil_div(a.dim_p, 64);
+  p.m_tiles = ceil_div(a.vdim_p, 128);
+  const int nh = a.heads > 16 && NFN_PAGE + a.dim_p / 2 + p.m_tiles * 32 <= 512 ? 32 : 16;
+  const int cols = NFN_PAGE + a.dim_p / 2 + std::max(p.m_tiles * nh, 8);      // the queries' last store may reach eight columns further
+  const uint32_t stage = p.panels * LD_PANEL, tail = latent_tail(p.panels, p.m_tiles, nh);
+  p.stages = 3 * stage + tail <= LIMIT ? 3 : 2;
+  p.smem = p.stages * stage + tail;
+  if (cols > 512 || p.smem > LIMIT || p.panels * nh * 128 > (int)stage) return 1;
+  p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;
   p.status = status_ptr();
-  const int mt = a.heads > 16 ? 2 : 1, nh = 16 * mt;
-  const size_t smem = (size_t)(nh + 2 * NFN_PAGE) * p.pitch * 2 + (size_t)2 * nh * LD_S * 4 + (size_t)nh * LD_P * 2;
-  if (smem > 220 * 1024) return 1;
-  // one wave of what is resident at a time, at least one page each
+  // one wave of what is resident at a time, at least a page each
   const long long ctas = (long long)a.rows * ceil_div(a.heads, nh), cells = (long long)a.rows * a.heads;
-  const int resident = (int)std::max<size_t>(1, (size_t)(220 * 1024) / smem);
-  long long splits = std::min<long long>(ceil_div(a.max_keys, NFN_PAGE) + 1, std::max<long long>(1, (long long)sm_count() * std::min(resident, 4) / ctas));
+  const int resident = std::min<int>(228 * 1024 / (p.smem + 3072), 512 / p.tmem_cols);
+  long long splits = std::min<long long>(ceil_div(a.max_keys, NFN_PAGE) + 1, std::max<long long>(1, (long long)sm_count() * std::max(resident, 1) / ctas));
   splits = std::min<long long>(std::min<long long>(splits, 64), (a.workspace_bytes - PAGED_COUNTER_BYTES) / (cells * (a.vdim_p * 4 + 8)));
   p.splits = (int)std::max<long long>(splits, 1);
   p.partial = reinterpret_cast<float*>(static_cast<char*>(a.workspace) + PAGED_COUNTER_BYTES);
   p.stats = reinterpret_cast<float2*>(p.partial + cells * p.splits * a.vdim_p);
-  if (mt == 1) return a.vdim_p <= 256 ? launch_latent_decode<1, 2>(p, smem, st) : launch_latent_decode<1, 4>(p, smem, st);
-  return a.vdim_p <= 256 ? launch_latent_decode<2, 2>(p, smem, st) : launch_latent_decode<2, 4>(p, smem, st);
+  CUtensorMap tq, tc;
+  if (!make_tmap_2d(&tq, a.q, 2, a.dim_p, (uint64_t)(a.row0 + a.rows) * a.heads, a.dim_p, 64, nh, 128)) return -3;
+  if (!make_tmap_2d(&tc, a.k_pool, 2, a.dim_p, (uint64_t)a.pages * NFN_PAGE, a.dim_p, 64, NFN_PAGE, 128)) return -3;
+  return nh == 32 ? launch_latent_decode<32>(p, tq, tc, st) : launch_latent_decode<16>(p, tq, tc, st);
 }
 
 }  // namespace nfn
