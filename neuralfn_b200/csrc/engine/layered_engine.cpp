@@ -169,7 +169,7 @@ struct layered_engine final : nfn_engine {
   void attention_args(const Layer& L, nfn_paged_attention_args* a);
   int post_pass(const Batch& b);
   // wkv: single tokens in one launch after the products, few rows through one launch for the four projections
-  bool wkv_step(const Layer& L, const Batch& b) const { return b.single && nfn_wkv_step_fits(b.rows, L.d.heads, L.dp); }
+  bool wkv_step(const Layer& L, const Batch& b) const { return b.single && nfn_wkv_step_fits(b.rows, L.dp); }
   bool grouped(const Layer& L, int rows) const { return c.dtype == 0 && L.d.experts <= 256 && L.d.top <= 32 && (long long)rows * L.d.top > 8LL * L.d.experts; }
   // single tokens of delta layers: convolution, rule, norm and gate in one launch
   bool one_step(const Layer& L, const Batch& b) const { return b.single && L.d.mixer == NFN_MIXER_DELTA && nfn_delta_step_fits(b.rows, L.d.heads, L.dp, L.vp); }

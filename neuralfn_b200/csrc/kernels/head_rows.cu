@@ -43,6 +43,18 @@ __device__ __forceinline__ float4 rotate4(const float4& v, const float2* cs, int
   return o;
 }
 
+// the same for dimensions c .. c + 7
+__device__ __forceinline__ void rotate8(float (&v)[8], const float2* cs, int c, int rot_dims) {
+#pragma unroll
+  for (int e = 0; e < 8; e += 2)
+    if (c + e + 1 < rot_dims) {
+      const float2 a = cs[(c + e) / 2];
+      const float x = v[e] * a.x - v[e + 1] * a.y;
+      v[e + 1] = v[e + 1] * a.x + v[e] * a.y;
+      v[e] = x;
+    }
+}
+
 __device__ __forceinline__ float warp_sum(float v) {
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
@@ -60,16 +72,27 @@ head_rows_kernel(const nfn_head_rows_args p) {
   if (t.slot < 0) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dims / 2;
   const int pos0 = t.e_pos0 + t.row0 - t.e_row0;
+  const int item = blockIdx.y * HR_WARPS + warp;
+  const bool key = item >= p.heads, on = item < p.heads + p.kv_heads;
+  const int head = key ? item - p.heads : item;
+  const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
+  const T* src = in + (key ? p.off_k : 0) + head * p.dim_p;
+  float4 v[R][NV];
+  auto fetch = [&](int i0) {
+#pragma unroll
+    for (int i = 0; i < R; ++i)
+#pragma unroll
+      for (int j = 0; j < NV; ++j) {
+        const int c = lane * 4 + j * 128;
+        v[i][j] = on && i0 + i < t.n && c < p.dim_p ? load4(src + (size_t)(i0 + i) * p.ld_in + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+  };
+  fetch(0);                                               // on their way while the angles are formed
   fill_rotations(hr_cs, p.freq, half, pos0, t.n);
   __syncthreads();
-  const int item = blockIdx.y * HR_WARPS + warp;
-  const bool key = item >= p.heads;
-  const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
   const size_t page = p.kv_heads > 0 ? (size_t)p.table[(size_t)t.slot * p.table_ld + pos0 / NFN_PAGE] : 0;
   const int in_page = pos0 % NFN_PAGE;
-  if (item < p.heads + p.kv_heads) {
-    const int head = key ? item - p.heads : item;
-    const T* src = in + (key ? p.off_k : 0) + head * p.dim_p;
+  if (on) {
     T* dst = key ? static_cast<T*>(p.k_pool) + ((page * p.kv_heads + head) * NFN_PAGE + in_page) * p.dim_p
                  : static_cast<T*>(p.q_out) + (size_t)t.row0 * p.ld_q + head * p.dim_p;
     const int ld_dst = key ? p.dim_p : p.ld_q;
@@ -81,14 +104,7 @@ head_rows_kernel(const nfn_head_rows_args p) {
       w[j] = weight && c < p.dim_p ? load4(weight + c) : make_float4(1.f, 1.f, 1.f, 1.f);
     }
     for (int i0 = 0; i0 < t.n; i0 += R) {
-      float4 v[R][NV];
-#pragma unroll
-      for (int i = 0; i < R; ++i)
-#pragma unroll
-        for (int j = 0; j < NV; ++j) {
-          const int c = lane * 4 + j * 128;
-          v[i][j] = i0 + i < t.n && c < p.dim_p ? load4(src + (size_t)(i0 + i) * p.ld_in + c) : make_float4(0.f, 0.f, 0.f, 0.f);
-        }
+      if (i0 > 0) fetch(i0);
 #pragma unroll
       for (int i = 0; i < R; ++i) {
         if (i0 + i >= t.n) break;
@@ -110,19 +126,30 @@ head_rows_kernel(const nfn_head_rows_args p) {
       }
     }
   }
-  // values, channel-major
+  // values, channel-major: two neighbouring channels per thread
   const int n_v = p.kv_heads * p.vdim_p;
-  for (int ch = blockIdx.y * HR_THREADS + threadIdx.x; ch < n_v; ch += gridDim.y * HR_THREADS) {
-    const T* src = in + p.off_v + ch;
+  struct alignas(2 * sizeof(T)) Pair { T a, b; };
+  for (int ch = 2 * (blockIdx.y * HR_THREADS + threadIdx.x); ch < n_v; ch += 2 * gridDim.y * HR_THREADS) {
+    const T* from = in + p.off_v + ch;
     T* dst = static_cast<T*>(p.v_pool) + (page * n_v + ch) * NFN_PAGE + in_page;
     if (t.n == HR_ROWS) {
-      T buf[HR_ROWS];
+      T buf[2][HR_ROWS];
 #pragma unroll
-      for (int i = 0; i < HR_ROWS; ++i) buf[i] = src[(size_t)i * p.ld_in];
+      for (int i = 0; i < HR_ROWS; ++i) {
+        const Pair f = *reinterpret_cast<const Pair*>(from + (size_t)i * p.ld_in);
+        buf[0][i] = f.a;
+        buf[1][i] = f.b;
+      }
 #pragma unroll
-      for (int q = 0; q < HR_ROWS * (int)sizeof(T) / 16; ++q) reinterpret_cast<uint4*>(dst)[q] = pack16(&buf[q * (16 / sizeof(T))]);
+      for (int e = 0; e < 2; ++e)
+#pragma unroll
+        for (int q = 0; q < HR_ROWS * (int)sizeof(T) / 16; ++q) reinterpret_cast<uint4*>(dst + e * NFN_PAGE)[q] = pack16(&buf[e][q * (16 / sizeof(T))]);
     } else {
-      for (int i = 0; i < t.n; ++i) dst[i] = src[(size_t)i * p.ld_in];
+      for (int i = 0; i < t.n; ++i) {
+        const Pair f = *reinterpret_cast<const Pair*>(from + (size_t)i * p.ld_in);
+        dst[i] = f.a;
+        dst[NFN_PAGE + i] = f.b;
+      }
     }
   }
 }
@@ -137,7 +164,6 @@ latent_rows_kernel(const nfn_latent_rows_args p) {
   if (t.slot < 0 || (of_keys && !p.k_pool)) return;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, half = p.rot_dim / 2;
   const int pos0 = t.e_pos0 + t.row0 - t.e_row0;
-  fill_rotations(hr_cs, p.freq, half, pos0, t.n);
   const int pitch = p.dim_p + p.rot_p, lp = p.rank_p + p.rot_p;
   const T* in = static_cast<const T*>(p.in) + (size_t)t.row0 * p.ld_in;
   if (!of_keys) {
@@ -147,24 +173,28 @@ latent_rows_kernel(const nfn_latent_rows_args p) {
     T* dst = lat ? static_cast<T*>(p.q_lat) + (size_t)t.row0 * p.heads * lp + (size_t)head * lp + p.rank_p
                  : static_cast<T*>(p.q_out) + (size_t)t.row0 * p.ld_q + head * pitch + p.dim_p;
     const size_t ld_dst = lat ? (size_t)p.heads * lp : (size_t)p.ld_q;
-    // pieces of four over the tile's rows, four per lane in flight: narrow rotated parts leave no lane idle
-    const int quads = p.rot_p / 4, total = on ? quads * t.n : 0;
-    float4 v[4];
+    // pieces of eight over the tile's rows, four per lane in flight: narrow rotated parts leave no lane idle
+    const int pieces = p.rot_p / 8, total = on ? pieces * t.n : 0;
+    float v[4][8];
     auto fetch = [&](int x0) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int x = x0 + 32 * e;
-        if (x < total) v[e] = load4(src + (size_t)(x / quads) * p.ld_in + p.dim_p + x % quads * 4);
+        if (x < total) load8(src + (size_t)(x / pieces) * p.ld_in + p.dim_p + x % pieces * 8, v[e]);
       }
     };
-    fetch(lane);
+    fetch(lane);                                          // on their way while the angles are formed
+    fill_rotations(hr_cs, p.freq, half, pos0, t.n);
     __syncthreads();
     for (int x0 = lane; x0 < total; x0 += 128) {
       if (x0 != lane) fetch(x0);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        const int x = x0 + 32 * e, i = x / quads, c = x % quads * 4;
-        if (x < total) store4(dst + i * ld_dst + c, rotate4(v[e], hr_cs + i * half, c, p.rot_dim));
+        const int x = x0 + 32 * e, i = x / pieces, c = x % pieces * 8;
+        if (x < total) {
+          rotate8(v[e], hr_cs + i * half, c, p.rot_dim);
+          store8(dst + i * ld_dst + c, v[e]);
+        }
       }
     }
     if (on && !lat && p.q_out != p.in)
@@ -172,6 +202,7 @@ latent_rows_kernel(const nfn_latent_rows_args p) {
         for (int c = lane * 4; c < p.dim_p; c += 128) store4(dst + i * ld_dst - p.dim_p + c, load4(src + (size_t)i * p.ld_in + c));
     return;
   }
+  fill_rotations(hr_cs, p.freq, half, pos0, t.n);
   __syncthreads();
   const size_t page = (size_t)p.table[(size_t)t.slot * p.table_ld + pos0 / NFN_PAGE];
   T* dst = static_cast<T*>(p.k_pool) + (page * NFN_PAGE + pos0 % NFN_PAGE) * lp;

@@ -545,7 +545,7 @@ int nfn_wkv_chunks(const nfn_wkv_args* args, int max_rows, void* workspace, long
 // left out in bf16, [rows][rank_p] in 32-bit mode.
 int nfn_tanh_split(int f32, const float* in, int ld_in, void* out, int ld_out, int rows, int rank_p, nfn_stream_t stream);
 // One token of every sequence: decay (with its outer projection w2 [heads * dim_p][ld_w2], low fp32 [rows][rank_p] before the tanh), rule, output norm, gate.
-// rkvg: rows [r | k | v | g]; tiles: one per row. nfn_wkv_step_fits: the sizes and row counts it takes.
+// rkvg: rows [r | k | v | g]; tiles: one per row. nfn_wkv_step_fits: the sizes it takes.
 typedef struct {
   int f32, rows;
   const void* rkvg; int ld_rkvg;
@@ -558,7 +558,7 @@ typedef struct {
   void* out; int ld_out;
   const nfn_row_tile* tiles;
 } nfn_wkv_step_args;
-int nfn_wkv_step_fits(int rows, int heads, int dim_p);
+int nfn_wkv_step_fits(int rows, int dim_p);
 int nfn_wkv_step(const nfn_wkv_step_args* args, nfn_stream_t stream);
 
 // ---- mixture of experts for the rows of a step (moe.cu, moe_rows.cu) ----------------------------------------------------------

@@ -288,15 +288,13 @@ extern "C" int nfn_tanh_split(int f32, const float* in, int ld_in, void* out, in
   return launch_check("tanh_split");
 }
 
-extern "C" int nfn_wkv_step_fits(int rows, int heads, int dim_p) {
-  return dim_p <= WS_THREADS / 32 * WR_COLS && (long long)rows * heads <= 4LL * sm_count();
-}
+extern "C" int nfn_wkv_step_fits(int rows, int dim_p) { return dim_p <= WS_THREADS / 32 * WR_COLS && rows <= 65535; }
 
 extern "C" int nfn_wkv_step(const nfn_wkv_step_args* args, nfn_stream_t stream) {
   if (!args) return fail(-1, "wkv step: null args");
   const nfn_wkv_step_args& a = *args;
   if (a.rows <= 0) return 0;
-  if (a.heads <= 0 || (a.dim_p & 15) || a.dim > a.dim_p || !nfn_wkv_step_fits(1, 1, a.dim_p)) return fail(-1, "wkv step: heads of at most 128 channels, padded to multiples of 16");
-  if ((a.rank_p & 15) || a.rank_p <= 0 || a.rank_p > 8192 || (a.ld_w2 & 3) || (a.ld_rkvg & 7) || a.rows > 65535) return fail(-1, "wkv step: misaligned rows, or too many");
+  if (a.heads <= 0 || (a.dim_p & 15) || a.dim > a.dim_p || !nfn_wkv_step_fits(a.rows, a.dim_p)) return fail(-1, "wkv step: heads of at most 128 channels, padded to multiples of 16, and at most 65535 rows");
+  if ((a.rank_p & 15) || a.rank_p <= 0 || a.rank_p > 8192 || (a.ld_w2 & 3) || (a.ld_rkvg & 7)) return fail(-1, "wkv step: misaligned rows");
   return a.f32 ? launch_wkv_step<float>(a, static_cast<cudaStream_t>(stream)) : launch_wkv_step<__nv_bfloat16>(a, static_cast<cudaStream_t>(stream));
 }
