@@ -22,6 +22,11 @@ struct DeltaChunkParams {
   unsigned char* blocks;      // [seq][chunk][head][dc_block_bytes]
   float* uo;                  // [seq][chunk][head][dc_uo_floats]
   int* status;
+  // segs > 1 (without corrections only): a round's chunks in segments of seg_chunks that run side by side
+  int segs, seg_chunks;
+  float* seg_init;            // [seq][head][dim_p][vdim_p]: the state before the round
+  float* seg_state;           // [seq][seg][head][dim_p][vdim_p]: what a segment adds (the first one: with seg_init decayed)
+  float* seg_gamma;           // [seq][seg][head][dk]: what it leaves of the state before it
 };
 
 // two fp32 values as bf16 pairs: the rounded values and what they leave out

@@ -13,7 +13,9 @@
 //                         and K arrive in fragment order by bulk copies through a ring of shared memory stages.
 //
 // The products with the state are formed from fp32 values split into two bf16 parts each (high x high + high x low + low x high), which
-// keeps sixteen bits of every factor. The scan also runs recurrences without corrections (U = V, no W: wkv_chunk.cu). Rounds of as many chunks as the workspace holds alternate between the two kernels, small enough
+// keeps sixteen bits of every factor. The scan also runs recurrences without corrections (U = V, no W: wkv_chunk.cu).
+// Their states are linear in what comes before, so where heads are few a round is cut into segments: segment_state_kernel runs every segment but the
+// last from zero, without read-outs, and the scan of each segment starts from the sum of what the earlier ones leave. Rounds of as many chunks as the workspace holds alternate between the two kernels, small enough
 // to stay in L2.
 #include <algorithm>
 
@@ -285,17 +287,18 @@ delta_scan_kernel(const DeltaChunkParams p) {
   __shared__ int cta_abort_s;
   volatile int* cta_abort = &cta_abort_s;
   const nfn_delta_args& a = p.a;
-  const nfn_seq_rows seq = a.seqs[blockIdx.z];
-  const int total = (seq.n + DC_T - 1) / DC_T, n_chunks = min(p.n_chunks, total - p.chunk0);
+  const int segs = CORRECTIONS ? 1 : p.segs, sq = blockIdx.z / segs, seg = blockIdx.z % segs, i0 = seg * (CORRECTIONS ? 0 : p.seg_chunks);
+  const nfn_seq_rows seq = a.seqs[sq];
+  const int total = (seq.n + DC_T - 1) / DC_T, here = min(p.n_chunks, total - p.chunk0), n_chunks = segs > 1 ? min(p.seg_chunks, here - i0) : here;
   if (seq.slot < 0 || n_chunks <= 0) return;
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, j = lane & 3;
   const int ks = warp % KS, h = blockIdx.y, DP = a.dim_p, VP = a.vdim_p;
   const int vt = blockIdx.x * TILES + warp / KS;
   const bool on = vt * 16 < VP;                                   // warps past the last column tile keep the others company
   float* xch = reinterpret_cast<float*>(dc_smem + STAGES * STAGE);
-  const unsigned char* blocks = p.blocks + ((size_t)blockIdx.z * p.n_chunks * a.heads + h) * BLOCK;
+  const unsigned char* blocks = p.blocks + (((size_t)sq * p.n_chunks + i0) * a.heads + h) * BLOCK;
   const size_t block_step = (size_t)a.heads * BLOCK;
-  const float* uo = p.uo + ((size_t)blockIdx.z * p.n_chunks * a.heads + h) * dc_uo_floats(VP) + blockIdx.x * TILES * 512;
+  const float* uo = p.uo + (((size_t)sq * p.n_chunks + i0) * a.heads + h) * dc_uo_floats(VP) + blockIdx.x * TILES * 512;
   const size_t uo_step = (size_t)a.heads * dc_uo_floats(VP);
   const uint32_t uo_bytes = min(TILES, VP / 16 - (int)blockIdx.x * TILES) * 2048;
 
@@ -315,13 +318,36 @@ delta_scan_kernel(const DeltaChunkParams p) {
   float* st = a.state + ((size_t)seq.slot * a.heads + h) * DP * VP + vt * 16 + g;
   const bool fresh = seq.pos0 == 0 && p.chunk0 == 0;
   float s[DS_N][4];
+  auto take = [&](const float* from, bool live) {                // a state as it lies in memory
 #pragma unroll
-  for (int t = 0; t < DS_N; ++t)
+    for (int t = 0; t < DS_N; ++t)
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
-      s[t][e] = (on && !fresh && d < DP) ? st[(size_t)d * VP + (e >> 1) * 8] : 0.f;
+      for (int e = 0; e < 4; ++e) {
+        const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
+        s[t][e] = (live && on && d < DP) ? from[(size_t)d * VP + (e >> 1) * 8] : 0.f;
+      }
+  };
+  if (segs == 1) {
+    take(st, !fresh);
+  } else if (seg == 0) {
+    take(p.seg_init + ((size_t)sq * a.heads + h) * DP * VP + vt * 16 + g, true);
+  } else {
+    const size_t cell = (size_t)sq * segs * a.heads + h;         // of the first segment
+    take(p.seg_state + cell * DP * VP + vt * 16 + g, true);
+    for (int q = 1; q < seg; ++q) {
+      const float* add = p.seg_state + (cell + (size_t)q * a.heads) * DP * VP + vt * 16 + g;
+      const float* left = p.seg_gamma + (cell + (size_t)q * a.heads) * DK + DS_CH * ks + 2 * j;
+#pragma unroll
+      for (int t = 0; t < DS_N; ++t) {
+        const float2 f = *reinterpret_cast<const float2*>(left + 8 * t);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
+          if (on && d < DP) s[t][e] = s[t][e] * ((e & 1) ? f.y : f.x) + add[(size_t)d * VP + (e >> 1) * 8];
+        }
+      }
     }
+  }
   __syncthreads();
   // Products that every warp of a column tile adds up: W S of this chunk, which the next state waits for, and Q S of the chunk before, which
   // nothing waits for and which is formed while the partial sums of W S cross shared memory.
@@ -382,7 +408,7 @@ delta_scan_kernel(const DeltaChunkParams p) {
         const float2 f = *reinterpret_cast<const float2*>(all + w * 512);
         t.x += f.x; t.y += f.y;
       }
-      const int r0 = (p.chunk0 + i) * DC_T + 8 * tile + 2 * j;
+      const int r0 = (p.chunk0 + i0 + i) * DC_T + 8 * tile + 2 * j;
       float* dst = a.o + (size_t)(seq.row0 + r0) * a.ld_o + (size_t)h * VP + vt * 16 + g + 4 * c;
       if (r0 < seq.n) dst[0] = t.x;
       if (r0 + 1 < seq.n) dst[a.ld_o] = t.y;
@@ -450,7 +476,7 @@ delta_scan_kernel(const DeltaChunkParams p) {
     for (int i = 0; i < 64; ++i) __nanosleep(1000);     // copies in flight land
     return;
   }
-  if (!on) return;
+  if (!on || i0 + n_chunks < here) return;                        // the last segment leaves the state
 #pragma unroll
   for (int t = 0; t < DS_N; ++t)
 #pragma unroll
@@ -458,6 +484,124 @@ delta_scan_kernel(const DeltaChunkParams p) {
       const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
       if (d < DP) st[(size_t)d * VP + (e >> 1) * 8] = s[t][e];
     }
+}
+
+// What each segment but the last adds to the state and leaves of the one before it. Roles and fragments as in the scan.
+constexpr int SG_STAGES = 4;
+__host__ __device__ constexpr int sg_stage_bytes(int ks) { return DS_CH * ks * 68 + DS_WARPS / ks * 1024; }      // K, e^G_last; V of the CTA's column tiles
+template <int KS>
+__global__ void __launch_bounds__(DS_WARPS * 32)
+segment_state_kernel(const DeltaChunkParams p) {
+  constexpr int DK = DS_CH * KS, TILES = DS_WARPS / KS, BLOCK = dc_block_bytes(DK, false), PART = DK * 68, STAGE = sg_stage_bytes(KS);
+  extern __shared__ __align__(128) unsigned char dc_smem[];       // [SG_STAGES][STAGE]
+  __shared__ __align__(8) uint64_t bar_full[SG_STAGES];
+  __shared__ int cta_abort_s;
+  volatile int* cta_abort = &cta_abort_s;
+  const nfn_delta_args& a = p.a;
+  const int sq = blockIdx.z / (p.segs - 1), seg = blockIdx.z % (p.segs - 1), i0 = seg * p.seg_chunks;
+  const nfn_seq_rows seq = a.seqs[sq];
+  const int total = (seq.n + DC_T - 1) / DC_T, here = min(p.n_chunks, total - p.chunk0);
+  if (seq.slot < 0 || i0 >= here) return;
+  const int n_chunks = i0 + p.seg_chunks < here ? p.seg_chunks : 0;      // 0: the last one, only the state before the round is noted
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, j = lane & 3;
+  const int ks = warp % KS, h = blockIdx.y, DP = a.dim_p, VP = a.vdim_p;
+  const int vt = blockIdx.x * TILES + warp / KS, tiles = min(TILES, VP / 16 - (int)blockIdx.x * TILES);
+  const bool on = vt * 16 < VP;
+  const unsigned char* blocks = p.blocks + (((size_t)sq * p.n_chunks + i0) * a.heads + h) * BLOCK + DK * 64;
+  const float* uo = p.uo + (((size_t)sq * p.n_chunks + i0) * a.heads + h) * dc_uo_floats(VP) + blockIdx.x * TILES * 512;
+  const size_t block_step = (size_t)a.heads * BLOCK, uo_step = (size_t)a.heads * dc_uo_floats(VP);
+  auto load = [&](int i) {
+    const uint32_t bar = smem_u32(&bar_full[i % SG_STAGES]), dst = smem_u32(dc_smem + (i % SG_STAGES) * STAGE);
+    mbar_expect_tx(bar, PART + tiles * 1024);
+    dc_bulk_load(dst, blocks + i * block_step, PART, bar);
+    for (int t = 0; t < tiles; ++t) dc_bulk_load(dst + PART + t * 1024, uo + i * uo_step + t * 512, 1024, bar);
+  };
+  if (tid == 0) {
+    cta_abort_s = 0;
+    for (int s = 0; s < SG_STAGES; ++s) mbar_init(smem_u32(&bar_full[s]), 1);
+    fence_mbar_init();
+    for (int i = 0; i < min(SG_STAGES, n_chunks); ++i) load(i);
+  }
+  const size_t cell = ((size_t)sq * p.segs + seg) * a.heads + h;
+  float s[DS_N][4], left[DS_N][2];
+#pragma unroll
+  for (int t = 0; t < DS_N; ++t) {
+    left[t][0] = left[t][1] = 1.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) s[t][e] = 0.f;
+  }
+  if (seg == 0 && on) {
+    const float* st = a.state + ((size_t)seq.slot * a.heads + h) * DP * VP + vt * 16 + g;
+    float* init = p.seg_init + ((size_t)sq * a.heads + h) * DP * VP + vt * 16 + g;
+    const bool fresh = seq.pos0 == 0 && p.chunk0 == 0;
+#pragma unroll
+    for (int t = 0; t < DS_N; ++t)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
+        if (d < DP) {
+          s[t][e] = fresh ? 0.f : st[(size_t)d * VP + (e >> 1) * 8];
+          init[(size_t)d * VP + (e >> 1) * 8] = s[t][e];
+        }
+      }
+  }
+  __syncthreads();
+  for (int i = 0; i < n_chunks; ++i) {
+    mbar_wait_bounded(smem_u32(&bar_full[i % SG_STAGES]), (i / SG_STAGES) & 1, cta_abort, p.status, NFN_ERR_WAIT_FULL);
+    const unsigned char* stage = dc_smem + (i % SG_STAGES) * STAGE;
+    const float* tv = reinterpret_cast<const float*>(stage + PART) + (on ? warp / KS : 0) * 256 + lane * 4;
+    const float4 v0 = *reinterpret_cast<const float4*>(tv), v1 = *reinterpret_cast<const float4*>(tv + 128);
+    const uint32_t uh[4] = {pack_bf16x2(v0.x, v0.y), pack_bf16x2(v0.z, v0.w), pack_bf16x2(v1.x, v1.y), pack_bf16x2(v1.z, v1.w)};
+    const float* gamma = reinterpret_cast<const float*>(stage + DK * 64) + DS_CH * ks + 2 * j;
+    uint4 kb[DS_N];
+#pragma unroll
+    for (int t = 0; t < DS_N; ++t) {
+      const float2 f = *reinterpret_cast<const float2*>(gamma + 8 * t);
+      kb[t] = *reinterpret_cast<const uint4*>(stage + dc_piece<false>(DS_N * ks + t, lane, true));
+      s[t][0] *= f.x; s[t][1] *= f.y; s[t][2] *= f.x; s[t][3] *= f.y;
+      left[t][0] *= f.x; left[t][1] *= f.y;
+    }
+#pragma unroll
+    for (int t = 0; t < DS_N; ++t) dc_mma(s[t], uh, kb[t].x, kb[t].z);
+#pragma unroll
+    for (int t = 0; t < DS_N; ++t) dc_mma(s[t], uh, kb[t].y, kb[t].w);
+    __syncthreads();                                    // every warp is done with the stage
+    if (*cta_abort) break;                              // set before the barrier: all leave together
+    if (tid == 0 && i + SG_STAGES < n_chunks) load(i + SG_STAGES);
+  }
+  if (*cta_abort) {
+    for (int i = 0; i < 64; ++i) __nanosleep(1000);     // copies in flight land
+    return;
+  }
+  if (n_chunks == 0 || !on) return;
+  float* add = p.seg_state + cell * DP * VP + vt * 16 + g;
+#pragma unroll
+  for (int t = 0; t < DS_N; ++t)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int d = DS_CH * ks + 8 * t + 2 * j + (e & 1);
+      if (d < DP) add[(size_t)d * VP + (e >> 1) * 8] = s[t][e];
+    }
+  if (vt == 0 && g == 0) {
+    float* gm = p.seg_gamma + cell * DK + DS_CH * ks + 2 * j;
+#pragma unroll
+    for (int t = 0; t < DS_N; ++t) *reinterpret_cast<float2*>(gm + 8 * t) = make_float2(left[t][0], left[t][1]);
+  }
+}
+
+template <int KS>
+static int launch_segments(const DeltaChunkParams& p, cudaStream_t st) {
+  constexpr int SMEM = SG_STAGES * sg_stage_bytes(KS);
+  auto kern = segment_state_kernel<KS>;
+  static bool raised[64] = {};
+  int dev = 0;
+  cudaGetDevice(&dev);
+  if (SMEM > 40 * 1024 && !raised[dev & 63]) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return launch_check("segment_state attr", 0);
+    raised[dev & 63] = true;
+  }
+  kern<<<dim3(ceil_div(p.a.vdim_p, 16 * (DS_WARPS / KS)), p.a.heads, p.a.n_seqs * (p.segs - 1)), DS_WARPS * 32, SMEM, st>>>(p);
+  return launch_check("segment_state");
 }
 
 template <int KS, bool CORRECTIONS>
@@ -471,12 +615,14 @@ static int launch_scan(const DeltaChunkParams& p, cudaStream_t st) {
     if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM) != cudaSuccess) return launch_check("delta_scan attr", 0);
     raised[dev & 63] = true;
   }
-  kern<<<dim3(ceil_div(p.a.vdim_p, 16 * (DS_WARPS / KS)), p.a.heads, p.a.n_seqs), DS_WARPS * 32, SMEM, st>>>(p);
+  kern<<<dim3(ceil_div(p.a.vdim_p, 16 * (DS_WARPS / KS)), p.a.heads, p.a.n_seqs * (CORRECTIONS ? 1 : p.segs)), DS_WARPS * 32, SMEM, st>>>(p);
   return launch_check("delta_scan");
 }
 
 int chunk_scan(const DeltaChunkParams& p, bool corrections, cudaStream_t st) {
   if (corrections) return p.dk == 64 ? launch_scan<1, true>(p, st) : p.dk == 128 ? launch_scan<2, true>(p, st) : launch_scan<4, true>(p, st);
+  if (p.segs > 1)
+    if (const int rc = p.dk == 64 ? launch_segments<1>(p, st) : p.dk == 128 ? launch_segments<2>(p, st) : launch_segments<4>(p, st)) return rc;
   return p.dk == 64 ? launch_scan<1, false>(p, st) : p.dk == 128 ? launch_scan<2, false>(p, st) : launch_scan<4, false>(p, st);
 }
 
@@ -513,8 +659,9 @@ extern "C" int nfn_delta_chunks(const nfn_delta_args* args, int max_rows, void* 
   if (args->n_seqs <= 0 || max_rows <= 0) return 0;
   if (const char* why = delta_args_problem(*args)) return fail(-1, why);
   if (args->f32 || args->dim_p > 256) return fail(-1, "delta rule: chunks are for bf16 activations and at most 256 key channels");
-  DeltaChunkParams p;
+  DeltaChunkParams p{};
   p.a = *args;
+  p.segs = 1;
   p.dk = args->dim_p <= 64 ? 64 : args->dim_p <= 128 ? 128 : 256;
   p.status = status_ptr();
   const long long per_chunk = (long long)args->n_seqs * args->heads * (dc_block_bytes(p.dk, true) + dc_uo_floats(args->vdim_p) * 4LL);

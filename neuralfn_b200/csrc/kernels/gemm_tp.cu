@@ -539,7 +539,9 @@ extern "C" int nfn_gemm_tp(const nfn_gemm_tp_args* args, nfn_stream_t stream_) {
     if (a.m <= 0 || a.n <= 0 || a.k <= 0 || (a.k & 7) || (a.n & 7) || (a.lda & 7) || (a.ldb & 7) || (a.ldc & 7)) return fail(-1, "gemm_tp: grouped sizes and leading dimensions must be multiples of 8");
     if (!a.a || !a.b || !a.c || !a.tile_group || !a.num_m_tiles_dev || a.groups <= 0) return fail(-1, "gemm_tp: grouped mode needs a, b, c, tile_group, num_m_tiles_dev and groups");
     if (a.m % TP_BM) return fail(-1, "gemm_tp: grouped row capacity must be a multiple of 128");
-    return (a.n >= 2048) ? launch_tp<256, 4>(a, stream) : launch_tp<128, 6>(a, stream);
+    // the wide tile, unless its last column tile would be mostly padding
+    const bool wide_tile = a.n >= 2048 || (a.n >= 1024 && (a.n + 255) / 256 * 256 - a.n <= a.n / 8);
+    return wide_tile ? launch_tp<256, 4>(a, stream) : launch_tp<128, 6>(a, stream);
   }
   if (a.m <= 0 || a.n <= 0 || a.k <= 0) return fail(-1, "gemm_tp: empty problem");
   if (a.world < 1 || a.world > TP_MAX_WORLD || a.rank < 0 || a.rank >= a.world) return fail(-1, "gemm_tp: bad rank / world (at most 8 ranks)");

@@ -202,10 +202,14 @@ using namespace nfn;
 
 static int wkv_dk(int dim_p) { return dim_p <= 64 ? 64 : dim_p <= 128 ? 128 : 256; }
 
+constexpr int WC_MAX_SEGS = 8, WC_MIN_SEG = 8;           // segments of a round, and fewest chunks of one
+// bytes the segments of a sequence take beside the operands
+static long long segment_bytes(int heads, int dim_p) { return (long long)heads * ((WC_MAX_SEGS + 1LL) * dim_p * dim_p + (long long)WC_MAX_SEGS * wkv_dk(dim_p)) * 4; }
+
 extern "C" long long nfn_wkv_chunk_workspace_bytes(int heads, int dim_p, int max_seqs) {
   if (dim_p > 256) return 0;
-  // at least one chunk of every head and sequence
-  return std::max<long long>(DC_WORKSPACE, (long long)max_seqs * heads * (dc_block_bytes(wkv_dk(dim_p), false) + dc_uo_floats(dim_p) * 4LL));
+  // at least one chunk of every head and sequence; segments are for few sequences
+  return std::max<long long>(DC_WORKSPACE, (long long)max_seqs * heads * (dc_block_bytes(wkv_dk(dim_p), false) + dc_uo_floats(dim_p) * 4LL)) + segment_bytes(heads, dim_p);
 }
 
 extern "C" int nfn_wkv_chunks(const nfn_wkv_args* args, int max_rows, void* workspace, long long workspace_bytes, nfn_stream_t stream) {
@@ -227,14 +231,26 @@ extern "C" int nfn_wkv_chunks(const nfn_wkv_args* args, int max_rows, void* work
   p.c.dk = wkv_dk(args->dim_p);
   p.c.status = status_ptr();
   const int block = dc_block_bytes(p.c.dk, false);
+  // where heads and columns leave SMs idle, a round runs in segments side by side
+  const int ctas = ceil_div(args->dim_p, 16 * (256 / p.c.dk)) * args->heads * args->n_seqs;
+  const long long seg_bytes = args->n_seqs * segment_bytes(args->heads, args->dim_p);
+  int segs = std::min(WC_MAX_SEGS, 2 * sm_count() / ctas);
+  // two would cost in extra passes what they gain
+  if (segs > 2 && workspace_bytes > 2 * seg_bytes) workspace_bytes = (workspace_bytes - seg_bytes) / 256 * 256;
+  else segs = 1;
   const long long per_chunk = (long long)args->n_seqs * args->heads * (block + dc_uo_floats(args->dim_p) * 4LL);
   const int total = ceil_div(max_rows, DC_T), round = (int)std::min<long long>(total, workspace_bytes / per_chunk);
   if (!workspace || round < 1) return fail(-1, "wkv: the workspace holds no chunk");
   p.c.blocks = static_cast<unsigned char*>(workspace);
   p.c.uo = reinterpret_cast<float*>(p.c.blocks + (size_t)round * args->n_seqs * args->heads * block);
+  p.c.seg_init = reinterpret_cast<float*>(static_cast<unsigned char*>(workspace) + workspace_bytes);
+  p.c.seg_state = p.c.seg_init + (size_t)args->n_seqs * args->heads * args->dim_p * args->dim_p;
+  p.c.seg_gamma = p.c.seg_state + (size_t)args->n_seqs * WC_MAX_SEGS * args->heads * args->dim_p * args->dim_p;
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   for (p.c.chunk0 = 0; p.c.chunk0 < total; p.c.chunk0 += round) {
     p.c.n_chunks = std::min(round, total - p.c.chunk0);
+    p.c.segs = std::max(1, std::min(segs, p.c.n_chunks / WC_MIN_SEG));
+    p.c.seg_chunks = ceil_div(p.c.n_chunks, p.c.segs);
     int rc = p.c.dk == 64 ? launch_wkv_prepare<32>(p, st) : p.c.dk == 128 ? launch_wkv_prepare<64>(p, st) : launch_wkv_prepare<128>(p, st);
     if (rc == 0) rc = chunk_scan(p.c, false, st);
     if (rc) return rc;

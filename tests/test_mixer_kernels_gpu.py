@@ -227,10 +227,13 @@ def wkv_reference(x, z, w0, u, state, heads, dim, dp):
     return out, S
 
 
-@pytest.mark.parametrize("heads,dim,dtype,form", [(h, d, t, f) for h, d in ((3, 64), (2, 24), (2, 128), (5, 80), (1, 200), (2, 16)) for t, f in ((torch.float32, "rows"), (torch.bfloat16, "rows"),
-                                                                                                                                              (torch.bfloat16, "chunks"))])
+FORMS = [(torch.float32, "rows"), (torch.bfloat16, "rows"), (torch.bfloat16, "chunks"), (torch.bfloat16, "segments")]
+
+
+@pytest.mark.parametrize("heads,dim,dtype,form", [(h, d, t, f) for h, d in ((3, 64), (2, 24), (2, 128), (5, 80), (1, 200), (2, 16)) for t, f in FORMS])
 def test_wkv_rule(heads, dim, dtype, form):
-    lengths = [1, 15, 16, 17, 100, 333]
+    """Token after token; sixteen at a time, a few chunks per round; rounds in segments that run side by side."""
+    lengths = [1, 15, 16, 17, 100, 333, 700]
     x, z, w0, u, state, dp = wkv_problem(heads, dim, lengths, dtype)
     seqs, base = [], 0
     for s, n in enumerate(lengths):
@@ -238,7 +241,7 @@ def test_wkv_rule(heads, dim, dtype, form):
         base += n
     before = state.clone()
     ws = torch.empty(len(lengths) * heads * 3 * 65536, device=DEV, dtype=torch.uint8) if form == "chunks" else None      # a few chunks per round
-    o = Y.wkv_rule(x, z, w0, u, state, ints(seqs + [[0, 5, -1, 0]]), dim=dim, form=form, workspace=ws, longest=333)
+    o = Y.wkv_rule(x, z, w0, u, state, ints(seqs + [[0, 5, -1, 0]]), dim=dim, form="rows" if form == "rows" else "chunks", workspace=ws, longest=700)
     tol = 3e-5 if form == "rows" else 1e-3
     for b, n, s, p in seqs:
         want, S = wkv_reference(x[b:b + n], z[b:b + n], w0, u, before[s] * (p > 0), heads, dim, dp)
