@@ -353,13 +353,13 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
         tmem_st_wait();
       } else {
 #pragma unroll
-      for (int c = 0; c < PP_BN / 8; ++c) {
-        const uint32_t* e = &s[c * 8];
-        st_swizzled_row_chunk(sP, PP_BM, r, c,
-                              make_uint4(pack_bf16x2(__uint_as_float(e[0]), __uint_as_float(e[1])), pack_bf16x2(__uint_as_float(e[2]), __uint_as_float(e[3])),
-                                         pack_bf16x2(__uint_as_float(e[4]), __uint_as_float(e[5])), pack_bf16x2(__uint_as_float(e[6]), __uint_as_float(e[7]))));
-      }
-      fence_proxy_async();
+        for (int c = 0; c < PP_BN / 8; ++c) {
+          const uint32_t* e = &s[c * 8];
+          st_swizzled_row_chunk(sP, PP_BM, r, c,
+                                make_uint4(pack_bf16x2(__uint_as_float(e[0]), __uint_as_float(e[1])), pack_bf16x2(__uint_as_float(e[2]), __uint_as_float(e[3])),
+                                           pack_bf16x2(__uint_as_float(e[4]), __uint_as_float(e[5])), pack_bf16x2(__uint_as_float(e[6]), __uint_as_float(e[7]))));
+        }
+        fence_proxy_async();
       }
       tc_fence_before();
       __syncwarp();
