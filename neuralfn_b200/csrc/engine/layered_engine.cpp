@@ -13,14 +13,14 @@
 // visible latents for the pass.
 //
 // Recurrent layers have no pages: a slot keeps one fp32 state per head, read and written in place (and, for the token shift, the previous input in two
-// halves like the convolutions' history). Layers of a loop share tensors and have caches and states of their own.
+// halves like the convolutions' history; convolutions on the sublayers' inputs keep theirs the same way, in every layer). Layers of a loop share tensors and have caches and states of their own.
 //
 // A step lays its rows out short entries first (single tokens and portions below kTileMin rows: one query row at a time), then
 // the long ones (tcgen05 tiles). Per layer it launches: input projection (q | k | v | gates | feed-forward in one product), the
 // row mix (convolution, temperature, cache append, feed-forward gate), attention with the output gate, one output product that
 // adds mixer and feed-forward to the 32-bit residual stream, and the token input's two products with their norm, which also
 // produces the next layer's normalised rows. `chained` models run mixer and feed-forward as two sublayers with a stream pass after each
-// (chained_pass). Steps of single tokens run with a padded row count and are replayed as CUDA graphs.
+// (chained_pass; post_pass where outputs are normed). Steps of single tokens run with a padded row count and are replayed as CUDA graphs.
 #include <cmath>
 #include <cstring>
 #include <memory>
@@ -59,10 +59,17 @@ struct Layer {
   const void *mu = nullptr, *w1 = nullptr, *w2 = nullptr, *w0 = nullptr, *u = nullptr;
   const void *w_shared_up = nullptr, *w_shared_down = nullptr, *correction = nullptr;
   float* prev = nullptr;                            // token shift: [2][slots][wp]
+  struct { const void *norm_b = nullptr, *conv = nullptr; void* history = nullptr; } sub[2];   // sandwich: mixer, feed-forward; [2][slots][taps - 1][wp]
+  const void *sinks = nullptr, *bias_gate_up = nullptr, *bias_down = nullptr;
+  float* powers = nullptr;                          // linear: [heads][NFN_LINEAR_CHUNK + 1]
+  std::vector<double> decay;
   bool paged() const { return d.mixer == NFN_MIXER_ATTENTION || d.mixer == NFN_MIXER_LATENT; }
   bool latent() const { return d.mixer == NFN_MIXER_LATENT; }
   int key_row() const { return latent() ? lr + rp : d.kv_heads * dp; }       // values of one token's key and value rows in the pages
   int value_row() const { return latent() ? 0 : d.kv_heads * vp; }
+  long long memory_floats() const { return d.mixer == NFN_MIXER_GRU ? vp : d.mixer == NFN_MIXER_DELTA || d.mixer == NFN_MIXER_WKV || d.mixer == NFN_MIXER_LINEAR ? (long long)d.heads * dp * vp : 0; }
+  nfn_gate_clamp clamp() const { return nfn_gate_clamp{d.ff_limit, d.ff_slope, 1.f}; }
+  bool has_ff() const { return d.experts > 0 || d.ff > 0; }
   int look() const { return d.chunk > 0 ? d.chunk : d.window; }              // most positions a query sees, 0: all
   struct { const void *in = nullptr, *out = nullptr, *mix = nullptr; } hc[2];   // streams: mixer, feed-forward
   int tile_rows = 0;                                // query rows per tcgen05 tile, 0: one row at a time
@@ -100,7 +107,7 @@ struct layered_engine final : nfn_engine {
   int es = 2;                                       // bytes per activation
   int wp = 0, vp = 0, sp = 0, max_pages = 0, rows_max = 0, logit_rows = 0, n_in_max = 0, nq_max = 0, cat_max = 0;
   float* x = nullptr;
-  void *xb = nullptr, *h = nullptr, *in = nullptr, *q = nullptr, *cat = nullptr, *s_act = nullptr, *y = nullptr, *hw = nullptr;
+  void *xb = nullptr, *h = nullptr, *hc = nullptr, *in = nullptr, *q = nullptr, *cat = nullptr, *s_act = nullptr, *y = nullptr, *hw = nullptr;
   float *s_gate = nullptr, *logits = nullptr, *saved = nullptr;
   float *decay = nullptr, *d_o = nullptr;           // delta: projected decays, read-outs
   void *d_gate = nullptr, *delta_ws = nullptr;
@@ -110,6 +117,10 @@ struct layered_engine final : nfn_engine {
   void *q_lat = nullptr, *o_lat = nullptr, *lat_rows = nullptr, *lat_x = nullptr;   // latent: absorbed queries and outputs of short rows; gathered latents, expansion
   int lat_cap = 0;                                  // rows of the last two
   void *shift = nullptr, *low_act = nullptr, *shared_mid = nullptr, *y_shared = nullptr;
+  const void* hx = nullptr;                         // what the sublayer at hand reads: h, or hc behind the convolution on its input
+  int* row_count = nullptr;                         // linear: one counter per row
+  void* linear_ws = nullptr;
+  long long linear_ws_bytes = 0;
   float* low = nullptr;
   void* wkv_ws = nullptr;
   long long wkv_ws_bytes = 0;
@@ -163,14 +174,18 @@ struct layered_engine final : nfn_engine {
   int rotated_attention(const Layer& L, const Batch& b);
   int latent_attention(const Layer& L, const Batch& b);
   int wkv(const Layer& L, const Batch& b);
+  int linear(const Layer& L, const Batch& b);
+  int gru(const Layer& L, const Batch& b);
   int mixer(const Layer& L, const Batch& b);
   int dense_ff(const Layer& L, int rows);
   bool rotated(const Layer& L) const { return L.d.mixer == NFN_MIXER_ATTENTION && (L.d.rot_dims > 0 || L.d.qk_norm || L.d.key_values); }
   void attention_args(const Layer& L, nfn_paged_attention_args* a);
   int post_pass(const Batch& b);
+  int enter(nfn_stream_args* s, const Layer& L, int which, const Batch& b);
   // wkv: single tokens in one launch after the products, few rows through one launch for the four projections
   bool wkv_step(const Layer& L, const Batch& b) const { return b.single && nfn_wkv_step_fits(b.rows, L.dp); }
   bool grouped(const Layer& L, int rows) const { return c.dtype == 0 && L.d.experts <= 256 && L.d.top <= 32 && (long long)rows * L.d.top > 8LL * L.d.experts; }
+  bool linear_step(const Layer& L, const Batch& b) const { return b.single && nfn_linear_step_fits(b.rows, L.dp, L.vp); }
   // single tokens of delta layers: convolution, rule, norm and gate in one launch
   bool one_step(const Layer& L, const Batch& b) const { return b.single && L.d.mixer == NFN_MIXER_DELTA && nfn_delta_step_fits(b.rows, L.d.heads, L.dp, L.vp); }
   int experts(const Layer& L, int rows, nfn_stream_args* sp);
@@ -214,15 +229,19 @@ int layered_engine::build() {
       if (d.weights_of >= l || layers[d.weights_of].d.weights_of >= 0) return efail(bad + " must take its tensors from an earlier layer that has its own");
       nfn_layer_desc a = d, o = layers[d.weights_of].d;
       a.weights_of = o.weights_of = -1;
+      a.decay = o.decay = nullptr;
+      if (L.decay != layers[d.weights_of].decay) return efail(bad + " and the layer whose tensors it uses differ");
       if (std::memcmp(&a, &o, sizeof a)) return efail(bad + " and the layer whose tensors it uses differ");
     }
-    if (c.chained ? (d.out_gate || (d.ff > 0 && d.experts > 0)) : (d.mixer != NFN_MIXER_ATTENTION || d.experts > 0 || d.qkv_bias || d.rot_dims > 0 || d.qk_norm || d.key_values))
+    if (c.chained ? ((d.out_gate && d.mixer != NFN_MIXER_LATENT) || (d.ff > 0 && d.experts > 0)) : (d.mixer != NFN_MIXER_ATTENTION || d.experts > 0 || d.qkv_bias || d.rot_dims > 0 || d.qk_norm || d.key_values))
       return efail(bad + (c.chained ? ": sublayers one after another have one feed-forward and no output gate"
                                     : ": recurrent and latent mixers, rotation, experts and biases need sublayers one after another"));
     if (d.mixer == NFN_MIXER_WKV && !c.post_norm) return efail(bad + ": the token shift reads the residual itself (post_norm)");
     if ((rotated(L) || d.mixer == NFN_MIXER_LATENT) && (d.conv_taps > 0 || d.q_temp_every > 0 || d.qkv_bias))
       return efail(bad + ": rotated and latent attention have no convolutions, query temperature or biases");
     if (!d.expert_plain && (d.shared_ff > 0 || d.route_correction || d.route_groups > 0 || d.route_normalise)) return efail(bad + ": gated experts have plain sigmoid routing and no shared expert");
+    if ((d.route_softmax || d.ff_act == NFN_ACT_CLAMPED) && d.experts > 0 && (d.expert_plain || !d.expert_weigh_out)) return efail(bad + ": softmax routing and clamped gates go with gated experts weighted at their output");
+    if ((d.mixer == NFN_MIXER_LINEAR || d.mixer == NFN_MIXER_GRU) && (d.conv_taps > 0 || (d.qkv_bias && d.mixer == NFN_MIXER_LINEAR))) return efail(bad + ": these recurrences have no convolution or such biases of their own");
     L.ep = d.experts > 0 ? up(d.experts, 16) : 0;
     L.ef = d.experts > 0 ? up(d.expert_ff, 16) : 0;
     L.dp = up(d.dim, 16);
@@ -251,11 +270,19 @@ int layered_engine::build() {
       L.rp = up(d.rot_dim, 16);
       L.nq = d.heads * (L.dp + L.rp);
       L.off_kv = L.nq;
-      L.n_in = L.nq + (own ? L.lr + L.rp : 0);
+      L.off_g = L.nq + (own ? L.lr + L.rp : 0);
+      L.n_in = L.off_g + (d.out_gate ? d.heads * L.vp : 0);
     } else if (d.mixer == NFN_MIXER_WKV) {
       L.ra = up(d.rank_decay, 16);
       L.nq = d.heads * L.dp;                       // each of r, k, v, g
       L.n_in = 4 * L.nq;
+    } else if (d.mixer == NFN_MIXER_LINEAR) {        // [q | k | v | gate]
+      L.nq = 2 * d.heads * L.dp + d.heads * L.vp;
+      L.off_g = L.nq;
+      L.n_in = L.nq + d.heads * L.vp;
+    } else if (d.mixer == NFN_MIXER_GRU) {           // [share | candidate | gate]
+      L.nq = 3 * L.vp;
+      L.n_in = L.nq;
     } else {
       L.nq = d.heads * L.dp;
       L.nk = own ? d.kv_heads * L.dp : 0;
@@ -272,7 +299,14 @@ int layered_engine::build() {
     if (!rotated(L) && (d.mixer == NFN_MIXER_ATTENTION || d.mixer == NFN_MIXER_DELTA)) nq_max = std::max(nq_max, L.nq);      // others keep their queries in place
     cat_max = std::max(cat_max, std::max(L.n_cat, L.ff));
     if (d.weights_of < 0) {
-      want(lname(l, "norm1"), wp);
+      const long long nw = c.scalar_norms ? 1 : wp;
+      want(lname(l, "norm1"), nw);
+      for (int q = 0; c.sandwich && q < (L.has_ff() ? 2 : 1); ++q) {
+        want(lname(l, q ? "norm2_b" : "norm1_b"), nw);
+        if (c.input_taps > 0) want(lname(l, q ? "in_conv2" : "in_conv1"), (long long)c.input_taps * wp);
+      }
+      if (d.sink == 2) want(lname(l, "sink"), d.heads);
+      if (d.mixer == NFN_MIXER_LINEAR) want(lname(l, "out_norm"), (long long)d.heads * L.vp);
       want(lname(l, "w_in"), (long long)L.n_in * wp);
       if (d.qk_norm) {
         want(lname(l, "q_norm"), L.dp);
@@ -292,9 +326,13 @@ int layered_engine::build() {
         want(lname(l, "out_norm"), L.nq);
       }
       if (c.chained && d.ff > 0) {
-        want(lname(l, "norm2"), wp);
+        want(lname(l, "norm2"), nw);
         want(lname(l, "w_gate_up"), 2LL * L.ff * wp);
         want(lname(l, "w_down"), (long long)wp * L.ff);
+        if (d.ff_bias) {
+          want(lname(l, "bias_gate_up"), 2LL * L.ff);
+          want(lname(l, "bias_down"), wp);
+        }
       }
       if (d.shared_ff > 0) {
         want(lname(l, "w_shared_up"), (long long)L.shp * wp);
@@ -317,7 +355,7 @@ int layered_engine::build() {
         want(lname(l, "out_norm"), L.vp);
       }
       if (d.experts > 0) {
-        want(lname(l, "norm2"), wp);
+        want(lname(l, "norm2"), nw);
         want(lname(l, "router"), (long long)L.ep * wp);
         want(lname(l, "w_gate_up"), (long long)d.experts * (d.expert_plain ? 1 : 2) * L.ef * wp);
         want(lname(l, "w_down"), (long long)d.experts * wp * L.ef);
@@ -333,7 +371,7 @@ int layered_engine::build() {
     L.tile_rows = L.latent() ? nfn_latent_tile_rows(c.dtype, L.dp, L.rp, L.vp) : nfn_paged_tile_rows(c.dtype, d.heads, d.kv_heads, L.dp, L.vp);
     if (L.tile_rows > 0 && std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) == tile_kinds.end()) tile_kinds.push_back(L.tile_rows);
   }
-  want("final_norm", wp);
+  want("final_norm", c.scalar_norms ? 1 : wp);
   // how far back the readers of each owner look, and one group per distinct answer
   for (int l = 0; l < c.n_layer; ++l) {
     if (layers[l].owner != l || !layers[l].paged()) continue;
@@ -376,7 +414,8 @@ extern "C" nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, 
   if (c.n_layer <= 0 || c.width <= 0 || c.vocab <= 0 || c.side_dim < 0 || (c.dtype != 0 && c.dtype != 1) || c.max_seq <= 0 || c.max_batch <= 0 ||
       c.kv_tokens < 0 || c.max_step_rows <= 0 || !(c.norm_eps >= 0.f) || c.streams < 0 || c.streams > NFN_MAX_STREAMS || (c.streams > 0 && !c.chained) ||
       (c.chained && c.side_dim > 0) || !(c.logit_softcap >= 0.f) || (!c.chained && c.norm_offset != 0.f) ||
-      (c.post_norm && (!c.chained || c.streams > 0 || c.norm_offset != 0.f))) {
+      (c.post_norm && (!c.chained || c.streams > 0 || c.norm_offset != 0.f)) || (c.sandwich && (!c.chained || c.streams > 0 || c.norm_offset != 0.f || c.post_norm)) ||
+      (!c.sandwich && (c.scalar_norms || c.input_taps)) || c.input_taps < 0) {
     efail("engine_create: invalid geometry");
     return nullptr;
   }
@@ -388,16 +427,20 @@ extern "C" nfn_engine* nfn_engine_create_layered(const nfn_layered_config* cfg, 
     const nfn_layer_desc& d = layers[l];
     if (d.heads <= 0 || d.kv_heads <= 0 || d.heads % d.kv_heads || d.dim <= 0 || d.vdim <= 0 || d.conv_taps < 0 || d.ff < 0 || d.window < 0 ||
         d.q_temp_every < 0 || d.keep_first < 0 || d.softcap < 0.f || d.experts < 0 || (d.experts > 0 && (d.top < 1 || d.top > d.experts || d.expert_ff < 1)) ||
-        d.mixer < NFN_MIXER_ATTENTION || d.mixer > NFN_MIXER_WKV || d.chunk < 0 || (d.chunk > 0 && (d.window > 0 || d.keep_first > 0)) || d.rot_dims < 0 ||
+        d.mixer < NFN_MIXER_ATTENTION || d.mixer > NFN_MIXER_GRU || d.chunk < 0 || (d.chunk > 0 && (d.window > 0 || d.keep_first > 0)) || d.rot_dims < 0 ||
         (d.rot_dims & 1) || (d.rot_dims > 0 && !(d.rot_base > 0.0)) || (d.mixer == NFN_MIXER_ATTENTION && (d.rot_dims > d.dim || (d.key_values && d.vdim != d.dim) || ((d.rot_dims > 0 || d.qk_norm) && d.dim > 512))) ||
-        (d.mixer == NFN_MIXER_LATENT && (d.kv_rank <= 0 || d.rot_dim <= 0 || d.rot_dims != d.rot_dim || d.rot_dim > 512 || d.kv_heads != 1 || d.keep_first > 0 || d.qk_norm || d.sink || d.softcap > 0.f || d.alibi != 0.f)) ||
+        (d.mixer == NFN_MIXER_LATENT && (d.kv_rank <= 0 || d.rot_dim <= 0 || d.rot_dims != d.rot_dim || d.rot_dim > 512 || d.kv_heads != 1 || d.keep_first > 0 || d.qk_norm || d.softcap > 0.f || d.alibi != 0.f)) ||
+        d.sink < 0 || d.sink > 2 || (d.sink && d.mixer != NFN_MIXER_ATTENTION && d.mixer != NFN_MIXER_LATENT) || (d.mixer == NFN_MIXER_LINEAR && (!d.decay || d.kv_heads != d.heads || d.dim > 512)) ||
+        (d.mixer == NFN_MIXER_GRU && (d.heads != 1 || d.dim != 1)) || (d.ff_act == NFN_ACT_CLAMPED && !(d.ff_limit > 0.f)) ||
         (d.mixer == NFN_MIXER_WKV && (d.rank_decay < 1 || d.dim > 512 || d.vdim != d.dim || d.kv_heads != d.heads)) || d.shared_ff < 0 || (d.shared_ff > 0 && d.experts <= 0) ||
         (d.route_groups > 0 && (d.experts % d.route_groups || d.route_keep < 1 || d.route_keep > d.route_groups || d.route_keep * (d.experts / d.route_groups) < d.top)) || d.route_groups < 0 ||
-        (d.mixer == NFN_MIXER_DELTA && (d.conv_taps < 1 || d.rank_decay < 1 || d.rank_gate < 1 || d.dim > 512)) || (d.ff_act != NFN_ACT_RELU && d.ff_act != NFN_ACT_SILU && d.ff_act != NFN_ACT_GELU_TANH && d.ff_act != NFN_ACT_RELU2)) {
+        (d.mixer == NFN_MIXER_DELTA && (d.conv_taps < 1 || d.rank_decay < 1 || d.rank_gate < 1 || d.dim > 512)) || (d.ff_act != NFN_ACT_RELU && d.ff_act != NFN_ACT_SILU && d.ff_act != NFN_ACT_GELU_TANH && d.ff_act != NFN_ACT_RELU2 && d.ff_act != NFN_ACT_CLAMPED)) {
       efail("engine_create: invalid sizes in layer " + std::to_string(l));
       return nullptr;
     }
     e->layers[l].d = d;
+    if (d.mixer == NFN_MIXER_LINEAR) e->layers[l].decay.assign(d.decay, d.decay + d.heads);
+    e->layers[l].d.decay = nullptr;
   }
   e->device = device;
   if (cudaSetDevice(device) != cudaSuccess || cudaStreamCreateWithFlags(&e->stream, cudaStreamNonBlocking) != cudaSuccess) {
@@ -425,11 +468,12 @@ int layered_engine::finalize() {
   if (c.dtype == 0 && zero(&xb, R * wp * 2)) return -1;
   if (sp && (zero((void**)&s_gate, R * sp * 4) || zero(&s_act, R * sp * es))) return -1;
   if ((sp || c.chained) && zero(&y, R * wp * es)) return -1;
+  if (c.input_taps > 0 && zero(&hc, R * wp * es)) return -1;
   // scratch of the delta mixers and of the experts: the largest any layer asks for
   long long n_q_lat = 0, n_o_lat = 0, n_lat = 0, n_lat_x = 0, n_low = 0, n_shift = 0, n_shared = 0;
   // rows that attend to latents themselves: short entries, or all of them where the sizes have no tiles
   const long long r_short = std::min<long long>(R, S * (kTileMin - 1));
-  long long n_dec = 0, n_do = 0, e_log = 0, e_max = 0, e_items = 0, e_sorted = 0, e_gu = 0, e_mid = 0, e_rows = 0;
+  long long n_dec = 0, n_do = 0, n_lin = 0, e_log = 0, e_max = 0, e_items = 0, e_sorted = 0, e_gu = 0, e_mid = 0, e_rows = 0;
   for (const Layer& L : layers) {
     const nfn_layer_desc& d = L.d;
     if (d.mixer == NFN_MIXER_DELTA) {
@@ -455,6 +499,10 @@ int layered_engine::finalize() {
       n_shift = 5 * R * wp;
       if (c.dtype == 0) wkv_ws_bytes = std::max(wkv_ws_bytes, nfn_wkv_chunk_workspace_bytes(d.heads, L.dp, c.max_batch));
     }
+    if (d.mixer == NFN_MIXER_LINEAR) {
+      n_lin = std::max(n_lin, R * d.heads * L.vp);
+      if (c.dtype == 0) linear_ws_bytes = std::max(linear_ws_bytes, nfn_linear_chunk_workspace_bytes(d.heads, L.dp, L.vp, c.max_batch));
+    }
     n_shared = std::max(n_shared, R * L.shp);
     if (d.experts > 0) {
       const bool g = grouped(L, (int)R);
@@ -475,7 +523,10 @@ int layered_engine::finalize() {
   if (n_shared && (zero(&shared_mid, n_shared * es) || zero(&y_shared, R * wp * es))) return -1;
   if (wkv_ws_bytes > 0 && add(&wkv_ws, wkv_ws_bytes)) return -1;
   if (delta_ws_bytes > 0 && add(&delta_ws, delta_ws_bytes)) return -1;
-  if (n_dec && (zero((void**)&decay, n_dec * 4) || zero((void**)&d_o, n_do * 4) || zero(&d_gate, n_do * es))) return -1;
+  if (n_dec && (zero((void**)&decay, n_dec * 4) || zero(&d_gate, n_do * es))) return -1;
+  if (std::max(n_do, n_lin) > 0 && zero((void**)&d_o, std::max(n_do, n_lin) * 4)) return -1;
+  if (n_lin && zero((void**)&row_count, R * 4)) return -1;
+  if (linear_ws_bytes > 0 && add(&linear_ws, linear_ws_bytes)) return -1;
   if (e_max && (zero((void**)&ex.logits, e_log * 4) || zero((void**)&ex.weight, e_items * 4) || zero((void**)&ex.idx, e_items * 4) ||
                 zero((void**)&ex.order, e_items * 4) || zero((void**)&ex.row_of, e_items * 4) || zero((void**)&ex.offsets, (e_max + 1) * 4) ||
                 zero((void**)&ex.active, (e_max + 1) * 4) || zero((void**)&ex.counts, e_max * 4) || zero((void**)&ex.cursor, e_max * 4) ||
@@ -498,10 +549,8 @@ int layered_engine::finalize() {
   for (int l = 0; l < c.n_layer; ++l) {
     Layer& L = layers[l];
     const nfn_layer_desc& d = L.d;
-    if (d.mixer == NFN_MIXER_DELTA) {
-      if (zero((void**)&L.memory, S * d.heads * L.dp * L.vp * 4)) return -1;
-    } else if (d.mixer == NFN_MIXER_WKV) {
-      if (zero((void**)&L.memory, S * d.heads * L.dp * L.dp * 4) || zero((void**)&L.prev, 2 * S * wp * 4)) return -1;
+    if (L.memory_floats() > 0) {
+      if (zero((void**)&L.memory, S * L.memory_floats() * 4) || (d.mixer == NFN_MIXER_WKV && zero((void**)&L.prev, 2 * S * wp * 4))) return -1;
     } else if (L.owner == l) {
       const long long tokens = (long long)groups[L.group].pages * kPage;
       if (zero(&L.k_pool, tokens * L.key_row() * es) || (L.value_row() > 0 && zero(&L.v_pool, tokens * L.value_row() * es))) return -1;
@@ -515,6 +564,21 @@ int layered_engine::finalize() {
     }
     const int wl = d.weights_of >= 0 ? d.weights_of : l;
     if (d.conv_taps > 0) L.conv = W(lname(wl, "conv"));
+    for (int q = 0; c.sandwich && q < (L.has_ff() ? 2 : 1); ++q) {
+      L.sub[q].norm_b = W(lname(wl, q ? "norm2_b" : "norm1_b"));
+      if (c.input_taps <= 0) continue;
+      L.sub[q].conv = W(lname(wl, q ? "in_conv2" : "in_conv1"));
+      if (c.input_taps > 1 && zero(&L.sub[q].history, 2 * S * (c.input_taps - 1) * wp * es)) return -1;
+    }
+    if (d.sink == 2) L.sinks = W(lname(wl, "sink"));
+    if (d.mixer == NFN_MIXER_LINEAR) {
+      L.out_norm = W(lname(wl, "out_norm"));
+      std::vector<float> pw((size_t)d.heads * (NFN_LINEAR_CHUNK + 1));
+      for (int i = 0; i < d.heads; ++i)
+        for (int n = 0; n <= NFN_LINEAR_CHUNK; ++n) pw[(size_t)i * (NFN_LINEAR_CHUNK + 1) + n] = (float)std::pow(L.decay[i], n);
+      if (zero((void**)&L.powers, (long long)pw.size() * 4)) return -1;
+      CU(cudaMemcpy(L.powers, pw.data(), pw.size() * 4, cudaMemcpyHostToDevice));
+    }
     if (d.alibi != 0.f) {
       std::vector<float> sl(d.heads);
       for (int i = 0; i < d.heads; ++i) sl[i] = (float)std::exp2(-(double)d.alibi * (i + 1) / d.heads);
@@ -553,6 +617,10 @@ int layered_engine::finalize() {
       L.norm2 = W(lname(wl, "norm2"));
       L.w_gate_up = W(lname(wl, "w_gate_up"));
       L.w_down = W(lname(wl, "w_down"));
+      if (d.ff_bias) {
+        L.bias_gate_up = W(lname(wl, "bias_gate_up"));
+        L.bias_down = W(lname(wl, "bias_down"));
+      }
     }
     if (d.shared_ff > 0) {
       L.w_shared_up = W(lname(wl, "w_shared_up"));
@@ -702,12 +770,18 @@ int layered_engine::fork(int src, int dst, int n) {
   parity[dst] = parity[src];
   for (const Layer& L : layers) {
     if (L.memory) {
-      const size_t n = (size_t)L.d.heads * L.dp * L.vp;
+      const size_t n = (size_t)L.memory_floats();
       CU(cudaMemcpyAsync(L.memory + dst * n, L.memory + src * n, n * 4, cudaMemcpyDeviceToDevice, stream));
     }
     if (L.prev) {
       float* half = L.prev + (size_t)parity[src] * c.max_batch * wp;
       CU(cudaMemcpyAsync(half + (size_t)dst * wp, half + (size_t)src * wp, (size_t)wp * 4, cudaMemcpyDeviceToDevice, stream));
+    }
+    for (const auto& u : L.sub) {
+      if (!u.history) continue;
+      const size_t row = (size_t)(c.input_taps - 1) * wp * es;
+      char* half = static_cast<char*>(u.history) + (size_t)parity[src] * c.max_batch * row;
+      CU(cudaMemcpyAsync(half + dst * row, half + src * row, row, cudaMemcpyDeviceToDevice, stream));
     }
     if (!L.state) continue;
     const size_t row = (size_t)(L.d.conv_taps - 1) * L.n_conv * es;
@@ -725,7 +799,7 @@ int layered_engine::fork(int src, int dst, int n) {
 int layered_engine::lin(const void* a, int lda, const void* wt, int rows, int n, int k, void* out, int ldo, int kind, const void* bias, int act) {
   if (c.dtype == 1) {
     K(nfn_gemm_f32(static_cast<const float*>(a), lda, wt, k, static_cast<float*>(out), ldo, rows, n, k, kind == kOutResidual, bias, stream));
-    if (act != NFN_ACT_NONE) K(nfn_ff_rows(1, out, ldo, 0, -1, n, act, out, ldo, rows, stream));
+    if (act != NFN_ACT_NONE) K(nfn_ff_rows(1, out, ldo, 0, -1, n, act, nullptr, out, ldo, rows, stream));
     return 0;
   }
   nfn_gemm_args g{};
@@ -775,7 +849,7 @@ void layered_engine::attention_args(const Layer& L, nfn_paged_attention_args* ou
   a.k_pool = L.k_pool; a.v_pool = L.v_pool; a.pages = groups[L.group].pages;
   a.table = groups[L.group].d_table; a.table_ld = max_pages;
   a.heads = d.heads; a.window = d.window; a.chunk = d.chunk; a.scale = d.scale; a.slopes = L.slopes;
-  a.keep_first = d.window > 0 ? d.keep_first : 0; a.softcap = d.softcap; a.sink = d.sink;
+  a.keep_first = d.window > 0 ? d.keep_first : 0; a.softcap = d.softcap; a.sink = d.sink == 1; a.sinks = L.sinks;
   a.row_slot = dev<int>(io.slot); a.row_pos = dev<int>(io.pos);
   a.max_keys = L.look() > 0 ? std::min(L.look() + d.keep_first, c.max_seq) : c.max_seq;
   a.workspace = att_ws; a.workspace_bytes = att_ws_bytes;
@@ -879,11 +953,13 @@ int layered_engine::latent_attention(const Layer& L, const Batch& b) {
     a.q = q_lat; a.ld_q = H * lp; a.kv_heads = 1; a.dim_p = lp; a.vdim_p = L.lr; a.v_pool = nullptr;
     a.out = o_lat; a.ld_o = H * L.lr; a.rows = single;
     K(nfn_paged_attention_rows(&a, stream));
+    if (d.out_gate) { g.gate = static_cast<const char*>(in) + (size_t)L.off_g * es; g.ld_gate = L.n_in; g.gate_group = L.vp; }
     g.n = L.vp; g.k = L.lr; g.in = o_lat; g.ld_in = (long long)H * L.lr; g.in_group = L.lr; g.w = L.w_uv; g.out = cat; g.ld_out = L.n_cat; g.out_group = L.vp;
     K(nfn_group_products(&g, stream));
   }
   const int l = (int)(&L - layers.data()), cols = H * (L.dp + L.vp);
   a.q = in; a.ld_q = L.n_in; a.kv_heads = H; a.dim_p = qp; a.vdim_p = L.vp; a.out = cat; a.ld_o = L.n_cat;
+  a.gate = d.out_gate ? static_cast<const char*>(in) + (size_t)L.off_g * es : nullptr; a.ld_gate = L.n_in;
   const int k = (int)(std::find(tile_kinds.begin(), tile_kinds.end(), L.tile_rows) - tile_kinds.begin());
   for (const Batch::Round& o : b.expand[l]) {
     K(nfn_latent_gather(f32, L.k_pool, lp, L.lr, groups[L.group].d_table, max_pages, dev<nfn_latent_span>(io.spans) + (size_t)l * c.max_batch + o.span0, o.n_spans, o.max_pages,
@@ -947,13 +1023,55 @@ int layered_engine::wkv(const Layer& L, const Batch& b) {
   return 0;
 }
 
-// A chained layer's mixer on the rows h -> y
+// Linear attention with a decay per head -> the first columns of `cat`
+int layered_engine::linear(const Layer& L, const Batch& b) {
+  const nfn_layer_desc& d = L.d;
+  const int f32 = c.dtype == 1, rows = b.rows, n_o = d.heads * L.vp;
+  if (linear_step(L, b)) {                               // the products in one, activations in the step
+    if (lin(hx, wp, L.w_in, rows, L.n_in, wp, in, L.n_in, kOutAct)) return -1;
+    nfn_linear_step_args t{};
+    t.f32 = f32; t.rows = rows; t.qkvg = in; t.ld_qkvg = L.n_in; t.powers = L.powers; t.heads = d.heads; t.vdim = d.vdim; t.dim_p = L.dp; t.vdim_p = L.vp;
+    t.state = L.memory; t.o = d_o; t.ld_o = n_o; t.counters = row_count; t.weight = L.out_norm; t.eps = c.norm_eps; t.out = cat; t.ld_out = L.n_cat;
+    t.tiles = dev<nfn_row_tile>(io.mix);
+    K(nfn_linear_step(&t, stream));
+    return 0;
+  }
+  char* gate = static_cast<char*>(in) + (size_t)L.off_g * es;
+  if (lin(hx, wp, L.w_in, rows, L.nq, wp, in, L.n_in, kOutAct, nullptr, NFN_ACT_SILU) ||
+      lin(hx, wp, static_cast<const char*>(L.w_in) + 2LL * L.off_g * wp, rows, n_o, wp, gate, L.n_in, kOutAct))
+    return -1;
+  nfn_linear_args a{};
+  a.f32 = f32; a.qkv = in; a.ld_qkv = L.n_in; a.powers = L.powers; a.heads = d.heads; a.dim_p = L.dp; a.vdim_p = L.vp; a.state = L.memory; a.o = d_o; a.ld_o = n_o;
+  const bool chunks = !f32 && nfn_linear_chunk_workspace_bytes(d.heads, L.dp, L.vp, 1) > 0;
+  a.seqs = dev<nfn_seq_rows>(io.seq); a.n_seqs = chunks ? b.n_short_seq : b.n_seq;
+  if (a.n_seqs > 0) K(nfn_linear_rows(&a, stream));
+  if (chunks && b.n_seq > b.n_short_seq) {
+    a.seqs += b.n_short_seq;
+    a.n_seqs = b.n_seq - b.n_short_seq;
+    K(nfn_linear_chunks(&a, b.longest, linear_ws, linear_ws_bytes, stream));
+  }
+  K(nfn_row_out(f32, d_o, n_o, gate, L.n_in, L.out_norm, c.norm_eps, cat, L.n_cat, rows, n_o, d.heads * d.vdim, stream));
+  return 0;
+}
+
+// The gated recurrence over the projected rows -> `cat`
+int layered_engine::gru(const Layer& L, const Batch& b) {
+  nfn_gru_args a{};
+  a.f32 = c.dtype == 1; a.width = L.vp; a.in = in; a.ld_in = L.n_in; a.state = L.memory; a.out = cat; a.ld_out = L.n_cat;
+  a.seqs = dev<nfn_seq_rows>(io.seq); a.n_seqs = b.n_seq; a.n_short = b.n_short_seq;
+  K(nfn_gru_rows(&a, stream));
+  return 0;
+}
+
+// A chained layer's mixer on the rows hx -> y
 int layered_engine::mixer(const Layer& L, const Batch& b) {
   const int kind = L.d.mixer;
-  if (kind != NFN_MIXER_WKV && lin(h, wp, L.w_in, b.rows, L.n_in, wp, in, L.n_in, kOutAct, L.bias_in)) return -1;
+  if (kind != NFN_MIXER_WKV && kind != NFN_MIXER_LINEAR && lin(hx, wp, L.w_in, b.rows, L.n_in, wp, in, L.n_in, kOutAct, L.bias_in)) return -1;
   int rc;
   if (kind == NFN_MIXER_WKV) rc = wkv(L, b);
   else if (kind == NFN_MIXER_LATENT) rc = latent_attention(L, b);
+  else if (kind == NFN_MIXER_LINEAR) rc = linear(L, b);
+  else if (kind == NFN_MIXER_GRU) rc = gru(L, b);
   else if (rotated(L)) rc = rotated_attention(L, b);
   else {
     if (!one_step(L, b) && mix_rows(L, b, nullptr)) return -1;
@@ -962,38 +1080,41 @@ int layered_engine::mixer(const Layer& L, const Batch& b) {
   return rc ? -1 : lin(cat, L.n_cat, L.w_out, b.rows, wp, L.n_cat, y, wp, kOutAct);
 }
 
-// A chained layer's gated feed-forward on the rows h -> y
+// A chained layer's gated feed-forward on the rows hx -> y
 int layered_engine::dense_ff(const Layer& L, int rows) {
-  if (lin(h, wp, L.w_gate_up, rows, 2 * L.ff, wp, in, 2 * L.ff, kOutAct)) return -1;
-  K(nfn_ff_rows(c.dtype == 1, in, 2 * L.ff, 0, L.ff, L.ff, L.d.ff_act, cat, L.ff, rows, stream));
-  return lin(cat, L.ff, L.w_down, rows, wp, L.ff, y, wp, kOutAct);
+  if (lin(hx, wp, L.w_gate_up, rows, 2 * L.ff, wp, in, 2 * L.ff, kOutAct, L.bias_gate_up)) return -1;
+  const nfn_gate_clamp clamp = L.clamp();
+  K(nfn_ff_rows(c.dtype == 1, in, 2 * L.ff, 0, L.ff, L.ff, L.d.ff_act, &clamp, cat, L.ff, rows, stream));
+  return lin(cat, L.ff, L.w_down, rows, wp, L.ff, y, wp, kOutAct, L.bias_down);
 }
 
-// Routed experts on the normalised rows h; says in `sp` where the next stream pass finds each row's outputs.
+// Routed experts on the rows hx; says in `sp` where the next stream pass finds each row's outputs.
 int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
   const nfn_layer_desc& d = L.d;
   const bool few = !grouped(L, rows), shared = d.shared_ff > 0;
   if (shared && c.dtype == 0 && rows <= kFewRows) {        // router and the shared expert's first product in one launch
     nfn_group_products_args g{};
-    g.rows = rows; g.groups = 1; g.n = L.shp; g.k = wp; g.in = h; g.ld_in = wp; g.w = L.w_shared_up; g.out = shared_mid; g.ld_out = L.shp; g.act = d.ff_act;
+    g.rows = rows; g.groups = 1; g.n = L.shp; g.k = wp; g.in = hx; g.ld_in = wp; g.w = L.w_shared_up; g.out = shared_mid; g.ld_out = L.shp; g.act = d.ff_act;
     g.tail_n = L.ep; g.tail_w = L.router; g.tail_out = ex.logits; g.ld_tail = L.ep;
     K(nfn_group_products(&g, stream));
-  } else if (lin(h, wp, L.router, rows, L.ep, wp, ex.logits, L.ep, kOutF32) || (shared && lin(h, wp, L.w_shared_up, rows, L.shp, wp, shared_mid, L.shp, kOutAct, nullptr, d.ff_act))) {
+  } else if (lin(hx, wp, L.router, rows, L.ep, wp, ex.logits, L.ep, kOutF32) || (shared && lin(hx, wp, L.w_shared_up, rows, L.shp, wp, shared_mid, L.shp, kOutAct, nullptr, d.ff_act))) {
     return -1;
   }
   if (shared && !few && lin(shared_mid, L.shp, L.w_shared_down, rows, wp, L.shp, y_shared, wp, kOutAct)) return -1;
   sp->y = ex.y;
   sp->y_rows = d.top;
-  sp->y_item = d.expert_plain ? ex.weight : nullptr;
+  const bool weigh_out = d.expert_plain || d.expert_weigh_out;
+  const nfn_gate_clamp clamp = L.clamp();
+  sp->y_item = weigh_out ? ex.weight : nullptr;
   sp->y_plus = shared ? y_shared : nullptr;
   nfn_route_rule rule{};
-  rule.correction = L.correction; rule.groups = d.route_groups; rule.keep_groups = d.route_keep; rule.normalise = d.route_normalise; rule.scale = d.route_scale;
+  rule.correction = L.correction; rule.groups = d.route_groups; rule.keep_groups = d.route_keep; rule.normalise = d.route_normalise; rule.scale = d.route_scale; rule.softmax = d.route_softmax;
   if (few) {
     nfn_moe_rows_args a{};
     a.f32 = c.dtype == 1; a.rows = rows; a.width = wp; a.ff = L.ef; a.experts = d.experts; a.top = d.top; a.act = d.ff_act;
-    a.logits = ex.logits; a.ld_logits = L.ep; a.h = h; a.ld_h = wp; a.w_gate_up = L.w_gate_up; a.w_down = L.w_down;
+    a.logits = ex.logits; a.ld_logits = L.ep; a.h = hx; a.ld_h = wp; a.w_gate_up = L.w_gate_up; a.w_down = L.w_down;
     a.idx = ex.idx; a.weight = ex.weight; a.order = ex.order; a.offsets = ex.offsets; a.active = ex.active;
-    a.mid = ex.mid; a.y = ex.y; a.ld_y = wp; a.plain = d.expert_plain; a.rule = rule;
+    a.mid = ex.mid; a.y = ex.y; a.ld_y = wp; a.plain = d.expert_plain; a.rule = rule; a.weigh_output = weigh_out; a.clamp = clamp;
     if (shared) { a.shared_ff = L.shp; a.shared_mid = shared_mid; a.w_shared_down = L.w_shared_down; a.y_shared = y_shared; }
     K(nfn_moe_rows(&a, stream));
     sp->y_index = nullptr;
@@ -1001,10 +1122,10 @@ int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
   }
   const int cap = (int)(((long long)rows * d.top + d.experts * 127LL + 127) / 128 * 128);
   CU(cudaMemsetAsync(ex.counts, 0, (size_t)d.experts * 4, stream));
-  if (d.expert_plain) K(nfn_moe_choose(ex.logits, L.ep, rows, d.experts, d.top, &rule, ex.idx, ex.weight, ex.counts, stream));
+  if (weigh_out) K(nfn_moe_choose(ex.logits, L.ep, rows, d.experts, d.top, &rule, ex.idx, ex.weight, ex.counts, stream));
   else K(nfn_moe_route(ex.logits, L.ep, rows, d.experts, d.top, 1, 0, 1.f, ex.idx, ex.weight, ex.counts, stream));
   K(nfn_moe_plan(ex.counts, d.experts, cap / 128, ex.offsets, ex.cursor, ex.tile_expert, ex.plan, stream));
-  K(nfn_moe_permute_weighted(h, wp, rows, d.top, wp, ex.idx, ex.weight, ex.offsets, ex.cursor, cap, ex.xs, ex.row_of, ex.row_w, stream));
+  K(nfn_moe_permute_weighted(hx, wp, rows, d.top, wp, ex.idx, ex.weight, ex.offsets, ex.cursor, cap, ex.xs, ex.row_of, ex.row_w, stream));
   nfn_gemm_tp_args g{};
   g.mode = NFN_TP_GROUPED;
   g.tile_group = ex.tile_expert; g.num_m_tiles_dev = ex.plan; g.groups = d.experts; g.m = cap;
@@ -1017,7 +1138,7 @@ int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
   } else {
     g.c = ex.gate_up; g.n = g.ldc = 2 * L.ef;
     K(nfn_gemm_tp(&g, stream));
-    K(nfn_moe_act_rows(ex.gate_up, ex.row_w, ex.plan, cap, L.ef, d.ff_act, ex.mid, stream));
+    K(nfn_moe_act_rows(ex.gate_up, weigh_out ? nullptr : ex.row_w, ex.plan, cap, L.ef, d.ff_act, &clamp, ex.mid, stream));
   }
   g.a = ex.mid; g.b = L.w_down; g.c = ex.y;
   g.n = wp; g.k = g.lda = g.ldb = L.ef; g.ldc = wp;
@@ -1028,7 +1149,8 @@ int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
 
 // Layers whose mixer and feed-forward read one norm
 int layered_engine::pass(const Batch& b) {
-  if (c.post_norm) return post_pass(b);
+  hx = h;
+  if (c.post_norm || c.sandwich) return post_pass(b);
   if (c.chained) return chained_pass(b);
   const int f32 = c.dtype == 1, rows = b.rows;
   nfn_row_norm_args rn{};
@@ -1088,26 +1210,47 @@ int layered_engine::chained_pass(const Batch& b) {
   return 0;
 }
 
-// Layers whose sublayers read the residual itself; the stream pass after each one norms its output, adds it and leaves the new rows in the activation
-// type. The last update is left to the head.
+// The stream pass in front of a sublayer (0: mixer, 1: feed-forward): its norm if it has one, and the convolution on its input - in the same launch when
+// every row is a sequence of its own.
+int layered_engine::enter(nfn_stream_args* s, const Layer& L, int which, const Batch& b) {
+  const auto& u = L.sub[which];
+  const long long half = (long long)c.max_batch * (c.input_taps - 1) * wp;
+  s->weight = !c.sandwich ? nullptr : which ? L.norm2 : L.norm1;
+  const bool fused = u.conv && b.single;
+  s->conv = fused ? u.conv : nullptr;
+  s->conv_taps = c.input_taps; s->history = u.history; s->history_half = half; s->tiles = dev<nfn_row_tile>(io.mix);
+  K(nfn_stream_pass(s, stream));
+  s->conv = nullptr;
+  hx = h;
+  if (!u.conv || fused) return 0;
+  nfn_input_conv_args a{};
+  a.f32 = c.dtype == 1; a.ld = wp; a.taps = c.input_taps; a.h = h; a.conv = u.conv; a.history = u.history; a.history_half = half; a.out = hc;
+  a.tiles = dev<nfn_row_tile>(io.mix); a.n_tiles = b.n_mix;
+  K(nfn_input_conv(&a, stream));
+  hx = hc;
+  return 0;
+}
+
+// Layers whose sublayers' outputs are normed before they are added. Sublayers read the residual itself, in the activation type, or (sandwich) its norm. The
+// last update is left to the head.
 int layered_engine::post_pass(const Batch& b) {
   nfn_stream_args s{};
   s.f32 = c.dtype == 1; s.rows = b.rows; s.width = c.width; s.ld = wp; s.streams = 1;
   s.eps = c.norm_eps; s.y_scale = c.residual_mult;
   s.tokens = dev<int>(io.tok); s.embed = W("embed"); s.embed_scale = c.embed_scale; s.vocab = c.vocab;
-  s.x = x; s.x_out = x; s.h = h;
-  K(nfn_stream_pass(&s, stream));
+  s.x = x; s.x_out = x; s.h = h; s.scalar_norms = c.scalar_norms;
+  if (enter(&s, layers[0], 0, b)) return -1;
   s.tokens = nullptr; s.embed = nullptr;
   for (int l = 0; l < c.n_layer; ++l) {
     const Layer& L = layers[l];
     if (mixer(L, b)) return -1;
-    s.y = y; s.y_rows = 1; s.y_index = nullptr; s.y_item = nullptr; s.y_plus = nullptr; s.y_weight = L.norm1;
-    if (L.d.experts > 0 || L.d.ff > 0) {
-      K(nfn_stream_pass(&s, stream));
+    s.y = y; s.y_rows = 1; s.y_index = nullptr; s.y_item = nullptr; s.y_plus = nullptr; s.y_weight = c.sandwich ? L.sub[0].norm_b : L.norm1;
+    if (L.has_ff()) {
+      if (enter(&s, L, 1, b)) return -1;
       if (L.d.experts > 0 ? experts(L, b.rows, &s) : dense_ff(L, b.rows)) return -1;
-      s.y_weight = L.norm2;
+      s.y_weight = c.sandwich ? L.sub[1].norm_b : L.norm2;
     }
-    if (l + 1 < c.n_layer) K(nfn_stream_pass(&s, stream));
+    if (l + 1 < c.n_layer && enter(&s, layers[l + 1], 0, b)) return -1;
   }
   pend = s;
   return 0;
@@ -1160,7 +1303,7 @@ int layered_engine::run(const std::vector<nfn_step_entry>& part, const int32_t* 
   int *tok = host<int>(io.tok), *slot = host<int>(io.slot), *pos = host<int>(io.pos);
   nfn_row_tile* mix = host<nfn_row_tile>(io.mix);
   int n_mix = 0, hist_max = 0;
-  for (const Layer& L : layers) hist_max = std::max(hist_max, L.prev ? 1 : L.d.conv_taps - 1);
+  for (const Layer& L : layers) hist_max = std::max(std::max(hist_max, c.input_taps - 1), L.prev ? 1 : L.d.conv_taps - 1);
   row_of.clear();
   for (size_t i = 0; i < part.size(); ++i) {
     const int s = part[i].slot, p0 = len[s], n = part[i].count;

@@ -65,7 +65,9 @@ typedef struct {
 // With `chained` set in the configuration mixer and feed-forward are two sublayers, each with a norm of its own, and the residual may be
 // several streams: u = sum_s in[s] x_s, y = sublayer(RMS(u) * norm), x_t <- sum_s mix[s][t] x_s + out[t] y.
 // With `post_norm` the sublayers of such a layer read the residual itself and their outputs are normed: x <- x + residual_mult * RMS(sublayer(x)) * norm.
-enum { NFN_MIXER_ATTENTION = 0, NFN_MIXER_DELTA = 1, NFN_MIXER_LATENT = 2, NFN_MIXER_WKV = 3 };
+// With `sandwich` they have a norm before and one after them: x <- x + residual_mult * RMS(sublayer(RMS(x) * norm)) * norm_b; `input_taps` then adds to what a
+// sublayer reads a short causal convolution of it over the sequence, h + conv(h).
+enum { NFN_MIXER_ATTENTION = 0, NFN_MIXER_DELTA = 1, NFN_MIXER_LATENT = 2, NFN_MIXER_WKV = 3, NFN_MIXER_LINEAR = 4, NFN_MIXER_GRU = 5 };
 typedef struct {
   int heads, kv_heads;   // query head h reads key / value head h / (heads / kv_heads)
   int dim, vdim;         // per-head query / key size and value size
@@ -78,12 +80,12 @@ typedef struct {
   int q_temp_every;
   int out_gate;          // heads *= sigmoid(W_g h)
   int ff;                // width of the gated feed-forward down(act(gate h) * (up h)); 0: none
-  int ff_act;            // NFN_ACT_RELU, NFN_ACT_SILU, NFN_ACT_GELU_TANH
+  int ff_act;            // NFN_ACT_RELU, NFN_ACT_SILU, NFN_ACT_GELU_TANH, NFN_ACT_RELU2, NFN_ACT_CLAMPED (gated ones, with ff_limit and ff_slope)
   int mixer;             // NFN_MIXER_*. Delta: gated delta rule with a decay per key channel (nfn_delta_rows); conv_taps >= 1 with SiLU after it
-  int qkv_bias;          // biases on the projected q, k, v
+  int qkv_bias;          // biases on the projected q, k, v (gru: on the share and the candidate)
   int keep_first;        // with a window: the sequence's first keys stay visible
   float softcap;         // score <- softcap * tanh(score / softcap); 0: off
-  int sink;              // one more score of 0, without a value, in the softmax
+  int sink;              // 1: one more score of 0, without a value, in the softmax; 2: one of a learned size per head
   int rank_decay, rank_gate;   // delta: inner sizes of the decay and output-gate projections
   int experts, top, expert_ff; // chained: routed experts instead of a dense feed-forward (sigmoid scores, weight on the expert's input)
   int weights_of;        // >= 0: this layer runs with the tensors of that earlier one (a loop over layers); -1: its own
@@ -100,8 +102,15 @@ typedef struct {
   int route_groups, route_keep;   // consecutive experts form groups, the choice is limited to the best of them (nfn_route_rule; 0: no groups)
   int route_normalise;   // weights divided by their sum
   float route_scale;     // times this; 0 counts as 1
+  int route_softmax;     // weights are the softmax over the chosen experts' logits
+  int expert_weigh_out;  // gated experts weighted at their output instead of their input
+  float ff_limit, ff_slope;   // NFN_ACT_CLAMPED: g = min(gate, limit), u = clamp(up, +-limit), g * sigmoid(slope * g) * (u + 1); feed-forward and experts
+  int ff_bias;           // biases on the dense feed-forward's three products
+  const double* decay;   // linear: factor of each head's state per token [heads], copied
 } nfn_layer_desc;
 // Latent (NFN_MIXER_LATENT): q per head [dim | rot_dim], c = RMS(W_dkv h) cached with the rotated key part; score = (q . W_uk c + q_rot . k_rot) * scale, value W_uv c.
+// Latent layers may have an output gate and a sink. Linear (NFN_MIXER_LINEAR): SiLU on q, k, v, the rule of nfn_linear_rows, RMS norm over all heads together,
+// sigmoid gate. Gru (NFN_MIXER_GRU): the rule of nfn_gru_rows over vdim channels (heads = kv_heads = dim = 1).
 // Wkv (NFN_MIXER_WKV): heads x dim, vdim = dim; token shift, bonus recurrence (nfn_wkv_rows), rank_decay the inner size of the decay projection.
 
 typedef struct {
@@ -121,7 +130,10 @@ typedef struct {
   float logit_scale;     // logits *= logit_scale
   float logit_softcap;   // logits <- cap * tanh(logits / cap); 0: off
   int post_norm;         // chained, one residual: norms on the sublayers' outputs
-  float residual_mult;   // post_norm: factor of the normed output
+  float residual_mult;   // post_norm, sandwich: factor of the normed output
+  int sandwich;          // chained, one residual: norms before and after every sublayer
+  int scalar_norms;      // sandwich: every norm of the residual has one factor for all channels
+  int input_taps;        // sandwich: taps of the convolution on the sublayers' inputs; 0: none
 } nfn_layered_config;
 
 enum { NFN_KV_PAGE = 64 };   // tokens per cache page

@@ -263,7 +263,10 @@ group_products_f32_kernel(const nfn_group_products_args p) {
   for (int i = 0; i < GP_ROWS; ++i) {
     if (i >= live) break;
     const float s = warp_sum(a[i]);
-    if (lane == 0) out[(size_t)i * (tail ? p.ld_tail : p.ld_out)] = tail ? s : ff_act(s, p.act);
+    if (lane != 0) continue;
+    float f = 1.f;
+    if (!tail && p.gate) f = sigmoid_exact(static_cast<const float*>(p.gate)[(size_t)(r0 + i) * p.ld_gate + (size_t)g * p.gate_group + n]);
+    out[(size_t)i * (tail ? p.ld_tail : p.ld_out)] = tail ? s : ff_act(s, p.act) * f;
   }
 }
 
@@ -358,8 +361,13 @@ group_products_mma_kernel(const nfn_group_products_args p) {
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < GM_WARPS; ++w) v += part[w][row][col];
-    if (tail) p.tail_out[(size_t)(r0 + col) * p.ld_tail + n0 + row] = v;
-    else static_cast<__nv_bfloat16*>(p.out)[(size_t)(r0 + col) * p.ld_out + (size_t)g * p.out_group + n0 + row] = __float2bfloat16(ff_act(v, p.act));
+    if (tail) {
+      p.tail_out[(size_t)(r0 + col) * p.ld_tail + n0 + row] = v;
+      continue;
+    }
+    v = ff_act(v, p.act);
+    if (p.gate) v *= sigmoid_for<__nv_bfloat16>(__bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[(size_t)(r0 + col) * p.ld_gate + (size_t)g * p.gate_group + n0 + row]));
+    static_cast<__nv_bfloat16*>(p.out)[(size_t)(r0 + col) * p.ld_out + (size_t)g * p.out_group + n0 + row] = __float2bfloat16(v);
   }
 }
 

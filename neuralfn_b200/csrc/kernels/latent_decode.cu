@@ -299,7 +299,7 @@ latent_decode_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
       if (lane == 0) mbar_arrive(smem_u32(bar_p));
     }
     // ---- O^T: a thread holds one channel of all heads ----
-    if (warp == 0) s_sum[head] = l_run;
+    if (warp == 0) s_sum[head] = l_run + (has_sink(a) && head < n_heads ? exp2f(sink_score(a, h0 + head) * 1.4426950408889634f - m_run) : 0.f);
     asm volatile("bar.sync 1, 128;" ::: "memory");
     if (*cta_abort) ok = false;
     if (ok) ok = mbar_wait_bounded(smem_u32(bar_o), (n - 1) & 1, cta_abort, p.status, 0x700 + 9);
@@ -348,7 +348,7 @@ latent_merge_kernel(const LatentDecodeParams p) {
   const size_t cell = (size_t)blockIdx.y * a.heads + h;
   const float2* stats = p.stats + cell * p.splits;
   const float* part = p.partial + cell * p.splits * a.vdim_p + c;
-  float m = -INFINITY, l = 0.f;
+  float m = has_sink(a) ? sink_score(a, h) * 1.4426950408889634f : -INFINITY, l = has_sink(a) ? 1.f : 0.f;
   float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
   for (int s0 = 0; s0 < p.splits; s0 += AT_ONCE) {
     float2 t[AT_ONCE];
@@ -401,7 +401,7 @@ static uint32_t latent_tail(int panels, int m_tiles, int nh) { return std::max<u
 // 1: sizes outside the kernel's limits
 int latent_decode(const nfn_paged_attention_args& a, cudaStream_t st) {
   constexpr uint32_t LIMIT = 227 * 1024 - 2048;            // static shared memory and the alignment of the dynamic part aside
-  if (a.vdim_p > 512 || ((a.dim_p | a.vdim_p) & 15) || a.ld_q != a.heads * a.dim_p || a.rows > 65535 || a.slopes || a.softcap > 0.f || a.sink || a.keep_first > 0 || a.gate) return 1;
+  if (a.vdim_p > 512 || ((a.dim_p | a.vdim_p) & 15) || a.ld_q != a.heads * a.dim_p || a.rows > 65535 || a.slopes || a.softcap > 0.f || a.keep_first > 0 || a.gate) return 1;
   LatentDecodeParams p{};
   p.a = a;
   p.panels = ceil_div(a.dim_p, 64);

@@ -199,6 +199,7 @@ extern "C" int nfn_moe_choose(const float* logits, int ld, int T, int E, int k, 
   if (E <= 0 || E > MOE_MAX_E || k <= 0 || k > E || ld < E) return fail(-1, "moe_choose: need 1 <= k <= E <= 256, ld >= E");
   if (rule->groups < 0 || (rule->groups > 0 && (E % rule->groups || rule->keep_groups < 1 || rule->keep_groups * (E / rule->groups) < k)))
     return fail(-1, "moe_choose: the kept groups must hold the chosen experts");
+  if (rule->softmax && (rule->correction || rule->groups > 0)) return fail(-1, "moe_choose: the softmax over chosen logits has no correction or groups");
   auto kern = E <= 32 ? moe_choose_kernel<1> : E <= 64 ? moe_choose_kernel<2> : E <= 128 ? moe_choose_kernel<4> : moe_choose_kernel<MOE_MAX_E / 32>;
   kern<<<(T + 7) / 8, 256, 0, static_cast<cudaStream_t>(stream)>>>(logits, ld, T, E, k, *rule, idx, weight, counts);
   return launch_check("moe_choose", 1);

@@ -84,22 +84,24 @@ __device__ __forceinline__ void choose_experts(const float* z, int experts, int 
     }
   }
   uint32_t taken = 0;
-  float sum = 0.f;
+  float sum = 0.f, first = 0.f;
   const float scale = rule.scale == 0.f ? 1.f : rule.scale;
   for (int j = 0; j < top; ++j) {
     float best;
     int e;
     best_of<PER>(c, taken, experts, lane, best, e);
     if ((e & 31) == lane) taken |= 1u << (e >> 5);
-    const float w = __shfl_sync(0xffffffffu, pick<PER>(s, e >> 5), e & 31);
+    float w = __shfl_sync(0xffffffffu, pick<PER>(s, e >> 5), e & 31);
+    if (j == 0) first = best;
+    if (rule.softmax) w = expf(best - first);               // the choice went by the logits, largest first
     sum += w;
     if (lane == (j & 31)) {
       idx[j] = e;
       weight[j] = w * scale;
     }
   }
-  if (rule.normalise) {
-    const float f = 1.f / (sum + 1e-20f);
+  if (rule.normalise || rule.softmax) {
+    const float f = 1.f / (rule.softmax ? sum : sum + 1e-20f);
     for (int j = lane; j < top; j += 32) weight[j] *= f;   // this lane's own entries
   }
 }

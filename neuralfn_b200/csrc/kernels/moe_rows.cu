@@ -131,8 +131,8 @@ moe_products_kernel(const nfn_moe_rows_args p) {
         } else if (!TWO) {
           static_cast<T*>(p.mid)[(size_t)item * p.ff + n] = from_float<T>(ff_act(a[i], p.act));
         } else {
-          const float w = p.weight[item];
-          static_cast<T*>(p.mid)[(size_t)item * p.ff + n] = from_float<T>(ff_act(w * a[i], p.act) * (w * b[i]));
+          const float w = p.weigh_output ? 1.f : p.weight[item];
+          static_cast<T*>(p.mid)[(size_t)item * p.ff + n] = from_float<T>(ff_gated<T>(w * a[i], w * b[i], p.act, p.clamp));
         }
       }
     }
@@ -241,8 +241,8 @@ moe_products_mma_kernel(const nfn_moe_rows_args p) {
           gv += part[w][0][row][col];
           uv += part[w][1][row][col];
         }
-        const float f = p.weight[item];
-        static_cast<__nv_bfloat16*>(p.mid)[(size_t)item * p.ff + n0 + row] = __float2bfloat16(ff_act(f * gv, p.act) * (f * uv));
+        const float f = p.weigh_output ? 1.f : p.weight[item];
+        static_cast<__nv_bfloat16*>(p.mid)[(size_t)item * p.ff + n0 + row] = __float2bfloat16(ff_gated<__nv_bfloat16>(f * gv, f * uv, p.act, p.clamp));
       }
     }
     __syncthreads();
@@ -252,15 +252,15 @@ moe_products_mma_kernel(const nfn_moe_rows_args p) {
 // Sorted prompt rows: mid = act(w g) * (w u). Rows past the plan's count stay untouched.
 __global__ void __launch_bounds__(256)
 moe_act_rows_kernel(const __nv_bfloat16* __restrict__ gate_up, const float* __restrict__ row_w, const int* __restrict__ plan, int ff, int act,
-                    __nv_bfloat16* __restrict__ mid) {
+                    nfn_gate_clamp clamp, __nv_bfloat16* __restrict__ mid) {
   const int r = blockIdx.x, c = (blockIdx.y * 256 + threadIdx.x) * 8;
   if (r >= plan[1] || c >= ff) return;
   float g[8], u[8];
   load8(gate_up + (size_t)r * 2 * ff + c, g);
   load8(gate_up + (size_t)r * 2 * ff + ff + c, u);
-  const float w = row_w[r];
+  const float w = row_w ? row_w[r] : 1.f;
 #pragma unroll
-  for (int i = 0; i < 8; ++i) g[i] = ff_act(w * g[i], act) * (w * u[i]);
+  for (int i = 0; i < 8; ++i) g[i] = ff_gated<__nv_bfloat16>(w * g[i], w * u[i], act, clamp);
   store8(mid + (size_t)r * ff + c, g);
 }
 
@@ -303,17 +303,21 @@ extern "C" int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream) 
   if (a.rule.groups < 0 || (a.rule.groups > 0 && (a.experts % a.rule.groups || a.rule.keep_groups < 1 || (long long)a.rule.keep_groups * (a.experts / a.rule.groups) < a.top)))
     return fail(-1, "moe_rows: the kept groups must hold the chosen experts");
   if (a.shared_ff < 0 || (a.shared_ff > 0 && ((a.shared_ff & 15) || !a.shared_mid || !a.w_shared_down || !a.y_shared))) return fail(-1, "moe_rows: the shared expert lacks an operand");
+  if (a.rule.softmax && (a.rule.correction || a.rule.groups > 0)) return fail(-1, "moe_rows: the softmax over chosen logits has no correction or groups");
+  if (a.plain && a.act == NFN_ACT_CLAMPED) return fail(-1, "moe_rows: the clamped gate needs gated experts");
   if ((a.width | a.ff | a.ld_h) & 15) return fail(-1, "moe_rows: widths must be multiples of 16");
   if ((long long)a.rows * a.top > 0x7fffffffLL / 2) return fail(-1, "moe_rows: too many rows");
   return launch_moe_rows(a, static_cast<cudaStream_t>(stream));
 }
 
-extern "C" int nfn_moe_act_rows(const void* gate_up, const float* row_w, const int* plan, int capacity_rows, int ff, int act, void* mid, nfn_stream_t stream) {
+extern "C" int nfn_moe_act_rows(const void* gate_up, const float* row_w, const int* plan, int capacity_rows, int ff, int act, const nfn_gate_clamp* clamp, void* mid,
+                                nfn_stream_t stream) {
   if (capacity_rows <= 0) return 0;
   if (ff & 7) return fail(-1, "moe_act_rows: the width must be a multiple of 8");
+  if (act == NFN_ACT_CLAMPED && !clamp) return fail(-1, "moe_act_rows: the clamped gate needs its limits");
   cudaStream_t st = static_cast<cudaStream_t>(stream);
   const __nv_bfloat16* gu = static_cast<const __nv_bfloat16*>(gate_up);
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(mid);
-  moe_act_rows_kernel<<<dim3(capacity_rows, ceil_div(ff, 256 * 8)), 256, 0, st>>>(gu, row_w, plan, ff, act, out);
+  moe_act_rows_kernel<<<dim3(capacity_rows, ceil_div(ff, 256 * 8)), 256, 0, st>>>(gu, row_w, plan, ff, act, clamp ? *clamp : nfn_gate_clamp{}, out);
   return launch_check("moe_act_rows");
 }

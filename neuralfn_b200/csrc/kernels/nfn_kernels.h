@@ -47,7 +47,8 @@ enum {
   NFN_EPI_ACT_SHIFT = 8,      // activation id in bits 8..11
 };
 enum { NFN_ACT_NONE = 0, NFN_ACT_GELU_TANH = 1, NFN_ACT_GELU_ERF = 2, NFN_ACT_SILU = 3,
-       NFN_ACT_RELU2 = 4, NFN_ACT_TANH_CAP = 5 /* cap*tanh(x/cap), cap = act_param */, NFN_ACT_RELU = 6 };
+       NFN_ACT_RELU2 = 4, NFN_ACT_TANH_CAP = 5 /* cap*tanh(x/cap), cap = act_param */, NFN_ACT_RELU = 6,
+       NFN_ACT_CLAMPED = 7 /* feed-forward gates only, see nfn_gate_clamp */ };
 
 typedef struct {
   const void* a; const void* b; void* c;
@@ -341,11 +342,15 @@ typedef struct {
   int rows;                               // rows of the call
 } nfn_mix_args;
 int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream);
-// out[r] = act(gate) * up of rows [.. off_gate: gate .. off_up: up ..]; off_up < 0: out[r] = act(gate).
-int nfn_ff_rows(int f32, const void* in, int ld_in, int off_gate, int off_up, int ff, int act, void* out, int ld_out, int rows, nfn_stream_t stream);
+// NFN_ACT_CLAMPED, the gate of a feed-forward with bounded inputs: g = min(gate, limit), u = max(-limit, min(up, limit)), g * sigmoid(slope * g) * (u + shift).
+typedef struct { float limit, slope, shift; } nfn_gate_clamp;
+// out[r] = act(gate) * up of rows [.. off_gate: gate .. off_up: up ..]; off_up < 0: out[r] = act(gate). clamp: with NFN_ACT_CLAMPED (which needs both).
+int nfn_ff_rows(int f32, const void* in, int ld_in, int off_gate, int off_up, int ff, int act, const nfn_gate_clamp* clamp, void* out, int ld_out, int rows,
+                nfn_stream_t stream);
 // Attention of a step's rows over the pages. score = q . k * scale, capped to softcap * tanh(score / softcap) (0: off), minus
 // slopes[h] * (i - j); keys 0 <= i - j < window (0: all) and the first keep_first ones of the sequence, with chunk > 0 only those of the query's own
-// chunk of that many positions; softmax, with sink != 0 over one more score of 0 that has no value; out = P V * sigmoid(gate) (gate optional).
+// chunk of that many positions; softmax, with sink != 0 over one more score of 0 that has no value, with sinks over one of
+// sinks[h] (not scaled, not capped); out = P V * sigmoid(gate) (gate optional).
 // q: [rows, heads * dim_p]; out: row pitch ld_o, head pitch vdim_p. v_pool = NULL: a key's value is its first vdim_p channels (latent caches).
 typedef struct {
   int f32;
@@ -365,6 +370,7 @@ typedef struct {
   int total_rows;                         // rows of the q buffer
   int keep_first; float softcap; int sink;
   int chunk;
+  const void* sinks;                      // bf16 [heads]
 } nfn_paged_attention_args;
 // One query row at a time (single tokens, very short portions): bf16 goes to the tensor cores in 32-key steps, fp32 and sizes
 // outside its limits to the plain kernel.
@@ -409,7 +415,7 @@ typedef struct {
 int nfn_latent_rows(const nfn_latent_rows_args* args, nfn_stream_t stream);
 // out[r][g][n] = act(sum_k in[r][g][k] w[g][n][k]): one small product per group and row (the per-head projections around a latent cache, several inputs
 // with a matrix each). in, out: activation type, group pitches in elements; w bf16. Sizes are multiples of 16. tail_n > 0: one more product of the same
-// depth, from the input tail_in elements into each row, with an fp32 result and no activation.
+// depth, from the input tail_in elements into each row, with an fp32 result and no activation. gate: out *= sigmoid(gate[r][g][n]).
 typedef struct {
   int f32, rows, groups, n, k;
   const void* in; long long ld_in, in_group;
@@ -419,6 +425,7 @@ typedef struct {
   long long tail_in;
   const void* tail_w;
   float* tail_out; int ld_tail;
+  const void* gate; long long ld_gate, gate_group;
 } nfn_group_products_args;
 int nfn_group_products(const nfn_group_products_args* args, nfn_stream_t stream);
 
@@ -450,7 +457,9 @@ int nfn_logit_cap(float* logits, int ld, int rows, int cols, float scale, float 
 // The base is embed[token] * embed_scale in every stream (tokens != NULL) or row src_rows[r] (NULL: r) of x; y is the row of the
 // same number, or with y_rows > 1 the sum of rows y_index[r * y_rows + j] (y_index NULL: r * y_rows + j), each times y_item[r * y_rows + j]
 // (NULL: 1), plus row r of y_plus (NULL: none). With y_weight the update is normed first: y <- y_scale * y / rms(y) * y_weight.
-// weight = NULL: h = u.
+// weight = NULL: h = u. scalar_norms: weight and y_weight are one number each, for all channels.
+// With conv (bf16 [conv_taps][ld]) every row is an entry of its own (tiles: one per row) and h gets a causal convolution of itself over the sequence added,
+// h + sum_j conv[j] h_(t - conv_taps + 1 + j), zero before its start; one stream. history: see nfn_input_conv.
 enum { NFN_MAX_STREAMS = 16 };
 typedef struct {
   int f32, rows, width, ld, streams;
@@ -462,8 +471,21 @@ typedef struct {
   float eps, weight_offset;
   const float* y_item; const void* y_plus;
   const void* y_weight; float y_scale;
+  int scalar_norms;
+  const void* conv; int conv_taps; void* history; long long history_half;
+  const nfn_row_tile* tiles;
 } nfn_stream_args;
 int nfn_stream_pass(const nfn_stream_args* args, nfn_stream_t stream);
+// The same convolution over the rows of any entries: out[r] = h[r] + sum_j conv[j] h_(t - taps + 1 + j). h and out are different buffers of pitch ld in the
+// activation type; history [2][slots][taps - 1][ld], its newest rows last: the half named by the tile's parity is read, the other written.
+typedef struct {
+  int f32, ld, taps;
+  const void* h; const void* conv;        // bf16 [taps][ld]
+  void* history; long long history_half;
+  void* out;
+  const nfn_row_tile* tiles; int n_tiles;
+} nfn_input_conv_args;
+int nfn_input_conv(const nfn_input_conv_args* args, nfn_stream_t stream);
 
 // ---- gated delta rule with a decay per key channel (delta_rows.cu, delta_chunk.cu) -------------------------------------------
 // Per head (query / key head h / (heads / kv_heads)), with the fp32 state S [dim][vdim] of the sequence:
@@ -561,13 +583,66 @@ typedef struct {
 int nfn_wkv_step_fits(int rows, int dim_p);
 int nfn_wkv_step(const nfn_wkv_step_args* args, nfn_stream_t stream);
 
+// ---- linear attention with a constant decay per head (linear_rows.cu, linear_chunk.cu) ------------------------------------------------------
+// Per head, with the fp32 state S [dim][vdim] of the sequence: S <- decay_h S + k v^T;  o = S^T q.
+// qkv: rows [q: heads * dim_p | k | v: heads * vdim_p], activated; state [slots][heads][dim_p][vdim_p]; a sequence at position 0 starts from zero.
+// powers: fp32 [heads][NFN_LINEAR_CHUNK + 1], decay_h^i. o: fp32 rows of heads * vdim_p. Padded channels are zero in q, k, v.
+enum { NFN_LINEAR_CHUNK = 64 };
+typedef struct {
+  int f32;
+  const void* qkv; int ld_qkv;
+  const float* powers;
+  int heads, dim_p, vdim_p;
+  float* state;
+  float* o; int ld_o;
+  const nfn_seq_rows* seqs; int n_seqs;
+} nfn_linear_args;
+int nfn_linear_rows(const nfn_linear_args* args, nfn_stream_t stream);      // token after token, any length
+// NFN_LINEAR_CHUNK tokens at a time on the tensor cores (bf16), for sequences of up to max_rows rows. The workspace lets the segments of a long sequence
+// run side by side; 0 bytes: these sizes go token after token.
+long long nfn_linear_chunk_workspace_bytes(int heads, int dim_p, int vdim_p, int max_seqs);
+int nfn_linear_chunks(const nfn_linear_args* args, int max_rows, void* workspace, long long workspace_bytes, nfn_stream_t stream);
+// One token of every sequence from the input product on: qkvg rows [q | k | v | g] before their activations; SiLU on q, k, v, the rule, then o / rms(o) *
+// weight * sigmoid(g), the norm over all heads of a row together (vdim values each). Tiles: one per row. o: scratch, fp32 rows of heads * vdim_p; counters:
+// one int per row, zero before the first call.
+typedef struct {
+  int f32, rows;
+  const void* qkvg; int ld_qkvg;
+  const float* powers;
+  int heads, vdim, dim_p, vdim_p;
+  float* state;
+  float* o; int ld_o; int* counters;
+  const void* weight; float eps;
+  void* out; int ld_out;
+  const nfn_row_tile* tiles;
+} nfn_linear_step_args;
+int nfn_linear_step_fits(int rows, int dim_p, int vdim_p);
+int nfn_linear_step(const nfn_linear_step_args* args, nfn_stream_t stream);
+// out = o / rms(o) * weight * sigmoid(gate) over whole rows of `cols` values of which `live` count; weight bf16 [cols], out and gate in the activation type.
+int nfn_row_out(int f32, const float* o, int ld_o, const void* gate, int ld_gate, const void* weight, float eps, void* out, int ld_out, int rows, int cols, int live,
+                nfn_stream_t stream);
+
+// ---- gated recurrence without a matrix in its loop (gru_rows.cu) ------------------------------------------------------------------------------------------
+// Per channel, with the fp32 state s of the sequence: z = sigmoid(a), c = b + 1/2 (b >= 0) or sigmoid(b), s <- (1 - z) s + z c, out = s * silu(g).
+// in: rows [a | b | g] of `width` channels each (a multiple of 16), biases added; state [slots][width]; a sequence at position 0 starts from zero. Entries
+// of at most 16 rows go token after token (n_short of them, first in seqs), longer ones in segments that a scan joins.
+typedef struct {
+  int f32, width;
+  const void* in; int ld_in;
+  float* state;
+  void* out; int ld_out;
+  const nfn_seq_rows* seqs; int n_seqs, n_short;
+} nfn_gru_args;
+int nfn_gru_rows(const nfn_gru_args* args, nfn_stream_t stream);
+
 // ---- mixture of experts for the rows of a step (moe.cu, moe_rows.cu) ----------------------------------------------------------
-// item i = token i / top, choice i % top. Gated experts take the routing weight at their INPUT: mid = act(w G h) * (w U h); plain ones (w_gate_up
-// [E][ff][width]) compute mid = act(U h) and leave the weight to whoever sums the items.
+// item i = token i / top, choice i % top. Gated experts take the routing weight at their INPUT: mid = act(w G h) * (w U h); with weigh_output, and plain
+// ones (w_gate_up [E][ff][width], mid = act(U h)), they leave it to whoever sums the items.
 // nfn_route_rule: how experts are chosen and weighted. s = sigmoid(logits). The choice goes by s + correction (bf16, NULL: by s). groups > 0: group g is
 // experts [g E / groups, (g + 1) E / groups); the keep_groups whose two best members add up to most stay open, the rest are out of the choice.
-// Weights: s, with normalise / (sum of the chosen ones + 1e-20), times scale. Ties: the lower index.
-typedef struct { const void* correction; int groups, keep_groups, normalise; float scale; } nfn_route_rule;
+// Weights: s, with normalise / (sum of the chosen ones + 1e-20), times scale. Ties: the lower index. softmax: the choice goes by the logits and the weights
+// are the softmax over the chosen ones alone, times scale (no correction, no groups).
+typedef struct { const void* correction; int groups, keep_groups, normalise; float scale; int softmax; } nfn_route_rule;
 int nfn_moe_choose(const float* logits, int ld, int T, int E, int k, const nfn_route_rule* rule, int* idx, float* weight, int* counts, nfn_stream_t stream);
 int nfn_moe_route(const float* logits, int ld, int T, int E, int k, int score_fn, int norm_topk, float route_scale, int* topk_idx, float* topk_w,
                   int* counts, nfn_stream_t stream);
@@ -575,8 +650,9 @@ int nfn_moe_plan(const int* counts, int E, int max_tiles, int* offsets, int* cur
 // nfn_moe_permute that also leaves each sorted row's routing weight in row_w.
 int nfn_moe_permute_weighted(const void* x, int ldx, int T, int k, int d, const int* topk_idx, const float* topk_w, const int* offsets, int* cursor,
                              int capacity_rows, void* xs, int* row_of, float* row_w, nfn_stream_t stream);
-// mid[r] = act(w G) * (w U) over the first plan[1] rows of gate_up [rows][2 * ff] (bf16), w = row_w[r].
-int nfn_moe_act_rows(const void* gate_up, const float* row_w, const int* plan, int capacity_rows, int ff, int act, void* mid, nfn_stream_t stream);
+// mid[r] = act(w G) * (w U) over the first plan[1] rows of gate_up [rows][2 * ff] (bf16), w = row_w[r] (NULL: 1); clamp as in nfn_ff_rows.
+int nfn_moe_act_rows(const void* gate_up, const float* row_w, const int* plan, int capacity_rows, int ff, int act, const nfn_gate_clamp* clamp, void* mid,
+                     nfn_stream_t stream);
 // Few rows: routing and a list of items per expert in one launch (order: items by expert; offsets: experts + 1; active: experts with items,
 // active[experts] their number), then the products of the chosen experts only, item by item. w_gate_up [E][2 ff][width], w_down [E][width][ff].
 typedef struct {
@@ -591,6 +667,8 @@ typedef struct {
   nfn_route_rule rule;                    // scale 0 counts as 1
   // shared_ff > 0: the second product of an expert that every row has, y_shared [rows][ld_y] = w_shared_down shared_mid [rows][shared_ff], beside the others
   int shared_ff; const void* shared_mid; const void* w_shared_down; void* y_shared;
+  int weigh_output;
+  nfn_gate_clamp clamp;                   // of NFN_ACT_CLAMPED
 } nfn_moe_rows_args;
 int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream);
 

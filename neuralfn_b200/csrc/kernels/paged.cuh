@@ -83,4 +83,19 @@ __device__ __forceinline__ float sigmoid_for(float v) {
 }
 __device__ __forceinline__ float sigmoid_exact(float v) { return 1.f / (1.f + expf(-v)); }
 
+// the product of a feed-forward's gate and up values
+template <typename T>
+__device__ __forceinline__ float ff_gated(float g, float u, int act, const nfn_gate_clamp& c) {
+  if (act != NFN_ACT_CLAMPED) return ff_act(g, act) * u;
+  g = fminf(g, c.limit);
+  u = fmaxf(-c.limit, fminf(u, c.limit));
+  return g * sigmoid_for<T>(c.slope * g) * (u + c.shift);
+}
+
+// the score without a key in a row's softmax: is there one, and its value
+__device__ __forceinline__ bool has_sink(const nfn_paged_attention_args& a) { return a.sink || a.sinks; }
+__device__ __forceinline__ float sink_score(const nfn_paged_attention_args& a, int h) {
+  return a.sinks ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.sinks)[h]) : 0.f;
+}
+
 }  // namespace nfn

@@ -252,7 +252,8 @@ paged_decode_kernel(const PagedDecodeParams p) {
   float* part = p.partial + (cell * p.splits + blockIdx.x) * NH * (VP + 2);
   for (int i = threadIdx.x; i < n_heads * VP; i += PD_THREADS) {
     const int h = i / VP, ch = i % VP;
-    float mx = p.splits == 1 && a.sink ? 0.f : -INFINITY;
+    const float sink = has_sink(a) ? sink_score(a, h0 + h) * LOG2E : -INFINITY;
+    float mx = p.splits == 1 ? sink : -INFINITY;
 #pragma unroll
     for (int w = 0; w < PD_WARPS; ++w) mx = fmaxf(mx, sm[w * NH + h]);
     float o = 0.f, sum = 0.f;
@@ -265,7 +266,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
       }
     }
     if (p.splits == 1) {
-      if (a.sink) sum += exp2f(-mx);
+      if (has_sink(a)) sum += exp2f(sink - mx);
       finish(h, ch, o / sum);
     } else {
       part[(size_t)h * (VP + 2) + ch] = o;
@@ -286,7 +287,8 @@ paged_decode_kernel(const PagedDecodeParams p) {
   const float* all = p.partial + cell * p.splits * NH * (VP + 2);
   for (int i = threadIdx.x; i < n_heads * VP; i += PD_THREADS) {
     const int h = i / VP, ch = i % VP;
-    float mx = a.sink ? 0.f : -INFINITY;
+    const float sink = has_sink(a) ? sink_score(a, h0 + h) * LOG2E : -INFINITY;
+    float mx = sink;
     for (int s2 = 0; s2 < p.splits; ++s2) mx = fmaxf(mx, __ldcg(&all[((size_t)s2 * NH + h) * (VP + 2) + VP]));
     float o = 0.f, sum = 0.f;
     for (int s2 = 0; s2 < p.splits; ++s2) {
@@ -295,7 +297,7 @@ paged_decode_kernel(const PagedDecodeParams p) {
       o += f * __ldcg(q + ch);
       sum += f * __ldcg(q + VP + 1);
     }
-    if (a.sink) sum += exp2f(-mx);
+    if (has_sink(a)) sum += exp2f(sink - mx);
     finish(h, ch, o / sum);
   }
   if (threadIdx.x == 0) p.counters[cell] = 0;

@@ -229,7 +229,7 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     const int v_lo = row_ok ? first_visible(a, pos) : 0;
     const int lo_last = first_visible(a, pos0 + n_rows - 1);
     const int v_keep = min(a.keep_first, v_hi);
-    float m_run = a.sink ? 0.f : -INFINITY, l_run = a.sink ? 1.f : 0.f;  // units of log2; the sink counts as seen before all keys
+    float m_run = has_sink(a) ? sink_score(a, h) * LOG2E : -INFINITY, l_run = has_sink(a) ? 1.f : 0.f;  // units of log2; the sink counts as seen before all keys
     bool ok = true;
     for (int j = 0; j < nblk; ++j) {
       ok = mbar_wait_bounded(smem_u32(bar_s), j & 1, cta_abort, p.status, 0x600 + 9);

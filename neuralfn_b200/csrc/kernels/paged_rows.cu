@@ -283,7 +283,7 @@ mix_rows_kernel(const nfn_mix_args p) {
 // out = act(gate) * up over all rows of a call: two rows per thread, few registers. off_up < 0: out = act(gate)
 template <typename T>
 __global__ void __launch_bounds__(256)
-ff_rows_kernel(const T* __restrict__ src, int ld_in, int off_gate, int off_up, int ff, int act, T* __restrict__ dst, int ld_out, int rows) {
+ff_rows_kernel(const T* __restrict__ src, int ld_in, int off_gate, int off_up, int ff, int act, nfn_gate_clamp clamp, T* __restrict__ dst, int ld_out, int rows) {
   const int c = (blockIdx.x * 256 + threadIdx.x) * 8, r0 = blockIdx.y * 2;
   if (c >= ff) return;
   const T* in = src + (size_t)r0 * ld_in + c;
@@ -300,14 +300,14 @@ ff_rows_kernel(const T* __restrict__ src, int ld_in, int off_gate, int off_up, i
   for (int i = 0; i < 2; ++i)
     if (i == 0 || two) {
 #pragma unroll
-      for (int e = 0; e < 8; ++e) g[i][e] = ff_act(g[i][e], act) * (up ? u[i][e] : 1.f);
+      for (int e = 0; e < 8; ++e) g[i][e] = up ? ff_gated<T>(g[i][e], u[i][e], act, clamp) : ff_act(g[i][e], act);
       store8(out + (size_t)i * ld_out, g[i]);
     }
 }
 
 template <typename T>
-static void launch_ff_rows(const void* in, int ld_in, int off_gate, int off_up, int ff, int act, void* out, int ld_out, int rows, cudaStream_t st) {
-  ff_rows_kernel<T><<<dim3(ceil_div(ff, 256 * 8), ceil_div(rows, 2)), 256, 0, st>>>(static_cast<const T*>(in), ld_in, off_gate, off_up, ff, act, static_cast<T*>(out),
+static void launch_ff_rows(const void* in, int ld_in, int off_gate, int off_up, int ff, int act, const nfn_gate_clamp& clamp, void* out, int ld_out, int rows, cudaStream_t st) {
+  ff_rows_kernel<T><<<dim3(ceil_div(ff, 256 * 8), ceil_div(rows, 2)), 256, 0, st>>>(static_cast<const T*>(in), ld_in, off_gate, off_up, ff, act, clamp, static_cast<T*>(out),
                                                                                     ld_out, rows);
 }
 
@@ -351,7 +351,7 @@ paged_attention_plain_kernel(const nfn_paged_attention_args p) {
   float acc[PLAIN_MAX_VEC];
 #pragma unroll
   for (int i = 0; i < PLAIN_MAX_VEC; ++i) acc[i] = 0.f;
-  float m = p.sink ? 0.f : -INFINITY, l = p.sink ? 1.f : 0.f;      // the sink is an element seen before all others
+  float m = has_sink(p) ? sink_score(p, h) : -INFINITY, l = has_sink(p) ? 1.f : 0.f;      // the sink is an element seen before all others
   for (int base = keep > 0 ? 0 : lo / 32 * 32; base <= pos; base += 32) {   // a chunk never crosses a page
     if (base >= keep && base + 32 <= lo) base = lo / 32 * 32;      // from the kept tokens to the window
     const size_t tile = (size_t)table[base / NFN_PAGE] * p.kv_heads + hk;
@@ -562,19 +562,22 @@ extern "C" int nfn_mix_rows(const nfn_mix_args* args, nfn_stream_t stream) {
   if (a.f32) launch_mix_rows<float>(a, grid, st);
   else launch_mix_rows<__nv_bfloat16>(a, grid, st);
   if (split) {
-    if (a.f32) launch_ff_rows<float>(a.in, a.ld_in, a.off_gate, a.off_up, a.ff, a.act, a.ff_out, a.ld_ff, a.rows, st);
-    else launch_ff_rows<__nv_bfloat16>(a.in, a.ld_in, a.off_gate, a.off_up, a.ff, a.act, a.ff_out, a.ld_ff, a.rows, st);
+    if (a.f32) launch_ff_rows<float>(a.in, a.ld_in, a.off_gate, a.off_up, a.ff, a.act, nfn_gate_clamp{}, a.ff_out, a.ld_ff, a.rows, st);
+    else launch_ff_rows<__nv_bfloat16>(a.in, a.ld_in, a.off_gate, a.off_up, a.ff, a.act, nfn_gate_clamp{}, a.ff_out, a.ld_ff, a.rows, st);
   }
   return launch_check("mix_rows", split ? 2 : 1);
 }
 
-extern "C" int nfn_ff_rows(int f32, const void* in, int ld_in, int off_gate, int off_up, int ff, int act, void* out, int ld_out, int rows, nfn_stream_t stream) {
+extern "C" int nfn_ff_rows(int f32, const void* in, int ld_in, int off_gate, int off_up, int ff, int act, const nfn_gate_clamp* clamp, void* out, int ld_out, int rows,
+                           nfn_stream_t stream) {
   if (rows <= 0 || ff <= 0) return 0;
   if ((ld_in | off_gate | ff | ld_out) & 7 || (off_up >= 0 && (off_up & 7))) return fail(-1, "ff_rows: widths and offsets must be multiples of 8");
   if (ceil_div(rows, 2) > 65535) return fail(-1, "ff_rows: too many rows in one launch");
+  if (act == NFN_ACT_CLAMPED && (!clamp || off_up < 0)) return fail(-1, "ff_rows: the clamped gate needs its limits and an up value");
+  const nfn_gate_clamp limits = clamp ? *clamp : nfn_gate_clamp{};
   cudaStream_t st = static_cast<cudaStream_t>(stream);
-  if (f32) launch_ff_rows<float>(in, ld_in, off_gate, off_up, ff, act, out, ld_out, rows, st);
-  else launch_ff_rows<__nv_bfloat16>(in, ld_in, off_gate, off_up, ff, act, out, ld_out, rows, st);
+  if (f32) launch_ff_rows<float>(in, ld_in, off_gate, off_up, ff, act, limits, out, ld_out, rows, st);
+  else launch_ff_rows<__nv_bfloat16>(in, ld_in, off_gate, off_up, ff, act, limits, out, ld_out, rows, st);
   return launch_check("ff_rows");
 }
 

@@ -2,7 +2,9 @@
 // output enters all of them through a small mixing matrix, the next sublayer reads a weighted sum of them through its norm. One CTA
 // per row does both: every stream is read and written once, the weighted sum waits in shared memory until its norm is known.
 // A single plain residual is the case of one stream with unit weights. The update may have a norm of its own (designs that norm a sublayer's output
-// instead of its input), its rows may carry weights (routed experts) and a row every token has (a shared expert).
+// instead of its input), its rows may carry weights (routed experts) and a row every token has (a shared expert). Where every row is the next token of
+// its own sequence the pass also adds the short convolution of designs whose sublayers read their input that way; other batches take a
+// launch of its own for it, since a row then needs its neighbours' norms.
 #include "common.h"
 #include "paged.cuh"
 
@@ -20,9 +22,19 @@ __device__ __forceinline__ float st_block_sum(float v, float* red) {
   return t;
 }
 
-// S: streams held in registers (an upper bound; the mixing weights past p.streams are zero). Few rows take many threads each, so that a
+constexpr int ST_HIST = 3;      // history rows fetched ahead
+
+// the norm's weights of channels 4 v .. 4 v + 3; one number for all of them
+__device__ __forceinline__ float4 st_weight(const void* w, int v, int scalar) {
+  const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(w);
+  if (!scalar) return load4(p + 4 * v);
+  const float f = __bfloat162float(*p);
+  return make_float4(f, f, f, f);
+}
+
+// S: streams held in registers (an upper bound; the mixing weights past p.streams are zero). CONV: with the short convolution. Few rows take many threads each, so that a
 // row's loads are all on their way at once
-template <typename T, int S, int ST_THREADS>
+template <typename T, int S, int ST_THREADS, bool CONV>
 __global__ void __launch_bounds__(ST_THREADS)
 stream_pass_kernel(const nfn_stream_args p) {
   extern __shared__ float st_row[];                        // [ld] u
@@ -73,7 +85,25 @@ stream_pass_kernel(const nfn_stream_args p) {
     fetch_y(threadIdx.x);
   }
   float4 wt = make_float4(0.f, 0.f, 0.f, 0.f);             // the norm's weights of the first piece come along
-  if (p.h && p.weight && threadIdx.x < vecs) wt = load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * threadIdx.x);
+  if (p.h && p.weight && threadIdx.x < vecs) wt = st_weight(p.weight, threadIdx.x, p.scalar_norms);
+  nfn_row_tile tile{};
+  const T* old = nullptr;                                  // the sequence's stored rows; none before its start
+  float4 past[ST_HIST], taps[ST_HIST + 1];
+  const int hist = p.conv_taps - 1;
+  const __nv_bfloat16* conv = static_cast<const __nv_bfloat16*>(p.conv);
+  auto stored = [&](int i, int v) { return old && tile.e_pos0 - hist + i >= 0 ? load4(old + (size_t)i * p.ld + 4 * v) : make_float4(0.f, 0.f, 0.f, 0.f); };
+  if constexpr (CONV) {
+    tile = p.tiles[r];
+    if (tile.slot >= 0 && hist > 0) old = static_cast<const T*>(p.history) + (size_t)tile.parity * p.history_half + (size_t)tile.slot * hist * p.ld;
+    if (threadIdx.x < vecs) {
+#pragma unroll
+      for (int i = 0; i < ST_HIST; ++i)
+        if (i < hist) past[i] = stored(i, threadIdx.x);
+#pragma unroll
+      for (int i = 0; i <= ST_HIST; ++i)
+        if (i <= hist) taps[i] = load4(conv + (size_t)i * p.ld + 4 * threadIdx.x);
+    }
+  }
   __syncthreads();
   float ry = 0.f;
   if (p.y_weight) {                                        // the update's own norm: its pieces past the first one wait in shared memory
@@ -95,7 +125,7 @@ stream_pass_kernel(const nfn_stream_args p) {
       else fetch_y(v);
     }
     if (p.y_weight) {
-      const float4 w = load4(static_cast<const __nv_bfloat16*>(p.y_weight) + 4 * v);
+      const float4 w = st_weight(p.y_weight, v, p.scalar_norms);
       f.x *= ry * w.x; f.y *= ry * w.y; f.z *= ry * w.z; f.w *= ry * w.w;
     }
     if (emb) {
@@ -142,16 +172,139 @@ stream_pass_kernel(const nfn_stream_args p) {
   const float rms = 1.f / sqrtf(st_block_sum<ST_THREADS>(ss, red) / (float)p.width + p.eps);
   T* h = static_cast<T*>(p.h) + (size_t)r * p.ld;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
-    const float4 u = load4(st_row + 4 * v), w = v == threadIdx.x ? wt : load4(static_cast<const __nv_bfloat16*>(p.weight) + 4 * v);
-    store4(h + 4 * v, make_float4(u.x * rms * (w.x + p.weight_offset), u.y * rms * (w.y + p.weight_offset), u.z * rms * (w.z + p.weight_offset),
-                                  u.w * rms * (w.w + p.weight_offset)));
+    const float4 u = load4(st_row + 4 * v), w = v == threadIdx.x ? wt : st_weight(p.weight, v, p.scalar_norms);
+    const float4 n = make_float4(u.x * rms * (w.x + p.weight_offset), u.y * rms * (w.y + p.weight_offset), u.z * rms * (w.z + p.weight_offset), u.w * rms * (w.w + p.weight_offset));
+    if constexpr (CONV) {
+      float4 c = n;
+      T* left = tile.slot >= 0 && hist > 0 ? static_cast<T*>(p.history) + (size_t)(1 - tile.parity) * p.history_half + (size_t)tile.slot * hist * p.ld + 4 * v : nullptr;
+      auto add = [&](int i, const float4& x, const float4& t) {
+        c.x += t.x * x.x; c.y += t.y * x.y; c.z += t.z * x.z; c.w += t.w * x.w;
+        if (left && i > 0) store4(left + (size_t)(i - 1) * p.ld, x);
+      };
+      const bool ahead = v == threadIdx.x && hist <= ST_HIST;
+      if (ahead) {
+#pragma unroll
+        for (int i = 0; i < ST_HIST; ++i)
+          if (i < hist) add(i, past[i], taps[i]);
+#pragma unroll
+        for (int i = 0; i <= ST_HIST; ++i)
+          if (i == hist) add(i, n, taps[i]);
+      } else {
+        for (int i = 0; i < hist; ++i) add(i, stored(i, v), load4(conv + (size_t)i * p.ld + 4 * v));
+        add(hist, n, load4(conv + (size_t)hist * p.ld + 4 * v));
+      }
+      store4(h + 4 * v, c);
+    } else {
+      store4(h + 4 * v, n);
+    }
   }
 }
 
-template <typename T, int S, int THREADS>
+// The convolution over the rows of any entries. A thread takes eight channels of a tile's rows; the window slides through registers (TAPS = 0: any
+// number of taps, rows are read again).
+constexpr int IC_THREADS = 128;
+
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(IC_THREADS)
+input_conv_kernel(const nfn_input_conv_args p) {
+  const nfn_row_tile t = p.tiles[blockIdx.x];
+  const int col = (blockIdx.y * IC_THREADS + threadIdx.x) * 8;
+  if (t.slot < 0 || col >= p.ld) return;
+  const int taps = TAPS ? TAPS : p.taps, hist = taps - 1, ti0 = t.row0 - t.e_row0;
+  const T* rows = static_cast<const T*>(p.h) + (size_t)t.e_row0 * p.ld + col;
+  const T* old = static_cast<const T*>(p.history) + (size_t)t.parity * p.history_half + (size_t)t.slot * hist * p.ld + col;
+  T* left = static_cast<T*>(p.history) + (size_t)(1 - t.parity) * p.history_half + (size_t)t.slot * hist * p.ld + col;
+  const __nv_bfloat16* conv = static_cast<const __nv_bfloat16*>(p.conv) + col;
+  T* out = static_cast<T*>(p.out) + (size_t)t.row0 * p.ld + col;
+  const bool last = hist > 0 && t.row0 + t.n == t.e_row0 + t.e_n;
+  // row `idx` of the entry: this step's, a stored one, or zero before the sequence's start
+  auto source = [&](int idx, float (&v)[8]) {
+    if (idx >= 0) {
+      load8(rows + (size_t)idx * p.ld, v);
+    } else if (t.e_pos0 + idx >= 0) {
+      load8(old + (size_t)(hist + idx) * p.ld, v);
+    } else {
+#pragma unroll
+      for (float& f : v) f = 0.f;
+    }
+  };
+  if constexpr (TAPS == 0) {
+    for (int i = 0; i < t.n; ++i) {
+      float acc[8], x[8], w[8];
+      source(ti0 + i, acc);
+      for (int j = 0; j < taps; ++j) {
+        source(ti0 + i - hist + j, x);
+        load8(conv + (size_t)j * p.ld, w);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) acc[e] += w[e] * x[e];
+      }
+      store8(out + (size_t)i * p.ld, acc);
+    }
+    if (last)
+      for (int i = 0; i < hist; ++i) {
+        float x[8];
+        source(t.e_n - hist + i, x);
+        store8(left + (size_t)i * p.ld, x);
+      }
+  } else {
+    constexpr int N = 4;                                   // rows in flight
+    float win[TAPS > 1 ? TAPS - 1 : 1][8], w[TAPS][8], v[N][8];
+    auto fetch = [&](int i0) {
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+        if (i0 + i < t.n) load8(rows + (size_t)(ti0 + i0 + i) * p.ld, v[i]);
+    };
+    fetch(0);
+#pragma unroll
+    for (int j = 0; j < TAPS - 1; ++j) source(ti0 - (TAPS - 1) + j, win[j]);
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) load8(conv + (size_t)j * p.ld, w[j]);
+    for (int i0 = 0; i0 < t.n; i0 += N) {
+      if (i0 > 0) fetch(i0);
+#pragma unroll
+      for (int i = 0; i < N; ++i)
+        if (i0 + i < t.n) {
+          float acc[8];
+#pragma unroll
+          for (int e = 0; e < 8; ++e) {
+            const float x = v[i][e];
+            float a = x + w[TAPS - 1][e] * x;
+#pragma unroll
+            for (int j = 0; j < TAPS - 1; ++j) a += w[j][e] * win[j][e];
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
+            if constexpr (TAPS > 1) win[TAPS - 2][e] = x;
+            acc[e] = a;
+          }
+          store8(out + (size_t)(i0 + i) * p.ld, acc);
+        }
+    }
+    if constexpr (TAPS > 1) {
+      if (last) {
+#pragma unroll
+        for (int j = 0; j < TAPS - 1; ++j) store8(left + (size_t)j * p.ld, win[j]);
+      }
+    }
+  }
+}
+
+template <typename T>
+static int pick_input_conv(const nfn_input_conv_args& a, cudaStream_t st) {
+  const dim3 grid(a.n_tiles, ceil_div(a.ld, IC_THREADS * 8));
+  switch (a.taps) {
+    case 1: input_conv_kernel<T, 1><<<grid, IC_THREADS, 0, st>>>(a); break;
+    case 2: input_conv_kernel<T, 2><<<grid, IC_THREADS, 0, st>>>(a); break;
+    case 3: input_conv_kernel<T, 3><<<grid, IC_THREADS, 0, st>>>(a); break;
+    case 4: input_conv_kernel<T, 4><<<grid, IC_THREADS, 0, st>>>(a); break;
+    default: input_conv_kernel<T, 0><<<grid, IC_THREADS, 0, st>>>(a); break;
+  }
+  return launch_check("input_conv");
+}
+
+template <typename T, int S, int THREADS, bool CONV = false>
 static int launch_stream(const nfn_stream_args& a, cudaStream_t st) {
   const size_t smem = a.h || a.y_weight ? (size_t)a.ld * sizeof(float) : 0;
-  auto kern = stream_pass_kernel<T, S, THREADS>;
+  auto kern = stream_pass_kernel<T, S, THREADS, CONV>;
   static bool raised[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -166,6 +319,7 @@ static int launch_stream(const nfn_stream_args& a, cudaStream_t st) {
 template <typename T>
 static int pick_stream(const nfn_stream_args& a, cudaStream_t st) {
   const bool few = a.rows <= 2 * sm_count() && a.ld >= 2048;
+  if (a.conv) return few ? launch_stream<T, 1, 1024, true>(a, st) : launch_stream<T, 1, 256, true>(a, st);
   switch (a.streams) {
     case 1: return few ? launch_stream<T, 1, 1024>(a, st) : launch_stream<T, 1, 256>(a, st);
     case 2: return few ? launch_stream<T, 2, 1024>(a, st) : launch_stream<T, 2, 256>(a, st);
@@ -188,5 +342,15 @@ extern "C" int nfn_stream_pass(const nfn_stream_args* args, nfn_stream_t stream)
   if (!a.tokens && !a.x) return fail(-1, "stream_pass: neither tokens nor rows");
   if (a.y && a.y_rows < 1) return fail(-1, "stream_pass: an update needs at least one row");
   if ((size_t)a.ld * 4 > 200 * 1024) return fail(-1, "stream_pass: rows too wide");
+  if (a.conv && (a.streams != 1 || !a.h || !a.weight || !a.tiles || a.conv_taps < 1 || (a.conv_taps > 1 && !a.history)))
+    return fail(-1, "stream_pass: the convolution goes with one stream, a norm, a tile per row and a history");
   return a.f32 ? pick_stream<float>(a, static_cast<cudaStream_t>(stream)) : pick_stream<__nv_bfloat16>(a, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int nfn_input_conv(const nfn_input_conv_args* args, nfn_stream_t stream) {
+  if (!args) return fail(-1, "input_conv: null args");
+  const nfn_input_conv_args& a = *args;
+  if (a.n_tiles <= 0) return 0;
+  if ((a.ld & 15) || a.taps < 1 || !a.h || !a.conv || !a.out || a.h == a.out || !a.tiles || (a.taps > 1 && !a.history)) return fail(-1, "input_conv: rows padded to multiples of 16, two buffers, a history");
+  return a.f32 ? pick_input_conv<float>(a, static_cast<cudaStream_t>(stream)) : pick_input_conv<__nv_bfloat16>(a, static_cast<cudaStream_t>(stream));
 }

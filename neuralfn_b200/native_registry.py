@@ -76,6 +76,7 @@ NATIVE_FAMILIES: dict[str, NativeTrainerSpec] = {s.family: s for s in (
     NativeTrainerSpec("bulidra", (), "", (), "serving-only", resident_inference=True, checkpoint_formats=("model-directory",)),
     NativeTrainerSpec("murilorn", (), "", (), "serving-only", resident_inference=True, checkpoint_formats=("model-directory",)),
     NativeTrainerSpec("vopozen", (), "", (), "serving-only", resident_inference=True, checkpoint_formats=("model-directory",)),
+    NativeTrainerSpec("kidolorn", (), "", (), "serving-only", resident_inference=True, checkpoint_formats=("model-directory",)),
     _spec("seq2seq", (), ("seq2seq",)), _spec("diffusion", (), ("diffusion",)), _spec("ttt-llama", (), ("ttt_llama",)),
     _spec("hnet-lm", (), ("hnet_lm",)), _spec("universal-llama", (), ("universal_llama",)),
 )}

@@ -65,7 +65,8 @@ def _compile_one(src: Path, obj: Path, extra: list[str], verbose: bool) -> str:
 # Components: the sources one kind of model needs, built into a library of their own by ``ensure_component``. "all" is the whole library.
 COMPONENTS: dict[str, tuple[str, ...]] = {
     "layered": ("common.cu", "gemm_tcgen05.cu", "gemm_2cta.cu", "gemv_bf16.cu", "gemm_skinny.cu", "sampling.cu", "paged_rows.cu", "paged_decode.cu",
-                "paged_prefill.cu", "stream_rows.cu", "delta_rows.cu", "delta_chunk.cu", "moe.cu", "moe_rows.cu", "gemm_tp.cu", "head_rows.cu", "latent_decode.cu", "wkv_rows.cu", "wkv_chunk.cu", "engine_core.cpp", "layered_engine.cpp"),
+                "paged_prefill.cu", "stream_rows.cu", "delta_rows.cu", "delta_chunk.cu", "moe.cu", "moe_rows.cu", "gemm_tp.cu", "head_rows.cu", "latent_decode.cu", "wkv_rows.cu", "wkv_chunk.cu", "linear_rows.cu", "linear_chunk.cu",
+                "gru_rows.cu", "engine_core.cpp", "layered_engine.cpp"),
 }
 
 

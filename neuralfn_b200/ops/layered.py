@@ -20,7 +20,8 @@ class _Stream(C.Structure):
                 ("src_rows", C.c_void_p), ("tokens", C.c_void_p), ("embed", C.c_void_p), ("embed_scale", C.c_float), ("vocab", C.c_int), ("y", C.c_void_p),
                 ("y_rows", C.c_int), ("y_index", C.c_void_p), ("mix", C.c_void_p), ("out", C.c_void_p), ("in_", C.c_void_p), ("h", C.c_void_p),
                 ("weight", C.c_void_p), ("eps", C.c_float), ("weight_offset", C.c_float), ("y_item", C.c_void_p), ("y_plus", C.c_void_p), ("y_weight", C.c_void_p),
-                ("y_scale", C.c_float)]
+                ("y_scale", C.c_float), ("scalar_norms", C.c_int), ("conv", C.c_void_p), ("conv_taps", C.c_int), ("history", C.c_void_p), ("history_half", C.c_longlong),
+                ("tiles", C.c_void_p)]
 
 
 class _Delta(C.Structure):
@@ -31,7 +32,7 @@ class _Delta(C.Structure):
 
 class RouteRule(C.Structure):
     """``nfn_route_rule``"""
-    _fields_ = [("correction", C.c_void_p), ("groups", C.c_int), ("keep_groups", C.c_int), ("normalise", C.c_int), ("scale", C.c_float)]
+    _fields_ = [("correction", C.c_void_p), ("groups", C.c_int), ("keep_groups", C.c_int), ("normalise", C.c_int), ("scale", C.c_float), ("softmax", C.c_int)]
 
 
 class _Experts(C.Structure):
@@ -39,7 +40,8 @@ class _Experts(C.Structure):
                 ("logits", C.c_void_p), ("ld_logits", C.c_int), ("h", C.c_void_p), ("ld_h", C.c_int), ("w_gate_up", C.c_void_p), ("w_down", C.c_void_p),
                 ("idx", C.c_void_p), ("weight", C.c_void_p), ("order", C.c_void_p), ("offsets", C.c_void_p), ("active", C.c_void_p), ("mid", C.c_void_p),
                 ("y", C.c_void_p), ("ld_y", C.c_int), ("plain", C.c_int), ("rule", RouteRule), ("shared_ff", C.c_int),
-                ("shared_mid", C.c_void_p), ("w_shared_down", C.c_void_p), ("y_shared", C.c_void_p)]
+                ("shared_mid", C.c_void_p), ("w_shared_down", C.c_void_p), ("y_shared", C.c_void_p), ("weigh_output", C.c_int), ("limit", C.c_float), ("slope", C.c_float),
+                ("shift", C.c_float)]
 
 
 def _p(t: torch.Tensor | None):
@@ -54,10 +56,13 @@ def stream_pass(x: torch.Tensor | None, h: torch.Tensor | None, *, width: int, s
                 weight_offset: float = 0.0, x_out: torch.Tensor | None = None, src_rows: torch.Tensor | None = None, y: torch.Tensor | None = None, y_rows: int = 1,
                 y_index: torch.Tensor | None = None, mix: torch.Tensor | None = None, out: torch.Tensor | None = None, into: torch.Tensor | None = None,
                 tokens: torch.Tensor | None = None, embed: torch.Tensor | None = None, embed_scale: float = 1.0, y_item: torch.Tensor | None = None,
-                y_plus: torch.Tensor | None = None, y_weight: torch.Tensor | None = None, y_scale: float = 1.0) -> None:
-    """x fp32 [rows, streams, ld]; see ``nfn_stream_args``. ``into``: weights of the streams in the next sublayer's input."""
+                y_plus: torch.Tensor | None = None, y_weight: torch.Tensor | None = None, y_scale: float = 1.0, scalar_norms: bool = False, conv: torch.Tensor | None = None,
+                history: torch.Tensor | None = None, tiles: torch.Tensor | None = None) -> None:
+    """x fp32 [rows, streams, ld]; see ``nfn_stream_args``. ``into``: weights of the streams in the next sublayer's input. conv bf16 [taps, ld], history
+    [2, slots, taps - 1, ld]: the convolution of rows that are entries of their own."""
     a = _Stream(int(f32), rows, width, ld, streams, _p(x), _p(x_out), _p(src_rows), _p(tokens), _p(embed), embed_scale, 0 if embed is None else embed.shape[0], _p(y), y_rows,
-                _p(y_index), _p(mix), _p(out), _p(into), _p(h), _p(weight), eps, weight_offset, _p(y_item), _p(y_plus), _p(y_weight), y_scale)
+                _p(y_index), _p(mix), _p(out), _p(into), _p(h), _p(weight), eps, weight_offset, _p(y_item), _p(y_plus), _p(y_weight), y_scale, int(scalar_norms), _p(conv),
+                0 if conv is None else conv.shape[0], _p(history), 0 if history is None else history.stride(0), _p(tiles))
     _call("stream_pass", a)
 
 
@@ -89,12 +94,12 @@ def delta_out(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, *, head
     return out
 
 
-def _rule(correction=None, groups=0, keep=0, normalise=False, scale=1.0) -> RouteRule:
-    return RouteRule(_p(correction), groups, keep, int(normalise), scale)
+def _rule(correction=None, groups=0, keep=0, normalise=False, scale=1.0, softmax=False) -> RouteRule:
+    return RouteRule(_p(correction), groups, keep, int(normalise), scale, int(softmax))
 
 
 def expert_choice(logits: torch.Tensor, top: int, **rule) -> tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
-    """Chosen experts [rows, top], weights, tokens per expert. ``rule``: correction (bf16 [experts]), groups, keep, normalise, scale."""
+    """Chosen experts [rows, top], weights, tokens per expert. ``rule``: correction (bf16 [experts]), groups, keep, normalise, scale, softmax."""
     T, E = logits.shape
     idx, weight = torch.zeros(T, top, dtype=torch.int32, device=logits.device), torch.zeros(T, top, device=logits.device)
     counts = torch.zeros(E, dtype=torch.int32, device=logits.device)
@@ -104,9 +109,10 @@ def expert_choice(logits: torch.Tensor, top: int, **rule) -> tuple[torch.Tensor,
 
 
 def expert_rows(h: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor, *, experts: int, top: int, act: int = 3, plain: bool = False,
-                shared_mid: torch.Tensor | None = None, shared_down: torch.Tensor | None = None, y_shared: torch.Tensor | None = None, **rule):
+                shared_mid: torch.Tensor | None = None, shared_down: torch.Tensor | None = None, y_shared: torch.Tensor | None = None, weigh_output: bool = False,
+                clamp: tuple[float, float, float] = (0.0, 0.0, 0.0), **rule):
     """Returns the chosen experts [rows, top], their weights and outputs y [rows, top, width]. plain: w_gate_up holds one matrix per expert. shared_mid [rows, f],
-    shared_down [width, f]: y_shared [rows, width] is their product."""
+    shared_down [width, f]: y_shared [rows, width] is their product. clamp: limit, slope and shift of activation 7."""
     rows, width, ff = h.shape[0], h.shape[1], w_down.shape[2]
     i32 = dict(dtype=torch.int32, device=h.device)
     idx, order, offsets, active = (torch.zeros(n, **i32) for n in (rows * top, rows * top, experts + 1, experts + 1))
@@ -114,7 +120,7 @@ def expert_rows(h: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, 
     mid, y = torch.zeros(rows * top, ff, device=h.device, dtype=h.dtype), torch.zeros(rows * top, width, device=h.device, dtype=h.dtype)
     a = _Experts(int(h.dtype == torch.float32), rows, width, ff, experts, top, act, _p(logits), logits.stride(0), _p(h), h.stride(0), _p(w_gate_up), _p(w_down), _p(idx),
                  _p(weight), _p(order), _p(offsets), _p(active), _p(mid), _p(y), y.stride(0), int(plain), _rule(**rule), 0 if shared_mid is None else shared_mid.shape[1], _p(shared_mid),
-                 _p(shared_down), _p(y_shared))
+                 _p(shared_down), _p(y_shared), int(weigh_output), *clamp)
     _call("moe_rows", a)
     return idx.view(rows, top), weight.view(rows, top), y.view(rows, top, width)
 
@@ -142,7 +148,7 @@ class _Latent(C.Structure):
 class _Groups(C.Structure):
     _fields_ = [("f32", C.c_int), ("rows", C.c_int), ("groups", C.c_int), ("n", C.c_int), ("k", C.c_int), ("in_", C.c_void_p), ("ld_in", C.c_longlong), ("in_group", C.c_longlong),
                 ("w", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_longlong), ("out_group", C.c_longlong), ("act", C.c_int), ("tail_n", C.c_int), ("tail_in", C.c_longlong),
-                ("tail_w", C.c_void_p), ("tail_out", C.c_void_p), ("ld_tail", C.c_int)]
+                ("tail_w", C.c_void_p), ("tail_out", C.c_void_p), ("ld_tail", C.c_int), ("gate", C.c_void_p), ("ld_gate", C.c_longlong), ("gate_group", C.c_longlong)]
 
 
 class _Expanded(C.Structure):
@@ -178,8 +184,9 @@ class LatentCache:
             part = rows[p * PAGE:(p + 1) * PAGE]
             self.k[int(self.table[slot, p]), 0, :part.shape[0]] = part.to(self.dtype)
 
-    def args(self, q: torch.Tensor, out: torch.Tensor, heads: int, window: int, scale: float) -> _Attention:
+    def args(self, q: torch.Tensor, out: torch.Tensor, heads: int, window: int, scale: float, sinks: torch.Tensor | None = None) -> _Attention:
         a = _Attention()
+        a.sinks = _p(sinks)
         a.f32, a.q, a.ld_q, a.k_pool, a.pages = int(self.dtype == torch.float32), _p(q), q.stride(0), _p(self.k), self.k.shape[0]
         a.table, a.table_ld, a.heads, a.window, a.scale, a.out, a.ld_o = _p(self.table), self.table.stride(0), heads, window, scale, _p(out), out.stride(0)
         a.workspace, a.workspace_bytes, a.total_rows = _p(self.ws), self.ws.numel(), q.shape[0]
@@ -195,19 +202,20 @@ def latent_rows(c: LatentCache, x: torch.Tensor, tiles: torch.Tensor, *, heads: 
 
 
 def group_products(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, *, act: int = 0, tail_w: torch.Tensor | None = None, tail_out: torch.Tensor | None = None,
-                   tail_in: int = 0) -> torch.Tensor:
+                   tail_in: int = 0, gate: torch.Tensor | None = None) -> torch.Tensor:
     """x [rows, groups, k], w bf16 [groups, n, k] -> out [rows, groups, n] (any strides over rows and groups); tail_w bf16 [m, k]: one more product, of the input
-    ``tail_in`` elements into each row, into tail_out fp32 [rows, m]."""
+    ``tail_in`` elements into each row, into tail_out fp32 [rows, m]. gate [rows, groups, n]: its sigmoid multiplies the result."""
     a = _Groups(int(x.dtype == torch.float32), x.shape[0], w.shape[0], w.shape[1], w.shape[2], _p(x), x.stride(0), x.stride(1), _p(w), _p(out), out.stride(0), out.stride(1), act,
-                0 if tail_w is None else tail_w.shape[0], tail_in, _p(tail_w), _p(tail_out), 0 if tail_out is None else tail_out.stride(0))
+                0 if tail_w is None else tail_w.shape[0], tail_in, _p(tail_w), _p(tail_out), 0 if tail_out is None else tail_out.stride(0),
+                _p(gate), 0 if gate is None else gate.stride(0), 0 if gate is None else gate.stride(1))
     _call("group_products", a)
     return out
 
 
 def latent_attention_rows(c: LatentCache, q: torch.Tensor, row_slot: torch.Tensor, row_pos: torch.Tensor, out: torch.Tensor, *, heads: int, window: int, scale: float,
-                          max_keys: int = 0) -> torch.Tensor:
+                          max_keys: int = 0, sinks: torch.Tensor | None = None) -> torch.Tensor:
     """q [rows, heads * (rank + rot)], out [rows, heads * rank]: sums of latents."""
-    a = c.args(q, out, heads, window, scale)
+    a = c.args(q, out, heads, window, scale, sinks)
     a.kv_heads, a.dim_p, a.vdim_p = 1, c.rank + c.rot, c.rank
     a.row_slot, a.row_pos, a.rows, a.max_keys = _p(row_slot), _p(row_pos), q.shape[0], max_keys or window or c.table.shape[1] * PAGE
     _call("paged_attention_rows", a)
@@ -223,9 +231,10 @@ def latent_gather(c: LatentCache, spans: torch.Tensor, out: torch.Tensor, max_pa
 
 
 def latent_attention_tiles(c: LatentCache, q: torch.Tensor, x: torch.Tensor, x_base: torch.Tensor, tiles: torch.Tensor, out: torch.Tensor, *, heads: int, dim: int, vdim: int,
-                           window: int, scale: float) -> torch.Tensor:
+                           window: int, scale: float, sinks: torch.Tensor | None = None, gate: torch.Tensor | None = None) -> torch.Tensor:
     """q [rows, heads * (dim + rot)]; x [n, heads * dim keys | heads * vdim values] formed from the gathered latents; tiles as in ``ops.paged.attention_tiles``."""
-    a = c.args(q, out, heads, window, scale)
+    a = c.args(q, out, heads, window, scale, sinks)
+    a.gate, a.ld_gate = _p(gate), 0 if gate is None else gate.stride(0)
     a.kv_heads, a.dim_p, a.vdim_p, a.tiles, a.n_tiles = heads, dim + c.rot, vdim, _p(tiles), tiles.shape[0]
     e = _Expanded(_p(x), x.shape[0], dim, c.rot, c.rank, _p(x_base))
     _lib.check(_lib.load().nfn_latent_attention_tiles(C.byref(a), C.byref(e), C.c_void_p(_lib.stream_ptr())), "latent_attention_tiles")
@@ -284,7 +293,11 @@ def wkv_step(rkvg: torch.Tensor, low: torch.Tensor, w2: torch.Tensor, w0: torch.
     return out
 
 
-def ff_rows(x: torch.Tensor, out: torch.Tensor, *, off_gate: int, off_up: int, act: int) -> torch.Tensor:
+class _Clamp(C.Structure):
+    _fields_ = [("limit", C.c_float), ("slope", C.c_float), ("shift", C.c_float)]
+
+
+def ff_rows(x: torch.Tensor, out: torch.Tensor, *, off_gate: int, off_up: int, act: int, clamp: tuple[float, float, float] = (0.0, 0.0, 0.0)) -> torch.Tensor:
     _lib.check(_lib.load().nfn_ff_rows(C.c_int(int(x.dtype == torch.float32)), C.c_void_p(_p(x)), C.c_int(x.stride(0)), C.c_int(off_gate), C.c_int(off_up), C.c_int(out.shape[1]),
-                                       C.c_int(act), C.c_void_p(_p(out)), C.c_int(out.stride(0)), C.c_int(x.shape[0]), C.c_void_p(_lib.stream_ptr())), "ff_rows")
+                                       C.c_int(act), C.byref(_Clamp(*clamp)), C.c_void_p(_p(out)), C.c_int(out.stride(0)), C.c_int(x.shape[0]), C.c_void_p(_lib.stream_ptr())), "ff_rows")
     return out

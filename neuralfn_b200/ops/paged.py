@@ -19,7 +19,7 @@ class _Attention(C.Structure):
                 ("window", C.c_int), ("scale", C.c_float), ("slopes", C.c_void_p), ("gate", C.c_void_p), ("ld_gate", C.c_int), ("out", C.c_void_p),
                 ("ld_o", C.c_int), ("row_slot", C.c_void_p), ("row_pos", C.c_void_p), ("rows", C.c_int), ("row0", C.c_int), ("max_keys", C.c_int),
                 ("workspace", C.c_void_p), ("workspace_bytes", C.c_longlong), ("tiles", C.c_void_p), ("n_tiles", C.c_int), ("total_rows", C.c_int),
-                ("keep_first", C.c_int), ("softcap", C.c_float), ("sink", C.c_int), ("chunk", C.c_int)]
+                ("keep_first", C.c_int), ("softcap", C.c_float), ("sink", C.c_int), ("chunk", C.c_int), ("sinks", C.c_void_p)]
 
 
 class _Mix(C.Structure):
@@ -63,9 +63,9 @@ class PagedCache:
             self.v[page, :, :, :n] = v[part].permute(1, 2, 0).to(self.dtype)
 
 
-def _args(c: PagedCache, q, out, heads, window, scale, slopes, gate, keep_first=0, softcap=0.0, sink=False, chunk=0) -> _Attention:
+def _args(c: PagedCache, q, out, heads, window, scale, slopes, gate, keep_first=0, softcap=0.0, sink=False, chunk=0, sinks=None) -> _Attention:
     a = _Attention()
-    a.keep_first, a.softcap, a.sink, a.chunk = keep_first, softcap, int(sink), chunk
+    a.keep_first, a.softcap, a.sink, a.chunk, a.sinks = keep_first, softcap, int(sink), chunk, _p(sinks)
     a.f32, a.q, a.ld_q, a.k_pool, a.v_pool = int(c.dtype == torch.float32), _p(q), q.stride(0), _p(c.k), _p(c.v)
     a.kv_heads, a.dim_p, a.vdim_p, a.pages, a.table, a.table_ld = c.kv_heads, c.dim, c.vdim, c.pages, _p(c.table), c.table.stride(0)
     a.heads, a.window, a.scale, a.slopes, a.gate, a.ld_gate = heads, window, scale, _p(slopes), _p(gate), gate.stride(0) if gate is not None else 0
@@ -75,8 +75,8 @@ def _args(c: PagedCache, q, out, heads, window, scale, slopes, gate, keep_first=
 
 def attention_rows(c: PagedCache, q: torch.Tensor, row_slot: torch.Tensor, row_pos: torch.Tensor, out: torch.Tensor, *, heads: int, window: int = 0,
                    scale: float, slopes: torch.Tensor | None = None, gate: torch.Tensor | None = None, max_keys: int = 0, keep_first: int = 0,
-                   softcap: float = 0.0, sink: bool = False, chunk: int = 0) -> torch.Tensor:
-    a = _args(c, q, out, heads, window, scale, slopes, gate, keep_first, softcap, sink, chunk)
+                   softcap: float = 0.0, sink: bool = False, chunk: int = 0, sinks: torch.Tensor | None = None) -> torch.Tensor:
+    a = _args(c, q, out, heads, window, scale, slopes, gate, keep_first, softcap, sink, chunk, sinks)
     a.row_slot, a.row_pos, a.rows = _p(row_slot), _p(row_pos), q.shape[0]
     a.max_keys = max_keys or chunk or (window + keep_first if window else c.table.shape[1] * PAGE)
     _lib.check(_lib.load().nfn_paged_attention_rows(C.byref(a), C.c_void_p(_lib.stream_ptr())), "paged_attention_rows")
@@ -89,9 +89,9 @@ def tile_rows(c: PagedCache, heads: int) -> int:
 
 def attention_tiles(c: PagedCache, q: torch.Tensor, tiles: torch.Tensor, out: torch.Tensor, *, heads: int, window: int = 0, scale: float,
                     slopes: torch.Tensor | None = None, gate: torch.Tensor | None = None, keep_first: int = 0, softcap: float = 0.0,
-                    sink: bool = False, chunk: int = 0) -> torch.Tensor:
+                    sink: bool = False, chunk: int = 0, sinks: torch.Tensor | None = None) -> torch.Tensor:
     """``tiles``: int32 [n, 4] = first row, rows (<= ``tile_rows``), slot, position of the first row."""
-    a = _args(c, q, out, heads, window, scale, slopes, gate, keep_first, softcap, sink, chunk)
+    a = _args(c, q, out, heads, window, scale, slopes, gate, keep_first, softcap, sink, chunk, sinks)
     a.tiles, a.n_tiles = _p(tiles), tiles.shape[0]
     _lib.check(_lib.load().nfn_paged_attention_tiles(C.byref(a), C.c_void_p(_lib.stream_ptr())), "paged_attention_tiles")
     return out

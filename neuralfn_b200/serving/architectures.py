@@ -53,6 +53,13 @@ def _build_vopozen(directory: Path, raw: Mapping[str, Any], **limits):
     return engine_config(cfg, **limits), pack_tensors(cfg, tensors)
 
 
+def _build_kidolorn(directory: Path, raw: Mapping[str, Any], **limits):
+    from ..checkpoint.safetensors_io import read_sharded_checkpoint
+    from ..models.kidolorn import KidolornConfig, engine_config, pack_tensors
+    cfg = KidolornConfig.from_dict(raw)
+    return engine_config(cfg, **limits), pack_tensors(cfg, read_sharded_checkpoint(directory))
+
+
 def _build_hf_llama(directory: Path, raw: Mapping[str, Any], *, max_batch: int = 1, max_seq: int | None = None, dtype: str = "bfloat16", **other):
     from ..checkpoint.safetensors_io import load_hf_llama_directory
     if dtype != "bfloat16":
@@ -66,6 +73,7 @@ ARCHITECTURES: dict[str, ModelArchitecture] = {a.name: a for a in (
     ModelArchitecture("Bulidra", "bulidra", "layered", ("bfloat16", "float32"), True, _build_bulidra),
     ModelArchitecture("Murilorn", "murilorn", "layered", ("bfloat16", "float32"), True, _build_murilorn),
     ModelArchitecture("Vopozen", "vopozen", "layered", ("bfloat16", "float32"), True, _build_vopozen),
+    ModelArchitecture("Kidolorn", "kidolorn", "layered", ("bfloat16", "float32"), True, _build_kidolorn),
     ModelArchitecture("LlamaForCausalLM", "llama", "all", ("bfloat16",), False, _build_hf_llama),
 )}
 

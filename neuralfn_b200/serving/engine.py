@@ -59,14 +59,16 @@ class _CLayer(C.Structure):
                 ("softcap", C.c_float), ("sink", C.c_int), ("rank_decay", C.c_int), ("rank_gate", C.c_int), ("experts", C.c_int), ("top", C.c_int),
                 ("expert_ff", C.c_int), ("weights_of", C.c_int), ("chunk", C.c_int), ("qk_norm", C.c_int), ("rot_dims", C.c_int), ("rot_base", C.c_double),
                 ("key_values", C.c_int), ("kv_rank", C.c_int), ("rot_dim", C.c_int), ("expert_plain", C.c_int), ("shared_ff", C.c_int), ("route_correction", C.c_int),
-                ("route_groups", C.c_int), ("route_keep", C.c_int), ("route_normalise", C.c_int), ("route_scale", C.c_float)]
+                ("route_groups", C.c_int), ("route_keep", C.c_int), ("route_normalise", C.c_int), ("route_scale", C.c_float),
+                ("route_softmax", C.c_int), ("expert_weigh_out", C.c_int), ("ff_limit", C.c_float), ("ff_slope", C.c_float), ("ff_bias", C.c_int), ("decay", C.POINTER(C.c_double))]
 
 
 class _CLayeredConfig(C.Structure):
     _fields_ = [("n_layer", C.c_int), ("width", C.c_int), ("vocab", C.c_int), ("side_dim", C.c_int), ("embed_scale", C.c_float),
                 ("norm_eps", C.c_float), ("dtype", C.c_int), ("max_seq", C.c_int), ("max_batch", C.c_int), ("kv_tokens", C.c_int),
                 ("max_step_rows", C.c_int), ("use_cuda_graph", C.c_int), ("chained", C.c_int), ("streams", C.c_int), ("untied_head", C.c_int),
-                ("norm_offset", C.c_float), ("logit_scale", C.c_float), ("logit_softcap", C.c_float), ("post_norm", C.c_int), ("residual_mult", C.c_float)]
+                ("norm_offset", C.c_float), ("logit_scale", C.c_float), ("logit_softcap", C.c_float), ("post_norm", C.c_int), ("residual_mult", C.c_float),
+                ("sandwich", C.c_int), ("scalar_norms", C.c_int), ("input_taps", C.c_int)]
 
 
 class _CEntry(C.Structure):
@@ -118,16 +120,23 @@ class LayerSpec:
     route_keep: int = 0
     route_normalise: int = 0
     route_scale: float = 0.0
+    route_softmax: int = 0
+    expert_weigh_out: int = 0
+    ff_limit: float = 0.0
+    ff_slope: float = 0.0
+    ff_bias: int = 0
+    decay: tuple[float, ...] = ()
 
-    FF_ACT_IDS = {"gelu": 1, "silu": 3, "relu2": 4, "relu": 6}
-    MIXER_IDS = {"attention": 0, "delta": 1, "latent": 2, "wkv": 3}
+    FF_ACT_IDS = {"gelu": 1, "silu": 3, "relu2": 4, "relu": 6, "clamped": 7}
+    MIXER_IDS = {"attention": 0, "delta": 1, "latent": 2, "wkv": 3, "linear": 4, "gru": 5}
 
     def c(self) -> _CLayer:
         return _CLayer(self.heads, self.kv_heads, self.dim, self.vdim, self.conv_taps, self.window, self.kv_from, self.scale, self.alibi,
                        self.q_temp_coef, self.q_temp_every, self.out_gate, self.ff, self.FF_ACT_IDS[self.ff_act], self.MIXER_IDS[self.mixer], self.qkv_bias, self.keep_first,
                        self.softcap, self.sink, self.rank_decay, self.rank_gate, self.experts, self.top, self.expert_ff, self.weights_of,
                        self.chunk, self.qk_norm, self.rot_dims, self.rot_base, self.key_values, self.kv_rank, self.rot_dim, self.expert_plain, self.shared_ff,
-                       self.route_correction, self.route_groups, self.route_keep, self.route_normalise, self.route_scale)
+                       self.route_correction, self.route_groups, self.route_keep, self.route_normalise, self.route_scale, self.route_softmax, self.expert_weigh_out, self.ff_limit,
+                       self.ff_slope, self.ff_bias, (C.c_double * len(self.decay))(*self.decay) if self.decay else None)
 
     @property
     def paged(self) -> bool:
@@ -171,6 +180,9 @@ class LayeredEngineConfig:
     logit_softcap: float = 0.0
     post_norm: int = 0
     residual_mult: float = 1.0
+    sandwich: int = 0
+    scalar_norms: int = 0
+    input_taps: int = 0
 
     family = 2
     kv_cache_mode = 0
@@ -199,8 +211,13 @@ class LayeredEngineConfig:
     def create(self, lib, device: int):
         cc = _CLayeredConfig(len(self.layers), self.width, self.vocab, self.side_dim, self.embed_scale, self.norm_eps,
                              int(self.dtype == "float32"), self.max_seq, self.max_batch, self.kv_tokens, self.max_step_rows, self.use_cuda_graph, self.chained,
-                             self.streams, self.untied_head, self.norm_offset, self.logit_scale, self.logit_softcap, self.post_norm, self.residual_mult)
-        arr = (_CLayer * len(self.layers))(*[y.c() for y in self.layers])
+                             self.streams, self.untied_head, self.norm_offset, self.logit_scale, self.logit_softcap, self.post_norm, self.residual_mult,
+                             self.sandwich, self.scalar_norms, self.input_taps)
+        for i, y in enumerate(self.layers):
+            if y.mixer == "linear" and len(y.decay) != y.heads:
+                raise ValueError(f"layer {i}: {len(y.decay)} decays for {y.heads} heads")
+        specs = [y.c() for y in self.layers]
+        arr = (_CLayer * len(specs))(*specs)
         return lib.nfn_engine_create_layered(C.byref(cc), arr, device)
 
     def estimate_device_bytes(self) -> int:
@@ -225,20 +242,29 @@ class LayeredEngineConfig:
                 widest = max(widest, n_in + 5 * wp + v + (4 // es) * (2 * q + up(y.rank_decay)) + 2 * up(y.rank_decay))
             elif y.mixer == "latent":
                 rank, rot = up(y.kv_rank), up(y.rot_dim)
-                n_in, own = y.heads * (dim + rot) + (0 if y.kv_from >= 0 else rank + rot), y.heads * rank * (2 * dim + vdim)
+                n_in, own = y.heads * (dim + rot) + (0 if y.kv_from >= 0 else rank + rot) + (v if y.out_gate else 0), y.heads * rank * (2 * dim + vdim)
                 cache += 0 if y.kv_from >= 0 else (rank + rot) * pool * es
                 short = rows if es == 4 else min(rows, 15 * self.max_batch)                # rows that attend to the latents, rows of the expansion
                 cache += short * y.heads * (2 * rank + rot) * es + (0 if es == 4 else (rows + min(y.look or self.max_seq, self.max_seq) + 2 * KV_PAGE) * (rank + y.heads * (dim + vdim)) * es)
+                widest = max(widest, n_in + v)
+            elif y.mixer == "linear":
+                n_in, own = 2 * (q + v), 0
+                cache += 4 * q * vdim * self.max_batch + (0 if es == 4 or dim > 128 else min(y.heads * self.max_batch, 160) * 9 * 4 * dim * vdim // sum(z.mixer == "linear" for z in self.layers))
+                widest = max(widest, n_in + v + (4 // es) * v)
+            elif y.mixer == "gru":
+                n_in, own = 3 * v, 0
+                cache += 4 * v * self.max_batch
                 widest = max(widest, n_in + v)
             else:
                 kv = 0 if y.kv_from >= 0 else y.kv_heads * (dim + vdim)
                 n_in, own = q + kv + (v if y.out_gate else 0) + (0 if self.chained else 2 * up(y.ff)), 0
                 cache += kv * pool * es
                 widest = max(widest, n_in + q + v + up(y.ff))
+            cache += 2 * 2 * self.max_batch * max(self.input_taps - 1, 0) * wp * es
             if y.weights_of < 0:
                 weights += wp * (n_in + v + up(y.ff) * (3 if self.chained else 1) + 2 * up(self.side_dim) + 2 * up(y.shared_ff)) + own + wp * (up(y.experts) + 3 * y.experts * up(y.expert_ff))
             routed = max(routed, (rows * y.top + 127 * y.experts) * es * (2 * wp + 3 * up(y.expert_ff)) if y.experts else 0)
-        acts = rows * (es * (3 * wp + widest + up(self.side_dim)) + 4 * (wp * max(self.streams, 1) + up(self.side_dim))) + 4 * 2 * max(self.max_batch, 64) * up(self.vocab)
+        acts = rows * (es * ((4 if self.input_taps else 3) * wp + widest + up(self.side_dim)) + 4 * (wp * max(self.streams, 1) + up(self.side_dim))) + 4 * 2 * max(self.max_batch, 64) * up(self.vocab)
         chunks = (96 << 20) * sum(any(y.mixer == m for y in self.layers) for m in ("delta", "wkv")) if es == 2 else 0        # operands of the recurrences' prompt chunks
         return int(2 * weights + cache + acts + routed + chunks)
 

@@ -22,10 +22,10 @@ def test_registry_resolution_and_proofs():
     with pytest.raises(ValueError):
         q.require("native_training")
     assert capability_proof_for("jamba").route == "tensor-runtime"
-    assert len(native_families_report()) == len(NATIVE_FAMILIES) == 19
+    assert len(native_families_report()) == len(NATIVE_FAMILIES) == 20
     trained = [s for s in NATIVE_FAMILIES.values() if s.route != "serving-only"]
     assert len(trained) == 16 and all(s.reference_binary.startswith("nfn_") and s.reference_binary.endswith("_native_train") for s in trained)
-    for name in ("bulidra", "murilorn", "vopozen"):
+    for name in ("bulidra", "murilorn", "vopozen", "kidolorn"):
         b = capability_proof_for(name)
         assert b.native_inference and not b.native_training and b.route == "serving-only" and len(b.reasons) == 1
 
