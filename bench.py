@@ -214,8 +214,8 @@ def main() -> None:
     ap.add_argument("--no-graph", action="store_true")
     ap.add_argument("--check-fused", action="store_true",
                     help="run the fused-collective kernel self-check also on one GPU (always on for N > 1)")
-    ap.add_argument("--serving", choices=["bulidra", "murilorn", "vopozen"], default=None,
-                    help="instead of the training benchmark: prefill and decode throughput of this design and of Glimmer blocks of equal size")
+    ap.add_argument("--serving", choices=["bulidra", "murilorn", "vopozen", "kidolorn"], default=None,
+                    help="instead of the training benchmark: prefill and decode throughput of this design and of the closest other model at equal size")
     args = ap.parse_args()
     if args.serving:
         from neuralfn_b200.bench.serving_bench import run as run_serving

@@ -563,7 +563,95 @@ def case_mixers(args):
     rep("expert_rows (gated)", lambda: Y.expert_rows(y1, z1, wg, down, experts=E, top=4), bytes_=6.0 * live * F * C, extra={"B": B, "experts_used": live})
 
 
-CASES = {"gemm": case_gemm, "paged": case_paged, "layered": case_layered, "mixers": case_mixers, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
+def case_recurrences(args):
+    """Linear attention with a decay per head, the gated recurrence, input convolutions, learned sinks, gates and clamped experts beside the like kernels of the other
+    designs, at one layer of ``--heads`` x ``--head-dim`` (the gated recurrence as wide as all heads together), width ``--k``, ``--experts`` experts of which four of
+    ``--n`` / 4 are used, latents of 512 + 64 channels over all earlier tokens."""
+    from neuralfn_b200.ops import layered as Y, paged as P
+    dev = torch.device("cuda")
+    H, D, T, B, C, E = args.heads, args.head_dim, args.seq, args.batch, args.k, args.experts
+    F, R, RANK, HD = args.n // 4, 64, 512, args.heads * args.head_dim
+    rand = lambda *s: torch.randn(*s, device=dev).bfloat16()  # noqa: E731
+    i32 = dict(dtype=torch.int32, device=dev)
+    rep = lambda name, fn, **kw: _report(name, time_kernel(fn, args.iters, args.warmup, args.flush), args=args, **kw)  # noqa: E731
+    one, pw = torch.tensor([[0, T, 0, 0]], **i32), Y.powers([1 - 2.0 ** (-1 - 9 * h / H) for h in range(H)], dev)
+    rt, st = P.row_tiles([(0, 0, T, 0)], dev), P.row_tiles([(b, 7, 1, 0) for b in range(B)], dev)
+
+    # ---- recurrences: prompts, then single tokens ----
+    qkvg, state = rand(T, 4 * HD) * 0.1, torch.zeros(1, H, D, D, device=dev)
+    lw = torch.empty(1, device=dev, dtype=torch.uint8)
+    rep("linear_chunks", lambda: Y.linear_rule(qkvg, pw, state, one, form="chunks"), bytes_=10.0 * T * HD, extra={"T": T, "heads": H, "dim": D})
+    rep("linear_chunks (no segments)", lambda: Y.linear_rule(qkvg, pw, state, one, form="chunks", workspace=lw), bytes_=10.0 * T * HD, extra={"T": T})
+    u, w0, wn = rand(HD), torch.full((HD,), -1.0, device=dev).bfloat16(), rand(HD)
+    z, wsp = torch.randn(T, HD, device=dev), torch.empty(96 << 20, device=dev, dtype=torch.uint8)
+    rep("wkv_chunks", lambda: Y.wkv_rule(qkvg, z, w0, u, state, one, dim=D, form="chunks", workspace=wsp), bytes_=14.0 * T * HD, extra={"T": T})
+    o, gate, out = torch.randn(T, HD, device=dev), rand(T, HD), torch.empty(T, HD, device=dev, dtype=torch.bfloat16)
+    rep("row_out", lambda: Y.row_out(o, gate, wn, live=HD, eps=1e-5), bytes_=8.0 * T * HD, extra={"T": T})
+    rep("delta_out (norm per head)", lambda: Y.delta_out(o, gate, wn[:D], heads=H, vdim=D, eps=1e-5), bytes_=8.0 * T * HD, extra={"T": T})
+    gx, gs = rand(T, 3 * HD), torch.zeros(B, HD, device=dev)
+    rep("gru_rows", lambda: Y.gru_rows(gx, gs, out, one, 0), bytes_=8.0 * T * HD, extra={"T": T, "width": HD})
+    mb = min(8, B)
+    parts = torch.tensor([[b * (T // mb), T // mb, b, 0] for b in range(mb)], **i32)
+    rep("gru_rows (several prompts)", lambda: Y.gru_rows(gx, gs, out, parts, 0), bytes_=8.0 * T * HD, extra={"T": T // mb, "prompts": mb})
+    for b in sorted({1, min(8, B), B}):
+        states, so, cnt = torch.zeros(b, H, D, D, device=dev), torch.empty(b, HD, device=dev, dtype=torch.bfloat16), torch.zeros(b, **i32)
+        low, w2 = torch.randn(b, 64, device=dev), rand(HD, 128) * 0.1
+        rep("linear_step", lambda: Y.linear_step(qkvg[:b], pw, states, wn, so, st[:b], cnt, vdim=D, eps=1e-5), bytes_=8.0 * b * HD * D, extra={"B": b})
+        rep("wkv_step", lambda: Y.wkv_step(qkvg[:b], low, w2, w0, u, states, wn, so, st[:b], dim=D, eps=1e-5), bytes_=8.0 * b * HD * D, extra={"B": b})
+        seqs = torch.tensor([[i, 1, i, 7] for i in range(b)], **i32)
+        rep("gru_rows (single tokens)", lambda: Y.gru_rows(gx[:b], gs, so, seqs, b), bytes_=16.0 * b * HD, extra={"B": b})
+    # ---- residual and convolution on the way into a sublayer ----
+    xs, y, h, hc, wt, g1 = torch.randn(T, C, device=dev), rand(T, C), torch.empty(T, C, device=dev, dtype=torch.bfloat16), torch.empty(T, C, device=dev, dtype=torch.bfloat16), rand(C), rand(1)
+    conv, hist = rand(4, C), torch.zeros(2, B, 3, C, device=dev, dtype=torch.bfloat16)
+    kw = dict(width=C, streams=1, ld=C, f32=False)
+    rep("stream_pass (norms on both sides, one factor)", lambda: Y.stream_pass(xs, h, rows=T, x_out=xs, y=y, y_weight=g1, weight=g1, scalar_norms=True, **kw), bytes_=12.0 * T * C, extra={"T": T})
+    rep("stream_pass (norm on the update)", lambda: Y.stream_pass(xs, h, rows=T, x_out=xs, y=y, y_weight=wt, **kw), bytes_=12.0 * T * C, extra={"T": T})
+    rep("input_conv", lambda: Y.input_conv(h, conv, hist, hc, rt), bytes_=4.0 * T * C, extra={"T": T, "width": C})
+    mu, prev, sh = rand(5, C), torch.zeros(2, 1, C, device=dev), torch.empty(5, T, C, device=dev, dtype=torch.bfloat16)
+    rep("shift_rows", lambda: Y.shift_rows(xs, mu, prev, sh, rt), bytes_=14.0 * T * C, extra={"T": T, "width": C})
+    del sh
+    rep("stream_pass (with the convolution, single tokens)", lambda: Y.stream_pass(xs, h, rows=B, x_out=xs, y=y, y_weight=g1, weight=g1, scalar_norms=True, conv=conv, history=hist, tiles=st, **kw),
+        bytes_=(12.0 + 12.0) * B * C, extra={"B": B})
+    rep("stream_pass (single tokens)", lambda: Y.stream_pass(xs, h, rows=B, x_out=xs, y=y, y_weight=wt, **kw), bytes_=12.0 * B * C, extra={"B": B})
+    # ---- latent attention: sinks, gate ----
+    lc = Y.LatentCache(1, T, RANK, R, dev)
+    lc.k.normal_()
+    sinks, ql, x, base = rand(H), rand(T, H * (D + R)), rand(T, 2 * HD), torch.zeros(1, **i32)
+    tiles = torch.tensor([[r, min(128, T - r), 0, r] for r in range(0, T, 128)], **i32)
+    flops = 2.0 * H * (2 * D + R) * T * (T + 1) / 2
+    la = dict(heads=H, dim=D, vdim=D, window=0, scale=(D + R) ** -0.5)
+    rep("latent_attention_tiles (sinks, gate)", lambda: Y.latent_attention_tiles(lc, ql, x, base, tiles, out, sinks=sinks, gate=gate, **la), flops=flops, extra={"T": T})
+    rep("latent_attention_tiles", lambda: Y.latent_attention_tiles(lc, ql, x, base, tiles, out, **la), flops=flops, extra={"T": T})
+    del lc, x, ql
+    keys = args.context
+    lc = Y.LatentCache(B, keys, RANK, R, dev)
+    lc.k.normal_()
+    slot, pos = torch.arange(B, **i32), torch.full((B,), keys - 1, **i32)
+    qa, oa = rand(B, H * (RANK + R)), torch.empty(B, H * RANK, device=dev, dtype=torch.bfloat16)
+    for b in sorted({1, min(8, B), B}):
+        lr = dict(heads=H, window=0, scale=(D + R) ** -0.5, max_keys=keys)
+        rep("latent_attention_rows (sinks)", lambda: Y.latent_attention_rows(lc, qa[:b], slot[:b], pos[:b], oa[:b], sinks=sinks, **lr), bytes_=2.0 * b * keys * (RANK + R), extra={"B": b, "keys": keys})
+        rep("latent_attention_rows", lambda: Y.latent_attention_rows(lc, qa[:b], slot[:b], pos[:b], oa[:b], **lr), bytes_=2.0 * b * keys * (RANK + R), extra={"B": b, "keys": keys})
+    wuv, ov, gb = rand(H, D, RANK), torch.empty(B, H, D, device=dev, dtype=torch.bfloat16), rand(B, H, D)
+    rep("group_products (values, gate)", lambda: Y.group_products(oa.view(B, H, RANK), wuv, ov, gate=gb), bytes_=2.0 * (HD * RANK + B * H * (RANK + 2 * D)), extra={"B": B})
+    rep("group_products (values)", lambda: Y.group_products(oa.view(B, H, RANK), wuv, ov), bytes_=2.0 * (HD * RANK + B * H * (RANK + D)), extra={"B": B})
+    # ---- feed-forward ----
+    gu, mid, cl = rand(T, 8 * F), torch.empty(T, 4 * F, device=dev, dtype=torch.bfloat16), (7.0, 1.702, 1.0)
+    rep("ff_rows (clamped)", lambda: Y.ff_rows(gu, mid, off_gate=0, off_up=4 * F, act=7, clamp=cl), bytes_=24.0 * T * F, extra={"T": T, "ff": 4 * F})
+    rep("ff_rows", lambda: Y.ff_rows(gu, mid, off_gate=0, off_up=4 * F, act=3), bytes_=24.0 * T * F, extra={"T": T, "ff": 4 * F})
+    del gu, mid
+    zt = torch.randn(T, E, device=dev)
+    rep("expert_choice (softmax)", lambda: Y.expert_choice(zt, 4, softmax=True), bytes_=4.0 * T * E + 32.0 * T, extra={"T": T})
+    rep("expert_choice (no groups)", lambda: Y.expert_choice(zt, 4), bytes_=4.0 * T * E + 32.0 * T, extra={"T": T})
+    wg, down = rand(E, 2 * F, C) * C ** -0.5, rand(E, C, F) * F ** -0.5
+    y1, z1 = rand(B, C), torch.randn(B, E, device=dev)
+    ex = dict(experts=E, top=4)
+    live = int(Y.expert_rows(y1, z1, wg, down, **ex)[0].unique().numel())
+    rep("expert_rows (clamped, softmax)", lambda: Y.expert_rows(y1, z1, wg, down, act=7, clamp=cl, weigh_output=True, softmax=True, **ex), bytes_=6.0 * live * F * C, extra={"B": B, "experts_used": live})
+    rep("expert_rows (gated)", lambda: Y.expert_rows(y1, z1, wg, down, **ex), bytes_=6.0 * live * F * C, extra={"B": B, "experts_used": live})
+
+
+CASES = {"gemm": case_gemm, "paged": case_paged, "layered": case_layered, "mixers": case_mixers, "recurrences": case_recurrences, "attention_fwd": case_attention, "attention_bwd": lambda a: case_attention(a, True),
          "cross_entropy": case_cross_entropy, "norm": case_norm, "adamw": case_adamw, "decode_attention": case_decode_attention,
          "skinny": case_skinny, "grouped_k": case_grouped_k, "kquant_gemv": case_kquant_gemv, "gemm_kquant": case_gemm_kquant, "block_attention": case_block_attention,
          "turboquant_attention": case_turboquant_attention, "engine_decode": case_engine_decode}

@@ -1,10 +1,12 @@
 """Prefill and decode throughput of Bulidra, Murilorn or Vopozen and, at equal size, of Glimmer blocks - the closest model the engine served before:
-grouped heads, sliding windows, gated attention, gated feed-forward. Random bf16 weights; one JSON line per model, size and phase.
+grouped heads, sliding windows, gated attention, gated feed-forward; of Kidolorn beside Vopozen. Random bf16 weights; one JSON line per model, size and
+phase.
 
 Murilorn at equal size: delta-rule and attention layers in turn with the same heads, the same active feed-forward width (four of thirty-two
 experts), four residual streams. Vopozen at equal size: chunked attention, latent attention, time mixing and latent attention on the earlier layer's
 cache in turn, the same heads, gated and routed feed-forwards in turn with the same active weights (four of thirty-two plain experts and a shared
-one).
+one). Kidolorn at equal size: linear attention, latent attention, the gated recurrence (as wide as all heads together) and latent attention on the
+earlier layer's cache in turn, without windows; dense and routed feed-forwards in turn (four of thirty-two gated experts).
 
 ``ms`` is device time (CUDA events on the engine's stream, median over repetitions of the public ``prefill`` / ``decode`` call,
 including its host-to-device copy of tokens and the read-back of the drawn token); weights and caches are larger than L2. Beside it
@@ -27,6 +29,8 @@ SIDE_DIM = 256
 EXPERTS, TOP, STREAMS, RANK, KEEP = 32, 4, 4, 128, 4
 LATENT, ROT, DECAY = 512, 64, 64
 VOPOZEN = ("attention", "latent", "wkv", "reader")
+KIDOLORN = ("lightning", "latent", "mingru", "reader")
+BESIDE = {"kidolorn": "vopozen"}                    # the closest model; others: Glimmer blocks
 
 
 def _peaks() -> tuple[float, float]:
@@ -39,7 +43,7 @@ def _peaks() -> tuple[float, float]:
 
 def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
     from ..models.bulidra import BulidraConfig, BulidraLayer, engine_config
-    from ..models import murilorn as M, vopozen as V
+    from ..models import kidolorn as Q, murilorn as M, vopozen as V
     from ..serving import EngineConfig, ResidentEngine
     L = z["layers"]
     if kind == "murilorn":
@@ -50,6 +54,8 @@ def _engine(kind: str, z: dict, max_batch: int, max_seq: int):
                               max_step_rows=max_seq)
     elif kind == "vopozen":
         cfg = V.engine_config(V.VopozenConfig(z["vocab"], z["width"], 1e-5, 0.5, tuple(_vopozen_layers(z))), max_batch=max_batch, max_seq=max_seq, max_step_rows=max_seq)
+    elif kind == "kidolorn":
+        cfg = Q.engine_config(Q.KidolornConfig(z["vocab"], z["width"], 1e-5, 4, tuple(_kidolorn_layers(z))), max_batch=max_batch, max_seq=max_seq, max_step_rows=max_seq)
     elif kind == "bulidra":
         layers = tuple(BulidraLayer(z["heads"], z["kv_heads"], z["dim"], z["dim"], 4, z["dim"] ** -0.5, z["window"], 0.1, 1024, None, z["ff"]) for _ in range(L))
         cfg = engine_config(BulidraConfig(z["vocab"], z["width"], 1.0, 1e-5, SIDE_DIM, layers), max_batch=max_batch, max_seq=max_seq, max_step_rows=max_seq)
@@ -91,6 +97,21 @@ def _vopozen_layers(z: dict) -> list:
     return out
 
 
+def _kidolorn_layers(z: dict) -> list:
+    from ..models import kidolorn as Q
+    out: list = []
+    for i in range(z["layers"]):
+        kind, H, d = KIDOLORN[i % 4], z["heads"], z["dim"]
+        f = dict(ff=z["ff"], limit=7.0) if i % 2 == 0 else dict(experts=EXPERTS, top=TOP, expert_ff=z["ff"] // TOP, limit=7.0)
+        if kind == "lightning":
+            out.append(Q.KidolornLayer("lightning", H, d, d, decay=tuple(1 - 2.0 ** (-1 - 9 * h / H) for h in range(H)), **f))
+        elif kind == "mingru":
+            out.append(Q.KidolornLayer("mingru", vdim=H * d, **f))
+        else:
+            out.append(Q.KidolornLayer("latent_attention", H, d, d, scale=d ** -0.5, rot_dim=ROT, kv_rank=LATENT, kv_from=i - 2 if kind == "reader" else -1, **f))
+    return out
+
+
 def _time(eng, fn, n: int, warmup: int) -> float:
     for _ in range(warmup):
         fn()
@@ -111,6 +132,8 @@ def _work(z: dict, kind: str, prompt: int, batch: int, context: int) -> tuple[fl
         return _murilorn_work(z, prompt, batch, context)
     if kind == "vopozen":
         return _vopozen_work(z, prompt, batch, context)
+    if kind == "kidolorn":
+        return _kidolorn_work(z, prompt, batch, context)
     per = w * (q + 2 * kv + q + 2 * z["ff"]) + w * (q + z["ff"]) + (2 * w * SIDE_DIM if kind == "bulidra" else 0)
     win = min(z["window"], prompt)
     keys = win * (win + 1) / 2 + (prompt - win) * win
@@ -162,11 +185,34 @@ def _vopozen_work(z: dict, prompt: int, batch: int, context: int) -> tuple[float
     return flops, byts
 
 
+def _kidolorn_work(z: dict, prompt: int, batch: int, context: int) -> tuple[float, float]:
+    w, q = z["width"], z["heads"] * z["dim"]
+    chosen = EXPERTS * (1 - (1 - TOP / EXPERTS) ** batch)       # experts a batch of uniform choices touches
+    flops, byts = 0.0, 2.0 * z["vocab"] * w
+    for y in _kidolorn_layers(z):
+        if y.type == "lightning":
+            per = 5 * w * q
+            flops += 5.0 * q * z["dim"] * prompt
+            byts += batch * 8.0 * q * z["dim"]
+        elif y.type == "mingru":
+            per = 4 * w * q
+            byts += batch * 8.0 * q
+        else:
+            row = LATENT + ROT
+            per = w * (z["heads"] * (z["dim"] + ROT) + (row if y.kv_from < 0 else 0)) + 2 * q * LATENT + 2 * q * w
+            flops += 2.0 * z["heads"] * (2 * z["dim"] + ROT) * prompt * (prompt + 1) / 2
+            byts += 2.0 * batch * context * row
+        act, read = (3 * w * y.ff,) * 2 if y.ff else (w * (3 * TOP * y.expert_ff + EXPERTS), w * (3 * chosen * y.expert_ff + EXPERTS))
+        flops += 2.0 * (per + act) * prompt
+        byts += 2.0 * (per + read)
+    return flops, byts
+
+
 def run(args, clock_sampler, sizes=None) -> None:
     hbm, tf = _peaks()
     for name in sizes or SIZES:
         z = SIZES[name]
-        for kind in ("glimmer", args.serving):
+        for kind in (BESIDE.get(args.serving, "glimmer"), args.serving):
             prompt, context = 8192, 4096
             eng = _engine(kind, z, 1, prompt + 64)
             g = torch.Generator().manual_seed(1)

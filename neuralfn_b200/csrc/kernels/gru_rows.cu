@@ -2,8 +2,11 @@
 // formed from b. Everything but the loads and stores is fp32.
 //
 // Short entries (single tokens, portions of a few rows) go token after token. Long ones are an affine scan: a CTA takes 32 channels, 16 lanes with two
-// channels each, and 256 rows at a time in 32 segments of eight; every segment's rows become one factor and one addend, the state in front
+// channels each, and 256 rows at a time in 32 segments of eight; every segment's rows become one step of the same form, the state in front
 // of a segment follows from those of the segments before it, and the rows are run again from there, out of registers.
+//
+// A step is taken as s <- s + z (c - s). Where z is small a state lasts for thousands of tokens, and a factor 1 - z that is rounded on its own would leave
+// each time a little less or more than the share z took.
 #include <type_traits>
 
 #include "common.h"
@@ -11,23 +14,13 @@
 
 namespace nfn {
 
-// what a token does to a channel: s <- keep * s + add
-struct GruStep { float keep, add; };
+// what a token does to a channel: s <- s + z (c - s)
+struct GruStep { float z, c; };
 template <typename T>
 __device__ __forceinline__ GruStep gru_step(float a, float b) {
-  float keep, z;
-  if constexpr (sizeof(T) == 4) {
-    const float e = expf(fminf(-a, 80.f));
-    z = 1.f / (1.f + e);
-    keep = e * z;                                           // 1 - z without its cancellation
-  } else {
-    const float e = fast_exp2(fminf(a * -1.4426950408889634f, 100.f));
-    z = fast_rcp(1.f + e);
-    keep = e * z;
-  }
-  const float c = b >= 0.f ? b + 0.5f : sigmoid_for<T>(b);
-  return GruStep{keep, z * c};
+  return GruStep{sigmoid_for<T>(a), b >= 0.f ? b + 0.5f : sigmoid_for<T>(b)};
 }
+__device__ __forceinline__ float gru_take(float s, float z, float c) { return s + z * (c - s); }
 template <typename T>
 __device__ __forceinline__ float gru_out(float s, float g) { return s * g * sigmoid_for<T>(g); }
 
@@ -53,7 +46,7 @@ gru_short_kernel(const nfn_gru_args p) {
     const float2 a = gru_unpack(*reinterpret_cast<const GruPair<T>*>(x)), b = gru_unpack(*reinterpret_cast<const GruPair<T>*>(x + p.width)),
                  g = gru_unpack(*reinterpret_cast<const GruPair<T>*>(x + 2 * p.width));
     const GruStep u = gru_step<T>(a.x, b.x), v = gru_step<T>(a.y, b.y);
-    s = make_float2(u.keep * s.x + u.add, v.keep * s.y + v.add);
+    s = make_float2(gru_take(s.x, u.z, u.c), gru_take(s.y, v.z, v.c));
     gru_store(static_cast<T*>(p.out) + (size_t)(seq.row0 + t) * p.ld_out + c, gru_out<T>(s.x, g.x), gru_out<T>(s.y, g.y));
   }
   *st = s;
@@ -64,7 +57,7 @@ template <typename T>
 __global__ void __launch_bounds__(GS_THREADS, 1)
 gru_scan_kernel(const nfn_gru_args p) {
   constexpr bool AHEAD = sizeof(T) == 2;                    // the next rows are on their way while these are used
-  __shared__ float4 segs[2][GS_SEGS][GS_LANES];             // factor and addend of both channels
+  __shared__ float4 segs[2][GS_SEGS][GS_LANES];             // of both channels: share of the state before it that goes, what comes in its place
   const nfn_seq_rows seq = p.seqs[p.n_short + blockIdx.y];
   if (seq.slot < 0) return;
   const int lane = threadIdx.x % GS_LANES, seg = threadIdx.x / GS_LANES, c = blockIdx.x * 2 * GS_LANES + 2 * lane;
@@ -92,16 +85,16 @@ gru_scan_kernel(const nfn_gru_args p) {
   for (int r0 = 0; r0 < seq.n; r0 += GS_SPAN, buf ^= 1) {
     if constexpr (AHEAD) fetch(r0 + GS_SPAN, na, nb, ng);
     const int live = on ? min(GS_ROWS, seq.n - r0 - seg * GS_ROWS) : 0;
-    float2 keep[GS_ROWS], add[GS_ROWS];
-    float4 f = make_float4(1.f, 0.f, 1.f, 0.f);
+    float2 z[GS_ROWS], cand[GS_ROWS];
+    float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < GS_ROWS; ++i)
       if (i < live) {
         const float2 x = gru_unpack(a[i]), y = gru_unpack(b[i]);
         const GruStep u = gru_step<T>(x.x, y.x), v = gru_step<T>(x.y, y.y);
-        keep[i] = make_float2(u.keep, v.keep);
-        add[i] = make_float2(u.add, v.add);
-        f = make_float4(f.x * u.keep, f.y * u.keep + u.add, f.z * v.keep, f.w * v.keep + v.add);
+        z[i] = make_float2(u.z, v.z);
+        cand[i] = make_float2(u.c, v.c);
+        f = make_float4(gru_take(f.x, u.z, 1.f), gru_take(f.y, u.z, u.c), gru_take(f.z, v.z, 1.f), gru_take(f.w, v.z, v.c));
       }
     segs[buf][seg][lane] = f;
     __syncthreads();                                        // the other buffer was read before the last one of these
@@ -110,12 +103,12 @@ gru_scan_kernel(const nfn_gru_args p) {
     for (int q = 0; q < GS_SEGS; ++q) {
       if (q == seg) mine = s;
       const float4 e = segs[buf][q][lane];
-      s = make_float2(s.x * e.x + e.y, s.y * e.z + e.w);
+      s = make_float2(s.x + (e.y - e.x * s.x), s.y + (e.w - e.z * s.y));
     }
 #pragma unroll
     for (int i = 0; i < GS_ROWS; ++i)
       if (i < live) {
-        mine = make_float2(keep[i].x * mine.x + add[i].x, keep[i].y * mine.y + add[i].y);
+        mine = make_float2(gru_take(mine.x, z[i].x, cand[i].x), gru_take(mine.y, z[i].y, cand[i].y));
         const float2 h = gru_unpack(g[i]);
         gru_store(out + (size_t)(r0 + seg * GS_ROWS + i) * p.ld_out, gru_out<T>(mine.x, h.x), gru_out<T>(mine.y, h.y));
       }

@@ -1,5 +1,5 @@
 """ctypes bindings of the layer-list engine's other kernels on torch tensors: residual streams (csrc/kernels/stream_rows.cu), the gated
-delta rule (delta_*.cu), the bonus recurrence (wkv_*.cu), rotated heads and latent attention (head_rows.cu, latent_decode.cu,
+delta rule (delta_*.cu), the bonus recurrence (wkv_*.cu), linear attention (linear_*.cu), the gated recurrence (gru_rows.cu), rotated heads and latent attention (head_rows.cu, latent_decode.cu,
 paged_prefill.cu) and routed experts (moe.cu, moe_rows.cu, the grouped GEMM). The engine calls them from C++; these wrappers serve kernel
 tests and timing."""
 from __future__ import annotations
@@ -11,8 +11,8 @@ import torch
 from . import _lib
 from .paged import PAGE, PagedCache, _Attention
 
-__all__ = ["LatentCache", "delta_out", "delta_rule", "expert_choice", "expert_rows", "ff_rows", "frequencies", "group_products", "head_rows", "latent_attention_rows",
-           "latent_attention_tiles", "latent_gather", "latent_rows", "logit_cap", "shift_rows", "stream_pass", "wkv_rule", "wkv_step"]
+__all__ = ["LatentCache", "delta_out", "delta_rule", "expert_choice", "expert_rows", "ff_rows", "frequencies", "group_products", "gru_rows", "head_rows", "input_conv",
+           "latent_attention_rows", "latent_attention_tiles", "latent_gather", "latent_rows", "linear_rule", "linear_step", "logit_cap", "row_out", "shift_rows", "stream_pass", "wkv_rule", "wkv_step"]
 
 
 class _Stream(C.Structure):
@@ -300,4 +300,82 @@ class _Clamp(C.Structure):
 def ff_rows(x: torch.Tensor, out: torch.Tensor, *, off_gate: int, off_up: int, act: int, clamp: tuple[float, float, float] = (0.0, 0.0, 0.0)) -> torch.Tensor:
     _lib.check(_lib.load().nfn_ff_rows(C.c_int(int(x.dtype == torch.float32)), C.c_void_p(_p(x)), C.c_int(x.stride(0)), C.c_int(off_gate), C.c_int(off_up), C.c_int(out.shape[1]),
                                        C.c_int(act), C.byref(_Clamp(*clamp)), C.c_void_p(_p(out)), C.c_int(out.stride(0)), C.c_int(x.shape[0]), C.c_void_p(_lib.stream_ptr())), "ff_rows")
+    return out
+
+
+# ---- linear attention, gated recurrence, convolutions on a sublayer's input ------------------------------------------------------
+class _Linear(C.Structure):
+    _fields_ = [("f32", C.c_int), ("qkv", C.c_void_p), ("ld_qkv", C.c_int), ("powers", C.c_void_p), ("heads", C.c_int), ("dim_p", C.c_int), ("vdim_p", C.c_int), ("state", C.c_void_p),
+                ("o", C.c_void_p), ("ld_o", C.c_int), ("seqs", C.c_void_p), ("n_seqs", C.c_int)]
+
+
+class _LinearStep(C.Structure):
+    _fields_ = [("f32", C.c_int), ("rows", C.c_int), ("qkvg", C.c_void_p), ("ld_qkvg", C.c_int), ("powers", C.c_void_p), ("heads", C.c_int), ("vdim", C.c_int), ("dim_p", C.c_int),
+                ("vdim_p", C.c_int), ("state", C.c_void_p), ("o", C.c_void_p), ("ld_o", C.c_int), ("counters", C.c_void_p), ("weight", C.c_void_p), ("eps", C.c_float), ("out", C.c_void_p),
+                ("ld_out", C.c_int), ("tiles", C.c_void_p)]
+
+
+class _Gru(C.Structure):
+    _fields_ = [("f32", C.c_int), ("width", C.c_int), ("in_", C.c_void_p), ("ld_in", C.c_int), ("state", C.c_void_p), ("out", C.c_void_p), ("ld_out", C.c_int), ("seqs", C.c_void_p),
+                ("n_seqs", C.c_int), ("n_short", C.c_int)]
+
+
+class _InputConv(C.Structure):
+    _fields_ = [("f32", C.c_int), ("ld", C.c_int), ("taps", C.c_int), ("h", C.c_void_p), ("conv", C.c_void_p), ("history", C.c_void_p), ("history_half", C.c_longlong), ("out", C.c_void_p),
+                ("tiles", C.c_void_p), ("n_tiles", C.c_int)]
+
+
+LINEAR_CHUNK = 64
+
+
+def powers(decay, device) -> torch.Tensor:
+    """decay_h^0 .. decay_h^LINEAR_CHUNK, fp32 [heads, LINEAR_CHUNK + 1]."""
+    d = torch.tensor(list(decay), dtype=torch.float64)[:, None]
+    return (d ** torch.arange(LINEAR_CHUNK + 1, dtype=torch.float64)).float().contiguous().to(device)
+
+
+def linear_rule(qkv: torch.Tensor, pw: torch.Tensor, state: torch.Tensor, seqs: torch.Tensor, *, form: str = "rows", workspace: torch.Tensor | None = None, longest: int = 0) -> torch.Tensor:
+    """qkv [rows, heads * (2 dim_p + vdim_p)] after its activation, state fp32 [slots, heads, dim_p, vdim_p], seqs int32 [n, 4] = first row, rows, slot, position. Returns
+    the read-outs, fp32 [rows, heads * vdim_p]. form: "rows" or "chunks" (without a workspace of its own: segments side by side where they pay)."""
+    _, heads, dim_p, vdim_p = state.shape
+    o = torch.zeros(qkv.shape[0], heads * vdim_p, device=qkv.device)
+    a = _Linear(int(qkv.dtype == torch.float32), _p(qkv), qkv.stride(0), _p(pw), heads, dim_p, vdim_p, _p(state), _p(o), o.stride(0), _p(seqs), seqs.shape[0])
+    if form == "rows":
+        _call("linear_rows", a)
+        return o
+    lib = _lib.load()
+    lib.nfn_linear_chunk_workspace_bytes.restype = C.c_longlong
+    ws = workspace if workspace is not None else torch.empty(lib.nfn_linear_chunk_workspace_bytes(heads, dim_p, vdim_p, seqs.shape[0]), device=qkv.device, dtype=torch.uint8)
+    _lib.check(lib.nfn_linear_chunks(C.byref(a), C.c_int(longest or qkv.shape[0]), C.c_void_p(_p(ws)), C.c_longlong(ws.numel()), C.c_void_p(_lib.stream_ptr())), "linear_chunks")
+    return o
+
+
+def linear_step(qkvg: torch.Tensor, pw: torch.Tensor, state: torch.Tensor, weight: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor, counters: torch.Tensor, *, vdim: int, eps: float) -> torch.Tensor:
+    """One token per row: qkvg [rows, heads * (2 dim_p + 2 vdim_p)] before its activations; counters int32 [rows], zero (and zero again afterwards)."""
+    _, heads, dim_p, vdim_p = state.shape
+    o = torch.zeros(qkvg.shape[0], heads * vdim_p, device=qkvg.device)
+    a = _LinearStep(int(qkvg.dtype == torch.float32), qkvg.shape[0], _p(qkvg), qkvg.stride(0), _p(pw), heads, vdim, dim_p, vdim_p, _p(state), _p(o), o.stride(0), _p(counters), _p(weight), eps,
+                    _p(out), out.stride(0), _p(tiles))
+    _call("linear_step", a)
+    return out
+
+
+def row_out(o: torch.Tensor, gate: torch.Tensor, weight: torch.Tensor, *, live: int, eps: float) -> torch.Tensor:
+    out = torch.empty_like(gate)
+    _lib.check(_lib.load().nfn_row_out(C.c_int(int(gate.dtype == torch.float32)), C.c_void_p(_p(o)), C.c_int(o.stride(0)), C.c_void_p(_p(gate)), C.c_int(gate.stride(0)), C.c_void_p(_p(weight)),
+                                       C.c_float(eps), C.c_void_p(_p(out)), C.c_int(out.stride(0)), C.c_int(o.shape[0]), C.c_int(o.shape[1]), C.c_int(live), C.c_void_p(_lib.stream_ptr())), "row_out")
+    return out
+
+
+def gru_rows(x: torch.Tensor, state: torch.Tensor, out: torch.Tensor, seqs: torch.Tensor, n_short: int) -> torch.Tensor:
+    """x [rows, 3 * width], state fp32 [slots, width], out [rows, width], seqs as in ``linear_rule``, the first ``n_short`` of them of few rows."""
+    a = _Gru(int(x.dtype == torch.float32), state.shape[1], _p(x), x.stride(0), _p(state), _p(out), out.stride(0), _p(seqs), seqs.shape[0], n_short)
+    _call("gru_rows", a)
+    return out
+
+
+def input_conv(h: torch.Tensor, conv: torch.Tensor, history: torch.Tensor, out: torch.Tensor, tiles: torch.Tensor) -> torch.Tensor:
+    """h, out [rows, ld], conv bf16 [taps, ld], history [2, slots, taps - 1, ld] of h's type."""
+    a = _InputConv(int(h.dtype == torch.float32), h.shape[1], conv.shape[0], _p(h), _p(conv), _p(history), history.stride(0), _p(out), _p(tiles), tiles.shape[0])
+    _call("input_conv", a)
     return out

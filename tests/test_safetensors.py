@@ -78,6 +78,13 @@ def _hf_llama(tmp_path, shards=True, tie=False):
     return root, sd
 
 
+def test_tensors_of_a_single_number(tmp_path):
+    t = {"g": torch.tensor(1.5).bfloat16(), "n": torch.tensor(3, dtype=torch.int32), "v": torch.ones(2).bfloat16()}
+    write_safetensors(tmp_path / "x.safetensors", t)
+    got, _ = read_safetensors(tmp_path / "x.safetensors")
+    assert all(torch.equal(got[k], v) and got[k].shape == v.shape for k, v in t.items())
+
+
 @pytest.mark.parametrize("shards,tie", [(True, False), (False, True)])
 def test_hf_llama_ingestion(tmp_path, shards, tie):
     root, sd = _hf_llama(tmp_path, shards, tie)
