@@ -2,13 +2,14 @@
 // formed from b. Everything but the loads and stores is fp32.
 //
 // Short entries (single tokens, portions of a few rows) go token after token. Long ones are an affine scan: a CTA takes 32 channels, 16 lanes with two
-// channels each, and 256 rows at a time in 32 segments of eight; every segment's rows become one step of the same form, the state in front
+// channels each, and 256 rows at a time in 32 segments of eight (two to a warp); every segment's rows become one step of the same form, the state in front
 // of a segment follows from those of the segments before it, and the rows are run again from there, out of registers.
 //
 // A step is taken as s <- s + z (c - s). Where z is small a state lasts for thousands of tokens, and a factor 1 - z that is rounded on its own would leave
 // each time a little less or more than the share z took.
 #include <type_traits>
 
+#include "attention_v2.cuh"
 #include "common.h"
 #include "paged.cuh"
 
@@ -18,9 +19,22 @@ namespace nfn {
 struct GruStep { float z, c; };
 template <typename T>
 __device__ __forceinline__ GruStep gru_step(float a, float b) {
-  return GruStep{sigmoid_for<T>(a), b >= 0.f ? b + 0.5f : sigmoid_for<T>(b)};
+  return GruStep{sigmoid_for<T>(a), fmaxf(b + 0.5f, sigmoid_for<T>(b))};      // the line is the larger one where b >= 0, the sigmoid where b < 0
 }
 __device__ __forceinline__ float gru_take(float s, float z, float c) { return s + z * (c - s); }
+__device__ __forceinline__ float2 gru_take2(float2 s, float2 z, float2 c) {
+  float2 d, r;
+  add2f(d.x, d.y, c.x, c.y, -s.x, -s.y);
+  fma2(r.x, r.y, z.x, z.y, d.x, d.y, s.x, s.y);
+  return r;
+}
+// the state behind several steps of which share `go` of it went and `come` came
+__device__ __forceinline__ float2 gru_after(float2 s, float2 go, float2 come) {
+  float2 d, r;
+  fma2(d.x, d.y, -go.x, -go.y, s.x, s.y, come.x, come.y);
+  add2f(r.x, r.y, s.x, s.y, d.x, d.y);
+  return r;
+}
 template <typename T>
 __device__ __forceinline__ float gru_out(float s, float g) { return s * g * sigmoid_for<T>(g); }
 
@@ -28,6 +42,13 @@ template <typename T>
 using GruPair = typename std::conditional<sizeof(T) == 4, float2, uint32_t>::type;      // two neighbouring channels as they lie in memory
 __device__ __forceinline__ float2 gru_unpack(float2 v) { return v; }
 __device__ __forceinline__ float2 gru_unpack(uint32_t v) { return unpack_bf16x2(v); }
+// a share's input of minus infinity
+template <typename T>
+__device__ __forceinline__ GruPair<T> gru_never();
+template <>
+__device__ __forceinline__ float2 gru_never<float>() { return make_float2(-INFINITY, -INFINITY); }
+template <>
+__device__ __forceinline__ uint32_t gru_never<__nv_bfloat16>() { return 0xff80ff80u; }
 __device__ __forceinline__ void gru_store(float* p, float x, float y) { *reinterpret_cast<float2*>(p) = make_float2(x, y); }
 __device__ __forceinline__ void gru_store(__nv_bfloat16* p, float x, float y) { *reinterpret_cast<uint32_t*>(p) = pack_bf16x2(x, y); }
 
@@ -52,16 +73,16 @@ gru_short_kernel(const nfn_gru_args p) {
   *st = s;
 }
 
-constexpr int GS_LANES = 16, GS_SEGS = 32, GS_ROWS = 8, GS_THREADS = GS_LANES * GS_SEGS, GS_SPAN = GS_SEGS * GS_ROWS;
+constexpr int GS_LANES = 16, GS_WARPS = 16, GS_ROWS = 8, GS_THREADS = GS_WARPS * 32, GS_SPAN = 2 * GS_WARPS * GS_ROWS;
 template <typename T>
 __global__ void __launch_bounds__(GS_THREADS, 1)
 gru_scan_kernel(const nfn_gru_args p) {
   constexpr bool AHEAD = sizeof(T) == 2;                    // the next rows are on their way while these are used
-  __shared__ float4 segs[2][GS_SEGS][GS_LANES];             // of both channels: share of the state before it that goes, what comes in its place
+  __shared__ float4 warps[2][GS_WARPS][GS_LANES];           // of a warp's two segments and both channels: share of the state that goes, what comes in its place
   const nfn_seq_rows seq = p.seqs[p.n_short + blockIdx.y];
   if (seq.slot < 0) return;
-  const int lane = threadIdx.x % GS_LANES, seg = threadIdx.x / GS_LANES, c = blockIdx.x * 2 * GS_LANES + 2 * lane;
-  const bool on = c < p.width;
+  const int warp = threadIdx.x / 32, lane = threadIdx.x % GS_LANES, seg = threadIdx.x / GS_LANES, c = blockIdx.x * 2 * GS_LANES + 2 * lane;
+  const bool on = c < p.width, second = seg & 1;
   float2* st = reinterpret_cast<float2*>(p.state + (size_t)seq.slot * p.width + c);
   float2 s = make_float2(0.f, 0.f);
   if (on && seq.pos0 > 0) s = *st;
@@ -69,11 +90,13 @@ gru_scan_kernel(const nfn_gru_args p) {
   T* out = static_cast<T*>(p.out) + (size_t)seq.row0 * p.ld_out + c;
   GruPair<T> a[GS_ROWS], b[GS_ROWS], g[GS_ROWS], na[AHEAD ? GS_ROWS : 1], nb[AHEAD ? GS_ROWS : 1], ng[AHEAD ? GS_ROWS : 1];
   auto fetch = [&](int r0, GruPair<T>* fa, GruPair<T>* fb, GruPair<T>* fg) {
+    const int first = r0 + seg * GS_ROWS;
+    const T* x = in + (size_t)first * p.ld_in;
 #pragma unroll
-    for (int i = 0; i < GS_ROWS; ++i) {
-      const int r = r0 + seg * GS_ROWS + i;
-      if (on && r < seq.n) {
-        const T* x = in + (size_t)r * p.ld_in;
+    for (int i = 0; i < GS_ROWS; ++i, x += p.ld_in) {
+      fa[i] = gru_never<T>();                               // rows that do not exist leave the state alone
+      fb[i] = fg[i] = GruPair<T>{};
+      if (on && first + i < seq.n) {
         fa[i] = *reinterpret_cast<const GruPair<T>*>(x);
         fb[i] = *reinterpret_cast<const GruPair<T>*>(x + p.width);
         fg[i] = *reinterpret_cast<const GruPair<T>*>(x + 2 * p.width);
@@ -84,34 +107,40 @@ gru_scan_kernel(const nfn_gru_args p) {
   int buf = 0;
   for (int r0 = 0; r0 < seq.n; r0 += GS_SPAN, buf ^= 1) {
     if constexpr (AHEAD) fetch(r0 + GS_SPAN, na, nb, ng);
-    const int live = on ? min(GS_ROWS, seq.n - r0 - seg * GS_ROWS) : 0;
-    float2 z[GS_ROWS], cand[GS_ROWS];
-    float4 f = make_float4(0.f, 0.f, 0.f, 0.f);
+    float2 z[GS_ROWS], cand[GS_ROWS], go = make_float2(0.f, 0.f), come = go;
 #pragma unroll
-    for (int i = 0; i < GS_ROWS; ++i)
-      if (i < live) {
-        const float2 x = gru_unpack(a[i]), y = gru_unpack(b[i]);
-        const GruStep u = gru_step<T>(x.x, y.x), v = gru_step<T>(x.y, y.y);
-        z[i] = make_float2(u.z, v.z);
-        cand[i] = make_float2(u.c, v.c);
-        f = make_float4(gru_take(f.x, u.z, 1.f), gru_take(f.y, u.z, u.c), gru_take(f.z, v.z, 1.f), gru_take(f.w, v.z, v.c));
-      }
-    segs[buf][seg][lane] = f;
+    for (int i = 0; i < GS_ROWS; ++i) {
+      const float2 x = gru_unpack(a[i]), y = gru_unpack(b[i]);
+      const GruStep u = gru_step<T>(x.x, y.x), v = gru_step<T>(x.y, y.y);
+      z[i] = make_float2(u.z, v.z);
+      cand[i] = make_float2(u.c, v.c);
+      go = gru_take2(go, z[i], make_float2(1.f, 1.f));
+      come = gru_take2(come, z[i], cand[i]);
+    }
+    // both segments of the warp as one step, the first one's kept for the second
+    const float2 go1 = make_float2(__shfl_xor_sync(0xffffffffu, go.x, GS_LANES), __shfl_xor_sync(0xffffffffu, go.y, GS_LANES));
+    const float2 come1 = make_float2(__shfl_xor_sync(0xffffffffu, come.x, GS_LANES), __shfl_xor_sync(0xffffffffu, come.y, GS_LANES));
+    if (!second) {
+      const float2 f = gru_after(go, go1, go1), e = gru_after(come, go1, come1);
+      warps[buf][warp][lane] = make_float4(f.x, f.y, e.x, e.y);
+    }
     __syncthreads();                                        // the other buffer was read before the last one of these
     float2 mine = s;
 #pragma unroll
-    for (int q = 0; q < GS_SEGS; ++q) {
-      if (q == seg) mine = s;
-      const float4 e = segs[buf][q][lane];
-      s = make_float2(s.x + (e.y - e.x * s.x), s.y + (e.w - e.z * s.y));
+    for (int q = 0; q < GS_WARPS; ++q) {
+      if (q == warp) mine = s;
+      const float4 e = warps[buf][q][lane];
+      s = gru_after(s, make_float2(e.x, e.y), make_float2(e.z, e.w));
     }
+    if (second) mine = gru_after(mine, go1, come1);
+    const int first = r0 + seg * GS_ROWS;
+    T* dst = out + (size_t)first * p.ld_out;
 #pragma unroll
-    for (int i = 0; i < GS_ROWS; ++i)
-      if (i < live) {
-        mine = make_float2(gru_take(mine.x, z[i].x, cand[i].x), gru_take(mine.y, z[i].y, cand[i].y));
-        const float2 h = gru_unpack(g[i]);
-        gru_store(out + (size_t)(r0 + seg * GS_ROWS + i) * p.ld_out, gru_out<T>(mine.x, h.x), gru_out<T>(mine.y, h.y));
-      }
+    for (int i = 0; i < GS_ROWS; ++i, dst += p.ld_out) {
+      mine = gru_take2(mine, z[i], cand[i]);
+      const float2 h = gru_unpack(g[i]);
+      if (on && first + i < seq.n) gru_store(dst, gru_out<T>(mine.x, h.x), gru_out<T>(mine.y, h.y));
+    }
     if constexpr (AHEAD) {
 #pragma unroll
       for (int i = 0; i < GS_ROWS; ++i) { a[i] = na[i]; b[i] = nb[i]; g[i] = ng[i]; }

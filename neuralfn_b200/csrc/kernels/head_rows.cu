@@ -306,6 +306,15 @@ group_products_mma_kernel(const nfn_group_products_args p) {
     on[t] = r < p.rows;
     src[t] = static_cast<const __nv_bfloat16*>(p.in) + (size_t)(on[t] ? r : r0) * p.ld_in + (tail ? (size_t)p.tail_in : (size_t)g * p.in_group) + 8 * j;
   }
+  const int live = min(M, p.rows - r0);
+  constexpr int GV = 32 * M / (GM_WARPS * 32);            // results of a thread, and their gates ahead of time
+  float gate[GV];
+#pragma unroll
+  for (int i = 0; i < GV; ++i) {
+    const int x = threadIdx.x + i * GM_WARPS * 32, col = x / 32, row = x % 32;
+    gate[i] = 0.f;
+    if (!tail && p.gate && col < live && n0 + row < N) gate[i] = __bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[(size_t)(r0 + col) * p.ld_gate + (size_t)g * p.gate_group + n0 + row]);
+  }
   float acc[2][NT][4];
 #pragma unroll
   for (int m = 0; m < 2; ++m)
@@ -354,10 +363,10 @@ group_products_mma_kernel(const nfn_group_products_args p) {
 #pragma unroll
       for (int c = 0; c < 4; ++c) part[warp][m * 16 + gr + (c >> 1) * 8][8 * t + 2 * j + (c & 1)] = acc[m][t][c];
   __syncthreads();
-  const int live = min(M, p.rows - r0);
-  for (int x = threadIdx.x; x < 32 * live; x += GM_WARPS * 32) {
-    const int col = x / 32, row = x % 32;
-    if (n0 + row >= N) continue;
+#pragma unroll
+  for (int i = 0; i < GV; ++i) {
+    const int x = threadIdx.x + i * GM_WARPS * 32, col = x / 32, row = x % 32;
+    if (col >= live || n0 + row >= N) continue;
     float v = 0.f;
 #pragma unroll
     for (int w = 0; w < GM_WARPS; ++w) v += part[w][row][col];
@@ -366,7 +375,7 @@ group_products_mma_kernel(const nfn_group_products_args p) {
       continue;
     }
     v = ff_act(v, p.act);
-    if (p.gate) v *= sigmoid_for<__nv_bfloat16>(__bfloat162float(static_cast<const __nv_bfloat16*>(p.gate)[(size_t)(r0 + col) * p.ld_gate + (size_t)g * p.gate_group + n0 + row]));
+    if (p.gate) v *= sigmoid_for<__nv_bfloat16>(gate[i]);
     static_cast<__nv_bfloat16*>(p.out)[(size_t)(r0 + col) * p.ld_out + (size_t)g * p.out_group + n0 + row] = __float2bfloat16(v);
   }
 }

@@ -19,7 +19,7 @@ namespace nfn {
 
 constexpr int LC_T = NFN_LINEAR_CHUNK, LC_WARPS = 4, LC_THREADS = LC_WARPS * 32, LC_COLS = 16 * LC_WARPS;
 constexpr int LC_VP = LC_COLS * 2 + 16, LC_PP = LC_T * 2 + 16;          // bytes of a row of values, of scores
-constexpr int LC_MAX_SEGS = 8, LC_MIN_SEG = 4;                          // segments of a sequence, and fewest chunks of one
+constexpr int LC_MAX_SEGS = 9, LC_MIN_SEG = 4;                          // segments of a sequence, and fewest chunks of one
 __host__ __device__ constexpr int lc_pitch(int dk) { return dk * 2 + 16; }
 __host__ __device__ constexpr int lc_stage(int dk) { return 2 * LC_T * lc_pitch(dk) + LC_T * LC_VP; }
 __host__ __device__ constexpr int lc_smem(int dk) { return 2 * lc_stage(dk) + 2 * LC_T * LC_PP; }
@@ -195,13 +195,18 @@ linear_chunk_kernel(const LinearChunkParams p) {
           split_bf16(s[2 * kk][2], s[2 * kk][3], hi[2], lo[2]);
           split_bf16(s[2 * kk + 1][2], s[2 * kk + 1][3], hi[3], lo[3]);
 #pragma unroll
-          for (int m = 0; m < 4; ++m) {
-            uint32_t q[4];
-            lc_load(q, sQ + (16 * m + (lane & 15)) * PITCH + kk * 32 + (lane >> 4) * 16);
-            lc_mma(o[m][0], q[0], q[1], q[2], q[3], hi[0], hi[1]);
-            lc_mma(o[m][1], q[0], q[1], q[2], q[3], hi[2], hi[3]);
-            lc_mma(o[m][0], q[0], q[1], q[2], q[3], lo[0], lo[1]);
-            lc_mma(o[m][1], q[0], q[1], q[2], q[3], lo[2], lo[3]);
+          for (int m0 = 0; m0 < 4; m0 += 2) {               // four products in a row that do not wait for one another
+            uint32_t q[2][4];
+#pragma unroll
+            for (int m = 0; m < 2; ++m) lc_load(q[m], sQ + (16 * (m0 + m) + (lane & 15)) * PITCH + kk * 32 + (lane >> 4) * 16);
+#pragma unroll
+            for (int m = 0; m < 2; ++m)
+#pragma unroll
+              for (int t = 0; t < 2; ++t) lc_mma(o[m0 + m][t], q[m][0], q[m][1], q[m][2], q[m][3], hi[2 * t], hi[2 * t + 1]);
+#pragma unroll
+            for (int m = 0; m < 2; ++m)
+#pragma unroll
+              for (int t = 0; t < 2; ++t) lc_mma(o[m0 + m][t], q[m][0], q[m][1], q[m][2], q[m][3], lo[2 * t], lo[2 * t + 1]);
           }
         }
 #pragma unroll
@@ -250,13 +255,14 @@ linear_chunk_kernel(const LinearChunkParams p) {
           }
         }
 #pragma unroll
-        for (int t = 0; t < NT; t += 2) {
-          uint32_t k[4];
-          lc_load_t(k, sK + (16 * kk + (lane & 15)) * PITCH + t * 16 + (lane >> 4) * 16);
-          lc_mma(s[t], hi[0], hi[1], hi[2], hi[3], k[0], k[1]);
-          lc_mma(s[t + 1], hi[0], hi[1], hi[2], hi[3], k[2], k[3]);
-          lc_mma(s[t], lo[0], lo[1], lo[2], lo[3], k[0], k[1]);
-          lc_mma(s[t + 1], lo[0], lo[1], lo[2], lo[3], k[2], k[3]);
+        for (int t0 = 0; t0 < NT; t0 += 4) {
+          uint32_t k[2][4];
+#pragma unroll
+          for (int t = 0; t < 2; ++t) lc_load_t(k[t], sK + (16 * kk + (lane & 15)) * PITCH + (t0 + 2 * t) * 16 + (lane >> 4) * 16);
+#pragma unroll
+          for (int t = 0; t < 4; ++t) lc_mma(s[t0 + t], hi[0], hi[1], hi[2], hi[3], k[t / 2][2 * (t & 1)], k[t / 2][2 * (t & 1) + 1]);
+#pragma unroll
+          for (int t = 0; t < 4; ++t) lc_mma(s[t0 + t], lo[0], lo[1], lo[2], lo[3], k[t / 2][2 * (t & 1)], k[t / 2][2 * (t & 1) + 1]);
         }
       }
     }
@@ -308,7 +314,17 @@ extern "C" int nfn_linear_chunks(const nfn_linear_args* args, int max_rows, void
   LinearChunkParams p{};
   p.a = a;
   const long long cells = (long long)a.heads * a.n_seqs, ctas = cells * ceil_div(a.vdim_p, LC_COLS);
-  p.segs = (int)std::min<long long>(std::min<long long>(LC_MAX_SEGS, 2LL * sm_count() / ctas), ceil_div(max_rows, LC_T) / LC_MIN_SEG);
+  // as many as leave the fewest chunks per slot, two CTAs to an SM; more of them only where it pays
+  const int chunks = ceil_div(max_rows, LC_T), slots = 2 * sm_count();
+  double best = 1e30;
+  p.segs = 1;
+  for (int n = 1; n <= LC_MAX_SEGS && (n == 1 || n * LC_MIN_SEG <= chunks); ++n) {
+    const double cost = (double)((ctas * n + slots - 1) / slots) * ceil_div(chunks, n) * (n > 1 ? 1.4 : 1.0) + n;      // the states in front take two fifths of a pass
+    if (cost < best) {
+      best = cost;
+      p.segs = n;
+    }
+  }
   if (!workspace || cells * linear_segment_bytes(a.dim_p, a.vdim_p) > workspace_bytes) p.segs = 1;
   p.segs = std::max(p.segs, 1);
   if ((long long)a.n_seqs * p.segs > 65535) return fail(-1, "linear attention: too many sequences for one launch");

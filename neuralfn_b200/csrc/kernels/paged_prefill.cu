@@ -37,8 +37,8 @@ struct PagedPrefillParams {
   int* status;
 };
 
-// tm_k, tm_v: the pages (EXPANDED: the pages for the rotated key part, the matrix of unrotated keys and values)
-template <bool EXPANDED>
+// GATED: with an output gate. tm_k, tm_v: the pages (EXPANDED: the pages for the rotated key part, the matrix of unrotated keys and values)
+template <bool EXPANDED, bool GATED>
 __global__ void __launch_bounds__(AV2_THREADS, 2)
 paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_constant__ CUtensorMap tm_k,
                      const __grid_constant__ CUtensorMap tm_v, const PagedPrefillParams p) {
@@ -367,12 +367,12 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
     }
     // ---- O / l, output gate -> global: 64 channels at a time, their gates on the way before O is waited for ----
     __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(a.out) + (size_t)(row0 + qi) * a.ld_o + (size_t)h * a.vdim_p;
-    const __nv_bfloat16* grow_ = (a.gate && row_ok) ? static_cast<const __nv_bfloat16*>(a.gate) + (size_t)(row0 + qi) * a.ld_gate + (size_t)h * a.vdim_p : nullptr;
+    const __nv_bfloat16* grow_ = (GATED && row_ok) ? static_cast<const __nv_bfloat16*>(a.gate) + (size_t)(row0 + qi) * a.ld_gate + (size_t)h * a.vdim_p : nullptr;
     uint4 gv[8];
     auto fetch_gate = [&](int c0) {
 #pragma unroll
       for (int g = 0; g < 8; ++g)
-        if (grow_ && c0 + g * 8 < a.vdim_p) gv[g] = __ldg(reinterpret_cast<const uint4*>(grow_ + c0 + g * 8));
+        if (GATED && grow_ && c0 + g * 8 < a.vdim_p) gv[g] = __ldg(reinterpret_cast<const uint4*>(grow_ + c0 + g * 8));
     };
     fetch_gate(0);
     if (ok) {
@@ -397,11 +397,11 @@ paged_prefill_kernel(const __grid_constant__ CUtensorMap tm_q, const __grid_cons
             float v[8];
 #pragma unroll
             for (int i = 0; i < 8; ++i) v[i] = __uint_as_float(o[g * 8 + i]) * inv;
-            if (grow_) {
+            if (GATED) {
               const float2 g0 = unpack_bf16x2(gv[g].x), g1 = unpack_bf16x2(gv[g].y), g2 = unpack_bf16x2(gv[g].z), g3 = unpack_bf16x2(gv[g].w);
               const float gf[8] = {g0.x, g0.y, g1.x, g1.y, g2.x, g2.y, g3.x, g3.y};
 #pragma unroll
-              for (int i = 0; i < 8; ++i) v[i] *= 1.f / (1.f + __expf(-gf[i]));
+              for (int i = 0; i < 8; ++i) v[i] *= sigmoid_for<__nv_bfloat16>(gf[i]);
             }
             store8(orow + c0 + g * 8, v);
           }
@@ -440,14 +440,14 @@ extern "C" int nfn_paged_tile_rows(int f32, int heads, int kv_heads, int dim_p, 
   return PP_BM / hg;
 }
 
-template <bool EXPANDED>
+template <bool EXPANDED, bool GATED>
 static int launch_paged_prefill(PagedPrefillParams& p, const CUtensorMap& tq, const CUtensorMap& tk, const CUtensorMap& tv, cudaStream_t st) {
   const nfn_paged_attention_args& a = p.a;
   p.o_col = EXPANDED ? PP_BN + PP_BN / 2 : PP_BN;
   const int cols = (int)p.o_col + (EXPANDED ? p.panels_v * 64 : a.vdim_p);
   p.tmem_cols = cols <= 128 ? 128 : cols <= 256 ? 256 : 512;
   p.status = status_ptr();
-  auto kern = paged_prefill_kernel<EXPANDED>;
+  auto kern = paged_prefill_kernel<EXPANDED, GATED>;
   static uint32_t raised[64] = {};
   int dev = 0;
   cudaGetDevice(&dev);
@@ -482,7 +482,8 @@ extern "C" int nfn_paged_attention_tiles(const nfn_paged_attention_args* args, n
   const uint64_t cells = (uint64_t)a.pages * a.kv_heads;
   if (!make_tmap_2d(&tk, a.k_pool, 2, a.dim_p, cells * NFN_PAGE, a.dim_p, 64, PP_BN, 128)) return -3;
   if (!make_tmap_2d(&tv, a.v_pool, 2, NFN_PAGE, cells * a.vdim_p, NFN_PAGE, NFN_PAGE, a.vdim_p, 128)) return -3;
-  return launch_paged_prefill<false>(p, tq, tk, tv, static_cast<cudaStream_t>(stream));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return a.gate ? launch_paged_prefill<false, true>(p, tq, tk, tv, st) : launch_paged_prefill<false, false>(p, tq, tk, tv, st);
 }
 
 // stages of values for these panels: two, or one where that lets a second CTA in or is all there is room for; 0: no room
@@ -522,5 +523,6 @@ extern "C" int nfn_latent_attention_tiles(const nfn_paged_attention_args* args, 
   if (!make_tmap_3d(&tq, a.q, 2, a.dim_p, a.heads, a.total_rows, a.dim_p, a.ld_q, 64, 1, PP_BM, 128)) return -3;
   if (!make_tmap_2d(&tk, a.k_pool, 2, lp, (uint64_t)a.pages * NFN_PAGE, lp, 64, PP_BN, 128)) return -3;
   if (!make_tmap_2d(&tx, x->x, 2, cols, x->x_rows, cols, 64, PP_BN, 128)) return -3;
-  return launch_paged_prefill<true>(p, tq, tk, tx, static_cast<cudaStream_t>(stream));
+  cudaStream_t st = static_cast<cudaStream_t>(stream);
+  return a.gate ? launch_paged_prefill<true, true>(p, tq, tk, tx, st) : launch_paged_prefill<true, false>(p, tq, tk, tx, st);
 }

@@ -200,7 +200,7 @@ stream_pass_kernel(const nfn_stream_args p) {
   }
 }
 
-// The convolution over the rows of any entries. A thread takes eight channels of a tile's rows; the window slides through registers (TAPS = 0: any
+// The convolution over the rows of any entries. A thread takes four channels of a tile's rows; the window slides through registers (TAPS = 0: any
 // number of taps, rows are read again).
 constexpr int IC_THREADS = 128;
 
@@ -208,7 +208,7 @@ template <typename T, int TAPS>
 __global__ void __launch_bounds__(IC_THREADS)
 input_conv_kernel(const nfn_input_conv_args p) {
   const nfn_row_tile t = p.tiles[blockIdx.x];
-  const int col = (blockIdx.y * IC_THREADS + threadIdx.x) * 8;
+  const int col = (blockIdx.y * IC_THREADS + threadIdx.x) * 4;
   if (t.slot < 0 || col >= p.ld) return;
   const int taps = TAPS ? TAPS : p.taps, hist = taps - 1, ti0 = t.row0 - t.e_row0;
   const T* rows = static_cast<const T*>(p.h) + (size_t)t.e_row0 * p.ld + col;
@@ -218,71 +218,53 @@ input_conv_kernel(const nfn_input_conv_args p) {
   T* out = static_cast<T*>(p.out) + (size_t)t.row0 * p.ld + col;
   const bool last = hist > 0 && t.row0 + t.n == t.e_row0 + t.e_n;
   // row `idx` of the entry: this step's, a stored one, or zero before the sequence's start
-  auto source = [&](int idx, float (&v)[8]) {
-    if (idx >= 0) {
-      load8(rows + (size_t)idx * p.ld, v);
-    } else if (t.e_pos0 + idx >= 0) {
-      load8(old + (size_t)(hist + idx) * p.ld, v);
-    } else {
-#pragma unroll
-      for (float& f : v) f = 0.f;
-    }
+  auto source = [&](int idx) {
+    if (idx >= 0) return load4(rows + (size_t)idx * p.ld);
+    return t.e_pos0 + idx >= 0 ? load4(old + (size_t)(hist + idx) * p.ld) : make_float4(0.f, 0.f, 0.f, 0.f);
   };
+  auto add = [](float4& a, const float4& w, const float4& x) { a.x += w.x * x.x; a.y += w.y * x.y; a.z += w.z * x.z; a.w += w.w * x.w; };
   if constexpr (TAPS == 0) {
     for (int i = 0; i < t.n; ++i) {
-      float acc[8], x[8], w[8];
-      source(ti0 + i, acc);
-      for (int j = 0; j < taps; ++j) {
-        source(ti0 + i - hist + j, x);
-        load8(conv + (size_t)j * p.ld, w);
-#pragma unroll
-        for (int e = 0; e < 8; ++e) acc[e] += w[e] * x[e];
-      }
-      store8(out + (size_t)i * p.ld, acc);
+      float4 a = source(ti0 + i);
+      for (int j = 0; j < taps; ++j) add(a, load4(conv + (size_t)j * p.ld), source(ti0 + i - hist + j));
+      store4(out + (size_t)i * p.ld, a);
     }
     if (last)
-      for (int i = 0; i < hist; ++i) {
-        float x[8];
-        source(t.e_n - hist + i, x);
-        store8(left + (size_t)i * p.ld, x);
-      }
+      for (int i = 0; i < hist; ++i) store4(left + (size_t)i * p.ld, source(t.e_n - hist + i));
   } else {
-    constexpr int N = 4;                                   // rows in flight
-    float win[TAPS > 1 ? TAPS - 1 : 1][8], w[TAPS][8], v[N][8];
+    constexpr int N = 8;                                   // rows in flight, as they lie in memory
+    struct alignas(4 * sizeof(T)) Raw { T v[4]; } raw[N];
+    float4 win[TAPS > 1 ? TAPS - 1 : 1], w[TAPS];
     auto fetch = [&](int i0) {
 #pragma unroll
       for (int i = 0; i < N; ++i)
-        if (i0 + i < t.n) load8(rows + (size_t)(ti0 + i0 + i) * p.ld, v[i]);
+        if (i0 + i < t.n) raw[i] = *reinterpret_cast<const Raw*>(rows + (size_t)(ti0 + i0 + i) * p.ld);
     };
     fetch(0);
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) source(ti0 - (TAPS - 1) + j, win[j]);
+    for (int j = 0; j < TAPS - 1; ++j) win[j] = source(ti0 - (TAPS - 1) + j);
 #pragma unroll
-    for (int j = 0; j < TAPS; ++j) load8(conv + (size_t)j * p.ld, w[j]);
+    for (int j = 0; j < TAPS; ++j) w[j] = load4(conv + (size_t)j * p.ld);
     for (int i0 = 0; i0 < t.n; i0 += N) {
       if (i0 > 0) fetch(i0);
 #pragma unroll
       for (int i = 0; i < N; ++i)
         if (i0 + i < t.n) {
-          float acc[8];
+          const float4 x = make_float4(to_float(raw[i].v[0]), to_float(raw[i].v[1]), to_float(raw[i].v[2]), to_float(raw[i].v[3]));
+          float4 a = x;
+          add(a, w[TAPS - 1], x);
 #pragma unroll
-          for (int e = 0; e < 8; ++e) {
-            const float x = v[i][e];
-            float a = x + w[TAPS - 1][e] * x;
+          for (int j = 0; j < TAPS - 1; ++j) add(a, w[j], win[j]);
 #pragma unroll
-            for (int j = 0; j < TAPS - 1; ++j) a += w[j][e] * win[j][e];
-#pragma unroll
-            for (int j = 0; j + 1 < TAPS - 1; ++j) win[j][e] = win[j + 1][e];
-            if constexpr (TAPS > 1) win[TAPS - 2][e] = x;
-            acc[e] = a;
-          }
-          store8(out + (size_t)(i0 + i) * p.ld, acc);
+          for (int j = 0; j + 1 < TAPS - 1; ++j) win[j] = win[j + 1];
+          if constexpr (TAPS > 1) win[TAPS - 2] = x;
+          store4(out + (size_t)(i0 + i) * p.ld, a);
         }
     }
     if constexpr (TAPS > 1) {
       if (last) {
 #pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) store8(left + (size_t)j * p.ld, win[j]);
+        for (int j = 0; j < TAPS - 1; ++j) store4(left + (size_t)j * p.ld, win[j]);
       }
     }
   }
@@ -290,7 +272,7 @@ input_conv_kernel(const nfn_input_conv_args p) {
 
 template <typename T>
 static int pick_input_conv(const nfn_input_conv_args& a, cudaStream_t st) {
-  const dim3 grid(a.n_tiles, ceil_div(a.ld, IC_THREADS * 8));
+  const dim3 grid(a.n_tiles, ceil_div(a.ld, IC_THREADS * 4));
   switch (a.taps) {
     case 1: input_conv_kernel<T, 1><<<grid, IC_THREADS, 0, st>>>(a); break;
     case 2: input_conv_kernel<T, 2><<<grid, IC_THREADS, 0, st>>>(a); break;
