@@ -1097,6 +1097,8 @@ int layered_engine::experts(const Layer& L, int rows, nfn_stream_args* sp) {
     g.rows = rows; g.groups = 1; g.n = L.shp; g.k = wp; g.in = hx; g.ld_in = wp; g.w = L.w_shared_up; g.out = shared_mid; g.ld_out = L.shp; g.act = d.ff_act;
     g.tail_n = L.ep; g.tail_w = L.router; g.tail_out = ex.logits; g.ld_tail = L.ep;
     K(nfn_group_products(&g, stream));
+  } else if (!shared && c.dtype == 0 && rows <= kFewRows) {
+    K(nfn_router_rows(hx, wp, L.router, rows, d.experts, wp, ex.logits, L.ep, stream));
   } else if (lin(hx, wp, L.router, rows, L.ep, wp, ex.logits, L.ep, kOutF32) || (shared && lin(hx, wp, L.w_shared_up, rows, L.shp, wp, shared_mid, L.shp, kOutAct, nullptr, d.ff_act))) {
     return -1;
   }

@@ -264,6 +264,49 @@ moe_act_rows_kernel(const __nv_bfloat16* __restrict__ gate_up, const float* __re
   store8(mid + (size_t)r * ff + c, g);
 }
 
+// Router logits: the warps of a CTA share the contraction of one expert's row with eight rows of h, every load of a thread on its way at once.
+constexpr int RT_WARPS = 8, RT_ROWS = 8;
+
+__global__ void __launch_bounds__(RT_WARPS * 32)
+router_rows_kernel(const __nv_bfloat16* __restrict__ h, int ld_h, const __nv_bfloat16* __restrict__ w, int rows, int width, float* __restrict__ logits, int ld_logits) {
+  __shared__ float part[RT_WARPS][RT_ROWS];
+  const int e = blockIdx.x, r0 = blockIdx.y * RT_ROWS, live = min(RT_ROWS, rows - r0), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  float a[RT_ROWS];
+#pragma unroll
+  for (int i = 0; i < RT_ROWS; ++i) a[i] = 0.f;
+  for (int k = threadIdx.x * 8; k < width; k += RT_WARPS * 32 * 8) {
+    uint4 x[RT_ROWS];
+    const uint4 u = *reinterpret_cast<const uint4*>(w + (size_t)e * width + k);
+#pragma unroll
+    for (int i = 0; i < RT_ROWS; ++i)
+      if (i < live) x[i] = *reinterpret_cast<const uint4*>(h + (size_t)(r0 + i) * ld_h + k);
+    const uint32_t uw[4] = {u.x, u.y, u.z, u.w};
+#pragma unroll
+    for (int i = 0; i < RT_ROWS; ++i) {
+      if (i >= live) break;
+      const uint32_t xw[4] = {x[i].x, x[i].y, x[i].z, x[i].w};
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const float2 f = unpack_bf16x2(uw[c]), g = unpack_bf16x2(xw[c]);
+        a[i] += f.x * g.x + f.y * g.y;
+      }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < RT_ROWS; ++i) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) a[i] += __shfl_xor_sync(0xffffffffu, a[i], o);
+    if (lane == 0) part[warp][i] = a[i];
+  }
+  __syncthreads();
+  if (threadIdx.x < live) {
+    float t = 0.f;
+#pragma unroll
+    for (int q = 0; q < RT_WARPS; ++q) t += part[q][threadIdx.x];
+    logits[(size_t)(r0 + threadIdx.x) * ld_logits + e] = t;
+  }
+}
+
 template <int NT>
 static void launch_products_mma(const nfn_moe_rows_args& a, int live, cudaStream_t st) {
   if (a.plain) moe_products_mma_kernel<kUp, NT><<<dim3(ceil_div(a.ff, 32), live), MM_WARPS * 32, 0, st>>>(a);
@@ -308,6 +351,15 @@ extern "C" int nfn_moe_rows(const nfn_moe_rows_args* args, nfn_stream_t stream) 
   if ((a.width | a.ff | a.ld_h) & 15) return fail(-1, "moe_rows: widths must be multiples of 16");
   if ((long long)a.rows * a.top > 0x7fffffffLL / 2) return fail(-1, "moe_rows: too many rows");
   return launch_moe_rows(a, static_cast<cudaStream_t>(stream));
+}
+
+extern "C" int nfn_router_rows(const void* h, int ld_h, const void* w, int rows, int experts, int width, float* logits, int ld_logits, nfn_stream_t stream) {
+  if (rows <= 0) return 0;
+  if (experts < 1 || experts > ld_logits || (width & 15) || width <= 0 || (ld_h & 7) || !h || !w || !logits) return fail(-1, "router_rows: rows padded to multiples of 16, a logit per expert");
+  if (ceil_div(rows, RT_ROWS) > 65535) return fail(-1, "router_rows: too many rows for one launch");
+  router_rows_kernel<<<dim3(experts, ceil_div(rows, RT_ROWS)), RT_WARPS * 32, 0, static_cast<cudaStream_t>(stream)>>>(static_cast<const __nv_bfloat16*>(h), ld_h, static_cast<const __nv_bfloat16*>(w),
+                                                                                                                 rows, width, logits, ld_logits);
+  return launch_check("router_rows");
 }
 
 extern "C" int nfn_moe_act_rows(const void* gate_up, const float* row_w, const int* plan, int capacity_rows, int ff, int act, const nfn_gate_clamp* clamp, void* mid,

@@ -643,6 +643,8 @@ int nfn_gru_rows(const nfn_gru_args* args, nfn_stream_t stream);
 // Weights: s, with normalise / (sum of the chosen ones + 1e-20), times scale. Ties: the lower index. softmax: the choice goes by the logits and the weights
 // are the softmax over the chosen ones alone, times scale (no correction, no groups).
 typedef struct { const void* correction; int groups, keep_groups, normalise; float scale; int softmax; } nfn_route_rule;
+// logits[r][e] = h[r] . w[e] for a handful of rows (bf16, fp32 sums): a CTA per expert and eight rows. width: a multiple of 16.
+int nfn_router_rows(const void* h, int ld_h, const void* w, int rows, int experts, int width, float* logits, int ld_logits, nfn_stream_t stream);
 int nfn_moe_choose(const float* logits, int ld, int T, int E, int k, const nfn_route_rule* rule, int* idx, float* weight, int* counts, nfn_stream_t stream);
 int nfn_moe_route(const float* logits, int ld, int T, int E, int k, int score_fn, int norm_topk, float route_scale, int* topk_idx, float* topk_w,
                   int* counts, nfn_stream_t stream);

@@ -22,14 +22,15 @@ __device__ __forceinline__ float st_block_sum(float v, float* red) {
   return t;
 }
 
+template <typename T>
+struct alignas(4 * sizeof(T)) StPiece { T v[4]; };
 constexpr int ST_HIST = 3;      // history rows fetched ahead
 
-// the norm's weights of channels 4 v .. 4 v + 3; one number for all of them
-__device__ __forceinline__ float4 st_weight(const void* w, int v, int scalar) {
+// a norm's weights of channels 4 v .. 4 v + 3, as they lie in memory; scalar: one number for all of them
+__device__ __forceinline__ StPiece<__nv_bfloat16> st_weight(const void* w, int v, int scalar) {
   const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(w);
-  if (!scalar) return load4(p + 4 * v);
-  const float f = __bfloat162float(*p);
-  return make_float4(f, f, f, f);
+  if (!scalar) return *reinterpret_cast<const StPiece<__nv_bfloat16>*>(p + 4 * v);
+  return StPiece<__nv_bfloat16>{{*p, *p, *p, *p}};
 }
 
 // S: streams held in registers (an upper bound; the mixing weights past p.streams are zero). CONV: with the short convolution. Few rows take many threads each, so that a
@@ -46,6 +47,8 @@ stream_pass_kernel(const nfn_stream_args p) {
   const float* x = p.x + (size_t)src * n * p.ld;
   float* x_out = p.x_out ? p.x_out + (size_t)r * n * p.ld : nullptr;
   const T* y = static_cast<const T*>(p.y);
+  nfn_row_tile tile{};
+  if constexpr (CONV) tile = p.tiles[r];                   // the first of all: the history's place depends on it
   float4 b[S], f;
   auto fetch_x = [&](int v) {
     if (emb) {
@@ -84,24 +87,22 @@ stream_pass_kernel(const nfn_stream_args p) {
     fetch_x(threadIdx.x);
     fetch_y(threadIdx.x);
   }
-  float4 wt = make_float4(0.f, 0.f, 0.f, 0.f);             // the norm's weights of the first piece come along
+  StPiece<__nv_bfloat16> wt{}, wy{};                       // the norms' weights of the first piece come along
+  if (p.y_weight && threadIdx.x < vecs) wy = st_weight(p.y_weight, threadIdx.x, p.scalar_norms);
   if (p.h && p.weight && threadIdx.x < vecs) wt = st_weight(p.weight, threadIdx.x, p.scalar_norms);
-  nfn_row_tile tile{};
   const T* old = nullptr;                                  // the sequence's stored rows; none before its start
-  float4 past[ST_HIST], taps[ST_HIST + 1];
+  StPiece<T> past[ST_HIST];                                // as they lie in memory
+  StPiece<__nv_bfloat16> taps[ST_HIST + 1];
   const int hist = p.conv_taps - 1;
   const __nv_bfloat16* conv = static_cast<const __nv_bfloat16*>(p.conv);
-  auto stored = [&](int i, int v) { return old && tile.e_pos0 - hist + i >= 0 ? load4(old + (size_t)i * p.ld + 4 * v) : make_float4(0.f, 0.f, 0.f, 0.f); };
+  auto stored = [&](int i, int v) { return old && tile.e_pos0 - hist + i >= 0 ? *reinterpret_cast<const StPiece<T>*>(old + (size_t)i * p.ld + 4 * v) : StPiece<T>{}; };
+  auto tap = [&](int i, int v) { return *reinterpret_cast<const StPiece<__nv_bfloat16>*>(conv + (size_t)i * p.ld + 4 * v); };
   if constexpr (CONV) {
-    tile = p.tiles[r];
     if (tile.slot >= 0 && hist > 0) old = static_cast<const T*>(p.history) + (size_t)tile.parity * p.history_half + (size_t)tile.slot * hist * p.ld;
     if (threadIdx.x < vecs) {
 #pragma unroll
       for (int i = 0; i < ST_HIST; ++i)
         if (i < hist) past[i] = stored(i, threadIdx.x);
-#pragma unroll
-      for (int i = 0; i <= ST_HIST; ++i)
-        if (i <= hist) taps[i] = load4(conv + (size_t)i * p.ld + 4 * threadIdx.x);
     }
   }
   __syncthreads();
@@ -125,7 +126,8 @@ stream_pass_kernel(const nfn_stream_args p) {
       else fetch_y(v);
     }
     if (p.y_weight) {
-      const float4 w = st_weight(p.y_weight, v, p.scalar_norms);
+      if (v != threadIdx.x) wy = st_weight(p.y_weight, v, p.scalar_norms);
+      const float4 w = load4(wy.v);
       f.x *= ry * w.x; f.y *= ry * w.y; f.z *= ry * w.z; f.w *= ry * w.w;
     }
     if (emb) {
@@ -169,10 +171,18 @@ stream_pass_kernel(const nfn_stream_args p) {
     }
   }
   if (!p.h || !p.weight) return;
+  if constexpr (CONV) {                                    // on their way during the sum
+    if (threadIdx.x < vecs) {
+#pragma unroll
+      for (int i = 0; i <= ST_HIST; ++i)
+        if (i <= hist) taps[i] = tap(i, threadIdx.x);
+    }
+  }
   const float rms = 1.f / sqrtf(st_block_sum<ST_THREADS>(ss, red) / (float)p.width + p.eps);
   T* h = static_cast<T*>(p.h) + (size_t)r * p.ld;
   for (int v = threadIdx.x; v < vecs; v += ST_THREADS) {
-    const float4 u = load4(st_row + 4 * v), w = v == threadIdx.x ? wt : st_weight(p.weight, v, p.scalar_norms);
+    if (v != threadIdx.x) wt = st_weight(p.weight, v, p.scalar_norms);
+    const float4 u = load4(st_row + 4 * v), w = load4(wt.v);
     const float4 n = make_float4(u.x * rms * (w.x + p.weight_offset), u.y * rms * (w.y + p.weight_offset), u.z * rms * (w.z + p.weight_offset), u.w * rms * (w.w + p.weight_offset));
     if constexpr (CONV) {
       float4 c = n;
@@ -185,12 +195,15 @@ stream_pass_kernel(const nfn_stream_args p) {
       if (ahead) {
 #pragma unroll
         for (int i = 0; i < ST_HIST; ++i)
-          if (i < hist) add(i, past[i], taps[i]);
+          if (i < hist) add(i, load4(past[i].v), load4(taps[i].v));
 #pragma unroll
         for (int i = 0; i <= ST_HIST; ++i)
-          if (i == hist) add(i, n, taps[i]);
+          if (i == hist) add(i, n, load4(taps[i].v));
       } else {
-        for (int i = 0; i < hist; ++i) add(i, stored(i, v), load4(conv + (size_t)i * p.ld + 4 * v));
+        for (int i = 0; i < hist; ++i) {
+          const StPiece<T> x = stored(i, v);
+          add(i, load4(x.v), load4(conv + (size_t)i * p.ld + 4 * v));
+        }
         add(hist, n, load4(conv + (size_t)hist * p.ld + 4 * v));
       }
       store4(h + 4 * v, c);

@@ -12,7 +12,7 @@ from . import _lib
 from .paged import PAGE, PagedCache, _Attention
 
 __all__ = ["LatentCache", "delta_out", "delta_rule", "expert_choice", "expert_rows", "ff_rows", "frequencies", "group_products", "gru_rows", "head_rows", "input_conv",
-           "latent_attention_rows", "latent_attention_tiles", "latent_gather", "latent_rows", "linear_rule", "linear_step", "logit_cap", "row_out", "shift_rows", "stream_pass", "wkv_rule", "wkv_step"]
+           "latent_attention_rows", "latent_attention_tiles", "latent_gather", "latent_rows", "linear_rule", "linear_step", "logit_cap", "router_rows", "row_out", "shift_rows", "stream_pass", "wkv_rule", "wkv_step"]
 
 
 class _Stream(C.Structure):
@@ -123,6 +123,14 @@ def expert_rows(h: torch.Tensor, logits: torch.Tensor, w_gate_up: torch.Tensor, 
                  _p(shared_down), _p(y_shared), int(weigh_output), *clamp)
     _call("moe_rows", a)
     return idx.view(rows, top), weight.view(rows, top), y.view(rows, top, width)
+
+
+def router_rows(h: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """h bf16 [rows, width], w bf16 [experts, width] -> fp32 [rows, experts]."""
+    out = torch.zeros(h.shape[0], w.shape[0], device=h.device)
+    _lib.check(_lib.load().nfn_router_rows(C.c_void_p(_p(h)), C.c_int(h.stride(0)), C.c_void_p(_p(w)), C.c_int(h.shape[0]), C.c_int(w.shape[0]), C.c_int(h.shape[1]), C.c_void_p(_p(out)),
+                                           C.c_int(out.stride(0)), C.c_void_p(_lib.stream_ptr())), "router_rows")
+    return out
 
 
 def logit_cap(logits: torch.Tensor, scale: float, cap: float) -> None:

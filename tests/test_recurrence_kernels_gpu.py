@@ -288,3 +288,10 @@ def test_softmax_routing_and_experts_weighted_at_their_output(experts, top, rows
             close(w[t], a, 1e-5)
         mid = torch.stack([oracle.clamped_gate(*(gu[k].double() @ h[t].double()).split(ff), 0.9) for k in e.tolist()])
         close(y[t], torch.einsum("ewf,ef->ew", down[e].double(), mid), 0.02 if dtype == torch.bfloat16 else 1e-5)
+
+
+@pytest.mark.parametrize("rows,experts,width", [(1, 1, 16), (8, 32, 4096), (9, 40, 2064), (32, 100, 336)])
+def test_router_rows(rows, experts, width):
+    rnd = gen(18)
+    h, w = rnd(rows, width), rnd(experts, width)
+    close(Y.router_rows(h, w), h.double() @ w.double().T, 3e-6)
