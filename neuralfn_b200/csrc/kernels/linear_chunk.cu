@@ -68,16 +68,32 @@ linear_chunk_kernel(const LinearChunkParams p) {
   auto load = [&](int c) {
     const uint32_t stage = smem + ((c - c0) & 1) * STAGE;
     const __nv_bfloat16* x = rows + (size_t)c * LC_T * a.ld_qkv;
-    const int n = seq.n - c * LC_T, pieces = DP / 8, vpieces = min(LC_COLS, VP - v0) / 8;
-    for (int i = tid; i < LC_T * pieces; i += LC_THREADS) {
-      const int r = i / pieces, q = i % pieces;
-      const __nv_bfloat16* src = x + (r < n ? (size_t)r * a.ld_qkv : 0) + h * DP + q * 8;
-      if (!STATE) lc_copy(stage + r * PITCH + q * 16, src, r < n);
-      lc_copy(stage + (LC_T + r) * PITCH + q * 16, src + HD, r < n);
+    const int n = seq.n - c * LC_T;
+    constexpr int PIECES = DK / 8, STEP = LC_THREADS / PIECES, VPIECES = LC_COLS / 8, VSTEP = LC_THREADS / VPIECES;      // 16 bytes each; rows at a time
+    {
+      const int q = tid % PIECES, r0 = tid / PIECES;
+      const __nv_bfloat16* src = x + (size_t)r0 * a.ld_qkv + h * DP + q * 8;
+      uint32_t dst = stage + r0 * PITCH + q * 16;
+      if (q * 8 < DP) {
+#pragma unroll
+        for (int r = 0; r < LC_T; r += STEP, src += (size_t)STEP * a.ld_qkv, dst += STEP * PITCH) {
+          const bool live = r0 + r < n;
+          if (!STATE) lc_copy(dst, live ? src : x, live);
+          lc_copy(dst + LC_T * PITCH, live ? src + HD : x, live);
+        }
+      }
     }
-    for (int i = tid; i < LC_T * vpieces; i += LC_THREADS) {
-      const int r = i / vpieces, q = i % vpieces;
-      lc_copy(stage + 2 * LC_T * PITCH + r * LC_VP + q * 16, x + (r < n ? (size_t)r * a.ld_qkv : 0) + 2 * HD + h * VP + v0 + q * 8, r < n);
+    {
+      const int q = tid % VPIECES, r0 = tid / VPIECES;
+      const __nv_bfloat16* src = x + (size_t)r0 * a.ld_qkv + 2 * HD + h * VP + v0 + q * 8;
+      uint32_t dst = stage + 2 * LC_T * PITCH + r0 * LC_VP + q * 16;
+      if (v0 + q * 8 < VP) {
+#pragma unroll
+        for (int r = 0; r < LC_T; r += VSTEP, src += (size_t)VSTEP * a.ld_qkv, dst += VSTEP * LC_VP) {
+          const bool live = r0 + r < n;
+          lc_copy(dst, live ? src : x, live);
+        }
+      }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };

@@ -213,85 +213,89 @@ stream_pass_kernel(const nfn_stream_args p) {
   }
 }
 
-// The convolution over the rows of any entries. A thread takes four channels of a tile's rows; the window slides through registers (TAPS = 0: any
-// number of taps, rows are read again).
-constexpr int IC_THREADS = 128;
+// The convolution over the rows of any entries. A warp takes 256 channels of four rows of a tile, a lane eight channels: the rows and the ones before
+// them are all on their way at once, and what the warps of a tile have in common comes out of L1.
+constexpr int IC_WARPS = 4, IC_ROWS = 4, IC_COLS = 256;
 
+template <typename T>
+struct alignas(16) Piece8 { T v[8]; };
+
+// TAPS = 0: any number of taps, one at a time
 template <typename T, int TAPS>
-__global__ void __launch_bounds__(IC_THREADS)
+__global__ void __launch_bounds__(IC_WARPS * 32)
 input_conv_kernel(const nfn_input_conv_args p) {
-  const nfn_row_tile t = p.tiles[blockIdx.x];
-  const int col = (blockIdx.y * IC_THREADS + threadIdx.x) * 4;
-  if (t.slot < 0 || col >= p.ld) return;
-  const int taps = TAPS ? TAPS : p.taps, hist = taps - 1, ti0 = t.row0 - t.e_row0;
+  const nfn_row_tile t = p.tiles[blockIdx.y];
+  const int i0 = threadIdx.x / 32 * IC_ROWS, col = blockIdx.x * IC_COLS + threadIdx.x % 32 * 8;
+  if (t.slot < 0 || col >= p.ld || i0 >= t.n) return;
+  const int taps = TAPS ? TAPS : p.taps, hist = taps - 1, at = t.row0 - t.e_row0 + i0, n = min(IC_ROWS, t.n - i0);      // of the entry
   const T* rows = static_cast<const T*>(p.h) + (size_t)t.e_row0 * p.ld + col;
   const T* old = static_cast<const T*>(p.history) + (size_t)t.parity * p.history_half + (size_t)t.slot * hist * p.ld + col;
-  T* left = static_cast<T*>(p.history) + (size_t)(1 - t.parity) * p.history_half + (size_t)t.slot * hist * p.ld + col;
   const __nv_bfloat16* conv = static_cast<const __nv_bfloat16*>(p.conv) + col;
-  T* out = static_cast<T*>(p.out) + (size_t)t.row0 * p.ld + col;
-  const bool last = hist > 0 && t.row0 + t.n == t.e_row0 + t.e_n;
+  T* out = static_cast<T*>(p.out) + (size_t)(t.row0 + i0) * p.ld + col;
   // row `idx` of the entry: this step's, a stored one, or zero before the sequence's start
   auto source = [&](int idx) {
-    if (idx >= 0) return load4(rows + (size_t)idx * p.ld);
-    return t.e_pos0 + idx >= 0 ? load4(old + (size_t)(hist + idx) * p.ld) : make_float4(0.f, 0.f, 0.f, 0.f);
+    if (idx >= 0) return *reinterpret_cast<const Piece8<T>*>(rows + (size_t)idx * p.ld);
+    return t.e_pos0 + idx >= 0 ? *reinterpret_cast<const Piece8<T>*>(old + (size_t)(hist + idx) * p.ld) : Piece8<T>{};
   };
-  auto add = [](float4& a, const float4& w, const float4& x) { a.x += w.x * x.x; a.y += w.y * x.y; a.z += w.z * x.z; a.w += w.w * x.w; };
+  auto tap = [&](int j) { return *reinterpret_cast<const Piece8<__nv_bfloat16>*>(conv + (size_t)j * p.ld); };
   if constexpr (TAPS == 0) {
-    for (int i = 0; i < t.n; ++i) {
-      float4 a = source(ti0 + i);
-      for (int j = 0; j < taps; ++j) add(a, load4(conv + (size_t)j * p.ld), source(ti0 + i - hist + j));
-      store4(out + (size_t)i * p.ld, a);
-    }
-    if (last)
-      for (int i = 0; i < hist; ++i) store4(left + (size_t)i * p.ld, source(t.e_n - hist + i));
-  } else {
-    constexpr int N = 8;                                   // rows in flight, as they lie in memory
-    struct alignas(4 * sizeof(T)) Raw { T v[4]; } raw[N];
-    float4 win[TAPS > 1 ? TAPS - 1 : 1], w[TAPS];
-    auto fetch = [&](int i0) {
+    for (int i = 0; i < n; ++i) {
+      float acc[8];
+      const Piece8<T> x = source(at + i);
 #pragma unroll
-      for (int i = 0; i < N; ++i)
-        if (i0 + i < t.n) raw[i] = *reinterpret_cast<const Raw*>(rows + (size_t)(ti0 + i0 + i) * p.ld);
-    };
-    fetch(0);
+      for (int e = 0; e < 8; ++e) acc[e] = to_float(x.v[e]);
+      for (int j = 0; j < taps; ++j) {
+        const Piece8<T> y = source(at + i - hist + j);
+        const Piece8<__nv_bfloat16> w = tap(j);
 #pragma unroll
-    for (int j = 0; j < TAPS - 1; ++j) win[j] = source(ti0 - (TAPS - 1) + j);
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) w[j] = load4(conv + (size_t)j * p.ld);
-    for (int i0 = 0; i0 < t.n; i0 += N) {
-      if (i0 > 0) fetch(i0);
-#pragma unroll
-      for (int i = 0; i < N; ++i)
-        if (i0 + i < t.n) {
-          const float4 x = make_float4(to_float(raw[i].v[0]), to_float(raw[i].v[1]), to_float(raw[i].v[2]), to_float(raw[i].v[3]));
-          float4 a = x;
-          add(a, w[TAPS - 1], x);
-#pragma unroll
-          for (int j = 0; j < TAPS - 1; ++j) add(a, w[j], win[j]);
-#pragma unroll
-          for (int j = 0; j + 1 < TAPS - 1; ++j) win[j] = win[j + 1];
-          if constexpr (TAPS > 1) win[TAPS - 2] = x;
-          store4(out + (size_t)(i0 + i) * p.ld, a);
-        }
-    }
-    if constexpr (TAPS > 1) {
-      if (last) {
-#pragma unroll
-        for (int j = 0; j < TAPS - 1; ++j) store4(left + (size_t)j * p.ld, win[j]);
+        for (int e = 0; e < 8; ++e) acc[e] += to_float(w.v[e]) * to_float(y.v[e]);
       }
+      store8(out + (size_t)i * p.ld, acc);
     }
+  } else {
+    Piece8<T> x[IC_ROWS + TAPS - 1];
+    Piece8<__nv_bfloat16> w[TAPS];
+    if (n == IC_ROWS && at >= TAPS - 1) {                  // inside the entry: nothing to decide between the loads
+      const T* first = rows + (size_t)(at - (TAPS - 1)) * p.ld;
+#pragma unroll
+      for (int i = 0; i < IC_ROWS + TAPS - 1; ++i) x[i] = *reinterpret_cast<const Piece8<T>*>(first + (size_t)i * p.ld);
+    } else {
+#pragma unroll
+      for (int i = 0; i < IC_ROWS + TAPS - 1; ++i)
+        if (i < n + TAPS - 1) x[i] = source(at - (TAPS - 1) + i);
+    }
+#pragma unroll
+    for (int j = 0; j < TAPS; ++j) w[j] = tap(j);
+#pragma unroll
+    for (int i = 0; i < IC_ROWS; ++i) {
+      if (i >= n) break;
+      float acc[8];
+#pragma unroll
+      for (int e = 0; e < 8; ++e) {
+        float a = to_float(x[i + TAPS - 1].v[e]);
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) a += to_float(w[j].v[e]) * to_float(x[i + j].v[e]);
+        acc[e] = a;
+      }
+      store8(out + (size_t)i * p.ld, acc);
+    }
+  }
+  // the history the entry leaves behind: its newest taps - 1 rows (older ones move up when it brought fewer)
+  if (i0 == 0 && hist > 0 && t.row0 + t.n == t.e_row0 + t.e_n) {
+    T* left = static_cast<T*>(p.history) + (size_t)(1 - t.parity) * p.history_half + (size_t)t.slot * hist * p.ld + col;
+    for (int i = 0; i < hist; ++i) *reinterpret_cast<Piece8<T>*>(left + (size_t)i * p.ld) = source(t.e_n - hist + i);
   }
 }
 
 template <typename T>
 static int pick_input_conv(const nfn_input_conv_args& a, cudaStream_t st) {
-  const dim3 grid(a.n_tiles, ceil_div(a.ld, IC_THREADS * 4));
+  const dim3 grid(ceil_div(a.ld, IC_COLS), a.n_tiles);                     // neighbouring CTAs read neighbouring columns of the same rows
   switch (a.taps) {
-    case 1: input_conv_kernel<T, 1><<<grid, IC_THREADS, 0, st>>>(a); break;
-    case 2: input_conv_kernel<T, 2><<<grid, IC_THREADS, 0, st>>>(a); break;
-    case 3: input_conv_kernel<T, 3><<<grid, IC_THREADS, 0, st>>>(a); break;
-    case 4: input_conv_kernel<T, 4><<<grid, IC_THREADS, 0, st>>>(a); break;
-    default: input_conv_kernel<T, 0><<<grid, IC_THREADS, 0, st>>>(a); break;
+    case 1: input_conv_kernel<T, 1><<<grid, IC_WARPS * 32, 0, st>>>(a); break;
+    case 2: input_conv_kernel<T, 2><<<grid, IC_WARPS * 32, 0, st>>>(a); break;
+    case 3: input_conv_kernel<T, 3><<<grid, IC_WARPS * 32, 0, st>>>(a); break;
+    case 4: input_conv_kernel<T, 4><<<grid, IC_WARPS * 32, 0, st>>>(a); break;
+    default: input_conv_kernel<T, 0><<<grid, IC_WARPS * 32, 0, st>>>(a); break;
   }
   return launch_check("input_conv");
 }
@@ -346,6 +350,7 @@ extern "C" int nfn_input_conv(const nfn_input_conv_args* args, nfn_stream_t stre
   if (!args) return fail(-1, "input_conv: null args");
   const nfn_input_conv_args& a = *args;
   if (a.n_tiles <= 0) return 0;
+  if (a.n_tiles > 65535) return fail(-1, "input_conv: too many row tiles in one launch");
   if ((a.ld & 15) || a.taps < 1 || !a.h || !a.conv || !a.out || a.h == a.out || !a.tiles || (a.taps > 1 && !a.history)) return fail(-1, "input_conv: rows padded to multiples of 16, two buffers, a history");
   return a.f32 ? pick_input_conv<float>(a, static_cast<cudaStream_t>(stream)) : pick_input_conv<__nv_bfloat16>(a, static_cast<cudaStream_t>(stream));
 }

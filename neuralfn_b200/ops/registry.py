@@ -41,15 +41,22 @@ KERNELS: tuple[KernelEntry, ...] = (
     _k("attention_backward", "nfn_attention_backward", ("bf16",), True, "dQ dK dV, delta pre-pass"),
     _k("block_attention", "nfn_block_attention", ("bf16",), True, "cache prefix + block, staging of block K/V, split-KV merge"),
     _k("decode_attention", "nfn_decode_attention", ("bf16",), False, "QK-norm, RoPE, cache append, split-KV merge"),
-    _k("paged attention, prompt tiles", "nfn_paged_attention_tiles", ("bf16",), True, "page table, window, kept first tokens, soft cap, sink, distance bias, GQA packing, output gate"),
-    _k("paged attention, single rows", "nfn_paged_attention_rows", ("bf16", "fp32"), False, "page table, window, kept first tokens, soft cap, sink, distance bias, split-KV merge, output gate"),
+    _k("paged attention, prompt tiles", "nfn_paged_attention_tiles", ("bf16",), True, "page table, window, kept first tokens, soft cap, zero or learned sink, distance bias, GQA packing, output gate"),
+    _k("paged attention, single rows", "nfn_paged_attention_rows", ("bf16", "fp32"), False, "page table, window, kept first tokens, soft cap, zero or learned sink, distance bias, split-KV merge, output gate"),
     _k("short convolution + cache append + feed-forward gate", "nfn_mix_rows", ("bf16", "fp32"), False, "per-sequence history, SiLU, query temperature, transposed value pages"),
     _k("gated delta rule, prompt chunks", "nfn_delta_chunks", ("bf16",), True, "per-channel decay, fp32 state, split-bf16 tensor-core scan"),
     _k("gated delta rule, rows", "nfn_delta_rows", ("bf16", "fp32"), False, "token after token, any length"),
     _k("gated delta rule, decode step", "nfn_delta_step", ("bf16", "fp32"), False, "convolution, SiLU, output norm and gate"),
     _k("delta rule output norm", "nfn_delta_out", ("bf16", "fp32"), False, "per-head RMS norm, sigmoid gate"),
-    _k("residual streams", "nfn_stream_pass", ("bf16", "fp32"), False, "mixing matrix, expert sum, next norm, row gather"),
-    _k("experts, few rows", "nfn_moe_rows", ("bf16", "fp32"), False, "routing, item lists, weight on the input"),
+    _k("linear attention with a decay per head, prompt chunks", "nfn_linear_chunks", ("bf16",), False, "64 tokens at a time, fp32 state in accumulators, split-bf16 products, segments side by side"),
+    _k("linear attention with a decay per head, rows", "nfn_linear_rows", ("bf16", "fp32"), False, "token after token, any length"),
+    _k("linear attention with a decay per head, decode step", "nfn_linear_step", ("bf16", "fp32"), False, "SiLU, norm over all heads, gate"),
+    _k("row norm and gate", "nfn_row_out", ("bf16", "fp32"), False, "RMS norm over all heads, weight, sigmoid gate"),
+    _k("gated recurrence", "nfn_gru_rows", ("bf16", "fp32"), False, "gates, affine scan, SiLU output gate"),
+    _k("convolution on a sublayer's input", "nfn_input_conv", ("bf16", "fp32"), False, "per-sequence history"),
+    _k("residual streams", "nfn_stream_pass", ("bf16", "fp32"), False, "mixing matrix, expert sum, norm of the update, next norm, short convolution of single tokens, row gather"),
+    _k("router logits, few rows", "nfn_router_rows", ("bf16",), False, "fp32 sums"),
+    _k("experts, few rows", "nfn_moe_rows", ("bf16", "fp32"), False, "routing, item lists, weight on the input or output, clamped gate"),
     _k("residual row pass", "nfn_row_norm", ("bf16", "fp32"), False, "embedding, branch norm + residual, next norm, row gather"),
     _k("per-layer token input gate", "nfn_side_mul", ("bf16", "fp32"), False, "GELU, embedding gather"),
     _k("gemm, 32-bit", "nfn_gemm_f32", ("fp32",), False, "accumulate"),
