@@ -1,4 +1,4 @@
-// A gated recurrence whose gates read only the current token: per channel s <- (1 - z) s + z c, out = s * silu(g), with z = sigmoid(a) and a candidate c
+// A gated recurrence that decides from the current token alone: per channel s <- (1 - z) s + z c, out = s * silu(g), with z = sigmoid(a) and a candidate c
 // formed from b. Everything but the loads and stores is fp32.
 //
 // Short entries (single tokens, portions of a few rows) go token after token. Long ones are an affine scan: a CTA takes 32 channels, 16 lanes with two

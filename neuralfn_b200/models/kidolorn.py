@@ -1,6 +1,6 @@
 """Kidolorn: a decoder whose sublayers have a norm before and one after them, each with a single factor, and read their input plus a short causal
-convolution of it. Three kinds of mixers: linear attention with a constant decay per head ("lightning"), a gated recurrence whose gates read only the
-current token ("mingru"), and latent attention over every earlier token with a learned sink per head and an output gate (a layer may read an earlier
+convolution of it. Three kinds of mixers: linear attention with a constant decay per head ("lightning"), a gated recurrence that decides from the
+current token alone ("mingru"), and latent attention over every earlier token with a learned sink per head and an output gate (a layer may read an earlier
 one's cache). Feed-forwards have a clamped gate, dense with biases or routed with the softmax over the chosen experts as weights.
 
 ``KidolornConfig.from_dict`` reads the model's ``config.json``, ``pack_tensors`` turns its tensors into the fused, padded ones of the layer-list engine
